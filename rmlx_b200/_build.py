@@ -39,6 +39,24 @@ NVCC_FLAGS = [
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-pthread"]
 
 
+# Kernel sets: what a model family needs, for a checkout in which nothing is built yet
+# (``_lib.prefer_kernels``; the full libraries win whenever they exist). "all" is every source.
+SETS = {
+    "parallel_block": {
+        "cuda": ("kernels/parallel_rows.cu", "kernels/parallel_gemv.cu", "kernels/gemm_tcgen05.cu",
+                 "kernels/gemm_f32.cu", "kernels/flash_prefill_tc.cu", "kernels/flash_decode_scored.cu",
+                 "kernels/attention_any.cu", "kernels/misc.cu", "runtime/graph_exec.cu"),
+        "host": ("host/serving.cpp", "host/sampler.cpp", "host/safetensors_io.cpp"),
+    },
+}
+
+
+def set_lib(kind: str, name: str) -> Path:
+    """Path of the ``kind`` ("cuda" or "host") library of a kernel set."""
+    full = CUDA_LIB if kind == "cuda" else HOST_LIB
+    return full if name == "all" else LIB / f"librmlx_b200_{kind}_{name}.so"
+
+
 def _nvcc() -> str | None:
     cand = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
     return cand if os.path.exists(cand) else None
@@ -82,15 +100,20 @@ def _sources(kind: str) -> list[Path]:
     return sorted((CSRC / "host").glob("*.cpp"))
 
 
-def build(kinds=("host", "cuda"), verbose: bool = False, force: bool = False) -> dict[str, Path]:
-    """Compile and link whatever is out of date. Returns the library paths."""
+def build(kinds=("host", "cuda"), verbose: bool = False, force: bool = False, only: str = "all") -> dict[str, Path]:
+    """Compile and link whatever is out of date. Returns the library paths. ``only``: a kernel set
+    (``SETS``) instead of every source; it goes into a library of its own."""
     OBJ.mkdir(exist_ok=True)
     LIB.mkdir(exist_ok=True)
     hdr = _headers_digest()
     out: dict[str, Path] = {}
     for kind in kinds:
-        srcs = _sources(kind)
-        lib = {"cuda": CUDA_LIB, "cuda_bounds": CUDA_BOUNDS_LIB}.get(kind, HOST_LIB)
+        if only == "all":
+            srcs = _sources(kind)
+            lib = {"cuda": CUDA_LIB, "cuda_bounds": CUDA_BOUNDS_LIB}.get(kind, HOST_LIB)
+        else:
+            srcs = [CSRC / s for s in SETS[only][kind]]
+            lib = set_lib(kind, only)
         if not srcs:
             continue
         if kind in ("cuda", "cuda_bounds"):
@@ -117,19 +140,21 @@ def build(kinds=("host", "cuda"), verbose: bool = False, force: bool = False) ->
             for o, did, log in results:
                 if did:
                     print(f"[build] compiled {o.name}", file=sys.stderr)
-        link_stamp = OBJ / f"{kind}.linkhash"
+        link_stamp = OBJ / (f"{kind}.linkhash" if only == "all" else f"{kind}_{only}.linkhash")
         link_digest = hashlib.sha256(
             "".join(sorted(j[3] for j in jobs)).encode()).hexdigest()
         if rebuilt or not lib.exists() or not link_stamp.exists() or \
                 link_stamp.read_text() != link_digest:
             objs = [str(r[0]) for r in results]
+            part = lib.with_suffix(f".{os.getpid()}.tmp")       # a link that is cut short leaves no half library
             if kind in ("cuda", "cuda_bounds"):
-                cmd = [_nvcc(), "-shared", "-o", str(lib), *objs, "-lpthread", "-ldl"]
+                cmd = [_nvcc(), "-shared", "-o", str(part), *objs, "-lpthread", "-ldl"]
             else:
-                cmd = [shutil.which("g++") or "g++", "-shared", "-o", str(lib), *objs, "-pthread"]
+                cmd = [shutil.which("g++") or "g++", "-shared", "-o", str(part), *objs, "-pthread"]
             proc = subprocess.run(cmd, capture_output=True, text=True)
             if proc.returncode != 0:
                 raise RuntimeError(f"link failed: {' '.join(cmd)}\n{proc.stdout}{proc.stderr}")
+            os.replace(part, lib)
             link_stamp.write_text(link_digest)
             if verbose:
                 print(f"[build] linked {lib.name}", file=sys.stderr)

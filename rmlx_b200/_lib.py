@@ -86,6 +86,27 @@ def register_cuda_sigs(sigs: Dict[str, tuple]) -> None:
         _bind(_cuda_lib, sigs)
 
 
+_kernel_set = "all"
+
+
+def prefer_kernels(name: str) -> None:
+    """In a checkout without the full libraries, build and load only the kernel set ``name``
+    (``_build.SETS``) instead of every source. Takes effect before the first kernel is loaded."""
+    global _kernel_set
+    _kernel_set = name
+
+
+def _library(kind: str) -> "_build.Path":
+    """The library to load, built first if there is none: the full one when it exists, else that of
+    the preferred kernel set."""
+    full = _build.set_lib(kind, "all")
+    if full.exists() or _kernel_set == "all":
+        if not full.exists():
+            _build.build(kinds=(kind,))
+        return full
+    return _build.build(kinds=(kind,), only=_kernel_set)[kind]
+
+
 def cuda() -> ctypes.CDLL:
     global _cuda_lib
     if _cuda_lib is None:
@@ -93,9 +114,9 @@ def cuda() -> ctypes.CDLL:
             if _cuda_lib is None:
                 # RMLX_BOUNDS=1: the bounds-checked build of the same kernels
                 bounds = os.environ.get("RMLX_BOUNDS", "0") == "1"
-                path = _build.CUDA_BOUNDS_LIB if bounds else _build.CUDA_LIB
-                if not path.exists():
-                    _build.build(kinds=("cuda_bounds" if bounds else "cuda",))
+                if bounds and not _build.CUDA_BOUNDS_LIB.exists():
+                    _build.build(kinds=("cuda_bounds",))
+                path = _build.CUDA_BOUNDS_LIB if bounds else _library("cuda")
                 lib = ctypes.CDLL(str(path))
                 lib.rmlx_bounds_build.restype = c_int
                 if bool(lib.rmlx_bounds_build()) != bounds:
@@ -126,9 +147,7 @@ def host() -> ctypes.CDLL:
     if _host_lib is None:
         with _lock:
             if _host_lib is None:
-                if not _build.HOST_LIB.exists():
-                    _build.build(kinds=("host",))
-                _host_lib = ctypes.CDLL(str(_build.HOST_LIB))
+                _host_lib = ctypes.CDLL(str(_library("host")))
     return _host_lib
 
 

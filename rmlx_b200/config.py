@@ -136,6 +136,91 @@ class TransformerConfig:
 
 
 @dataclass
+class ScoredAttentionSpec:
+    """Attention whose scores are modified before the softmax: ``scale``, a soft cap (0: none), and
+    the per-head temperature, distance bias and sink that come with the weights. Query / key heads
+    are ``dim`` wide, value heads ``vdim``."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    softcap: float = 0.0
+
+    def validate(self) -> "ScoredAttentionSpec":
+        _require(self.heads > 0 and self.kv_heads > 0, "head counts must be positive")
+        _require(self.heads % self.kv_heads == 0, "heads must be a multiple of kv_heads")
+        _require(self.dim > 0 and self.vdim > 0, "head sizes must be positive")
+        _require(self.softcap >= 0, "softcap must be >= 0 (0: no cap)")
+        return self
+
+
+@dataclass
+class ParallelLayerSpec:
+    """One layer of a parallel-block decoder: attention and (unless ``ff`` is 0) a dense feed-forward
+    that read the same normalised input."""
+    mixer: ScoredAttentionSpec
+    ff: int = 0
+
+    def validate(self) -> "ParallelLayerSpec":
+        self.mixer.validate()
+        _require(self.ff >= 0, "ff must be >= 0 (0: no feed-forward)")
+        return self
+
+
+@dataclass
+class PosudraConfig:
+    """Posudra: parallel-block decoder without rotation; every layer states its own sizes."""
+    vocab_size: int
+    width: int
+    layers: "list[ParallelLayerSpec]"
+    norm_eps: float = 1e-6
+    embedding_scale: float = 1.0
+    max_seq_len: int = 0             # 0: bounded by the cache only (positions enter as distances)
+    name: str = "posudra"
+
+    sliding_window = 0               # every key stays visible
+
+    def validate(self) -> "PosudraConfig":
+        _require(self.vocab_size > 0 and self.width > 0 and len(self.layers) > 0, "bad sizes")
+        _require(self.norm_eps > 0, "norm_eps must be positive")
+        for layer in self.layers:
+            layer.validate()
+        return self
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def hidden_size(self) -> int:
+        return self.width
+
+    @staticmethod
+    def from_json(c: dict) -> "PosudraConfig":
+        layers = []
+        for i, e in enumerate(c["layers"]):
+            _require(e.get("type") == "attention", f"layer {i}: unknown mixer type {e.get('type')!r}")
+            m, mlp = e["mixer"], e.get("mlp")
+            _require(mlp is None or mlp.get("kind") == "dense",
+                     f"layer {i}: unknown feed-forward kind {None if mlp is None else mlp.get('kind')!r}")
+            layers.append(ParallelLayerSpec(
+                ScoredAttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]),
+                                    float(m["scale"]), float(m.get("softcap") or 0.0)),
+                0 if mlp is None else int(mlp["ff"])))
+        return PosudraConfig(int(c["vocab"]), int(c["width"]), layers, float(c["norm"]["eps"]),
+                             float(c["embedding"]["scale"])).validate()
+
+    def to_json(self) -> dict:
+        return {"architecture": "Posudra", "vocab": self.vocab_size, "width": self.width,
+                "norm": {"eps": self.norm_eps}, "embedding": {"scale": self.embedding_scale},
+                "layers": [{"type": "attention",
+                            "mixer": {"heads": l.mixer.heads, "kv_heads": l.mixer.kv_heads, "dim": l.mixer.dim,
+                                      "vdim": l.mixer.vdim, "scale": l.mixer.scale, "softcap": l.mixer.softcap},
+                            "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None} for l in self.layers]}
+
+
+@dataclass
 class AttentionConfig:
     num_heads: int
     num_kv_heads: int

@@ -1,0 +1,79 @@
+// Attention-score modifiers shared by the attention kernels that take them: what happens to q . k
+// between the product and the softmax. Every part is optional, so designs pick what they need:
+//
+//   s = (q . k) * scale * temp[h]               per-head temperature (temp == nullptr: 1)
+//   s = softcap * tanh(s / softcap)             logit soft cap       (softcap <= 0: none)
+//   s = s - r1[h] * ln(1 + r2[h] * (i - j))     logarithmic distance bias (r1 == nullptr: none)
+//   weights = exp(s) / (sum exp(s) + exp(sink[h]))    sink without key or value (nullptr: none)
+//
+// The tensor-core kernels work in base 2 (scores times log2 e), which leaves one ex2 per weight.
+#pragma once
+#include "ptx.cuh"
+
+namespace rb {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+struct ScoreMod {
+  float scale = 1.f;
+  float softcap = 0.f;
+  const float* temp = nullptr;
+  const float* r1 = nullptr;
+  const float* r2 = nullptr;
+  const float* sink = nullptr;
+};
+
+// tanh(u) / u as a polynomial in u^2, |u| <= kTanhPolyMax: Chebyshev interpolation of degree 4 in
+// u^2, largest relative error 1.6e-7 (fp32 evaluation included).
+constexpr float kTanhPolyMax = 0.625f;
+constexpr float kTanhP0 = 0.9999998807907104f, kTanhP1 = -0.33331942558288574f,
+                kTanhP2 = 0.1330437958240509f, kTanhP3 = -0.05181591212749481f,
+                kTanhP4 = 0.015043356455862522f;
+
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// tanh with small relative error everywhere: the polynomial near zero, 1 - 2 / (1 + e^(2u)) beyond
+// (which saturates to +-1 without overflow trouble: the exponential may become 0 or inf).
+__device__ __forceinline__ float tanh_score(float u) {
+  const float w = u * u;
+  const float near = u * fmaf(fmaf(fmaf(fmaf(kTanhP4, w, kTanhP3), w, kTanhP2), w, kTanhP1), w, kTanhP0);
+  const float far = 1.f - __fdividef(2.f, 1.f + ex2_approx(fminf(u, 40.f) * (2.f * kLog2e)));
+  return fabsf(u) <= kTanhPolyMax ? near : far;
+}
+
+// One head's modifiers, in base-2 units.
+struct HeadScore {
+  float lin;       // scale * temp * log2 e
+  float inner;     // scale * temp / softcap, 0 without a cap
+  float capl;      // softcap * log2 e, 0 without a cap
+  float r1, r2;    // r1 as given: r1 * log2(1 + r2 d) is already r1 * ln(..) in base-2 units
+  float sink;      // sink * log2 e; -inf without one
+};
+
+__device__ __forceinline__ HeadScore head_score(const ScoreMod& m, int h) {
+  HeadScore s;
+  const float st = m.scale * (m.temp ? m.temp[h] : 1.f);
+  s.lin = st * kLog2e;
+  s.inner = m.softcap > 0.f ? st / m.softcap : 0.f;
+  s.capl = m.softcap > 0.f ? m.softcap * kLog2e : 0.f;
+  s.r1 = m.r1 ? m.r1[h] : 0.f;
+  s.r2 = m.r1 ? m.r2[h] : 0.f;
+  s.sink = m.sink ? m.sink[h] * kLog2e : -INFINITY;
+  return s;
+}
+
+__device__ __forceinline__ float distance_bias(const HeadScore& s, float dist) {
+  return s.r1 * __log2f(fmaf(s.r2, dist, 1.f));
+}
+
+// Base-2 score of a dot product at distance i - j >= 0.
+__device__ __forceinline__ float score_base2(float dot, const HeadScore& s, float dist) {
+  const float t = s.capl > 0.f ? s.capl * tanh_score(dot * s.inner) : dot * s.lin;
+  return t - distance_bias(s, dist);
+}
+
+}  // namespace rb

@@ -1,0 +1,172 @@
+// Paged causal attention for any head sizes, in fp32 or bf16 storage with fp32 arithmetic on the
+// CUDA cores: the attention of models run in 32-bit, and of head sizes the tensor-core kernels do
+// not take. Rows are single query tokens (a ragged batch of prompt portions and decoded tokens);
+// each has a position and a row of the block table.
+//
+// A block owns one (token, query head); its four warps take 32-key chunks in turn. Lane j scores
+// key j (its row read straight from the page), the chunk's softmax update is a warp reduction, and
+// the values are accumulated with lanes along the value dimension. The warps merge through shared
+// memory at the end.
+#include "../common/launch.cuh"
+#include "../common/score_mod.cuh"
+
+namespace rb {
+
+constexpr int kAaWarps = 4;
+
+struct AaParams {
+  const void* q;            // [T, Hq, dkp]
+  const void* k_cache;      // [blocks, Hkv, page, dkp]
+  const void* v_cache;      // [blocks, Hkv, page, dvp]
+  const int* block_table;
+  const int* positions;     // [T]
+  const int* token_seq;     // [T] row of the block table, or null: token t has row t
+  void* out;                // [T, Hq, dvp]
+  int Hq, Hkv, dkp, dvp, max_blocks, page, window;
+  ScoreMod mod;
+};
+
+__device__ __forceinline__ float aa_dot8(const float* k, const float* q) {
+  const float4 a = *reinterpret_cast<const float4*>(k), b = *reinterpret_cast<const float4*>(k + 4);
+  float s = a.x * q[0];
+  s = fmaf(a.y, q[1], s); s = fmaf(a.z, q[2], s); s = fmaf(a.w, q[3], s);
+  s = fmaf(b.x, q[4], s); s = fmaf(b.y, q[5], s); s = fmaf(b.z, q[6], s); s = fmaf(b.w, q[7], s);
+  return s;
+}
+__device__ __forceinline__ float aa_dot8(const __nv_bfloat16* k, const float* q) {
+  const uint4 v = *reinterpret_cast<const uint4*>(k);
+  float s = bf16lo(v.x) * q[0];
+  s = fmaf(bf16hi(v.x), q[1], s); s = fmaf(bf16lo(v.y), q[2], s); s = fmaf(bf16hi(v.y), q[3], s);
+  s = fmaf(bf16lo(v.z), q[4], s); s = fmaf(bf16hi(v.z), q[5], s); s = fmaf(bf16lo(v.w), q[6], s);
+  s = fmaf(bf16hi(v.w), q[7], s);
+  return s;
+}
+__device__ __forceinline__ float aa_f32(float v) { return v; }
+__device__ __forceinline__ float aa_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void aa_put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void aa_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// NV: 32-wide slices of the value dimension kept per lane.
+template <class T, int NV>
+__global__ void __launch_bounds__(kAaWarps * 32) attention_any_kernel(AaParams p) {
+  extern __shared__ float smem[];
+  float* sq = smem;                                   // the query, fp32
+  float* so = smem + p.dkp;                           // [warps][dvp]
+  __shared__ float s_m[kAaWarps], s_l[kAaWarps];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, h = blockIdx.y, kvh = h / (p.Hq / p.Hkv);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = p.positions[t];
+  const int seq = p.token_seq ? p.token_seq[t] : t;
+  const int* bt = p.block_table + size_t(seq) * p.max_blocks;
+  const T* q = static_cast<const T*>(p.q) + (size_t(t) * p.Hq + h) * p.dkp;
+  for (int i = threadIdx.x; i < p.dkp; i += kAaWarps * 32) sq[i] = aa_f32(q[i]);
+  __syncthreads();
+  // natural units here: the all-32-bit mode uses the full-precision functions
+  const float st = p.mod.scale * (p.mod.temp ? p.mod.temp[h] : 1.f);
+  const float cap = p.mod.softcap;
+  const float r1 = p.mod.r1 ? p.mod.r1[h] : 0.f, r2 = p.mod.r1 ? p.mod.r2[h] : 0.f;
+  const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+
+  float m = -INFINITY, l = 0.f, o[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) o[i] = 0.f;
+  for (int c0 = (first & ~31) + warp * 32; c0 <= pos; c0 += kAaWarps * 32) {
+    const int key = c0 + lane;
+    const bool ok = key >= first && key <= pos && RB_BOUNDS(key / p.page, p.max_blocks);
+    float s = -INFINITY;
+    if (ok) {
+      const size_t row = (size_t(bt[key / p.page]) * p.Hkv + kvh) * p.page + key % p.page;
+      const T* k = static_cast<const T*>(p.k_cache) + row * p.dkp;
+      float dot = 0.f;
+      for (int d = 0; d < p.dkp; d += 8) dot += aa_dot8(k + d, sq + d);
+      s = dot * st;
+      if (cap > 0.f) s = cap * tanhf(s / cap);
+      if (p.mod.r1) s -= r1 * log1pf(r2 * float(pos - key));
+    }
+    const float nm = fmaxf(m, warp_max(s));
+    if (nm == -INFINITY) continue;                    // no visible key in this chunk
+    const float f = expf(m - nm), w = expf(s - nm);   // exp(-inf) = 0
+    m = nm;
+    l = l * f + warp_sum(w);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) o[i] *= f;
+    const int n = min(32, pos - c0 + 1);
+    for (int j = 0; j < n; ++j) {
+      const float wj = __shfl_sync(0xffffffffu, w, j);
+      if (wj == 0.f) continue;                        // warp-uniform
+      const int kj = c0 + j;
+      const size_t row = (size_t(bt[kj / p.page]) * p.Hkv + kvh) * p.page + kj % p.page;
+      const T* v = static_cast<const T*>(p.v_cache) + row * p.dvp;
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (i * 32 + lane < p.dvp) o[i] = fmaf(wj, aa_f32(v[i * 32 + lane]), o[i]);
+    }
+  }
+  if (lane == 0) { s_m[warp] = m; s_l[warp] = l; }
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (i * 32 + lane < p.dvp) so[warp * p.dvp + i * 32 + lane] = o[i];
+  __syncthreads();
+  float M = p.mod.sink ? p.mod.sink[h] : -INFINITY;
+#pragma unroll
+  for (int w = 0; w < kAaWarps; ++w) M = fmaxf(M, s_m[w]);
+  float L = p.mod.sink ? expf(p.mod.sink[h] - M) : 0.f;
+  float f[kAaWarps];
+#pragma unroll
+  for (int w = 0; w < kAaWarps; ++w) {
+    f[w] = s_m[w] == -INFINITY ? 0.f : expf(s_m[w] - M);
+    L += s_l[w] * f[w];
+  }
+  T* out = static_cast<T*>(p.out) + (size_t(t) * p.Hq + h) * p.dvp;
+  for (int i = threadIdx.x; i < p.dvp; i += kAaWarps * 32) {
+    float acc = 0.f;
+#pragma unroll
+    for (int w = 0; w < kAaWarps; ++w) acc += so[w * p.dvp + i] * f[w];
+    aa_put(out + i, L > 0.f ? acc / L : 0.f);
+  }
+}
+
+template <class T, int NV>
+static int launch_any(const AaParams& p, int rows, int pdl, cudaStream_t st) {
+  const size_t smem = (size_t(p.dkp) + size_t(kAaWarps) * p.dvp) * sizeof(float);
+  auto kern = attention_any_kernel<T, NV>;
+  RB_CHECK(set_max_smem(kern, smem));
+  return launch(kern, dim3(rows, p.Hq), dim3(kAaWarps * 32), smem, st, pdl != 0, p);
+}
+template <class T>
+static int dispatch_any(const AaParams& p, int rows, int pdl, cudaStream_t st) {
+  if (p.dvp <= 64) return launch_any<T, 2>(p, rows, pdl, st);
+  if (p.dvp <= 128) return launch_any<T, 4>(p, rows, pdl, st);
+  if (p.dvp <= 256) return launch_any<T, 8>(p, rows, pdl, st);
+  if (p.dvp <= 1024) return launch_any<T, 32>(p, rows, pdl, st);
+  return -2;
+}
+
+}  // namespace rb
+
+using namespace rb;
+RB_BOUNDS_REGISTER("attention_any.cu")
+
+// q [T, Hq, dkp], out [T, Hq, dvp], caches [blocks, Hkv, page, dkp / dvp]: fp32 (f32) or bf16; dkp and
+// dvp multiples of eight, dvp <= 1024. Token t sits at positions[t] and sees keys 0 .. positions[t]
+// (the last `window` of them when window > 0) of row token_seq[t] of the block table.
+extern "C" int rmlx_attention_any(const void* q, const void* k_cache, const void* v_cache,
+                                  const int* block_table, const int* positions, const int* token_seq,
+                                  void* out, int T, int Hq, int Hkv, int dkp, int dvp, int max_blocks,
+                                  int page, int window, float scale, float softcap, const float* temp,
+                                  const float* r1, const float* r2, const float* sink, int f32, int pdl,
+                                  cudaStream_t st) {
+  if (T < 1 || Hkv < 1 || Hq % Hkv || Hq > 65535 || dkp < 8 || dkp % 8 || dvp < 8 || dvp % 8 ||
+      dkp > 8192 || (r1 && !r2))
+    return -2;
+  AaParams p;
+  p.q = q; p.k_cache = k_cache; p.v_cache = v_cache; p.block_table = block_table;
+  p.positions = positions; p.token_seq = token_seq; p.out = out;
+  p.Hq = Hq; p.Hkv = Hkv; p.dkp = dkp; p.dvp = dvp; p.max_blocks = max_blocks; p.page = page;
+  p.window = window;
+  p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2;
+  p.mod.sink = sink;
+  return f32 ? dispatch_any<float>(p, T, pdl, st) : dispatch_any<__nv_bfloat16>(p, T, pdl, st);
+}

@@ -1,6 +1,20 @@
 // Paged causal flash attention for prompt processing on the 5th-generation tensor cores
 // (head_dim 128, optional sliding window; other head dimensions use the mma.sync kernel in
-// flash_prefill.cu).
+// flash_prefill.cu), and its form with score modifiers (score_mod.cuh: temperature, soft cap,
+// logarithmic distance bias, sink) over ragged batches, for key and value widths up to 128 each.
+//
+// KP / VP: 64-column panels of a key / value row. Widths that are not a multiple of 64 cost no extra
+// global memory: the tensor maps end at the real width and TMA fills the rest of a panel with zeros.
+// Ragged batches come as a table of query tiles ({first row, rows, position of the first row, row of
+// the block table}), so prompt portions of several sequences share one launch.
+//
+// Score modifiers run between S and the softmax, in base 2: t = P(s) - bias(i - j), where P is
+// softcap * tanh(s scale temp / softcap) as s times a polynomial in s^2 with the head's constants
+// folded in (all FMA), or, in a step where some |argument| leaves the polynomial's range, by
+// ex2 / rcp. The bias depends on the distance only: every softmax warp keeps the values for the
+// 95 distances a step can hold in a ring in shared memory (128 entries, stored twice so that a
+// step reads a straight run) and adds the 64 new ones of each step. The sink is a first key of
+// weight one and no value: it initialises the running maximum and sum.
 //
 // A CTA owns LANES (1 or 2) tiles of 128 query tokens of one query head and walks the keys 64 at a
 // time; the K and V tiles of a step serve every lane. A kernel that allocates tensor memory gets one
@@ -33,6 +47,7 @@
 #include "../common/ptx.cuh"
 #include "../common/launch.cuh"
 #include "../common/tensormap.cuh"
+#include "../common/score_mod.cuh"
 
 namespace rb {
 
@@ -42,54 +57,57 @@ constexpr int kTcHd = 128;
 constexpr int kTcPage = 16;
 constexpr int kTcPages = kTcKeys / kTcPage;   // pages per step
 constexpr int kTcQPanel = 128 * 128;          // 128 rows x 64 bf16 columns
-constexpr int kTcQTile = 2 * kTcQPanel;       // 128 x 128 bf16
 constexpr int kTcKvPanel = kTcKeys * 128;     // 64 rows x 64 bf16 columns
-constexpr int kTcKvTile = 2 * kTcKvPanel;     // 64 x 128 bf16
+constexpr int kTcBiasRing = 256;              // floats per softmax warp: 128 distances, twice
 constexpr int kTcPTile = kTcQPanel;           // 128 rows x 64 keys bf16
 constexpr int kTcPageBytes = kTcPage * 128;   // one page inside a 64-column panel
 constexpr float kTcRescaleStep = 8.f;         // log2 of the growth tolerated before O is rescaled
 
-template <int LANES>
+template <int LANES, int KP, int VP, bool MOD>
 struct TcCfg {
+  static constexpr int kQTile = KP * kTcQPanel;     // 128 query rows
+  static constexpr int kKTile = KP * kTcKvPanel;    // 64 keys
+  static constexpr int kVTile = VP * kTcKvPanel;
   static constexpr int kThreads = 64 + 128 * LANES;
-  // per lane: S0 [0,64) S1 [64,128); then per lane O (128 columns)
+  // per lane: S0 [0,64) S1 [64,128); then per lane O (VP * 64 columns)
   static constexpr uint32_t kTmemCols = 256 * LANES;
   static constexpr int kBars = 9 + 6 * LANES;
   // Q per lane, K x2, V x2, P per lane, barriers. No slack for alignment: the kernel checks that
   // the dynamic shared-memory window starts on a 1024-byte boundary and refuses to run otherwise.
-  static constexpr int kSmem = LANES * kTcQTile + 4 * kTcKvTile + LANES * kTcPTile + 256;
+  static constexpr int kBiasBytes = MOD ? LANES * 4 * kTcBiasRing * 4 : 0;
+  static constexpr int kSmem = LANES * kQTile + 2 * kKTile + 2 * kVTile + LANES * kTcPTile + 256 + kBiasBytes;
 };
 
 struct TcParams {
-  const int* block_table;   // this sequence's pages
-  __nv_bfloat16* out;       // [T, Hq, 128]
+  const int* block_table;   // this sequence's pages (with tiles: the whole table)
+  __nv_bfloat16* out;       // [T, Hq, dv]
   int T, Hq, Hkv, pos0, n_qt;
+  int dk, dv;               // key and value row widths in memory
+  const int4* tiles;        // ragged batches: {first row, rows, position of the first row, table row}
+  int max_blocks;
   int window;               // > 0: a query sees only its last `window` keys
   float scale_log2;
+  ScoreMod mod;             // MOD instances
   int* status;
 };
 
-__device__ __forceinline__ float tc_ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
+__device__ __forceinline__ float tc_ex2(float x) { return ex2_approx(x); }
 
-template <int LANES>
-__global__ void __launch_bounds__(TcCfg<LANES>::kThreads, 1)
+template <int LANES, int KP, int VP, bool MOD>
+__global__ void __launch_bounds__(TcCfg<LANES, KP, VP, MOD>::kThreads, 1)
 flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
                         const __grid_constant__ CUtensorMap tmap_k,
                         const __grid_constant__ CUtensorMap tmap_v, TcParams p) {
-  using C = TcCfg<LANES>;
+  using C = TcCfg<LANES, KP, VP, MOD>;
   extern __shared__ __align__(1024) char smem[];
   if (smem_u32(smem) & 1023u) {       // the swizzled tiles need 1024-byte alignment
     if (threadIdx.x == 0 && p.status) atomicExch(p.status, kStatusBadArgument);
     return;
   }
   char* sQ = smem;                        // one tile per lane
-  char* sK = sQ + LANES * kTcQTile;       // two stages
-  char* sV = sK + 2 * kTcKvTile;          // two stages
-  char* sP = sV + 2 * kTcKvTile;          // one tile per lane
+  char* sK = sQ + LANES * C::kQTile;      // two stages
+  char* sV = sK + 2 * C::kKTile;          // two stages
+  char* sP = sV + 2 * C::kVTile;          // one tile per lane
   uint64_t* bars = reinterpret_cast<uint64_t*>(sP + LANES * kTcPTile);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;            // [2]
@@ -101,21 +119,34 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   volatile uint32_t* abort_flag = tmem_slot + 1;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  // long rows of work first: the last query tile walks the most keys
-  const int qt = p.n_qt - 1 - int(blockIdx.x) / p.Hq, h = int(blockIdx.x) % p.Hq;
+  const int h = int(blockIdx.x) % p.Hq;
   const int kvh = h / (p.Hq / p.Hkv);
-  const int q0 = qt * (kTcRows * LANES);
+  // q0: the block's first query row; rows: how many rows from there on are its sequence's; pos_q0:
+  // position of row q0; bt: the sequence's pages
+  int q0, rows, pos_q0;
+  const int* bt;
+  if (p.tiles) {
+    pdl_wait();      // the table may have been written by the launch before this one
+    const int4 tile = p.tiles[int(blockIdx.x) / p.Hq];
+    q0 = tile.x; rows = tile.y; pos_q0 = tile.z;
+    bt = p.block_table + size_t(tile.w) * p.max_blocks;
+  } else {
+    // long rows of work first: the last query tile walks the most keys
+    q0 = (p.n_qt - 1 - int(blockIdx.x) / p.Hq) * (kTcRows * LANES);
+    rows = p.T - q0; pos_q0 = p.pos0 + q0;
+    bt = p.block_table;
+  }
   // steps of lane L: it sees keys [0, kv_end_L); a lane that starts past the last token is idle.
   // With a sliding window the block's steps start at j0, the step that holds the first key its
   // first row can see (later rows mask what lies before their own window).
-  const int j0 = p.window > 0 ? max(0, p.pos0 + q0 - p.window + 1) / kTcKeys : 0;
+  const int j0 = p.window > 0 ? max(0, pos_q0 - p.window + 1) / kTcKeys : 0;
   int n_steps[LANES];
   int n_max = 0, kv_end_max = 1;
 #pragma unroll
   for (int L = 0; L < LANES; ++L) {
-    const int first = q0 + L * kTcRows;
-    const int kv_end = p.pos0 + min(first + kTcRows - 1, p.T - 1) + 1;
-    n_steps[L] = first < p.T ? (kv_end + kTcKeys - 1) / kTcKeys - j0 : 0;
+    const int first = L * kTcRows;
+    const int kv_end = pos_q0 + min(first + kTcRows, rows);
+    n_steps[L] = first < rows ? (kv_end + kTcKeys - 1) / kTcKeys - j0 : 0;
     if (n_steps[L] > 0) { n_max = max(n_max, n_steps[L]); kv_end_max = max(kv_end_max, kv_end); }
   }
   const int last_page = (kv_end_max - 1) / kTcPage;
@@ -160,12 +191,13 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         int active = 0;
 #pragma unroll
         for (int L = 0; L < LANES; ++L) active += n_steps[L] > 0;
-        mbar_arrive_expect_tx(q_full, active * kTcQTile);
+        mbar_arrive_expect_tx(q_full, active * C::kQTile);
 #pragma unroll
         for (int L = 0; L < LANES; ++L) {
           if (n_steps[L] == 0) continue;
-          tma_load_2d(sQ + L * kTcQTile, &tmap_q, q_full, h * kTcHd, q0 + L * kTcRows);
-          tma_load_2d(sQ + L * kTcQTile + kTcQPanel, &tmap_q, q_full, h * kTcHd + 64, q0 + L * kTcRows);
+#pragma unroll
+          for (int c = 0; c < KP; ++c)
+            tma_load_2d(sQ + L * C::kQTile + c * kTcQPanel, &tmap_q, q_full, h * p.dk + c * 64, q0 + L * kTcRows);
         }
       }
       for (int j = 0; j < n_max; ++j) {
@@ -177,26 +209,26 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         for (int pg = 0; pg < kTcPages; ++pg) {
           // pages past the last one this CTA can see repeat it (their keys are masked)
           const int page = min((j + j0) * kTcPages + pg, last_page);
-          y[pg] = (p.block_table[page] * p.Hkv + kvh) * kTcPage;
+          y[pg] = (bt[page] * p.Hkv + kvh) * kTcPage;
         }
         if (!mbar_wait(k_free + s, par, abort_flag)) break;
-        mbar_arrive_expect_tx(k_full + s, kTcKvTile);
+        mbar_arrive_expect_tx(k_full + s, C::kKTile);
         last_k[s] = j;
-        char* kd = sK + s * kTcKvTile;
+        char* kd = sK + s * C::kKTile;
 #pragma unroll
-        for (int pg = 0; pg < kTcPages; ++pg) {
-          tma_load_2d(kd + pg * kTcPageBytes, &tmap_k, k_full + s, 0, y[pg]);
-          tma_load_2d(kd + kTcKvPanel + pg * kTcPageBytes, &tmap_k, k_full + s, 64, y[pg]);
-        }
+        for (int pg = 0; pg < kTcPages; ++pg)
+#pragma unroll
+          for (int c = 0; c < KP; ++c)
+            tma_load_2d(kd + c * kTcKvPanel + pg * kTcPageBytes, &tmap_k, k_full + s, c * 64, y[pg]);
         if (!mbar_wait(v_free + s, par, abort_flag)) break;
-        mbar_arrive_expect_tx(v_full + s, kTcKvTile);
+        mbar_arrive_expect_tx(v_full + s, C::kVTile);
         last_v[s] = j;
-        char* vd = sV + s * kTcKvTile;
+        char* vd = sV + s * C::kVTile;
 #pragma unroll
-        for (int pg = 0; pg < kTcPages; ++pg) {
-          tma_load_2d(vd + pg * kTcPageBytes, &tmap_v, v_full + s, 0, y[pg]);
-          tma_load_2d(vd + kTcKvPanel + pg * kTcPageBytes, &tmap_v, v_full + s, 64, y[pg]);
-        }
+        for (int pg = 0; pg < kTcPages; ++pg)
+#pragma unroll
+          for (int c = 0; c < VP; ++c)
+            tma_load_2d(vd + c * kTcKvPanel + pg * kTcPageBytes, &tmap_v, v_full + s, c * 64, y[pg]);
       }
       if (*abort_flag) {
         // leaving early: let the copies already in flight land before the CTA gives up its
@@ -216,23 +248,23 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     // ---------------------------------------------------------------- MMA issuer
     if (elect_one()) {
       constexpr uint32_t idesc_s = umma_idesc_bf16_f32(128, kTcKeys);
-      constexpr uint32_t idesc_pv = umma_idesc_bf16_f32(128, 128) | kUmmaBMajorMN;
+      constexpr uint32_t idesc_pv = umma_idesc_bf16_f32(128, VP * 64) | kUmmaBMajorMN;
       bool ok = mbar_wait(q_full, 0, abort_flag);
       // S of step j for every lane that still has work
       auto issue_s = [&](int j) -> bool {
         const int s = j & 1;
         const uint32_t u = (j >> 1) & 1;
         if (!mbar_wait(k_full + s, u, abort_flag)) return false;
-        const uint32_t k_addr = smem_u32(sK + s * kTcKvTile);
+        const uint32_t k_addr = smem_u32(sK + s * C::kKTile);
 #pragma unroll
         for (int L = 0; L < LANES; ++L) {
           if (j >= n_steps[L]) continue;
           uint64_t* lb = lane_bars + 6 * L;
           if (!mbar_wait(lb + 2 + s, u ^ 1u, abort_flag)) return false;   // s_free
           tc_fence_after_sync();
-          const uint32_t q_addr = smem_u32(sQ + L * kTcQTile);
+          const uint32_t q_addr = smem_u32(sQ + L * C::kQTile);
 #pragma unroll
-          for (int ks = 0; ks < 8; ++ks) {       // 16 of the 128 head dimensions per product
+          for (int ks = 0; ks < KP * 4; ++ks) {  // 16 of the head dimensions per product
             const uint32_t in_row = (ks & 3) * 32;
             tc_mma_f16(tmem_base + L * 128 + s * kTcKeys,
                        umma_desc_sw128_kmajor(q_addr + (ks >> 2) * kTcQPanel + in_row),
@@ -249,7 +281,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         if (j + 1 < n_max && !issue_s(j + 1)) { ok = false; break; }
         const int s = j & 1;
         if (!mbar_wait(v_full + s, (j >> 1) & 1, abort_flag)) { ok = false; break; }
-        const uint32_t v_addr = smem_u32(sV + s * kTcKvTile);
+        const uint32_t v_addr = smem_u32(sV + s * C::kVTile);
 #pragma unroll
         for (int L = 0; L < LANES; ++L) {
           if (j >= n_steps[L]) continue;
@@ -259,7 +291,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
           const uint32_t p_addr = smem_u32(sP + L * kTcPTile);
 #pragma unroll
           for (int ks = 0; ks < kTcKeys / 16; ++ks) {       // 16 keys per product
-            tc_mma_f16(tmem_base + LANES * 128 + L * 128, umma_desc_sw128_kmajor(p_addr + ks * 32),
+            tc_mma_f16(tmem_base + LANES * 128 + L * (VP * 64), umma_desc_sw128_kmajor(p_addr + ks * 32),
                        umma_desc_sw128_mnmajor(v_addr + ks * 2048, kTcKvPanel), idesc_pv,
                        (j | ks) != 0 ? 1u : 0u);
           }
@@ -276,20 +308,48 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     const int row = quarter * 32 + lane;
     const uint32_t t_lane = uint32_t(quarter * 32) << 16;
     const uint32_t tmem_s = tmem_base + L * 128 + t_lane;
-    const uint32_t tmem_o = tmem_base + LANES * 128 + L * 128 + t_lane;
+    const uint32_t tmem_o = tmem_base + LANES * 128 + L * (VP * 64) + t_lane;
     uint64_t* s_full = lane_bars + 6 * L;
     uint64_t* s_free = s_full + 2;
     uint64_t* p_full = s_full + 4;
     uint64_t* o_done = s_full + 5;
-    const int lane_q0 = q0 + L * kTcRows;
-    const int qrow = lane_q0 + row;
-    const int pos = p.pos0 + qrow;
+    const int lrow = L * kTcRows + row;                // row inside the block
+    const int pos = pos_q0 + lrow;
     const int my_steps = n_steps[LANES == 1 ? 0 : L];
-    const float sc = p.scale_log2;
+    const float sc = MOD ? 1.f : p.scale_log2;         // MOD: scores are final, in base 2
     char* prow = sP + L * kTcPTile + row * 128;
     float m_used = -INFINITY, l = 0.f;
     bool ok = true;
     pdl_wait();
+    // score modifiers of this head; polynomial coefficients with every constant folded in
+    HeadScore hs{};
+    float c0 = 0.f, c1 = 0.f, c2 = 0.f, c3 = 0.f, c4 = 0.f, far_in = 0.f;
+    float* ring = nullptr;
+    int d_low = 0;                                     // smallest distance this warp's step can hold
+    if (MOD) {
+      hs = head_score(p.mod, h);
+      if (hs.capl > 0.f) {
+        const float w = hs.inner * hs.inner;
+        c0 = hs.capl * hs.inner * kTanhP0;
+        c1 = hs.capl * hs.inner * w * kTanhP1;
+        c2 = hs.capl * hs.inner * (w * w) * kTanhP2;
+        c3 = hs.capl * hs.inner * (w * w) * w * kTanhP3;
+        c4 = hs.capl * hs.inner * (w * w) * (w * w) * kTanhP4;
+        far_in = 2.f * kLog2e * hs.inner;
+      } else {
+        c0 = hs.lin;
+      }
+      if (hs.sink != -INFINITY) { m_used = hs.sink; l = 1.f; }
+      ring = reinterpret_cast<float*>(reinterpret_cast<char*>(bars) + 256) + (warp - 2) * kTcBiasRing;
+      d_low = pos_q0 + L * kTcRows + quarter * 32 - j0 * kTcKeys - (kTcKeys - 1);
+      for (int i = lane; i < 128; i += 32) {
+        const int d = d_low + i;
+        const float v = distance_bias(hs, float(max(d, 0)));
+        ring[d & 127] = v;
+        ring[(d & 127) + 128] = v;
+      }
+      __syncwarp();
+    }
 #pragma unroll 1
     for (int j = 0; j < my_steps; ++j) {
       const int sb = j & 1;
@@ -307,7 +367,46 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       if (lane == 0) mbar_arrive(s_free + sb);         // the issuer may overwrite this S now
 
       const int k0 = (j + j0) * kTcKeys;
-      if (k0 + kTcKeys - 1 > p.pos0 + lane_q0) {       // the step touches the diagonal
+      if (MOD) {
+        float amax[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; ++i) amax[i & 3] = fmaxf(amax[i & 3], fabsf(__uint_as_float(r[c][i])));
+        const float top = fmaxf(fmaxf(amax[0], amax[1]), fmaxf(amax[2], amax[3]));
+        const float* bias = ring + (d_low & 127) + lane + (kTcKeys - 1);   // bias[-i]: key k0 + i
+        if (!__any_sync(0xffffffffu, top * fabsf(hs.inner) > kTanhPolyMax)) {
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const float a = __uint_as_float(r[c][i]), w = a * a;
+              const float poly = fmaf(fmaf(fmaf(fmaf(c4, w, c3), w, c2), w, c1), w, c0);
+              r[c][i] = __float_as_uint(fmaf(a, poly, -bias[-(c * 32 + i)]));
+            }
+        } else {
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const float a = __uint_as_float(r[c][i]);
+              const float e = tc_ex2(fminf(a * far_in, 80.f));
+              r[c][i] = __float_as_uint(hs.capl - __fdividef(2.f * hs.capl, 1.f + e) - bias[-(c * 32 + i)]);
+            }
+        }
+        // the next step's 64 new distances (all below the ones held)
+        __syncwarp();
+        d_low -= kTcKeys;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int d = d_low + lane + i * 32;
+          const float v = distance_bias(hs, float(max(d, 0)));
+          ring[d & 127] = v;
+          ring[(d & 127) + 128] = v;
+        }
+        __syncwarp();
+      }
+      if (k0 + kTcKeys - 1 > pos_q0 + L * kTcRows) {   // the step touches the diagonal
         const int vis = pos - k0;                      // keys k0 .. k0+vis are visible to this row
 #pragma unroll
         for (int c = 0; c < NC; ++c)
@@ -342,7 +441,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
           waited = true;
           tc_fence_after_sync();
 #pragma unroll 1
-          for (int c = 0; c < 4; ++c) {
+          for (int c = 0; c < VP * 2; ++c) {
             uint32_t o[32];
             tmem_ld_32x32(tmem_o + c * 32, o);
             tmem_ld_wait();
@@ -387,15 +486,16 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     if (ok && my_steps > 0) {
       tc_fence_after_sync();
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.out + (size_t(min(qrow, p.T - 1)) * p.Hq + h) * kTcHd;
+      __nv_bfloat16* dst = p.out + (size_t(q0 + min(lrow, rows - 1)) * p.Hq + h) * p.dv;
 #pragma unroll 1
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < VP * 2; ++c) {
         uint32_t o[32];
         tmem_ld_32x32(tmem_o + c * 32, o);
         tmem_ld_wait();
-        if (qrow < p.T) {
+        if (lrow < rows) {
 #pragma unroll
           for (int v = 0; v < 4; ++v) {
+            if (c * 32 + v * 8 >= p.dv) break;           // dv is a multiple of 8
             uint4 pk;
             pk.x = pack_bf16(__uint_as_float(o[v * 8]) * inv, __uint_as_float(o[v * 8 + 1]) * inv);
             pk.y = pack_bf16(__uint_as_float(o[v * 8 + 2]) * inv, __uint_as_float(o[v * 8 + 3]) * inv);
@@ -419,15 +519,25 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   pdl_launch_dependents();
 }
 
-template <int LANES>
+template <int LANES, int KP, int VP, bool MOD>
 static int launch_prefill_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
                              TcParams p, int pdl, cudaStream_t st) {
-  auto kern = flash_prefill_tc_kernel<LANES>;
-  constexpr size_t smem = TcCfg<LANES>::kSmem;
+  auto kern = flash_prefill_tc_kernel<LANES, KP, VP, MOD>;
+  using C = TcCfg<LANES, KP, VP, MOD>;
+  constexpr size_t smem = C::kSmem;
   RB_CHECK(set_max_smem(kern, smem));
-  p.n_qt = (p.T + kTcRows * LANES - 1) / (kTcRows * LANES);
-  return launch(kern, dim3(p.n_qt * p.Hq), dim3(TcCfg<LANES>::kThreads), smem, st, pdl != 0, tq, tk,
-                tv, p);
+  if (!p.tiles) p.n_qt = (p.T + kTcRows * LANES - 1) / (kTcRows * LANES);
+  return launch(kern, dim3(p.n_qt * p.Hq), dim3(C::kThreads), smem, st, pdl != 0, tq, tk, tv, p);
+}
+
+static int prefill_tc_maps(CUtensorMap* tq, CUtensorMap* tk, CUtensorMap* tv, const void* q, const void* k_cache,
+                           const void* v_cache, int T, int Hq, int Hkv, int dk, int dv, int num_blocks) {
+  int rc = make_tmap_2d_bf16(tq, q, uint64_t(Hq) * dk, uint64_t(T), uint64_t(Hq) * dk * 2, 64, kTcRows);
+  if (rc) return rc;
+  const uint64_t rows = uint64_t(num_blocks) * Hkv * kTcPage;
+  rc = make_tmap_2d_bf16(tk, k_cache, uint64_t(dk), rows, uint64_t(dk) * 2, 64, kTcPage);
+  if (rc) return rc;
+  return make_tmap_2d_bf16(tv, v_cache, uint64_t(dv), rows, uint64_t(dv) * 2, 64, kTcPage);
 }
 
 }  // namespace rb
@@ -456,22 +566,58 @@ extern "C" int rmlx_flash_prefill_tc(const void* q, const void* k_cache, const v
        reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(out)) & 15)
     return -2;
   CUtensorMap tq, tk, tv;
-  int rc = make_tmap_2d_bf16(&tq, q, uint64_t(Hq) * kTcHd, uint64_t(T), uint64_t(Hq) * kTcHd * 2, 64,
-                             kTcRows);
+  const int rc = prefill_tc_maps(&tq, &tk, &tv, q, k_cache, v_cache, T, Hq, Hkv, kTcHd, kTcHd, num_blocks);
   if (rc) return rc;
-  const uint64_t rows = uint64_t(num_blocks) * Hkv * kTcPage;
-  rc = make_tmap_2d_bf16(&tk, k_cache, kTcHd, rows, kTcHd * 2, 64, kTcPage);
-  if (rc) return rc;
-  rc = make_tmap_2d_bf16(&tv, v_cache, kTcHd, rows, kTcHd * 2, 64, kTcPage);
-  if (rc) return rc;
-  TcParams p;
+  TcParams p{};
   p.block_table = block_table;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.pos0 = pos0;
   p.n_qt = 0;
+  p.dk = p.dv = kTcHd;
+  p.tiles = nullptr; p.max_blocks = 0;
   p.window = window > 0 ? window : 0;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  p.scale_log2 = scale * kLog2e;
   p.status = status;
-  return lanes == 2 ? launch_prefill_tc<2>(tq, tk, tv, p, pdl, st)
-                    : launch_prefill_tc<1>(tq, tk, tv, p, pdl, st);
+  return lanes == 2 ? launch_prefill_tc<2, 2, 2, false>(tq, tk, tv, p, pdl, st)
+                    : launch_prefill_tc<1, 2, 2, false>(tq, tk, tv, p, pdl, st);
+}
+
+// 1 when the form with score modifiers takes these key and value row widths.
+extern "C" int rmlx_flash_prefill_scored_supported(int dk, int dv) {
+  return dk >= 8 && dv >= 8 && dk % 8 == 0 && dv % 8 == 0 && dk <= 128 && dv <= 128;
+}
+
+// Ragged batch with score modifiers. q [T, Hq, dk] and out [T, Hq, dv] bf16, caches [num_blocks, Hkv, 16,
+// dk / dv] bf16 already holding the rows' own keys and values; tiles: n_tiles x {first row, rows (1..128),
+// position of the first row, row of block_table [.., max_blocks]} (int32, device), heaviest first.
+extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, const void* v_cache,
+                                         const int* block_table, int max_blocks, const int* tiles, int n_tiles,
+                                         void* out, int T, int Hq, int Hkv, int dk, int dv, int num_blocks,
+                                         int window, float scale, float softcap, const float* temp,
+                                         const float* r1, const float* r2, const float* sink, int* status,
+                                         int pdl, cudaStream_t st) {
+  if (T < 1 || Hkv < 1 || Hq % Hkv || num_blocks < 1 || n_tiles < 1 || !tiles || (r1 && !r2) ||
+      !rmlx_flash_prefill_scored_supported(dk, dv))
+    return -2;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) |
+       reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(out) |
+       reinterpret_cast<uintptr_t>(tiles)) & 15)
+    return -2;
+  CUtensorMap tq, tk, tv;
+  const int rc = prefill_tc_maps(&tq, &tk, &tv, q, k_cache, v_cache, T, Hq, Hkv, dk, dv, num_blocks);
+  if (rc) return rc;
+  TcParams p{};
+  p.block_table = block_table; p.max_blocks = max_blocks;
+  p.tiles = reinterpret_cast<const int4*>(tiles); p.n_qt = n_tiles;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.pos0 = 0;
+  p.dk = dk; p.dv = dv;
+  p.window = window > 0 ? window : 0;
+  p.scale_log2 = 1.f;
+  p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2; p.mod.sink = sink;
+  p.status = status;
+  if (dk > 64) return dv > 64 ? launch_prefill_tc<1, 2, 2, true>(tq, tk, tv, p, pdl, st)
+                              : launch_prefill_tc<1, 2, 1, true>(tq, tk, tv, p, pdl, st);
+  return dv > 64 ? launch_prefill_tc<1, 1, 2, true>(tq, tk, tv, p, pdl, st)
+                 : launch_prefill_tc<1, 1, 1, true>(tq, tk, tv, p, pdl, st);
 }

@@ -228,18 +228,25 @@ class PagedKvCache:
     ``[blocks, Hkv, page, D/64, 2]`` of (scale, bias) per token and group of 64): half the bytes
     per token. The device kernels quantise on append and expand inside attention
     (csrc/kernels/kv_q8.cu, flash_decode.cu); the counterpart of the reference's host-side
-    QuantizedKvCache (crates/rmlx-nn/src/attention.rs:4438-4680)."""
+    QuantizedKvCache (crates/rmlx-nn/src/attention.rs:4438-4680).
+
+    ``layer_shapes``: one ``(kv_heads, key width, value width)`` per layer, for models whose layers
+    differ or whose keys and values have different widths (``kv_heads`` / ``head_dim`` are then only
+    the first layer's)."""
 
     def __init__(self, num_blocks: int, num_layers: int, kv_heads: int, head_dim: int,
                  dtype=torch.bfloat16, device="cpu", max_seqs: int = 64,
                  max_blocks_per_seq: int = 512, block_size: int = PAGE,
-                 kv_quant: Optional[str] = None):
+                 kv_quant: Optional[str] = None, layer_shapes: Optional[List[tuple]] = None):
         self.manager = make_block_manager(num_blocks, block_size, reserved=1)
         self.num_layers, self.kv_heads, self.head_dim = num_layers, kv_heads, head_dim
         self.block_size = block_size
         if kv_quant not in (None, "q8"):
             raise ValueError(f"unsupported KV quantisation {kv_quant}")
         self.quantized = kv_quant == "q8"
+        if layer_shapes is not None and (self.quantized or len(layer_shapes) != num_layers):
+            raise ValueError("layer_shapes: one entry per layer, 16- or 32-bit caches only")
+        self.layer_shapes = layer_shapes or [(kv_heads, head_dim, head_dim)] * num_layers
         self.dtype = dtype
         if self.quantized:
             if head_dim % 64:
@@ -250,10 +257,10 @@ class PagedKvCache:
             self.k_sb = [torch.zeros(sbs, dtype=torch.bfloat16, device=device) for _ in range(num_layers)]
             self.v_sb = [torch.zeros(sbs, dtype=torch.bfloat16, device=device) for _ in range(num_layers)]
         else:
-            self.k = [torch.zeros(num_blocks, kv_heads, block_size, head_dim, dtype=dtype, device=device)
-                      for _ in range(num_layers)]
-            self.v = [torch.zeros(num_blocks, kv_heads, block_size, head_dim, dtype=dtype, device=device)
-                      for _ in range(num_layers)]
+            self.k = [torch.zeros(num_blocks, h, block_size, dk, dtype=dtype, device=device)
+                      for h, dk, _ in self.layer_shapes]
+            self.v = [torch.zeros(num_blocks, h, block_size, dv, dtype=dtype, device=device)
+                      for h, _, dv in self.layer_shapes]
             self.k_sb = self.v_sb = None
         self.device = torch.device(device)
         self.max_blocks_per_seq = max_blocks_per_seq
@@ -389,6 +396,7 @@ class PagedKvCache:
 
     def bytes_per_token(self) -> int:
         """Cache bytes one token occupies over all layers (K and V)."""
-        per = self.head_dim + (self.head_dim // 64) * 4 if self.quantized else \
-            self.head_dim * torch.empty(0, dtype=self.dtype).element_size()
-        return 2 * self.num_layers * self.kv_heads * per
+        if self.quantized:
+            return 2 * self.num_layers * self.kv_heads * (self.head_dim + (self.head_dim // 64) * 4)
+        size = torch.empty(0, dtype=self.dtype).element_size()
+        return sum(h * (dk + dv) for h, dk, dv in self.layer_shapes) * size

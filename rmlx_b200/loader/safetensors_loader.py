@@ -189,9 +189,11 @@ def build_weights(cfg: TransformerConfig, tensors: Dict[str, torch.Tensor],
 
 def load_model(model_dir: str, device="cpu", dtype=torch.bfloat16,
                layout: Optional[ParallelLayout] = None):
-    """``(TransformerModel-ready ModelWeights, config)`` for one rank from a checkpoint folder."""
-    cfg, quant = read_config(model_dir)
-    return build_weights(cfg, load_tensors(model_dir), quant, device, dtype, layout), cfg
+    """``(weights, config)`` for one rank from a checkpoint folder: what the model class of its family
+    (``models.registry``) is built from."""
+    from ..models.registry import family_of, read_json
+    config = read_json(model_dir)
+    return family_of(config).weights(model_dir, config, device, dtype, layout)
 
 
 def save_checkpoint(model_dir: str, cfg: TransformerConfig, state_dict: Dict[str, torch.Tensor],

@@ -1,0 +1,93 @@
+"""Ragged batches: one forward pass over the new tokens of several sequences at once, prompt portions
+beside single decoded tokens.
+
+``RaggedBatch`` turns (sequence, tokens) entries into the device arrays the kernels read: token ids,
+positions, the block-table row of every token, the query tiles of the entries with several tokens
+(tensor-core prompt attention) and the rows of those with one (split-KV decode attention). Everything
+travels in one pinned copy."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import List, Optional, Sequence
+
+import torch
+
+TILE_ROWS = 128
+
+
+@dataclass
+class Entry:
+    """The next tokens of one sequence and the places among them whose logits are wanted."""
+    seq_id: int
+    tokens: Sequence[int]
+    want: Sequence[int] = ()
+
+
+def query_tiles(starts: Sequence[int], lens: Sequence[int], pos0: Sequence[int], slots: Sequence[int],
+                tile_rows: int = TILE_ROWS) -> List[tuple]:
+    """(first row, rows, position of the first row, table row) of every query tile of the entries with
+    more than one token, the tiles that see most keys first."""
+    tiles = []
+    for start, n, pos, slot in zip(starts, lens, pos0, slots):
+        if n < 2:
+            continue
+        for lo in range(0, n, tile_rows):
+            tiles.append((start + lo, min(tile_rows, n - lo), pos + lo, slot))
+    tiles.sort(key=lambda t: -(t[2] + t[1]))
+    return tiles
+
+
+class RaggedBatch:
+    """``plan`` is host arithmetic; ``upload`` puts the arrays on the cache's device."""
+
+    def __init__(self, entries: Sequence[Entry], pos0: Sequence[int], slots: Sequence[int]):
+        if not entries or any(len(e.tokens) < 1 for e in entries):
+            raise ValueError("a batch needs at least one entry, and every entry at least one token")
+        if len({e.seq_id for e in entries}) != len(entries):
+            raise ValueError("a sequence appears twice in one batch")
+        self.entries = list(entries)
+        self.lens = [len(e.tokens) for e in entries]
+        self.starts, n = [], 0
+        for l in self.lens:
+            self.starts.append(n)
+            n += l
+        self.num_tokens = n
+        self.pos0, self.slots = list(pos0), list(slots)
+        self.tiles_host = query_tiles(self.starts, self.lens, self.pos0, self.slots)
+        self.single_host = [s for s, l in zip(self.starts, self.lens) if l == 1]
+        self.want_host = [s + w for s, e, l in zip(self.starts, self.entries, self.lens) for w in e.want]
+        for e, l in zip(self.entries, self.lens):
+            if any(not 0 <= w < l for w in e.want):
+                raise ValueError("wanted place outside the entry's tokens")
+        # longest context a single-token row sees (plans its KV splits)
+        self.single_len = max([p + 1 for p, l in zip(self.pos0, self.lens) if l == 1], default=0)
+        self.tokens: Optional[torch.Tensor] = None
+
+    @staticmethod
+    def plan(entries: Sequence[Entry], cache) -> "RaggedBatch":
+        """Positions and table rows from the cache's current state."""
+        return RaggedBatch(entries, [cache.seq_len(e.seq_id) for e in entries],
+                           [cache.slot_of[e.seq_id] for e in entries])
+
+    def upload(self, device) -> "RaggedBatch":
+        n, tiles = self.num_tokens, self.tiles_host
+        parts = [torch.tensor([x for t in tiles for x in t], dtype=torch.int32),     # 16-byte records first
+                 torch.cat([torch.as_tensor(e.tokens, dtype=torch.int32).reshape(-1) for e in self.entries]),
+                 torch.cat([torch.arange(p, p + l, dtype=torch.int32) for p, l in zip(self.pos0, self.lens)]),
+                 torch.repeat_interleave(torch.tensor(self.slots, dtype=torch.int32), torch.tensor(self.lens)),
+                 torch.tensor(self.single_host, dtype=torch.int32),
+                 torch.tensor(self.want_host, dtype=torch.int32)]
+        flat = torch.cat(parts)
+        device = torch.device(device)
+        if device.type == "cuda":
+            flat = flat.pin_memory().to(device, non_blocking=True)
+        out, at = [], 0
+        for p in parts:
+            out.append(flat[at:at + p.numel()])
+            at += p.numel()
+        self.tiles = out[0].view(-1, 4) if tiles else None
+        self.tokens, self.positions, self.token_seq = out[1], out[2], out[3]
+        self.single = out[4] if self.single_host else None
+        self.want = out[5]
+        assert self.tokens.numel() == n
+        return self

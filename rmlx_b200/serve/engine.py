@@ -3,16 +3,21 @@
 crates/rmlx-nn/src/prefix_cache.rs:9-17): requests are admitted by the continuous-batching
 scheduler, prompts run in chunks through ``TransformerModel.prefill``, decode steps run batched,
 on CUDA through the graph-captured ``CachedDecode``, on CPU through the library-kernel forward.
+
+Models with ``mixed_batches`` run a step that has a prompt chunk as ONE ragged batch, the chunk beside
+the decoded tokens (``run_entries``); steps without one go through their captured decode engine.
+``open_sequence`` / ``run_entries`` / ``close_sequence`` are the same step under the caller's control:
+which tokens of which sequences run next, and which positions' logits come back.
 """
 from __future__ import annotations
 
 import itertools
-import os
-from typing import Dict, List, Optional
+from typing import Dict, List, Optional, Sequence
 
 import torch
 
 from ..config import SamplerConfig, SchedulerConfig
+from ..models.ragged import Entry
 from ..models.transformer import TransformerModel
 from ..parallel.warmup import Warmup, WarmupResult
 from ..utils.metrics import PERF
@@ -60,6 +65,7 @@ class ServingEngine:
         self.released_pages = 0               # sliding-window models: pages returned to the pool
         self._engine = None
         self._bound: List[int] = []
+        self.mixed = bool(getattr(model, "mixed_batches", False))
         self.guard = precision_guard
         self.guard_every = max(1, guard_every)
         self.guard_warnings = 0
@@ -69,23 +75,7 @@ class ServingEngine:
         self._comm = comm
         self._warmup = Warmup()
         if model.device.type == "cuda":
-            # prompts through the tensor-core path; decode through the mat-vec engine for small
-            # batches and through the tensor-core path (batch = GEMM rows) for larger ones
-            from .. import _lib
-            from ..models.decode_engine import CachedDecode
-            from ..models.prefill import BatchedDecode, enable_native_prefill
-            enable_native_prefill(model)
-            # measured on the 60-layer MoE model (4-bit weights): the mat-vec engine takes 377 us
-            # per layer at 8 rows against 434 for the tensor-core path, which wins from 16 rows on
-            matvec_max = int(os.environ.get("RMLX_MATVEC_MAX_BATCH", "8"))
-            if scfg.max_batch_size <= matvec_max:
-                self._engine = CachedDecode(model, self.cache, max_batch=scfg.max_batch_size, comm=comm,
-                                            greedy=True)
-            else:
-                try:
-                    self._engine = BatchedDecode(model, self.cache, max_batch=scfg.max_batch_size)
-                except ImportError:
-                    self._engine = None          # shapes outside the kernels: library-kernel forward
+            self._engine = model.make_decode_engine(self.cache, scfg.max_batch_size, comm)
 
     def _on_admit(self, seq_id: int) -> int:
         """New sequence; with a prefix cache, start it from the cached pages of the longest
@@ -175,6 +165,63 @@ class ServingEngine:
         self.outputs[sid] = []
         return sid
 
+    # ------------------------------------------------------------------ explicit steps
+    def open_sequence(self) -> int:
+        """A sequence outside the scheduler's queue; its tokens come through ``run_entries``."""
+        sid = next(self._ids)
+        self.cache.add_sequence(sid)
+        return sid
+
+    def close_sequence(self, seq_id: int) -> None:
+        """Give back the sequence's pages and slot."""
+        self.cache.free_sequence(seq_id)
+        self._bound = []
+
+    @torch.no_grad()
+    def run_entries(self, entries: Sequence[Entry]) -> torch.Tensor:
+        """One step over the given tokens: every entry continues its sequence from what the cache
+        holds. Returns the wanted logits, fp32 [wanted, vocab], in the order of the entries and of
+        their ``want``. A step of single tokens runs through the captured decode engine, any other
+        as one ragged batch (models without ``mixed_batches``: entry by entry)."""
+        if len({e.seq_id for e in entries}) != len(entries):
+            raise ValueError("a sequence appears twice in one step")
+        self._bound = []
+        if self._engine is not None and len(entries) <= self.sched.cfg.max_batch_size and \
+                all(len(e.tokens) == 1 for e in entries):
+            self._engine.bind([e.seq_id for e in entries], [int(e.tokens[0]) for e in entries])
+            self._engine.reserve(1)
+            self._engine.step()
+            rows = [i for i, e in enumerate(entries) for _ in e.want]
+            return self._engine.logits[rows].float()
+        if self.mixed:
+            return self.model.forward_batch(entries, self.cache)
+        parts = []
+        for e in entries:
+            toks = torch.tensor(list(e.tokens), device=self.model.device)
+            logits = self.model.prefill(toks, self.cache, e.seq_id, all_logits=True)
+            parts.append(logits[list(e.want)].float())
+        return torch.cat(parts, 0)
+
+    def _run_mixed(self, plan) -> Dict[int, int]:
+        """The plan's prompt chunk and decoded tokens as one batch; returns the sampled tokens."""
+        lo, hi = plan.prefill_chunk_range
+        entries = [Entry(m.seq_id, self.sched.prompt_chunk(m.seq_id, (lo, hi)),
+                         [hi - lo - 1] if hi >= m.prompt_len else ()) for m in plan.prefill_seqs]
+        self.prefill_tokens += (hi - lo) * len(entries)
+        self._decode_steps += bool(plan.decode_seqs)
+        entries += [Entry(m.seq_id, [self.last_token[m.seq_id]], [0]) for m in plan.decode_seqs]
+        ids = [e.seq_id for e in entries if len(e.want)]
+        logits = self.run_entries(entries)
+        if not ids:
+            return {}
+        if self.guard is not None:
+            self._guard_check(logits)
+        if not self.sample_on_device:
+            PERF.record_d2h(logits)
+            logits = logits.cpu()
+        toks = self.sampler.sample_batch(logits, [self.outputs[s] for s in ids])
+        return {s: int(t) for s, t in zip(ids, toks)}
+
     def step(self) -> Dict[int, int]:
         """One scheduler step. Returns the tokens produced in it (seq_id -> token)."""
         waiting_len = self.sched.first_waiting_prompt_len() if self.prefix is not None else None
@@ -188,7 +235,10 @@ class ServingEngine:
         self._finished = {}
         produced: Dict[int, int] = {}
         dev = self.model.device
-        for meta in plan.prefill_seqs:
+        mixed = self.mixed and bool(plan.prefill_seqs)
+        if mixed:
+            produced = self._run_mixed(plan)
+        for meta in () if mixed else plan.prefill_seqs:
             lo, hi = plan.prefill_chunk_range
             chunk = torch.tensor(self.sched.prompt_chunk(meta.seq_id, (lo, hi)), device=dev)
             logits = self.model.prefill(chunk, self.cache, meta.seq_id)
@@ -199,7 +249,7 @@ class ServingEngine:
                 tok = self.sampler.sample_token(logits[0].float().cpu(), self.outputs[meta.seq_id])
                 produced[meta.seq_id] = tok
         ids = [m.seq_id for m in plan.decode_seqs]
-        if ids:
+        if ids and not mixed:
             toks = self._decode(ids)
             for sid, tok in zip(ids, toks):
                 produced[sid] = tok
