@@ -55,7 +55,15 @@ def parse():
     ap.add_argument("--arms", default="auto",
                     help="comma list of extra arms: bf16, nccl_cublas; 'auto' = both from 2 GPUs on, "
                          "'none' = headline only")
-    return ap.parse_args()
+    ap.add_argument("--suite", default="headline", choices=["headline", "parallel_block"],
+                    help="parallel_block: the parallel-block decoder beside the dense one at equal size "
+                         "(benchmarks/bench_parallel_block.py, which takes the remaining options); the default "
+                         "is the headline workload")
+    args, rest = ap.parse_known_args()
+    if args.suite == "headline" and rest:
+        ap.error(f"unrecognized arguments: {' '.join(rest)}")
+    args.rest = rest
+    return args
 
 
 class ClockSampler:
@@ -313,6 +321,10 @@ def main():
     args = parse()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.suite == "parallel_block":
+        sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "benchmarks"))
+        import bench_parallel_block
+        return bench_parallel_block.main(args.rest)
     world = int(os.environ.get("WORLD_SIZE", "1"))
     if args.gpus != world and world == 1 and args.gpus > 1:
         print(f"bench.py: --gpus {args.gpus} needs torchrun with {args.gpus} ranks", file=sys.stderr)

@@ -36,18 +36,21 @@ __device__ __forceinline__ float ex2_approx(float x) {
   return y;
 }
 
-// tanh with small relative error everywhere: the polynomial near zero, 1 - 2 / (1 + e^(2u)) beyond
-// (which saturates to +-1 without overflow trouble: the exponential may become 0 or inf).
-__device__ __forceinline__ float tanh_score(float u) {
+// tanh for |u| <= kTanhPolyMax.
+__device__ __forceinline__ float tanh_near(float u) {
   const float w = u * u;
-  const float near = u * fmaf(fmaf(fmaf(fmaf(kTanhP4, w, kTanhP3), w, kTanhP2), w, kTanhP1), w, kTanhP0);
+  return u * fmaf(fmaf(fmaf(fmaf(kTanhP4, w, kTanhP3), w, kTanhP2), w, kTanhP1), w, kTanhP0);
+}
+// tanh with small relative error everywhere: the polynomial near zero, 1 - 2 / (1 + e^(2u)) beyond
+// (which saturates to +-1 without overflow trouble).
+__device__ __forceinline__ float tanh_any(float u) {
   const float far = 1.f - __fdividef(2.f, 1.f + ex2_approx(fminf(u, 40.f) * (2.f * kLog2e)));
-  return fabsf(u) <= kTanhPolyMax ? near : far;
+  return fabsf(u) <= kTanhPolyMax ? tanh_near(u) : far;
 }
 
 // One head's modifiers, in base-2 units.
 struct HeadScore {
-  float lin;       // scale * temp * log2 e
+  float lin;       // scale * temp * log2 e without a cap, else 0
   float inner;     // scale * temp / softcap, 0 without a cap
   float capl;      // softcap * log2 e, 0 without a cap
   float r1, r2;    // r1 as given: r1 * log2(1 + r2 d) is already r1 * ln(..) in base-2 units
@@ -57,7 +60,7 @@ struct HeadScore {
 __device__ __forceinline__ HeadScore head_score(const ScoreMod& m, int h) {
   HeadScore s;
   const float st = m.scale * (m.temp ? m.temp[h] : 1.f);
-  s.lin = st * kLog2e;
+  s.lin = m.softcap > 0.f ? 0.f : st * kLog2e;
   s.inner = m.softcap > 0.f ? st / m.softcap : 0.f;
   s.capl = m.softcap > 0.f ? m.softcap * kLog2e : 0.f;
   s.r1 = m.r1 ? m.r1[h] : 0.f;
@@ -70,10 +73,22 @@ __device__ __forceinline__ float distance_bias(const HeadScore& s, float dist) {
   return s.r1 * __log2f(fmaf(s.r2, dist, 1.f));
 }
 
-// Base-2 score of a dot product at distance i - j >= 0.
-__device__ __forceinline__ float score_base2(float dot, const HeadScore& s, float dist) {
-  const float t = s.capl > 0.f ? s.capl * tanh_score(dot * s.inner) : dot * s.lin;
-  return t - distance_bias(s, dist);
+// Base-2 scores of N dot products of one head at distances dist[i] (i - j, taken as 0 where
+// negative), in place and without branches per score. `near`: every |dot * inner| is within the
+// polynomial's range.
+template <int N>
+__device__ __forceinline__ void scores_base2(float* dot, const HeadScore& s, const float* dist, bool near) {
+  float th[N];
+  if (near) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) th[i] = tanh_near(dot[i] * s.inner);
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) th[i] = tanh_any(dot[i] * s.inner);
+  }
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+    dot[i] = fmaf(s.capl, th[i], dot[i] * s.lin) - distance_bias(s, fmaxf(dist[i], 0.f));
 }
 
 }  // namespace rb

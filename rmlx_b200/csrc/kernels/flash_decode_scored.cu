@@ -75,6 +75,24 @@ __device__ __forceinline__ float fs_block_sum(float v, float* red) {
   return t;
 }
 
+// One warp copies a page of 16 rows of `chunks` 16-byte pieces into swizzled rows of ROW_BYTES.
+template <int ROW_BYTES>
+__device__ __forceinline__ void fs_copy_page(char* dst, const char* src, int chunks, int lane) {
+  constexpr int FULL = ROW_BYTES / 16;
+  if (chunks == FULL) {
+#pragma unroll
+    for (int u = 0; u < kFsPage * FULL / 32; ++u) {
+      const int i = u * 32 + lane, r = i / FULL, c = i % FULL;
+      fs_cp_async16(dst + r * ROW_BYTES + ((c ^ (r & 7)) << 4), src + i * 16);
+    }
+  } else {
+    for (int i = lane; i < kFsPage * chunks; i += 32) {
+      const int r = i / chunks, c = i - r * chunks;
+      fs_cp_async16(dst + r * ROW_BYTES + ((c ^ (r & 7)) << 4), src + i * 16);
+    }
+  }
+}
+
 template <int DK, int DV, int NST>
 __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParams p) {
   constexpr int KS = DK / 16;            // k-steps of the QK^T product
@@ -95,8 +113,9 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   const int g = lane >> 2, t = lane & 3;
 
   pdl_launch_dependents();
-  // shared memory starts at zero: the columns past dkp / dvp are never written again
-  for (int i = lane; i < NST * STAGE / 16; i += 32) reinterpret_cast<uint4*>(wsm)[i] = make_uint4(0u, 0u, 0u, 0u);
+  // narrow heads: shared memory starts at zero, the columns past dkp / dvp are never written again
+  if (p.dkp < DK || p.dvp < DV)
+    for (int i = lane; i < NST * STAGE / 16; i += 32) reinterpret_cast<uint4*>(wsm)[i] = make_uint4(0u, 0u, 0u, 0u);
   pdl_wait();
   const int b = p.rows ? p.rows[lb] : lb;
   const int len = p.positions[b] + 1;
@@ -108,29 +127,74 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   const int pg1 = min(pg0 + pg_per_split, pg_end);
   const int* bt = p.block_table + size_t(p.table_rows ? p.table_rows[b] : b) * p.max_blocks;
 
+  // ---- ask for the first pages before anything else, so that their latency runs beside the query
+  // staging. Fused form: the page of the new token waits until the key and value are in it. ----
+  const int kch = p.dkp >> 3, vch = p.dvp >> 3;      // 16-byte chunks per row in global memory
+  auto issue = [&](int pg, int stage) {
+    const int blk = RB_BOUNDS(pg, p.max_blocks) ? bt[pg] : 0;
+    const size_t pgi = (size_t(blk) * p.Hkv + kvh) * kFsPage;
+    char* kd = wsm + stage * STAGE;
+    fs_copy_page<DK * 2>(kd, reinterpret_cast<const char*>(p.k_cache + pgi * p.dkp), kch, lane);
+    fs_copy_page<DV * 2>(kd + K_PAGE, reinterpret_cast<const char*>(p.v_cache + pgi * p.dvp), vch, lane);
+  };
+
+  const bool owner = p.raw && pg0 < pg1 && pg1 == pg_end;    // this split ends the sequence
+  const int late = owner ? pg_end - 1 : -1;
+  __syncwarp();                                              // the warp's zero fill is complete
+  int pg = pg0 + warp;
+#pragma unroll
+  for (int s = 0; s < NST; ++s) {
+    if (pg + s * kFsWarps < pg1 && pg + s * kFsWarps != late) issue(pg + s * kFsWarps, s);
+    fs_commit();
+  }
+
   // ---- queries of this tile: 16 rows (heads beyond G are zero) ----
   if (p.raw) {
     const float* row = p.raw + size_t(b) * p.raw_ld;
     const int nq = p.Hq * p.dim, nk = p.Hkv * p.dim;
+    // this thread's share of the tile's queries, un-normalised but weighted (independent loads)
+    constexpr int QPT = 16 * DK / kFsThreads;
+    float qv[QPT];
+    const int q_rows = min(16, p.G - gt * 16);
+#pragma unroll
+    for (int u = 0; u < QPT; ++u) {
+      const int i = u * kFsThreads + threadIdx.x, r = i / DK, d = i % DK;
+      const int src = (kvh * p.G + gt * 16 + r) * p.dim + d;
+      qv[u] = (r < q_rows && d < p.dim) ? __ldcg(row + src) * p.q_w[src] : 0.f;
+    }
     float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < nq + nk; i += kFsThreads) {
-      const float v = __ldcg(row + i);
-      if (i < nq) sq += v * v; else sk += v * v;
+    if (((nq | nk | p.raw_ld) & 3) == 0) {
+      const float4* row4 = reinterpret_cast<const float4*>(row);
+      const int n4 = (nq + nk) >> 2, q4 = nq >> 2;
+      for (int i0 = threadIdx.x; i0 < n4; i0 += kFsThreads * 8) {
+        float4 v[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+          const int i = i0 + u * kFsThreads;
+          v[u] = i < n4 ? __ldcg(row4 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+          const float s = v[u].x * v[u].x + v[u].y * v[u].y + v[u].z * v[u].z + v[u].w * v[u].w;
+          if (i0 + u * kFsThreads < q4) sq += s; else sk += s;
+        }
+      }
+    } else {
+      for (int i = threadIdx.x; i < nq + nk; i += kFsThreads) {
+        const float v = __ldcg(row + i);
+        if (i < nq) sq += v * v; else sk += v * v;
+      }
     }
     sq = fs_block_sum(sq, red);
     sk = fs_block_sum(sk, red);
     const float iq = 1.f / sqrtf(sq / float(nq) + p.eps), ik = 1.f / sqrtf(sk / float(nk) + p.eps);
-    for (int i = threadIdx.x; i < 16 * DK; i += kFsThreads) {
-      const int r = i / DK, d = i % DK, h = gt * 16 + r;
-      float v = 0.f;
-      if (h < p.G && d < p.dim) {
-        const int src = (kvh * p.G + h) * p.dim + d;
-        v = __ldcg(row + src) * iq * p.q_w[src];
-      }
-      sQ[r][d] = __float2bfloat16_rn(v);
+#pragma unroll
+    for (int u = 0; u < QPT; ++u) {
+      const int i = u * kFsThreads + threadIdx.x;
+      sQ[i / DK][i % DK] = __float2bfloat16_rn(qv[u] * iq);
     }
-    if (pg0 < pg1 && pg1 == pg_end && RB_BOUNDS((len - 1) / kFsPage, p.max_blocks)) {
-      // this split ends the sequence: append the new key and value before reading its page
+    if (owner && RB_BOUNDS((len - 1) / kFsPage, p.max_blocks)) {
+      // append the new key and value before this block reads their page
       const size_t slot = (size_t(bt[(len - 1) / kFsPage]) * p.Hkv + kvh) * kFsPage + (len - 1) % kFsPage;
       __nv_bfloat16* kd = p.k_cache + slot * p.dkp;
       __nv_bfloat16* vd = p.v_cache + slot * p.dvp;
@@ -155,7 +219,8 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
     const int h = gt * 16 + threadIdx.x;
     s_sink[threadIdx.x] = (h < p.G && p.mod.sink) ? p.mod.sink[kvh * p.G + h] * kLog2e : -INFINITY;
   }
-  __syncthreads();      // queries staged, zero fill done, the appended key / value written
+  const bool upper = p.G - gt * 16 > 8;      // rows 8 .. 15 of the tile hold heads
+  __syncthreads();      // queries staged, the appended key / value written
 
   uint32_t qa[KS][4];
 #pragma unroll
@@ -171,34 +236,12 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   for (int j = 0; j < NT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
 
-  const int kch = p.dkp >> 3, vch = p.dvp >> 3;      // 16-byte chunks per row in global memory
-  auto copy_page = [&](char* dst, const char* src, int chunks, int row_bytes) {
-    if (chunks * 16 == row_bytes) {                  // full rows: the page is one contiguous run
-      const int sh = row_bytes == 256 ? 4 : 3;
-      for (int i = lane; i < kFsPage * chunks; i += 32) {
-        const int r = i >> sh, c = i & (chunks - 1);
-        fs_cp_async16(dst + r * row_bytes + ((c ^ (r & 7)) << 4), src + i * 16);
-      }
-    } else {
-      for (int i = lane; i < kFsPage * chunks; i += 32) {
-        const int r = i / chunks, c = i - r * chunks;
-        fs_cp_async16(dst + r * row_bytes + ((c ^ (r & 7)) << 4), src + i * 16);
-      }
-    }
-  };
-  auto issue = [&](int pg, int stage) {
-    const int blk = RB_BOUNDS(pg, p.max_blocks) ? bt[pg] : 0;
-    const size_t pgi = (size_t(blk) * p.Hkv + kvh) * kFsPage;
-    char* kd = wsm + stage * STAGE;
-    copy_page(kd, reinterpret_cast<const char*>(p.k_cache + pgi * p.dkp), kch, DK * 2);
-    copy_page(kd + K_PAGE, reinterpret_cast<const char*>(p.v_cache + pgi * p.dvp), vch, DV * 2);
-  };
-
-  int pg = pg0 + warp;
+  if (owner) {
 #pragma unroll
-  for (int s = 0; s < NST; ++s) {
-    if (pg + s * kFsWarps < pg1) issue(pg + s * kFsWarps, s);
+    for (int s = 0; s < NST; ++s)
+      if (pg + s * kFsWarps == late) issue(late, s);
     fs_commit();
+    fs_wait<0>();
   }
   int stage = 0;
   for (; pg < pg1; pg += kFsWarps) {
@@ -218,12 +261,21 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
     const int tok0 = pg * kFsPage + t * 2;
     float sv[8] = {s0[0], s0[1], s1[0], s1[1], s0[2], s0[3], s1[2], s1[3]};
     const int tk[4] = {tok0, tok0 + 1, tok0 + 8, tok0 + 9};
+    float dist[4], top0 = 0.f, top1 = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      dist[i] = float(len - 1 - tk[i]);
+      top0 = fmaxf(top0, fabsf(sv[i]));
+      top1 = fmaxf(top1, fabsf(sv[4 + i]));
+    }
+    const bool near = !__any_sync(0xffffffffu, fmaxf(top0 * fabsf(hs0.inner), top1 * fabsf(hs1.inner)) > kTanhPolyMax);
+    scores_base2<4>(sv, hs0, dist, near);
+    if (upper) scores_base2<4>(sv + 4, hs1, dist, near);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const bool ok = tk[i] < len && tk[i] >= first;
-      const float dist = float(len - 1 - tk[i]);
-      sv[i] = ok ? score_base2(sv[i], hs0, dist) : -INFINITY;
-      sv[4 + i] = ok ? score_base2(sv[4 + i], hs1, dist) : -INFINITY;
+      sv[i] = ok ? sv[i] : -INFINITY;
+      sv[4 + i] = ok ? sv[4 + i] : -INFINITY;
     }
     float mx0 = fmaxf(fmaxf(sv[0], sv[1]), fmaxf(sv[2], sv[3]));
     float mx1 = fmaxf(fmaxf(sv[4], sv[5]), fmaxf(sv[6], sv[7]));

@@ -93,6 +93,26 @@ struct TcParams {
 
 __device__ __forceinline__ float tc_ex2(float x) { return ex2_approx(x); }
 
+// Pairs of fp32 values in one 64-bit register (one issue slot for two operations).
+__device__ __forceinline__ uint64_t pair2(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ void unpair2(uint64_t v, uint32_t& lo, uint32_t& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=r"(lo), "=r"(hi) : "l"(v));
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
 template <int LANES, int KP, int VP, bool MOD>
 __global__ void __launch_bounds__(TcCfg<LANES, KP, VP, MOD>::kThreads, 1)
 flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
@@ -323,28 +343,30 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     pdl_wait();
     // score modifiers of this head; polynomial coefficients with every constant folded in
     HeadScore hs{};
-    float c0 = 0.f, c1 = 0.f, c2 = 0.f, c3 = 0.f, c4 = 0.f, far_in = 0.f;
+    float far_in = 0.f;
+    uint64_t p0 = 0, p1 = 0, p2 = 0, p3 = 0, p4 = 0;
     float* ring = nullptr;
     int d_low = 0;                                     // smallest distance this warp's step can hold
     if (MOD) {
       hs = head_score(p.mod, h);
       if (hs.capl > 0.f) {
-        const float w = hs.inner * hs.inner;
-        c0 = hs.capl * hs.inner * kTanhP0;
-        c1 = hs.capl * hs.inner * w * kTanhP1;
-        c2 = hs.capl * hs.inner * (w * w) * kTanhP2;
-        c3 = hs.capl * hs.inner * (w * w) * w * kTanhP3;
-        c4 = hs.capl * hs.inner * (w * w) * (w * w) * kTanhP4;
+        const float w = hs.inner * hs.inner, f = hs.capl * hs.inner;
+        auto both = [](float v) { return pair2(v, v); };
+        p0 = both(f * kTanhP0);
+        p1 = both(f * w * kTanhP1);
+        p2 = both(f * (w * w) * kTanhP2);
+        p3 = both(f * (w * w) * w * kTanhP3);
+        p4 = both(f * (w * w) * (w * w) * kTanhP4);
         far_in = 2.f * kLog2e * hs.inner;
       } else {
-        c0 = hs.lin;
+        p0 = pair2(hs.lin, hs.lin);
       }
       if (hs.sink != -INFINITY) { m_used = hs.sink; l = 1.f; }
       ring = reinterpret_cast<float*>(reinterpret_cast<char*>(bars) + 256) + (warp - 2) * kTcBiasRing;
       d_low = pos_q0 + L * kTcRows + quarter * 32 - j0 * kTcKeys - (kTcKeys - 1);
       for (int i = lane; i < 128; i += 32) {
         const int d = d_low + i;
-        const float v = distance_bias(hs, float(max(d, 0)));
+        const float v = -distance_bias(hs, float(max(d, 0)));
         ring[d & 127] = v;
         ring[(d & 127) + 128] = v;
       }
@@ -379,10 +401,11 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
 #pragma unroll
           for (int c = 0; c < NC; ++c)
 #pragma unroll
-            for (int i = 0; i < 32; ++i) {
-              const float a = __uint_as_float(r[c][i]), w = a * a;
-              const float poly = fmaf(fmaf(fmaf(fmaf(c4, w, c3), w, c2), w, c1), w, c0);
-              r[c][i] = __float_as_uint(fmaf(a, poly, -bias[-(c * 32 + i)]));
+            for (int i = 0; i < 32; i += 2) {
+              const uint64_t a = pair2(__uint_as_float(r[c][i]), __uint_as_float(r[c][i + 1]));
+              const uint64_t w = mul2(a, a);
+              const uint64_t poly = fma2(fma2(fma2(fma2(p4, w, p3), w, p2), w, p1), w, p0);
+              unpair2(fma2(a, poly, pair2(bias[-(c * 32 + i)], bias[-(c * 32 + i + 1)])), r[c][i], r[c][i + 1]);
             }
         } else {
 #pragma unroll
@@ -391,7 +414,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
             for (int i = 0; i < 32; ++i) {
               const float a = __uint_as_float(r[c][i]);
               const float e = tc_ex2(fminf(a * far_in, 80.f));
-              r[c][i] = __float_as_uint(hs.capl - __fdividef(2.f * hs.capl, 1.f + e) - bias[-(c * 32 + i)]);
+              r[c][i] = __float_as_uint(hs.capl - __fdividef(2.f * hs.capl, 1.f + e) + bias[-(c * 32 + i)]);
             }
         }
         // the next step's 64 new distances (all below the ones held)
@@ -400,7 +423,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
           const int d = d_low + lane + i * 32;
-          const float v = distance_bias(hs, float(max(d, 0)));
+          const float v = -distance_bias(hs, float(max(d, 0)));
           ring[d & 127] = v;
           ring[(d & 127) + 128] = v;
         }
@@ -588,15 +611,15 @@ extern "C" int rmlx_flash_prefill_scored_supported(int dk, int dv) {
 }
 
 // Ragged batch with score modifiers. q [T, Hq, dk] and out [T, Hq, dv] bf16, caches [num_blocks, Hkv, 16,
-// dk / dv] bf16 already holding the rows' own keys and values; tiles: n_tiles x {first row, rows (1..128),
+// dk / dv] bf16 already holding the rows' own keys and values; tiles: n_tiles x {first row, rows (1 .. lanes * 128),
 // position of the first row, row of block_table [.., max_blocks]} (int32, device), heaviest first.
 extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, const void* v_cache,
                                          const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                                          void* out, int T, int Hq, int Hkv, int dk, int dv, int num_blocks,
                                          int window, float scale, float softcap, const float* temp,
-                                         const float* r1, const float* r2, const float* sink, int* status,
-                                         int pdl, cudaStream_t st) {
-  if (T < 1 || Hkv < 1 || Hq % Hkv || num_blocks < 1 || n_tiles < 1 || !tiles || (r1 && !r2) ||
+                                         const float* r1, const float* r2, const float* sink, int lanes,
+                                         int* status, int pdl, cudaStream_t st) {
+  if (T < 1 || (lanes != 1 && lanes != 2) || Hkv < 1 || Hq % Hkv || num_blocks < 1 || n_tiles < 1 || !tiles || (r1 && !r2) ||
       !rmlx_flash_prefill_scored_supported(dk, dv))
     return -2;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) |
@@ -616,8 +639,11 @@ extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, con
   p.scale_log2 = 1.f;
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2; p.mod.sink = sink;
   p.status = status;
-  if (dk > 64) return dv > 64 ? launch_prefill_tc<1, 2, 2, true>(tq, tk, tv, p, pdl, st)
-                              : launch_prefill_tc<1, 2, 1, true>(tq, tk, tv, p, pdl, st);
-  return dv > 64 ? launch_prefill_tc<1, 1, 2, true>(tq, tk, tv, p, pdl, st)
-                 : launch_prefill_tc<1, 1, 1, true>(tq, tk, tv, p, pdl, st);
+#define RB_FPS(KP_, VP_)                                                             \
+  return lanes == 2 ? launch_prefill_tc<2, KP_, VP_, true>(tq, tk, tv, p, pdl, st)   \
+                    : launch_prefill_tc<1, KP_, VP_, true>(tq, tk, tv, p, pdl, st)
+  if (dk > 64) { if (dv > 64) RB_FPS(2, 2); RB_FPS(2, 1); }
+  if (dv > 64) RB_FPS(1, 2);
+  RB_FPS(1, 1);
+#undef RB_FPS
 }

@@ -341,7 +341,7 @@ class PosudraModel:
         called with (layer, residual rows [T, width]) after every layer."""
         if self.device.type != "cuda":
             raise _lib.NativeError("Posudra runs on this package's CUDA kernels only")
-        batch = RaggedBatch.plan(entries, cache)
+        batch = RaggedBatch.plan(entries, cache, min(l.mixer.heads for l in self.cfg.layers))
         for e, l in zip(batch.entries, batch.lens):
             cache.reserve(e.seq_id, l)
         batch.upload(self.device)
@@ -368,7 +368,7 @@ class PosudraModel:
             P.attention_any(q, k, v, cache.block_table, batch.positions, batch.token_seq, lw.mods, attn)
             return
         if batch.tiles is not None:
-            P.flash_prefill_scored(q, k, v, cache.block_table, batch.tiles, lw.mods, attn)
+            P.flash_prefill_scored(q, k, v, cache.block_table, batch.tiles, lw.mods, attn, lanes=batch.lanes)
         if batch.single is not None:
             n = len(batch.single_host)
             splits = self.decode_splits(lw, n, batch.single_len)

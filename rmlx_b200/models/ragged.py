@@ -37,10 +37,19 @@ def query_tiles(starts: Sequence[int], lens: Sequence[int], pos0: Sequence[int],
     return tiles
 
 
+def query_lanes(lens: Sequence[int], heads: int, sm_count: int = 148) -> int:
+    """Query tiles of 128 rows a block of the prompt attention takes: 2 (two softmax warps per
+    scheduler, shared key / value tiles) when blocks of 256 rows still fill the machine and few of
+    their second tiles are empty, else 1. The result does not depend on it."""
+    tiles = sum(-(-n // TILE_ROWS) for n in lens if n > 1)
+    pairs = sum(-(-n // (2 * TILE_ROWS)) for n in lens if n > 1)
+    return 2 if pairs * heads >= sm_count and tiles >= 1.5 * pairs else 1
+
+
 class RaggedBatch:
     """``plan`` is host arithmetic; ``upload`` puts the arrays on the cache's device."""
 
-    def __init__(self, entries: Sequence[Entry], pos0: Sequence[int], slots: Sequence[int]):
+    def __init__(self, entries: Sequence[Entry], pos0: Sequence[int], slots: Sequence[int], heads: int = 1):
         if not entries or any(len(e.tokens) < 1 for e in entries):
             raise ValueError("a batch needs at least one entry, and every entry at least one token")
         if len({e.seq_id for e in entries}) != len(entries):
@@ -53,7 +62,8 @@ class RaggedBatch:
             n += l
         self.num_tokens = n
         self.pos0, self.slots = list(pos0), list(slots)
-        self.tiles_host = query_tiles(self.starts, self.lens, self.pos0, self.slots)
+        self.lanes = query_lanes(self.lens, heads)
+        self.tiles_host = query_tiles(self.starts, self.lens, self.pos0, self.slots, TILE_ROWS * self.lanes)
         self.single_host = [s for s, l in zip(self.starts, self.lens) if l == 1]
         self.want_host = [s + w for s, e, l in zip(self.starts, self.entries, self.lens) for w in e.want]
         for e, l in zip(self.entries, self.lens):
@@ -64,10 +74,11 @@ class RaggedBatch:
         self.tokens: Optional[torch.Tensor] = None
 
     @staticmethod
-    def plan(entries: Sequence[Entry], cache) -> "RaggedBatch":
-        """Positions and table rows from the cache's current state."""
+    def plan(entries: Sequence[Entry], cache, heads: int = 1) -> "RaggedBatch":
+        """Positions and table rows from the cache's current state; ``heads``: query heads of the
+        model (of its narrowest layer), which with the lengths decides the tile height."""
         return RaggedBatch(entries, [cache.seq_len(e.seq_id) for e in entries],
-                           [cache.slot_of[e.seq_id] for e in entries])
+                           [cache.slot_of[e.seq_id] for e in entries], heads)
 
     def upload(self, device) -> "RaggedBatch":
         n, tiles = self.num_tokens, self.tiles_host

@@ -29,7 +29,7 @@ _lib.register_cuda_sigs({
     "rmlx_sgemm_scaled_add": ("pipippiiiiip", "i"),
     "rmlx_attention_any": ("pppppppiiiiiiiiffppppiip", "i"),
     "rmlx_flash_prefill_scored_supported": ("ii", "i"),
-    "rmlx_flash_prefill_scored": ("ppppipipiiiiiiiffpppppip", "i"),
+    "rmlx_flash_prefill_scored": ("ppppipipiiiiiiiffppppipip", "i"),
     "rmlx_flash_decode_scored_supported": ("ii", "i"),
     "rmlx_flash_decode_scored_part_o_elems": ("iiiii", "q"),
     "rmlx_flash_decode_scored_part_ml_elems": ("iiii", "q"),
@@ -213,10 +213,10 @@ def decode_scored_supported(dk: int, dv: int) -> bool:
 
 
 def flash_prefill_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
-                         tiles: torch.Tensor, mods: ScoreMods, out: torch.Tensor, window: int = 0,
+                         tiles: torch.Tensor, mods: ScoreMods, out: torch.Tensor, window: int = 0, lanes: int = 1,
                          pdl: bool = False) -> torch.Tensor:
     """Ragged causal attention over pages on the tensor cores: q [T, H, dk] bf16; ``tiles`` int32
-    [n, 4] = (first row, rows <= 128, position of the first row, row of ``block_table``)."""
+    [n, 4] = (first row, rows <= lanes * 128, position of the first row, row of ``block_table``)."""
     _lib.require_cuda_tensor(q, k_cache, v_cache, block_table, tiles, out)
     t, h, dk = q.shape
     assert q.is_contiguous() and out.is_contiguous() and tiles.dtype == torch.int32 and tiles.is_contiguous()
@@ -224,7 +224,8 @@ def flash_prefill_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
     rc = _lib.cuda().rmlx_flash_prefill_scored(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), block_table.stride(0),
         tiles.data_ptr(), tiles.shape[0], out.data_ptr(), t, h, k_cache.shape[1], dk, v_cache.shape[3],
-        k_cache.shape[0], window, *mods.args(), GemmStatus.get(q.device).data_ptr(), int(pdl), _lib.stream_ptr())
+        k_cache.shape[0], window, *mods.args(), lanes, GemmStatus.get(q.device).data_ptr(), int(pdl),
+        _lib.stream_ptr())
     _lib.check(rc, "flash_prefill_scored")
     return out
 
