@@ -1,6 +1,6 @@
 #!/usr/bin/env python
-"""Generate tokens from a model: random weights of a small MoE decoder by default, or an MLX-style
-safetensors directory (``--model-dir``; packed Q4 triplets are used as they are).
+"""Generate tokens from a model: random weights of a small MoE decoder by default, or a safetensors
+directory of any registered family (``--model-dir``; packed Q4 triplets are used as they are).
 
 On a GPU the prompt runs through the tensor-core prefill and every new token is one replay of the
 captured decode graph; on CPU the library-kernel forward runs the same model.
@@ -18,6 +18,7 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 from rmlx_b200.config import FeedForwardType, MoeConfig, TransformerConfig  # noqa: E402
+from rmlx_b200.models.registry import from_pretrained  # noqa: E402
 from rmlx_b200.models.transformer import TransformerModel  # noqa: E402
 from rmlx_b200.models.weights import from_state_dict, random_state_dict  # noqa: E402
 
@@ -39,24 +40,20 @@ def main(argv=None) -> list:
     a = ap.parse_args(argv)
     dev = torch.device(a.device)
     if a.model_dir:
-        from rmlx_b200.loader.safetensors_loader import load_model
-        weights, _ = load_model(a.model_dir, device=dev)
+        model = from_pretrained(a.model_dir, dev)
     else:
         cfg = small_moe()
         quant = None if (a.quant == "none" or dev.type == "cpu") else a.quant
         dtype = torch.bfloat16 if dev.type == "cuda" else torch.float32
         weights = from_state_dict(cfg, random_state_dict(cfg, 0), device=dev, quant=quant, dtype=dtype)
-    model = TransformerModel(weights)
+        model = TransformerModel(weights)
     prompt = torch.tensor([int(t) for t in a.prompt.split(",")], device=dev)
     if dev.type == "cuda":
-        from rmlx_b200.models.decode_engine import CachedDecode
-        from rmlx_b200.models.prefill import enable_native_prefill
-        enable_native_prefill(model)
         cache = model.new_cache((prompt.numel() + a.steps + 15) // 16 + 2, max_seqs=1)
         cache.add_sequence(0)
         logits = model.prefill(prompt, cache, 0)
         first = int(logits[0].argmax())
-        eng = CachedDecode(model, cache, max_batch=1)
+        eng = model.make_decode_engine(cache, 1)
         eng.bind([0], [first])
         toks = [first] + (eng.generate(a.steps - 1)[0].tolist() if a.steps > 1 else [])
     else:

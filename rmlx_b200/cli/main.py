@@ -1,5 +1,8 @@
-"""``python -m rmlx_b200.cli {config,launch}`` — the single-box counterpart of the reference's
-``rmlx`` binary (crates/rmlx-cli/src/main.rs:18-32).
+"""``python -m rmlx_b200.cli {config,launch,plan,generate,trace-run}`` — the single-box counterpart of
+the reference's ``rmlx`` binary (crates/rmlx-cli/src/main.rs:18-32).
+
+``generate`` runs prompts through the serving engine (any model family of ``models.registry``);
+``trace-run`` replays given token ids and writes logits (cli/trace.py).
 
 ``config`` probes the machine (GPUs, peer access, NVLink) and writes a hostfile-like JSON
 (crates/rmlx-cli/src/config.rs:115-345 does this over SSH with Thunderbolt discovery).
@@ -160,6 +163,10 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
     c.add_argument("--ssh", default="localhost", help="ssh target recorded in the hostfile")
     sub.add_parser("plan", add_help=False,
                    help="memory and decode plans of a model on B200s (see `rmlx_b200 plan --help`)")
+    sub.add_parser("generate", add_help=False,
+                   help="generate tokens from a checkpoint folder (see `rmlx_b200 generate --help`)")
+    sub.add_parser("trace-run", add_help=False,
+                   help="replay token ids and write logits (see `rmlx_b200 trace-run --help`)")
     l = sub.add_parser("launch", help="run a command as one rank per GPU")
     l.add_argument("--nproc", "-n", type=int, default=0, help="ranks (default: all GPUs)")
     l.add_argument("--backend", default="auto")
@@ -172,6 +179,12 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
     l.add_argument("--dry-run", action="store_true", help="with --hosts: print the ssh commands only")
     l.add_argument("command", nargs=argparse.REMAINDER)
     args = list(sys.argv[1:] if argv is None else argv)
+    if args and args[0] == "generate":
+        from .generate import main as generate_main
+        return generate_main(args[1:])
+    if args and args[0] == "trace-run":
+        from .trace import main as trace_main
+        return trace_main(args[1:])
     if args and args[0] == "plan":                  # the planner owns its own options
         from .plan import main as plan_main
         return plan_main(args[1:])

@@ -14,6 +14,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import os
 from typing import Dict, Optional, Sequence
 
 from ..config import TransformerConfig, moe_a22b_config
@@ -74,6 +75,15 @@ def kv_bytes_per_token_per_gpu(cfg: TransformerConfig, tp: int, kv_quant: Option
     return int(cfg.num_layers * 2 * hkv * cfg.head_dim * per_value)
 
 
+def decode_hbm_gbs() -> float:
+    path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))),
+                        "MEASURED_PEAKS.json")
+    if not os.path.exists(path):
+        return 6650.0
+    with open(path) as f:
+        return json.load(f)["hbm_gbs"]
+
+
 def decode_roofline(cfg: TransformerConfig, weights: str, tp: int, ctx: int, batch: int = 1,
                     hbm_gbs: Optional[float] = None) -> Dict[str, float]:
     """Bytes one decode step must read per GPU (each active weight once, the cached keys and
@@ -81,10 +91,7 @@ def decode_roofline(cfg: TransformerConfig, weights: str, tp: int, ctx: int, bat
     measured step time is reported against. ``hbm_gbs`` defaults to the pool's measured figure
     (``MEASURED_PEAKS.json`` beside the package) or 6650 GB/s."""
     if hbm_gbs is None:
-        import os
-        path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))),
-                            "MEASURED_PEAKS.json")
-        hbm_gbs = json.load(open(path))["hbm_gbs"] if os.path.exists(path) else 6650.0
+        hbm_gbs = decode_hbm_gbs()
     layout = ParallelLayout(0, tp)
     hq, _, hkv, _ = layout.heads(cfg)
     d, hd, bits = cfg.hidden_size, cfg.head_dim, BITS[weights]
@@ -180,11 +187,51 @@ def plan_deepseek(weights: str = "q4", ranks: int = 8, batch: int = 1, ctx: int 
     }
 
 
+def plan_posudra(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, budget_fraction: float = 0.90,
+                 cfg=None) -> dict:
+    """A Posudra model (bf16, one GPU): per-layer sizes from its configuration, keys and values of their
+    own widths, the activations of a prompt chunk as ``BlockBuffers`` allocates them."""
+    from ..models.posudra import posudra_8b, tensor_shapes
+    from ..ops.parallel_block import pad8
+    c = cfg or posudra_8b()
+    parts = {"attention": 0, "feed_forward": 0, "norms": 0, "embedding": 0, "lm_head": 0}
+    for name, shape in tensor_shapes(c).items():
+        n = 1
+        for s in shape:
+            n *= s
+        part = {"embed": "embedding", "head": "lm_head"}.get(name) or (
+            "norms" if len(shape) == 1 else "feed_forward" if ".mlp." in name else "attention")
+        parts[part] += n * (4 if len(shape) == 1 else 2)               # per-channel vectors are kept in fp32
+    parts["total"] = sum(parts.values())
+    mx = [l.mixer for l in c.layers]
+    kv_layer = [m.kv_heads * (pad8(m.dim) + pad8(m.vdim)) * 2 for m in mx]
+    row = 6 * c.width + 2 * max((m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim for m in mx) + \
+        2 * max(l.ff for l in c.layers) + 2 * max(m.heads * (pad8(m.dim) + pad8(m.vdim)) for m in mx)
+    budget, scratch, need = int(HBM_BYTES * budget_fraction), prefill_chunk * row, batch * ctx * sum(kv_layer)
+    step = parts["attention"] + parts["feed_forward"] + need + parts["lm_head"]
+    hbm = decode_hbm_gbs()
+    layer = (step - parts["lm_head"]) / c.num_layers
+    return {
+        "model": c.name, "weights": "bf16", "tp": 1, "expert_parallel": False, "batch": batch, "ctx": ctx,
+        "kv_quant": "bf16", "weight_bytes_per_gpu": parts, "kv_bytes_per_token_per_gpu": sum(kv_layer),
+        "prefill_chunk": prefill_chunk, "prefill_scratch_bytes": scratch, "budget_bytes_per_gpu": budget,
+        "kv_bytes_needed": need, "kv_tokens_that_fit": max(0, (budget - parts["total"] - scratch) // sum(kv_layer)),
+        "fits": parts["total"] + scratch + need <= budget,
+        "decode_roofline": {"bytes_per_layer": layer, "us_per_layer": layer / (hbm * 1e3), "us_per_step": step / (hbm * 1e3),
+                            "tokens_per_s": batch * hbm * 1e9 / step, "hbm_gbs": hbm},
+        "decode_stream_plans": {},
+    }
+
+
 def plan(model: str = "moe-a22b", weights: str = "q4", tp: int = 1, batch: int = 1, ctx: int = 4096,
          kv_quant: Optional[str] = None, expert_parallel: bool = False, prefill_chunk: int = 2048,
          budget_fraction: float = 0.90, cfg: Optional[TransformerConfig] = None) -> dict:
     if model == "deepseek-v3" and cfg is None:
         return plan_deepseek(weights, tp, batch, ctx, budget_fraction)
+    if model == "posudra-8b" and cfg is None:
+        if weights != "bf16" or tp != 1 or kv_quant is not None:
+            raise ValueError("Posudra runs on one GPU with bf16 weights and cache")
+        return plan_posudra(batch, ctx, prefill_chunk, budget_fraction)
     cfg = cfg or presets()[model]
     w = weight_bytes_per_gpu(cfg, weights, tp, expert_parallel)
     kv_tok = kv_bytes_per_token_per_gpu(cfg, tp, kv_quant)
@@ -246,7 +293,7 @@ def render(p: dict) -> str:
 
 def main(argv: Optional[Sequence[str]] = None) -> int:
     ap = argparse.ArgumentParser(prog="rmlx plan", description=__doc__.split("\n\n")[0])
-    ap.add_argument("--model", default="moe-a22b", choices=sorted(presets()) + ["deepseek-v3"])
+    ap.add_argument("--model", default="moe-a22b", choices=sorted(presets()) + ["deepseek-v3", "posudra-8b"])
     ap.add_argument("--weights", default="q4", choices=sorted(BITS))
     ap.add_argument("--tp", type=int, default=1)
     ap.add_argument("--expert-parallel", action="store_true")
@@ -257,7 +304,11 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
     ap.add_argument("--budget", type=float, default=0.90, help="fraction of 180 GB that may be used")
     ap.add_argument("--json", action="store_true")
     a = ap.parse_args(argv)
-    p = plan(a.model, a.weights, a.tp, a.batch, a.ctx, a.kv_quant, a.expert_parallel, a.prefill_chunk, a.budget)
+    try:
+        p = plan(a.model, a.weights, a.tp, a.batch, a.ctx, a.kv_quant, a.expert_parallel, a.prefill_chunk,
+                 a.budget)
+    except ValueError as e:
+        ap.error(str(e))
     print(json.dumps(p) if a.json else render(p))
     return 0 if p["fits"] else 1
 

@@ -43,24 +43,32 @@ def sink_softmax(scores, sink):
     return e / (e.sum(-1, keepdim=True) + torch.exp(sink[:, None, None] - top))
 
 
-def attention(h, w, mixer, eps):
-    """h [T, width]; w maps 'q', 'k', ... to the layer's tensors. Returns [T, width]."""
-    t = h.shape[0]
-    heads, groups = mixer["heads"], mixer["kv_heads"]
-    q = rms_norm(h @ w["q"].T, w["q.norm"], eps)
-    k = rms_norm(h @ w["k"].T, w["k.norm"], eps)
-    v = h @ w["v"].T
-    q, k, v = split_heads(q, heads), split_heads(k, groups), split_heads(v, groups)
-    per = heads // groups
-    k = torch.stack([k[i // per] for i in range(heads)])
-    v = torch.stack([v[i // per] for i in range(heads)])
-    score = (q @ k.transpose(1, 2)) * mixer["scale"]
-    score = score * w["temp"][:, None, None]
-    score = soft_cap(score, mixer["softcap"])
-    score = score - distance_bias(t, w["r1"], w["r2"], h.dtype)
+def scored_attention(q, k, v, scale, temp, cap, r1, r2, sink):
+    """q [heads, T, d], k and v per query head; causal over one sequence. Returns [heads, T, dv]."""
+    t = q.shape[1]
+    score = (q @ k.transpose(1, 2)) * scale
+    score = score * temp[:, None, None]
+    score = soft_cap(score, cap)
+    score = score - distance_bias(t, r1, r2, q.dtype)
     visible = torch.ones(t, t, dtype=torch.bool).tril()
     score = score.masked_fill(~visible, -math.inf)
-    out = sink_softmax(score, w["sink"]) @ v
+    return sink_softmax(score, sink) @ v
+
+
+def repeat_groups(kv, heads):
+    """Query head i uses key / value head i // (heads / groups)."""
+    per = heads // kv.shape[0]
+    return torch.stack([kv[i // per] for i in range(heads)])
+
+
+def attention(h, w, mixer, eps):
+    """h [T, width]; w maps 'q', 'k', ... to the layer's tensors. Returns [T, width]."""
+    t, heads, groups = h.shape[0], mixer["heads"], mixer["kv_heads"]
+    q = split_heads(rms_norm(h @ w["q"].T, w["q.norm"], eps), heads)
+    k = split_heads(rms_norm(h @ w["k"].T, w["k.norm"], eps), groups)
+    v = split_heads(h @ w["v"].T, groups)
+    out = scored_attention(q, repeat_groups(k, heads), repeat_groups(v, heads), mixer["scale"], w["temp"],
+                           mixer["softcap"], w["r1"], w["r2"], w["sink"])
     return out.permute(1, 0, 2).reshape(t, -1) @ w["o"].T
 
 
