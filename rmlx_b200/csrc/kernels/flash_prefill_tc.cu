@@ -113,6 +113,23 @@ __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
   return d;
 }
 
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+// Largest of three values / of three magnitudes, one instruction each.
+__device__ __forceinline__ float max3(float a, float b, float c) {
+  float d;
+  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+  return d;
+}
+__device__ __forceinline__ float max3_abs(float a, float b, float c) {
+  float d;
+  asm("max.abs.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
+  return d;
+}
+
 template <int LANES, int KP, int VP, bool MOD>
 __global__ void __launch_bounds__(TcCfg<LANES, KP, VP, MOD>::kThreads, 1)
 flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
@@ -394,7 +411,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
 #pragma unroll
         for (int c = 0; c < NC; ++c)
 #pragma unroll
-          for (int i = 0; i < 32; ++i) amax[i & 3] = fmaxf(amax[i & 3], fabsf(__uint_as_float(r[c][i])));
+          for (int i = 0; i < 32; i += 2)
+            amax[(i >> 1) & 3] = max3_abs(amax[(i >> 1) & 3], __uint_as_float(r[c][i]), __uint_as_float(r[c][i + 1]));
         const float top = fmaxf(fmaxf(amax[0], amax[1]), fmaxf(amax[2], amax[3]));
         const float* bias = ring + (d_low & 127) + lane + (kTcKeys - 1);   // bias[-i]: key k0 + i
         if (!__any_sync(0xffffffffu, top * fabsf(hs.inner) > kTanhPolyMax)) {
@@ -449,7 +467,14 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
 #pragma unroll
       for (int c = 0; c < NC; ++c)
 #pragma unroll
-        for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(r[c][i]));
+        for (int i = 0; i < 32; i += 2) {
+          if (MOD) {
+            mx4[(i >> 1) & 3] = max3(mx4[(i >> 1) & 3], __uint_as_float(r[c][i]), __uint_as_float(r[c][i + 1]));
+          } else {
+            mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(r[c][i]));
+            mx4[(i & 3) + 1] = fmaxf(mx4[(i & 3) + 1], __uint_as_float(r[c][i + 1]));
+          }
+        }
       const float m_new = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * sc;
       bool waited = false;
       if (__any_sync(0xffffffffu, m_new > m_used + kTcRescaleStep)) {
@@ -478,6 +503,23 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       const float sub = (m_used == -INFINITY) ? 0.f : m_used;
       uint32_t w[kTcKeys / 2];
       float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+      if (MOD) {
+        const uint64_t sub2 = pair2(-sub, -sub);
+        uint64_t acc[2] = {0, 0};
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) {
+            uint32_t x0, x1;
+            unpair2(add2(pair2(__uint_as_float(r[c][i]), __uint_as_float(r[c][i + 1])), sub2), x0, x1);
+            const float e0 = tc_ex2(__uint_as_float(x0)), e1 = tc_ex2(__uint_as_float(x1));
+            acc[(i >> 1) & 1] = add2(acc[(i >> 1) & 1], pair2(e0, e1));
+            w[c * 16 + (i >> 1)] = pack_bf16(e0, e1);
+          }
+        uint32_t lo, hi;
+        unpair2(add2(acc[0], acc[1]), lo, hi);
+        sum4[0] = __uint_as_float(lo) + __uint_as_float(hi);
+      } else
 #pragma unroll
       for (int c = 0; c < NC; ++c)
 #pragma unroll

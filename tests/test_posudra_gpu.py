@@ -557,6 +557,18 @@ def test_sampling_through_the_engine(bench):
             hist.append(t)
 
 
+def test_cached_prefix_is_reused(bench):
+    eng = ServingEngine(bench.model, 60, SchedulerConfig(max_batch_size=2, max_prefill_chunk=32), use_prefix_cache=True)
+    head = bench.tokens(48, 30)
+    prompts = [head + bench.tokens(9, 31), head + bench.tokens(14, 32)]
+    for p, ran in zip(prompts, (57, 14)):
+        before = eng.prefill_tokens
+        sid = eng.submit(p, 4)
+        _check_greedy(bench, p, eng.run_until_done()[sid])
+        eng.step()
+        assert eng.prefill_tokens - before == ran
+
+
 def test_warm_up_and_other_entry_points(bench):
     eng = bench.engine(batch=2)
     eng.warm_up(prompt_len=5, new_tokens=2)
