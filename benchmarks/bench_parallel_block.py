@@ -10,7 +10,8 @@ feed-forward of inner width I has three matrices, the xIELU one two, so ff = 3 I
 effect (both LM heads are 32768 rows). Prefill: one prompt of ``--tokens``; decode: B sequences of
 ``--ctx`` cached tokens, one captured step per token. Timing: CUDA events after warm-up, the layers'
 weights together exceed L2, so nothing is reused between steps. Kernel times: graph-captured
-loops over all layers (each with its own weights and pages). "roofline" is the larger of bytes / copy
+loops over all layers (each with its own weights and pages), after a pause in which the clocks recover
+from the power cap. "roofline" is the larger of bytes / copy
 bandwidth and FLOPs / burst GEMM rate of MEASURED_PEAKS.json."""
 from __future__ import annotations
 
@@ -18,6 +19,7 @@ import argparse
 import json
 import os
 import sys
+import time
 
 import torch
 
@@ -77,6 +79,7 @@ def graph_us(fn, launches: int, iters: int = 10) -> float:
     """Microseconds per launch of ``fn`` (a loop of ``launches`` launches), captured and replayed."""
     fn()
     torch.cuda.synchronize()
+    time.sleep(0.3)          # the GEMM loops before may have pushed the part into its power cap
     g = torch.cuda.CUDAGraph()
     with torch.cuda.graph(g):
         fn()

@@ -277,3 +277,20 @@ def test_engine_explicit_steps_on_the_transformer_family():
     got = [eng.run_entries([Entry(a, toks[:9], range(9)), Entry(b, [1, 2], ())])]
     got += [eng.run_entries([Entry(b, [3], ()), Entry(a, toks[9:], range(11))])]
     assert torch.allclose(torch.cat(got), want, atol=1e-4)
+
+
+def test_kernel_sets_name_existing_sources_and_give_way_to_the_full_library(monkeypatch, tmp_path):
+    from rmlx_b200 import _build, _lib
+    for name, kinds in _build.SETS.items():
+        for sources in kinds.values():
+            assert all((_build.CSRC / s).exists() for s in sources), name
+    built = []
+    monkeypatch.setattr(_build, "LIB", tmp_path)
+    monkeypatch.setattr(_build, "CUDA_LIB", tmp_path / "full.so")
+    monkeypatch.setattr(_build, "build", lambda kinds, only="all": built.append((kinds, only)) or
+                        {k: _build.set_lib(k, only) for k in kinds})
+    monkeypatch.setattr(_lib, "_kernel_set", "all")
+    _lib.prefer_kernels("parallel_block")
+    assert _lib._library("cuda").name == "librmlx_b200_cuda_parallel_block.so"
+    (tmp_path / "full.so").touch()
+    assert _lib._library("cuda").name == "full.so" and built == [(("cuda",), "parallel_block")]

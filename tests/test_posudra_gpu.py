@@ -338,7 +338,7 @@ def test_decode_projections(dev, b, ff):
 
 
 @pytest.mark.parametrize("dtype,tol", [(F32, 1e-6), (BF, 4e-3)])
-@pytest.mark.parametrize("hq,hkv,dk,dv", [(3, 1, 20, 10), (4, 2, 64, 48)])
+@pytest.mark.parametrize("hq,hkv,dk,dv", [(3, 1, 20, 10), (6, 3, 72, 40)])
 def test_norms_append_and_embedding(dev, dtype, tol, hq, hkv, dk, dv):
     g = torch.Generator().manual_seed(1)
     r = lambda *s: torch.randn(*s, generator=g)                           # noqa: E731
