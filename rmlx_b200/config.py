@@ -221,6 +221,205 @@ class PosudraConfig:
 
 
 @dataclass
+class WindowAttentionSpec:
+    """Grouped-query attention without positions, per-head query / key norm, a sigmoid gate per head on
+    the output and a sliding window (0: none)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int = 0
+
+    kind = "attention"
+
+    def validate(self) -> "WindowAttentionSpec":
+        _require(self.heads > 0 and self.kv_heads > 0, "head counts must be positive")
+        _require(self.heads % self.kv_heads == 0, "heads must be a multiple of kv_heads")
+        _require(self.dim > 0 and self.vdim > 0, "head sizes must be positive")
+        _require(self.window >= 0, "window must be >= 0 (0: none)")
+        return self
+
+    @staticmethod
+    def from_json(m: dict) -> "WindowAttentionSpec":
+        return WindowAttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                                   int((m.get("mask") or {}).get("size") or 0))
+
+    def to_json(self) -> dict:
+        return {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale,
+                "mask": {"size": self.window} if self.window else None}
+
+
+@dataclass
+class LatentAttentionSpec:
+    """Attention over one latent of ``kv_rank`` values and one rotated key part of ``rot_dim`` values per
+    token; heads have ``dim`` unrotated and ``rot_dim`` rotated query / key values, of which the first
+    ``rot_dims`` turn, and ``vdim`` value channels."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot_base: float = 10000.0
+    rot_dims: Optional[int] = None       # default: all of rot_dim
+
+    kind = "latent_attention"
+
+    def __post_init__(self):
+        if self.rot_dims is None:
+            self.rot_dims = self.rot_dim
+
+    def validate(self) -> "LatentAttentionSpec":
+        _require(self.heads > 0 and self.dim > 0 and self.vdim > 0 and self.kv_rank > 0, "sizes must be positive")
+        _require(self.rot_dim >= 0 and self.rot_dims % 2 == 0 and self.rot_dims <= self.rot_dim,
+                 "rotated dimensions come in pairs, at most rot_dim of them")
+        _require(self.kv_rank <= 1024, "kv_rank must be <= 1024")
+        _require(self.rot_base > 0, "rot_base must be positive")
+        return self
+
+    @staticmethod
+    def from_json(m: dict) -> "LatentAttentionSpec":
+        rot = m.get("rot") or {}
+        rot_dim = int(m["rot_dim"])
+        return LatentAttentionSpec(int(m["heads"]), int(m["dim"]), rot_dim, int(m["vdim"]), int(m["kv_rank"]),
+                                   float(m["scale"]), float(rot.get("base", 10000.0)), int(rot.get("dims", rot_dim)))
+
+    def to_json(self) -> dict:
+        return {"heads": self.heads, "dim": self.dim, "rot_dim": self.rot_dim, "vdim": self.vdim, "kv_rank": self.kv_rank,
+                "scale": self.scale, "rot": {"base": self.rot_base, "dims": self.rot_dims}}
+
+
+@dataclass
+class WkvSpec:
+    """RWKV-style time mixing: ``heads`` states of dim x dim, decays from a low-rank projection (its
+    rank comes with the weights; ``decay_rank`` is what random weights use)."""
+    heads: int
+    dim: int
+    decay_rank: int = 16
+
+    kind = "wkv"
+
+    def validate(self) -> "WkvSpec":
+        _require(self.heads > 0 and 0 < self.dim <= 256, "wkv: heads must be positive, dim in [1, 256]")
+        return self
+
+    @staticmethod
+    def from_json(m: dict) -> "WkvSpec":
+        return WkvSpec(int(m["heads"]), int(m["dim"]))
+
+    def to_json(self) -> dict:
+        return {"heads": self.heads, "dim": self.dim}
+
+
+@dataclass
+class ClampedFfSpec:
+    """Gated feed-forward whose gate and up values are clamped to ``limit``."""
+    ff: int
+    limit: float
+
+    def validate(self) -> "ClampedFfSpec":
+        _require(self.ff > 0 and self.limit > 0, "feed-forward: ff and limit must be positive")
+        return self
+
+    def to_json(self) -> dict:
+        return {"kind": "dense", "ff": self.ff, "limit": self.limit}
+
+
+@dataclass
+class RoutedFfSpec:
+    """``experts`` clamped feed-forwards of width ``ff`` and ``identity`` experts that return their input;
+    each token uses ``top`` of them, chosen by corrected softmax scores."""
+    experts: int
+    identity: int
+    top: int
+    ff: int
+    limit: float
+
+    def validate(self) -> "RoutedFfSpec":
+        _require(self.experts > 0 and self.identity >= 0 and self.ff > 0 and self.limit > 0, "bad expert sizes")
+        _require(self.experts <= 256 and self.experts + self.identity <= 512, "at most 256 experts and 512 router outputs")
+        _require(1 <= self.top <= min(32, self.experts + self.identity), "top must be in [1, 32] and <= the router outputs")
+        return self
+
+    def to_json(self) -> dict:
+        return {"kind": "moe", "expert": {"ff": self.ff, "limit": self.limit},
+                "router": {"experts": self.experts, "identity": self.identity, "top": self.top}}
+
+
+_MIXERS = {c.kind: c for c in (WindowAttentionSpec, LatentAttentionSpec, WkvSpec)}
+
+
+@dataclass
+class PostNormLayerSpec:
+    """One layer: a mixer and (unless None) a feed-forward, each followed by a norm of its output."""
+    mixer: "WindowAttentionSpec | LatentAttentionSpec | WkvSpec"
+    mlp: "ClampedFfSpec | RoutedFfSpec | None" = None
+
+    def validate(self) -> "PostNormLayerSpec":
+        self.mixer.validate()
+        if self.mlp is not None:
+            self.mlp.validate()
+        return self
+
+    @staticmethod
+    def from_json(e: dict) -> "PostNormLayerSpec":
+        _require(e.get("type") in _MIXERS, f"unknown mixer type {e.get('type')!r}")
+        m, mlp = e.get("mlp"), None
+        if m is not None:
+            _require(m.get("kind") in ("dense", "moe"), f"unknown feed-forward kind {m.get('kind')!r}")
+            if m["kind"] == "dense":
+                mlp = ClampedFfSpec(int(m["ff"]), float(m["limit"]))
+            else:
+                r, x = m["router"], m["expert"]
+                mlp = RoutedFfSpec(int(r["experts"]), int(r.get("identity") or 0), int(r["top"]), int(x["ff"]),
+                                   float(x["limit"]))
+        return PostNormLayerSpec(_MIXERS[e["type"]].from_json(e["mixer"]), mlp)
+
+    def to_json(self) -> dict:
+        return {"type": self.mixer.kind, "mixer": self.mixer.to_json(),
+                "mlp": None if self.mlp is None else self.mlp.to_json()}
+
+
+@dataclass
+class RodapelConfig:
+    """Rodapel: a decoder that mixes windowed attention, latent attention and WKV recurrence, with norms on
+    the sublayers' outputs; every layer states its own kind and sizes."""
+    vocab_size: int
+    width: int
+    layers: "list[PostNormLayerSpec]"
+    norm_eps: float = 1e-6
+    max_seq_len: int = 0             # 0: bounded by the cache only
+    name: str = "rodapel"
+
+    sliding_window = 0               # pages are shared by every layer: none can be dropped early
+
+    def validate(self) -> "RodapelConfig":
+        _require(self.vocab_size > 0 and self.width > 0 and len(self.layers) > 0, "bad sizes")
+        _require(self.norm_eps > 0, "norm_eps must be positive")
+        for layer in self.layers:
+            layer.validate()
+        return self
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def hidden_size(self) -> int:
+        return self.width
+
+    @staticmethod
+    def from_json(c: dict) -> "RodapelConfig":
+        return RodapelConfig(int(c["vocab"]), int(c["width"]), [PostNormLayerSpec.from_json(e) for e in c["layers"]],
+                             float(c["norm"]["eps"])).validate()
+
+    def to_json(self) -> dict:
+        return {"architecture": "Rodapel", "vocab": self.vocab_size, "width": self.width,
+                "norm": {"eps": self.norm_eps}, "layers": [l.to_json() for l in self.layers]}
+
+
+@dataclass
 class AttentionConfig:
     num_heads: int
     num_kv_heads: int

@@ -5,6 +5,7 @@
 //   s = softcap * tanh(s / softcap)             logit soft cap       (softcap <= 0: none)
 //   s = s - r1[h] * ln(1 + r2[h] * (i - j))     logarithmic distance bias (r1 == nullptr: none)
 //   weights = exp(s) / (sum exp(s) + exp(sink[h]))    sink without key or value (nullptr: none)
+//   o = o * sigmoid(gate[t, h])                 output gate, one logit per token and head (nullptr: none)
 //
 // The tensor-core kernels work in base 2 (scores times log2 e), which leaves one ex2 per weight.
 #pragma once
@@ -22,6 +23,17 @@ struct ScoreMod {
   const float* r2 = nullptr;
   const float* sink = nullptr;
 };
+
+// Gate logits of token t, head h at gate[t * ld + h], in the activations' type.
+struct HeadGate {
+  const void* gate = nullptr;
+  int ld = 0;
+};
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+template <class T>
+__device__ __forceinline__ float head_gate(const HeadGate& g, size_t t, int h) {
+  return g.gate ? sigmoid_f(float(static_cast<const T*>(g.gate)[t * g.ld + h])) : 1.f;
+}
 
 // tanh(u) / u as a polynomial in u^2, |u| <= kTanhPolyMax: Chebyshev interpolation of degree 4 in
 // u^2, largest relative error 1.6e-7 (fp32 evaluation included).

@@ -16,14 +16,16 @@ constexpr int kAaWarps = 4;
 
 struct AaParams {
   const void* q;            // [T, Hq, dkp]
-  const void* k_cache;      // [blocks, Hkv, page, dkp]
-  const void* v_cache;      // [blocks, Hkv, page, dvp]
+  const void* k_cache;      // [blocks, Hkv, page, ldk], the first dkp values of a row are the key
+  const void* v_cache;      // [blocks, Hkv, page, ldv], the first dvp the value (latent rows are both)
   const int* block_table;
   const int* positions;     // [T]
   const int* token_seq;     // [T] row of the block table, or null: token t has row t
   void* out;                // [T, Hq, dvp]
-  int Hq, Hkv, dkp, dvp, max_blocks, page, window;
+  int Hq, Hkv, dkp, dvp, ldk, ldv, max_blocks, page, window;
   ScoreMod mod;
+  HeadGate gate;
+  const int* rows;          // [n] batch rows to run, or null: all
 };
 
 __device__ __forceinline__ float aa_dot8(const float* k, const float* q) {
@@ -55,7 +57,7 @@ __global__ void __launch_bounds__(kAaWarps * 32) attention_any_kernel(AaParams p
   __shared__ float s_m[kAaWarps], s_l[kAaWarps];
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, h = blockIdx.y, kvh = h / (p.Hq / p.Hkv);
+  const int t = p.rows ? p.rows[blockIdx.x] : blockIdx.x, h = blockIdx.y, kvh = h / (p.Hq / p.Hkv);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pos = p.positions[t];
   const int seq = p.token_seq ? p.token_seq[t] : t;
@@ -78,7 +80,7 @@ __global__ void __launch_bounds__(kAaWarps * 32) attention_any_kernel(AaParams p
     float s = -INFINITY;
     if (ok) {
       const size_t row = (size_t(bt[key / p.page]) * p.Hkv + kvh) * p.page + key % p.page;
-      const T* k = static_cast<const T*>(p.k_cache) + row * p.dkp;
+      const T* k = static_cast<const T*>(p.k_cache) + row * p.ldk;
       float dot = 0.f;
       for (int d = 0; d < p.dkp; d += 8) dot += aa_dot8(k + d, sq + d);
       s = dot * st;
@@ -98,7 +100,7 @@ __global__ void __launch_bounds__(kAaWarps * 32) attention_any_kernel(AaParams p
       if (wj == 0.f) continue;                        // warp-uniform
       const int kj = c0 + j;
       const size_t row = (size_t(bt[kj / p.page]) * p.Hkv + kvh) * p.page + kj % p.page;
-      const T* v = static_cast<const T*>(p.v_cache) + row * p.dvp;
+      const T* v = static_cast<const T*>(p.v_cache) + row * p.ldv;
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         if (i * 32 + lane < p.dvp) o[i] = fmaf(wj, aa_f32(v[i * 32 + lane]), o[i]);
@@ -119,12 +121,13 @@ __global__ void __launch_bounds__(kAaWarps * 32) attention_any_kernel(AaParams p
     f[w] = s_m[w] == -INFINITY ? 0.f : expf(s_m[w] - M);
     L += s_l[w] * f[w];
   }
+  const float scale = L > 0.f ? head_gate<T>(p.gate, t, h) / L : 0.f;
   T* out = static_cast<T*>(p.out) + (size_t(t) * p.Hq + h) * p.dvp;
   for (int i = threadIdx.x; i < p.dvp; i += kAaWarps * 32) {
     float acc = 0.f;
 #pragma unroll
     for (int w = 0; w < kAaWarps; ++w) acc += so[w * p.dvp + i] * f[w];
-    aa_put(out + i, L > 0.f ? acc / L : 0.f);
+    aa_put(out + i, acc * scale);
   }
 }
 
@@ -149,24 +152,27 @@ static int dispatch_any(const AaParams& p, int rows, int pdl, cudaStream_t st) {
 using namespace rb;
 RB_BOUNDS_REGISTER("attention_any.cu")
 
-// q [T, Hq, dkp], out [T, Hq, dvp], caches [blocks, Hkv, page, dkp / dvp]: fp32 (f32) or bf16; dkp and
-// dvp multiples of eight, dvp <= 1024. Token t sits at positions[t] and sees keys 0 .. positions[t]
-// (the last `window` of them when window > 0) of row token_seq[t] of the block table.
+// q [T, Hq, dkp], out [T, Hq, dvp], caches [blocks, Hkv, page, ldk / ldv]: fp32 (f32) or bf16; dkp, dvp, ldk
+// and ldv multiples of eight, dvp <= 1024. Token t sits at positions[t] and sees keys 0 .. positions[t]
+// (the last `window` of them when window > 0) of row token_seq[t] of the block table. rows: the n_rows
+// batch rows to run (null: all T). gate [T, ldg] in the same type, or null.
 extern "C" int rmlx_attention_any(const void* q, const void* k_cache, const void* v_cache,
                                   const int* block_table, const int* positions, const int* token_seq,
-                                  void* out, int T, int Hq, int Hkv, int dkp, int dvp, int max_blocks,
-                                  int page, int window, float scale, float softcap, const float* temp,
-                                  const float* r1, const float* r2, const float* sink, int f32, int pdl,
-                                  cudaStream_t st) {
+                                  const int* rows, int n_rows, void* out, int T, int Hq, int Hkv, int dkp, int dvp,
+                                  int ldk, int ldv, int max_blocks, int page, int window, float scale, float softcap,
+                                  const float* temp, const float* r1, const float* r2, const float* sink,
+                                  const void* gate, int ldg, int f32, int pdl, cudaStream_t st) {
   if (T < 1 || Hkv < 1 || Hq % Hkv || Hq > 65535 || dkp < 8 || dkp % 8 || dvp < 8 || dvp % 8 ||
-      dkp > 8192 || (r1 && !r2))
+      dkp > 8192 || ldk < dkp || ldk % 8 || ldv < dvp || ldv % 8 || (r1 && !r2) || (rows && n_rows < 1))
     return -2;
   AaParams p;
   p.q = q; p.k_cache = k_cache; p.v_cache = v_cache; p.block_table = block_table;
-  p.positions = positions; p.token_seq = token_seq; p.out = out;
-  p.Hq = Hq; p.Hkv = Hkv; p.dkp = dkp; p.dvp = dvp; p.max_blocks = max_blocks; p.page = page;
+  p.positions = positions; p.token_seq = token_seq; p.out = out; p.rows = rows;
+  p.Hq = Hq; p.Hkv = Hkv; p.dkp = dkp; p.dvp = dvp; p.ldk = ldk; p.ldv = ldv; p.max_blocks = max_blocks; p.page = page;
   p.window = window;
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2;
   p.mod.sink = sink;
-  return f32 ? dispatch_any<float>(p, T, pdl, st) : dispatch_any<__nv_bfloat16>(p, T, pdl, st);
+  p.gate.gate = gate; p.gate.ld = ldg;
+  const int n = rows ? n_rows : T;
+  return f32 ? dispatch_any<float>(p, n, pdl, st) : dispatch_any<__nv_bfloat16>(p, n, pdl, st);
 }

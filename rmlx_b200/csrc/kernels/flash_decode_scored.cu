@@ -62,8 +62,11 @@ struct FsParams {
   float* part_ml;                // [B, Hkv*gtiles, S, 16, 2]
   unsigned int* tickets;         // [B * Hkv*gtiles], zero on entry, zero on exit
   int raw_ld, max_blocks, Hq, Hkv, G, gtiles, S, window, dim, vdim, dkp, dvp;
+  int head_norm;                 // fused form: q_w / k_w are [dim] and every head is normed on its own
+  int gate_col;                  // fused form: gate logits at raw[b][gate_col + head] (< 0: none)
   float eps;
   ScoreMod mod;
+  HeadGate gate;                 // plain form
 };
 
 __device__ __forceinline__ float fs_block_sum(float v, float* red) {
@@ -102,7 +105,7 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   extern __shared__ __align__(128) char smem[];
   char* wsm = smem + (threadIdx.x >> 5) * (NST * STAGE);   // reused for the merges afterwards
   __shared__ float s_m[kFsWarps][16], s_l[kFsWarps][16];
-  __shared__ float s_sink[16];
+  __shared__ float s_sink[16], s_gate[16];
   __shared__ float red[kFsWarps];
   __shared__ __align__(16) __nv_bfloat16 sQ[16][DK + 8];
   __shared__ unsigned int s_last;
@@ -152,6 +155,53 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   if (p.raw) {
     const float* row = p.raw + size_t(b) * p.raw_ld;
     const int nq = p.Hq * p.dim, nk = p.Hkv * p.dim;
+    if (p.head_norm) {
+      // one warp per query head in turn; the owner's last warp also takes the new key's root mean square
+      constexpr int PL = DK / 32;
+      const int q_rows = min(16, p.G - gt * 16);
+      float v[4][PL];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int r = warp * 4 + u;
+        const float* src = row + (kvh * p.G + gt * 16 + r) * p.dim;
+#pragma unroll
+        for (int i = 0; i < PL; ++i) v[u][i] = (r < q_rows && i * 32 + lane < p.dim) ? __ldcg(src + i * 32 + lane) : 0.f;
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int r = warp * 4 + u;
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < PL; ++i) ss += v[u][i] * v[u][i];
+        const float iq = 1.f / sqrtf(warp_sum(ss) / float(p.dim) + p.eps);
+#pragma unroll
+        for (int i = 0; i < PL; ++i) {
+          const int d = i * 32 + lane;
+          sQ[r][d] = __float2bfloat16_rn(d < p.dim ? v[u][i] * iq * p.q_w[d] : 0.f);
+        }
+      }
+      if (owner && RB_BOUNDS((len - 1) / kFsPage, p.max_blocks)) {
+        const size_t slot = (size_t(bt[(len - 1) / kFsPage]) * p.Hkv + kvh) * kFsPage + (len - 1) % kFsPage;
+        __nv_bfloat16* kd = p.k_cache + slot * p.dkp;
+        __nv_bfloat16* vd = p.v_cache + slot * p.dvp;
+        if (warp == kFsWarps - 1) {
+          float f[PL], ss = 0.f;
+#pragma unroll
+          for (int i = 0; i < PL; ++i) {
+            f[i] = i * 32 + lane < p.dim ? __ldcg(row + nq + kvh * p.dim + i * 32 + lane) : 0.f;
+            ss += f[i] * f[i];
+          }
+          const float ik = 1.f / sqrtf(warp_sum(ss) / float(p.dim) + p.eps);
+#pragma unroll
+          for (int i = 0; i < PL; ++i) {
+            const int d = i * 32 + lane;
+            if (d < p.dim) kd[d] = __float2bfloat16_rn(f[i] * ik * p.k_w[d]);
+          }
+        }
+        for (int d = threadIdx.x; d < p.vdim; d += kFsThreads)
+          vd[d] = __float2bfloat16_rn(__ldcg(row + nq + nk + kvh * p.vdim + d));
+      }
+    } else {
     // this thread's share of the tile's queries, un-normalised but weighted (independent loads)
     constexpr int QPT = 16 * DK / kFsThreads;
     float qv[QPT];
@@ -203,6 +253,7 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
       for (int d = threadIdx.x; d < p.vdim; d += kFsThreads)
         vd[d] = __float2bfloat16_rn(__ldcg(row + nq + nk + kvh * p.vdim + d));
     }
+    }
   } else {
     for (int i = threadIdx.x; i < 16 * (DK / 8); i += kFsThreads) {
       const int r = i / (DK / 8), c = i % (DK / 8), h = gt * 16 + r;
@@ -218,6 +269,12 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   if (threadIdx.x < 16) {
     const int h = gt * 16 + threadIdx.x;
     s_sink[threadIdx.x] = (h < p.G && p.mod.sink) ? p.mod.sink[kvh * p.G + h] * kLog2e : -INFINITY;
+    float gate = 1.f;
+    if (h < p.G) {
+      if (!p.raw) gate = head_gate<__nv_bfloat16>(p.gate, b, kvh * p.G + h);
+      else if (p.gate_col >= 0) gate = sigmoid_f(__ldcg(p.raw + size_t(b) * p.raw_ld + p.gate_col + kvh * p.G + h));
+    }
+    s_gate[threadIdx.x] = gate;
   }
   const bool upper = p.G - gt * 16 > 8;      // rows 8 .. 15 of the tile hold heads
   __syncthreads();      // queries staged, the appended key / value written
@@ -342,7 +399,7 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
     if (p.S == 1) {
       if (s_sink[row] != -INFINITY) L += ex2_approx(s_sink[row] - M);
       if (h < p.G && d < p.dvp)
-        p.out[(size_t(b) * p.Hq + size_t(kvh) * p.G + h) * p.dvp + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+        p.out[(size_t(b) * p.Hq + size_t(kvh) * p.G + h) * p.dvp + d] = __float2bfloat16_rn(L > 0.f ? acc * s_gate[row] / L : 0.f);
     } else {
       p.part_o[((tile * p.S + split) * 16 + row) * DV + d] = acc;
       if (d == 0) {
@@ -375,7 +432,7 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
       wgt[s * 16 + row] = f;
       L += mls[s * 32 + row * 2 + 1] * f;
     }
-    const float inv = L > 0.f ? 1.f / L : 0.f;
+    const float inv = L > 0.f ? s_gate[row] / L : 0.f;
     for (int s = 0; s < p.S; ++s) wgt[s * 16 + row] *= inv;
   }
   __syncthreads();
@@ -426,7 +483,8 @@ extern "C" long long rmlx_flash_decode_scored_part_ml_elems(int B, int Hq, int H
 extern "C" long long rmlx_flash_decode_scored_ticket_elems(int B, int Hq, int Hkv) { return fs_tiles(B, Hq, Hkv); }
 
 // q (bf16) or raw (fp32, with q_w, k_w, eps: the fused form), exactly one of them. dkp / dvp: dim /
-// vdim rounded up to eight. `tickets` is zero on the first call; the kernel leaves it zero.
+// vdim rounded up to eight. gate: bf16 [rows, ldg] output gate logits of the plain form, or null; head_norm,
+// gate_col (-1: none): the fused form's. `tickets` is zero on the first call; the kernel leaves it zero.
 extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw_ld, const float* q_w,
                                         const float* k_w, float eps, void* k_cache, void* v_cache,
                                         const int* block_table, const int* positions, const int* rows,
@@ -434,7 +492,8 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
                                         unsigned int* tickets, int B, int Hq, int Hkv, int dim, int vdim,
                                         int dkp, int dvp, int max_blocks, int splits, int window,
                                         float scale, float softcap, const float* temp, const float* r1,
-                                        const float* r2, const float* sink, int pdl, cudaStream_t st) {
+                                        const float* r2, const float* sink, const void* gate, int ldg,
+                                        int head_norm, int gate_col, int pdl, cudaStream_t st) {
   if (B < 1 || B > 65535 || Hkv < 1 || Hq % Hkv || splits < 1 || splits > kFsMaxSplits || (!q) == (!raw) ||
       dkp % 8 || dvp % 8 || dim > dkp || vdim > dvp || dim < 1 || vdim < 1 || (r1 && !r2))
     return -2;
@@ -449,6 +508,8 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
   p.max_blocks = max_blocks; p.Hq = Hq; p.Hkv = Hkv; p.G = Hq / Hkv; p.gtiles = (p.G + 15) / 16;
   p.S = splits; p.window = window; p.dim = dim; p.vdim = vdim; p.dkp = dkp; p.dvp = dvp;
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2; p.mod.sink = sink;
+  p.gate.gate = gate; p.gate.ld = ldg; p.head_norm = head_norm; p.gate_col = gate_col;
+  if (raw && gate_col >= 0 && raw_ld < gate_col + Hq) return -2;
   if (p.Hkv * p.gtiles > 65535) return -2;
   const dim3 grid(splits, Hkv * p.gtiles, B);
   const bool deep = size_t(splits) * Hkv * p.gtiles * B <= size_t(2 * sm_count());

@@ -88,6 +88,7 @@ struct TcParams {
   int window;               // > 0: a query sees only its last `window` keys
   float scale_log2;
   ScoreMod mod;             // MOD instances
+  HeadGate gate;            // MOD instances
   int* status;
 };
 
@@ -550,7 +551,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     }
     if (ok && my_steps > 0) {
       tc_fence_after_sync();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (MOD) inv *= head_gate<__nv_bfloat16>(p.gate, size_t(q0 + min(lrow, rows - 1)), h);
       __nv_bfloat16* dst = p.out + (size_t(q0 + min(lrow, rows - 1)) * p.Hq + h) * p.dv;
 #pragma unroll 1
       for (int c = 0; c < VP * 2; ++c) {
@@ -655,12 +657,13 @@ extern "C" int rmlx_flash_prefill_scored_supported(int dk, int dv) {
 // Ragged batch with score modifiers. q [T, Hq, dk] and out [T, Hq, dv] bf16, caches [num_blocks, Hkv, 16,
 // dk / dv] bf16 already holding the rows' own keys and values; tiles: n_tiles x {first row, rows (1 .. lanes * 128),
 // position of the first row, row of block_table [.., max_blocks]} (int32, device), heaviest first.
+// gate: bf16 [T, ldg] output gate logits, or null.
 extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, const void* v_cache,
                                          const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                                          void* out, int T, int Hq, int Hkv, int dk, int dv, int num_blocks,
                                          int window, float scale, float softcap, const float* temp,
-                                         const float* r1, const float* r2, const float* sink, int lanes,
-                                         int* status, int pdl, cudaStream_t st) {
+                                         const float* r1, const float* r2, const float* sink, const void* gate,
+                                         int ldg, int lanes, int* status, int pdl, cudaStream_t st) {
   if (T < 1 || (lanes != 1 && lanes != 2) || Hkv < 1 || Hq % Hkv || num_blocks < 1 || n_tiles < 1 || !tiles || (r1 && !r2) ||
       !rmlx_flash_prefill_scored_supported(dk, dv))
     return -2;
@@ -680,6 +683,7 @@ extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, con
   p.window = window > 0 ? window : 0;
   p.scale_log2 = 1.f;
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2; p.mod.sink = sink;
+  p.gate.gate = gate; p.gate.ld = ldg;
   p.status = status;
 #define RB_FPS(KP_, VP_)                                                             \
   return lanes == 2 ? launch_prefill_tc<2, KP_, VP_, true>(tq, tk, tv, p, pdl, st)   \

@@ -4,7 +4,7 @@
 //
 // Epilogues: plain store; split (columns before n_raw stored as they are, the others through xIELU
 // into a second matrix); scaled accumulate (X[m, n] += s[n] * C[m, n], a layer scale and the
-// residual sum).
+// residual sum). Grouped form: rows sorted by expert, blockIdx.z picks the expert's matrix and rows.
 #include "../common/ptx.cuh"
 #include "../common/launch.cuh"
 #include "../common/xielu.cuh"
@@ -20,6 +20,7 @@ struct SgemmOut {
   int n_raw;
   float ap, an;
   const float* scale;         // accumulate
+  const int* offsets;         // grouped: rows offsets[z] .. offsets[z + 1] take matrix z of the stack
 };
 
 template <int EPI>
@@ -29,7 +30,15 @@ sgemm_kernel(const float* __restrict__ A, int lda, const float* __restrict__ W, 
   __shared__ float sA[kSgK][kSgTile + 4], sW[kSgK][kSgTile + 4];
   pdl_launch_dependents();
   pdl_wait();
+  if (o.offsets) {
+    const int at = o.offsets[blockIdx.z];
+    M = o.offsets[blockIdx.z + 1] - at;
+    A += size_t(at) * lda;
+    W += size_t(blockIdx.z) * N * ldw;
+    o.c += size_t(at) * o.ldc;
+  }
   const int m0 = blockIdx.y * kSgTile, n0 = blockIdx.x * kSgTile;
+  if (m0 >= M) return;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   // loader: thread i brings four consecutive k of row i / 4
   const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;
@@ -87,8 +96,8 @@ sgemm_kernel(const float* __restrict__ A, int lda, const float* __restrict__ W, 
 
 template <int EPI>
 static int launch_sgemm(const float* A, int lda, const float* W, int ldw, int M, int N, int K, SgemmOut o,
-                        int pdl, cudaStream_t st) {
-  const dim3 grid((N + kSgTile - 1) / kSgTile, (M + kSgTile - 1) / kSgTile);
+                        int pdl, cudaStream_t st, int groups = 1) {
+  const dim3 grid((N + kSgTile - 1) / kSgTile, (M + kSgTile - 1) / kSgTile, groups);
   if (grid.y > 65535u) return -2;
   return launch(sgemm_kernel<EPI>, grid, dim3(256), 0, st, pdl != 0, A, lda, W, ldw, M, N, K, o);
 }
@@ -120,4 +129,13 @@ extern "C" int rmlx_sgemm_scaled_add(const float* A, int lda, const float* W, in
   if (M < 1 || N < 1 || K < 1 || !scale) return -2;
   SgemmOut o{}; o.c = x; o.ldc = ldx; o.scale = scale;
   return launch_sgemm<kSgAccumulate>(A, lda, W, ldw, M, N, K, o, pdl, st);
+}
+
+// Grouped: A's rows are sorted by expert, W is the stack [E, N, ldw], offsets int32 [E + 1] on the device;
+// M bounds the rows of one expert.
+extern "C" int rmlx_sgemm_grouped(const float* A, int lda, const float* W, int ldw, const int* offsets, int E,
+                                  float* c, int ldc, int M, int N, int K, int pdl, cudaStream_t st) {
+  if (M < 1 || N < 1 || K < 1 || E < 1 || E > 65535 || !offsets) return -2;
+  SgemmOut o{}; o.c = c; o.ldc = ldc; o.offsets = offsets;
+  return launch_sgemm<kSgPlain>(A, lda, W, ldw, M, N, K, o, pdl, st, E);
 }

@@ -231,9 +231,17 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
         if (OUT_F32) {
           if (row < M && col0 < N) {
             float* dstf = static_cast<float*>(Cv) + size_t(row) * ldc + col0;
+            if (col0 + 32 <= N && (ldc & 3) == 0 && (reinterpret_cast<uintptr_t>(Cv) & 15) == 0) {
 #pragma unroll
-            for (int j = 0; j < 32; ++j)
-              if (col0 + j < N) dstf[j] = __uint_as_float(r[j]);
+              for (int v = 0; v < 8; ++v)
+                *reinterpret_cast<float4*>(dstf + v * 4) =
+                    make_float4(__uint_as_float(r[v * 4]), __uint_as_float(r[v * 4 + 1]),
+                                __uint_as_float(r[v * 4 + 2]), __uint_as_float(r[v * 4 + 3]));
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j)
+                if (col0 + j < N) dstf[j] = __uint_as_float(r[j]);
+            }
           }
         } else if (row < M && col0 < N) {
           __nv_bfloat16* dst = C + size_t(row) * ldc + col0;

@@ -1,0 +1,338 @@
+// RWKV-style time mixing: token shift, the WKV recurrence with its fp32 state, and the per-head norm
+// with the output gate.
+//
+// Per head, with S [dim, dim] (rows: key channels, columns: value channels) carried per sequence:
+//     o_t = (S + diag(u) k_t v_t^T)^T r_t,   S <- diag(w_t) S + k_t v_t^T,
+//     w_t = exp(-exp(dl_t + w0))
+// Columns are independent of each other. A block owns one (sequence, head, group of columns) and walks
+// the sequence's new tokens; a thread holds 16 rows of one column in registers, LANES threads share a
+// column. Half of the block's warps fetch the next chunk of tokens (and take the exponentials and
+// r . (u k)) while the other half runs the current one; r, k and w are read from shared memory in
+// 16-row groups that start in different banks. Arithmetic on the state runs on pairs (fma.rn.f32x2).
+//
+// The state of a sequence lives in its slot's row of a flat fp32 pool, beside the last token's
+// residual row, which the token shift of the sequence's next token needs.
+#include "../common/launch.cuh"
+#include "../common/rows.cuh"
+
+namespace rb {
+
+constexpr int kShiftParts = 5;            // r, k, v, g, w
+
+// out[s][t] = x[t] + (prev[t] - x[t]) * mu[s]; prev: the row before in the batch, or for a sequence's
+// first row of the batch the row kept in its slot. slots [T]; each_row: no two rows share a sequence.
+template <class T>
+__global__ void __launch_bounds__(kRowThreads)
+token_shift_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ mu, const float* __restrict__ prev,
+                   long long prev_stride, const int* __restrict__ slots, int each_row, T* __restrict__ out, int rows) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const bool first = each_row || t == 0 || slots[t - 1] != slots[t];
+  const float* before = first ? prev + size_t(slots[t]) * prev_stride : x + size_t(t - 1) * ldx;
+  const float* row = x + size_t(t) * ldx;
+  for (int c = threadIdx.x; c < ldx >> 3; c += kRowThreads) {
+    float a[8], b[8];
+    load8(row + c * 8, a);
+    load8(before + c * 8, b);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) b[i] -= a[i];
+#pragma unroll
+    for (int s = 0; s < kShiftParts; ++s) {
+      float m[8];
+      load8(mu + s * ldx + c * 8, m);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) m[i] = fmaf(b[i], m[i], a[i]);
+      store8(out + (size_t(s) * rows + t) * ldx + c * 8, m);
+    }
+  }
+}
+
+__device__ __forceinline__ uint64_t wk_pair(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ void wk_unpair(uint64_t v, float& lo, float& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ uint64_t wk_fma(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t wk_mul(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
+struct WkvParams {
+  const void* r;            // [rows, ld] each, head h at column h * dim
+  const void* k;
+  const void* v;
+  int ld;
+  const float* dl;          // [rows, ld_dl] decay logits before w0
+  int ld_dl;
+  const float* w0;          // [H * dim]
+  const float* u;           // [H * dim]
+  const int4* segs;         // {first row, rows, slot, -}; null: segment i is row i with slot slots[i]
+  const int* slots;
+  float* state;             // slot s: state + s * stride, [H, dim, dim]
+  float* prev;              // slot s: prev + s * stride, [ldx]
+  long long stride;
+  const float* x;           // [rows, ldx] what the sublayer read
+  int ldx;
+  float* out;               // [rows, ld_out] fp32
+  int ld_out;
+  int H, dim;
+};
+
+constexpr int kWkThreads = 256, kWkHalf = 128, kWkRows = 16, kWkGroup = 20;
+template <int LANES>
+struct WkCfg {
+  static constexpr int kCols = kWkHalf / LANES;                  // columns per block
+  static constexpr int kChunk = LANES >= 16 ? 8 : 16;            // tokens per chunk
+  static constexpr int kVec = LANES * kWkGroup;                  // floats of one staged r / k / w vector
+  static constexpr int kTok = 3 * kVec + kCols + 4;              // + v, + r . (u k)
+  static constexpr int kSmem = 2 * kChunk * kTok * 4;
+};
+
+template <class T, int LANES>
+__global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
+  using C = WkCfg<LANES>;
+  extern __shared__ __align__(16) float smem[];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.y, col0 = blockIdx.x * C::kCols;
+  int row0, len, slot;
+  if (p.segs) {
+    const int4 s = p.segs[blockIdx.z];
+    row0 = s.x; len = s.y; slot = s.z;
+  } else {
+    row0 = blockIdx.z; len = 1; slot = p.slots[blockIdx.z];
+  }
+  const int dim = p.dim, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool stager = warp >= 4;
+  const int chunks = (len + C::kChunk - 1) / C::kChunk;
+
+  auto stage = [&](int ch) {
+    float* buf = smem + (ch & 1) * C::kChunk * C::kTok;
+    const T* r = static_cast<const T*>(p.r) + h * dim;
+    const T* k = static_cast<const T*>(p.k) + h * dim;
+    const T* v = static_cast<const T*>(p.v) + h * dim;
+    const float* dl = p.dl + h * dim;
+    constexpr int M = (LANES * kWkRows + 31) / 32;               // key channels per lane
+    constexpr int VM = (C::kCols + 31) / 32;
+    constexpr int PER = C::kChunk / 4;                           // tokens per warp
+    constexpr int U = M <= 4 ? 2 : 1;                            // tokens whose loads are in flight together
+#pragma unroll
+    for (int q0 = 0; q0 < PER; q0 += U) {
+      float fr[U][M], fk[U][M], fd[U][M], fv[U][VM];
+#pragma unroll
+      for (int q = 0; q < U; ++q) {
+        const int tok = (q0 + q) * 4 + (warp - 4), t = ch * C::kChunk + tok;
+        const size_t row = size_t(row0 + min(t, len - 1));
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          const int i = m * 32 + lane;
+          const bool in = t < len && i < dim;
+          fr[q][m] = in ? to_f32(r[row * p.ld + i]) : 0.f;
+          fk[q][m] = in ? to_f32(k[row * p.ld + i]) : 0.f;
+          fd[q][m] = in ? dl[row * p.ld_dl + i] : -INFINITY;     // decay 1: the state stays as it is
+        }
+#pragma unroll
+        for (int m = 0; m < VM; ++m) {
+          const int c = m * 32 + lane;
+          fv[q][m] = (t < len && c < C::kCols && col0 + c < dim) ? to_f32(v[row * p.ld + col0 + c]) : 0.f;
+        }
+      }
+#pragma unroll
+      for (int q = 0; q < U; ++q) {
+        const int tok = (q0 + q) * 4 + (warp - 4);
+        float* b = buf + tok * C::kTok;
+        float ruk = 0.f;
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          const int i = m * 32 + lane;
+          if (i >= LANES * kWkRows) continue;
+          const int at = (i >> 4) * kWkGroup + (i & 15);
+          const bool in = i < dim;
+          b[at] = fr[q][m];
+          b[C::kVec + at] = fk[q][m];
+          b[2 * C::kVec + at] = expf(-expf(fd[q][m] + (in ? p.w0[h * dim + i] : 0.f)));
+          ruk = fmaf(fr[q][m] * (in ? p.u[h * dim + i] : 0.f), fk[q][m], ruk);
+        }
+#pragma unroll
+        for (int m = 0; m < VM; ++m) {
+          const int c = m * 32 + lane;
+          if (c < C::kCols) b[3 * C::kVec + c] = fv[q][m];
+        }
+        ruk = warp_sum(ruk);
+        if (lane == 0) b[3 * C::kVec + C::kCols] = ruk;
+      }
+    }
+  };
+
+  // compute threads: rows g * 16 .. + 15 of column `col`
+  const int g = threadIdx.x % LANES, cl = (threadIdx.x & (kWkHalf - 1)) / LANES, col = col0 + cl;
+  uint64_t s2[kWkRows / 2];
+  float* sp = p.state + size_t(slot) * p.stride + size_t(h) * dim * dim + col;
+  if (!stager) {
+#pragma unroll
+    for (int i = 0; i < kWkRows / 2; ++i) {
+      const int r0 = g * kWkRows + 2 * i;
+      s2[i] = wk_pair((r0 < dim && col < dim) ? sp[size_t(r0) * dim] : 0.f,
+                      (r0 + 1 < dim && col < dim) ? sp[size_t(r0 + 1) * dim] : 0.f);
+    }
+  } else {
+    stage(0);
+  }
+  __syncthreads();
+  for (int ch = 0; ch < chunks; ++ch) {
+    if (stager) {
+      if (ch + 1 < chunks) stage(ch + 1);
+    } else {
+      const float* buf = smem + (ch & 1) * C::kChunk * C::kTok;
+      const int n = min(C::kChunk, len - ch * C::kChunk);
+      for (int t0 = 0; t0 < n; t0 += 4) {                        // tokens past the end are staged as no-ops
+        float o[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const float* b = buf + (t0 + q) * C::kTok;
+          const float v = b[3 * C::kVec + cl];
+          const uint64_t v2 = wk_pair(v, v);
+          uint64_t acc0 = 0, acc1 = 0;
+#pragma unroll
+          for (int i = 0; i < kWkRows / 4; ++i) {
+            const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(b + g * kWkGroup + i * 4);
+            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(b + C::kVec + g * kWkGroup + i * 4);
+            const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(b + 2 * C::kVec + g * kWkGroup + i * 4);
+            acc0 = wk_fma(r.x, s2[2 * i], acc0);
+            acc1 = wk_fma(r.y, s2[2 * i + 1], acc1);
+            s2[2 * i] = wk_fma(w.x, s2[2 * i], wk_mul(k.x, v2));
+            s2[2 * i + 1] = wk_fma(w.y, s2[2 * i + 1], wk_mul(k.y, v2));
+          }
+          float a, c, d, e;
+          wk_unpair(acc0, a, c);
+          wk_unpair(acc1, d, e);
+          o[q] = (a + c) + (d + e);
+          if (g == 0) o[q] = fmaf(b[3 * C::kVec + C::kCols], v, o[q]);
+        }
+#pragma unroll
+        for (int off = LANES / 2; off > 0; off >>= 1)
+#pragma unroll
+          for (int q = 0; q < 4; ++q) o[q] += __shfl_xor_sync(0xffffffffu, o[q], off);
+        if (g == 0 && col < dim) {
+#pragma unroll
+          for (int q = 0; q < 4; ++q)
+            if (t0 + q < n) p.out[size_t(row0 + ch * C::kChunk + t0 + q) * p.ld_out + h * dim + col] = o[q];
+        }
+      }
+    }
+    __syncthreads();
+  }
+  if (!stager) {
+#pragma unroll
+    for (int i = 0; i < kWkRows / 2; ++i) {
+      const int r0 = g * kWkRows + 2 * i;
+      float lo, hi;
+      wk_unpair(s2[i], lo, hi);
+      if (col < dim) {
+        if (r0 < dim) sp[size_t(r0) * dim] = lo;
+        if (r0 + 1 < dim) sp[size_t(r0 + 1) * dim] = hi;
+      }
+    }
+  } else if (blockIdx.x == 0 && h == 0) {
+    const float* last = p.x + size_t(row0 + len - 1) * p.ldx;
+    float* keep = p.prev + size_t(slot) * p.stride;
+    for (int i = threadIdx.x - kWkHalf; i < p.ldx; i += kWkHalf) keep[i] = last[i];
+  }
+}
+
+// a[t, h*dim + i] = o / rms(o over the head) * norm * silu(gate). One warp per (row, head).
+template <class T>
+__global__ void __launch_bounds__(kRowThreads)
+wkv_finish_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ gate, int ld_g,
+                  const float* __restrict__ norm, float eps, T* __restrict__ a, int ld_a, int rows, int H, int dim) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int unit = blockIdx.x * (kRowThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (unit >= rows * H) return;
+  const int t = unit / H, h = unit - t * H;
+  const float* src = o + size_t(t) * ld_o + h * dim;
+  float ssq = 0.f;
+  for (int i = lane; i < dim; i += 32) ssq += src[i] * src[i];
+  const float inv = 1.f / sqrtf(warp_sum(ssq) / float(dim) + eps);
+  for (int i = lane; i < dim; i += 32) {
+    const float z = to_f32(gate[size_t(t) * ld_g + h * dim + i]);
+    a[size_t(t) * ld_a + h * dim + i] = from_f32<T>(src[i] * inv * norm[h * dim + i] * (z / (1.f + expf(-z))));
+  }
+}
+
+template <class T, int LANES>
+static int launch_wkv(const WkvParams& p, int n_segs, int pdl, cudaStream_t st) {
+  using C = WkCfg<LANES>;
+  auto kern = wkv_scan_kernel<T, LANES>;
+  RB_CHECK(set_max_smem(kern, C::kSmem));
+  return launch(kern, dim3((p.dim + C::kCols - 1) / C::kCols, p.H, n_segs), dim3(kWkThreads), C::kSmem, st, pdl != 0, p);
+}
+template <class T>
+static int dispatch_wkv(const WkvParams& p, int n, int pdl, cudaStream_t st) {
+  const int groups = (p.dim + kWkRows - 1) / kWkRows;
+  if (groups <= 1) return launch_wkv<T, 1>(p, n, pdl, st);
+  if (groups <= 2) return launch_wkv<T, 2>(p, n, pdl, st);
+  if (groups <= 4) return launch_wkv<T, 4>(p, n, pdl, st);
+  if (groups <= 8) return launch_wkv<T, 8>(p, n, pdl, st);
+  if (groups <= 16) return launch_wkv<T, 16>(p, n, pdl, st);
+  return -2;
+}
+
+}  // namespace rb
+
+using namespace rb;
+
+// Largest head size of the recurrence.
+extern "C" int rmlx_wkv_max_dim() { return 16 * kWkRows; }
+
+// x fp32 [T, ldx], mu fp32 [5, ldx], out [5, T, ldx] fp32 (f32) or bf16; ldx a multiple of eight, prev
+// rows 16-byte aligned. slots int32 [T].
+extern "C" int rmlx_token_shift(const float* x, int ldx, const float* mu, const float* prev, long long prev_stride,
+                                const int* slots, int each_row, void* out, int T, int f32, int pdl, cudaStream_t st) {
+  if (T < 1 || ldx < 8 || ldx % 8 || prev_stride % 4 || !slots) return -2;
+  if (f32)
+    return launch(token_shift_kernel<float>, dim3(T), dim3(kRowThreads), 0, st, pdl != 0, x, ldx, mu, prev, prev_stride,
+                  slots, each_row, static_cast<float*>(out), T);
+  return launch(token_shift_kernel<__nv_bfloat16>, dim3(T), dim3(kRowThreads), 0, st, pdl != 0, x, ldx, mu, prev,
+                prev_stride, slots, each_row, static_cast<__nv_bfloat16*>(out), T);
+}
+
+// r, k, v [rows, ld] fp32 (f32) or bf16; dl fp32 [rows, ld_dl]; segs int32 [n_segs, 4] (16-byte aligned) or
+// null with slots [n_segs]: then every row is a segment. No slot occurs twice except one that nobody reads.
+extern "C" int rmlx_wkv_scan(const void* r, const void* k, const void* v, int ld, const float* dl, int ld_dl,
+                             const float* w0, const float* u, const int* segs, const int* slots, int n_segs,
+                             float* state, float* prev, long long stride, const float* x, int ldx, float* out,
+                             int ld_out, int H, int dim, int f32, int pdl, cudaStream_t st) {
+  if (n_segs < 1 || n_segs > 65535 || H < 1 || H > 65535 || dim < 1 || ld < H * dim || ld_dl < H * dim ||
+      ld_out < H * dim || (!segs && !slots) || (reinterpret_cast<uintptr_t>(segs) & 15))
+    return -2;
+  WkvParams p;
+  p.r = r; p.k = k; p.v = v; p.ld = ld; p.dl = dl; p.ld_dl = ld_dl; p.w0 = w0; p.u = u;
+  p.segs = reinterpret_cast<const int4*>(segs); p.slots = slots;
+  p.state = state; p.prev = prev; p.stride = stride; p.x = x; p.ldx = ldx; p.out = out; p.ld_out = ld_out;
+  p.H = H; p.dim = dim;
+  return f32 ? dispatch_wkv<float>(p, n_segs, pdl, st) : dispatch_wkv<__nv_bfloat16>(p, n_segs, pdl, st);
+}
+
+extern "C" int rmlx_wkv_finish(const float* o, int ld_o, const void* gate, int ld_g, const float* norm, float eps,
+                               void* a, int ld_a, int rows, int H, int dim, int f32, int pdl, cudaStream_t st) {
+  const long long units = 1LL * rows * H;
+  if (rows < 1 || H < 1 || dim < 1 || units > 0x7fffffffLL) return -2;
+  const dim3 grid(unsigned((units + kRowThreads / 32 - 1) / (kRowThreads / 32)));
+  if (f32)
+    return launch(wkv_finish_kernel<float>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o,
+                  static_cast<const float*>(gate), ld_g, norm, eps, static_cast<float*>(a), ld_a, rows, H, dim);
+  return launch(wkv_finish_kernel<__nv_bfloat16>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o,
+                static_cast<const __nv_bfloat16*>(gate), ld_g, norm, eps, static_cast<__nv_bfloat16*>(a), ld_a, rows,
+                H, dim);
+}

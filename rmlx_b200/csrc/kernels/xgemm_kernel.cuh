@@ -3,7 +3,7 @@
 //   * W bf16 (TMA-fed) or MLX-affine Q4 dequantised inside the main loop by eight dequant warps;
 //   * GROUPED: rows of A sorted by expert, tile table derived on the device from offsets[E+1];
 //   * swiglu: a tile holds BN/2 gate rows and the matching BN/2 up rows of W; the epilogue writes
-//     silu(gate) * up straight from the fp32 accumulators;
+//     the gated activation (gated.cuh) straight from the fp32 accumulators;
 //   * COMM = kCommReduce: this rank holds a K-shard; every finished accumulator tile is stored
 //     straight into the staging slab of the rank that owns the tile (peer stores over NVLink; a
 //     signalling warp publishes a release counter per tile); four collective warps of the owner
@@ -22,6 +22,7 @@
 #include "../common/ptx.cuh"
 #include "../common/launch.cuh"
 #include "../common/tensormap.cuh"
+#include "../common/gated.cuh"
 
 namespace rb {
 
@@ -189,7 +190,7 @@ xgemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__
              const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_s,
              const __grid_constant__ CUtensorMap tmap_b, __nv_bfloat16* __restrict__ C,
              const __nv_bfloat16* __restrict__ residual, const int* __restrict__ offsets, int E, int M,
-             int N, int K, int ldc, int* __restrict__ status, const XComm cm, int swiglu) {
+             int N, int K, int ldc, int* __restrict__ status, const XComm cm, int swiglu, float gate_limit) {
   static_assert(COMM == kCommNone || !GROUPED, "collective modes are for plain GEMMs");
   static_assert(MT == 1 || (COMM == kCommNone && 2 * BN * MT <= 512), "stacked tiles: no collective modes");
   using S = XSmem<BN, WQ4, MT>;
@@ -425,8 +426,7 @@ xgemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__
             float f[32];
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
-              const float g = __uint_as_float(rg[j]);
-              f[j] = g / (1.f + __expf(-g)) * __uint_as_float(ru[j]);
+              f[j] = gated_act_fast(__uint_as_float(rg[j]), __uint_as_float(ru[j]), gate_limit);
             }
             if (col0 + 32 <= n_out) {
 #pragma unroll
@@ -678,7 +678,7 @@ template <int BN, bool WQ4, bool GROUPED, bool RESIDUAL, int COMM = kCommNone, i
 static int launch_x(const CUtensorMap& ta, const CUtensorMap& ta2, const CUtensorMap& tw,
                     const CUtensorMap& ts, const CUtensorMap& tb, void* C, const void* residual,
                     const int* offsets, int E, int M, int N, int K, int ldc, int* status, int pdl,
-                    cudaStream_t st, const XComm& cm = XComm(), int swiglu = 0) {
+                    cudaStream_t st, const XComm& cm = XComm(), int swiglu = 0, float gate_limit = 0.f) {
   using S = XSmem<BN, WQ4, MT>;
   auto kern = xgemm_kernel<BN, WQ4, GROUPED, RESIDUAL, COMM, MT>;
   RB_CHECK(set_max_smem(kern, S::kBytes));
@@ -687,7 +687,7 @@ static int launch_x(const CUtensorMap& ta, const CUtensorMap& ta2, const CUtenso
   const int grid = tiles < sm_count() ? (tiles > 0 ? tiles : 1) : sm_count();
   return launch(kern, dim3(grid), dim3(S::kThreads + (COMM != kCommNone ? kCommThreads : 0)), size_t(S::kBytes), st, pdl != 0, ta, ta2, tw, ts, tb,
                 static_cast<__nv_bfloat16*>(C), static_cast<const __nv_bfloat16*>(residual), offsets, E,
-                M, N, K, ldc, status, cm, swiglu);
+                M, N, K, ldc, status, cm, swiglu, gate_limit);
 }
 
 // Tensor maps of the weight operand (and of its scales/biases for Q4).

@@ -29,12 +29,13 @@ extern "C" int rmlx_qgemm_supported(int K) { return K % 512 == 0; }
 //   offsets == nullptr: plain GEMM, rowsW = N.
 //   offsets != nullptr: grouped; A rows are sorted by expert, offsets[E+1] (device, int32),
 //                       rowsW = E*N, N must be a multiple of the tile width.
-//   swiglu != 0: W's N rows (per expert) are [gate; up]; C gets N/2 columns of silu(gate)*up,
-//                computed in the epilogue from the fp32 accumulators (no residual in this mode).
+//   swiglu != 0: W's N rows (per expert) are [gate; up]; C gets N/2 columns of the gated activation
+//                (gate_limit 0: silu(gate)*up, else the clamped gate of gated.cuh), computed in the
+//                epilogue from the fp32 accumulators (no residual in this mode).
 extern "C" int rmlx_xgemm(int w_kind, const void* A, const void* W, const void* scales,
                           const void* biases, void* C, const void* residual, const int* offsets,
                           int E, int M, int N, int K, int lda, int ldc, int bn, int swiglu,
-                          int* status, int pdl, cudaStream_t st) {
+                          float gate_limit, int* status, int pdl, cudaStream_t st) {
   if (M < 1 || N < 1 || K < 8 || K % 8 || lda % 8) return -2;
   if (w_kind == 1 && !rmlx_qgemm_supported(K)) return -2;
   const bool grouped = offsets != nullptr;
@@ -65,19 +66,19 @@ extern "C" int rmlx_xgemm(int w_kind, const void* A, const void* W, const void* 
   if (rc) return rc;
 #define RB_X(BN_, Q_, G_)                                                                          \
   return residual ? launch_x<BN_, Q_, G_, true>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st) \
-                  : launch_x<BN_, Q_, G_, false>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu)
+                  : launch_x<BN_, Q_, G_, false>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu, gate_limit)
   if (mt == 2 && grouped) {
     if (w_kind == 1)
-      return launch_x<128, true, true, false, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu);
-    return launch_x<128, false, true, false, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu);
+      return launch_x<128, true, true, false, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu, gate_limit);
+    return launch_x<128, false, true, false, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu, gate_limit);
   }
   if (mt == 2) {
     if (w_kind == 1) {
       return residual ? launch_x<128, true, false, true, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st)
-                      : launch_x<128, true, false, false, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu);
+                      : launch_x<128, true, false, false, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu, gate_limit);
     }
     return residual ? launch_x<128, false, false, true, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st)
-                    : launch_x<128, false, false, false, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu);
+                    : launch_x<128, false, false, false, kCommNone, 2>(ta, ta, tw, ts, tb, C, residual, offsets, E, M, N, K, ldc, status, pdl, st, XComm(), swiglu, gate_limit);
   }
   if (bn == 256) {
     if (w_kind == 1) { if (grouped) { RB_X(256, true, true); } else { RB_X(256, true, false); } }

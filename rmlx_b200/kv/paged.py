@@ -11,6 +11,7 @@ tensor so a captured decode graph sees growth without re-capture.
 """
 from __future__ import annotations
 
+import math
 from typing import Dict, List, Optional
 
 import torch
@@ -232,12 +233,20 @@ class PagedKvCache:
 
     ``layer_shapes``: one ``(kv_heads, key width, value width)`` per layer, for models whose layers
     differ or whose keys and values have different widths (``kv_heads`` / ``head_dim`` are then only
-    the first layer's)."""
+    the first layer's). A value width of 0 stands for rows that are key and value at once (latent
+    attention: ``v`` is the same pool as ``k``), None for a layer without keys (a recurrent one).
+
+    ``layer_states``: per layer a dict name -> shape of what a recurrent layer carries from token to
+    token (None: nothing). The states of one sequence are one fp32 row of ``state``, at the sequence's
+    slot: cleared when the sequence is added, copied by ``fork``. The last row, ``idle_slot``, belongs
+    to no sequence (idle batch rows write there). A state cannot be rolled back or started from cached
+    pages: ``trim`` and ``adopt_prefix`` refuse."""
 
     def __init__(self, num_blocks: int, num_layers: int, kv_heads: int, head_dim: int,
                  dtype=torch.bfloat16, device="cpu", max_seqs: int = 64,
                  max_blocks_per_seq: int = 512, block_size: int = PAGE,
-                 kv_quant: Optional[str] = None, layer_shapes: Optional[List[tuple]] = None):
+                 kv_quant: Optional[str] = None, layer_shapes: Optional[List[Optional[tuple]]] = None,
+                 layer_states: Optional[List[Optional[Dict[str, tuple]]]] = None):
         self.manager = make_block_manager(num_blocks, block_size, reserved=1)
         self.num_layers, self.kv_heads, self.head_dim = num_layers, kv_heads, head_dim
         self.block_size = block_size
@@ -257,11 +266,22 @@ class PagedKvCache:
             self.k_sb = [torch.zeros(sbs, dtype=torch.bfloat16, device=device) for _ in range(num_layers)]
             self.v_sb = [torch.zeros(sbs, dtype=torch.bfloat16, device=device) for _ in range(num_layers)]
         else:
-            self.k = [torch.zeros(num_blocks, h, block_size, dk, dtype=dtype, device=device)
-                      for h, dk, _ in self.layer_shapes]
-            self.v = [torch.zeros(num_blocks, h, block_size, dv, dtype=dtype, device=device)
-                      for h, _, dv in self.layer_shapes]
+            def pool(h, width):
+                return torch.zeros(num_blocks, h, block_size, width, dtype=dtype, device=device)
+            self.k = [None if s is None else pool(s[0], s[1]) for s in self.layer_shapes]
+            self.v = [k if s is None or not s[2] else pool(s[0], s[2]) for k, s in zip(self.k, self.layer_shapes)]
             self.k_sb = self.v_sb = None
+        self.state = None
+        if layer_states is not None and any(layer_states):
+            if len(layer_states) != num_layers:
+                raise ValueError("layer_states: one entry per layer")
+            self._state_at, total = {}, 0
+            for l, pieces in enumerate(layer_states):
+                for name, shape in (pieces or {}).items():
+                    self._state_at[l, name] = (total, tuple(shape))
+                    total += (math.prod(shape) + 3) // 4 * 4          # 16-byte rows
+            self.state = torch.zeros(max_seqs + 1, total, dtype=torch.float32, device=device)
+        self.idle_slot = max_seqs
         self.device = torch.device(device)
         self.max_blocks_per_seq = max_blocks_per_seq
         # row r of the device table belongs to the sequence bound to slot r
@@ -280,7 +300,15 @@ class PagedKvCache:
         self.manager.add_sequence(seq_id)
         slot = self._free_slots.pop()
         self.slot_of[seq_id] = slot
+        if self.state is not None:
+            self.state[slot].zero_()
         return slot
+
+    def layer_state(self, layer: int, name: str) -> torch.Tensor:
+        """One piece of a recurrent layer's state for every slot, [max_seqs + 1, *shape]: a view whose
+        slots are ``state.stride(0)`` apart."""
+        at, shape = self._state_at[layer, name]
+        return self.state[:, at:at + math.prod(shape)].unflatten(1, shape)
 
     def free_sequence(self, seq_id: int) -> None:
         self.manager.free_sequence(seq_id)
@@ -293,11 +321,15 @@ class PagedKvCache:
         self.manager.fork(parent, child)
         slot = self._free_slots.pop()
         self.slot_of[child] = slot
+        if self.state is not None:
+            self.state[slot].copy_(self.state[self.slot_of[parent]])
         self._sync_slot(child)
         return slot
 
     def adopt_prefix(self, seq_id: int, blocks: List[int], num_tokens: int) -> None:
         """Start an (empty, already added) sequence from cached prefix pages."""
+        if self.state is not None:
+            raise ValueError("a recurrent layer's state is not part of the cached pages")
         self.manager.adopt(seq_id, blocks, num_tokens)
         self._sync_slot(seq_id)
 
@@ -331,8 +363,11 @@ class PagedKvCache:
         copies = self.manager.reserve(seq_id, new_tokens)
         for src, dst in copies:
             for l in range(self.num_layers):
+                if self.k[l] is None:
+                    continue
                 self.k[l][dst].copy_(self.k[l][src])
-                self.v[l][dst].copy_(self.v[l][src])
+                if self.v[l] is not self.k[l]:
+                    self.v[l][dst].copy_(self.v[l][src])
                 if self.quantized:
                     self.k_sb[l][dst].copy_(self.k_sb[l][src])
                     self.v_sb[l][dst].copy_(self.v_sb[l][src])
@@ -343,6 +378,8 @@ class PagedKvCache:
         self.manager.commit(seq_id, new_tokens)
 
     def trim(self, seq_id: int, num_tokens: int) -> None:
+        if self.state is not None and num_tokens > 0:
+            raise ValueError("a recurrent layer's state cannot be rolled back")
         self.manager.trim(seq_id, num_tokens)
         self._sync_slot(seq_id)
 
@@ -399,4 +436,8 @@ class PagedKvCache:
         if self.quantized:
             return 2 * self.num_layers * self.kv_heads * (self.head_dim + (self.head_dim // 64) * 4)
         size = torch.empty(0, dtype=self.dtype).element_size()
-        return sum(h * (dk + dv) for h, dk, dv in self.layer_shapes) * size
+        return sum(s[0] * (s[1] + s[2]) for s in self.layer_shapes if s is not None) * size
+
+    def bytes_per_sequence(self) -> int:
+        """Recurrent state one sequence occupies whatever its length."""
+        return 0 if self.state is None else self.state.shape[1] * 4

@@ -56,6 +56,8 @@ class DecodeEngineBase:
         self.active = torch.zeros(max_batch, **i32)
         self.next_tokens = torch.zeros(max_batch, **i32)
         self.block_table = torch.zeros(max_batch, cache.max_blocks_per_seq, **i32)
+        # models with recurrent layers: the state slot of every batch row (idle rows: nobody's)
+        self.state_slots = None if cache.state is None else torch.full((max_batch,), cache.idle_slot, **i32)
         self.vocab_local = model.w.lm_head.n
         self.logits = torch.zeros(max_batch, cfg.vocab_size, dtype=torch.float32, device=dev)
         # One captured graph per batch bucket (1, 2, 4, ... max_batch): a step runs the smallest
@@ -94,6 +96,9 @@ class DecodeEngineBase:
         # inactive rows still run (shape-stable graph): give them a harmless one-token context
         if n < self.B:
             self.seq_lens[n:] = 1
+        if self.state_slots is not None:
+            self.state_slots.copy_(torch.tensor([self.cache.slot_of[s] for s in seq_ids] +
+                                                [self.cache.idle_slot] * (self.B - n), dtype=torch.int32))
         self.refresh_tables()
 
     def refresh_tables(self) -> None:
@@ -138,10 +143,15 @@ class DecodeEngineBase:
         nb = self.bucket() if nb is None else nb
         state = (self.tokens, self.positions, self.seq_lens)
         saved = [t.clone() for t in state]
+        if self.state_slots is not None:      # a run also advances the bound sequences' recurrent state
+            slots = self.state_slots.long()
+            saved_rows = self.cache.state.index_select(0, slots)
 
         def restore():
             for t, sv in zip(state, saved):
                 t.copy_(sv)
+            if self.state_slots is not None:
+                self.cache.state.index_copy_(0, slots, saved_rows)
 
         return self.graphs.get_or_capture(("decode", nb), lambda: self._run_step(nb), warmup=1,
                                           restore=restore, device=self.model.device)

@@ -3,8 +3,8 @@ beside single decoded tokens.
 
 ``RaggedBatch`` turns (sequence, tokens) entries into the device arrays the kernels read: token ids,
 positions, the block-table row of every token, the query tiles of the entries with several tokens
-(tensor-core prompt attention) and the rows of those with one (split-KV decode attention). Everything
-travels in one pinned copy."""
+(tensor-core prompt attention), the rows of those with one (split-KV decode attention) and the run of
+rows of every entry (recurrent layers). Everything travels in one pinned copy."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -82,7 +82,9 @@ class RaggedBatch:
 
     def upload(self, device) -> "RaggedBatch":
         n, tiles = self.num_tokens, self.tiles_host
+        runs = [x for s, l, slot, p in zip(self.starts, self.lens, self.slots, self.pos0) for x in (s, l, slot, p)]
         parts = [torch.tensor([x for t in tiles for x in t], dtype=torch.int32),     # 16-byte records first
+                 torch.tensor(runs, dtype=torch.int32),
                  torch.cat([torch.as_tensor(e.tokens, dtype=torch.int32).reshape(-1) for e in self.entries]),
                  torch.cat([torch.arange(p, p + l, dtype=torch.int32) for p, l in zip(self.pos0, self.lens)]),
                  torch.repeat_interleave(torch.tensor(self.slots, dtype=torch.int32), torch.tensor(self.lens)),
@@ -97,8 +99,9 @@ class RaggedBatch:
             out.append(flat[at:at + p.numel()])
             at += p.numel()
         self.tiles = out[0].view(-1, 4) if tiles else None
-        self.tokens, self.positions, self.token_seq = out[1], out[2], out[3]
-        self.single = out[4] if self.single_host else None
-        self.want = out[5]
+        self.runs = out[1].view(-1, 4)            # (first row, rows, slot, position of the first row) per entry
+        self.tokens, self.positions, self.token_seq = out[2], out[3], out[4]
+        self.single = out[5] if self.single_host else None
+        self.want = out[6]
         assert self.tokens.numel() == n
         return self

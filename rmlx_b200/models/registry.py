@@ -86,6 +86,23 @@ def _posudra_model(weights):
     return PosudraModel(weights)
 
 
+def _rodapel_weights(model_dir, config, device, dtype, layout):
+    from ..config import RodapelConfig
+    from ..loader.safetensors_loader import load_tensors
+    from .rodapel import build_weights
+    if layout is not None and layout.world != 1:
+        raise ValueError("Rodapel runs on one GPU")
+    cfg = RodapelConfig.from_json(config)
+    return build_weights(cfg, load_tensors(model_dir), device, dtype), cfg
+
+
+def _rodapel_model(weights):
+    from .rodapel import RodapelModel
+    return RodapelModel(weights)
+
+
 register(ModelFamily("transformer", lambda c: "num_attention_heads" in c, _transformer_weights, _transformer_model))
 register(ModelFamily("posudra", lambda c: c.get("architecture") == "Posudra", _posudra_weights, _posudra_model,
                      kernels="parallel_block"))
+register(ModelFamily("rodapel", lambda c: c.get("architecture") == "Rodapel", _rodapel_weights, _rodapel_model,
+                     kernels="post_norm"))

@@ -27,14 +27,14 @@ _lib.register_cuda_sigs({
     "rmlx_sgemm": ("pipipiiiiip", "i"),
     "rmlx_sgemm_split_xielu": ("pipipiipiffiiiip", "i"),
     "rmlx_sgemm_scaled_add": ("pipippiiiiip", "i"),
-    "rmlx_attention_any": ("pppppppiiiiiiiiffppppiip", "i"),
+    "rmlx_attention_any": ("pppppppipiiiiiiiiii" "ffpppp" "piiip", "i"),
     "rmlx_flash_prefill_scored_supported": ("ii", "i"),
-    "rmlx_flash_prefill_scored": ("ppppipipiiiiiiiffppppipip", "i"),
+    "rmlx_flash_prefill_scored": ("ppppipipiiiiiiiffpppp" "piipip", "i"),
     "rmlx_flash_decode_scored_supported": ("ii", "i"),
     "rmlx_flash_decode_scored_part_o_elems": ("iiiii", "q"),
     "rmlx_flash_decode_scored_part_ml_elems": ("iiii", "q"),
     "rmlx_flash_decode_scored_ticket_elems": ("iii", "q"),
-    "rmlx_flash_decode_scored": ("ppippfpppppppppp" "iiiiiiiiii" "ffppppip", "i"),
+    "rmlx_flash_decode_scored": ("ppippfpppppppppp" "iiiiiiiiii" "ffpppp" "piiiip", "i"),
 })
 
 
@@ -204,6 +204,13 @@ def qk_norm_append(raw: torch.Tensor, q_w: torch.Tensor, k_w: torch.Tensor, eps:
     _lib.check(rc, "qk_norm_append")
 
 
+def _gate_args(gate: Optional[torch.Tensor], t: int, h: int, dtype):
+    if gate is None:
+        return None, 0
+    assert gate.shape == (t, h) and gate.stride(1) == 1 and gate.dtype == dtype
+    return gate.data_ptr(), gate.stride(0)
+
+
 def prefill_scored_supported(dk: int, dv: int) -> bool:
     return bool(_lib.cuda().rmlx_flash_prefill_scored_supported(dk, dv))
 
@@ -214,9 +221,10 @@ def decode_scored_supported(dk: int, dv: int) -> bool:
 
 def flash_prefill_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                          tiles: torch.Tensor, mods: ScoreMods, out: torch.Tensor, window: int = 0, lanes: int = 1,
-                         pdl: bool = False) -> torch.Tensor:
+                         gate: Optional[torch.Tensor] = None, pdl: bool = False) -> torch.Tensor:
     """Ragged causal attention over pages on the tensor cores: q [T, H, dk] bf16; ``tiles`` int32
-    [n, 4] = (first row, rows <= lanes * 128, position of the first row, row of ``block_table``)."""
+    [n, 4] = (first row, rows <= lanes * 128, position of the first row, row of ``block_table``).
+    ``gate`` [T, H]: logits of a sigmoid each head's output is multiplied by."""
     _lib.require_cuda_tensor(q, k_cache, v_cache, block_table, tiles, out)
     t, h, dk = q.shape
     assert q.is_contiguous() and out.is_contiguous() and tiles.dtype == torch.int32 and tiles.is_contiguous()
@@ -224,7 +232,7 @@ def flash_prefill_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
     rc = _lib.cuda().rmlx_flash_prefill_scored(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), block_table.stride(0),
         tiles.data_ptr(), tiles.shape[0], out.data_ptr(), t, h, k_cache.shape[1], dk, v_cache.shape[3],
-        k_cache.shape[0], window, *mods.args(), lanes, GemmStatus.get(q.device).data_ptr(), int(pdl),
+        k_cache.shape[0], window, *mods.args(), *_gate_args(gate, t, h, q.dtype), lanes, GemmStatus.get(q.device).data_ptr(), int(pdl),
         _lib.stream_ptr())
     _lib.check(rc, "flash_prefill_scored")
     return out
@@ -250,10 +258,12 @@ def flash_decode_scored(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tabl
                         raw: Optional[torch.Tensor] = None, q_w: Optional[torch.Tensor] = None,
                         k_w: Optional[torch.Tensor] = None, eps: float = 0.0, rows: Optional[torch.Tensor] = None,
                         table_rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None, window: int = 0,
+                        gate: Optional[torch.Tensor] = None, head_norm: bool = False, gate_col: int = -1,
                         pdl: bool = False) -> torch.Tensor:
     """One token per row: q [T, H, dk] (keys already appended) or the fused form on the un-normalised
-    fp32 projection ``raw`` [T, >= q|k|v], which also appends the key and value. ``rows`` int32: the
-    batch rows to run (default: the first ``n_rows``)."""
+    fp32 projection ``raw`` [T, >= q|k|v], which also appends the key and value (``head_norm``: the
+    norms are per head, their weights [dim]; ``gate_col``: where the output gate's logits start in a
+    row). ``rows`` int32: the batch rows to run (default: the first ``n_rows``)."""
     _lib.require_cuda_tensor(k_cache, v_cache, block_table, positions, out, q, raw)
     src = q if q is not None else raw
     n = rows.numel() if rows is not None else (n_rows or src.shape[0])
@@ -265,22 +275,28 @@ def flash_decode_scored(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tabl
         k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), positions.data_ptr(), _lib.ptr(rows),
         _lib.ptr(table_rows), out.data_ptr(), scratch.part_o.data_ptr(), scratch.part_ml.data_ptr(),
         scratch.tickets.data_ptr(), n, heads, k_cache.shape[1], dim, vdim, k_cache.shape[3], v_cache.shape[3],
-        block_table.stride(0), scratch.splits, window, *mods.args(), int(pdl), _lib.stream_ptr())
+        block_table.stride(0), scratch.splits, window, *mods.args(),
+        *_gate_args(gate, 0 if q is None else q.shape[0], heads, torch.bfloat16), int(head_norm), gate_col, int(pdl),
+        _lib.stream_ptr())
     _lib.check(rc, "flash_decode_scored")
     return out
 
 
 def attention_any(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                   positions: torch.Tensor, token_seq: Optional[torch.Tensor], mods: ScoreMods, out: torch.Tensor,
-                  window: int = 0, pdl: bool = False) -> torch.Tensor:
-    """Attention of single query tokens over pages for any head widths, bf16 or fp32 storage."""
+                  window: int = 0, gate: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+                  pdl: bool = False) -> torch.Tensor:
+    """Attention of single query tokens over pages for any head widths, bf16 or fp32 storage. Cache rows
+    may be wider than the query (key) and the output (value): ``k_cache`` and ``v_cache`` may be one
+    pool whose rows hold both (latent attention). ``rows``: batch rows to run (default: all)."""
     _lib.require_cuda_tensor(q, k_cache, v_cache, block_table, positions, token_seq, out)
     t, h, dk = q.shape
     assert q.is_contiguous() and out.is_contiguous() and q.dtype == k_cache.dtype == out.dtype
-    assert k_cache.shape[3] == dk and out.shape == (t, h, v_cache.shape[3])
+    assert k_cache.shape[3] >= dk and out.shape[:2] == (t, h) and v_cache.shape[3] >= out.shape[2]
     rc = _lib.cuda().rmlx_attention_any(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), positions.data_ptr(),
-        _lib.ptr(token_seq), out.data_ptr(), t, h, k_cache.shape[1], dk, v_cache.shape[3], block_table.stride(0),
-        k_cache.shape[2], window, *mods.args(), _f32(q), int(pdl), _lib.stream_ptr())
+        _lib.ptr(token_seq), _lib.ptr(rows), 0 if rows is None else rows.numel(), out.data_ptr(), t, h,
+        k_cache.shape[1], dk, out.shape[2], k_cache.shape[3], v_cache.shape[3], block_table.stride(0),
+        k_cache.shape[2], window, *mods.args(), *_gate_args(gate, t, h, q.dtype), _f32(q), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "attention_any")
     return out

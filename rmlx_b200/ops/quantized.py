@@ -16,7 +16,7 @@ from .weights import LinearWeight, W_Q4
 
 _lib.register_cuda_sigs({
     "rmlx_qgemm_supported": ("i", "i"),
-    "rmlx_xgemm": ("ipppppppiiiiiiiipip", "i"),
+    "rmlx_xgemm": ("ipppppppiiiiiiiifpip", "i"),
     "rmlx_moe_scatter_rows": ("pipppppiiiip", "i"),
     "rmlx_moe_combine": ("ppppipiiiip", "i"),
 })
@@ -24,10 +24,11 @@ _lib.register_cuda_sigs({
 
 def xgemm(x: torch.Tensor, w: LinearWeight, residual: Optional[torch.Tensor] = None,
           out: Optional[torch.Tensor] = None, offsets: Optional[torch.Tensor] = None, bn: int = 0,
-          pdl: bool = False, swiglu: bool = False) -> torch.Tensor:
+          pdl: bool = False, swiglu: bool = False, gate_limit: float = 0.0) -> torch.Tensor:
     """Plain (offsets None) or grouped tensor-core GEMM with bf16 or Q4 weights.
     Grouped: x rows sorted by expert, ``offsets`` int32 [E+1] on the device, w stacked [E, N, K].
-    ``swiglu``: w's rows are [gate; up]; the result has N/2 columns of silu(gate) * up."""
+    ``swiglu``: w's rows are [gate; up]; the result has N/2 columns of silu(gate) * up, or of the
+    clamped gate (csrc/common/gated.cuh) when ``gate_limit`` is positive."""
     _lib.require_cuda_tensor(x, w.w)
     assert x.dtype == torch.bfloat16 and x.dim() == 2 and x.stride(1) == 1
     m, k = x.shape
@@ -41,6 +42,7 @@ def xgemm(x: torch.Tensor, w: LinearWeight, residual: Optional[torch.Tensor] = N
     rc = _lib.cuda().rmlx_xgemm(w.kind, x.data_ptr(), w.w.data_ptr(), _lib.ptr(w.scales),
                                 _lib.ptr(w.biases), out.data_ptr(), _lib.ptr(residual),
                                 _lib.ptr(offsets), e, m, n, k, x.stride(0), out.stride(0), bn, int(swiglu),
+                                gate_limit,
                                 GemmStatus.get(x.device).data_ptr(), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "xgemm")
     return out

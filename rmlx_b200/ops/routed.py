@@ -1,0 +1,93 @@
+"""Routing by corrected scores with identity experts (csrc/kernels/moe_route.cu) and the grouped expert
+feed-forward around it for any number of tokens: route -> rows sorted by expert -> gate/up with the gated
+activation -> down. The combination with the output norm is ``combine_post_norm`` (postnorm_rows.cu)."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from .. import _lib
+from .parallel_block import _f32
+from .post_norm import gated_act
+from .quantized import xgemm
+from .weights import LinearWeight
+
+ROUTE_MAX_OUTPUTS, ROUTE_MAX_TOP = 512, 32       # of the routing kernel
+
+_lib.register_cuda_sigs({
+    "rmlx_route_max_outputs": ("", "i"),
+    "rmlx_route_max_top": ("", "i"),
+    "rmlx_route_corrected": ("pippppppiiiiip", "i"),
+    "rmlx_route_scatter": ("pipppp" "iiiiip", "i"),
+    "rmlx_moe_combine_post_norm": ("pipppipfppiiiiip", "i"),
+    "rmlx_sgemm_grouped": ("pipipipiiiiip", "i"),
+})
+
+
+@dataclass
+class Routing:
+    """Device arrays of one routed batch (views of preallocated buffers)."""
+    idx: torch.Tensor            # int32 [T, top]; identity experts have idx >= experts
+    weights: torch.Tensor        # fp32 [T, top]
+    identity: torch.Tensor       # fp32 [T] summed weight of the identity experts
+    counts: torch.Tensor         # int32 [experts]
+    offsets: torch.Tensor        # int32 [experts + 1]
+    row_of_pair: torch.Tensor    # int32 [T, top]; -1: no row
+
+
+def route_corrected(logits: torch.Tensor, correction: torch.Tensor, experts: int, r: Routing, grouped: bool = True,
+                    pdl: bool = False) -> None:
+    """Chooses by softmax + correction, weights by the softmax alone. ``grouped``: also the experts' row ranges."""
+    _lib.require_cuda_tensor(logits, correction, r.idx)
+    t, outputs = logits.shape
+    assert logits.dtype == correction.dtype == torch.float32 and correction.numel() == outputs
+    rc = _lib.cuda().rmlx_route_corrected(
+        logits.data_ptr(), logits.stride(0), correction.data_ptr(), r.idx.data_ptr(), r.weights.data_ptr(),
+        r.identity.data_ptr(), r.counts.data_ptr() if grouped else None, r.offsets.data_ptr() if grouped else None, t,
+        experts, outputs, r.idx.shape[1], int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "route_corrected")
+
+
+def route_scatter(h: torch.Tensor, r: Routing, xs: torch.Tensor, pdl: bool = False) -> None:
+    """Copies every routed (token, slot) row of ``h`` into ``xs`` [T * top, width], sorted by expert."""
+    _lib.require_cuda_tensor(h, xs)
+    t, top = r.idx.shape
+    assert h.is_contiguous() and xs.is_contiguous() and xs.shape == (t * top, h.shape[1]) and xs.dtype == h.dtype
+    rc = _lib.cuda().rmlx_route_scatter(h.data_ptr(), h.stride(0), r.idx.data_ptr(), r.counts.data_ptr(), xs.data_ptr(),
+                                        r.row_of_pair.data_ptr(), t, top, r.counts.numel(), _f32(h), int(pdl),
+                                        _lib.stream_ptr())
+    _lib.check(rc, "route_scatter")
+
+
+def _sgemm_grouped(x, w, offsets, out, max_rows, pdl):
+    rc = _lib.cuda().rmlx_sgemm_grouped(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(1), offsets.data_ptr(),
+                                        w.shape[0], out.data_ptr(), out.stride(0), max_rows, w.shape[1], w.shape[2],
+                                        int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "sgemm_grouped")
+
+
+def grouped_gated_ffn(xs: torch.Tensor, offsets: torch.Tensor, gate_up: LinearWeight, down: LinearWeight, limit: float,
+                      tokens: int, scratch, act: torch.Tensor, y: torch.Tensor, pdl: bool = False) -> None:
+    """y rows = expert feed-forward of the expert-sorted rows ``xs``; ``tokens`` bounds the rows of one expert.
+    fp32 goes through ``scratch`` [rows, 2 n]."""
+    if not _f32(xs):
+        xgemm(xs, gate_up, offsets=offsets, out=act, swiglu=True, gate_limit=limit, pdl=pdl)
+        xgemm(act, down, offsets=offsets, out=y, pdl=pdl)
+        return
+    _sgemm_grouped(xs, gate_up.w, offsets, scratch, tokens, pdl)
+    gated_act(scratch, act, limit, pdl=pdl)
+    _sgemm_grouped(act, down.w, offsets, y, tokens, pdl)
+
+
+def combine_post_norm(y: torch.Tensor, r: Routing, w: torch.Tensor, eps: float, width: int, x: torch.Tensor,
+                      h: torch.Tensor, pdl: bool = False) -> None:
+    """x += RMSNorm(sum of weighted expert rows + identity weight * x) * w; h = x in the compute type."""
+    _lib.require_cuda_tensor(y, w, x, h)
+    t, ldx = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and h.shape == x.shape and h.dtype == y.dtype
+    rc = _lib.cuda().rmlx_moe_combine_post_norm(
+        y.data_ptr(), y.stride(0), r.row_of_pair.data_ptr(), r.weights.data_ptr(), r.identity.data_ptr(),
+        r.idx.shape[1], w.data_ptr(), eps, x.data_ptr(), h.data_ptr(), t, width, ldx, _f32(y), int(pdl),
+        _lib.stream_ptr())
+    _lib.check(rc, "moe_combine_post_norm")

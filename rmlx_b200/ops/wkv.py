@@ -1,0 +1,67 @@
+"""RWKV-style time mixing (csrc/kernels/wkv.cu): token shift, the WKV recurrence and the gated head norm.
+A sequence's state is its slot's row of a flat fp32 pool (``PagedKvCache.layer_state`` views)."""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from .. import _lib
+from .parallel_block import _f32
+
+SHIFT_PARTS = ("r", "k", "v", "g", "w")
+
+_lib.register_cuda_sigs({
+    "rmlx_wkv_max_dim": ("", "i"),
+    "rmlx_token_shift": ("pippqpipiiip", "i"),
+    "rmlx_wkv_scan": ("pppipippppi" "ppqpipi" "iiiip", "i"),
+    "rmlx_wkv_finish": ("pipipfpiiiiiip", "i"),
+})
+
+WKV_MAX_DIM = 256        # of the recurrence kernel
+
+
+def token_shift(x: torch.Tensor, mu: torch.Tensor, prev: torch.Tensor, slots: torch.Tensor, each_row: bool,
+                out: torch.Tensor, pdl: bool = False) -> None:
+    """out[s, t] = x[t] + (x[t - 1] - x[t]) * mu[s]; the row before a sequence's first row of the batch comes
+    from ``prev`` [slots, width] at the row's slot. ``each_row``: every row is another sequence."""
+    _lib.require_cuda_tensor(x, mu, prev, slots, out)
+    t, ldx = x.shape
+    assert x.dtype == mu.dtype == prev.dtype == torch.float32 and x.is_contiguous() and mu.is_contiguous()
+    assert mu.shape == (len(SHIFT_PARTS), ldx) and out.shape == (len(SHIFT_PARTS), t, ldx) and out.is_contiguous()
+    assert prev.shape[1] == ldx and prev.stride(1) == 1 and slots.dtype == torch.int32
+    rc = _lib.cuda().rmlx_token_shift(x.data_ptr(), ldx, mu.data_ptr(), prev.data_ptr(), prev.stride(0),
+                                      slots.data_ptr(), int(each_row), out.data_ptr(), t, _f32(out), int(pdl),
+                                      _lib.stream_ptr())
+    _lib.check(rc, "token_shift")
+
+
+def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, w0: torch.Tensor, u: torch.Tensor,
+             state: torch.Tensor, prev: torch.Tensor, x: torch.Tensor, out: torch.Tensor,
+             runs: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None, pdl: bool = False) -> None:
+    """Runs every sequence's new tokens through the recurrence on top of ``state`` [slots, H, d, d] and
+    leaves the new state (and in ``prev`` the last row of ``x``) behind. r, k, v [T, >= H d] in the compute type,
+    ``decay`` fp32 logits (w = exp(-exp(decay + w0))), out fp32. ``runs`` int32 [n, 4] (first row, rows, slot, -),
+    or ``slots``: every row its own sequence."""
+    _lib.require_cuda_tensor(r, k, v, decay, w0, u, state, prev, x, out, runs, slots)
+    _, h, d, _ = state.shape
+    assert r.stride(0) == k.stride(0) == v.stride(0) and r.dtype == k.dtype == v.dtype
+    assert decay.dtype == out.dtype == x.dtype == state.dtype == torch.float32 and state.stride()[1:] == (d * d, d, 1)
+    assert w0.numel() == u.numel() == h * d and state.stride(0) == prev.stride(0)
+    n = runs.shape[0] if runs is not None else slots.numel()
+    rc = _lib.cuda().rmlx_wkv_scan(
+        r.data_ptr(), k.data_ptr(), v.data_ptr(), r.stride(0), decay.data_ptr(), decay.stride(0), w0.data_ptr(),
+        u.data_ptr(), _lib.ptr(runs), _lib.ptr(slots), n, state.data_ptr(), prev.data_ptr(), state.stride(0),
+        x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), h, d, _f32(r), int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "wkv_scan")
+
+
+def wkv_finish(o: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor, eps: float, heads: int, dim: int,
+               out: torch.Tensor, pdl: bool = False) -> None:
+    """out = o / rms(o per head) * norm * silu(gate)."""
+    _lib.require_cuda_tensor(o, gate, norm, out)
+    assert o.dtype == norm.dtype == torch.float32 and gate.dtype == out.dtype and norm.numel() == heads * dim
+    rc = _lib.cuda().rmlx_wkv_finish(o.data_ptr(), o.stride(0), gate.data_ptr(), gate.stride(0), norm.data_ptr(), eps,
+                                     out.data_ptr(), out.stride(0), o.shape[0], heads, dim, _f32(out), int(pdl),
+                                     _lib.stream_ptr())
+    _lib.check(rc, "wkv_finish")

@@ -58,6 +58,8 @@ class ServingEngine:
         self.last_token: Dict[int, int] = {}
         self._ids = itertools.count()
         self._finished: Dict[int, int] = {}
+        if use_prefix_cache and self.cache.state is not None:
+            raise ValueError("a prefix cache keeps pages, not the state of recurrent layers: this model has such layers")
         prefix_cls = native.NativePrefixCache if self.native else PrefixCache
         self.prefix = prefix_cls(self.cache.block_size) if use_prefix_cache else None
         self._prompts: Dict[int, List[int]] = {}
