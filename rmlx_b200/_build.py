@@ -52,8 +52,8 @@ SETS = {
         "cuda": ("kernels/postnorm_rows.cu", "kernels/wkv.cu", "kernels/moe_route.cu",
                  "kernels/head_gemv.cu", "kernels/gemm_tcgen05.cu", "kernels/xgemm_tcgen05.cu",
                  "kernels/gemm_f32.cu", "kernels/flash_prefill_tc.cu", "kernels/flash_decode_scored.cu",
-                 "kernels/attention_any.cu", "kernels/mla_decode.cu", "kernels/parallel_rows.cu", "kernels/misc.cu",
-                 "runtime/graph_exec.cu"),
+                 "kernels/attention_any.cu", "kernels/mla_decode.cu", "kernels/parallel_rows.cu", "kernels/postnorm_gemv.cu",
+                 "kernels/parallel_gemv.cu", "kernels/misc.cu", "runtime/graph_exec.cu"),
         "host": ("host/serving.cpp", "host/sampler.cpp", "host/safetensors_io.cpp"),
     },
 }

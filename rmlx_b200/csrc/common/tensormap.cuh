@@ -52,4 +52,20 @@ inline int make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t inner,
                       row_stride_bytes, box_inner, box_outer);
 }
 
+// Three-dimensional bf16 map with the 128-byte swizzle: extents d0 (contiguous), d1, d2 in elements, byte
+// strides of d1 and d2 (multiples of 16).
+inline int make_tmap_3d_bf16(CUtensorMap* out, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t stride1,
+                             uint64_t stride2, uint32_t box0, uint32_t box1, uint32_t box2) {
+  EncodeTiledFn fn = encode_tiled_fn();
+  if (!fn) return -3;
+  cuuint64_t dims[3] = {d0, d1, d2};
+  cuuint64_t strides[2] = {stride1, stride2};
+  cuuint32_t box[3] = {box0, box1, box2};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -4;
+}
+
 }  // namespace rb

@@ -7,6 +7,10 @@
 // global memory: the tensor maps end at the real width and TMA fills the rest of a panel with zeros.
 // Ragged batches come as a table of query tiles ({first row, rows, position of the first row, row of
 // the block table}), so prompt portions of several sequences share one launch.
+// Latent attention (LAT): the keys and values of the batch's contexts are expanded from their latents
+// beforehand, [context rows, H, dim + vdim] in position order, and read through three-dimensional tensor
+// maps (a head's columns past its width read as zero); the rotated key part, shared by all heads, is the
+// last panel of a key row and comes straight from the latent cache's pages.
 //
 // Score modifiers run between S and the softmax, in base 2: t = P(s) - bias(i - j), where P is
 // softcap * tanh(s scale temp / softcap) as s times a polynomial in s^2 with the head's constants
@@ -89,6 +93,10 @@ struct TcParams {
   float scale_log2;
   ScoreMod mod;             // MOD instances
   HeadGate gate;            // MOD instances
+  // LAT instances: panels of the unrotated key part, where the rotated part starts in a query row and in
+  // a cache row, first context row of every tile's sequence
+  int kn, q_rot, c_rot;
+  const int* tile_ctx;
   int* status;
 };
 
@@ -131,11 +139,12 @@ __device__ __forceinline__ float max3_abs(float a, float b, float c) {
   return d;
 }
 
-template <int LANES, int KP, int VP, bool MOD>
+template <int LANES, int KP, int VP, bool MOD, bool LAT>
 __global__ void __launch_bounds__(TcCfg<LANES, KP, VP, MOD>::kThreads, 1)
 flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
                         const __grid_constant__ CUtensorMap tmap_k,
-                        const __grid_constant__ CUtensorMap tmap_v, TcParams p) {
+                        const __grid_constant__ CUtensorMap tmap_v,
+                        const __grid_constant__ CUtensorMap tmap_kr, TcParams p) {
   using C = TcCfg<LANES, KP, VP, MOD>;
   extern __shared__ __align__(1024) char smem[];
   if (smem_u32(smem) & 1023u) {       // the swizzled tiles need 1024-byte alignment
@@ -161,13 +170,14 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   const int kvh = h / (p.Hq / p.Hkv);
   // q0: the block's first query row; rows: how many rows from there on are its sequence's; pos_q0:
   // position of row q0; bt: the sequence's pages
-  int q0, rows, pos_q0;
+  int q0, rows, pos_q0, ctx0 = 0;
   const int* bt;
   if (p.tiles) {
     pdl_wait();      // the table may have been written by the launch before this one
     const int4 tile = p.tiles[int(blockIdx.x) / p.Hq];
     q0 = tile.x; rows = tile.y; pos_q0 = tile.z;
     bt = p.block_table + size_t(tile.w) * p.max_blocks;
+    if (LAT) ctx0 = p.tile_ctx[int(blockIdx.x) / p.Hq];
   } else {
     // long rows of work first: the last query tile walks the most keys
     q0 = (p.n_qt - 1 - int(blockIdx.x) / p.Hq) * (kTcRows * LANES);
@@ -235,7 +245,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
           if (n_steps[L] == 0) continue;
 #pragma unroll
           for (int c = 0; c < KP; ++c)
-            tma_load_2d(sQ + L * C::kQTile + c * kTcQPanel, &tmap_q, q_full, h * p.dk + c * 64, q0 + L * kTcRows);
+            tma_load_2d(sQ + L * C::kQTile + c * kTcQPanel, &tmap_q, q_full,
+                        h * p.dk + (LAT && c >= p.kn ? p.q_rot + (c - p.kn) * 64 : c * 64), q0 + L * kTcRows);
         }
       }
       for (int j = 0; j < n_max; ++j) {
@@ -247,26 +258,45 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         for (int pg = 0; pg < kTcPages; ++pg) {
           // pages past the last one this CTA can see repeat it (their keys are masked)
           const int page = min((j + j0) * kTcPages + pg, last_page);
-          y[pg] = (bt[page] * p.Hkv + kvh) * kTcPage;
+          y[pg] = (LAT ? bt[page] : bt[page] * p.Hkv + kvh) * kTcPage;
         }
         if (!mbar_wait(k_free + s, par, abort_flag)) break;
         mbar_arrive_expect_tx(k_full + s, C::kKTile);
         last_k[s] = j;
         char* kd = sK + s * C::kKTile;
+        if (LAT) {
 #pragma unroll
-        for (int pg = 0; pg < kTcPages; ++pg)
+          for (int c = 0; c < KP; ++c) {
+            if (c < p.kn) {
+              tma_load_3d(kd + c * kTcKvPanel, &tmap_k, k_full + s, c * 64, h, ctx0 + j * kTcKeys);
+            } else {
 #pragma unroll
-          for (int c = 0; c < KP; ++c)
-            tma_load_2d(kd + c * kTcKvPanel + pg * kTcPageBytes, &tmap_k, k_full + s, c * 64, y[pg]);
+              for (int pg = 0; pg < kTcPages; ++pg)
+                tma_load_2d(kd + c * kTcKvPanel + pg * kTcPageBytes, &tmap_kr, k_full + s, p.c_rot + (c - p.kn) * 64, y[pg]);
+            }
+          }
+        } else {
+#pragma unroll
+          for (int pg = 0; pg < kTcPages; ++pg)
+#pragma unroll
+            for (int c = 0; c < KP; ++c)
+              tma_load_2d(kd + c * kTcKvPanel + pg * kTcPageBytes, &tmap_k, k_full + s, c * 64, y[pg]);
+        }
         if (!mbar_wait(v_free + s, par, abort_flag)) break;
         mbar_arrive_expect_tx(v_full + s, C::kVTile);
         last_v[s] = j;
         char* vd = sV + s * C::kVTile;
-#pragma unroll
-        for (int pg = 0; pg < kTcPages; ++pg)
+        if (LAT) {
 #pragma unroll
           for (int c = 0; c < VP; ++c)
-            tma_load_2d(vd + c * kTcKvPanel + pg * kTcPageBytes, &tmap_v, v_full + s, c * 64, y[pg]);
+            tma_load_3d(vd + c * kTcKvPanel, &tmap_v, v_full + s, c * 64, h, ctx0 + j * kTcKeys);
+        } else {
+#pragma unroll
+          for (int pg = 0; pg < kTcPages; ++pg)
+#pragma unroll
+            for (int c = 0; c < VP; ++c)
+              tma_load_2d(vd + c * kTcKvPanel + pg * kTcPageBytes, &tmap_v, v_full + s, c * 64, y[pg]);
+        }
       }
       if (*abort_flag) {
         // leaving early: let the copies already in flight land before the CTA gives up its
@@ -586,15 +616,16 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   pdl_launch_dependents();
 }
 
-template <int LANES, int KP, int VP, bool MOD>
+template <int LANES, int KP, int VP, bool MOD, bool LAT = false>
 static int launch_prefill_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
-                             TcParams p, int pdl, cudaStream_t st) {
-  auto kern = flash_prefill_tc_kernel<LANES, KP, VP, MOD>;
+                             TcParams p, int pdl, cudaStream_t st, const CUtensorMap* tkr = nullptr) {
+  auto kern = flash_prefill_tc_kernel<LANES, KP, VP, MOD, LAT>;
   using C = TcCfg<LANES, KP, VP, MOD>;
   constexpr size_t smem = C::kSmem;
   RB_CHECK(set_max_smem(kern, smem));
   if (!p.tiles) p.n_qt = (p.T + kTcRows * LANES - 1) / (kTcRows * LANES);
-  return launch(kern, dim3(p.n_qt * p.Hq), dim3(C::kThreads), smem, st, pdl != 0, tq, tk, tv, p);
+  return launch(kern, dim3(p.n_qt * p.Hq), dim3(C::kThreads), smem, st, pdl != 0, tq, tk, tv,
+                tkr ? *tkr : tk, p);
 }
 
 static int prefill_tc_maps(CUtensorMap* tq, CUtensorMap* tk, CUtensorMap* tv, const void* q, const void* k_cache,
@@ -692,4 +723,51 @@ extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, con
   if (dv > 64) RB_FPS(1, 2);
   RB_FPS(1, 1);
 #undef RB_FPS
+}
+
+// 1 when the latent form takes these (eight-padded) widths: unrotated, rotated, value.
+extern "C" int rmlx_flash_prefill_latent_supported(int dim, int rot, int dv) {
+  return dim >= 8 && dim <= 128 && dim % 8 == 0 && rot >= 8 && rot <= 64 && rot % 8 == 0 && dv >= 8 && dv <= 128 && dv % 8 == 0;
+}
+
+// Latent attention over a ragged batch. q [T, H, dim + rot], out [T, H, dv]; kv [ctx_rows, H, dim + dv]: keys and
+// values of the contexts, tile i's sequence from row tile_ctx[i] (a multiple of 16) on; cache [num_blocks, 16,
+// ldc] with the rotated key part at column c_rot of a row; all bf16. tiles and block_table as above.
+extern "C" int rmlx_flash_prefill_latent(const void* q, const void* kv, const void* cache, const int* block_table,
+                                         int max_blocks, const int* tiles, const int* tile_ctx, int n_tiles, void* out,
+                                         int T, int H, int dim, int rot, int dv, int ctx_rows, int num_blocks, int ldc,
+                                         int c_rot, float scale, int lanes, int* status, int pdl, cudaStream_t st) {
+  if (T < 1 || H < 1 || (lanes != 1 && lanes != 2) || n_tiles < 1 || !tiles || !tile_ctx || ctx_rows < 1 || num_blocks < 1 ||
+      ldc % 8 || c_rot % 8 || c_rot + rot > ldc || !rmlx_flash_prefill_latent_supported(dim, rot, dv))
+    return -2;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(cache) |
+       reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(tiles)) & 15)
+    return -2;
+  const int dk = dim + rot, per = dim + dv;
+  CUtensorMap tq, tk, tv, tkr;
+  int rc = make_tmap_2d_bf16(&tq, q, uint64_t(H) * dk, uint64_t(T), uint64_t(H) * dk * 2, 64, kTcRows);
+  if (rc) return rc;
+  rc = make_tmap_3d_bf16(&tk, kv, dim, H, ctx_rows, uint64_t(per) * 2, uint64_t(H) * per * 2, 64, 1, kTcKeys);
+  if (rc) return rc;
+  rc = make_tmap_3d_bf16(&tv, static_cast<const __nv_bfloat16*>(kv) + dim, dv, H, ctx_rows, uint64_t(per) * 2,
+                         uint64_t(H) * per * 2, 64, 1, kTcKeys);
+  if (rc) return rc;
+  rc = make_tmap_2d_bf16(&tkr, cache, uint64_t(c_rot) + rot, uint64_t(num_blocks) * kTcPage, uint64_t(ldc) * 2, 64, kTcPage);
+  if (rc) return rc;
+  TcParams p{};
+  p.block_table = block_table; p.max_blocks = max_blocks;
+  p.tiles = reinterpret_cast<const int4*>(tiles); p.n_qt = n_tiles; p.tile_ctx = tile_ctx;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.T = T; p.Hq = H; p.Hkv = H; p.pos0 = 0;
+  p.dk = dk; p.dv = dv;
+  p.kn = dim > 64 ? 2 : 1; p.q_rot = dim; p.c_rot = c_rot;
+  p.scale_log2 = scale * kLog2e;
+  p.status = status;
+#define RB_FPL(KP_, VP_)                                                                          \
+  return lanes == 2 ? launch_prefill_tc<2, KP_, VP_, false, true>(tq, tk, tv, p, pdl, st, &tkr)   \
+                    : launch_prefill_tc<1, KP_, VP_, false, true>(tq, tk, tv, p, pdl, st, &tkr)
+  if (dim > 64) { if (dv > 64) RB_FPL(3, 2); RB_FPL(3, 1); }
+  if (dv > 64) RB_FPL(2, 2);
+  RB_FPL(2, 1);
+#undef RB_FPL
 }

@@ -59,6 +59,11 @@ struct MlaParams {
   const int* block_table;        // [slots, max_blocks]
   const int* seq_lens;           // [slots] tokens in the cache including the current one
   const int* slots;              // [B] cache slot of each query row (null: row b uses slot b)
+  // ragged batches: launch row b is row rows[b] of q and out (null: b), its token sits at positions[row] and
+  // its pages are row table_rows[row] of the block table (null: row); seq_lens and slots are then unused
+  const int* rows;
+  const int* positions;
+  const int* table_rows;
   __nv_bfloat16* out;            // [B, H, LAT]
   float* part_o;                 // [B, HT, S, 16, LAT]
   float* part_ml;                // [B, HT, S, 16, 2]
@@ -105,8 +110,9 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 4 ? 2 : 1) mla_decode_ker
   }
   pdl_launch_dependents();
   pdl_wait();
-  const int slot = p.slots ? p.slots[b] : b;
-  const int len = p.seq_lens[slot];
+  const int row_id = p.rows ? p.rows[b] : b;
+  const int slot = p.positions ? (p.table_rows ? p.table_rows[row_id] : row_id) : p.slots ? p.slots[b] : b;
+  const int len = p.positions ? p.positions[row_id] + 1 : p.seq_lens[slot];
   const int pg_total = (len + kMlaPage - 1) / kMlaPage;
   const int per = ((pg_total + p.S - 1) / p.S + kMlaStepPages - 1) / kMlaStepPages * kMlaStepPages;
   const int pg0 = split * per, pg1 = min(pg0 + per, pg_total);
@@ -138,7 +144,7 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 4 ? 2 : 1) mla_decode_ker
     const int r = idx / CH, c = idx - r * CH;
     const int h = ht * 16 + r;
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (h < p.H) v = *reinterpret_cast<const uint4*>(p.q + (size_t(b) * p.H + h) * W + c * 8);
+    if (h < p.H) v = *reinterpret_cast<const uint4*>(p.q + (size_t(row_id) * p.H + h) * W + c * 8);
     *reinterpret_cast<uint4*>(qs + r * ROW_PAD + c * 16) = v;
   }
   __syncthreads();              // the barriers are initialised, the queries staged
@@ -261,7 +267,7 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 4 ? 2 : 1) mla_decode_ker
       if (p.S == 1) {
         if (h < p.H) {
           const float inv = L > 0.f ? 1.f / L : 0.f;
-          *reinterpret_cast<uint32_t*>(p.out + (size_t(b) * p.H + h) * LAT + d) = pack_bf16(v0 * inv, v1 * inv);
+          *reinterpret_cast<uint32_t*>(p.out + (size_t(row_id) * p.H + h) * LAT + d) = pack_bf16(v0 * inv, v1 * inv);
         }
       } else {
         *reinterpret_cast<float2*>(p.part_o + (tile * 16 + row) * LAT + d) = make_float2(v0, v1);
@@ -284,6 +290,7 @@ __global__ void __launch_bounds__(256) mla_merge_kernel(MlaParams p) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t tile0 = (size_t(b) * p.HT + ht) * p.S;
+  const int row_id = p.rows ? p.rows[b] : b;
   {
     const int row = threadIdx.x >> 4, ls = threadIdx.x & 15;
     float ms[4], lsum[4], M = -INFINITY;
@@ -329,7 +336,7 @@ __global__ void __launch_bounds__(256) mla_merge_kernel(MlaParams p) {
       const float w = wgt[s * 16 + row];
       a0 = fmaf(v.x, w, a0); a1 = fmaf(v.y, w, a1);
     }
-    *reinterpret_cast<uint32_t*>(p.out + (size_t(b) * p.H + h) * LAT + d) = pack_bf16(a0, a1);
+    *reinterpret_cast<uint32_t*>(p.out + (size_t(row_id) * p.H + h) * LAT + d) = pack_bf16(a0, a1);
   }
 }
 
@@ -355,10 +362,12 @@ extern "C" int rmlx_mla_status() {
 
 // q [B, H, LAT + ROPE] bf16 (absorbed), cache [blocks, 16, row_elems = LAT + ROPE + 8] bf16 (the
 // last 8 values of a row are padding), out [B, H, LAT] bf16.
-// block_table / seq_lens are the cache's own tables, indexed by slots[b] (by b when slots is null).
+// block_table / seq_lens are the cache's own tables, indexed by slots[b] (by b when slots is null);
+// with `positions` (and optionally rows, table_rows) the launch rows are rows of a ragged batch instead.
 // (LAT, ROPE) in {(512, 64), (128, 64)}; splits in [1, 64]; part_* needed when splits > 1.
 extern "C" int rmlx_mla_decode_paged(const void* q, const void* cache, const int* block_table,
-                                     const int* seq_lens, const int* slots, void* out, float* part_o, float* part_ml,
+                                     const int* seq_lens, const int* slots, const int* rows, const int* positions,
+                                     const int* table_rows, void* out, float* part_o, float* part_ml,
                                      int B, int H, int LAT, int ROPE, int row_elems, int max_blocks,
                                      int splits, float scale, int pdl, cudaStream_t st) {
   if (B < 1 || H < 1 || splits < 1 || splits > 64) return -2;
@@ -368,6 +377,7 @@ extern "C" int rmlx_mla_decode_paged(const void* q, const void* cache, const int
   p.q = static_cast<const __nv_bfloat16*>(q);
   p.cache = static_cast<const __nv_bfloat16*>(cache);
   p.block_table = block_table; p.seq_lens = seq_lens; p.slots = slots;
+  p.rows = rows; p.positions = positions; p.table_rows = table_rows;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.part_o = part_o; p.part_ml = part_ml;
   p.max_blocks = max_blocks; p.H = H; p.HT = (H + 15) / 16; p.S = splits;

@@ -1,0 +1,577 @@
+// Decode projections of decoders with norms on the sublayers' outputs (x <- x + norm(y), fp32 residual),
+// one warp per weight-row pair as in decode_gemv.cu. The kernels that read the residual take the previous
+// sublayer's output y along and finish that sublayer first: every block forms x + norm(y) while it stages
+// its activations (a few thousand values from L2), and block 0 writes it to a second residual buffer.
+//
+//   postnorm_in       out = W x: fp32 rows, or (gated) the activation of row pairs (i, n + i) in bf16, or
+//                     (shift) row segments that each read their own token-shift mix of x
+//   postnorm_router   router logits, softmax, corrected top-k (the last block to finish chooses)
+//   postnorm_expert   gate / up projections of each token's chosen experts with the gated activation
+//   expert_out        y = sum over slots of weight * Wdown[e] act + identity weight * x
+//   matvec_out        y = W a
+//   wkv_decode        one token of the WKV recurrence: decay from its low-rank projection, state update,
+//                     head norm, output gate
+#include "../common/gated.cuh"
+#include "../common/gemv_core.cuh"
+#include "../common/launch.cuh"
+#include "../common/route.cuh"
+
+namespace rb {
+
+constexpr int kPnRows = 2;        // weight rows a warp accumulates together
+constexpr size_t kPnMaxSmem = 220 * 1024;
+
+// The residual a kernel reads: x + y / rms(y) * w (y == nullptr: x itself), D real columns of ldx.
+struct PostNormIn {
+  const float* x;
+  const float* y;
+  const float* w;
+  float eps;
+  int D, ldx;
+  float* x_out;                   // written by block 0; not x itself
+};
+// Token shift: rows seg * seg_rows .. of W read x + (prev - x) * mu[seg].
+struct ShiftIn {
+  const float* mu;                // [5, ldx]
+  const float* prev;              // slot s: prev + s * stride
+  const int* slots;
+  long long stride;
+  int seg_rows;                   // rows of the first four segments; the rest is the fifth
+};
+
+// Stages row b of the residual into `xs` (split-chunk layout of gemv_core.cuh). 256 threads.
+__device__ __forceinline__ void stage_post_norm(const PostNormIn& in, int b, char* xs, float* red, bool write,
+                                                const float* mu, const float* prev) {
+  constexpr int kKeep = 4;
+  const int chunks = in.ldx >> 3;
+  const float* x = in.x + size_t(b) * in.ldx;
+  const float* y = in.y ? in.y + size_t(b) * in.ldx : nullptr;
+  float4* dst = reinterpret_cast<float4*>(xs);
+  auto ld = [](const float* p, int c, float (&f)[8]) {
+    const float4 a = __ldcg(reinterpret_cast<const float4*>(p + c * 8));
+    const float4 e = __ldcg(reinterpret_cast<const float4*>(p + c * 8 + 4));
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = e.x; f[5] = e.y; f[6] = e.z; f[7] = e.w;
+  };
+  float fy[kKeep][8], fx[kKeep][8];
+  float ssq = 0.f;
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int c = u * kGemvThreads + threadIdx.x;
+    if (c < chunks) {
+      ld(x, c, fx[u]);
+      if (y) {
+        ld(y, c, fy[u]);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) ssq += fy[u][i] * fy[u][i];
+      }
+    }
+  }
+  float inv = 0.f;
+  if (y) {
+    for (int c = kKeep * kGemvThreads + threadIdx.x; c < chunks; c += kGemvThreads) {
+      float f[8];
+      ld(y, c, f);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ssq += f[i] * f[i];
+    }
+    inv = 1.f / sqrtf(block_sum_256(ssq, red) / float(in.D) + in.eps);
+  }
+  auto put = [&](int c, float (&a)[8], const float (&e)[8]) {
+    if (y) {
+      float g[8];
+      ld(in.w, c, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) a[i] = fmaf(e[i] * inv, g[i], a[i]);
+    }
+    if (write) {
+      float4* o = reinterpret_cast<float4*>(in.x_out + size_t(b) * in.ldx + c * 8);
+      o[0] = make_float4(a[0], a[1], a[2], a[3]);
+      o[1] = make_float4(a[4], a[5], a[6], a[7]);
+    }
+    if (mu) {
+      float m[8], p[8];
+      ld(mu, c, m);
+      ld(prev, c, p);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) a[i] = fmaf(p[i] - a[i], m[i], a[i]);
+    }
+    dst[c] = make_float4(a[0], a[1], a[2], a[3]);
+    dst[chunks + c] = make_float4(a[4], a[5], a[6], a[7]);
+  };
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int c = u * kGemvThreads + threadIdx.x;
+    if (c < chunks) put(c, fx[u], fy[u]);
+  }
+  for (int c = kKeep * kGemvThreads + threadIdx.x; c < chunks; c += kGemvThreads) {
+    float a[8], e[8];
+    ld(x, c, a);
+    if (y) ld(y, c, e);
+    put(c, a, e);
+  }
+}
+
+// GATED: N counts output columns, W has 2 N rows (gate then up). One tile of rows per warp: the grid
+// covers N (a block's rows then belong to one shift segment).
+template <int B, bool GATED>
+__global__ void __launch_bounds__(kGemvThreads)
+postnorm_in_kernel(Matrix<WBf16> W, PostNormIn in, ShiftIn sh, float* __restrict__ out, int ld_out,
+                   __nv_bfloat16* __restrict__ act, int ld_act, int N, float limit) {
+  extern __shared__ __align__(16) char smem[];
+  __shared__ float red[kGemvWarps];
+  constexpr int R = GATED ? 2 * kPnRows : kPnRows;
+  const int K = W.K, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const size_t bstride = XStage<WBf16>::bytes(K);
+  const int n0 = (blockIdx.x * kGemvWarps + warp) * kPnRows;
+  RowBf16 rows[R];
+  Tile<RowBf16, R> t0;
+  if (n0 < N) {                 // weights wait for nothing: ask for the first tile at once
+#pragma unroll
+    for (int r = 0; r < kPnRows; ++r) {
+      const int n = min(n0 + r, N - 1);
+      rows[r] = W.row(n);
+      if (GATED) rows[kPnRows + r] = W.row(size_t(N) + n);
+    }
+    load_tile<R>(rows, K, 0, t0);
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* mu = nullptr;
+  if (sh.mu) mu = sh.mu + size_t(min(blockIdx.x * kGemvWarps * kPnRows / sh.seg_rows, 4)) * in.ldx;
+#pragma unroll
+  for (int b = 0; b < B; ++b)
+    stage_post_norm(in, b, smem + b * bstride, red, blockIdx.x == 0, mu, mu ? sh.prev + sh.slots[b] * sh.stride : nullptr);
+  __syncthreads();
+  if (n0 >= N) return;
+  float acc[R][B];
+#pragma unroll
+  for (int r = 0; r < R; ++r)
+#pragma unroll
+    for (int b = 0; b < B; ++b) acc[r][b] = 0.f;
+  warp_dot<R, B, RowBf16>(rows, smem, bstride, K, acc, t0);
+#pragma unroll
+  for (int r = 0; r < kPnRows; ++r)
+#pragma unroll
+    for (int b = 0; b < B; ++b) {
+      const float v = warp_sum(acc[r][b]);
+      const float u = GATED ? warp_sum(acc[GATED ? kPnRows + r : r][b]) : 0.f;
+      const int n = n0 + r;
+      if (lane == r * B + b && n < N) {
+        if (GATED) act[size_t(b) * ld_act + n] = __float2bfloat16_rn(gated_act_fast(v, u, limit));
+        else out[size_t(b) * ld_out + n] = v;
+      }
+    }
+}
+
+// One warp per router output; the last block to arrive chooses for every token.
+template <int B>
+__global__ void __launch_bounds__(kGemvThreads)
+postnorm_router_kernel(Matrix<WBf16> W, PostNormIn in, const float* __restrict__ correction, float* __restrict__ logits,
+                       int* __restrict__ idx, float* __restrict__ weights, float* __restrict__ identity,
+                       unsigned int* __restrict__ ticket, int experts, int outputs, int top_k) {
+  extern __shared__ __align__(16) char smem[];
+  __shared__ float red[kGemvWarps];
+  __shared__ unsigned int last;
+  const int K = W.K, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const size_t bstride = XStage<WBf16>::bytes(K);
+  const int n = blockIdx.x * kGemvWarps + warp;
+  RowBf16 rows[1] = {W.row(min(n, outputs - 1))};
+  Tile<RowBf16, 1> t0;
+  load_tile<1>(rows, K, 0, t0);
+  pdl_launch_dependents();
+  pdl_wait();
+#pragma unroll
+  for (int b = 0; b < B; ++b) stage_post_norm(in, b, smem + b * bstride, red, blockIdx.x == 0, nullptr, nullptr);
+  __syncthreads();
+  float acc[1][B];
+#pragma unroll
+  for (int b = 0; b < B; ++b) acc[0][b] = 0.f;
+  warp_dot<1, B, RowBf16>(rows, smem, bstride, K, acc, t0);
+#pragma unroll
+  for (int b = 0; b < B; ++b) {
+    const float v = warp_sum(acc[0][b]);
+    if (lane == 0 && n < outputs) logits[size_t(b) * outputs + n] = v;
+  }
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) last = (atomicAdd(ticket, 1u) == gridDim.x - 1) ? 1u : 0u;
+  __syncthreads();
+  if (last) {
+    __threadfence();
+    for (int b = warp; b < B; b += kGemvWarps) {
+      // through L2: other blocks wrote the logits
+      float* row = reinterpret_cast<float*>(smem) + b * outputs;
+      for (int i = lane; i < outputs; i += 32) row[i] = __ldcg(logits + size_t(b) * outputs + i);
+      __syncwarp();
+      warp_route_corrected(row, correction, experts, outputs, top_k, idx + size_t(b) * top_k, weights + size_t(b) * top_k,
+                           identity + b, nullptr);
+    }
+    if (threadIdx.x == 0) *ticket = 0u;
+  }
+}
+
+// grid (column blocks, token * slot). x: the finished residual.
+__global__ void __launch_bounds__(kGemvThreads, 2)
+postnorm_expert_kernel(const __nv_bfloat16* __restrict__ w, int K, const float* __restrict__ x, int ldx,
+                       const int* __restrict__ idx, __nv_bfloat16* __restrict__ act, int ld_act, int N, int top_k,
+                       int experts, float limit) {
+  extern __shared__ __align__(16) char smem[];
+  constexpr int R = 2 * kPnRows;
+  const int pair = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int e = idx[pair];
+  if (e >= experts) return;                           // an identity expert has no tensors
+  Matrix<WBf16> W{w + size_t(e) * 2 * N * K, K};
+  const int n0 = (blockIdx.x * kGemvWarps + warp) * kPnRows;
+  RowBf16 rows[R];
+  Tile<RowBf16, R> t0;
+  if (n0 < N) {
+#pragma unroll
+    for (int r = 0; r < kPnRows; ++r) {
+      const int n = min(n0 + r, N - 1);
+      rows[r] = W.row(n);
+      rows[kPnRows + r] = W.row(size_t(N) + n);
+    }
+    load_tile<R>(rows, K, 0, t0);
+  }
+  const float* src = x + size_t(pair / top_k) * ldx;
+  auto ld = [&](int c, float (&f)[8]) {
+    const float4 a = __ldcg(reinterpret_cast<const float4*>(src + c * 8));
+    const float4 b = __ldcg(reinterpret_cast<const float4*>(src + c * 8 + 4));
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  };
+  XStage<WBf16>::stage_with(smem, K, ld);
+  if (n0 >= N) return;
+  float acc[R][1];
+#pragma unroll
+  for (int r = 0; r < R; ++r) acc[r][0] = 0.f;
+  warp_dot<R, 1, RowBf16>(rows, smem, 0, K, acc, t0);
+#pragma unroll
+  for (int r = 0; r < kPnRows; ++r) {
+    const float g = warp_sum(acc[r][0]), u = warp_sum(acc[kPnRows + r][0]);
+    if (lane == r && n0 + r < N) act[size_t(pair) * ld_act + n0 + r] = __float2bfloat16_rn(gated_act_fast(g, u, limit));
+  }
+}
+
+// grid (row blocks, tokens): y[b, n] = sum_s weight_s * (Wdown[e_s] act_s)[n] + identity * x[b, n], n < N.
+__global__ void __launch_bounds__(kGemvThreads, 2)
+expert_out_kernel(const __nv_bfloat16* __restrict__ w, int rows_e, int K, const __nv_bfloat16* __restrict__ act, int ld_act,
+                  const int* __restrict__ idx, const float* __restrict__ weights, const float* __restrict__ identity,
+                  const float* __restrict__ x, float* __restrict__ y, int ldx, int N, int top_k, int experts) {
+  extern __shared__ __align__(16) char smem[];        // [top_k] staged activations
+  __shared__ int s_e[kRouteMaxTop];
+  __shared__ float s_w[kRouteMaxTop];
+  const int b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const size_t bstride = XStage<WBf16>::bytes(K);
+  pdl_launch_dependents();
+  pdl_wait();
+  if (threadIdx.x < top_k) {
+    const int e = idx[b * top_k + threadIdx.x];
+    s_e[threadIdx.x] = e < experts ? e : -1;
+    s_w[threadIdx.x] = weights[b * top_k + threadIdx.x];
+  }
+  __syncthreads();
+  auto next = [&](int s) { while (s < top_k && s_e[s] < 0) ++s; return s; };
+  const int n0 = (blockIdx.x * kGemvWarps + warp) * kPnRows;
+  int s = next(0);
+  RowBf16 rows[kPnRows];
+  Tile<RowBf16, kPnRows> cur;
+  auto point = [&](int slot, RowBf16 (&r)[kPnRows]) {
+#pragma unroll
+    for (int i = 0; i < kPnRows; ++i) r[i] = RowBf16{w + (size_t(s_e[slot]) * rows_e + min(n0 + i, N - 1)) * K};
+  };
+  if (n0 < N && s < top_k) { point(s, rows); load_tile<kPnRows>(rows, K, 0, cur); }
+  for (int q = 0; q < top_k; ++q) {
+    if (s_e[q] < 0) continue;
+    XLoadBf16 ld{act + size_t(b * top_k + q) * ld_act, nullptr, 0.f};
+    XStage<WBf16>::stage_part(smem + q * bstride, K, ld, threadIdx.x, kGemvThreads);
+  }
+  __syncthreads();
+  if (n0 >= N) return;
+  float tot[kPnRows];
+#pragma unroll
+  for (int r = 0; r < kPnRows; ++r) tot[r] = 0.f;
+  while (s < top_k) {                                  // the next expert's first tile is asked for early
+    const int sn = next(s + 1);
+    RowBf16 rn[kPnRows];
+    Tile<RowBf16, kPnRows> nxt;
+    if (sn < top_k) { point(sn, rn); load_tile<kPnRows>(rn, K, 0, nxt); }
+    float acc[kPnRows][1];
+#pragma unroll
+    for (int r = 0; r < kPnRows; ++r) acc[r][0] = 0.f;
+    warp_dot<kPnRows, 1, RowBf16>(rows, smem + s * bstride, 0, K, acc, cur);
+#pragma unroll
+    for (int r = 0; r < kPnRows; ++r) tot[r] = fmaf(s_w[s], acc[r][0], tot[r]);
+    if (sn < top_k) {
+      cur = nxt;
+#pragma unroll
+      for (int r = 0; r < kPnRows; ++r) rows[r] = rn[r];
+    }
+    s = sn;
+  }
+#pragma unroll
+  for (int r = 0; r < kPnRows; ++r) {
+    const float v = warp_sum(tot[r]);
+    const int n = n0 + r;
+    if (lane == r && n < N) y[size_t(b) * ldx + n] = fmaf(identity[b], __ldcg(x + size_t(b) * ldx + n), v);
+  }
+}
+
+template <int B>
+__global__ void __launch_bounds__(kGemvThreads)
+matvec_out_kernel(Matrix<WBf16> W, const __nv_bfloat16* __restrict__ a, int ld_a, float* __restrict__ y, int ld_y, int N) {
+  extern __shared__ __align__(16) char smem[];
+  const int K = W.K, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const size_t bstride = XStage<WBf16>::bytes(K);
+  const int n0 = (blockIdx.x * kGemvWarps + warp) * kPnRows;
+  RowBf16 rows[kPnRows];
+  Tile<RowBf16, kPnRows> t0;
+  if (n0 < N) {
+#pragma unroll
+    for (int r = 0; r < kPnRows; ++r) rows[r] = W.row(min(n0 + r, N - 1));
+    load_tile<kPnRows>(rows, K, 0, t0);
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+#pragma unroll
+  for (int b = 0; b < B; ++b) {
+    XLoadBf16 ld{a + size_t(b) * ld_a, nullptr, 0.f};
+    XStage<WBf16>::stage_part(smem + b * bstride, K, ld, threadIdx.x, kGemvThreads);
+  }
+  __syncthreads();
+  if (n0 >= N) return;
+  float acc[kPnRows][B];
+#pragma unroll
+  for (int r = 0; r < kPnRows; ++r)
+#pragma unroll
+    for (int b = 0; b < B; ++b) acc[r][b] = 0.f;
+  warp_dot<kPnRows, B, RowBf16>(rows, smem, bstride, K, acc, t0);
+#pragma unroll
+  for (int r = 0; r < kPnRows; ++r)
+#pragma unroll
+    for (int b = 0; b < B; ++b) {
+      const float v = warp_sum(acc[r][b]);
+      if (lane == r * B + b && n0 + r < N) y[size_t(b) * ld_y + n0 + r] = v;
+    }
+}
+
+// raw row b = [r | k | v | g: `inner` values apart | low: rank]. One block per (head, row).
+__global__ void __launch_bounds__(256)
+wkv_decode_kernel(const float* __restrict__ raw, int ld_raw, int inner, const __nv_bfloat16* __restrict__ w2, int rank,
+                  const float* __restrict__ w0, const float* __restrict__ u, const float* __restrict__ norm, float eps,
+                  const int* __restrict__ slots, float* __restrict__ state, float* __restrict__ prev, long long stride,
+                  const float* __restrict__ x, int ldx, __nv_bfloat16* __restrict__ a, int ld_a, int dim, int dim_pad) {
+  extern __shared__ float sm[];
+  float* sr = sm;                    // [dim] r, k, decay
+  float* sk = sr + dim;
+  float* sw = sk + dim;
+  float* low = sw + dim;             // [rank] tanh
+  float* part = low + rank;          // [256 / dim_pad][dim_pad]
+  __shared__ float red[8];
+  pdl_launch_dependents();
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
+  pdl_wait();
+  const float* row = raw + size_t(b) * ld_raw;
+  const int slot = slots[b];
+  // the column this thread works on and its group's share of the rows
+  const int groups = 256 / dim_pad, g = tid / dim_pad, col = tid - g * dim_pad;
+  const int per = (dim + groups - 1) / groups, i0 = g * per, i1 = min(i0 + per, dim);
+  for (int i = tid; i < rank; i += 256) low[i] = tanhf(__ldcg(row + 4 * inner + i));
+  float ruk = 0.f;
+  for (int i = tid; i < dim; i += 256) {
+    const float r = __ldcg(row + h * dim + i), k = __ldcg(row + inner + h * dim + i);
+    sr[i] = r;
+    sk[i] = k;
+    ruk = fmaf(r * u[h * dim + i], k, ruk);
+  }
+  ruk = block_sum_256(ruk, red);     // low, sr and sk are visible, too
+  for (int i = tid; i < dim; i += 256) {
+    const __nv_bfloat16* wr = w2 + size_t(h * dim + i) * rank;
+    float d = w0[h * dim + i];
+    for (int j = 0; j < rank; j += 8) {
+      const uint4 q = *reinterpret_cast<const uint4*>(wr + j);
+      d = fmaf(bf16lo(q.x), low[j], d); d = fmaf(bf16hi(q.x), low[j + 1], d);
+      d = fmaf(bf16lo(q.y), low[j + 2], d); d = fmaf(bf16hi(q.y), low[j + 3], d);
+      d = fmaf(bf16lo(q.z), low[j + 4], d); d = fmaf(bf16hi(q.z), low[j + 5], d);
+      d = fmaf(bf16lo(q.w), low[j + 6], d); d = fmaf(bf16hi(q.w), low[j + 7], d);
+    }
+    sw[i] = expf(-expf(d));
+  }
+  __syncthreads();
+  const float v = col < dim ? __ldcg(row + 2 * inner + h * dim + col) : 0.f;
+  float o = 0.f;
+  if (col < dim && g < groups) {
+    float* sp = state + size_t(slot) * stride + size_t(h) * dim * dim + col;
+#pragma unroll 8
+    for (int i = i0; i < i1; ++i) {
+      const float s = sp[size_t(i) * dim];
+      o = fmaf(sr[i], s, o);
+      sp[size_t(i) * dim] = fmaf(sw[i], s, sk[i] * v);
+    }
+  }
+  if (g < groups) part[g * dim_pad + col] = o;
+  __syncthreads();
+  float ssq = 0.f;
+  if (tid < dim) {
+    o = ruk * v;
+    for (int q = 0; q < groups; ++q) o += part[q * dim_pad + tid];
+    ssq = o * o;
+  }
+  ssq = block_sum_256(ssq, red);
+  if (tid < dim) {
+    const float inv = 1.f / sqrtf(ssq / float(dim) + eps);
+    const float z = __ldcg(row + 3 * inner + h * dim + tid);
+    a[size_t(b) * ld_a + h * dim + tid] = __float2bfloat16_rn(o * inv * norm[h * dim + tid] * (z / (1.f + expf(-z))));
+  }
+  if (h == 0) {
+    float* keep = prev + size_t(slot) * stride;
+    for (int i = tid; i < ldx; i += 256) keep[i] = __ldcg(x + size_t(b) * ldx + i);
+  }
+}
+
+static int pn_grid(int rows) { return (rows + kGemvWarps * kPnRows - 1) / (kGemvWarps * kPnRows); }
+
+}  // namespace rb
+
+using namespace rb;
+
+// Rows one launch takes for K staged values: at most four, fewer when the fp32 staging would not fit.
+extern "C" int rmlx_postnorm_max_rows(int K) {
+  int b = 4;
+  while (b > 0 && size_t(K) * 4 * b > kPnMaxSmem) --b;
+  return b;
+}
+
+#define RB_PN_DISPATCH(B_, CALL)                     \
+  switch (B_) {                                      \
+    case 1: { constexpr int kB = 1; return CALL; }   \
+    case 2: { constexpr int kB = 2; return CALL; }   \
+    case 3: { constexpr int kB = 3; return CALL; }   \
+    case 4: { constexpr int kB = 4; return CALL; }   \
+    default: return -2;                              \
+  }
+
+template <int B, bool GATED>
+static int launch_in(const void* w, const PostNormIn& in, const ShiftIn& sh, float* out, int ld_out, void* act, int ld_act,
+                     int N, float limit, int pdl, cudaStream_t st) {
+  const size_t smem = XStage<WBf16>::bytes(in.ldx) * B;
+  auto kern = postnorm_in_kernel<B, GATED>;
+  RB_CHECK(set_max_smem(kern, smem));
+  return launch(kern, dim3(pn_grid(N)), dim3(kGemvThreads), smem, st, pdl != 0,
+                Matrix<WBf16>{static_cast<const __nv_bfloat16*>(w), in.ldx}, in, sh, out, ld_out,
+                static_cast<__nv_bfloat16*>(act), ld_act, N, limit);
+}
+
+// w bf16 [N, ldx]; x, y (or null) and x_out fp32 [B, ldx], norm_w fp32 [ldx]; out fp32 [B, ld_out]. mu (or
+// null): fp32 [5, ldx], prev rows `stride` apart by slots [B]; then w's rows are four segments of seg_rows (a
+// multiple of 16) and a fifth.
+extern "C" int rmlx_postnorm_in(const void* w, const float* x, const float* y, const float* norm_w, float eps, float* x_out,
+                                int D, int ldx, const float* mu, const float* prev, const int* slots, long long stride,
+                                int seg_rows, float* out, int ld_out, int B, int N, int pdl, cudaStream_t st) {
+  if (ldx < 8 || ldx % 8 || D < 1 || D > ldx || N < 1 || ld_out < N || !x_out || x_out == x || B > rmlx_postnorm_max_rows(ldx) ||
+      (y && !norm_w) || (mu && (!prev || !slots || stride % 4 || seg_rows < 16 || seg_rows % 16)))
+    return -2;
+  const PostNormIn in{x, y, norm_w, eps, D, ldx, x_out};
+  const ShiftIn sh{mu, prev, slots, stride, mu ? seg_rows : 1};
+  RB_PN_DISPATCH(B, (launch_in<kB, false>(w, in, sh, out, ld_out, nullptr, 0, N, 0.f, pdl, st)))
+}
+
+// w bf16 [2 N, ldx] = [gate; up]; act bf16 [B, ld_act].
+extern "C" int rmlx_postnorm_gated(const void* w, const float* x, const float* y, const float* norm_w, float eps,
+                                   float* x_out, int D, int ldx, void* act, int ld_act, int B, int N, float limit, int pdl,
+                                   cudaStream_t st) {
+  if (ldx < 8 || ldx % 8 || D < 1 || D > ldx || N < 1 || ld_act < N || !x_out || x_out == x || B > rmlx_postnorm_max_rows(ldx) ||
+      (y && !norm_w))
+    return -2;
+  const PostNormIn in{x, y, norm_w, eps, D, ldx, x_out};
+  const ShiftIn sh{nullptr, nullptr, nullptr, 0, 1};
+  RB_PN_DISPATCH(B, (launch_in<kB, true>(w, in, sh, nullptr, 0, act, ld_act, N, limit, pdl, st)))
+}
+
+template <int B>
+static int launch_router(const void* w, const PostNormIn& in, const float* correction, float* logits, int* idx,
+                         float* weights, float* identity, unsigned int* ticket, int experts, int outputs, int top_k, int pdl,
+                         cudaStream_t st) {
+  size_t smem = XStage<WBf16>::bytes(in.ldx) * B;
+  if (smem < size_t(B) * outputs * 4) smem = size_t(B) * outputs * 4;
+  auto kern = postnorm_router_kernel<B>;
+  RB_CHECK(set_max_smem(kern, smem));
+  return launch(kern, dim3((outputs + kGemvWarps - 1) / kGemvWarps), dim3(kGemvThreads), smem, st, pdl != 0,
+                Matrix<WBf16>{static_cast<const __nv_bfloat16*>(w), in.ldx}, in, correction, logits, idx, weights, identity,
+                ticket, experts, outputs, top_k);
+}
+
+// w bf16 [outputs, ldx]; logits fp32 [B, outputs] scratch; ticket: one word, zero on entry and on exit.
+extern "C" int rmlx_postnorm_router(const void* w, const float* x, const float* y, const float* norm_w, float eps,
+                                    float* x_out, int D, int ldx, const float* correction, float* logits, int* idx,
+                                    float* weights, float* identity, unsigned int* ticket, int B, int experts, int outputs,
+                                    int top_k, int pdl, cudaStream_t st) {
+  if (ldx < 8 || ldx % 8 || D < 1 || D > ldx || !x_out || x_out == x || (y && !norm_w) || experts < 1 || outputs < experts ||
+      outputs > kRouteMaxOutputs || top_k < 1 || top_k > kRouteMaxTop || top_k > outputs || B > rmlx_postnorm_max_rows(ldx))
+    return -2;
+  const PostNormIn in{x, y, norm_w, eps, D, ldx, x_out};
+  RB_PN_DISPATCH(B, (launch_router<kB>(w, in, correction, logits, idx, weights, identity, ticket, experts, outputs, top_k,
+                                       pdl, st)))
+}
+
+// w bf16 [experts, 2 N, ldx]; x fp32 [B, ldx]; idx [B, top_k]; act bf16 [B * top_k, ld_act].
+extern "C" int rmlx_postnorm_expert(const void* w, const float* x, int ldx, const int* idx, void* act, int ld_act, int B,
+                                    int top_k, int N, int experts, float limit, int pdl, cudaStream_t st) {
+  if (B < 1 || top_k < 1 || B * top_k > 65535 || ldx < 8 || ldx % 8 || N < 1 || ld_act < N || experts < 1 ||
+      XStage<WBf16>::bytes(ldx) > kPnMaxSmem)
+    return -2;
+  const size_t smem = XStage<WBf16>::bytes(ldx);
+  RB_CHECK(set_max_smem(postnorm_expert_kernel, smem));
+  return launch(postnorm_expert_kernel, dim3(pn_grid(N), B * top_k), dim3(kGemvThreads), smem, st, pdl != 0,
+                static_cast<const __nv_bfloat16*>(w), ldx, x, ldx, idx, static_cast<__nv_bfloat16*>(act), ld_act, N, top_k,
+                experts, limit);
+}
+
+// w bf16 [experts, rows_e, K], N <= rows_e; act bf16 [B * top_k, ld_act >= K]; x, y fp32 [B, ldx].
+extern "C" int rmlx_expert_out(const void* w, int rows_e, int K, const void* act, int ld_act, const int* idx,
+                               const float* weights, const float* identity, const float* x, float* y, int ldx, int B, int N,
+                               int top_k, int experts, int pdl, cudaStream_t st) {
+  if (B < 1 || B > 65535 || top_k < 1 || top_k > kRouteMaxTop || K < 8 || K % 8 || ld_act % 8 || ld_act < K || N < 1 ||
+      N > rows_e || N > ldx || XStage<WBf16>::bytes(K) * top_k > kPnMaxSmem)
+    return -2;
+  const size_t smem = XStage<WBf16>::bytes(K) * top_k;
+  RB_CHECK(set_max_smem(expert_out_kernel, smem));
+  return launch(expert_out_kernel, dim3(pn_grid(N), B), dim3(kGemvThreads), smem, st, pdl != 0,
+                static_cast<const __nv_bfloat16*>(w), rows_e, K, static_cast<const __nv_bfloat16*>(act), ld_act, idx, weights,
+                identity, x, y, ldx, N, top_k, experts);
+}
+
+template <int B>
+static int launch_matvec(const void* w, const void* a, int ld_a, float* y, int ld_y, int N, int K, int pdl, cudaStream_t st) {
+  const size_t smem = XStage<WBf16>::bytes(K) * B;
+  auto kern = matvec_out_kernel<B>;
+  RB_CHECK(set_max_smem(kern, smem));
+  return launch(kern, dim3(pn_grid(N)), dim3(kGemvThreads), smem, st, pdl != 0,
+                Matrix<WBf16>{static_cast<const __nv_bfloat16*>(w), K}, static_cast<const __nv_bfloat16*>(a), ld_a, y, ld_y, N);
+}
+
+// w bf16 [N, K], a bf16 [B, ld_a], y fp32 [B, ld_y].
+extern "C" int rmlx_matvec_out(const void* w, const void* a, int ld_a, float* y, int ld_y, int B, int N, int K, int pdl,
+                               cudaStream_t st) {
+  if (K < 8 || K % 8 || ld_a % 8 || ld_a < K || N < 1 || ld_y < N || B > rmlx_postnorm_max_rows(K)) return -2;
+  RB_PN_DISPATCH(B, (launch_matvec<kB>(w, a, ld_a, y, ld_y, N, K, pdl, st)))
+}
+
+// raw fp32 [B, ld_raw] = [r | k | v | g] `inner` apart, then `rank` values (a multiple of eight); w2 bf16
+// [>= H * dim, rank]; a bf16 [B, ld_a]; state / prev as in rmlx_wkv_scan; x fp32 [B, ldx] what the layer read.
+extern "C" int rmlx_wkv_decode(const float* raw, int ld_raw, int inner, const void* w2, int rank, const float* w0,
+                               const float* u, const float* norm, float eps, const int* slots, float* state, float* prev,
+                               long long stride, const float* x, int ldx, void* a, int ld_a, int B, int H, int dim, int pdl,
+                               cudaStream_t st) {
+  if (B < 1 || B > 65535 || H < 1 || dim < 1 || dim > 256 || inner < H * dim || rank < 8 || rank % 8 ||
+      ld_raw < 4 * inner + rank || ld_a < H * dim || !slots || rank > 4096)
+    return -2;
+  int dim_pad = 8;
+  while (dim_pad < dim) dim_pad *= 2;
+  const size_t smem = size_t(3 * dim + rank + 256) * sizeof(float);
+  RB_CHECK(set_max_smem(wkv_decode_kernel, smem));
+  return launch(wkv_decode_kernel, dim3(H, B), dim3(256), smem, st, pdl != 0, raw, ld_raw, inner,
+                static_cast<const __nv_bfloat16*>(w2), rank, w0, u, norm, eps, slots, state, prev, stride, x, ldx,
+                static_cast<__nv_bfloat16*>(a), ld_a, dim, dim_pad);
+}

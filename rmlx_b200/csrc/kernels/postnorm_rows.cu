@@ -254,6 +254,23 @@ latent_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restr
   }
 }
 
+// The latents of whole contexts in position order: page i of the result is page pages[i].y of the sequence
+// in row pages[i].x of the block table. One block per page.
+__global__ void __launch_bounds__(kRowThreads)
+latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, int ldc, const int* __restrict__ block_table, int max_blocks,
+                     const int2* __restrict__ pages, __nv_bfloat16* __restrict__ out, int lat, int page) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int2 pg = pages[blockIdx.x];
+  const int blk = RB_BOUNDS(pg.y, max_blocks) ? block_table[size_t(pg.x) * max_blocks + pg.y] : 0;
+  const int units = lat / 8;
+  for (int i = threadIdx.x; i < page * units; i += kRowThreads) {
+    const int r = i / units, c = i - r * units;
+    reinterpret_cast<uint4*>(out + (size_t(blockIdx.x) * page + r) * lat)[c] =
+        reinterpret_cast<const uint4*>(cache + (size_t(blk) * page + r) * ldc)[c];
+  }
+}
+
 // out[r, i] = act(in[r, i], in[r, n + i]); n a multiple of eight.
 template <class T>
 __global__ void __launch_bounds__(kRowThreads)
@@ -377,6 +394,15 @@ extern "C" int rmlx_latent_append(const void* raw, int ldraw, int raw_f32, const
   if (raw_f32) RB_LA(float, __nv_bfloat16);
   RB_LA(__nv_bfloat16, __nv_bfloat16);
 #undef RB_LA
+}
+
+// cache [.., page, ldc] bf16, pages int32 [n, 2], out bf16 [n * page, lat]; lat and ldc multiples of eight.
+extern "C" int rmlx_latent_gather(const void* cache, int ldc, const int* block_table, int max_blocks, const int* pages,
+                                  void* out, int n, int lat, int page, int pdl, cudaStream_t st) {
+  if (n < 1 || lat < 8 || lat % 8 || ldc % 8 || ldc < lat || page < 1 || (reinterpret_cast<uintptr_t>(pages) & 7)) return -2;
+  return launch(latent_gather_kernel, dim3(n), dim3(kRowThreads), 0, st, pdl != 0,
+                static_cast<const __nv_bfloat16*>(cache), ldc, block_table, max_blocks,
+                reinterpret_cast<const int2*>(pages), static_cast<__nv_bfloat16*>(out), lat, page);
 }
 
 // in [R, 2 n] = [gate | up], out [R, n], both fp32 (f32) or bf16; n a multiple of eight.

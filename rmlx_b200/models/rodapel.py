@@ -23,6 +23,7 @@ from .. import _lib
 from ..config import (ClampedFfSpec, LatentAttentionSpec, PostNormLayerSpec, RodapelConfig, RoutedFfSpec,
                       WindowAttentionSpec, WkvSpec)
 from ..kv.paged import PAGE, PagedKvCache
+from ..ops import latent as L
 from ..ops import parallel_block as P
 from ..ops import post_norm as N
 from ..ops import routed as R
@@ -35,6 +36,9 @@ from ..ops.weights import LinearWeight, W_BF16
 from .ragged import Entry, RaggedBatch
 from .weights import ParallelLayout
 
+# Latent attention: batch entries of up to this many tokens attend to the cached latents; longer ones to keys
+# and values expanded for their whole context (which costs about as much as 0.8 * kv_rank query tokens).
+LATENT_ABSORB = 4
 LATENT_ROW_PAD = 8       # unused values behind a latent cache row (csrc/kernels/mla_decode.cu)
 
 
@@ -72,6 +76,7 @@ class LatentWeights:
     c_norm: torch.Tensor             # fp32 [rank]
     w_uk: torch.Tensor               # [heads, lat_p, dim_p]: queries into the latent space
     w_uv: torch.Tensor               # [heads, vdim_p, lat_p]: attended latents to values
+    w_ukv: LinearWeight              # [heads * (dim_p + vdim_p), lat_p]: latents to keys and values
     w_o: LinearWeight                # [width_p, heads * vdim_p]
     inv_freq: torch.Tensor           # fp32 [rotated pairs]
     mods: ScoreMods
@@ -97,8 +102,7 @@ class LatentWeights:
 class WkvWeights:
     spec: WkvSpec
     mu: torch.Tensor                 # fp32 [5, width_p] (r, k, v, g, w)
-    w_rkvg: LinearWeight             # [4, inner_p, width_p]
-    w1: torch.Tensor                 # [rank_p, width_p]
+    w_in: LinearWeight               # [4 * inner_p + rank_p, width_p]: r | k | v | g | decay rank
     w2: torch.Tensor                 # [inner_p, rank_p]
     w0: torch.Tensor                 # fp32 [heads * dim]
     u: torch.Tensor                  # fp32 [heads * dim]
@@ -108,6 +112,15 @@ class WkvWeights:
     @property
     def inner_p(self) -> int:
         return self.w_o.k
+
+    @property
+    def rank_p(self) -> int:
+        return self.w2.shape[1]
+
+    def part(self, s: int) -> torch.Tensor:
+        """Projection of shift part ``s`` (r, k, v, g; 4: the decay's first factor)."""
+        at = s * self.inner_p
+        return self.w_in.w[at:at + (self.inner_p if s < 4 else self.rank_p)]
 
 
 @dataclass
@@ -265,17 +278,17 @@ def build_weights(cfg: RodapelConfig, tensors: Dict[str, torch.Tensor], device="
             uk[:, :m.kv_rank, :m.dim] = dev(g("uk")).view(m.heads, m.dim, m.kv_rank).transpose(1, 2)
             uv = torch.zeros(m.heads, pad8(m.vdim), pad8(m.kv_rank), dtype=dtype, device=device)
             uv[:, :m.vdim, :m.kv_rank] = dev(g("uv")).view(m.heads, m.vdim, m.kv_rank)
+            ukv = torch.cat([uk.transpose(1, 2), uv], 1).reshape(-1, pad8(m.kv_rank)).contiguous()
             pairs = torch.arange(m.rot_dims // 2, dtype=torch.float64)
             return LatentWeights(m, lin([g("q"), g("dkv")], pad8(rows), wp), vec(g("dkv.norm")), uk, uv,
-                                 out_proj(g("o"), m.heads, m.vdim), vec(m.rot_base ** (-2.0 * pairs / max(m.rot_dims, 1))),
+                                 LinearWeight(W_BF16, ukv), out_proj(g("o"), m.heads, m.vdim), vec(m.rot_base ** (-2.0 * pairs / max(m.rot_dims, 1))),
                                  ScoreMods(m.scale))
         n = m.heads * m.dim
-        inner, rank, rank_p = pad8(n), ranks[i], pad8(ranks[i])
+        inner, rank, rank_p = pad_to(n, 16), ranks[i], pad_to(ranks[i], 16)
         m = replace(m, decay_rank=rank)
-        return WkvWeights(m, torch.stack([vec(g("mu." + s), wp) for s in W.SHIFT_PARTS]),
-                          LinearWeight(W_BF16, torch.stack([mat([g(s)], inner, wp) for s in "rkvg"])),
-                          mat([g("w1")], rank_p, wp), mat([g("w2")], inner, rank_p), vec(g("w0")), vec(g("u")),
-                          vec(g("norm")), lin([g("o")], wp, inner))
+        w_in = torch.cat([mat([g(s)], inner, wp) for s in "rkvg"] + [mat([g("w1")], rank_p, wp)])
+        return WkvWeights(m, torch.stack([vec(g("mu." + s), wp) for s in W.SHIFT_PARTS]), LinearWeight(W_BF16, w_in),
+                          mat([g("w2")], inner, rank_p), vec(g("w0")), vec(g("u")), vec(g("norm")), lin([g("o")], wp, inner))
 
     def feed_forward(i: int, f):
         p = f"l{i}.mlp."
@@ -342,6 +355,17 @@ class Buffers:
             buf = self._store[name, dtype] = torch.zeros(self.rows * per, dtype=dtype, device=self.device)
         return buf[:t * per].view(t, *shape)
 
+    def rows_of(self, name: str, n: int, *shape: int, dtype) -> torch.Tensor:
+        """[n, *shape] where ``n`` is not bounded by the batch (expanded contexts): grows as needed."""
+        per = 1
+        for s in shape:
+            per *= s
+        buf = self._store.get((name, dtype))
+        if buf is None or buf.numel() < n * per:
+            self._store.pop((name, dtype), None)
+            buf = self._store[name, dtype] = torch.zeros(n * per, dtype=dtype, device=self.device)
+        return buf[:n * per].view(n, *shape)
+
 
 @dataclass
 class StepContext:
@@ -372,7 +396,9 @@ class RodapelModel:
         self.width_p = pad8(self.cfg.width)
         self.allgather_logits = None
         self._bufs: Optional[Buffers] = None
-        self._scratch: Dict[tuple, P.ScoredDecodeScratch] = {}
+        self._scratch: Dict[tuple, object] = {}
+        latent = [l.mix for l in weights.layers if isinstance(l.mix, LatentWeights)]
+        self._absorb = LATENT_ABSORB if self.device.type == "cuda" and any(map(self.latent_prefill, latent)) else None
 
     @classmethod
     def from_config(cls, cfg: Optional[RodapelConfig] = None, seed: int = 0, device="cuda", dtype=torch.bfloat16
@@ -471,20 +497,56 @@ class RodapelModel:
                                       rows=b.single, table_rows=c.token_seq, window=m.window, gate=gate)
         return self._output(attn.view(t, -1), mw.w_o, c)
 
-    def latent_attention(self, li: int, mw: LatentWeights, h: torch.Tensor, c: StepContext) -> torch.Tensor:
+    def latent_prefill(self, mw: LatentWeights) -> bool:
+        return self.dtype == torch.bfloat16 and L.prefill_supported(mw.dim_p, mw.rot_p, mw.vdim_p)
+
+    def absorbed_attention(self, mw: LatentWeights, pool: torch.Tensor, q: torch.Tensor, q_abs: torch.Tensor,
+                           attn: torch.Tensor, c: StepContext, rows: Optional[torch.Tensor], longest: int) -> None:
+        """Queries into the latent space, attention over the cached latents, attended latents to values."""
+        m, pdl = mw.spec, c.pdl
+        o_lat = c.bufs.get("o_lat", c.t, m.heads, mw.lat_p, dtype=self.dtype)
+        N.head_gemv(mw.w_uk, q, q_abs, rows=rows, pdl=pdl)
+        if self.dtype == torch.bfloat16 and (m.kv_rank, m.rot_dim) in L.DECODE_WIDTHS:
+            n = c.t if rows is None else rows.numel()
+            splits = L.decode_splits(n, m.heads, longest)
+            key = ("latent", m.heads, mw.lat_p, n, splits)
+            if key not in self._scratch:
+                self._scratch[key] = L.LatentDecodeScratch(n, m.heads, splits, mw.lat_p, self.device)
+            L.latent_decode(q_abs, pool, c.block_table, c.positions, m.scale, o_lat, self._scratch[key], rows=rows,
+                            table_rows=c.token_seq, pdl=pdl)
+        else:
+            P.attention_any(q_abs, pool, pool, c.block_table, c.positions, c.token_seq, mw.mods, o_lat, rows=rows, pdl=pdl)
+        N.head_gemv(mw.w_uv, o_lat, attn, rows=rows, pdl=pdl)
+
+    def latent_core(self, li: int, mw: LatentWeights, raw: torch.Tensor, c: StepContext) -> torch.Tensor:
+        """Everything between the two projections: raw [T, q | latent | key part] -> attention output rows."""
         m, t, dt, pdl = mw.spec, c.t, self.dtype, c.pdl
-        pool = c.cache.k[li]
-        raw = N.linear(h, mw.w_in.w, c.bufs.get("raw", t, mw.w_in.n, dtype=dt), pdl=pdl)
+        pool, b = c.cache.k[li], c.batch
         q = c.bufs.get("q", t, m.heads, mw.dim_p + mw.rot_p, dtype=dt)
         q_abs = c.bufs.get("q_abs", t, m.heads, mw.lat_p + mw.rot_p, dtype=dt)
-        o_lat = c.bufs.get("o_lat", t, m.heads, mw.lat_p, dtype=dt)
         attn = c.bufs.get("attn", t, m.heads, mw.vdim_p, dtype=dt)
-        N.latent_append(raw, mw.c_norm, self.cfg.norm_eps, mw.inv_freq, q, q_abs, pool, c.block_table, c.positions,
-                        c.token_seq, m.heads, m.dim, m.rot_dim, m.kv_rank, mw.dim_p, mw.rot_p, mw.lat_p, pdl=pdl)
-        N.head_gemv(mw.w_uk, q, q_abs, pdl=pdl)
-        P.attention_any(q_abs, pool, pool, c.block_table, c.positions, c.token_seq, mw.mods, o_lat, pdl=pdl)
-        N.head_gemv(mw.w_uv, o_lat, attn, pdl=pdl)
-        return self._output(attn.view(t, -1), mw.w_o, c)
+        expand = b is not None and b.latent_tiles is not None and self.latent_prefill(mw)
+        some_absorbed = not expand or b.absorbed is not None
+        N.latent_append(raw, mw.c_norm, self.cfg.norm_eps, mw.inv_freq, q, q_abs if some_absorbed else None, pool,
+                        c.block_table, c.positions, c.token_seq, m.heads, m.dim, m.rot_dim, m.kv_rank, mw.dim_p, mw.rot_p,
+                        mw.lat_p, pdl=pdl)
+        if expand:
+            n = b.ctx_pages.shape[0] * PAGE
+            ctx = c.bufs.rows_of("ctx", n, mw.lat_p, dtype=dt)
+            kv = c.bufs.rows_of("ctx_kv", n, m.heads, mw.dim_p + mw.vdim_p, dtype=dt)
+            L.latent_gather(pool, c.block_table, b.ctx_pages, ctx)
+            N.linear(ctx, mw.w_ukv.w, kv.view(n, -1))
+            L.flash_prefill_latent(q, kv, pool, mw.lat_p, c.block_table, b.latent_tiles, b.tile_ctx, m.scale, attn, mw.dim_p,
+                                   lanes=b.latent_lanes)
+        if some_absorbed:
+            rows = b.absorbed if expand else None
+            longest = c.max_len if b is None else b.absorbed_len if expand else max(p + l for p, l in zip(b.pos0, b.lens))
+            self.absorbed_attention(mw, pool, q, q_abs, attn, c, rows, longest)
+        return attn
+
+    def latent_attention(self, li: int, mw: LatentWeights, h: torch.Tensor, c: StepContext) -> torch.Tensor:
+        raw = N.linear(h, mw.w_in.w, c.bufs.get("raw", c.t, mw.w_in.n, dtype=self.dtype), pdl=c.pdl)
+        return self._output(self.latent_core(li, mw, raw, c).view(c.t, -1), mw.w_o, c)
 
     def time_mix(self, li: int, mw: WkvWeights, x: torch.Tensor, c: StepContext) -> torch.Tensor:
         m, t, dt, pdl, inner = mw.spec, c.t, self.dtype, c.pdl, mw.inner_p
@@ -494,9 +556,9 @@ class RodapelModel:
         W.token_shift(x, mw.mu, prev, c.slots, c.runs is None, mix, pdl=pdl)
         rkvg = c.bufs.get("rkvg", t, 4, inner, dtype=dt).view(4, t, inner)
         for s in range(4):
-            N.linear(mix[s], mw.w_rkvg.w[s], rkvg[s], pdl=pdl)
-        low = P.logits_f32(mix[4], mw.w1, c.bufs.get("low", t, mw.w1.shape[0], dtype=torch.float32))
-        low_t = N.tanh_rows(low, c.bufs.get("low_t", t, mw.w1.shape[0], dtype=dt), pdl=pdl)
+            N.linear(mix[s], mw.part(s), rkvg[s], pdl=pdl)
+        low = P.logits_f32(mix[4], mw.part(4), c.bufs.get("low", t, mw.rank_p, dtype=torch.float32))
+        low_t = N.tanh_rows(low, c.bufs.get("low_t", t, mw.rank_p, dtype=dt), pdl=pdl)
         decay = P.logits_f32(low_t, mw.w2, c.bufs.get("decay", t, inner, dtype=torch.float32))
         o = c.bufs.get("wkv_o", t, inner, dtype=torch.float32)
         W.wkv_scan(rkvg[0], rkvg[1], rkvg[2], decay, mw.w0, mw.u, state, prev, x, o, runs=c.runs,
@@ -586,7 +648,8 @@ class RodapelModel:
         called with (layer, residual rows [T, width]) after every layer."""
         if self.device.type != "cuda":
             raise _lib.NativeError("Rodapel runs on this package's CUDA kernels only")
-        batch = RaggedBatch.plan(entries, cache, min(l.mixer.heads for l in self.cfg.layers))
+        batch = RaggedBatch.plan(entries, cache, min(l.mixer.heads for l in self.cfg.layers),
+                                 self._absorb)
         for e, l in zip(batch.entries, batch.lens):
             cache.reserve(e.seq_id, l)
         batch.upload(self.device)

@@ -194,24 +194,14 @@ def _mla_decode_kernel(q_abs: torch.Tensor, cache: MlaPagedCache, slots: torch.T
     """q_abs [B, H, LAT + ROPE] bf16 (absorbed queries) -> o_lat [B, H, LAT] bf16 on the device
     kernel; row b attends to the sequence in cache slot ``slots[b]``."""
     from .. import _lib
-    _lib.register_cuda_sigs({
-        "rmlx_mla_decode_paged": ("ppppppppiiiiiiifip", "i"),
-        "rmlx_mla_decode_part_o_elems": ("iiii", "q"),
-        "rmlx_mla_decode_part_ml_elems": ("iii", "q"),
-    })
+    from ..ops.latent import decode_splits
     lib = _lib.cuda()
     b, h, w = q_abs.shape
     lat = cache.cfg.kv_lora_rank
     table, lens = cache.block_table, cache.seq_lens      # the kernel indexes both by slots[b]
     slots = slots.to(torch.int32)
     if splits <= 0:
-        # Up to 16 head tiles: wide blocks (eight warps, one per SM), one wave of 148. More: narrow
-        # blocks (four warps, two per SM; the launcher picks them once the grid exceeds the SMs),
-        # one wave of 296. At least 8 pages per split.
-        tiles = b * ((h + 15) // 16)
-        longest = int(table.shape[1]) * MlaPagedCache.PAGE
-        slots_per_wave = 148 if tiles <= 16 else 296
-        splits = max(1, min(64, slots_per_wave // tiles, longest // 128))
+        splits = decode_splits(b, h, int(table.shape[1]) * MlaPagedCache.PAGE)
     out = torch.empty(b, h, lat, dtype=torch.bfloat16, device=q_abs.device)
     part_o = part_ml = None
     if splits > 1:
@@ -220,7 +210,7 @@ def _mla_decode_kernel(q_abs: torch.Tensor, cache: MlaPagedCache, slots: torch.T
         part_ml = torch.empty(lib.rmlx_mla_decode_part_ml_elems(b, h, splits), dtype=torch.float32,
                               device=q_abs.device)
     rc = lib.rmlx_mla_decode_paged(q_abs.data_ptr(), cache.store.data_ptr(), table.data_ptr(),
-                                   lens.data_ptr(), slots.data_ptr(), out.data_ptr(), _lib.ptr(part_o), _lib.ptr(part_ml),
+                                   lens.data_ptr(), slots.data_ptr(), None, None, None, out.data_ptr(), _lib.ptr(part_o), _lib.ptr(part_ml),
                                    b, h, lat, w - lat, cache.store.shape[2], table.shape[1], splits, scale, 0,
                                    _lib.stream_ptr())
     _lib.check(rc, "mla_decode_paged")

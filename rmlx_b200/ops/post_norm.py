@@ -3,6 +3,7 @@ plain projections in the activations' type, and the per-head products of absorbe
 (head_gemv.cu). Activations are bf16 or fp32; the dtype of the tensors picks the kernels."""
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -21,6 +22,10 @@ _lib.register_cuda_sigs({
     "rmlx_gated_act": ("ppiifiip", "i"),
     "rmlx_tanh_rows": ("ppqiip", "i"),
     "rmlx_head_gemv": ("ppiipiipiiiiiip", "i"),
+    "rmlx_postnorm_max_rows": ("i", "i"),
+    "rmlx_postnorm_in": ("ppppfpii" "pppqi" "piiiip", "i"),
+    "rmlx_postnorm_gated": ("ppppfpii" "piiifip", "i"),
+    "rmlx_matvec_out": ("ppipiiiiip", "i"),
 })
 
 
@@ -140,3 +145,68 @@ def tanh_rows(x: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> torch.Te
     rc = _lib.cuda().rmlx_tanh_rows(x.data_ptr(), out.data_ptr(), x.numel(), _f32(out), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "tanh_rows")
     return out
+
+
+# ------------------------------------------------------------------ decode projections (csrc/kernels/postnorm_gemv.cu)
+def max_rows(k: int) -> int:
+    """Rows one launch of the decode projections takes for ``k`` staged values (0: none)."""
+    return int(_lib.cuda().rmlx_postnorm_max_rows(k))
+
+
+def _chunks(b: int, k: int):
+    step = max_rows(k)
+    if step < 1:
+        raise _lib.NativeError(f"decode projections: {k} values do not fit a block's shared memory")
+    return [(lo, min(b, lo + step)) for lo in range(0, b, step)]
+
+
+@dataclass
+class Pending:
+    """A finished sublayer's output that still has to be normed and added to the residual: what the next kernel
+    that reads the residual does on the way."""
+    y: Optional[torch.Tensor]        # fp32 [B, width_p]; None: nothing pending
+    w: Optional[torch.Tensor]        # fp32 [width_p]
+
+
+def postnorm_in(x: torch.Tensor, pending: Pending, eps: float, width: int, x_out: torch.Tensor, w: torch.Tensor,
+                out: torch.Tensor, shift=None, pdl: bool = False) -> None:
+    """x_out = x + RMSNorm(pending); out = W x_out in fp32. ``shift``: (mu [5, width_p], prev [slots, width_p],
+    slots, segment rows) - the row segments of W then read their token-shift mixes of x_out."""
+    _lib.require_cuda_tensor(x, x_out, w, out, pending.y)
+    b, k = x.shape
+    assert x.dtype == x_out.dtype == out.dtype == torch.float32 and w.dtype == torch.bfloat16 and w.is_contiguous()
+    assert w.shape[1] == k and x.is_contiguous() and x_out.is_contiguous() and out.shape[0] == b
+    for lo, hi in _chunks(b, k):
+        y = None if pending.y is None else pending.y[lo:].data_ptr()
+        sh = (None, None, None, 0, 0) if shift is None else (
+            shift[0].data_ptr(), shift[1].data_ptr(), shift[2][lo:].data_ptr(), shift[1].stride(0), shift[3])
+        rc = _lib.cuda().rmlx_postnorm_in(w.data_ptr(), x[lo:].data_ptr(), y, _lib.ptr(pending.w), eps, x_out[lo:].data_ptr(),
+                                          width, k, *sh, out[lo:].data_ptr(), out.stride(0), hi - lo, w.shape[0], int(pdl),
+                                          _lib.stream_ptr())
+        _lib.check(rc, "postnorm_in")
+
+
+def postnorm_gated(x: torch.Tensor, pending: Pending, eps: float, width: int, x_out: torch.Tensor, w: torch.Tensor,
+                   limit: float, act: torch.Tensor, pdl: bool = False) -> None:
+    """x_out = x + RMSNorm(pending); act = gated activation of W x_out, W = [gate; up]."""
+    _lib.require_cuda_tensor(x, x_out, w, act, pending.y)
+    b, k = x.shape
+    assert w.shape == (2 * act.shape[1], k) and w.is_contiguous() and act.dtype == w.dtype == torch.bfloat16
+    for lo, hi in _chunks(b, k):
+        y = None if pending.y is None else pending.y[lo:].data_ptr()
+        rc = _lib.cuda().rmlx_postnorm_gated(w.data_ptr(), x[lo:].data_ptr(), y, _lib.ptr(pending.w), eps,
+                                             x_out[lo:].data_ptr(), width, k, act[lo:].data_ptr(), act.stride(0), hi - lo,
+                                             act.shape[1], limit, int(pdl), _lib.stream_ptr())
+        _lib.check(rc, "postnorm_gated")
+
+
+def matvec_out(a: torch.Tensor, w: torch.Tensor, y: torch.Tensor, pdl: bool = False) -> torch.Tensor:
+    """y = a w^T, bf16 in, fp32 out, a few rows."""
+    _lib.require_cuda_tensor(a, w, y)
+    b, k = a.shape
+    assert a.dtype == w.dtype == torch.bfloat16 and y.dtype == torch.float32 and w.is_contiguous() and w.shape[1] == k
+    for lo, hi in _chunks(b, k):
+        rc = _lib.cuda().rmlx_matvec_out(w.data_ptr(), a[lo:].data_ptr(), a.stride(0), y[lo:].data_ptr(), y.stride(0), hi - lo,
+                                         w.shape[0], k, int(pdl), _lib.stream_ptr())
+        _lib.check(rc, "matvec_out")
+    return y

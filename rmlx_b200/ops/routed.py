@@ -9,7 +9,7 @@ import torch
 
 from .. import _lib
 from .parallel_block import _f32
-from .post_norm import gated_act
+from .post_norm import Pending, _chunks, gated_act, max_rows
 from .quantized import xgemm
 from .weights import LinearWeight
 
@@ -21,6 +21,9 @@ _lib.register_cuda_sigs({
     "rmlx_route_corrected": ("pippppppiiiiip", "i"),
     "rmlx_route_scatter": ("pipppp" "iiiiip", "i"),
     "rmlx_moe_combine_post_norm": ("pipppipfppiiiiip", "i"),
+    "rmlx_postnorm_router": ("ppppfpii" "pppppp" "iiiiip", "i"),
+    "rmlx_postnorm_expert": ("ppippiiiiifip", "i"),
+    "rmlx_expert_out": ("piipippppp" "iiiiiip", "i"),
     "rmlx_sgemm_grouped": ("pipipipiiiiip", "i"),
 })
 
@@ -91,3 +94,48 @@ def combine_post_norm(y: torch.Tensor, r: Routing, w: torch.Tensor, eps: float, 
         r.idx.shape[1], w.data_ptr(), eps, x.data_ptr(), h.data_ptr(), t, width, ldx, _f32(y), int(pdl),
         _lib.stream_ptr())
     _lib.check(rc, "moe_combine_post_norm")
+
+
+# ------------------------------------------------------------------ decode (csrc/kernels/postnorm_gemv.cu)
+def postnorm_router(x: torch.Tensor, pending: Pending, eps: float, width: int, x_out: torch.Tensor, w: torch.Tensor,
+                    correction: torch.Tensor, experts: int, logits: torch.Tensor, ticket: torch.Tensor, r: Routing,
+                    pdl: bool = False) -> None:
+    """x_out = x + RMSNorm(pending), router logits and the choice. ``ticket``: one int32 word, zero."""
+    _lib.require_cuda_tensor(x, x_out, w, logits, ticket)
+    b, k = x.shape
+    outputs, top = w.shape[0], r.idx.shape[1]
+    assert w.dtype == torch.bfloat16 and w.is_contiguous() and logits.is_contiguous() and correction.numel() == outputs
+    for lo, hi in _chunks(b, k):
+        y = None if pending.y is None else pending.y[lo:].data_ptr()
+        rc = _lib.cuda().rmlx_postnorm_router(
+            w.data_ptr(), x[lo:].data_ptr(), y, _lib.ptr(pending.w), eps, x_out[lo:].data_ptr(), width, k,
+            correction.data_ptr(), logits[lo:].data_ptr(), r.idx[lo:].data_ptr(), r.weights[lo:].data_ptr(),
+            r.identity[lo:].data_ptr(), ticket.data_ptr(), hi - lo, experts, outputs, top, int(pdl), _lib.stream_ptr())
+        _lib.check(rc, "postnorm_router")
+
+
+def postnorm_expert(x: torch.Tensor, w: torch.Tensor, limit: float, r: Routing, act: torch.Tensor, pdl: bool = False) -> None:
+    """act [B * top, n] = gated activation of the chosen experts' [gate; up] projections of x (fp32)."""
+    _lib.require_cuda_tensor(x, w, act)
+    e, n2, k = w.shape
+    assert x.shape[1] == k and w.is_contiguous() and act.shape == (r.idx.numel(), n2 // 2) and act.is_contiguous()
+    rc = _lib.cuda().rmlx_postnorm_expert(w.data_ptr(), x.data_ptr(), k, r.idx.data_ptr(), act.data_ptr(), act.stride(0),
+                                          x.shape[0], r.idx.shape[1], n2 // 2, e, limit, int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "postnorm_expert")
+
+
+def expert_out(act: torch.Tensor, w: torch.Tensor, r: Routing, x: torch.Tensor, y: torch.Tensor, pdl: bool = False) -> None:
+    """y = sum of the slots' weighted down projections + identity weight * x."""
+    _lib.require_cuda_tensor(act, w, x, y)
+    e, rows, k = w.shape
+    b, ldx = x.shape
+    assert y.shape == x.shape and act.stride(0) >= k and w.is_contiguous()
+    rc = _lib.cuda().rmlx_expert_out(w.data_ptr(), rows, k, act.data_ptr(), act.stride(0), r.idx.data_ptr(),
+                                     r.weights.data_ptr(), r.identity.data_ptr(), x.data_ptr(), y.data_ptr(), ldx, b, ldx,
+                                     r.idx.shape[1], e, int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "expert_out")
+
+
+def expert_decode_fits(k: int, top: int) -> bool:
+    """Whether ``expert_out`` can stage ``top`` activations of ``k`` values."""
+    return max_rows(k * top) > 0

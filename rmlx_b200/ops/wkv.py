@@ -15,6 +15,7 @@ _lib.register_cuda_sigs({
     "rmlx_wkv_max_dim": ("", "i"),
     "rmlx_token_shift": ("pippqpipiiip", "i"),
     "rmlx_wkv_scan": ("pppipippppi" "ppqpipi" "iiiip", "i"),
+    "rmlx_wkv_decode": ("piipipppfp" "ppqpipiiiiip", "i"),
     "rmlx_wkv_finish": ("pipipfpiiiiiip", "i"),
 })
 
@@ -65,3 +66,19 @@ def wkv_finish(o: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor, eps: flo
                                      out.data_ptr(), out.stride(0), o.shape[0], heads, dim, _f32(out), int(pdl),
                                      _lib.stream_ptr())
     _lib.check(rc, "wkv_finish")
+
+
+def wkv_decode(raw: torch.Tensor, inner: int, w2: torch.Tensor, w0: torch.Tensor, u: torch.Tensor, norm: torch.Tensor,
+               eps: float, slots: torch.Tensor, state: torch.Tensor, prev: torch.Tensor, x: torch.Tensor,
+               out: torch.Tensor, pdl: bool = False) -> None:
+    """One token per row through recurrence, head norm and gate: raw fp32 [B, 4 * inner + rank] = r | k | v | g | decay
+    rank, ``x`` the rows the layer read (kept in ``prev``); out bf16 [B, >= H d] (csrc/kernels/postnorm_gemv.cu)."""
+    _lib.require_cuda_tensor(raw, w2, w0, u, norm, slots, state, prev, x, out)
+    _, h, d, _ = state.shape
+    assert raw.dtype == x.dtype == torch.float32 and w2.dtype == out.dtype == torch.bfloat16 and w2.is_contiguous()
+    assert state.stride()[1:] == (d * d, d, 1) and state.stride(0) == prev.stride(0) and slots.dtype == torch.int32
+    rc = _lib.cuda().rmlx_wkv_decode(
+        raw.data_ptr(), raw.stride(0), inner, w2.data_ptr(), w2.shape[1], w0.data_ptr(), u.data_ptr(), norm.data_ptr(), eps,
+        slots.data_ptr(), state.data_ptr(), prev.data_ptr(), state.stride(0), x.data_ptr(), x.stride(0), out.data_ptr(),
+        out.stride(0), raw.shape[0], h, d, int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "wkv_decode")
