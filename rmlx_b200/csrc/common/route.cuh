@@ -7,12 +7,11 @@ namespace rb {
 constexpr int kRouteMaxOutputs = 512;
 constexpr int kRouteMaxTop = 32;
 
-// logits, correction: fp32 [outputs], the first `experts` of them with weights of their own. Ties go to
+// N: outputs a lane holds. logits, correction: fp32 [outputs], the first `experts` of them with weights of their own. Ties go to
 // the lower index. counts (may be null) gets one more for every chosen expert.
-__device__ __forceinline__ void warp_route_corrected(const float* logits, const float* correction, int experts,
-                                                     int outputs, int top_k, int* idx, float* weights, float* identity,
-                                                     int* counts) {
-  constexpr int N = kRouteMaxOutputs / 32;
+template <int N>
+__device__ __forceinline__ void warp_route_n(const float* logits, const float* correction, int experts, int outputs,
+                                             int top_k, int* idx, float* weights, float* identity, int* counts) {
   const int lane = threadIdx.x & 31;
   float s[N], c[N], m = -INFINITY;
 #pragma unroll
@@ -59,6 +58,14 @@ __device__ __forceinline__ void warp_route_corrected(const float* logits, const 
     if (counts && my_e < experts) atomicAdd(counts + my_e, 1);
   }
   if (lane == 0) *identity = id_w;
+}
+
+__device__ __forceinline__ void warp_route_corrected(const float* logits, const float* correction, int experts,
+                                                     int outputs, int top_k, int* idx, float* weights, float* identity,
+                                                     int* counts) {
+  if (outputs <= 64) warp_route_n<2>(logits, correction, experts, outputs, top_k, idx, weights, identity, counts);
+  else if (outputs <= 256) warp_route_n<8>(logits, correction, experts, outputs, top_k, idx, weights, identity, counts);
+  else warp_route_n<kRouteMaxOutputs / 32>(logits, correction, experts, outputs, top_k, idx, weights, identity, counts);
 }
 
 }  // namespace rb

@@ -44,4 +44,20 @@ __device__ __forceinline__ float row_block_sum(float v, float* red) {
   return t;
 }
 
+// Eight elements of which the first n exist (the rest read as zero); `aligned`: all eight, 16-byte aligned.
+template <class T>
+__device__ __forceinline__ void load8_upto(const T* p, int n, bool aligned, float (&f)[8]) {
+  if (aligned) { load8(p, f); return; }
+#pragma unroll
+  for (int i = 0; i < 8; ++i) f[i] = i < n ? to_f32(p[i]) : 0.f;
+}
+
+// Sum over groups of L consecutive lanes (L a power of two).
+template <int L>
+__device__ __forceinline__ float group_sum(float v) {
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+
 }  // namespace rb

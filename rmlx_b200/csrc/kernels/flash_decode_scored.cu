@@ -96,7 +96,8 @@ __device__ __forceinline__ void fs_copy_page(char* dst, const char* src, int chu
   }
 }
 
-template <int DK, int DV, int NST>
+// MOD = false: no modifier but the scale.
+template <int DK, int DV, int NST, bool MOD>
 __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParams p) {
   constexpr int KS = DK / 16;            // k-steps of the QK^T product
   constexpr int NT = DV / 8;             // n-tiles of the PV product
@@ -263,6 +264,7 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
       *reinterpret_cast<uint4*>(&sQ[r][c * 8]) = v;
     }
   }
+  const float lin = p.mod.scale * kLog2e;
   HeadScore hs0{}, hs1{};
   if (gt * 16 + g < p.G) hs0 = head_score(p.mod, kvh * p.G + gt * 16 + g);
   if (gt * 16 + g + 8 < p.G) hs1 = head_score(p.mod, kvh * p.G + gt * 16 + g + 8);
@@ -318,16 +320,21 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
     const int tok0 = pg * kFsPage + t * 2;
     float sv[8] = {s0[0], s0[1], s1[0], s1[1], s0[2], s0[3], s1[2], s1[3]};
     const int tk[4] = {tok0, tok0 + 1, tok0 + 8, tok0 + 9};
-    float dist[4], top0 = 0.f, top1 = 0.f;
+    if (MOD) {
+      float dist[4], top0 = 0.f, top1 = 0.f;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      dist[i] = float(len - 1 - tk[i]);
-      top0 = fmaxf(top0, fabsf(sv[i]));
-      top1 = fmaxf(top1, fabsf(sv[4 + i]));
+      for (int i = 0; i < 4; ++i) {
+        dist[i] = float(len - 1 - tk[i]);
+        top0 = fmaxf(top0, fabsf(sv[i]));
+        top1 = fmaxf(top1, fabsf(sv[4 + i]));
+      }
+      const bool near = !__any_sync(0xffffffffu, fmaxf(top0 * fabsf(hs0.inner), top1 * fabsf(hs1.inner)) > kTanhPolyMax);
+      scores_base2<4>(sv, hs0, dist, near);
+      if (upper) scores_base2<4>(sv + 4, hs1, dist, near);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) sv[i] *= lin;
     }
-    const bool near = !__any_sync(0xffffffffu, fmaxf(top0 * fabsf(hs0.inner), top1 * fabsf(hs1.inner)) > kTanhPolyMax);
-    scores_base2<4>(sv, hs0, dist, near);
-    if (upper) scores_base2<4>(sv + 4, hs1, dist, near);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const bool ok = tk[i] < len && tk[i] >= first;
@@ -512,6 +519,7 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
   if (raw && gate_col >= 0 && raw_ld < gate_col + Hq) return -2;
   if (p.Hkv * p.gtiles > 65535) return -2;
   const dim3 grid(splits, Hkv * p.gtiles, B);
+  const bool plain = softcap <= 0.f && !temp && !r1 && !sink;
   const bool deep = size_t(splits) * Hkv * p.gtiles * B <= size_t(2 * sm_count());
   // staging (>= 4 x 2 x 4 KB) covers the warp merge (4 x 16 x DV floats) and the split tables (12 KB)
 #define RB_FS(DK_, DV_, NST_)                                                      \
@@ -519,7 +527,8 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
     constexpr size_t smem = size_t(kFsWarps) * NST_ * kFsPage * (DK_ + DV_) * 2;   \
     static_assert(smem >= size_t(kFsWarps) * 16 * DV_ * 4, "warp merge");          \
     static_assert(smem >= size_t(kFsMaxSplits) * 16 * 3 * 4, "split tables");      \
-    auto kern = flash_decode_scored_kernel<DK_, DV_, NST_>;                        \
+    auto kern = plain ? flash_decode_scored_kernel<DK_, DV_, NST_, false>          \
+                      : flash_decode_scored_kernel<DK_, DV_, NST_, true>;          \
     RB_CHECK(set_max_smem(kern, smem));                                            \
     return launch(kern, grid, dim3(kFsThreads), smem, st, pdl != 0, p);            \
   }

@@ -92,7 +92,7 @@ struct TcParams {
   int window;               // > 0: a query sees only its last `window` keys
   float scale_log2;
   ScoreMod mod;             // MOD instances
-  HeadGate gate;            // MOD instances
+  HeadGate gate;            // ragged batches
   // LAT instances: panels of the unrotated key part, where the rotated part starts in a query row and in
   // a cache row, first context row of every tile's sequence
   int kn, q_rot, c_rot;
@@ -582,7 +582,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     if (ok && my_steps > 0) {
       tc_fence_after_sync();
       float inv = l > 0.f ? 1.f / l : 0.f;
-      if (MOD) inv *= head_gate<__nv_bfloat16>(p.gate, size_t(q0 + min(lrow, rows - 1)), h);
+      if (p.gate.gate) inv *= head_gate<__nv_bfloat16>(p.gate, size_t(q0 + min(lrow, rows - 1)), h);
       __nv_bfloat16* dst = p.out + (size_t(q0 + min(lrow, rows - 1)) * p.Hq + h) * p.dv;
 #pragma unroll 1
       for (int c = 0; c < VP * 2; ++c) {
@@ -716,11 +716,20 @@ extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, con
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2; p.mod.sink = sink;
   p.gate.gate = gate; p.gate.ld = ldg;
   p.status = status;
+  // no modifier but the scale: the plain softmax
+  const bool plain = softcap <= 0.f && !temp && !r1 && !sink;
+  if (plain) p.scale_log2 = scale * kLog2e;
 #define RB_FPS(KP_, VP_)                                                             \
+  if (plain)                                                                         \
+    return lanes == 2 ? launch_prefill_tc<2, KP_, VP_, false>(tq, tk, tv, p, pdl, st)  \
+                      : launch_prefill_tc<1, KP_, VP_, false>(tq, tk, tv, p, pdl, st); \
   return lanes == 2 ? launch_prefill_tc<2, KP_, VP_, true>(tq, tk, tv, p, pdl, st)   \
                     : launch_prefill_tc<1, KP_, VP_, true>(tq, tk, tv, p, pdl, st)
-  if (dk > 64) { if (dv > 64) RB_FPS(2, 2); RB_FPS(2, 1); }
-  if (dv > 64) RB_FPS(1, 2);
+  if (dk > 64) {
+    if (dv > 64) { RB_FPS(2, 2); }
+    RB_FPS(2, 1);
+  }
+  if (dv > 64) { RB_FPS(1, 2); }
   RB_FPS(1, 1);
 #undef RB_FPS
 }

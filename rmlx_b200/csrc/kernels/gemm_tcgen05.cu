@@ -360,12 +360,14 @@ extern "C" int rmlx_gemm_bf16_f32(const void* A, const void* W, void* C, int M, 
                                   int ldw, int ldc, int* status, int pdl, cudaStream_t st) {
   if (M < 1 || N < 1 || K < 8 || K % 8 || lda % 8 || ldw % 8) return -2;
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) return -2;
-  const int bn = rmlx_gemm_pick_bn(M, N) >= 128 ? 128 : 64;
+  int bn = rmlx_gemm_pick_bn(M, N);
+  if (bn < 64) bn = 64;
   CUtensorMap ta, tw;
   int rc = make_tmap_2d_bf16(&ta, A, uint64_t(K), uint64_t(M), uint64_t(lda) * 2, kBK, kBM);
   if (rc) return rc;
   rc = make_tmap_2d_bf16(&tw, W, uint64_t(K), uint64_t(N), uint64_t(ldw) * 2, kBK, bn);
   if (rc) return rc;
+  if (bn == 256) return launch_gemm<256, kEpiF32>(ta, tw, C, nullptr, M, N, K, ldc, status, pdl, st);
   if (bn == 128) return launch_gemm<128, kEpiF32>(ta, tw, C, nullptr, M, N, K, ldc, status, pdl, st);
   return launch_gemm<64, kEpiF32>(ta, tw, C, nullptr, M, N, K, ldc, status, pdl, st);
 }

@@ -9,16 +9,20 @@ namespace rb {
 
 constexpr int kHgRows = 4;          // rows of the batch per block
 constexpr int kHgWarps = 8;
-constexpr int kHgTile = 64;         // output channels per block
 
-template <class T, int L>
+// TILE: output channels per block (few rows: small tiles, so that the weights come from many SMs at once).
+template <class T, int L, int TILE>
 __global__ void __launch_bounds__(kHgWarps * 32)
 head_gemv_kernel(const T* __restrict__ w, const T* __restrict__ in, int in_t, int in_h, T* __restrict__ out, int out_t,
                  int out_h, const int* __restrict__ row_ids, int rows, int N, int K) {
   extern __shared__ __align__(16) float xs[];       // [kHgRows][2][K / 2]: first and second halves of the chunks
-  const int h = blockIdx.y, n0 = blockIdx.x * kHgTile, t0 = blockIdx.z * kHgRows;
+  const int h = blockIdx.y, n0 = blockIdx.x * TILE, t0 = blockIdx.z * kHgRows;
   const int nt = min(kHgRows, rows - t0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, chunks = K >> 3;
+  constexpr int PER = 32 / L;                        // weight rows a warp holds at once
+  const int sub = lane / L, sl = lane % L;
+  float f0[8];                                       // weights wait for nothing: the first chunk is asked for at once
+  load8(w + (size_t(h) * N + min(n0 + warp * PER + sub, N - 1)) * K + min(sl, chunks - 1) * 8, f0);
   pdl_launch_dependents();
   pdl_wait();
   for (int i = threadIdx.x; i < kHgRows * chunks; i += kHgWarps * 32) {
@@ -33,15 +37,18 @@ head_gemv_kernel(const T* __restrict__ w, const T* __restrict__ in, int in_t, in
     d[chunks + c] = make_float4(f[4], f[5], f[6], f[7]);
   }
   __syncthreads();
-  constexpr int PER = 32 / L;                        // weight rows a warp holds at once
-  const int sub = lane / L, sl = lane % L;
-  for (int r = warp * PER + sub; r < kHgTile; r += kHgWarps * PER) {
+  for (int r = warp * PER + sub; r < TILE; r += kHgWarps * PER) {
     const int n = n0 + r;                            // the lanes of a row leave the loop together with their warp
     const T* row = w + (size_t(h) * N + min(n, N - 1)) * K;
     float acc[kHgRows] = {0.f, 0.f, 0.f, 0.f};
     for (int c = sl; c < chunks; c += L) {
       float f[8];
-      load8(row + c * 8, f);
+      if (r == warp * PER + sub && c == sl) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = f0[i];
+      } else {
+        load8(row + c * 8, f);
+      }
 #pragma unroll
       for (int b = 0; b < kHgRows; ++b) {
         const float4* d = reinterpret_cast<const float4*>(xs + b * K);
@@ -66,20 +73,19 @@ head_gemv_kernel(const T* __restrict__ w, const T* __restrict__ in, int in_t, in
   }
 }
 
-template <class T>
+template <class T, int TILE>
 static int launch_head_gemv(const T* w, const T* in, int in_t, int in_h, T* out, int out_t, int out_h,
                             const int* row_ids, int rows, int H, int N, int K, int pdl, cudaStream_t st) {
-  const dim3 grid((N + kHgTile - 1) / kHgTile, H, (rows + kHgRows - 1) / kHgRows);
+  const dim3 grid((N + TILE - 1) / TILE, H, (rows + kHgRows - 1) / kHgRows);
   const size_t smem = size_t(kHgRows) * K * sizeof(float);
   auto go = [&](auto kern) -> int {
     RB_CHECK(set_max_smem(kern, smem));
     return launch(kern, grid, dim3(kHgWarps * 32), smem, st, pdl != 0, w, in, in_t, in_h, out, out_t, out_h, row_ids,
                   rows, N, K);
   };
-  if (K <= 32) return go(head_gemv_kernel<T, 4>);
-  if (K <= 64) return go(head_gemv_kernel<T, 8>);
-  if (K <= 128) return go(head_gemv_kernel<T, 16>);
-  return go(head_gemv_kernel<T, 32>);
+  if (K <= 64) return go(head_gemv_kernel<T, 8, TILE>);
+  if (K <= 128) return go(head_gemv_kernel<T, 16, TILE>);
+  return go(head_gemv_kernel<T, 32, TILE>);
 }
 
 }  // namespace rb
@@ -93,9 +99,11 @@ extern "C" int rmlx_head_gemv(const void* w, const void* in, int in_t, int in_h,
   if (rows < 1 || (rows + kHgRows - 1) / kHgRows > 65535 || H < 1 || H > 65535 || N < 1 || K < 8 || K % 8 || in_t % 8 ||
       in_h % 8 || K > 8192)
     return -2;
-  if (f32)
-    return launch_head_gemv(static_cast<const float*>(w), static_cast<const float*>(in), in_t, in_h,
-                            static_cast<float*>(out), out_t, out_h, row_ids, rows, H, N, K, pdl, st);
-  return launch_head_gemv(static_cast<const __nv_bfloat16*>(w), static_cast<const __nv_bfloat16*>(in), in_t, in_h,
-                          static_cast<__nv_bfloat16*>(out), out_t, out_h, row_ids, rows, H, N, K, pdl, st);
+#define RB_HG(T_, TILE_)                                                                                            \
+  return launch_head_gemv<T_, TILE_>(static_cast<const T_*>(w), static_cast<const T_*>(in), in_t, in_h,            \
+                                     static_cast<T_*>(out), out_t, out_h, row_ids, rows, H, N, K, pdl, st)
+  if (f32) RB_HG(float, 64);
+  if (rows <= 2 * kHgRows) RB_HG(__nv_bfloat16, 32);
+  RB_HG(__nv_bfloat16, 64);
+#undef RB_HG
 }

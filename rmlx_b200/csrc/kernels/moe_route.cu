@@ -61,7 +61,7 @@ route_scatter_kernel(const T* __restrict__ x, int ldx, const int* __restrict__ i
     row_of_pair[p] = row;
   }
   row = __shfl_sync(0xffffffffu, row, 0);
-  if (row < 0 || !RB_BOUNDS(row, pairs)) return;
+  if (row < 0 || row >= pairs) return;              // (row >= pairs: cursors that belong to another choice)
   const uint4* src = reinterpret_cast<const uint4*>(x + size_t(p / top_k) * ldx);
   uint4* dst = reinterpret_cast<uint4*>(xs + size_t(row) * ldx);
   const int units = ldx * int(sizeof(T)) / 16;

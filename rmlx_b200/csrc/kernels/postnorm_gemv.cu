@@ -111,10 +111,10 @@ __device__ __forceinline__ void stage_post_norm(const PostNormIn& in, int b, cha
   }
 }
 
-// GATED: N counts output columns, W has 2 N rows (gate then up). One tile of rows per warp: the grid
-// covers N (a block's rows then belong to one shift segment).
+// GATED: N counts output columns, W has 2 N rows (gate then up). Blocks stay and walk the rows (the norm and
+// the staging are paid once per block); grid y: the shift segment whose rows a block takes.
 template <int B, bool GATED>
-__global__ void __launch_bounds__(kGemvThreads)
+__global__ void __launch_bounds__(kGemvThreads, 2)
 postnorm_in_kernel(Matrix<WBf16> W, PostNormIn in, ShiftIn sh, float* __restrict__ out, int ld_out,
                    __nv_bfloat16* __restrict__ act, int ld_act, int N, float limit) {
   extern __shared__ __align__(16) char smem[];
@@ -122,10 +122,12 @@ postnorm_in_kernel(Matrix<WBf16> W, PostNormIn in, ShiftIn sh, float* __restrict
   constexpr int R = GATED ? 2 * kPnRows : kPnRows;
   const int K = W.K, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const size_t bstride = XStage<WBf16>::bytes(K);
-  const int n0 = (blockIdx.x * kGemvWarps + warp) * kPnRows;
+  const int seg = blockIdx.y, n_lo = sh.mu ? seg * sh.seg_rows : 0, n_hi = sh.mu && seg < 4 ? n_lo + sh.seg_rows : N;
+  int n0 = n_lo + (blockIdx.x * kGemvWarps + warp) * kPnRows;
+  if (n_lo + int(blockIdx.x) * kGemvWarps * kPnRows >= n_hi) return;        // a short segment
   RowBf16 rows[R];
   Tile<RowBf16, R> t0;
-  if (n0 < N) {                 // weights wait for nothing: ask for the first tile at once
+  auto point = [&]() {
 #pragma unroll
     for (int r = 0; r < kPnRows; ++r) {
       const int n = min(n0 + r, N - 1);
@@ -133,37 +135,40 @@ postnorm_in_kernel(Matrix<WBf16> W, PostNormIn in, ShiftIn sh, float* __restrict
       if (GATED) rows[kPnRows + r] = W.row(size_t(N) + n);
     }
     load_tile<R>(rows, K, 0, t0);
-  }
+  };
+  if (n0 < n_hi) point();       // weights wait for nothing: ask for the first tile at once
   pdl_launch_dependents();
   pdl_wait();
-  const float* mu = nullptr;
-  if (sh.mu) mu = sh.mu + size_t(min(blockIdx.x * kGemvWarps * kPnRows / sh.seg_rows, 4)) * in.ldx;
+  const float* mu = sh.mu ? sh.mu + size_t(seg) * in.ldx : nullptr;
 #pragma unroll
   for (int b = 0; b < B; ++b)
-    stage_post_norm(in, b, smem + b * bstride, red, blockIdx.x == 0, mu, mu ? sh.prev + sh.slots[b] * sh.stride : nullptr);
+    stage_post_norm(in, b, smem + b * bstride, red, blockIdx.x == 0 && seg == 0, mu,
+                    mu ? sh.prev + sh.slots[b] * sh.stride : nullptr);
   __syncthreads();
-  if (n0 >= N) return;
-  float acc[R][B];
+  for (bool first = true; n0 < n_hi; n0 += gridDim.x * kGemvWarps * kPnRows, first = false) {
+    if (!first) point();
+    float acc[R][B];
 #pragma unroll
-  for (int r = 0; r < R; ++r)
+    for (int r = 0; r < R; ++r)
 #pragma unroll
-    for (int b = 0; b < B; ++b) acc[r][b] = 0.f;
-  warp_dot<R, B, RowBf16>(rows, smem, bstride, K, acc, t0);
+      for (int b = 0; b < B; ++b) acc[r][b] = 0.f;
+    warp_dot<R, B, RowBf16>(rows, smem, bstride, K, acc, t0);
 #pragma unroll
-  for (int r = 0; r < kPnRows; ++r)
+    for (int r = 0; r < kPnRows; ++r)
 #pragma unroll
-    for (int b = 0; b < B; ++b) {
-      const float v = warp_sum(acc[r][b]);
-      const float u = GATED ? warp_sum(acc[GATED ? kPnRows + r : r][b]) : 0.f;
-      const int n = n0 + r;
-      if (lane == r * B + b && n < N) {
-        if (GATED) act[size_t(b) * ld_act + n] = __float2bfloat16_rn(gated_act_fast(v, u, limit));
-        else out[size_t(b) * ld_out + n] = v;
+      for (int b = 0; b < B; ++b) {
+        const float v = warp_sum(acc[r][b]);
+        const float u = GATED ? warp_sum(acc[GATED ? kPnRows + r : r][b]) : 0.f;
+        const int n = n0 + r;
+        if (lane == r * B + b && n < n_hi) {
+          if (GATED) act[size_t(b) * ld_act + n] = __float2bfloat16_rn(gated_act_fast(v, u, limit));
+          else out[size_t(b) * ld_out + n] = v;
+        }
       }
-    }
+  }
 }
 
-// One warp per router output; the last block to arrive chooses for every token.
+// One block per router output, its warps share the row; the last block to arrive chooses for every token.
 template <int B>
 __global__ void __launch_bounds__(kGemvThreads)
 postnorm_router_kernel(Matrix<WBf16> W, PostNormIn in, const float* __restrict__ correction, float* __restrict__ logits,
@@ -171,28 +176,59 @@ postnorm_router_kernel(Matrix<WBf16> W, PostNormIn in, const float* __restrict__
                        unsigned int* __restrict__ ticket, int experts, int outputs, int top_k) {
   extern __shared__ __align__(16) char smem[];
   __shared__ float red[kGemvWarps];
+  __shared__ float part[kGemvWarps][B];
   __shared__ unsigned int last;
-  const int K = W.K, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int K = W.K, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, chunks = K >> 3;
   const size_t bstride = XStage<WBf16>::bytes(K);
-  const int n = blockIdx.x * kGemvWarps + warp;
-  RowBf16 rows[1] = {W.row(min(n, outputs - 1))};
-  Tile<RowBf16, 1> t0;
-  load_tile<1>(rows, K, 0, t0);
+  const int n = blockIdx.x;
+  const __nv_bfloat16* row = W.w + size_t(n) * K;
+  constexpr int kKeep = 4;
+  uint4 wv[kKeep];
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int c = u * kGemvThreads + threadIdx.x;
+    wv[u] = c < chunks ? ldg_stream(row + (size_t(c) << 3)) : make_uint4(0u, 0u, 0u, 0u);
+  }
   pdl_launch_dependents();
   pdl_wait();
 #pragma unroll
-  for (int b = 0; b < B; ++b) stage_post_norm(in, b, smem + b * bstride, red, blockIdx.x == 0, nullptr, nullptr);
+  for (int b = 0; b < B; ++b) stage_post_norm(in, b, smem + b * bstride, red, n == 0, nullptr, nullptr);
   __syncthreads();
-  float acc[1][B];
+  float acc[B];
 #pragma unroll
-  for (int b = 0; b < B; ++b) acc[0][b] = 0.f;
-  warp_dot<1, B, RowBf16>(rows, smem, bstride, K, acc, t0);
+  for (int b = 0; b < B; ++b) acc[b] = 0.f;
+  auto dot = [&](int c, const uint4& w) {
+#pragma unroll
+    for (int b = 0; b < B; ++b) {
+      const float4* xs = reinterpret_cast<const float4*>(smem + b * bstride);
+      const float4 x0 = xs[c], x1 = xs[chunks + c];
+      float a = acc[b];
+      a = fmaf(bf16lo(w.x), x0.x, a); a = fmaf(bf16hi(w.x), x0.y, a);
+      a = fmaf(bf16lo(w.y), x0.z, a); a = fmaf(bf16hi(w.y), x0.w, a);
+      a = fmaf(bf16lo(w.z), x1.x, a); a = fmaf(bf16hi(w.z), x1.y, a);
+      a = fmaf(bf16lo(w.w), x1.z, a); a = fmaf(bf16hi(w.w), x1.w, a);
+      acc[b] = a;
+    }
+  };
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int c = u * kGemvThreads + threadIdx.x;
+    if (c < chunks) dot(c, wv[u]);
+  }
+  for (int c = kKeep * kGemvThreads + threadIdx.x; c < chunks; c += kGemvThreads) dot(c, ldg_stream(row + (size_t(c) << 3)));
 #pragma unroll
   for (int b = 0; b < B; ++b) {
-    const float v = warp_sum(acc[0][b]);
-    if (lane == 0 && n < outputs) logits[size_t(b) * outputs + n] = v;
+    const float v = warp_sum(acc[b]);
+    if (lane == 0) part[warp][b] = v;
   }
-  __threadfence();
+  __syncthreads();
+  if (threadIdx.x < B) {
+    float v = 0.f;
+#pragma unroll
+    for (int q = 0; q < kGemvWarps; ++q) v += part[q][threadIdx.x];
+    logits[size_t(threadIdx.x) * outputs + n] = v;
+    __threadfence();
+  }
   __syncthreads();
   if (threadIdx.x == 0) last = (atomicAdd(ticket, 1u) == gridDim.x - 1) ? 1u : 0u;
   __syncthreads();
@@ -200,10 +236,10 @@ postnorm_router_kernel(Matrix<WBf16> W, PostNormIn in, const float* __restrict__
     __threadfence();
     for (int b = warp; b < B; b += kGemvWarps) {
       // through L2: other blocks wrote the logits
-      float* row = reinterpret_cast<float*>(smem) + b * outputs;
-      for (int i = lane; i < outputs; i += 32) row[i] = __ldcg(logits + size_t(b) * outputs + i);
+      float* z = reinterpret_cast<float*>(smem) + b * outputs;
+      for (int i = lane; i < outputs; i += 32) z[i] = __ldcg(logits + size_t(b) * outputs + i);
       __syncwarp();
-      warp_route_corrected(row, correction, experts, outputs, top_k, idx + size_t(b) * top_k, weights + size_t(b) * top_k,
+      warp_route_corrected(z, correction, experts, outputs, top_k, idx + size_t(b) * top_k, weights + size_t(b) * top_k,
                            identity + b, nullptr);
     }
     if (threadIdx.x == 0) *ticket = 0u;
@@ -356,64 +392,80 @@ matvec_out_kernel(Matrix<WBf16> W, const __nv_bfloat16* __restrict__ a, int ld_a
     }
 }
 
-// raw row b = [r | k | v | g: `inner` values apart | low: rank]. One block per (head, row).
+// raw row b = [r | k | v | g: `inner` values apart | low: rank]. One block per (head, row). ROWS: state rows a
+// thread holds; they belong to this kernel alone within a step, so they are asked for before the wait (the
+// step's first kernel has waited for everything before it).
+template <int ROWS>
 __global__ void __launch_bounds__(256)
 wkv_decode_kernel(const float* __restrict__ raw, int ld_raw, int inner, const __nv_bfloat16* __restrict__ w2, int rank,
                   const float* __restrict__ w0, const float* __restrict__ u, const float* __restrict__ norm, float eps,
                   const int* __restrict__ slots, float* __restrict__ state, float* __restrict__ prev, long long stride,
                   const float* __restrict__ x, int ldx, __nv_bfloat16* __restrict__ a, int ld_a, int dim, int dim_pad) {
   extern __shared__ float sm[];
-  float* sr = sm;                    // [dim] r, k, decay
-  float* sk = sr + dim;
-  float* sw = sk + dim;
-  float* low = sw + dim;             // [rank] tanh
-  float* part = low + rank;          // [256 / dim_pad][dim_pad]
+  float* sr = sm;                    // [dim_pad] r, k, decay
+  float* sk = sr + dim_pad;
+  float* sw = sk + dim_pad;
+  float* low = sw + dim_pad;         // [rank] tanh
+  float* part = low + rank;          // [256]
   __shared__ float red[8];
-  pdl_launch_dependents();
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
-  pdl_wait();
-  const float* row = raw + size_t(b) * ld_raw;
   const int slot = slots[b];
   // the column this thread works on and its group's share of the rows
   const int groups = 256 / dim_pad, g = tid / dim_pad, col = tid - g * dim_pad;
   const int per = (dim + groups - 1) / groups, i0 = g * per, i1 = min(i0 + per, dim);
+  float* sp = state + size_t(slot) * stride + size_t(h) * dim * dim + col;
+  float s[ROWS];
+#pragma unroll
+  for (int q = 0; q < ROWS; ++q) s[q] = (col < dim && i0 + q < i1) ? __ldcg(sp + size_t(i0 + q) * dim) : 0.f;
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* row = raw + size_t(b) * ld_raw;
   for (int i = tid; i < rank; i += 256) low[i] = tanhf(__ldcg(row + 4 * inner + i));
   float ruk = 0.f;
-  for (int i = tid; i < dim; i += 256) {
-    const float r = __ldcg(row + h * dim + i), k = __ldcg(row + inner + h * dim + i);
-    sr[i] = r;
-    sk[i] = k;
-    ruk = fmaf(r * u[h * dim + i], k, ruk);
+  if (tid < dim) {
+    const float r = __ldcg(row + h * dim + tid), k = __ldcg(row + inner + h * dim + tid);
+    sr[tid] = r;
+    sk[tid] = k;
+    ruk = r * u[h * dim + tid] * k;
   }
-  ruk = block_sum_256(ruk, red);     // low, sr and sk are visible, too
-  for (int i = tid; i < dim; i += 256) {
-    const __nv_bfloat16* wr = w2 + size_t(h * dim + i) * rank;
-    float d = w0[h * dim + i];
-    for (int j = 0; j < rank; j += 8) {
-      const uint4 q = *reinterpret_cast<const uint4*>(wr + j);
-      d = fmaf(bf16lo(q.x), low[j], d); d = fmaf(bf16hi(q.x), low[j + 1], d);
-      d = fmaf(bf16lo(q.y), low[j + 2], d); d = fmaf(bf16hi(q.y), low[j + 3], d);
-      d = fmaf(bf16lo(q.z), low[j + 4], d); d = fmaf(bf16hi(q.z), low[j + 5], d);
-      d = fmaf(bf16lo(q.w), low[j + 6], d); d = fmaf(bf16hi(q.w), low[j + 7], d);
-    }
-    sw[i] = expf(-expf(d));
-  }
-  __syncthreads();
   const float v = col < dim ? __ldcg(row + 2 * inner + h * dim + col) : 0.f;
+  ruk = block_sum_256(ruk, red);     // low, sr and sk are visible, too
+  {                                  // decay of row `col`, the rank's chunks dealt to the groups
+    float d = 0.f;
+    if (col < dim) {
+      const __nv_bfloat16* wr = w2 + size_t(h * dim + col) * rank;
+      for (int j = g * 8; j < rank; j += groups * 8) {
+        const uint4 q = *reinterpret_cast<const uint4*>(wr + j);
+        d = fmaf(bf16lo(q.x), low[j], d); d = fmaf(bf16hi(q.x), low[j + 1], d);
+        d = fmaf(bf16lo(q.y), low[j + 2], d); d = fmaf(bf16hi(q.y), low[j + 3], d);
+        d = fmaf(bf16lo(q.z), low[j + 4], d); d = fmaf(bf16hi(q.z), low[j + 5], d);
+        d = fmaf(bf16lo(q.w), low[j + 6], d); d = fmaf(bf16hi(q.w), low[j + 7], d);
+      }
+    }
+    part[tid] = d;
+    __syncthreads();
+    if (tid < dim) {
+      d = w0[h * dim + tid];
+      for (int q = 0; q < groups; ++q) d += part[q * dim_pad + tid];
+      sw[tid] = expf(-expf(d));
+    }
+    __syncthreads();
+  }
   float o = 0.f;
-  if (col < dim && g < groups) {
-    float* sp = state + size_t(slot) * stride + size_t(h) * dim * dim + col;
-#pragma unroll 8
-    for (int i = i0; i < i1; ++i) {
-      const float s = sp[size_t(i) * dim];
-      o = fmaf(sr[i], s, o);
-      sp[size_t(i) * dim] = fmaf(sw[i], s, sk[i] * v);
+  if (col < dim) {
+#pragma unroll
+    for (int q = 0; q < ROWS; ++q) {
+      const int i = i0 + q;
+      if (i < i1) {
+        o = fmaf(sr[i], s[q], o);
+        sp[size_t(i) * dim] = fmaf(sw[i], s[q], sk[i] * v);
+      }
     }
   }
-  if (g < groups) part[g * dim_pad + col] = o;
+  part[tid] = o;
   __syncthreads();
   float ssq = 0.f;
-  if (tid < dim) {
+  if (tid < dim) {                   // tid is this thread's column
     o = ruk * v;
     for (int q = 0; q < groups; ++q) o += part[q * dim_pad + tid];
     ssq = o * o;
@@ -458,7 +510,13 @@ static int launch_in(const void* w, const PostNormIn& in, const ShiftIn& sh, flo
   const size_t smem = XStage<WBf16>::bytes(in.ldx) * B;
   auto kern = postnorm_in_kernel<B, GATED>;
   RB_CHECK(set_max_smem(kern, smem));
-  return launch(kern, dim3(pn_grid(N)), dim3(kGemvThreads), smem, st, pdl != 0,
+  // as many blocks as stay resident, the rows spread evenly over them
+  int per_sm = 1;
+  RB_CHECK(cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, kern, kGemvThreads, smem));
+  const int segs = sh.mu ? 5 : 1, longest = sh.mu ? sh.seg_rows : N;
+  const int cap = sm_count() * (per_sm > 0 ? per_sm : 1) / (sh.mu ? 4 : 1), tiles = pn_grid(longest);
+  const int passes = (tiles + cap - 1) / cap;
+  return launch(kern, dim3((tiles + passes - 1) / passes, segs), dim3(kGemvThreads), smem, st, pdl != 0,
                 Matrix<WBf16>{static_cast<const __nv_bfloat16*>(w), in.ldx}, in, sh, out, ld_out,
                 static_cast<__nv_bfloat16*>(act), ld_act, N, limit);
 }
@@ -497,7 +555,7 @@ static int launch_router(const void* w, const PostNormIn& in, const float* corre
   if (smem < size_t(B) * outputs * 4) smem = size_t(B) * outputs * 4;
   auto kern = postnorm_router_kernel<B>;
   RB_CHECK(set_max_smem(kern, smem));
-  return launch(kern, dim3((outputs + kGemvWarps - 1) / kGemvWarps), dim3(kGemvThreads), smem, st, pdl != 0,
+  return launch(kern, dim3(outputs), dim3(kGemvThreads), smem, st, pdl != 0,
                 Matrix<WBf16>{static_cast<const __nv_bfloat16*>(w), in.ldx}, in, correction, logits, idx, weights, identity,
                 ticket, experts, outputs, top_k);
 }
@@ -565,13 +623,20 @@ extern "C" int rmlx_wkv_decode(const float* raw, int ld_raw, int inner, const vo
                                long long stride, const float* x, int ldx, void* a, int ld_a, int B, int H, int dim, int pdl,
                                cudaStream_t st) {
   if (B < 1 || B > 65535 || H < 1 || dim < 1 || dim > 256 || inner < H * dim || rank < 8 || rank % 8 ||
-      ld_raw < 4 * inner + rank || ld_a < H * dim || !slots || rank > 4096)
+      ld_raw < 4 * inner + rank || ld_a < H * dim || !slots || rank > 4096 || w2 == nullptr)
     return -2;
   int dim_pad = 8;
   while (dim_pad < dim) dim_pad *= 2;
-  const size_t smem = size_t(3 * dim + rank + 256) * sizeof(float);
-  RB_CHECK(set_max_smem(wkv_decode_kernel, smem));
-  return launch(wkv_decode_kernel, dim3(H, B), dim3(256), smem, st, pdl != 0, raw, ld_raw, inner,
-                static_cast<const __nv_bfloat16*>(w2), rank, w0, u, norm, eps, slots, state, prev, stride, x, ldx,
-                static_cast<__nv_bfloat16*>(a), ld_a, dim, dim_pad);
+  const size_t smem = size_t(3 * dim_pad + rank + 256) * sizeof(float);
+  const int groups = 256 / dim_pad, per = (dim + groups - 1) / groups;
+  auto go = [&](auto kern) -> int {
+    RB_CHECK(set_max_smem(kern, smem));
+    return launch(kern, dim3(H, B), dim3(256), smem, st, pdl != 0, raw, ld_raw, inner,
+                  static_cast<const __nv_bfloat16*>(w2), rank, w0, u, norm, eps, slots, state, prev, stride, x, ldx,
+                  static_cast<__nv_bfloat16*>(a), ld_a, dim, dim_pad);
+  };
+  if (per <= 4) return go(wkv_decode_kernel<4>);
+  if (per <= 16) return go(wkv_decode_kernel<16>);
+  if (per <= 64) return go(wkv_decode_kernel<64>);
+  return go(wkv_decode_kernel<256>);
 }

@@ -60,14 +60,24 @@ struct ExpertSource {
   __device__ __forceinline__ void load(int t, int c, const float (&x)[8], float (&f)[8]) const {
 #pragma unroll
     for (int i = 0; i < 8; ++i) f[i] = id_w * x[i];
-    for (int s = 0; s < top_k; ++s) {
-      const int row = row_of_pair[t * top_k + s];
-      if (row < 0) continue;
-      const float a = weights[t * top_k + s];
-      float g[8];
-      load8(y + size_t(row) * ldy + c * 8, g);
+    for (int s0 = 0; s0 < top_k; s0 += 4) {            // four slots' rows in flight
+      float g[4][8], a[4];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = fmaf(a, g[i], f[i]);
+      for (int u = 0; u < 4; ++u) {
+        const int p = t * top_k + min(s0 + u, top_k - 1);
+        const int row = s0 + u < top_k ? row_of_pair[p] : -1;
+        a[u] = row >= 0 ? weights[p] : 0.f;
+        if (row >= 0) {
+          load8(y + size_t(row) * ldy + c * 8, g[u]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) g[u][i] = 0.f;
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = fmaf(a[u], g[u][i], f[i]);
     }
   }
 };
@@ -77,7 +87,7 @@ template <class SRC, class T>
 __global__ void __launch_bounds__(kRowThreads)
 post_norm_add_kernel(SRC src, const float* __restrict__ w, float eps, float* __restrict__ x, T* __restrict__ h,
                      int D, int ldx) {
-  constexpr int kKeep = 4;                 // chunks of eight a thread keeps in registers
+  constexpr int kKeep = 2;                 // chunks of eight a thread keeps in registers
   __shared__ float red[kRowThreads / 32];
   pdl_launch_dependents();
   pdl_wait();
@@ -129,17 +139,10 @@ post_norm_add_kernel(SRC src, const float* __restrict__ w, float eps, float* __r
   }
 }
 
-template <class TR>
-__device__ __forceinline__ void load8_upto(const TR* p, int n, bool aligned, float (&f)[8]) {
-  if (aligned) { load8(p, f); return; }
-#pragma unroll
-  for (int i = 0; i < 8; ++i) f[i] = i < n ? to_f32(p[i]) : 0.f;
-}
-
 // raw row t = [q: Hq*dim | k: Hkv*dim | v: Hkv*vdim | ..]. Every query and key head is divided by its
 // own root mean square and multiplied by q_w / k_w [dim]; q goes to q_out [T, Hq, dkp], k and v to the
-// token's slot of its sequence's pages. One warp per head.
-template <class TR, class T>
+// token's slot of its sequence's pages. L lanes per head.
+template <class TR, class T, int L>
 __global__ void __launch_bounds__(kRowThreads)
 head_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restrict__ q_w,
                         const float* __restrict__ k_w, float eps, T* __restrict__ q_out,
@@ -148,46 +151,53 @@ head_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __re
                         int Hkv, int dim, int vdim, int dkp, int dvp, int max_blocks, int page) {
   pdl_launch_dependents();
   pdl_wait();
-  const int per = Hq + 2 * Hkv;
-  const int unit = blockIdx.x * (kRowThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (unit >= rows * per) return;
-  const int t = unit / per, r = unit - t * per;
+  const int per = Hq + 2 * Hkv, units = rows * per;
+  const int unit = (blockIdx.x * kRowThreads + threadIdx.x) / L, lane = threadIdx.x % L;
+  const bool live = unit < units;                      // the lanes of a warp stay together for the sums
+  const int t = live ? unit / per : 0, r = live ? unit - t * per : 0;
   const bool is_q = r < Hq, is_v = r >= Hq + Hkv;
   const int head = is_q ? r : is_v ? r - Hq - Hkv : r - Hq;
   const int width = is_v ? vdim : dim, padded = is_v ? dvp : dkp;
   const int src0 = is_q ? head * dim : is_v ? (Hq + Hkv) * dim + head * vdim : (Hq + head) * dim;
   const TR* src = raw + size_t(t) * ldraw + src0;
   const bool vec = width % 8 == 0 && src0 % 8 == 0 && ldraw % 8 == 0;
-  T* dst;
+  T* dst = nullptr;
   if (is_q) {
     dst = q_out + (size_t(t) * Hq + head) * dkp;
   } else {
     const int pos = positions[t];
-    if (!RB_BOUNDS(pos / page, max_blocks)) return;
-    const int seq = token_seq ? token_seq[t] : t;
-    const int blk = block_table[size_t(seq) * max_blocks + pos / page];
-    dst = (is_v ? v_cache : k_cache) + ((size_t(blk) * Hkv + head) * page + pos % page) * padded;
-  }
-  float inv = 1.f;
-  if (!is_v) {
-    float ssq = 0.f;
-    for (int d0 = lane * 8; d0 < dim; d0 += 256) {
-      float f[8];
-      load8_upto(src + d0, dim - d0, vec, f);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) ssq += f[i] * f[i];
+    if (RB_BOUNDS(pos / page, max_blocks)) {
+      const int seq = token_seq ? token_seq[t] : t;
+      const int blk = block_table[size_t(seq) * max_blocks + pos / page];
+      dst = (is_v ? v_cache : k_cache) + ((size_t(blk) * Hkv + head) * page + pos % page) * padded;
     }
-    inv = 1.f / sqrtf(warp_sum(ssq) / float(dim) + eps);
   }
-  const float* w = is_q ? q_w : k_w;
-  for (int d0 = lane * 8; d0 < padded; d0 += 256) {
+  float first[8], ssq = 0.f;
+  load8_upto(src + lane * 8, width - lane * 8, vec && lane * 8 < width, first);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ssq += first[i] * first[i];
+  for (int d0 = (lane + L) * 8; d0 < width; d0 += L * 8) {
     float f[8];
-    load8_upto(src + d0, width - d0, vec && d0 < width, f);
+    load8_upto(src + d0, width - d0, vec, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ssq += f[i] * f[i];
+  }
+  ssq = group_sum<L>(ssq);
+  if (!live || !dst) return;
+  const float inv = is_v ? 1.f : 1.f / sqrtf(ssq / float(dim) + eps);
+  const float* w = is_q ? q_w : k_w;
+  auto put = [&](int d0, float (&f)[8]) {
     if (!is_v) {
 #pragma unroll
       for (int i = 0; i < 8; ++i) f[i] = d0 + i < dim ? f[i] * inv * w[d0 + i] : 0.f;
     }
     store8(dst + d0, f);
+  };
+  if (lane * 8 < padded) put(lane * 8, first);
+  for (int d0 = (lane + L) * 8; d0 < padded; d0 += L * 8) {
+    float f[8];
+    load8_upto(src + d0, width - d0, vec && d0 < width, f);
+    put(d0, f);
   }
 }
 
@@ -195,7 +205,7 @@ head_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __re
 // [T, H, dimp + rotp] with their last `rot` values rotated (pairs (2i, 2i+1) of the first `dims` by
 // position * inv_freq[i]), the rotated part also behind the latent part of q_abs [T, H, latp + rotp]
 // when that is given. The latent is divided by its root mean square, times c_w; it and the rotated
-// shared key part form the token's cache row [latp | rotp | ..] of `ldc` elements. One block per token.
+// shared key part form the token's cache row [latp | rotp | ..] of `ldc` elements. One block per token, or (grid y) several.
 template <class TR, class T>
 __global__ void __launch_bounds__(kRowThreads)
 latent_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restrict__ c_w, float eps,
@@ -220,37 +230,49 @@ latent_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restr
   }
   ssq = row_block_sum(ssq, red);           // the angles are in shared memory, too
   const float inv = 1.f / sqrtf(ssq / float(rank) + eps);
-  auto rotated = [&](const TR* p, int i) {   // value i of a rotated vector
-    const float a = to_f32(p[i]);
-    if (i >= dims) return a;
-    const float b = to_f32(p[i ^ 1]), c = trig[i >> 1], s = trig[dims / 2 + (i >> 1)];
-    return i & 1 ? fmaf(a, c, b * s) : fmaf(a, c, -b * s);
+  const bool vec = dim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && ldraw % 8 == 0;
+  // values i0 .. i0 + 7 of a vector whose first `dims` values turn
+  auto rotate = [&](int i0, float (&f)[8]) {
+#pragma unroll
+    for (int i = 0; i < 8; i += 2)
+      if (i0 + i < dims) {
+        const float c = trig[(i0 + i) >> 1], s = trig[dims / 2 + ((i0 + i) >> 1)], u = f[i], v = f[i + 1];
+        f[i] = fmaf(u, c, -v * s);
+        f[i + 1] = fmaf(v, c, u * s);
+      }
   };
-  const int wq = dimp + rotp;
-  for (int u = threadIdx.x; u < H * wq; u += kRowThreads) {
-    const int h = u / wq, i = u - h * wq;
-    const TR* p = row + h * (dim + rot);
-    float v = 0.f;
-    if (i < dimp) {
-      if (i < dim) v = to_f32(p[i]);
-    } else {
-      if (i - dimp < rot) v = rotated(p + dim, i - dimp);
-      if (q_abs) q_abs[(size_t(t) * H + h) * (latp + rotp) + latp + (i - dimp)] = from_f32<T>(v);
-    }
-    q_out[size_t(t) * H * wq + u] = from_f32<T>(v);
-  }
-  if (!RB_BOUNDS(pos / page, max_blocks)) return;
   const int seq = token_seq ? token_seq[t] : t;
-  const int blk = block_table[size_t(seq) * max_blocks + pos / page];
-  T* dst = cache + (size_t(blk) * page + pos % page) * ldc;
-  for (int i = threadIdx.x; i < latp + rotp; i += kRowThreads) {
-    float v = 0.f;
-    if (i < latp) {
-      if (i < rank) v = to_f32(down[i]) * inv * c_w[i];
-    } else if (i - latp < rot) {
-      v = rotated(down + rank, i - latp);
+  const bool in_table = RB_BOUNDS(pos / page, max_blocks);
+  const int blk = in_table ? block_table[size_t(seq) * max_blocks + pos / page] : 0;
+  T* cdst = cache + (size_t(blk) * page + pos % page) * ldc;
+  const int ud = dimp >> 3, uq = (dimp + rotp) >> 3, ul = latp >> 3, uc = (latp + rotp) >> 3;
+  for (int u = blockIdx.y * kRowThreads + threadIdx.x; u < H * uq + uc; u += gridDim.y * kRowThreads) {
+    float f[8];
+    if (u < H * uq) {                      // a query
+      const int h = u / uq, c = u - h * uq;
+      const TR* p = row + h * (dim + rot);
+      if (c < ud) {
+        load8_upto(p + c * 8, dim - c * 8, vec, f);
+      } else {
+        const int i0 = (c - ud) * 8;
+        load8_upto(p + dim + i0, rot - i0, vec, f);
+        rotate(i0, f);
+        if (q_abs) store8(q_abs + (size_t(t) * H + h) * (latp + rotp) + latp + i0, f);
+      }
+      store8(q_out + (size_t(t) * H + h) * (dimp + rotp) + c * 8, f);
+    } else if (in_table) {                 // the token's cache row
+      const int c = u - H * uq;
+      if (c < ul) {
+        load8_upto(down + c * 8, rank - c * 8, vec, f);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = c * 8 + i < rank ? f[i] * inv * c_w[c * 8 + i] : 0.f;
+      } else {
+        const int i0 = (c - ul) * 8;
+        load8_upto(down + rank + i0, rot - i0, vec, f);
+        rotate(i0, f);
+      }
+      store8(cdst + c * 8, f);
     }
-    dst[i] = from_f32<T>(v);
   }
 }
 
@@ -361,17 +383,25 @@ extern "C" int rmlx_head_norm_append(const void* raw, int ldraw, int raw_f32, co
       ldraw < (Hq + Hkv) * dim + Hkv * vdim || (f32 && !raw_f32))
     return -2;
   const long long units = 1LL * T * (Hq + 2 * Hkv);
-  if (units > 0x7fffffffLL) return -2;
-  const dim3 grid(unsigned((units + kRowThreads / 32 - 1) / (kRowThreads / 32)));
-#define RB_HN(TR_, T_)                                                                                            \
-  return launch(head_norm_append_kernel<TR_, T_>, grid, dim3(kRowThreads), 0, st, pdl != 0,                       \
+  if (units * 32 > 0x7fffffffLL) return -2;
+  const int widest = dkp > dvp ? dkp : dvp, lanes = widest <= 64 ? 8 : widest <= 128 ? 16 : 32;
+  const dim3 grid(unsigned((units * lanes + kRowThreads - 1) / kRowThreads));
+#define RB_HN_L(TR_, T_, L_)                                                                                      \
+  return launch(head_norm_append_kernel<TR_, T_, L_>, grid, dim3(kRowThreads), 0, st, pdl != 0,                   \
                 static_cast<const TR_*>(raw), ldraw, q_w, k_w, eps, static_cast<T_*>(q_out),                      \
                 static_cast<T_*>(k_cache), static_cast<T_*>(v_cache), block_table, positions, token_seq, T, Hq,   \
                 Hkv, dim, vdim, dkp, dvp, max_blocks, page)
+#define RB_HN(TR_, T_)                     \
+  {                                        \
+    if (lanes == 8) RB_HN_L(TR_, T_, 8);   \
+    if (lanes == 16) RB_HN_L(TR_, T_, 16); \
+    RB_HN_L(TR_, T_, 32);                  \
+  }
   if (f32) RB_HN(float, float);
   if (raw_f32) RB_HN(float, __nv_bfloat16);
   RB_HN(__nv_bfloat16, __nv_bfloat16);
 #undef RB_HN
+#undef RB_HN_L
 }
 
 // Types as above. dims: how many of the rotated part's values turn (even, <= rot); inv_freq fp32 [dims / 2].
@@ -385,8 +415,10 @@ extern "C" int rmlx_latent_append(const void* raw, int ldraw, int raw_f32, const
     return -2;
   const size_t smem = size_t(dims) * sizeof(float);
   if (smem > 32 * 1024) return -2;
+  const int work = (H * (dimp + rotp) + latp + rotp) / 8;            // few tokens: several blocks share one
+  const int split = T >= 64 ? 1 : (work + kRowThreads - 1) / kRowThreads;
 #define RB_LA(TR_, T_)                                                                                            \
-  return launch(latent_append_kernel<TR_, T_>, dim3(T), dim3(kRowThreads), smem, st, pdl != 0,                    \
+  return launch(latent_append_kernel<TR_, T_>, dim3(T, split), dim3(kRowThreads), smem, st, pdl != 0,                    \
                 static_cast<const TR_*>(raw), ldraw, c_w, eps, inv_freq, dims, static_cast<T_*>(q_out),           \
                 static_cast<T_*>(q_abs), static_cast<T_*>(cache), ldc, block_table, positions, token_seq, H, dim, \
                 rot, rank, dimp, rotp, latp, max_blocks, page)

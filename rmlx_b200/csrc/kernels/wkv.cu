@@ -116,61 +116,60 @@ __global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
   const bool stager = warp >= 4;
   const int chunks = (len + C::kChunk - 1) / C::kChunk;
 
-  auto stage = [&](int ch) {
+  // A stager warp holds the raw values of its tokens of one chunk: they are asked for one chunk before they
+  // are converted, so that the loads run beside the recurrence.
+  constexpr int M = (LANES * kWkRows + 31) / 32;                 // key channels per lane
+  constexpr int VM = (C::kCols + 31) / 32;
+  constexpr int PER = C::kChunk / 4;                             // tokens per warp
+  T fr[PER][M], fk[PER][M], fv[PER][VM];
+  float fd[PER][M], w0[M], uu[M];
+  const T* rp = static_cast<const T*>(p.r) + h * dim;
+  const T* kp = static_cast<const T*>(p.k) + h * dim;
+  const T* vp = static_cast<const T*>(p.v) + h * dim + col0;
+  const float* dp = p.dl + h * dim;
+  auto fetch = [&](int ch) {
+#pragma unroll
+    for (int q = 0; q < PER; ++q) {
+      const int t = ch * C::kChunk + q * 4 + (warp - 4);
+      const size_t row = size_t(row0 + min(t, len - 1));
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        const int i = min(m * 32 + lane, dim - 1);               // always in bounds; masked below
+        fr[q][m] = rp[row * p.ld + i];
+        fk[q][m] = kp[row * p.ld + i];
+        fd[q][m] = dp[row * p.ld_dl + i];
+      }
+#pragma unroll
+      for (int m = 0; m < VM; ++m) fv[q][m] = vp[row * p.ld + min(m * 32 + lane, dim - 1 - col0)];
+    }
+  };
+  auto convert = [&](int ch) {
     float* buf = smem + (ch & 1) * C::kChunk * C::kTok;
-    const T* r = static_cast<const T*>(p.r) + h * dim;
-    const T* k = static_cast<const T*>(p.k) + h * dim;
-    const T* v = static_cast<const T*>(p.v) + h * dim;
-    const float* dl = p.dl + h * dim;
-    constexpr int M = (LANES * kWkRows + 31) / 32;               // key channels per lane
-    constexpr int VM = (C::kCols + 31) / 32;
-    constexpr int PER = C::kChunk / 4;                           // tokens per warp
-    constexpr int U = M <= 4 ? 2 : 1;                            // tokens whose loads are in flight together
 #pragma unroll
-    for (int q0 = 0; q0 < PER; q0 += U) {
-      float fr[U][M], fk[U][M], fd[U][M], fv[U][VM];
+    for (int q = 0; q < PER; ++q) {
+      const int tok = q * 4 + (warp - 4);
+      const bool there = ch * C::kChunk + tok < len;             // tokens past the end leave the state as it is
+      float* b = buf + tok * C::kTok;
+      float ruk = 0.f;
 #pragma unroll
-      for (int q = 0; q < U; ++q) {
-        const int tok = (q0 + q) * 4 + (warp - 4), t = ch * C::kChunk + tok;
-        const size_t row = size_t(row0 + min(t, len - 1));
-#pragma unroll
-        for (int m = 0; m < M; ++m) {
-          const int i = m * 32 + lane;
-          const bool in = t < len && i < dim;
-          fr[q][m] = in ? to_f32(r[row * p.ld + i]) : 0.f;
-          fk[q][m] = in ? to_f32(k[row * p.ld + i]) : 0.f;
-          fd[q][m] = in ? dl[row * p.ld_dl + i] : -INFINITY;     // decay 1: the state stays as it is
-        }
-#pragma unroll
-        for (int m = 0; m < VM; ++m) {
-          const int c = m * 32 + lane;
-          fv[q][m] = (t < len && c < C::kCols && col0 + c < dim) ? to_f32(v[row * p.ld + col0 + c]) : 0.f;
-        }
+      for (int m = 0; m < M; ++m) {
+        const int i = m * 32 + lane;
+        if (LANES * kWkRows < 32 && i >= LANES * kWkRows) continue;
+        const int at = (i >> 4) * kWkGroup + (i & 15);
+        const bool in = there && i < dim;
+        const float r = in ? to_f32(fr[q][m]) : 0.f, k = in ? to_f32(fk[q][m]) : 0.f;
+        b[at] = r;
+        b[C::kVec + at] = k;
+        b[2 * C::kVec + at] = in ? __expf(-__expf(fd[q][m] + w0[m])) : 1.f;
+        ruk = fmaf(r * uu[m], k, ruk);
       }
 #pragma unroll
-      for (int q = 0; q < U; ++q) {
-        const int tok = (q0 + q) * 4 + (warp - 4);
-        float* b = buf + tok * C::kTok;
-        float ruk = 0.f;
-#pragma unroll
-        for (int m = 0; m < M; ++m) {
-          const int i = m * 32 + lane;
-          if (i >= LANES * kWkRows) continue;
-          const int at = (i >> 4) * kWkGroup + (i & 15);
-          const bool in = i < dim;
-          b[at] = fr[q][m];
-          b[C::kVec + at] = fk[q][m];
-          b[2 * C::kVec + at] = expf(-expf(fd[q][m] + (in ? p.w0[h * dim + i] : 0.f)));
-          ruk = fmaf(fr[q][m] * (in ? p.u[h * dim + i] : 0.f), fk[q][m], ruk);
-        }
-#pragma unroll
-        for (int m = 0; m < VM; ++m) {
-          const int c = m * 32 + lane;
-          if (c < C::kCols) b[3 * C::kVec + c] = fv[q][m];
-        }
-        ruk = warp_sum(ruk);
-        if (lane == 0) b[3 * C::kVec + C::kCols] = ruk;
+      for (int m = 0; m < VM; ++m) {
+        const int c = m * 32 + lane;
+        if (c < C::kCols) b[3 * C::kVec + c] = there && col0 + c < dim ? to_f32(fv[q][m]) : 0.f;
       }
+      ruk = warp_sum(ruk);
+      if (lane == 0) b[3 * C::kVec + C::kCols] = ruk;
     }
   };
 
@@ -186,12 +185,23 @@ __global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
                       (r0 + 1 < dim && col < dim) ? sp[size_t(r0 + 1) * dim] : 0.f);
     }
   } else {
-    stage(0);
+    fetch(0);
+#pragma unroll
+    for (int m = 0; m < M; ++m) {
+      const bool in = m * 32 + lane < dim;
+      w0[m] = in ? p.w0[h * dim + m * 32 + lane] : 0.f;
+      uu[m] = in ? p.u[h * dim + m * 32 + lane] : 0.f;
+    }
+    convert(0);
+    if (chunks > 1) fetch(1);
   }
   __syncthreads();
   for (int ch = 0; ch < chunks; ++ch) {
     if (stager) {
-      if (ch + 1 < chunks) stage(ch + 1);
+      if (ch + 1 < chunks) {
+        convert(ch + 1);
+        if (ch + 2 < chunks) fetch(ch + 2);
+      }
     } else {
       const float* buf = smem + (ch & 1) * C::kChunk * C::kTok;
       const int n = min(C::kChunk, len - ch * C::kChunk);
@@ -250,23 +260,35 @@ __global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
   }
 }
 
-// a[t, h*dim + i] = o / rms(o over the head) * norm * silu(gate). One warp per (row, head).
-template <class T>
+// a[t, h*dim + i] = o / rms(o over the head) * norm * silu(gate). L lanes per (row, head).
+template <class T, int L>
 __global__ void __launch_bounds__(kRowThreads)
 wkv_finish_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ gate, int ld_g,
                   const float* __restrict__ norm, float eps, T* __restrict__ a, int ld_a, int rows, int H, int dim) {
   pdl_launch_dependents();
   pdl_wait();
-  const int unit = blockIdx.x * (kRowThreads / 32) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (unit >= rows * H) return;
-  const int t = unit / H, h = unit - t * H;
-  const float* src = o + size_t(t) * ld_o + h * dim;
-  float ssq = 0.f;
-  for (int i = lane; i < dim; i += 32) ssq += src[i] * src[i];
-  const float inv = 1.f / sqrtf(warp_sum(ssq) / float(dim) + eps);
-  for (int i = lane; i < dim; i += 32) {
-    const float z = to_f32(gate[size_t(t) * ld_g + h * dim + i]);
-    a[size_t(t) * ld_a + h * dim + i] = from_f32<T>(src[i] * inv * norm[h * dim + i] * (z / (1.f + expf(-z))));
+  const int unit = (blockIdx.x * kRowThreads + threadIdx.x) / L, lane = threadIdx.x % L;
+  const bool live = unit < rows * H;                   // the lanes of a warp stay together for the sums
+  const int t = live ? unit / H : 0, h = live ? unit - t * H : 0;
+  const int at = h * dim + lane * 8, n = dim - lane * 8;
+  const bool vec = dim % 8 == 0 && ld_o % 8 == 0 && ld_g % 8 == 0 && ld_a % 8 == 0 && n > 0;
+  float f[8], ssq = 0.f;
+  load8_upto(o + size_t(t) * ld_o + at, n, vec, f);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ssq += f[i] * f[i];
+  ssq = group_sum<L>(ssq);
+  if (!live || n <= 0) return;
+  const float inv = 1.f / sqrtf(ssq / float(dim) + eps);
+  float z[8], w[8];
+  load8_upto(gate + size_t(t) * ld_g + at, n, vec, z);
+  load8_upto(norm + at, n, vec, w);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) f[i] = f[i] * inv * w[i] * (z[i] / (1.f + expf(-z[i])));
+  T* dst = a + size_t(t) * ld_a + at;
+  if (vec) {
+    store8(dst, f);
+  } else {
+    for (int i = 0; i < 8 && i < n; ++i) dst[i] = from_f32<T>(f[i]);
   }
 }
 
@@ -328,11 +350,20 @@ extern "C" int rmlx_wkv_finish(const float* o, int ld_o, const void* gate, int l
                                void* a, int ld_a, int rows, int H, int dim, int f32, int pdl, cudaStream_t st) {
   const long long units = 1LL * rows * H;
   if (rows < 1 || H < 1 || dim < 1 || units > 0x7fffffffLL) return -2;
-  const dim3 grid(unsigned((units + kRowThreads / 32 - 1) / (kRowThreads / 32)));
-  if (f32)
-    return launch(wkv_finish_kernel<float>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o,
-                  static_cast<const float*>(gate), ld_g, norm, eps, static_cast<float*>(a), ld_a, rows, H, dim);
-  return launch(wkv_finish_kernel<__nv_bfloat16>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o,
-                static_cast<const __nv_bfloat16*>(gate), ld_g, norm, eps, static_cast<__nv_bfloat16*>(a), ld_a, rows,
-                H, dim);
+  const int lanes = dim <= 64 ? 8 : dim <= 128 ? 16 : 32;
+  if (dim > 256 || units * lanes > 0x7fffffffLL) return -2;
+  const dim3 grid(unsigned((units * lanes + kRowThreads - 1) / kRowThreads));
+#define RB_WF(T_, L_)                                                                                              \
+  return launch(wkv_finish_kernel<T_, L_>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o,                      \
+                static_cast<const T_*>(gate), ld_g, norm, eps, static_cast<T_*>(a), ld_a, rows, H, dim)
+#define RB_WFL(T_)                 \
+  {                                \
+    if (lanes == 8) RB_WF(T_, 8);  \
+    if (lanes == 16) RB_WF(T_, 16); \
+    RB_WF(T_, 32);                 \
+  }
+  if (f32) RB_WFL(float)
+  RB_WFL(__nv_bfloat16)
+#undef RB_WFL
+#undef RB_WF
 }
