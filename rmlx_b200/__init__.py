@@ -20,7 +20,8 @@ _EXPORTS = {
     "random_state_dict": "models.weights", "CachedDecode": "models.decode_engine", "BatchedDecode": "models.prefill",
     "NativePrefill": "models.prefill", "enable_native_prefill": "models.prefill",
     "Qwen2Model": "models.qwen", "MixtralModel": "models.mixtral", "DeepSeekV3Model": "models.deepseek",
-    "PosudraModel": "models.posudra", "PosudraConfig": "config", "from_pretrained": "models.registry",
+    "PosudraModel": "models.posudra", "PosudraConfig": "config", "RodapelModel": "models.rodapel", "RodapelConfig": "config",
+    "from_pretrained": "models.registry",
     "ModelFamily": "models.registry", "Entry": "models.ragged", "ParallelBlockDecode": "models.parallel_decode",
     # weights, caches, serving
     "LinearWeight": "ops.weights", "PagedKvCache": "kv.paged", "BlockManager": "kv.paged",

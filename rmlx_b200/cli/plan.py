@@ -14,6 +14,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import math
 import os
 from typing import Dict, Optional, Sequence
 
@@ -223,6 +224,50 @@ def plan_posudra(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, bud
     }
 
 
+def plan_rodapel(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, budget_fraction: float = 0.90,
+                 cfg=None) -> dict:
+    """A Rodapel model (bf16, one GPU): pages for its attention layers, recurrent state per sequence for its
+    WKV layers, the widest activations of a prompt chunk (with expanded keys and values of ``ctx`` tokens)."""
+    from ..config import LatentAttentionSpec, RoutedFfSpec, WkvSpec
+    from ..models.rodapel import kv_shapes, rodapel_4096, state_shapes, tensor_shapes
+    c = cfg or rodapel_4096()
+    parts = {"attention": 0, "feed_forward": 0, "norms": 0, "embedding": 0, "lm_head": 0}
+    routed, active = 0, 0
+    for name, shape in tensor_shapes(c).items():
+        n = math.prod(shape)
+        part = {"embed": "embedding", "head": "lm_head"}.get(name) or (
+            "norms" if len(shape) == 1 else "feed_forward" if ".mlp." in name else "attention")
+        parts[part] += n * (4 if len(shape) == 1 else 2)               # per-channel vectors are kept in fp32
+        routed += n * 2 if ".mlp.e" in name else 0
+    for l in c.layers:
+        if isinstance(l.mlp, RoutedFfSpec):
+            active += min(l.mlp.experts, batch * l.mlp.top) * 3 * l.mlp.ff * c.width * 2
+    parts["total"] = sum(parts.values())
+    kv_tok = sum(s[0] * (s[1] + s[2]) * 2 for s in kv_shapes(c) if s is not None)
+    state = sum(4 * math.prod(shape) for p in state_shapes(c) if p for shape in p.values())
+    lat = [l.mixer for l in c.layers if isinstance(l.mixer, LatentAttentionSpec)]
+    row = 10 * c.width + max([0] + [12 * l.mixer.heads * l.mixer.dim + 10 * c.width for l in c.layers
+                                    if isinstance(l.mixer, WkvSpec)]) + \
+        max([0] + [l.mlp.top * 2 * (2 * c.width + l.mlp.ff) if isinstance(l.mlp, RoutedFfSpec) else 2 * l.mlp.ff
+                   for l in c.layers if l.mlp is not None])
+    scratch = prefill_chunk * row + ctx * max([0] + [2 * (m.heads * (m.dim + m.vdim) + m.kv_rank) for m in lat])
+    budget, need = int(HBM_BYTES * budget_fraction), batch * (ctx * kv_tok + state)
+    step = parts["attention"] + parts["feed_forward"] - routed + active + need + parts["lm_head"]
+    hbm = decode_hbm_gbs()
+    layer = (step - parts["lm_head"]) / c.num_layers
+    return {
+        "model": c.name, "weights": "bf16", "tp": 1, "expert_parallel": False, "batch": batch, "ctx": ctx,
+        "kv_quant": "bf16", "weight_bytes_per_gpu": parts, "kv_bytes_per_token_per_gpu": kv_tok,
+        "state_bytes_per_sequence": state, "prefill_chunk": prefill_chunk, "prefill_scratch_bytes": scratch,
+        "budget_bytes_per_gpu": budget, "kv_bytes_needed": need,
+        "kv_tokens_that_fit": max(0, (budget - parts["total"] - scratch - batch * state) // max(kv_tok, 1)),
+        "fits": parts["total"] + scratch + need <= budget,
+        "decode_roofline": {"bytes_per_layer": layer, "us_per_layer": layer / (hbm * 1e3), "us_per_step": step / (hbm * 1e3),
+                            "tokens_per_s": batch * hbm * 1e9 / step, "hbm_gbs": hbm},
+        "decode_stream_plans": {},
+    }
+
+
 def plan(model: str = "moe-a22b", weights: str = "q4", tp: int = 1, batch: int = 1, ctx: int = 4096,
          kv_quant: Optional[str] = None, expert_parallel: bool = False, prefill_chunk: int = 2048,
          budget_fraction: float = 0.90, cfg: Optional[TransformerConfig] = None) -> dict:
@@ -232,6 +277,10 @@ def plan(model: str = "moe-a22b", weights: str = "q4", tp: int = 1, batch: int =
         if weights != "bf16" or tp != 1 or kv_quant is not None:
             raise ValueError("Posudra runs on one GPU with bf16 weights and cache")
         return plan_posudra(batch, ctx, prefill_chunk, budget_fraction)
+    if model == "rodapel-4096" and cfg is None:
+        if weights != "bf16" or tp != 1 or kv_quant is not None:
+            raise ValueError("Rodapel runs on one GPU with bf16 weights and cache")
+        return plan_rodapel(batch, ctx, prefill_chunk, budget_fraction)
     cfg = cfg or presets()[model]
     w = weight_bytes_per_gpu(cfg, weights, tp, expert_parallel)
     kv_tok = kv_bytes_per_token_per_gpu(cfg, tp, kv_quant)
@@ -277,6 +326,8 @@ def render(p: dict) -> str:
              f"  weights per GPU      {_gb(w['total'])}  (attention {_gb(w['attention']).strip()}, feed-forward "
              f"{_gb(w['feed_forward']).strip()}, embedding {_gb(w['embedding']).strip()}, LM head {_gb(w['lm_head']).strip()})",
              f"  KV per token per GPU {p['kv_bytes_per_token_per_gpu']:8d} B   needed for this batch and context {_gb(p['kv_bytes_needed']).strip()}",
+             *([f"  recurrent state per sequence {_gb(p['state_bytes_per_sequence']).strip()}"]
+               if p.get("state_bytes_per_sequence") else []),
              f"  prompt chunk {p['prefill_chunk']}: scratch {_gb(p['prefill_scratch_bytes']).strip()}",
              f"  budget per GPU       {_gb(p['budget_bytes_per_gpu'])}  -> {'fits' if p['fits'] else 'DOES NOT FIT'}; "
              f"room for {p['kv_tokens_that_fit']:,} cached tokens per GPU"]
@@ -293,7 +344,7 @@ def render(p: dict) -> str:
 
 def main(argv: Optional[Sequence[str]] = None) -> int:
     ap = argparse.ArgumentParser(prog="rmlx plan", description=__doc__.split("\n\n")[0])
-    ap.add_argument("--model", default="moe-a22b", choices=sorted(presets()) + ["deepseek-v3", "posudra-8b"])
+    ap.add_argument("--model", default="moe-a22b", choices=sorted(presets()) + ["deepseek-v3", "posudra-8b", "rodapel-4096"])
     ap.add_argument("--weights", default="q4", choices=sorted(BITS))
     ap.add_argument("--tp", type=int, default=1)
     ap.add_argument("--expert-parallel", action="store_true")

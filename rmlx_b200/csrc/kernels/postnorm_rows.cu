@@ -56,28 +56,40 @@ struct ExpertSource {
   const float* identity;      // [T] summed weight of the identity experts
   int top_k;
   float id_w;
-  __device__ __forceinline__ void prepare(int t) { id_w = identity[t]; }
+  int rows[4];                // the first four slots
+  float wts[4];
+  __device__ __forceinline__ void prepare(int t) {
+    id_w = identity[t];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      rows[u] = u < top_k ? row_of_pair[t * top_k + u] : -1;
+      wts[u] = u < top_k ? weights[t * top_k + u] : 0.f;
+    }
+  }
   __device__ __forceinline__ void load(int t, int c, const float (&x)[8], float (&f)[8]) const {
 #pragma unroll
     for (int i = 0; i < 8; ++i) f[i] = id_w * x[i];
-    for (int s0 = 0; s0 < top_k; s0 += 4) {            // four slots' rows in flight
-      float g[4][8], a[4];
+    float g[4][8];
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int p = t * top_k + min(s0 + u, top_k - 1);
-        const int row = s0 + u < top_k ? row_of_pair[p] : -1;
-        a[u] = row >= 0 ? weights[p] : 0.f;
-        if (row >= 0) {
-          load8(y + size_t(row) * ldy + c * 8, g[u]);
-        } else {
+    for (int u = 0; u < 4; ++u) {                      // four slots' rows in flight
+      if (rows[u] >= 0) {
+        load8(y + size_t(rows[u]) * ldy + c * 8, g[u]);
+      } else {
 #pragma unroll
-          for (int i = 0; i < 8; ++i) g[u][i] = 0.f;
-        }
+        for (int i = 0; i < 8; ++i) g[u][i] = 0.f;
       }
+    }
 #pragma unroll
-      for (int u = 0; u < 4; ++u)
+    for (int u = 0; u < 4; ++u)
 #pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] = fmaf(a[u], g[u][i], f[i]);
+      for (int i = 0; i < 8; ++i) f[i] = fmaf(wts[u], g[u][i], f[i]);
+    for (int s = 4; s < top_k; ++s) {
+      const int row = row_of_pair[t * top_k + s];
+      if (row < 0) continue;
+      const float a = weights[t * top_k + s];
+      load8(y + size_t(row) * ldy + c * 8, g[0]);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] = fmaf(a, g[0][i], f[i]);
     }
   }
 };
@@ -368,9 +380,9 @@ extern "C" int rmlx_moe_combine_post_norm(const void* y, int ldy, const int* row
   if (T < 1 || D < 1 || ldx < D || ldx % 8 || ldy % 8 || ldy < ldx || top_k < 1) return -2;
   if (f32)
     return launch_post_norm(ExpertSource<float>{static_cast<const float*>(y), ldy, row_of_pair, weights, identity,
-                                                top_k, 0.f}, w, eps, x, h, T, D, ldx, 1, pdl, st);
+                                                top_k}, w, eps, x, h, T, D, ldx, 1, pdl, st);
   return launch_post_norm(ExpertSource<__nv_bfloat16>{static_cast<const __nv_bfloat16*>(y), ldy, row_of_pair, weights,
-                                                      identity, top_k, 0.f}, w, eps, x, h, T, D, ldx, 0, pdl, st);
+                                                      identity, top_k}, w, eps, x, h, T, D, ldx, 0, pdl, st);
 }
 
 // f32: q_out and the caches are fp32, else bf16; raw_f32: raw is fp32.

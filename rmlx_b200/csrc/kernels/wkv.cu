@@ -5,10 +5,11 @@
 //     o_t = (S + diag(u) k_t v_t^T)^T r_t,   S <- diag(w_t) S + k_t v_t^T,
 //     w_t = exp(-exp(dl_t + w0))
 // Columns are independent of each other. A block owns one (sequence, head, group of columns) and walks
-// the sequence's new tokens; a thread holds 16 rows of one column in registers, LANES threads share a
-// column. Half of the block's warps fetch the next chunk of tokens (and take the exponentials and
-// r . (u k)) while the other half runs the current one; r, k and w are read from shared memory in
-// 16-row groups that start in different banks. Arithmetic on the state runs on pairs (fma.rn.f32x2).
+// the sequence's new tokens. A thread holds ROWS rows of four columns in registers (each r, k and w read from
+// shared memory then serves four columns: shared-memory wavefronts, not arithmetic, are what one column per
+// thread is bound by); LANES threads share a column and add their parts by a transposing butterfly. Half of the
+// block's warps fetch tokens ahead, take the exponentials and r . (u k), and stage the next chunk while the
+// other half runs the current one. Arithmetic on the state runs on pairs (fma.rn.f32x2).
 //
 // The state of a sequence lives in its slot's row of a flat fp32 pool, beside the last token's
 // residual row, which the token shift of the sequence's next token needs.
@@ -88,19 +89,19 @@ struct WkvParams {
   int H, dim;
 };
 
-constexpr int kWkThreads = 256, kWkHalf = 128, kWkRows = 16, kWkGroup = 20;
-template <int LANES>
+constexpr int kWkHalf = 64, kWkCols = 4;            // compute (and staging) threads; columns per thread
+template <int ROWS, int LANES>
 struct WkCfg {
-  static constexpr int kCols = kWkHalf / LANES;                  // columns per block
-  static constexpr int kChunk = LANES >= 16 ? 8 : 16;            // tokens per chunk
-  static constexpr int kVec = LANES * kWkGroup;                  // floats of one staged r / k / w vector
-  static constexpr int kTok = 3 * kVec + kCols + 4;              // + v, + r . (u k)
+  static constexpr int kDim = ROWS * LANES;          // padded rows of the state
+  static constexpr int kCols = kWkHalf / LANES * kWkCols;        // columns per block
+  static constexpr int kChunk = kDim > 128 ? 4 : kDim > 64 ? 8 : 16;   // tokens per chunk
+  static constexpr int kTok = 3 * kDim + kCols + 4;              // r, k, w, v, r . (u k)
   static constexpr int kSmem = 2 * kChunk * kTok * 4;
 };
 
-template <class T, int LANES>
-__global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
-  using C = WkCfg<LANES>;
+template <class T, int ROWS, int LANES>
+__global__ void __launch_bounds__(2 * kWkHalf) wkv_scan_kernel(WkvParams p) {
+  using C = WkCfg<ROWS, LANES>;
   extern __shared__ __align__(16) float smem[];
   pdl_launch_dependents();
   pdl_wait();
@@ -113,14 +114,15 @@ __global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
     row0 = blockIdx.z; len = 1; slot = p.slots[blockIdx.z];
   }
   const int dim = p.dim, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const bool stager = warp >= 4;
+  constexpr int SW = kWkHalf / 32;                               // staging warps
+  const bool stager = warp >= SW;
   const int chunks = (len + C::kChunk - 1) / C::kChunk;
 
   // A stager warp holds the raw values of its tokens of one chunk: they are asked for one chunk before they
   // are converted, so that the loads run beside the recurrence.
-  constexpr int M = (LANES * kWkRows + 31) / 32;                 // key channels per lane
+  constexpr int M = (C::kDim + 31) / 32;                         // key channels per lane
   constexpr int VM = (C::kCols + 31) / 32;
-  constexpr int PER = C::kChunk / 4;                             // tokens per warp
+  constexpr int PER = C::kChunk / SW;                            // tokens per warp
   T fr[PER][M], fk[PER][M], fv[PER][VM];
   float fd[PER][M], w0[M], uu[M];
   const T* rp = static_cast<const T*>(p.r) + h * dim;
@@ -130,7 +132,7 @@ __global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
   auto fetch = [&](int ch) {
 #pragma unroll
     for (int q = 0; q < PER; ++q) {
-      const int t = ch * C::kChunk + q * 4 + (warp - 4);
+      const int t = ch * C::kChunk + q * SW + (warp - SW);
       const size_t row = size_t(row0 + min(t, len - 1));
 #pragma unroll
       for (int m = 0; m < M; ++m) {
@@ -147,43 +149,46 @@ __global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
     float* buf = smem + (ch & 1) * C::kChunk * C::kTok;
 #pragma unroll
     for (int q = 0; q < PER; ++q) {
-      const int tok = q * 4 + (warp - 4);
+      const int tok = q * SW + (warp - SW);
       const bool there = ch * C::kChunk + tok < len;             // tokens past the end leave the state as it is
       float* b = buf + tok * C::kTok;
       float ruk = 0.f;
 #pragma unroll
       for (int m = 0; m < M; ++m) {
         const int i = m * 32 + lane;
-        if (LANES * kWkRows < 32 && i >= LANES * kWkRows) continue;
-        const int at = (i >> 4) * kWkGroup + (i & 15);
+        if (C::kDim < 32 && i >= C::kDim) continue;
+        // row group g's values four at a time: 16-byte pieces of consecutive groups are neighbours
+        const int at = (i % ROWS) / 4 * (LANES * 4) + i / ROWS * 4 + i % 4;
         const bool in = there && i < dim;
         const float r = in ? to_f32(fr[q][m]) : 0.f, k = in ? to_f32(fk[q][m]) : 0.f;
         b[at] = r;
-        b[C::kVec + at] = k;
-        b[2 * C::kVec + at] = in ? __expf(-__expf(fd[q][m] + w0[m])) : 1.f;
+        b[C::kDim + at] = k;
+        b[2 * C::kDim + at] = in ? __expf(-__expf(fd[q][m] + w0[m])) : 1.f;
         ruk = fmaf(r * uu[m], k, ruk);
       }
 #pragma unroll
       for (int m = 0; m < VM; ++m) {
         const int c = m * 32 + lane;
-        if (c < C::kCols) b[3 * C::kVec + c] = there && col0 + c < dim ? to_f32(fv[q][m]) : 0.f;
+        if (c < C::kCols) b[3 * C::kDim + c] = there && col0 + c < dim ? to_f32(fv[q][m]) : 0.f;
       }
       ruk = warp_sum(ruk);
-      if (lane == 0) b[3 * C::kVec + C::kCols] = ruk;
+      if (lane == 0) b[3 * C::kDim + C::kCols] = ruk;
     }
   };
 
-  // compute threads: rows g * 16 .. + 15 of column `col`
-  const int g = threadIdx.x % LANES, cl = (threadIdx.x & (kWkHalf - 1)) / LANES, col = col0 + cl;
-  uint64_t s2[kWkRows / 2];
-  float* sp = p.state + size_t(slot) * p.stride + size_t(h) * dim * dim + col;
+  // compute threads: rows g * ROWS .. of columns c0 .. c0 + 3 (of the block)
+  const int g = threadIdx.x % LANES, c0 = (threadIdx.x & (kWkHalf - 1)) / LANES * kWkCols;
+  uint64_t s2[ROWS / 2][kWkCols];
+  float* sp = p.state + size_t(slot) * p.stride + size_t(h) * dim * dim;
   if (!stager) {
 #pragma unroll
-    for (int i = 0; i < kWkRows / 2; ++i) {
-      const int r0 = g * kWkRows + 2 * i;
-      s2[i] = wk_pair((r0 < dim && col < dim) ? sp[size_t(r0) * dim] : 0.f,
-                      (r0 + 1 < dim && col < dim) ? sp[size_t(r0 + 1) * dim] : 0.f);
-    }
+    for (int i = 0; i < ROWS / 2; ++i)
+#pragma unroll
+      for (int c = 0; c < kWkCols; ++c) {
+        const int r0 = g * ROWS + 2 * i, col = col0 + c0 + c;
+        s2[i][c] = wk_pair((r0 < dim && col < dim) ? sp[size_t(r0) * dim + col] : 0.f,
+                           (r0 + 1 < dim && col < dim) ? sp[size_t(r0 + 1) * dim + col] : 0.f);
+      }
   } else {
     fetch(0);
 #pragma unroll
@@ -196,6 +201,10 @@ __global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
     if (chunks > 1) fetch(1);
   }
   __syncthreads();
+  // after the butterfly, the lanes of a column group hold column `mine` of the four
+  const int mine = (g & (LANES / 2) ? 2 : 0) + (g & (LANES / 4) ? 1 : 0);
+  const bool writer = g % (LANES / 4) == 0 && col0 + c0 + mine < dim;
+  float* op = p.out + size_t(row0) * p.ld_out + h * dim + col0 + c0 + mine;
   for (int ch = 0; ch < chunks; ++ch) {
     if (stager) {
       if (ch + 1 < chunks) {
@@ -205,38 +214,56 @@ __global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
     } else {
       const float* buf = smem + (ch & 1) * C::kChunk * C::kTok;
       const int n = min(C::kChunk, len - ch * C::kChunk);
-      for (int t0 = 0; t0 < n; t0 += 4) {                        // tokens past the end are staged as no-ops
-        float o[4];
+      constexpr int TU = 4;                                      // tokens whose sums are in flight together
+      for (int t0 = 0; t0 < n; t0 += TU) {
+        float o[TU][kWkCols];
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
+        for (int q = 0; q < TU; ++q) {
           const float* b = buf + (t0 + q) * C::kTok;
-          const float v = b[3 * C::kVec + cl];
-          const uint64_t v2 = wk_pair(v, v);
-          uint64_t acc0 = 0, acc1 = 0;
+          const float4 v = *reinterpret_cast<const float4*>(b + 3 * C::kDim + c0);
+          const uint64_t v2[kWkCols] = {wk_pair(v.x, v.x), wk_pair(v.y, v.y), wk_pair(v.z, v.z), wk_pair(v.w, v.w)};
+          uint64_t acc[kWkCols] = {0, 0, 0, 0};
 #pragma unroll
-          for (int i = 0; i < kWkRows / 4; ++i) {
-            const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(b + g * kWkGroup + i * 4);
-            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(b + C::kVec + g * kWkGroup + i * 4);
-            const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(b + 2 * C::kVec + g * kWkGroup + i * 4);
-            acc0 = wk_fma(r.x, s2[2 * i], acc0);
-            acc1 = wk_fma(r.y, s2[2 * i + 1], acc1);
-            s2[2 * i] = wk_fma(w.x, s2[2 * i], wk_mul(k.x, v2));
-            s2[2 * i + 1] = wk_fma(w.y, s2[2 * i + 1], wk_mul(k.y, v2));
+          for (int i = 0; i < ROWS / 4; ++i) {
+            const int at = i * (LANES * 4) + g * 4;
+            const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(b + at);
+            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(b + C::kDim + at);
+            const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(b + 2 * C::kDim + at);
+#pragma unroll
+            for (int c = 0; c < kWkCols; ++c) {
+              acc[c] = wk_fma(r.x, s2[2 * i][c], acc[c]);
+              acc[c] = wk_fma(r.y, s2[2 * i + 1][c], acc[c]);
+              s2[2 * i][c] = wk_fma(w.x, s2[2 * i][c], wk_mul(k.x, v2[c]));
+              s2[2 * i + 1][c] = wk_fma(w.y, s2[2 * i + 1][c], wk_mul(k.y, v2[c]));
+            }
           }
-          float a, c, d, e;
-          wk_unpair(acc0, a, c);
-          wk_unpair(acc1, d, e);
-          o[q] = (a + c) + (d + e);
-          if (g == 0) o[q] = fmaf(b[3 * C::kVec + C::kCols], v, o[q]);
+#pragma unroll
+          for (int c = 0; c < kWkCols; ++c) {
+            float lo, hi;
+            wk_unpair(acc[c], lo, hi);
+            o[q][c] = lo + hi;
+          }
+        }
+        float sum[TU];
+#pragma unroll
+        for (int q = 0; q < TU; ++q) {
+          const bool up = g & (LANES / 2), up2 = g & (LANES / 4);
+          const float k0 = up ? o[q][2] : o[q][0], k1 = up ? o[q][3] : o[q][1];
+          const float x0 = up ? o[q][0] : o[q][2], x1 = up ? o[q][1] : o[q][3];
+          const float y0 = k0 + __shfl_xor_sync(0xffffffffu, x0, LANES / 2);
+          const float y1 = k1 + __shfl_xor_sync(0xffffffffu, x1, LANES / 2);
+          sum[q] = (up2 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, up2 ? y0 : y1, LANES / 4);
         }
 #pragma unroll
-        for (int off = LANES / 2; off > 0; off >>= 1)
+        for (int off = LANES / 8; off > 0; off >>= 1)
 #pragma unroll
-          for (int q = 0; q < 4; ++q) o[q] += __shfl_xor_sync(0xffffffffu, o[q], off);
-        if (g == 0 && col < dim) {
+          for (int q = 0; q < TU; ++q) sum[q] += __shfl_xor_sync(0xffffffffu, sum[q], off);
+        if (writer) {
 #pragma unroll
-          for (int q = 0; q < 4; ++q)
-            if (t0 + q < n) p.out[size_t(row0 + ch * C::kChunk + t0 + q) * p.ld_out + h * dim + col] = o[q];
+          for (int q = 0; q < TU; ++q) {
+            const float* b = buf + (t0 + q) * C::kTok + 3 * C::kDim;
+            if (t0 + q < n) op[size_t(ch * C::kChunk + t0 + q) * p.ld_out] = fmaf(b[C::kCols], b[c0 + mine], sum[q]);
+          }
         }
       }
     }
@@ -244,15 +271,17 @@ __global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
   }
   if (!stager) {
 #pragma unroll
-    for (int i = 0; i < kWkRows / 2; ++i) {
-      const int r0 = g * kWkRows + 2 * i;
-      float lo, hi;
-      wk_unpair(s2[i], lo, hi);
-      if (col < dim) {
-        if (r0 < dim) sp[size_t(r0) * dim] = lo;
-        if (r0 + 1 < dim) sp[size_t(r0 + 1) * dim] = hi;
+    for (int i = 0; i < ROWS / 2; ++i)
+#pragma unroll
+      for (int c = 0; c < kWkCols; ++c) {
+        const int r0 = g * ROWS + 2 * i, col = col0 + c0 + c;
+        float lo, hi;
+        wk_unpair(s2[i][c], lo, hi);
+        if (col < dim) {
+          if (r0 < dim) sp[size_t(r0) * dim + col] = lo;
+          if (r0 + 1 < dim) sp[size_t(r0 + 1) * dim + col] = hi;
+        }
       }
-    }
   } else if (blockIdx.x == 0 && h == 0) {
     const float* last = p.x + size_t(row0 + len - 1) * p.ldx;
     float* keep = p.prev + size_t(slot) * p.stride;
@@ -292,21 +321,20 @@ wkv_finish_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ g
   }
 }
 
-template <class T, int LANES>
+template <class T, int ROWS, int LANES>
 static int launch_wkv(const WkvParams& p, int n_segs, int pdl, cudaStream_t st) {
-  using C = WkCfg<LANES>;
-  auto kern = wkv_scan_kernel<T, LANES>;
+  using C = WkCfg<ROWS, LANES>;
+  auto kern = wkv_scan_kernel<T, ROWS, LANES>;
   RB_CHECK(set_max_smem(kern, C::kSmem));
-  return launch(kern, dim3((p.dim + C::kCols - 1) / C::kCols, p.H, n_segs), dim3(kWkThreads), C::kSmem, st, pdl != 0, p);
+  return launch(kern, dim3((p.dim + C::kCols - 1) / C::kCols, p.H, n_segs), dim3(2 * kWkHalf), C::kSmem, st, pdl != 0, p);
 }
 template <class T>
 static int dispatch_wkv(const WkvParams& p, int n, int pdl, cudaStream_t st) {
-  const int groups = (p.dim + kWkRows - 1) / kWkRows;
-  if (groups <= 1) return launch_wkv<T, 1>(p, n, pdl, st);
-  if (groups <= 2) return launch_wkv<T, 2>(p, n, pdl, st);
-  if (groups <= 4) return launch_wkv<T, 4>(p, n, pdl, st);
-  if (groups <= 8) return launch_wkv<T, 8>(p, n, pdl, st);
-  if (groups <= 16) return launch_wkv<T, 16>(p, n, pdl, st);
+  if (p.dim <= 16) return launch_wkv<T, 4, 4>(p, n, pdl, st);
+  if (p.dim <= 32) return launch_wkv<T, 4, 8>(p, n, pdl, st);
+  if (p.dim <= 64) return launch_wkv<T, 4, 16>(p, n, pdl, st);
+  if (p.dim <= 128) return launch_wkv<T, 4, 32>(p, n, pdl, st);
+  if (p.dim <= 256) return launch_wkv<T, 8, 32>(p, n, pdl, st);
   return -2;
 }
 
@@ -315,7 +343,7 @@ static int dispatch_wkv(const WkvParams& p, int n, int pdl, cudaStream_t st) {
 using namespace rb;
 
 // Largest head size of the recurrence.
-extern "C" int rmlx_wkv_max_dim() { return 16 * kWkRows; }
+extern "C" int rmlx_wkv_max_dim() { return 256; }
 
 // x fp32 [T, ldx], mu fp32 [5, ldx], out [5, T, ldx] fp32 (f32) or bf16; ldx a multiple of eight, prev
 // rows 16-byte aligned. slots int32 [T].

@@ -51,6 +51,18 @@ def rodapel_tiny() -> RodapelConfig:
         PostNormLayerSpec(WindowAttentionSpec(2, 2, 24, 16, 0.25, 9), None)]).validate()
 
 
+def rodapel_4096(num_layers: int = 32) -> RodapelConfig:
+    """Layers of width 4096 (memory plan, benchmarks): in fours, windowed attention + dense, WKV + routed,
+    latent attention + routed, windowed attention + routed."""
+    win = WindowAttentionSpec(32, 8, 128, 128, 128 ** -0.5, 1024)
+    lat = LatentAttentionSpec(32, 128, 64, 128, 512, 192 ** -0.5)
+    moe = RoutedFfSpec(32, 8, 4, 3584, 7.0)
+    four = [PostNormLayerSpec(win, ClampedFfSpec(14336, 7.0)), PostNormLayerSpec(WkvSpec(64, 64, 64), moe),
+            PostNormLayerSpec(lat, moe), PostNormLayerSpec(win, moe)]
+    return RodapelConfig(vocab_size=128256, width=4096, layers=(four * ((num_layers + 3) // 4))[:num_layers],
+                         norm_eps=1e-6, name="rodapel-4096").validate()
+
+
 # ------------------------------------------------------------------------------------------------
 # Weights
 # ------------------------------------------------------------------------------------------------
@@ -168,8 +180,28 @@ class RodapelWeights:
         return sum(size(v) for p in parts for v in vars(p).values())
 
 
-def tensor_shapes(cfg: RodapelConfig, ranks: Optional[Dict[int, int]] = None) -> Dict[str, tuple]:
-    """Checkpoint tensor names and shapes. ``ranks``: layer -> decay rank, where a checkpoint has its own."""
+def kv_shapes(cfg: RodapelConfig) -> List[Optional[tuple]]:
+    """Per layer (kv heads, key row, value row) of the paged cache; latent rows are key and value at once."""
+    out: List[Optional[tuple]] = []
+    for l in cfg.layers:
+        m = l.mixer
+        if isinstance(m, WindowAttentionSpec):
+            out.append((m.kv_heads, pad8(m.dim), pad8(m.vdim)))
+        elif isinstance(m, LatentAttentionSpec):
+            out.append((1, pad8(m.kv_rank) + pad8(m.rot_dim) + LATENT_ROW_PAD, 0))
+        else:
+            out.append(None)
+    return out
+
+
+def state_shapes(cfg: RodapelConfig) -> List[Optional[Dict[str, tuple]]]:
+    """Per layer what a sequence carries: the WKV state and the last token's residual row."""
+    return [{"wkv": (l.mixer.heads, l.mixer.dim, l.mixer.dim), "prev": (pad8(cfg.width),)}
+            if isinstance(l.mixer, WkvSpec) else None for l in cfg.layers]
+
+
+def tensor_shapes(cfg: RodapelConfig) -> Dict[str, tuple]:
+    """Checkpoint tensor names and shapes."""
     d = cfg.width
     out = {"embed": (cfg.vocab_size, d), "embed.norm": (d,)}
     for i, l in enumerate(cfg.layers):
@@ -185,7 +217,7 @@ def tensor_shapes(cfg: RodapelConfig, ranks: Optional[Dict[int, int]] = None) ->
                         p + "dkv.norm": (m.kv_rank,), p + "uk": (m.heads * m.dim, m.kv_rank),
                         p + "uv": (m.heads * m.vdim, m.kv_rank), p + "o": (d, m.heads * m.vdim)})
         else:
-            n, rank = m.heads * m.dim, (ranks or {}).get(i, m.decay_rank)
+            n, rank = m.heads * m.dim, m.decay_rank
             out.update({p + "mu." + s: (d,) for s in W.SHIFT_PARTS})
             out.update({p + s: (n, d) for s in "rkvg"})
             out.update({p + "w1": (rank, d), p + "w2": (n, rank), p + "w0": (n,), p + "u": (m.heads, m.dim),
@@ -234,7 +266,9 @@ def build_weights(cfg: RodapelConfig, tensors: Dict[str, torch.Tensor], device="
         raise ValueError("Rodapel runs in bfloat16 or float32")
     ranks = {i: tensors[f"l{i}.mix.w1"].shape[0] for i, l in enumerate(cfg.layers)
              if isinstance(l.mixer, WkvSpec) and f"l{i}.mix.w1" in tensors}
-    for name, shape in tensor_shapes(cfg, ranks).items():
+    cfg = replace(cfg, layers=[replace(l, mixer=replace(l.mixer, decay_rank=ranks[i])) if i in ranks else l
+                               for i, l in enumerate(cfg.layers)])
+    for name, shape in tensor_shapes(cfg).items():
         if name not in tensors:
             raise KeyError(f"checkpoint has no tensor {name!r}")
         if tuple(tensors[name].shape) != shape:
@@ -284,8 +318,7 @@ def build_weights(cfg: RodapelConfig, tensors: Dict[str, torch.Tensor], device="
                                  LinearWeight(W_BF16, ukv), out_proj(g("o"), m.heads, m.vdim), vec(m.rot_base ** (-2.0 * pairs / max(m.rot_dims, 1))),
                                  ScoreMods(m.scale))
         n = m.heads * m.dim
-        inner, rank, rank_p = pad_to(n, 16), ranks[i], pad_to(ranks[i], 16)
-        m = replace(m, decay_rank=rank)
+        inner, rank_p = pad_to(n, 16), pad_to(m.decay_rank, 16)
         w_in = torch.cat([mat([g(s)], inner, wp) for s in "rkvg"] + [mat([g("w1")], rank_p, wp)])
         return WkvWeights(m, torch.stack([vec(g("mu." + s), wp) for s in W.SHIFT_PARTS]), LinearWeight(W_BF16, w_in),
                           mat([g("w2")], inner, rank_p), vec(g("w0")), vec(g("u")), vec(g("norm")), lin([g("o")], wp, inner))
@@ -414,22 +447,6 @@ class RodapelModel:
         return from_pretrained(model_dir, device, dtype)
 
     # ------------------------------------------------------------------ cache
-    def kv_shapes(self) -> List[Optional[tuple]]:
-        out: List[Optional[tuple]] = []
-        for l in self.cfg.layers:
-            m = l.mixer
-            if isinstance(m, WindowAttentionSpec):
-                out.append((m.kv_heads, pad8(m.dim), pad8(m.vdim)))
-            elif isinstance(m, LatentAttentionSpec):
-                out.append((1, pad8(m.kv_rank) + pad8(m.rot_dim) + LATENT_ROW_PAD, 0))
-            else:
-                out.append(None)
-        return out
-
-    def state_shapes(self) -> List[Optional[Dict[str, tuple]]]:
-        return [{"wkv": (l.mixer.heads, l.mixer.dim, l.mixer.dim), "prev": (self.width_p,)}
-                if isinstance(l.mixer, WkvSpec) else None for l in self.cfg.layers]
-
     def new_cache(self, num_blocks: int, max_seqs: int = 64, max_blocks_per_seq: Optional[int] = None,
                   dtype=None, kv_quant: Optional[str] = None) -> PagedKvCache:
         """``num_blocks`` pages of 16 tokens (page 0 is reserved). Without ``max_blocks_per_seq`` one
@@ -440,11 +457,11 @@ class RodapelModel:
             max_blocks_per_seq = max(1, num_blocks - 1)
             if self.cfg.max_seq_len:
                 max_blocks_per_seq = min(max_blocks_per_seq, (self.cfg.max_seq_len + PAGE - 1) // PAGE)
-        shapes = self.kv_shapes()
+        shapes = kv_shapes(self.cfg)
         first = next((s for s in shapes if s is not None), (1, 8, 8))
         return PagedKvCache(num_blocks, len(shapes), first[0], first[1], dtype=dtype or self.dtype, device=self.device,
                             max_seqs=max_seqs, max_blocks_per_seq=max_blocks_per_seq, layer_shapes=shapes,
-                            layer_states=self.state_shapes())
+                            layer_states=state_shapes(self.cfg))
 
     def make_decode_engine(self, cache: PagedKvCache, max_batch: int, comm=None):
         from .post_norm_decode import PostNormDecode

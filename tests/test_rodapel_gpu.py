@@ -1,0 +1,840 @@
+"""Rodapel on the GPU against the plain restatement in ``oracle/rodapel.py``: every mechanism alone, then the
+model through its ragged batches, its decode engine, the serving engine and the command line, in 32-bit
+(tight) and bf16."""
+import io
+import json
+import struct
+import sys
+
+import pytest
+import torch
+from oracle import rodapel as O
+
+from rmlx_b200.config import (ClampedFfSpec, LatentAttentionSpec, PostNormLayerSpec, RodapelConfig, RoutedFfSpec,
+                              SamplerConfig, SchedulerConfig, WindowAttentionSpec, WkvSpec)
+from rmlx_b200.models import rodapel as M
+from rmlx_b200.models.post_norm_decode import PostNormDecode
+from rmlx_b200.models.ragged import Entry, query_tiles
+from rmlx_b200.ops import latent as L
+from rmlx_b200.ops import parallel_block as P
+from rmlx_b200.ops import post_norm as N
+from rmlx_b200.ops import routed as R
+from rmlx_b200.ops import wkv as W
+from rmlx_b200.ops.post_norm import pad_to
+from rmlx_b200.ops.quantized import xgemm
+from rmlx_b200.ops.weights import LinearWeight, W_BF16
+from rmlx_b200.serve.engine import ServingEngine
+
+pytestmark = pytest.mark.gpu
+BF, F32 = torch.bfloat16, torch.float32
+pad8 = P.pad8
+
+
+def rel(got, want):
+    got, want = got.double().cpu(), want.double().cpu()
+    return float((got - want).norm() / want.norm().clamp_min(1e-30))
+
+
+def worst_row(got, want):
+    """Largest error of a row of logits (mean taken off) over the rms of the logits."""
+    d = got.double().cpu() - want.double().cpu()
+    d = d - d.mean(-1, keepdim=True)
+    return float(d.pow(2).mean(-1).sqrt().max() / want.double().pow(2).mean().sqrt())
+
+
+def rand(seed):
+    g = torch.Generator().manual_seed(seed)
+    return lambda *s: torch.randn(*s, generator=g)
+
+
+def i32(x, dev):
+    return torch.tensor(x, dtype=torch.int32, device=dev)
+
+
+def shuffled_pages(lens, seed=5):
+    """Block table [sequences, pages] of pages in shuffled order (page 0 stays reserved), and their count."""
+    npg = [(n + 15) // 16 for n in lens]
+    order = torch.randperm(sum(npg), generator=torch.Generator().manual_seed(seed)) + 1
+    table, at = torch.zeros(len(lens), max(npg), dtype=torch.int32), 0
+    for i, n in enumerate(npg):
+        table[i, :n] = order[at:at + n].int()
+        at += n
+    return table, sum(npg) + 1
+
+
+# ------------------------------------------------------------------ windowed attention
+class WindowHeads:
+    """Normed q, k and v of several sequences in pages; attention with a window and a gate by the oracle."""
+
+    def __init__(self, dev, lens, hq, hkv, dk, dv, dtype=BF, seed=0):
+        r = rand(seed)
+        self.dev, self.lens, self.hq, self.hkv, self.dk, self.dv, self.dtype = dev, lens, hq, hkv, dk, dv, dtype
+        self.q, self.k = [r(n, hq, dk).to(dtype) for n in lens], [r(n, hkv, dk).to(dtype) for n in lens]
+        self.v, self.gate = [r(n, hkv, dv).to(dtype) for n in lens], [(2 * r(n, hq)).to(dtype) for n in lens]
+        self.scale = dk ** -0.5
+
+    def build(self):
+        table, count = shuffled_pages(self.lens)
+        kc = torch.zeros(count, self.hkv, 16, pad8(self.dk), dtype=self.dtype)
+        vc = torch.zeros(count, self.hkv, 16, pad8(self.dv), dtype=self.dtype)
+        for s, n in enumerate(self.lens):
+            for t in range(n):
+                kc[table[s, t // 16], :, t % 16, :self.dk] = self.k[s][t]
+                vc[table[s, t // 16], :, t % 16, :self.dv] = self.v[s][t]
+        return kc.to(self.dev), vc.to(self.dev), table.to(self.dev)
+
+    def rows(self, rows):
+        q = torch.zeros(len(rows), self.hq, pad8(self.dk), dtype=self.dtype)
+        for i, (s, t) in enumerate(rows):
+            q[i, :, :self.dk] = self.q[s][t]
+        wide = torch.zeros(len(rows), self.hq + 5, dtype=self.dtype)         # gate logits inside wider rows
+        wide[:, 3:3 + self.hq] = torch.stack([self.gate[s][t] for s, t in rows])
+        return q.to(self.dev), wide.to(self.dev)[:, 3:3 + self.hq]
+
+    def want(self, rows, window):
+        outs = {}
+        for s in {s for s, _ in rows}:
+            q, k, v = (x[s].double().permute(1, 0, 2) for x in (self.q, self.k, self.v))
+            k, v = k.repeat_interleave(self.hq // self.hkv, 0), v.repeat_interleave(self.hq // self.hkv, 0)
+            o = O.softmax_attention(q @ k.transpose(1, 2) * self.scale, O.visible(self.lens[s], window or None), v)
+            outs[s] = o * torch.sigmoid(self.gate[s].double()).T[:, :, None]
+        return torch.stack([outs[s][:, t] for s, t in rows])
+
+    def every_kernel(self, rows, starts, window):
+        """The rows (sequences' tails from ``starts``) through every attention kernel that takes them."""
+        kc, vc, table = self.build()
+        q, gate = self.rows(rows)
+        mods = P.ScoreMods(self.scale)
+        pos, seq = i32([t for _, t in rows], self.dev), i32([s for s, _ in rows], self.dev)
+        new = lambda: torch.full((len(rows), self.hq, pad8(self.dv)), 5.0, dtype=self.dtype, device=self.dev)   # noqa: E731
+        outs = {"any": P.attention_any(q, kc, vc, table, pos, seq, mods, new(), window=window, gate=gate)}
+        if self.dtype == BF and P.prefill_scored_supported(pad8(self.dk), pad8(self.dv)):
+            lens = [n - lo for n, lo in zip(self.lens, starts)]
+            firsts = [sum(lens[:i]) for i in range(len(lens))]
+            for lanes in (1, 2):
+                tiles = i32(query_tiles(firsts, lens, starts, list(range(len(lens))), 128 * lanes), self.dev)
+                outs[f"prompt{lanes}"] = P.flash_prefill_scored(q, kc, vc, table, tiles, mods, new(), window=window,
+                                                                lanes=lanes, gate=gate)
+            for splits in (1, 3):
+                scr = P.ScoredDecodeScratch(len(rows), self.hq, self.hkv, pad8(self.dv), splits, self.dev)
+                outs[f"decode{splits}"] = P.flash_decode_scored(kc, vc, table, pos, mods, new(), scr, self.hq, self.dk,
+                                                                self.dv, q=q, table_rows=seq, window=window, gate=gate)
+        return {n: o[..., :self.dv] for n, o in outs.items()}
+
+
+@pytest.mark.parametrize("shape", [(4, 2, 32, 40), (6, 6, 72, 16), (8, 1, 128, 128), (3, 1, 20, 70), (2, 1, 136, 24)], ids=str)
+@pytest.mark.parametrize("dtype,tol", [(F32, 2e-6), (BF, 7e-3)])
+@pytest.mark.parametrize("window", [0, 1, 16, 37, 1000])
+def test_window_attention_with_gate(dev, shape, dtype, tol, window):
+    h = WindowHeads(dev, [3, 18, 150], *shape, dtype=dtype)
+    starts = [0, 1, 45]
+    rows = [(s, t) for s, lo in enumerate(starts) for t in range(lo, h.lens[s])]
+    want = h.want(rows, window)
+    for name, got in h.every_kernel(rows, starts, window).items():
+        assert rel(got, want) < tol, name
+
+
+def test_window_edge_and_page_borders_stand_out(dev):
+    """A key just inside the window carries most of one query's weight, a like key just outside none."""
+    for window in (1, 15, 16, 17, 33, 64):
+        h = WindowHeads(dev, [220], 2, 1, 64, 32, seed=7)
+        for t in (150, 160, 175, 191):
+            for key in (t - window + 1, t - window):
+                h.k[0][key] = (h.q[0][t].float()[0] * 3).to(BF)
+        rows = [(0, t) for t in range(100, 220)]
+        want = h.want(rows, window)
+        for off in (-1, 1):                                # on the CPU: one token more or less is far off
+            if window + off >= 1:
+                assert rel(h.want(rows, window + off)[[50, 60, 75, 91]], want[[50, 60, 75, 91]]) > 0.2
+        for name, got in h.every_kernel(rows, [100], window).items():
+            assert rel(got, want) < 8e-3, (name, window)
+            for t in (50, 60, 75, 91):
+                assert rel(got[t], want[t]) < 2e-2, (name, window, t)
+
+
+@pytest.mark.parametrize("shape", [(4, 2, 32, 40), (2, 2, 20, 70), (40, 2, 64, 64), (16, 1, 128, 128)], ids=str)
+@pytest.mark.parametrize("window", [0, 17])
+def test_fused_head_norm_append_attention_gate(dev, shape, window):
+    hq, hkv, dk, dv = shape
+    r, lens = rand(3), [1, 16, 17, 200]
+    h = WindowHeads(dev, lens, *shape, seed=2)
+    nq, nk, nv = hq * dk, hkv * dk, hkv * dv
+    raw, qw, kw = torch.randn(4, nq + nk + nv + hq + 3), 1 + 0.3 * r(dk), 1 + 0.3 * r(dk)
+    raw[:, :nq + nk + nv] = r(4, nq + nk + nv)
+    for s, n in enumerate(lens):                          # the oracle's view of the new token
+        h.q[s][n - 1] = O.rms_norm(raw[s, :nq].view(hq, dk), 1e-5, qw).to(BF)
+        h.k[s][n - 1] = O.rms_norm(raw[s, nq:nq + nk].view(hkv, dk), 1e-5, kw).to(BF)
+        h.v[s][n - 1] = raw[s, nq + nk:nq + nk + nv].view(hkv, dv).to(BF)
+        h.gate[s] = h.gate[s].float()
+        h.gate[s][n - 1] = raw[s, nq + nk + nv:nq + nk + nv + hq]
+    want_k, want_v, table = h.build()
+    kc, vc = want_k.clone(), want_v.clone()
+    for s, n in enumerate(lens):                          # the slot of the new token starts dirty
+        kc[table[s, (n - 1) // 16], :, (n - 1) % 16, :dk] = 9.0
+        vc[table[s, (n - 1) // 16], :, (n - 1) % 16, :dv] = -9.0
+    for splits in (1, 5):
+        out = torch.zeros(4, hq, pad8(dv), dtype=BF, device=dev)
+        scr = P.ScoredDecodeScratch(4, hq, hkv, pad8(dv), splits, dev)
+        P.flash_decode_scored(kc, vc, table, i32([n - 1 for n in lens], dev), P.ScoreMods(h.scale), out, scr, hq, dk, dv,
+                              raw=raw.to(dev), q_w=qw.to(dev), k_w=kw.to(dev), eps=1e-5, window=window, head_norm=True,
+                              gate_col=nq + nk + nv)
+        assert rel(out[..., :dv], h.want([(s, n - 1) for s, n in enumerate(lens)], window)) < 7e-3
+        assert rel(kc, want_k) < 2e-3 and torch.equal(vc, want_v)
+
+
+@pytest.mark.parametrize("dtype,tol", [(F32, 1e-6), (BF, 4e-3)])
+@pytest.mark.parametrize("hq,hkv,dk,dv", [(3, 1, 20, 10), (6, 3, 72, 40), (2, 2, 300, 8)])
+def test_head_norm_and_append(dev, dtype, tol, hq, hkv, dk, dv):
+    r, t = rand(1), 37
+    nq, nk, nv = hq * dk, hkv * dk, hkv * dv
+    raw = r(t, pad8(nq + nk + nv)).to(dtype)
+    qw, kw = 1 + 0.2 * r(dk), 1 + 0.2 * r(dk)
+    kc = torch.zeros(9, hkv, 16, pad8(dk), dtype=dtype, device=dev)
+    vc = torch.zeros(9, hkv, 16, pad8(dv), dtype=dtype, device=dev)
+    table = i32([[4, 2, 8], [7, 1, 3]], dev)
+    seq, pos = [0] * 17 + [1] * 20, list(range(14, 31)) + list(range(20))
+    q = torch.full((t, hq, pad8(dk)), 5.0, dtype=dtype, device=dev)
+    N.head_norm_append(raw.to(dev), qw.to(dev), kw.to(dev), 1e-3, q, kc, vc, table, i32(pos, dev), i32(seq, dev), hq, dk, dv)
+    d = raw.double()
+    assert rel(q[..., :dk], O.rms_norm(d[:, :nq].view(t, hq, dk), 1e-3, qw.double())) < tol and not q[..., dk:].any()
+    blk, off = [int(table[s, p // 16]) for s, p in zip(seq, pos)], [p % 16 for p in pos]
+    assert rel(kc[blk, :, off, :dk], O.rms_norm(d[:, nq:nq + nk].view(t, hkv, dk), 1e-3, kw.double())) < tol
+    assert torch.equal(vc[blk, :, off, :dv].cpu(), raw[:, nq + nk:nq + nk + nv].view(t, hkv, dv))
+    assert not kc[..., dk:].any() and not vc[..., dv:].any() and not kc[[0, 5, 6]].any()
+
+
+# ------------------------------------------------------------------ latent attention
+class LatentCase:
+    """A latent-attention sublayer over whole sequences by the oracle, its cache filled by the kernels."""
+
+    def __init__(self, dev, lens, spec, dtype, seed=0, plant=()):
+        self.dev, self.lens, self.m, self.dtype = dev, lens, spec, dtype
+        r = rand(seed)
+        self.width = 40
+        cfg = RodapelConfig(16, self.width, [PostNormLayerSpec(spec, None)], 1e-5).validate()
+        t = {k: v.float() for k, v in M.random_tensors(cfg, seed).items()}
+        self.w = {k[7:]: v.to(dtype) for k, v in t.items() if k.startswith("l0.mix.")}
+        self.w["dkv.norm"] = t["l0.mix.dkv.norm"]
+        self.mw = M.build_weights(cfg, {**t, **{"l0.mix." + k: v for k, v in self.w.items()}}, dev, dtype).layers[0].mix
+        self.h = [r(n, self.width).to(dtype) for n in lens]
+        for s, t, j, gain in plant:                       # token t asks for what token j holds
+            self.h[s][t] = (self.h[s][j].float() * gain).to(dtype)
+
+    def want(self, spec=None):
+        """Attention output before the output projection, per sequence [T, heads * vdim]."""
+        w = {k: v.double() for k, v in self.w.items()}
+        w["o"] = torch.eye(self.m.heads * self.m.vdim, dtype=torch.float64)
+        return [O.latent_attention(w, (spec or self.m).to_json(), 1e-5, h.double()) for h in self.h]
+
+    def run(self, how):
+        """All tokens of all sequences through one form; [sum of lengths, heads, vdim]."""
+        m, mw, dev, dt = self.m, self.mw, self.dev, self.dtype
+        h = torch.zeros(sum(self.lens), pad8(self.width), dtype=dt, device=dev)
+        h[:, :self.width] = torch.cat(self.h).to(dev)
+        t = h.shape[0]
+        raw = N.linear(h, mw.w_in.w, torch.empty(t, mw.w_in.n, dtype=dt, device=dev))
+        table, count = shuffled_pages(self.lens)
+        table = table.to(dev)
+        pool = torch.zeros(count, 1, 16, mw.lat_p + mw.rot_p + 8, dtype=dt, device=dev)
+        pos = i32([p for n in self.lens for p in range(n)], dev)
+        seq = i32([s for s, n in enumerate(self.lens) for _ in range(n)], dev)
+        q = torch.empty(t, m.heads, mw.dim_p + mw.rot_p, dtype=dt, device=dev)
+        q_abs = torch.zeros(t, m.heads, mw.lat_p + mw.rot_p, dtype=dt, device=dev)
+        out = torch.full((t, m.heads, mw.vdim_p), 5.0, dtype=dt, device=dev)
+        N.latent_append(raw, mw.c_norm, 1e-5, mw.inv_freq, q, q_abs, pool, table, pos, seq, m.heads, m.dim, m.rot_dim,
+                        m.kv_rank, mw.dim_p, mw.rot_p, mw.lat_p)
+        if how.startswith("expanded"):
+            first = [sum(self.lens[:i]) for i in range(len(self.lens))]
+            pages = [(s, p) for s, n in enumerate(self.lens) for p in range((n + 15) // 16)]
+            base = {s: 16 * pages.index((s, 0)) for s in range(len(self.lens))}
+            lanes = int(how[-1])
+            tiles = query_tiles(first, self.lens, [0] * len(self.lens), list(range(len(self.lens))), 128 * lanes)
+            ctx = L.latent_gather(pool, table, i32(pages, dev), torch.empty(16 * len(pages), mw.lat_p, dtype=dt, device=dev))
+            kv = torch.empty(16 * len(pages), m.heads, mw.dim_p + mw.vdim_p, dtype=dt, device=dev)
+            N.linear(ctx, mw.w_ukv.w, kv.view(len(ctx), -1))
+            L.flash_prefill_latent(q, kv, pool, mw.lat_p, table, i32(tiles, dev), i32([base[x[3]] for x in tiles], dev),
+                                   m.scale, out, mw.dim_p, lanes=lanes)
+            return out[..., :m.vdim]
+        rows = i32(list(range(t)), dev)
+        N.head_gemv(mw.w_uk, q, q_abs, rows=rows)
+        o_lat = torch.zeros(t, m.heads, mw.lat_p, dtype=dt, device=dev)
+        if how == "any":
+            P.attention_any(q_abs, pool, pool, table, pos, seq, mw.mods, o_lat, rows=rows)
+        else:
+            scr = L.LatentDecodeScratch(t, m.heads, int(how), mw.lat_p, dev)
+            L.latent_decode(q_abs, pool, table, pos, m.scale, o_lat, scr, rows=rows, table_rows=seq)
+        N.head_gemv(mw.w_uv, o_lat, out)
+        return out[..., :m.vdim]
+
+
+LATENT = [LatentAttentionSpec(3, 24, 16, 40, 72, 0.2, 100.0), LatentAttentionSpec(5, 12, 6, 10, 21, 0.3, 500.0),
+          LatentAttentionSpec(2, 128, 64, 128, 128, 0.07, 1e4), LatentAttentionSpec(4, 72, 40, 24, 200, 0.1, 1e4),
+          LatentAttentionSpec(1, 64, 64, 72, 512, 0.09, 1e4, 32)]
+
+
+@pytest.mark.parametrize("spec", LATENT, ids=lambda s: f"{s.heads}-{s.dim}-{s.rot_dim}-{s.vdim}-{s.kv_rank}")
+@pytest.mark.parametrize("dtype,tol", [(F32, 3e-6), (BF, 2e-2)])
+def test_latent_attention_in_every_form(dev, spec, dtype, tol):
+    c = LatentCase(dev, [2, 17, 140], spec, dtype)
+    want = torch.cat(c.want())
+    forms = ["any"]
+    if dtype == BF:
+        if L.prefill_supported(c.mw.dim_p, c.mw.rot_p, c.mw.vdim_p):
+            forms += ["expanded1", "expanded2"]
+        if (spec.kv_rank, spec.rot_dim) in L.DECODE_WIDTHS:
+            forms += ["1", "3"]
+    for how in forms:
+        got = c.run(how)
+        assert rel(got.reshape(len(want), -1), want) < tol, how
+
+
+@pytest.mark.parametrize("spec", [LATENT[0], LATENT[2]], ids=["small", "decode-kernel"])
+def test_a_far_latent_key_stands_out(dev, spec):
+    """Queries that ask strongly for one far token (on page borders, the first token): losing it, or turning
+    it by a wrong angle, shows."""
+    from dataclasses import replace
+    spec = replace(spec, scale=spec.scale * 4)
+    plant = [(0, 290, 0, 1.0), (0, 291, 15, 1.0), (0, 292, 16, 1.0), (0, 299, 143, 1.0)]
+    c = LatentCase(dev, [300], spec, BF, seed=3, plant=plant)
+    want = c.want()[0]
+    rows = [290, 291, 292, 299]
+    lost = LatentCase(dev, [300], spec, BF, seed=3, plant=plant)
+    for _, _, j, _ in plant:
+        lost.h[0][j] = 0
+    turned = replace(spec, rot_base=spec.rot_base * 1.5)
+    assert rel(lost.want()[0][rows], want[rows]) > 0.1 and rel(c.want(turned)[0], want) > 5e-2
+    forms = ["any", "expanded1"] + (["2"] if (spec.kv_rank, spec.rot_dim) in L.DECODE_WIDTHS else [])
+    for how in forms:
+        got = c.run(how).reshape(300, -1)
+        assert rel(got, want) < 3e-2 and rel(got[rows], want[rows]) < 4e-2, how
+
+
+# ------------------------------------------------------------------ WKV
+class WkvCase:
+    def __init__(self, heads, dim, width, rank, seed):
+        self.m, self.width = WkvSpec(heads, dim, rank), width
+        cfg = RodapelConfig(16, width, [PostNormLayerSpec(self.m, None)], 1e-5).validate()
+        self.cfg, self.t = cfg, M.random_tensors(cfg, seed)
+        self.w = {k[7:]: v.double() for k, v in self.t.items() if k.startswith("l0.mix.")}
+
+    def model(self, dev, dtype):
+        return M.RodapelModel(M.build_weights(self.cfg, self.t, dev, dtype))
+
+
+@pytest.mark.parametrize("heads,dim", [(3, 7), (2, 16), (3, 20), (2, 33), (1, 64), (2, 100), (1, 200)])
+@pytest.mark.parametrize("dtype,tol", [(F32, 3e-6), (BF, 6e-3)])
+def test_recurrence_in_portions(dev, heads, dim, dtype, tol):
+    """Several sequences at once, continued over portions of every kind of length, states in shuffled slots."""
+    r, n, ldx = rand(dim), heads * dim, 24
+    lens, slots = [1, 5, 50, 33], [3, 0, 4, 1]
+    ld = pad_to(n, 8)
+    stack = lambda: [r(t, n).to(dtype) for t in lens]                     # noqa: E731
+    rr, k, v = stack(), stack(), stack()
+    dl, u, w0 = [r(t, n) for t in lens], r(heads, dim), -1 + r(n)
+    hf = lambda x: O.heads_first(x.double(), heads)                       # noqa: E731
+    want = [O.heads_last(O.wkv_recurrence(hf(a), hf(b), hf(c), hf(torch.exp(-torch.exp((d + w0).double()))), u.double()))
+            for a, b, c, d in zip(rr, k, v, dl)]
+    pool = torch.zeros(6, n * dim + ldx + (-(n * dim)) % 4, device=dev)
+    pool[5] = 1e4                                         # the idle slot's contents matter to nobody
+    state = pool[:, :n * dim].unflatten(1, (heads, dim, dim))
+    prev = pool[:, pool.shape[1] - ldx:]
+    got, at = [[] for _ in lens], [0] * 4
+    for cut in ([1, 1, 2, 3], [0, 2, 17, 16], [0, 1, 1, 1], [0, 1, 30, 13]):
+        live = [i for i in range(4) if cut[i]]
+        if len(live) == 4 and max(cut) == 3:
+            live = [2, 0, 3, 1]                           # order in the batch does not matter
+        runs, first = [], 0
+        cat = lambda xs: torch.cat([xs[i][at[i]:at[i] + cut[i]] for i in live])             # noqa: E731, B023
+        wide = lambda x: torch.nn.functional.pad(x, (0, ld - n)).to(dev)                    # noqa: E731
+        for i in live:
+            runs.append([first, cut[i], slots[i], at[i]])
+            first += cut[i]
+        x = r(first, ldx).to(dev)
+        o = torch.zeros(first, ld, device=dev)
+        W.wkv_scan(wide(cat(rr)), wide(cat(k)), wide(cat(v)), wide(cat(dl)), w0.to(dev), u.reshape(-1).to(dev), state, prev,
+                   x, o, runs=i32(runs, dev))
+        for (f, c, slot, _), i in zip(runs, live):
+            got[i].append(o[f:f + c, :n].cpu())
+            assert torch.equal(prev[slot], x[f + c - 1])
+            at[i] += c
+    assert at == lens
+    for a, b in zip(got, want):
+        assert rel(torch.cat(a), b) < tol
+    assert not pool[2].any() and float(pool[5].min()) == 1e4
+
+
+def test_state_decays_exactly_over_a_long_past(dev):
+    """One strong key at the start read back hundreds of tokens later through slow decays: a lost or repeated
+    decay step shows."""
+    n, d, t = 2, 32, 600
+    r = rand(9)
+    rr, k, v = 0.01 * r(t, n * d), 0.01 * r(t, n * d), r(t, n * d)
+    k[3], rr[t - 1] = 3.0, 1.0
+    dl, w0 = torch.full((t, n * d), -6.0) + 0.3 * r(t, n * d), torch.zeros(n * d)
+    u = torch.zeros(n * d)
+    hf = lambda x: O.heads_first(x.double(), n)                           # noqa: E731
+    decay = torch.exp(-torch.exp(dl.double()))
+    want = O.heads_last(O.wkv_recurrence(hf(rr), hf(k), hf(v), hf(decay), u.view(n, d).double()))
+    lost = O.heads_last(O.wkv_recurrence(hf(rr), hf(k), hf(v), hf(decay * (torch.arange(t)[:, None] != 300) +
+                                                                  (torch.arange(t)[:, None] == 300)), u.view(n, d).double()))
+    assert rel(lost[-1], want[-1]) > 1e-3
+    pool = torch.zeros(1, n * d * d + 8, device=dev)
+    o = torch.zeros(t, n * d, device=dev)
+    W.wkv_scan(rr.to(dev), k.to(dev), v.to(dev), dl.to(dev), w0.to(dev), u.to(dev), pool[:, :n * d * d].unflatten(1, (n, d, d)),
+               pool[:, n * d * d:], torch.zeros(t, 8, device=dev), o, runs=i32([[0, t, 0, 0]], dev))
+    assert rel(o[-1], want[-1]) < 2e-5
+
+
+@pytest.mark.parametrize("dtype,tol", [(F32, 1e-6), (BF, 4e-3)])
+def test_token_shift_and_head_gate(dev, dtype, tol):
+    r, width, ldx = rand(2), 20, 24
+    x, mu, prev = torch.zeros(9, ldx), torch.zeros(5, ldx), torch.zeros(4, ldx + 4)
+    x[:, :width], mu[:, :width], prev[:, :width] = r(9, width), r(5, width), r(4, width)
+    slots = [2, 2, 2, 0, 3, 3, 3, 3, 1]
+    out = torch.empty(5, 9, ldx, dtype=dtype, device=dev)
+    W.token_shift(x.to(dev), mu.to(dev), prev.to(dev)[:, :ldx], i32(slots, dev), False, out)
+    for lo, hi in ((0, 3), (3, 4), (4, 8), (8, 9)):
+        for s in range(5):
+            seq = torch.cat([prev[slots[lo]:slots[lo] + 1, :ldx], x[lo:hi]]).double()
+            assert rel(out[s, lo:hi], O.token_shift(seq, mu[s].double())[1:]) < tol
+    W.token_shift(x.to(dev), mu.to(dev), prev.to(dev)[:, :ldx], i32(slots, dev), True, out)
+    alone = x.double() + (prev[slots, :ldx].double() - x.double()) * mu[1].double()
+    assert rel(out[1], alone) < tol
+    for heads, dim in ((3, 20), (2, 64), (1, 136)):
+        o, z, w = r(7, heads * dim), r(7, heads * dim).to(dtype), r(heads * dim)
+        a = torch.empty(7, heads * dim, dtype=dtype, device=dev)
+        W.wkv_finish(o.to(dev), z.to(dev), w.to(dev), 1e-3, heads, dim, a)
+        want = O.rms_norm(o.double().view(7, heads, dim), 1e-3).view(7, -1) * w.double() * torch.nn.functional.silu(z.double())
+        assert rel(a, want) < tol
+
+
+@pytest.mark.parametrize("heads,dim,rank", [(3, 20, 5), (2, 64, 64), (1, 130, 16), (2, 256, 8)])
+@pytest.mark.parametrize("b", [1, 3, 6])
+def test_wkv_decode_projections_and_step(dev, heads, dim, rank, b):
+    """Token shift + projections + recurrence + norm + gate of one token per row, twice in a row."""
+    c = WkvCase(heads, dim, 44, rank, 4)
+    model = c.model(dev, BF)
+    mw, wp, r = model.w.layers[0].mix, 48, rand(b)
+    cache = model.new_cache(4, max_seqs=8)
+    slots = torch.randperm(8, generator=torch.Generator().manual_seed(1))[:b]
+    h = r(b, 6, 44)
+    want = [O.time_mix({**c.w, "o": torch.eye(heads * dim, dtype=torch.float64)}, c.m.to_json(), 1e-5, h[i].double())
+            for i in range(b)]
+    state, prev = cache.layer_state(0, "wkv"), cache.layer_state(0, "prev")
+    for t in range(6):
+        x = torch.zeros(b, wp, device=dev)
+        x[:, :44] = h[:, t].to(dev)
+        x2, raw = torch.empty_like(x), torch.empty(b, mw.w_in.n, device=dev)
+        N.postnorm_in(x, N.Pending(None, None), 1e-5, 44, x2, mw.w_in.w, raw,
+                      shift=(mw.mu, prev, slots.int().to(dev), mw.inner_p))
+        a = torch.zeros(b, mw.inner_p, dtype=BF, device=dev)
+        W.wkv_decode(raw, mw.inner_p, mw.w2, mw.w0, mw.u, mw.norm, 1e-5, slots.int().to(dev), state, prev, x2, a)
+        assert torch.equal(x, x2) and torch.equal(prev[slots.to(dev)], x)
+        assert rel(a[:, :heads * dim], torch.stack([w[t] for w in want])) < 6e-3, t
+
+
+# ------------------------------------------------------------------ norms, feed-forward, routing
+@pytest.mark.parametrize("width", [20, 104, 2100])
+@pytest.mark.parametrize("dtype,tol", [(F32, 1e-6), (BF, 4e-3)])
+def test_embedding_norm_and_output_norm(dev, width, dtype, tol):
+    r, t, ldx = rand(width), 7, pad8(width)
+    vec = lambda: torch.nn.functional.pad(1 + 0.3 * r(width), (0, ldx - width))             # noqa: E731
+    table, ids, w = r(30, width).to(dtype), torch.tensor([0, 29, 3, 3, 7, 8, 1]), vec()
+    x, h = torch.full((t, ldx), 9.0, device=dev), torch.full((t, ldx), 9.0, dtype=dtype, device=dev)
+    N.embed_norm(table.to(dev), ids.int().to(dev), w.to(dev), 1e-2, x, h)
+    want = O.rms_norm(table[ids].double(), 1e-2, w[:width].double())
+    assert rel(x[:, :width], want) < 1e-6 and rel(h[:, :width], want) < tol and not x[:, width:].any() and not h[:, width:].any()
+    for ydt in (F32, dtype):
+        y, n = torch.nn.functional.pad(5 * r(t, width), (0, ldx - width)).to(ydt), vec()
+        before = x.clone()
+        N.post_norm_add(y.to(dev), n.to(dev), 1e-2, width, x, h)
+        want = before[:, :width].double().cpu() + O.rms_norm(y[:, :width].double(), 1e-2, n[:width].double())
+        assert rel(x[:, :width], want) < 1e-6 and rel(h[:, :width], want) < tol and not x[:, width:].any()
+
+
+@pytest.mark.parametrize("dtype,tol", [(F32, 3e-6), (BF, 5e-3)])
+@pytest.mark.parametrize("t,width,ff,limit", [(1, 24, 40, 1.0), (130, 104, 200, 0.5), (77, 512, 64, 7.0)])
+def test_clamped_gate_projection(dev, dtype, tol, t, width, ff, limit):
+    r, ffp = rand(t), pad_to(ff, 64)
+    h, g, u = r(t, width).to(dtype), (r(ff, width) / width ** 0.5).to(dtype), (r(ff, width) / width ** 0.5).to(dtype)
+    gu = torch.zeros(2 * ffp, width, dtype=dtype)
+    gu[:ff], gu[ffp:ffp + ff] = g, u
+    act = torch.empty(t, ffp, dtype=dtype, device=dev)
+    N.gated_linear(h.to(dev), LinearWeight(W_BF16, gu.to(dev)), limit, act, torch.empty(t, 2 * ffp, dtype=dtype, device=dev))
+    want = O.clamped_gate_ffn(g.double(), u.double(), torch.eye(ff, dtype=torch.float64), limit, h.double())
+    assert rel(act[:, :ff], want) < tol and not act[:, ff:].any()
+
+
+def _experts(r, e, identity, width, ff, dtype):
+    w = {"router": r(e + identity, width) / width ** 0.5, "correction": 0.3 * r(e + identity)}
+    for i in range(e):
+        w.update({f"e{i}.gate": r(ff, width) / width ** 0.5, f"e{i}.up": r(ff, width) / width ** 0.5,
+                  f"e{i}.down": r(width, ff) / ff ** 0.5})
+    return {k: v if k == "correction" else v.to(dtype) for k, v in w.items()}
+
+
+@pytest.mark.parametrize("e,identity,top", [(5, 0, 1), (6, 3, 3), (3, 2, 5), (40, 30, 8), (200, 100, 12)])
+def test_corrected_routing(dev, e, identity, top):
+    r, t = rand(e), 53
+    n = e + identity
+    z, corr = 2 * r(t, n), 0.2 * r(n)
+    i = lambda *s: torch.zeros(*s, dtype=torch.int32, device=dev)         # noqa: E731
+    rt = R.Routing(i(t, top), torch.zeros(t, top, device=dev), torch.zeros(t, device=dev), i(e), i(e + 1), i(t, top))
+    R.route_corrected(z.to(dev), corr.to(dev), e, rt)
+    idx, wt = O.route(torch.eye(n, dtype=torch.float64), corr.double(), top, z.double())
+    assert torch.equal(rt.idx.cpu().sort(1).values.long(), idx.sort(1).values)
+    order = rt.idx.cpu().long()
+    s = torch.softmax(z.double(), -1).gather(1, order)
+    assert rel(rt.weights, s) < 1e-6
+    assert torch.allclose(rt.identity.cpu().double(), (s * (order >= e)).sum(1), atol=1e-6)
+    count = torch.bincount(order[order < e], minlength=e)
+    assert torch.equal(rt.offsets.cpu().long(), torch.cat([torch.zeros(1, dtype=torch.long), count.cumsum(0)]))
+    x = r(t, 24).to(BF)
+    xs = torch.zeros(t * top, 24, dtype=BF, device=dev)
+    R.route_scatter(x.to(dev), rt, xs)
+    rows = rt.row_of_pair.cpu().long()
+    assert ((rows < 0) == (order >= e)).all() and len(set(rows[rows >= 0].tolist())) == int((order < e).sum())
+    for a in range(t):
+        for b in range(top):
+            if rows[a, b] >= 0:
+                lo, hi = rt.offsets[order[a, b]], rt.offsets[order[a, b] + 1]
+                assert lo <= rows[a, b] < hi and torch.equal(xs[rows[a, b]].cpu(), x[a])
+
+
+@pytest.mark.parametrize("dtype,tol", [(F32, 5e-6), (BF, 1e-2)])
+@pytest.mark.parametrize("t,e,identity,top", [(1, 3, 1, 2), (70, 6, 2, 3), (300, 4, 0, 1), (9, 2, 6, 6)])
+def test_routed_feed_forward_with_its_norm(dev, dtype, tol, t, e, identity, top):
+    width, ff = 44, 40
+    cfg = RodapelConfig(16, width, [PostNormLayerSpec(WkvSpec(1, 8), RoutedFfSpec(e, identity, top, ff, 1.2))], 1e-4).validate()
+    r = rand(t)
+    tensors = M.random_tensors(cfg, 7, dtype=F32)
+    mlp = {k[7:]: v.to(dtype) for k, v in tensors.items() if k.startswith("l0.mlp.")}
+    mlp.update(_experts(r, e, identity, width, ff, dtype))
+    tensors.update({"l0.mlp." + k: v for k, v in mlp.items()})
+    model = M.RodapelModel(M.build_weights(cfg, tensors, dev, dtype))
+    lw = model.w.layers[0]
+    x = torch.zeros(t, 48, device=dev)
+    x[:, :width] = r(t, width).to(dtype).float().to(dev)
+    before, h = x[:, :width].double().cpu(), x.to(dtype)
+    bufs = M.Buffers(max(t, 8), dev)
+    c = M.StepContext(t, bufs, None, None, None, None, None, None)
+    model.routed_ff(lw, lw.mlp, x, h, c)
+    y = O.expert_mix({k: v.double() for k, v in mlp.items()}, cfg.layers[0].mlp.to_json(), before)
+    want = before + O.rms_norm(y, 1e-4, tensors["l0.norm2"].double())
+    assert rel(x[:, :width] - before.to(dev), want - before) < tol
+    assert rel(h[:, :width], want) < (1e-6 if dtype == F32 else 5e-3) and not x[:, width:].any()
+
+
+@pytest.mark.parametrize("b", [1, 3, 6])
+@pytest.mark.parametrize("pending", [False, True])
+def test_decode_projections(dev, b, pending):
+    """The mat-vec kernels that finish the previous sublayer on the way: projection, gated, router, experts."""
+    r, d, k = rand(b), 100, 104
+    pad = lambda v: torch.nn.functional.pad(v, (0, k - v.shape[-1]))      # noqa: E731
+    x, y, nw = pad(3 * r(b, d)), pad(2 * r(b, d)), pad(1 + 0.2 * r(d))
+    pend = N.Pending(y.to(dev), nw.to(dev)) if pending else N.Pending(None, None)
+    xf = x[:, :d].double()
+    if pending:
+        xf = xf + O.rms_norm(y[:, :d].double(), 1e-4, nw[:d].double())
+    w = pad(r(75, d) / 10).to(BF)
+    x2, out = torch.full((b, k), 7.0, device=dev), torch.empty(b, 75, device=dev)
+    N.postnorm_in(x.to(dev), pend, 1e-4, d, x2, w.to(dev), out)
+    assert rel(x2[:, :d], xf) < 1e-6 and not x2[:, d:].any() and rel(out, xf @ w[:, :d].double().T) < 3e-6
+    gu = pad(r(2 * 40, d) / 10).to(BF)
+    act = torch.empty(b, 40, dtype=BF, device=dev)
+    N.postnorm_gated(x.to(dev), pend, 1e-4, d, x2, gu.to(dev), 1.1, act)
+    want = O.clamped_gate_ffn(gu[:40, :d].double(), gu[40:, :d].double(), torch.eye(40, dtype=torch.float64), 1.1, xf)
+    assert rel(act, want) < 5e-3
+    wd = r(d, 40).to(BF)
+    assert rel(N.matvec_out(act, wd.to(dev), torch.empty(b, d, device=dev)), act.double().cpu() @ wd.double().T) < 3e-6
+    e, identity, top, ff = 5, 3, 4, 64
+    ew = _experts(r, e, identity, d, ff, BF)
+    i = lambda *s: torch.zeros(*s, dtype=torch.int32, device=dev)         # noqa: E731
+    rt = R.Routing(i(b, top), torch.zeros(b, top, device=dev), torch.zeros(b, device=dev), i(e), i(e + 1), i(b, top))
+    z, ticket = torch.empty(b, e + identity, device=dev), i(1)
+    for _ in range(2):                                    # the ticket is left clean
+        R.postnorm_router(x.to(dev), pend, 1e-4, d, x2, pad(ew["router"].float()).to(BF).to(dev), ew["correction"].to(dev), e,
+                          z, ticket, rt)
+    stack = lambda n: torch.stack([ew[f"e{j}.{n}"] for j in range(e)])    # noqa: E731
+    gus = pad(torch.cat([stack("gate"), stack("up")], 1).float()).to(BF).to(dev)
+    downs = torch.zeros(e, 128, ff, dtype=BF, device=dev)
+    downs[:, :d] = stack("down").to(dev)
+    acte, yo = torch.zeros(b * top, ff, dtype=BF, device=dev), torch.full((b, k), 7.0, device=dev)
+    R.postnorm_expert(x2, gus, 1.1, rt, acte)
+    R.expert_out(acte, downs, rt, x2, yo)
+    want = O.expert_mix({n: v.double() for n, v in ew.items()}, RoutedFfSpec(e, identity, top, ff, 1.1).to_json(), xf)
+    assert rel(yo[:, :d], want) < 8e-3 and not yo[:, d:].any()
+
+
+def test_gate_limit_of_the_grouped_gemm_switches_the_activation(dev):
+    r = rand(1)
+    x, w = r(200, 64).to(BF), (r(256, 64) / 8).to(BF)
+    lw = LinearWeight(W_BF16, w.to(dev))
+    g, u = (x.double() @ w.double().T).chunk(2, 1)
+    assert rel(xgemm(x.to(dev), lw, swiglu=True), torch.nn.functional.silu(g) * u) < 5e-3
+    g, u = g.clamp(max=0.7), u.clamp(-0.7, 0.7)
+    assert rel(xgemm(x.to(dev), lw, swiglu=True, gate_limit=0.7), g * torch.sigmoid(1.702 * g) * (u + 1)) < 5e-3
+
+
+# ------------------------------------------------------------------ the model
+def odd_cfg():
+    """Widths and ranks that are not multiples of eight, single heads, a layer without feed-forward, top equal
+    to the outputs, no identity experts; latent widths of the decode kernel; two WKV layers in a row."""
+    A, K, Q, S = WindowAttentionSpec, LatentAttentionSpec, WkvSpec, PostNormLayerSpec
+    return RodapelConfig(83, 100, [
+        S(K(3, 20, 10, 14, 50, 0.2, 300.0), RoutedFfSpec(3, 0, 2, 50, 1.0)), S(Q(1, 72, 12), None), S(Q(5, 9, 20), ClampedFfSpec(70, 4.0)),
+        S(A(5, 5, 12, 20, 0.3, 1), ClampedFfSpec(33, 0.8)), S(K(2, 64, 64, 72, 128, 0.1, 1e4), RoutedFfSpec(2, 2, 4, 64, 2.0)),
+        S(A(3, 1, 100, 36, 0.12, 65), RoutedFfSpec(9, 1, 1, 40, 1.5))], 1e-3).validate()
+
+
+def wide_cfg():
+    """Head sizes outside the tensor-core attention kernels; attention without a window."""
+    A, K, Q, S = WindowAttentionSpec, LatentAttentionSpec, WkvSpec, PostNormLayerSpec
+    return RodapelConfig(65, 44, [S(A(2, 1, 136, 20, 0.1, 0), ClampedFfSpec(30, 2.0)), S(K(2, 140, 16, 30, 40, 0.1, 1e3), None),
+                                  S(Q(1, 144, 4), RoutedFfSpec(4, 2, 2, 24, 1.0))], 1e-4).validate()
+
+
+CFGS = {"tiny": M.rodapel_tiny, "odd": odd_cfg, "wide": wide_cfg}
+TOL = {F32: 3e-5, BF: 6e-2}
+
+
+class Bench:
+    """A random model with its plain counterpart; prompts' logits are computed once."""
+
+    def __init__(self, dev, name, dtype):
+        self.cfg = CFGS[name]()
+        # router logits well apart, so that rounding does not change who is chosen
+        self.tensors = {k: (v.float() * 3 if k.endswith(".router") else v.float()).to(BF)
+                        for k, v in M.random_tensors(self.cfg, 11).items()}
+        self.model = M.RodapelModel(M.build_weights(self.cfg, self.tensors, dev, dtype))
+        self.dtype, self._ref, self._w = dtype, {}, {k: v.double() for k, v in self.tensors.items()}
+
+    def tokens(self, n, seed):
+        return torch.randint(0, self.cfg.vocab_size, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+    def ref(self, toks):
+        key = tuple(toks)
+        if key not in self._ref:
+            self._ref[key] = O.forward(self.cfg.to_json(), self._w, toks)
+        return self._ref[key]
+
+    def engine(self, blocks=80, batch=4, **kw):
+        return ServingEngine(self.model, blocks, SchedulerConfig(max_batch_size=batch, **kw))
+
+    def close(self, got, want):
+        """32-bit: every row. bf16: nearly every row (a close choice of experts may flip), and all on average."""
+        if self.dtype == F32:
+            return worst_row(got, want) < TOL[F32]
+        d = got.double().cpu() - want.double().cpu()
+        d = d - d.mean(-1, keepdim=True)
+        err = d.pow(2).mean(-1).sqrt() / want.double().pow(2).mean().sqrt()
+        return float((err > TOL[BF]).double().mean()) <= 0.06 and float(err.median()) < TOL[BF] / 2
+
+
+@pytest.fixture(scope="module", params=[(n, d) for n in CFGS for d in (F32, BF)], ids=lambda p: f"{p[0]}-{str(p[1])[6:]}")
+def bench(request):
+    return Bench(torch.device("cuda:0"), *request.param)
+
+
+def test_layers_one_by_one(bench):
+    toks, want = bench.tokens(23, 1), []
+    O.forward(bench.cfg.to_json(), bench._w, toks, lambda i, x: want.append(x))
+    cache = bench.model.new_cache(4, max_seqs=1)
+    cache.add_sequence(0)
+    errs = []
+    bench.model.forward_batch([Entry(0, toks, [22])], cache, observe=lambda li, x: errs.append(rel(x, want[li])))
+    assert len(errs) == bench.cfg.num_layers and max(errs) < (2e-5 if bench.dtype == F32 else 6e-2)
+
+
+@pytest.mark.parametrize("cuts", [[150], [2] * 20 + [110], [1] * 9 + [141], [16, 16, 15, 17, 3, 83], [64, 1, 64, 1, 1, 19],
+                                  [129, 2, 2, 1, 1, 1, 14], [5] * 30], ids=str)
+def test_a_prompt_in_portions(bench, cuts):
+    toks = bench.tokens(150, 2)
+    want = bench.ref(toks)
+    eng = bench.engine()
+    sid, at, got = eng.open_sequence(), 0, []
+    for n in cuts:
+        got.append(eng.run_entries([Entry(sid, toks[at:at + n], range(n))]))
+        at += n
+    assert at == 150 and bench.close(torch.cat(got), want)
+
+
+def test_unequal_requests_together_and_slots_again(bench):
+    """Four slots, ten requests of different lengths whose portions and decoded tokens share steps; pages and
+    slots are used again, some requests pause, the pool is just large enough."""
+    lens = [1, 2, 17, 70, 33, 5, 128, 16, 40, 64]
+    reqs = [bench.tokens(n, 20 + i) for i, n in enumerate(lens)]
+    eng = bench.engine(blocks=1 + (128 + 64 + 64 + 80) // 16)
+    gen = torch.Generator().manual_seed(4)
+    live, waiting, got, step = {}, list(range(10)), {i: [] for i in range(10)}, 0
+    while live or waiting:
+        while waiting and len(live) < 4:
+            i = waiting.pop(0)
+            live[i] = [eng.open_sequence(), 0]
+        step += 1
+        batch, order = [], []
+        for i, (sid, at) in live.items():
+            if (step + i) % 5 == 0 and len(live) > 1:
+                continue                                  # this one pauses
+            n = min(lens[i] - at, int(torch.tensor([1, 1, 2, 3, 13, 40])[torch.randint(6, (1,), generator=gen)]))
+            batch.append(Entry(sid, reqs[i][at:at + n], range(n)))
+            order.append((i, n))
+        if not batch:
+            continue
+        out, lo = eng.run_entries(batch), 0
+        for i, n in order:
+            got[i].append(out[lo:lo + n].cpu())
+            lo += n
+            live[i][1] += n
+            if live[i][1] == lens[i]:
+                eng.close_sequence(live.pop(i)[0])
+    for i, toks in enumerate(reqs):
+        assert bench.close(torch.cat(got[i]), bench.ref(toks)) or len(toks) < 20, i
+    assert bench.close(torch.cat([torch.cat(got[i]) for i in range(10)]), torch.cat([bench.ref(t) for t in reqs]))
+
+
+def test_result_does_not_depend_on_company_or_pages(bench):
+    """One request alone on fresh pages, and in a crowd on used pages: the same up to rounding."""
+    toks = bench.tokens(60, 40)
+    a = bench.engine()
+    s = a.open_sequence()
+    alone = torch.cat([a.run_entries([Entry(s, toks[:50], range(50))])] +
+                      [a.run_entries([Entry(s, [t], [0])]) for t in toks[50:]])
+    b = bench.engine()
+    junk = [b.open_sequence() for _ in range(3)]
+    b.run_entries([Entry(j, bench.tokens(30 + j, 50 + j), ()) for j in junk])
+    b.close_sequence(junk[1])
+    s = b.open_sequence()
+    crowd = [b.run_entries([Entry(junk[0], [3, 4], ()), Entry(s, toks[:50], range(50))])]
+    for t in toks[50:]:
+        crowd.append(b.run_entries([Entry(junk[2], [5], ()), Entry(s, [t], [0])]))
+    assert worst_row(torch.cat(crowd), alone) < 2e-5 if bench.dtype == F32 else bench.close(torch.cat(crowd), alone)
+
+
+def test_long_decoding(bench):
+    toks = bench.tokens(310, 60)
+    want = bench.ref(toks)
+    eng = bench.engine()
+    s = eng.open_sequence()
+    got = [eng.run_entries([Entry(s, toks[:3], range(3))])]
+    got += [eng.run_entries([Entry(s, [t], [0])]) for t in toks[3:]]
+    assert bench.close(torch.cat(got), want)
+
+
+@pytest.mark.parametrize("rows", [1, 3, 5, 16])
+def test_decode_engine_buckets(bench, rows):
+    """The captured step at several batch sizes (mat-vec and GEMM forms, idle rows), graph and eager; recording a
+    step leaves no trace in the recurrent state, and rows keep their own."""
+    prompts = [bench.tokens(4 + 7 * i % 40, 70 + i) for i in range(rows)]
+    for use_graph in (True, False):
+        cache = bench.model.new_cache(120, max_seqs=16)
+        eng = PostNormDecode(bench.model, cache, max_batch=16, use_graph=use_graph)
+        for i, p in enumerate(prompts):
+            cache.add_sequence(i)
+            bench.model.prefill(torch.tensor(p[:-2]), cache, i)
+        eng.bind(list(range(rows)), [p[-2] for p in prompts])
+        eng.reserve(2)
+        got = []
+        for k in (-1, 0):
+            eng.step()
+            got.append(eng.logits[:rows].clone())
+            if k:
+                eng.set_next_tokens([p[-1] for p in prompts])
+        for j in (0, 1):
+            want = torch.stack([bench.ref(p)[j - 2] for p in prompts])
+            assert bench.close(got[j], want) or (bench.dtype == BF and rows < 16 and
+                                                 rel(got[j], want) < 0.3), (use_graph, j)
+        assert eng.launches_per_step > 0
+
+
+def test_fork_copies_the_state(bench):
+    toks = bench.tokens(40, 3)
+    cache = bench.model.new_cache(20, max_seqs=3)
+    cache.add_sequence(0)
+    bench.model.prefill(torch.tensor(toks[:30]), cache, 0)
+    cache.fork(0, 1)
+    a = bench.model.forward_batch([Entry(1, toks[30:], range(10)), Entry(0, [1, 2, 3], ())], cache)
+    assert bench.close(a, bench.ref(toks)[30:])
+
+
+def _check_greedy(bench, prompt, got):
+    """Every chosen token is the plain model's, or within rounding of its best logit."""
+    hist = list(prompt)
+    for t in got:
+        lg = bench.ref(hist)[-1]
+        slack = (2e-4 if bench.dtype == F32 else 0.3) * float(lg.std())
+        assert float(lg.max() - lg[t]) <= slack
+        hist.append(t)
+
+
+def test_greedy_generation_through_the_scheduler(bench):
+    prompts = [bench.tokens(n, 90 + n) for n in (1, 19, 50, 3, 33, 16)]
+    eng = bench.engine(batch=3, max_prefill_chunk=16)
+    ids = [eng.submit(p, 5) for p in prompts]
+    out = eng.run_until_done()
+    for sid, p in zip(ids, prompts):
+        assert len(out[sid]) == 5
+        _check_greedy(bench, p, out[sid])
+    p = prompts[1]
+    got = bench.model.generate_greedy(torch.tensor(p), 5)
+    assert len(got) == 5
+    _check_greedy(bench, p, got)
+
+
+def test_sampling_through_the_engine(bench):
+    eng = ServingEngine(bench.model, 60, SchedulerConfig(max_batch_size=2, max_prefill_chunk=16),
+                        SamplerConfig(temperature=0.8, top_k=5, seed=3))
+    ids = [eng.submit(bench.tokens(20, 7), 6), eng.submit(bench.tokens(4, 8), 6)]
+    out = eng.run_until_done()
+    for sid, seed, n in zip(ids, (7, 8), (20, 4)):
+        hist = bench.tokens(n, seed)
+        for t in out[sid]:
+            assert t in bench.ref(hist)[-1].topk(14).indices.tolist()
+            hist.append(t)
+
+
+def test_warm_up_and_other_entry_points(bench):
+    eng = bench.engine(batch=2)
+    eng.warm_up(prompt_len=5, new_tokens=2)
+    assert eng.cache.manager.num_free_blocks() >= 70
+    toks = bench.tokens(40, 5)
+    assert bench.close(bench.model.forward(torch.tensor(toks)), bench.ref(toks))
+    s = eng.open_sequence()                               # a slot the warm-up has used
+    assert bench.close(eng.run_entries([Entry(s, toks, range(40))]), bench.ref(toks))
+
+
+def test_command_line_generation_and_trace(tmp_path, dev):
+    from rmlx_b200.cli.main import main
+    b = Bench(dev, "odd", F32)
+    M.save_checkpoint(str(tmp_path / "m"), b.cfg, b.tensors)
+    prompt = [5, 9, 80, 3]
+    out, real = io.StringIO(), sys.stdout
+    sys.stdout = out
+    try:
+        assert main(["generate", "--model", str(tmp_path / "m"), "--prompt", "5,9,80,3", "--steps", "4",
+                     "--dtype", "float32"]) == 0
+    finally:
+        sys.stdout = real
+    toks = json.loads(out.getvalue().splitlines()[-1])["tokens"]
+    assert len(toks) == 1 and len(toks[0]) == 4
+    _check_greedy(b, prompt, toks[0])
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": prompt[:3], "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "x", "tokens": prompt[3:], "want": [0]},
+                                     {"id": "y", "tokens": [1, 2], "want": [1, 0]}], "end": ["x", "y"]},
+             {"step": 2, "entries": [{"id": "x", "tokens": [1, 2], "want": [1]}], "end": ["x"]}]
+    (tmp_path / "o").mkdir()
+    out, real_in = io.StringIO(), sys.stdin
+    sys.stdin, sys.stdout = io.StringIO("".join(json.dumps(s) + "\n" for s in steps)), out
+    try:
+        assert main(["trace-run", "--model", str(tmp_path / "m"), "--dtype", "float32", "--out", str(tmp_path / "o"),
+                     "--max-tokens", "128"]) == 0
+    finally:
+        sys.stdin, sys.stdout = real_in, real
+    assert out.getvalue().split() == ["done", "0", "done", "1", "done", "2"] and not (tmp_path / "o" / "0.f32").exists()
+
+    def read(name):
+        data = (tmp_path / "o" / name).read_bytes()
+        return torch.tensor(struct.unpack(f"<{len(data) // 4}f", data)).view(-1, b.cfg.vocab_size)
+
+    want = torch.stack([b.ref(prompt)[-1], b.ref([1, 2])[1], b.ref([1, 2])[0]])
+    assert worst_row(read("1.f32"), want) < TOL[F32] and worst_row(read("2.f32"), b.ref([1, 2])[1:]) < TOL[F32]
