@@ -295,7 +295,8 @@ def prefill_kernels(tab: Table, model: RodapelModel, t: int):
     tab.add(ph, "wkv: decay, first factor", [lambda w=w: P.logits_f32(mix[4], w.part(4), low) for _, w, _ in wkv], gemm(w0.rank_p, d, 4))
     tab.add(ph, "wkv: decay, second factor", [lambda w=w: P.logits_f32(low_t, w.w2, decay) for _, w, _ in wkv],
             gemm(inner, w0.rank_p, 4))
-    tab.add(ph, "wkv: recurrence", [lambda i=i, w=w: W.wkv_scan(rkvg[0], rkvg[1], rkvg[2], decay, w.w0, w.u, *st(i), x, o,
+    rec = torch.empty(t * m.heads * W.record(m.dim), device=dev)
+    tab.add(ph, "wkv: recurrence", [lambda i=i, w=w: W.wkv_scan(rkvg[0], rkvg[1], rkvg[2], decay, w.w0, w.u, *st(i), x, o, rec,
                                                                 runs=batch.runs) for i, w, _ in wkv],
             (t * inner * (6 + 4 + 4), 0, 3.0 * t * inner * m.dim))
     tab.add(ph, "wkv: head norm + gate", [lambda w=w: W.wkv_finish(o, rkvg[3], w.norm, 1e-6, m.heads, m.dim, a) for _, w, _ in wkv],

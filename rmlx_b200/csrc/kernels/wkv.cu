@@ -4,12 +4,14 @@
 // Per head, with S [dim, dim] (rows: key channels, columns: value channels) carried per sequence:
 //     o_t = (S + diag(u) k_t v_t^T)^T r_t,   S <- diag(w_t) S + k_t v_t^T,
 //     w_t = exp(-exp(dl_t + w0))
-// Columns are independent of each other. A block owns one (sequence, head, group of columns) and walks
-// the sequence's new tokens. A thread holds ROWS rows of four columns in registers (each r, k and w read from
-// shared memory then serves four columns: shared-memory wavefronts, not arithmetic, are what one column per
-// thread is bound by); LANES threads share a column and add their parts by a transposing butterfly. Half of the
-// block's warps fetch tokens ahead, take the exponentials and r . (u k), and stage the next chunk while the
-// other half runs the current one. Arithmetic on the state runs on pairs (fma.rn.f32x2).
+// Columns are independent of each other. wkv_prepare takes the exponentials once per head and writes one fp32
+// record per (head, token): r, k, w, v and r . (u k), the records of a head in token order. wkv_scan: a block
+// owns one (sequence, head, group of columns) and walks the sequence's new tokens, whose records arrive in
+// shared memory by one bulk copy per chunk, two chunks ahead: no instruction of the scan is spent on staging
+// (when the block converted its own inputs, that took more issue slots than the recurrence). A thread holds
+// ROWS rows of four columns in registers, so that each r, k and w it reads serves four columns; LANES threads
+// share a column and add their parts by a transposing butterfly. Arithmetic on the state runs on pairs
+// (fma.rn.f32x2).
 //
 // The state of a sequence lives in its slot's row of a flat fp32 pool, beside the last token's
 // residual row, which the token shift of the sequence's next token needs.
@@ -68,15 +70,83 @@ __device__ __forceinline__ uint64_t wk_mul(uint64_t a, uint64_t b) {
   return d;
 }
 
+constexpr int kWkThreads = 64, kWkCols = 4, kWkStages = 3;       // columns per thread; chunks in flight
+template <int ROWS, int LANES>
+struct WkCfg {
+  static constexpr int kDim = ROWS * LANES;          // padded rows of the state
+  static constexpr int kCols = kWkThreads / LANES * kWkCols;     // columns per block
+  static constexpr int kChunk = kDim > 128 ? 8 : 16;             // tokens per chunk
+  static constexpr int kV = (kDim + kCols - 1) / kCols * kCols;  // padded columns
+  static constexpr int kRec = 3 * kDim + kV + 4;                 // floats of a record
+  static constexpr int kSmem = kWkStages * kChunk * kRec * 4 + 64;
+};
+
+// Where value i of r, k or w sits in a record: row group g's values four at a time, so that the 16-byte pieces
+// of consecutive groups are neighbours.
+template <int ROWS, int LANES>
+__device__ __forceinline__ int wk_at(int i) {
+  return (i % ROWS) / 4 * (LANES * 4) + i / ROWS * 4 + i % 4;
+}
+
+// rec[h][t] of all heads and rows. LU lanes per record, four values each per turn.
+template <class T, int ROWS, int LANES, int LU>
+__global__ void __launch_bounds__(kRowThreads)
+wkv_prepare_kernel(const T* __restrict__ r, const T* __restrict__ k, const T* __restrict__ v, int ld,
+                   const float* __restrict__ dl, int ld_dl, const float* __restrict__ w0, const float* __restrict__ u,
+                   float* __restrict__ rec, int rows, int H, int dim) {
+  using C = WkCfg<ROWS, LANES>;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int unit = (blockIdx.x * kRowThreads + threadIdx.x) / LU, lane = threadIdx.x % LU;
+  const bool live = unit < rows * H;                 // the lanes of a warp stay together for the sum
+  const int t = live ? unit / H : 0, h = live ? unit - t * H : 0;
+  float* out = rec + (size_t(h) * rows + t) * C::kRec;
+  const bool vec = dim % 4 == 0 && ld % 4 == 0 && ld_dl % 4 == 0;
+  auto load4 = [&](const T* p, int i, float (&f)[4]) {
+    if (vec && i < dim) {
+      if (sizeof(T) == 2) {
+        const uint2 q = *reinterpret_cast<const uint2*>(p + i);
+        f[0] = bf16lo(q.x); f[1] = bf16hi(q.x); f[2] = bf16lo(q.y); f[3] = bf16hi(q.y);
+      } else {
+        const float4 q = *reinterpret_cast<const float4*>(p + i);
+        f[0] = q.x; f[1] = q.y; f[2] = q.z; f[3] = q.w;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) f[j] = i + j < dim ? to_f32(p[i + j]) : 0.f;
+    }
+  };
+  const size_t at = size_t(t) * ld + h * dim;
+  const float* dp = dl + size_t(t) * ld_dl + h * dim;
+  float ruk = 0.f;
+  for (int i = lane * 4; i < C::kV || i < C::kDim; i += LU * 4) {
+    float fr[4], fk[4], fv[4], fw[4];
+    load4(r + at, i, fr);
+    load4(k + at, i, fk);
+    load4(v + at, i, fv);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const bool in = i + j < dim;
+      fw[j] = in ? expf(-expf(dp[in ? i + j : 0] + w0[h * dim + (in ? i + j : 0)])) : 1.f;
+      ruk = fmaf(fr[j] * (in ? u[h * dim + i + j] : 0.f), fk[j], ruk);
+    }
+    if (live) {
+      if (i < C::kDim) {
+        float* o = out + wk_at<ROWS, LANES>(i);
+        *reinterpret_cast<float4*>(o) = make_float4(fr[0], fr[1], fr[2], fr[3]);
+        *reinterpret_cast<float4*>(o + C::kDim) = make_float4(fk[0], fk[1], fk[2], fk[3]);
+        *reinterpret_cast<float4*>(o + 2 * C::kDim) = make_float4(fw[0], fw[1], fw[2], fw[3]);
+      }
+      if (i < C::kV) *reinterpret_cast<float4*>(out + 3 * C::kDim + i) = make_float4(fv[0], fv[1], fv[2], fv[3]);
+    }
+  }
+  ruk = group_sum<LU>(ruk);
+  if (live && lane == 0) *reinterpret_cast<float4*>(out + 3 * C::kDim + C::kV) = make_float4(ruk, 0.f, 0.f, 0.f);
+}
+
 struct WkvParams {
-  const void* r;            // [rows, ld] each, head h at column h * dim
-  const void* k;
-  const void* v;
-  int ld;
-  const float* dl;          // [rows, ld_dl] decay logits before w0
-  int ld_dl;
-  const float* w0;          // [H * dim]
-  const float* u;           // [H * dim]
+  const float* rec;         // [H, rows, kRec]
+  int rows;
   const int4* segs;         // {first row, rows, slot, -}; null: segment i is row i with slot slots[i]
   const int* slots;
   float* state;             // slot s: state + s * stride, [H, dim, dim]
@@ -87,25 +157,23 @@ struct WkvParams {
   float* out;               // [rows, ld_out] fp32
   int ld_out;
   int H, dim;
+  int* status;
 };
 
-constexpr int kWkHalf = 64, kWkCols = 4;            // compute (and staging) threads; columns per thread
 template <int ROWS, int LANES>
-struct WkCfg {
-  static constexpr int kDim = ROWS * LANES;          // padded rows of the state
-  static constexpr int kCols = kWkHalf / LANES * kWkCols;        // columns per block
-  static constexpr int kChunk = kDim > 128 ? 4 : kDim > 64 ? 8 : 16;   // tokens per chunk
-  static constexpr int kTok = 3 * kDim + kCols + 4;              // r, k, w, v, r . (u k)
-  static constexpr int kSmem = 2 * kChunk * kTok * 4;
-};
-
-template <class T, int ROWS, int LANES>
-__global__ void __launch_bounds__(2 * kWkHalf) wkv_scan_kernel(WkvParams p) {
+__global__ void __launch_bounds__(kWkThreads) wkv_scan_kernel(WkvParams p) {
   using C = WkCfg<ROWS, LANES>;
-  extern __shared__ __align__(16) float smem[];
+  extern __shared__ __align__(128) float smem[];
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem + kWkStages * C::kChunk * C::kRec);      // [stages]
+  __shared__ uint32_t gave_up;
+  const int h = blockIdx.y, col0 = blockIdx.x * C::kCols, dim = p.dim;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kWkStages; ++i) mbar_init(full + i, 1);
+    gave_up = 0u;
+    fence_mbar_init();
+  }
   pdl_launch_dependents();
   pdl_wait();
-  const int h = blockIdx.y, col0 = blockIdx.x * C::kCols;
   int row0, len, slot;
   if (p.segs) {
     const int4 s = p.segs[blockIdx.z];
@@ -113,179 +181,146 @@ __global__ void __launch_bounds__(2 * kWkHalf) wkv_scan_kernel(WkvParams p) {
   } else {
     row0 = blockIdx.z; len = 1; slot = p.slots[blockIdx.z];
   }
-  const int dim = p.dim, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  constexpr int SW = kWkHalf / 32;                               // staging warps
-  const bool stager = warp >= SW;
+  __syncthreads();                                   // the barriers are initialised
   const int chunks = (len + C::kChunk - 1) / C::kChunk;
-
-  // A stager warp holds the raw values of its tokens of one chunk: they are asked for one chunk before they
-  // are converted, so that the loads run beside the recurrence.
-  constexpr int M = (C::kDim + 31) / 32;                         // key channels per lane
-  constexpr int VM = (C::kCols + 31) / 32;
-  constexpr int PER = C::kChunk / SW;                            // tokens per warp
-  T fr[PER][M], fk[PER][M], fv[PER][VM];
-  float fd[PER][M], w0[M], uu[M];
-  const T* rp = static_cast<const T*>(p.r) + h * dim;
-  const T* kp = static_cast<const T*>(p.k) + h * dim;
-  const T* vp = static_cast<const T*>(p.v) + h * dim + col0;
-  const float* dp = p.dl + h * dim;
-  auto fetch = [&](int ch) {
-#pragma unroll
-    for (int q = 0; q < PER; ++q) {
-      const int t = ch * C::kChunk + q * SW + (warp - SW);
-      const size_t row = size_t(row0 + min(t, len - 1));
-#pragma unroll
-      for (int m = 0; m < M; ++m) {
-        const int i = min(m * 32 + lane, dim - 1);               // always in bounds; masked below
-        fr[q][m] = rp[row * p.ld + i];
-        fk[q][m] = kp[row * p.ld + i];
-        fd[q][m] = dp[row * p.ld_dl + i];
-      }
-#pragma unroll
-      for (int m = 0; m < VM; ++m) fv[q][m] = vp[row * p.ld + min(m * 32 + lane, dim - 1 - col0)];
-    }
+  const float* src = p.rec + (size_t(h) * p.rows + row0) * C::kRec;
+  auto issue = [&](int ch) {
+    const int n = min(C::kChunk, len - ch * C::kChunk), st = ch % kWkStages;
+    const uint32_t bytes = uint32_t(n) * C::kRec * 4;
+    mbar_arrive_expect_tx(full + st, bytes);
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                     smem_u32(smem + st * C::kChunk * C::kRec)),
+                 "l"(src + size_t(ch) * C::kChunk * C::kRec), "r"(bytes), "r"(smem_u32(full + st))
+                 : "memory");
   };
-  auto convert = [&](int ch) {
-    float* buf = smem + (ch & 1) * C::kChunk * C::kTok;
-#pragma unroll
-    for (int q = 0; q < PER; ++q) {
-      const int tok = q * SW + (warp - SW);
-      const bool there = ch * C::kChunk + tok < len;             // tokens past the end leave the state as it is
-      float* b = buf + tok * C::kTok;
-      float ruk = 0.f;
-#pragma unroll
-      for (int m = 0; m < M; ++m) {
-        const int i = m * 32 + lane;
-        if (C::kDim < 32 && i >= C::kDim) continue;
-        // row group g's values four at a time: 16-byte pieces of consecutive groups are neighbours
-        const int at = (i % ROWS) / 4 * (LANES * 4) + i / ROWS * 4 + i % 4;
-        const bool in = there && i < dim;
-        const float r = in ? to_f32(fr[q][m]) : 0.f, k = in ? to_f32(fk[q][m]) : 0.f;
-        b[at] = r;
-        b[C::kDim + at] = k;
-        b[2 * C::kDim + at] = in ? __expf(-__expf(fd[q][m] + w0[m])) : 1.f;
-        ruk = fmaf(r * uu[m], k, ruk);
-      }
-#pragma unroll
-      for (int m = 0; m < VM; ++m) {
-        const int c = m * 32 + lane;
-        if (c < C::kCols) b[3 * C::kDim + c] = there && col0 + c < dim ? to_f32(fv[q][m]) : 0.f;
-      }
-      ruk = warp_sum(ruk);
-      if (lane == 0) b[3 * C::kDim + C::kCols] = ruk;
-    }
-  };
+  if (threadIdx.x == 0)
+    for (int ch = 0; ch < kWkStages && ch < chunks; ++ch) issue(ch);
 
-  // compute threads: rows g * ROWS .. of columns c0 .. c0 + 3 (of the block)
-  const int g = threadIdx.x % LANES, c0 = (threadIdx.x & (kWkHalf - 1)) / LANES * kWkCols;
+  // rows g * ROWS .. of columns c0 .. c0 + 3 (of the block)
+  const int g = threadIdx.x % LANES, c0 = threadIdx.x / LANES * kWkCols;
   uint64_t s2[ROWS / 2][kWkCols];
   float* sp = p.state + size_t(slot) * p.stride + size_t(h) * dim * dim;
-  if (!stager) {
 #pragma unroll
-    for (int i = 0; i < ROWS / 2; ++i)
+  for (int i = 0; i < ROWS / 2; ++i)
 #pragma unroll
-      for (int c = 0; c < kWkCols; ++c) {
-        const int r0 = g * ROWS + 2 * i, col = col0 + c0 + c;
-        s2[i][c] = wk_pair((r0 < dim && col < dim) ? sp[size_t(r0) * dim + col] : 0.f,
-                           (r0 + 1 < dim && col < dim) ? sp[size_t(r0 + 1) * dim + col] : 0.f);
-      }
-  } else {
-    fetch(0);
-#pragma unroll
-    for (int m = 0; m < M; ++m) {
-      const bool in = m * 32 + lane < dim;
-      w0[m] = in ? p.w0[h * dim + m * 32 + lane] : 0.f;
-      uu[m] = in ? p.u[h * dim + m * 32 + lane] : 0.f;
+    for (int c = 0; c < kWkCols; ++c) {
+      const int r0 = g * ROWS + 2 * i, col = col0 + c0 + c;
+      s2[i][c] = wk_pair((r0 < dim && col < dim) ? sp[size_t(r0) * dim + col] : 0.f,
+                         (r0 + 1 < dim && col < dim) ? sp[size_t(r0 + 1) * dim + col] : 0.f);
     }
-    convert(0);
-    if (chunks > 1) fetch(1);
-  }
-  __syncthreads();
   // after the butterfly, the lanes of a column group hold column `mine` of the four
   const int mine = (g & (LANES / 2) ? 2 : 0) + (g & (LANES / 4) ? 1 : 0);
   const bool writer = g % (LANES / 4) == 0 && col0 + c0 + mine < dim;
+  const int at_v = 3 * C::kDim + col0 + c0, at_ruk = 3 * C::kDim + C::kV;
   float* op = p.out + size_t(row0) * p.ld_out + h * dim + col0 + c0 + mine;
-  for (int ch = 0; ch < chunks; ++ch) {
-    if (stager) {
-      if (ch + 1 < chunks) {
-        convert(ch + 1);
-        if (ch + 2 < chunks) fetch(ch + 2);
-      }
-    } else {
-      const float* buf = smem + (ch & 1) * C::kChunk * C::kTok;
-      const int n = min(C::kChunk, len - ch * C::kChunk);
-      constexpr int TU = 4;                                      // tokens whose sums are in flight together
-      for (int t0 = 0; t0 < n; t0 += TU) {
-        float o[TU][kWkCols];
+
+  // one token: the state's part of o, then the state's update
+  auto token = [&](const float* b, float (&o)[kWkCols]) {
+    const float4 v = *reinterpret_cast<const float4*>(b + at_v);
+    const uint64_t v2[kWkCols] = {wk_pair(v.x, v.x), wk_pair(v.y, v.y), wk_pair(v.z, v.z), wk_pair(v.w, v.w)};
+    uint64_t acc[kWkCols] = {0, 0, 0, 0};
 #pragma unroll
-        for (int q = 0; q < TU; ++q) {
-          const float* b = buf + (t0 + q) * C::kTok;
-          const float4 v = *reinterpret_cast<const float4*>(b + 3 * C::kDim + c0);
-          const uint64_t v2[kWkCols] = {wk_pair(v.x, v.x), wk_pair(v.y, v.y), wk_pair(v.z, v.z), wk_pair(v.w, v.w)};
-          uint64_t acc[kWkCols] = {0, 0, 0, 0};
-#pragma unroll
-          for (int i = 0; i < ROWS / 4; ++i) {
-            const int at = i * (LANES * 4) + g * 4;
-            const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(b + at);
-            const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(b + C::kDim + at);
-            const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(b + 2 * C::kDim + at);
-#pragma unroll
-            for (int c = 0; c < kWkCols; ++c) {
-              acc[c] = wk_fma(r.x, s2[2 * i][c], acc[c]);
-              acc[c] = wk_fma(r.y, s2[2 * i + 1][c], acc[c]);
-              s2[2 * i][c] = wk_fma(w.x, s2[2 * i][c], wk_mul(k.x, v2[c]));
-              s2[2 * i + 1][c] = wk_fma(w.y, s2[2 * i + 1][c], wk_mul(k.y, v2[c]));
-            }
-          }
-#pragma unroll
-          for (int c = 0; c < kWkCols; ++c) {
-            float lo, hi;
-            wk_unpair(acc[c], lo, hi);
-            o[q][c] = lo + hi;
-          }
-        }
-        float sum[TU];
-#pragma unroll
-        for (int q = 0; q < TU; ++q) {
-          const bool up = g & (LANES / 2), up2 = g & (LANES / 4);
-          const float k0 = up ? o[q][2] : o[q][0], k1 = up ? o[q][3] : o[q][1];
-          const float x0 = up ? o[q][0] : o[q][2], x1 = up ? o[q][1] : o[q][3];
-          const float y0 = k0 + __shfl_xor_sync(0xffffffffu, x0, LANES / 2);
-          const float y1 = k1 + __shfl_xor_sync(0xffffffffu, x1, LANES / 2);
-          sum[q] = (up2 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, up2 ? y0 : y1, LANES / 4);
-        }
-#pragma unroll
-        for (int off = LANES / 8; off > 0; off >>= 1)
-#pragma unroll
-          for (int q = 0; q < TU; ++q) sum[q] += __shfl_xor_sync(0xffffffffu, sum[q], off);
-        if (writer) {
-#pragma unroll
-          for (int q = 0; q < TU; ++q) {
-            const float* b = buf + (t0 + q) * C::kTok + 3 * C::kDim;
-            if (t0 + q < n) op[size_t(ch * C::kChunk + t0 + q) * p.ld_out] = fmaf(b[C::kCols], b[c0 + mine], sum[q]);
-          }
-        }
-      }
-    }
-    __syncthreads();
-  }
-  if (!stager) {
-#pragma unroll
-    for (int i = 0; i < ROWS / 2; ++i)
+    for (int i = 0; i < ROWS / 4; ++i) {
+      const int at = i * (LANES * 4) + g * 4;
+      const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(b + at);
+      const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(b + C::kDim + at);
+      const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(b + 2 * C::kDim + at);
 #pragma unroll
       for (int c = 0; c < kWkCols; ++c) {
-        const int r0 = g * ROWS + 2 * i, col = col0 + c0 + c;
-        float lo, hi;
-        wk_unpair(s2[i][c], lo, hi);
-        if (col < dim) {
-          if (r0 < dim) sp[size_t(r0) * dim + col] = lo;
-          if (r0 + 1 < dim) sp[size_t(r0 + 1) * dim + col] = hi;
+        acc[c] = wk_fma(r.x, s2[2 * i][c], acc[c]);
+        acc[c] = wk_fma(r.y, s2[2 * i + 1][c], acc[c]);
+        s2[2 * i][c] = wk_fma(w.x, s2[2 * i][c], wk_mul(k.x, v2[c]));
+        s2[2 * i + 1][c] = wk_fma(w.y, s2[2 * i + 1][c], wk_mul(k.y, v2[c]));
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < kWkCols; ++c) {
+      float lo, hi;
+      wk_unpair(acc[c], lo, hi);
+      o[c] = lo + hi;
+    }
+  };
+  const bool up = g & (LANES / 2), up2 = g & (LANES / 4);
+  auto fold = [&](const float (&o)[kWkCols]) {
+    const float k0 = up ? o[2] : o[0], k1 = up ? o[3] : o[1], x0 = up ? o[0] : o[2], x1 = up ? o[1] : o[3];
+    const float y0 = k0 + __shfl_xor_sync(0xffffffffu, x0, LANES / 2);
+    const float y1 = k1 + __shfl_xor_sync(0xffffffffu, x1, LANES / 2);
+    float sum = (up2 ? y1 : y0) + __shfl_xor_sync(0xffffffffu, up2 ? y0 : y1, LANES / 4);
+#pragma unroll
+    for (int off = LANES / 8; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+    return sum;
+  };
+
+  bool ok = true;
+  for (int ch = 0; ch < chunks; ++ch) {
+    const int st = ch % kWkStages;
+    ok = mbar_wait(full + st, uint32_t(ch / kWkStages) & 1u, &gave_up) && ok;
+    const float* buf = smem + st * C::kChunk * C::kRec;
+    const int n = min(C::kChunk, len - ch * C::kChunk);
+    float* oc = op + size_t(ch) * C::kChunk * p.ld_out;
+    // groups of TU tokens; a group's sums are taken beside the next group's arithmetic
+    constexpr int TU = 4;
+    auto put = [&](int t, const float (&o)[TU][kWkCols]) {
+      float sum[TU];
+#pragma unroll
+      for (int q = 0; q < TU; ++q) sum[q] = fold(o[q]);
+      if (writer) {
+#pragma unroll
+        for (int q = 0; q < TU; ++q) {
+          const float* b = buf + (t + q) * C::kRec;
+          oc[size_t(t + q) * p.ld_out] = fmaf(b[at_ruk], b[at_v + mine], sum[q]);
         }
       }
-  } else if (blockIdx.x == 0 && h == 0) {
+    };
+    int t = 0;
+    if (n >= TU) {
+      float o[TU][kWkCols];
+#pragma unroll
+      for (int q = 0; q < TU; ++q) token(buf + q * C::kRec, o[q]);
+      for (t = TU; t + TU <= n; t += TU) {
+        float next[TU][kWkCols];
+#pragma unroll
+        for (int q = 0; q < TU; ++q) token(buf + (t + q) * C::kRec, next[q]);
+        put(t - TU, o);
+#pragma unroll
+        for (int q = 0; q < TU; ++q)
+#pragma unroll
+          for (int c = 0; c < kWkCols; ++c) o[q][c] = next[q][c];
+      }
+      put(t - TU, o);
+    }
+    for (; t < n; ++t) {
+      const float* b = buf + t * C::kRec;
+      float o[kWkCols];
+      token(b, o);
+      const float sum = fold(o);
+      if (writer) oc[size_t(t) * p.ld_out] = fmaf(b[at_ruk], b[at_v + mine], sum);
+    }
+    __syncthreads();                                 // the stage has been read
+    if (threadIdx.x == 0 && ch + kWkStages < chunks) issue(ch + kWkStages);
+  }
+  if (!ok) {                                         // let the copies in flight land, as far as that goes
+    for (int i = 0; threadIdx.x == 0 && i < kWkStages; ++i)
+      for (uint32_t k = 0; k < (1u << 16); ++k)
+        if (mbar_try_wait(full + i, uint32_t((chunks - 1 - (chunks - 1 - i) % kWkStages) / kWkStages) & 1u)) break;
+    if (p.status) atomicExch(p.status, int(kStatusMbarTimeout));
+  }
+#pragma unroll
+  for (int i = 0; i < ROWS / 2; ++i)
+#pragma unroll
+    for (int c = 0; c < kWkCols; ++c) {
+      const int r0 = g * ROWS + 2 * i, col = col0 + c0 + c;
+      float lo, hi;
+      wk_unpair(s2[i][c], lo, hi);
+      if (col < dim) {
+        if (r0 < dim) sp[size_t(r0) * dim + col] = lo;
+        if (r0 + 1 < dim) sp[size_t(r0 + 1) * dim + col] = hi;
+      }
+    }
+  if (blockIdx.x == 0 && h == 0) {
     const float* last = p.x + size_t(row0 + len - 1) * p.ldx;
     float* keep = p.prev + size_t(slot) * p.stride;
-    for (int i = threadIdx.x - kWkHalf; i < p.ldx; i += kWkHalf) keep[i] = last[i];
+    for (int i = threadIdx.x; i < p.ldx; i += kWkThreads) keep[i] = last[i];
   }
 }
 
@@ -321,20 +356,32 @@ wkv_finish_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ g
   }
 }
 
+struct WkvIn {
+  const void* r; const void* k; const void* v; int ld;
+  const float* dl; int ld_dl; const float* w0; const float* u; float* rec;
+};
+
 template <class T, int ROWS, int LANES>
-static int launch_wkv(const WkvParams& p, int n_segs, int pdl, cudaStream_t st) {
+static int launch_wkv(const WkvIn& in, WkvParams p, int n_segs, int pdl, cudaStream_t st) {
   using C = WkCfg<ROWS, LANES>;
-  auto kern = wkv_scan_kernel<T, ROWS, LANES>;
+  constexpr int LU = C::kDim >= 128 ? 32 : C::kDim / 4;
+  const long long threads = 1LL * p.rows * p.H * LU;
+  if (threads > 0x7fffffffLL) return -2;
+  const int rc = launch(wkv_prepare_kernel<T, ROWS, LANES, LU>, dim3(unsigned((threads + kRowThreads - 1) / kRowThreads)),
+                        dim3(kRowThreads), 0, st, pdl != 0, static_cast<const T*>(in.r), static_cast<const T*>(in.k),
+                        static_cast<const T*>(in.v), in.ld, in.dl, in.ld_dl, in.w0, in.u, in.rec, p.rows, p.H, p.dim);
+  if (rc) return rc;
+  auto kern = wkv_scan_kernel<ROWS, LANES>;
   RB_CHECK(set_max_smem(kern, C::kSmem));
-  return launch(kern, dim3((p.dim + C::kCols - 1) / C::kCols, p.H, n_segs), dim3(2 * kWkHalf), C::kSmem, st, pdl != 0, p);
+  return launch(kern, dim3((p.dim + C::kCols - 1) / C::kCols, p.H, n_segs), dim3(kWkThreads), C::kSmem, st, pdl != 0, p);
 }
 template <class T>
-static int dispatch_wkv(const WkvParams& p, int n, int pdl, cudaStream_t st) {
-  if (p.dim <= 16) return launch_wkv<T, 4, 4>(p, n, pdl, st);
-  if (p.dim <= 32) return launch_wkv<T, 4, 8>(p, n, pdl, st);
-  if (p.dim <= 64) return launch_wkv<T, 4, 16>(p, n, pdl, st);
-  if (p.dim <= 128) return launch_wkv<T, 4, 32>(p, n, pdl, st);
-  if (p.dim <= 256) return launch_wkv<T, 8, 32>(p, n, pdl, st);
+static int dispatch_wkv(const WkvIn& in, const WkvParams& p, int n, int pdl, cudaStream_t st) {
+  if (p.dim <= 16) return launch_wkv<T, 4, 4>(in, p, n, pdl, st);
+  if (p.dim <= 32) return launch_wkv<T, 4, 8>(in, p, n, pdl, st);
+  if (p.dim <= 64) return launch_wkv<T, 4, 16>(in, p, n, pdl, st);
+  if (p.dim <= 128) return launch_wkv<T, 4, 32>(in, p, n, pdl, st);
+  if (p.dim <= 256) return launch_wkv<T, 8, 32>(in, p, n, pdl, st);
   return -2;
 }
 
@@ -344,6 +391,14 @@ using namespace rb;
 
 // Largest head size of the recurrence.
 extern "C" int rmlx_wkv_max_dim() { return 256; }
+// Floats of the scratch record of one (token, head).
+extern "C" int rmlx_wkv_record(int dim) {
+  if (dim <= 16) return WkCfg<4, 4>::kRec;
+  if (dim <= 32) return WkCfg<4, 8>::kRec;
+  if (dim <= 64) return WkCfg<4, 16>::kRec;
+  if (dim <= 128) return WkCfg<4, 32>::kRec;
+  return WkCfg<8, 32>::kRec;
+}
 
 // x fp32 [T, ldx], mu fp32 [5, ldx], out [5, T, ldx] fp32 (f32) or bf16; ldx a multiple of eight, prev
 // rows 16-byte aligned. slots int32 [T].
@@ -357,21 +412,25 @@ extern "C" int rmlx_token_shift(const float* x, int ldx, const float* mu, const 
                 prev_stride, slots, each_row, static_cast<__nv_bfloat16*>(out), T);
 }
 
-// r, k, v [rows, ld] fp32 (f32) or bf16; dl fp32 [rows, ld_dl]; segs int32 [n_segs, 4] (16-byte aligned) or
-// null with slots [n_segs]: then every row is a segment. No slot occurs twice except one that nobody reads.
+// r, k, v [rows, ld] fp32 (f32) or bf16; dl fp32 [rows, ld_dl]; rec: scratch, fp32 [H, rows, record], 16-byte
+// aligned; segs int32 [n_segs, 4] (16-byte aligned) or null with slots [n_segs]: then every row is a segment.
+// No slot occurs twice except one that nobody reads. status: set when a wait for a chunk gave up.
 extern "C" int rmlx_wkv_scan(const void* r, const void* k, const void* v, int ld, const float* dl, int ld_dl,
-                             const float* w0, const float* u, const int* segs, const int* slots, int n_segs,
-                             float* state, float* prev, long long stride, const float* x, int ldx, float* out,
-                             int ld_out, int H, int dim, int f32, int pdl, cudaStream_t st) {
-  if (n_segs < 1 || n_segs > 65535 || H < 1 || H > 65535 || dim < 1 || ld < H * dim || ld_dl < H * dim ||
-      ld_out < H * dim || (!segs && !slots) || (reinterpret_cast<uintptr_t>(segs) & 15))
+                             const float* w0, const float* u, float* rec, int rows, const int* segs, const int* slots,
+                             int n_segs, float* state, float* prev, long long stride, const float* x, int ldx, float* out,
+                             int ld_out, int H, int dim, int f32, int* status, int pdl, cudaStream_t st) {
+  if (rows < 1 || n_segs < 1 || n_segs > 65535 || H < 1 || H > 65535 || dim < 1 || ld < H * dim || ld_dl < H * dim ||
+      ld_out < H * dim || (!segs && !slots) || ((reinterpret_cast<uintptr_t>(segs) | reinterpret_cast<uintptr_t>(rec)) & 15) ||
+      ((reinterpret_cast<uintptr_t>(r) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) |
+        reinterpret_cast<uintptr_t>(dl)) & 15))
     return -2;
+  const WkvIn in{r, k, v, ld, dl, ld_dl, w0, u, rec};
   WkvParams p;
-  p.r = r; p.k = k; p.v = v; p.ld = ld; p.dl = dl; p.ld_dl = ld_dl; p.w0 = w0; p.u = u;
+  p.rec = rec; p.rows = rows;
   p.segs = reinterpret_cast<const int4*>(segs); p.slots = slots;
   p.state = state; p.prev = prev; p.stride = stride; p.x = x; p.ldx = ldx; p.out = out; p.ld_out = ld_out;
-  p.H = H; p.dim = dim;
-  return f32 ? dispatch_wkv<float>(p, n_segs, pdl, st) : dispatch_wkv<__nv_bfloat16>(p, n_segs, pdl, st);
+  p.H = H; p.dim = dim; p.status = status;
+  return f32 ? dispatch_wkv<float>(in, p, n_segs, pdl, st) : dispatch_wkv<__nv_bfloat16>(in, p, n_segs, pdl, st);
 }
 
 extern "C" int rmlx_wkv_finish(const float* o, int ld_o, const void* gate, int ld_g, const float* norm, float eps,

@@ -136,11 +136,8 @@ class DecodeEngineBase:
             _lib.check(rc, "decode_advance")
         self._launches_per_step = _lib.launch_count() - n0
 
-    def capture(self, nb: Optional[int] = None):
-        """The captured step of bucket ``nb`` (default: the bucket of the bound rows), captured on
-        first use: one eager warm-up run (sets kernel attributes), then the capture; the state
-        the runs advance is put back after each."""
-        nb = self.bucket() if nb is None else nb
+    def _snapshot(self):
+        """Remembers what a step advances; the function returned puts it back."""
         state = (self.tokens, self.positions, self.seq_lens)
         saved = [t.clone() for t in state]
         if self.state_slots is not None:      # a run also advances the bound sequences' recurrent state
@@ -153,8 +150,17 @@ class DecodeEngineBase:
             if self.state_slots is not None:
                 self.cache.state.index_copy_(0, slots, saved_rows)
 
-        return self.graphs.get_or_capture(("decode", nb), lambda: self._run_step(nb), warmup=1,
-                                          restore=restore, device=self.model.device)
+        return restore
+
+    def capture(self, nb: Optional[int] = None):
+        """The captured step of bucket ``nb`` (default: the bucket of the bound rows), captured on
+        first use: one eager warm-up run (sets kernel attributes), then the capture; the state
+        the runs advance is put back after each."""
+        nb = self.bucket() if nb is None else nb
+        key = ("decode", nb)
+        return self.graphs.get_or_capture(key, lambda: self._run_step(nb), warmup=1,
+                                          restore=None if key in self.graphs else self._snapshot(),
+                                          device=self.model.device)
 
     def step(self) -> torch.Tensor:
         """Run one decode step for every bound row. Returns the device tensor of sampled tokens

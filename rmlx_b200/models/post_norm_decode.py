@@ -38,6 +38,7 @@ class PostNormDecode(DecodeEngineBase):
         self.bufs = Buffers(max_batch, model.device)
         self.matvec_rows = matvec_rows
         self.max_len = cache.max_blocks_per_seq * cache.block_size
+        self._planned = set()
         self.ticket = torch.zeros(1, dtype=torch.int32, device=model.device)
         self.fused = model.dtype == torch.bfloat16 and all(self._fits(lw) for lw in model.w.layers) and \
             P.gemv_max_rows(model.width_p) > 0
@@ -52,6 +53,17 @@ class PostNormDecode(DecodeEngineBase):
         if isinstance(f, DenseFfWeights):
             return N.max_rows(f.w_down.k) > 0
         return f is None or R.expert_decode_fits(f.w_down.k, f.spec.top)
+
+    def capture(self, nb: Optional[int] = None):
+        """Buffers and scratch of a bucket come with its first run: one plain run first, so that the recorded
+        step allocates nothing (which the native graph store asks for)."""
+        nb = self.bucket() if nb is None else nb
+        if nb not in self._planned:
+            self._planned.add(nb)
+            restore = self._snapshot()
+            self._run_step(nb)
+            restore()
+        return super().capture(nb)
 
     def _context(self, nb: int) -> StepContext:
         return StepContext(nb, self.bufs, self.cache, self.block_table[:nb], self.positions[:nb], None,

@@ -578,7 +578,8 @@ class RodapelModel:
         low_t = N.tanh_rows(low, c.bufs.get("low_t", t, mw.rank_p, dtype=dt), pdl=pdl)
         decay = P.logits_f32(low_t, mw.w2, c.bufs.get("decay", t, inner, dtype=torch.float32))
         o = c.bufs.get("wkv_o", t, inner, dtype=torch.float32)
-        W.wkv_scan(rkvg[0], rkvg[1], rkvg[2], decay, mw.w0, mw.u, state, prev, x, o, runs=c.runs,
+        rec = c.bufs.get("wkv_rec", t, m.heads, W.record(m.dim), dtype=torch.float32)
+        W.wkv_scan(rkvg[0], rkvg[1], rkvg[2], decay, mw.w0, mw.u, state, prev, x, o, rec, runs=c.runs,
                    slots=None if c.runs is not None else c.slots, pdl=pdl)
         a = c.bufs.get("wkv_a", t, inner, dtype=dt)
         W.wkv_finish(o, rkvg[3], mw.norm, self.cfg.norm_eps, m.heads, m.dim, a, pdl=pdl)

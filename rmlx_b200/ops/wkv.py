@@ -7,6 +7,7 @@ from typing import Optional
 import torch
 
 from .. import _lib
+from .gemm import GemmStatus
 from .parallel_block import _f32
 
 SHIFT_PARTS = ("r", "k", "v", "g", "w")
@@ -14,7 +15,8 @@ SHIFT_PARTS = ("r", "k", "v", "g", "w")
 _lib.register_cuda_sigs({
     "rmlx_wkv_max_dim": ("", "i"),
     "rmlx_token_shift": ("pippqpipiiip", "i"),
-    "rmlx_wkv_scan": ("pppipippppi" "ppqpipi" "iiiip", "i"),
+    "rmlx_wkv_record": ("i", "i"),
+    "rmlx_wkv_scan": ("pppipippp" "ippi" "ppqpipi" "iiipip", "i"),
     "rmlx_wkv_decode": ("piipipppfp" "ppqpipiiiiip", "i"),
     "rmlx_wkv_finish": ("pipipfpiiiiiip", "i"),
 })
@@ -37,23 +39,30 @@ def token_shift(x: torch.Tensor, mu: torch.Tensor, prev: torch.Tensor, slots: to
     _lib.check(rc, "token_shift")
 
 
+def record(dim: int) -> int:
+    """Scratch floats of ``wkv_scan`` per row and head."""
+    return int(_lib.cuda().rmlx_wkv_record(dim))
+
+
 def wkv_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, w0: torch.Tensor, u: torch.Tensor,
-             state: torch.Tensor, prev: torch.Tensor, x: torch.Tensor, out: torch.Tensor,
+             state: torch.Tensor, prev: torch.Tensor, x: torch.Tensor, out: torch.Tensor, rec: torch.Tensor,
              runs: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None, pdl: bool = False) -> None:
     """Runs every sequence's new tokens through the recurrence on top of ``state`` [slots, H, d, d] and
     leaves the new state (and in ``prev`` the last row of ``x``) behind. r, k, v [T, >= H d] in the compute type,
-    ``decay`` fp32 logits (w = exp(-exp(decay + w0))), out fp32. ``runs`` int32 [n, 4] (first row, rows, slot, -),
-    or ``slots``: every row its own sequence."""
+    ``decay`` fp32 logits (w = exp(-exp(decay + w0))), out fp32, ``rec`` scratch of T * H * ``record(d)`` floats.
+    ``runs`` int32 [n, 4] (first row, rows, slot, -), or ``slots``: every row its own sequence."""
     _lib.require_cuda_tensor(r, k, v, decay, w0, u, state, prev, x, out, runs, slots)
     _, h, d, _ = state.shape
     assert r.stride(0) == k.stride(0) == v.stride(0) and r.dtype == k.dtype == v.dtype
     assert decay.dtype == out.dtype == x.dtype == state.dtype == torch.float32 and state.stride()[1:] == (d * d, d, 1)
     assert w0.numel() == u.numel() == h * d and state.stride(0) == prev.stride(0)
-    n = runs.shape[0] if runs is not None else slots.numel()
+    n, t = runs.shape[0] if runs is not None else slots.numel(), r.shape[0]
+    assert rec.dtype == torch.float32 and rec.is_contiguous() and rec.numel() >= t * h * record(d)
     rc = _lib.cuda().rmlx_wkv_scan(
         r.data_ptr(), k.data_ptr(), v.data_ptr(), r.stride(0), decay.data_ptr(), decay.stride(0), w0.data_ptr(),
-        u.data_ptr(), _lib.ptr(runs), _lib.ptr(slots), n, state.data_ptr(), prev.data_ptr(), state.stride(0),
-        x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), h, d, _f32(r), int(pdl), _lib.stream_ptr())
+        u.data_ptr(), rec.data_ptr(), t, _lib.ptr(runs), _lib.ptr(slots), n, state.data_ptr(), prev.data_ptr(),
+        state.stride(0), x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), h, d, _f32(r),
+        GemmStatus.get(r.device).data_ptr(), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "wkv_scan")
 
 

@@ -61,6 +61,9 @@ class GraphCache:
     def __len__(self) -> int:
         return len(self._g)
 
+    def __contains__(self, key: Hashable) -> bool:
+        return key in self._g
+
     def get_or_capture(self, key: Hashable, fn: Callable[[], None], warmup: int = 1,
                        restore: Optional[Callable[[], None]] = None, device=None):
         """Returns a replayable object for ``fn`` (a CUDA graph; on CPU, ``fn`` itself).

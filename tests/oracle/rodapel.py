@@ -58,7 +58,7 @@ def window_attention(w, m, eps, h):
     v = heads_first(h @ w["v"].T, m["kv_heads"])
     group = m["heads"] // m["kv_heads"]
     k, v = k.repeat_interleave(group, 0), v.repeat_interleave(group, 0)
-    o = softmax_attention(q @ k.transpose(1, 2) * m["scale"], visible(len(h), m["mask"]["size"]), v)
+    o = softmax_attention(q @ k.transpose(1, 2) * m["scale"], visible(len(h), (m.get("mask") or {}).get("size")), v)
     gate = torch.sigmoid(h @ w["g"].T)                       # [T, heads]
     return heads_last(o * gate.T[:, :, None]) @ w["o"].T
 

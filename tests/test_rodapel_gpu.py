@@ -215,10 +215,20 @@ class LatentCase:
         t = {k: v.float() for k, v in M.random_tensors(cfg, seed).items()}
         self.w = {k[7:]: v.to(dtype) for k, v in t.items() if k.startswith("l0.mix.")}
         self.w["dkv.norm"] = t["l0.mix.dkv.norm"]
-        self.mw = M.build_weights(cfg, {**t, **{"l0.mix." + k: v for k, v in self.w.items()}}, dev, dtype).layers[0].mix
         self.h = [r(n, self.width).to(dtype) for n in lens]
-        for s, t, j, gain in plant:                       # token t asks for what token j holds
-            self.h[s][t] = (self.h[s][j].float() * gain).to(dtype)
+        if plant:
+            # keys come from the first half of h, queries from the second and with the keys' own projections:
+            # token t asks for exactly what token j holds, without holding it itself
+            half, d, n = self.width // 2, spec.dim, spec.dim + spec.rot_dim
+            self.w["dkv"][:, half:] = 0
+            down = self.w["dkv"][:, :half].float()
+            q = torch.zeros(spec.heads, n, self.width)
+            q[:, :d, half:] = self.w["uk"].float().view(spec.heads, d, -1) @ down[:spec.kv_rank]
+            q[:, d:, half:] = down[spec.kv_rank:]
+            self.w["q"] = q.reshape(-1, self.width).to(dtype)
+            for s, t_, j, gain in plant:
+                self.h[s][t_, half:] = (self.h[s][j, :half].float() * gain).to(dtype)
+        self.mw = M.build_weights(cfg, {**t, **{"l0.mix." + k: v for k, v in self.w.items()}}, dev, dtype).layers[0].mix
 
     def want(self, spec=None):
         """Attention output before the output projection, per sequence [T, heads * vdim]."""
@@ -294,7 +304,7 @@ def test_a_far_latent_key_stands_out(dev, spec):
     it by a wrong angle, shows."""
     from dataclasses import replace
     spec = replace(spec, scale=spec.scale * 4)
-    plant = [(0, 290, 0, 1.0), (0, 291, 15, 1.0), (0, 292, 16, 1.0), (0, 299, 143, 1.0)]
+    plant = [(0, 290, 0, 4.0), (0, 291, 15, 4.0), (0, 292, 16, 4.0), (0, 299, 143, 4.0)]
     c = LatentCase(dev, [300], spec, BF, seed=3, plant=plant)
     want = c.want()[0]
     rows = [290, 291, 292, 299]
@@ -302,7 +312,7 @@ def test_a_far_latent_key_stands_out(dev, spec):
     for _, _, j, _ in plant:
         lost.h[0][j] = 0
     turned = replace(spec, rot_base=spec.rot_base * 1.5)
-    assert rel(lost.want()[0][rows], want[rows]) > 0.1 and rel(c.want(turned)[0], want) > 5e-2
+    assert rel(lost.want()[0][rows], want[rows]) > 0.15 and rel(c.want(turned)[0], want) > 0.1
     forms = ["any", "expanded1"] + (["2"] if (spec.kv_rank, spec.rot_dim) in L.DECODE_WIDTHS else [])
     for how in forms:
         got = c.run(how).reshape(300, -1)
@@ -352,7 +362,7 @@ def test_recurrence_in_portions(dev, heads, dim, dtype, tol):
         x = r(first, ldx).to(dev)
         o = torch.zeros(first, ld, device=dev)
         W.wkv_scan(wide(cat(rr)), wide(cat(k)), wide(cat(v)), wide(cat(dl)), w0.to(dev), u.reshape(-1).to(dev), state, prev,
-                   x, o, runs=i32(runs, dev))
+                   x, o, torch.empty(first * heads * W.record(dim), device=dev), runs=i32(runs, dev))
         for (f, c, slot, _), i in zip(runs, live):
             got[i].append(o[f:f + c, :n].cpu())
             assert torch.equal(prev[slot], x[f + c - 1])
@@ -378,10 +388,10 @@ def test_state_decays_exactly_over_a_long_past(dev):
     lost = O.heads_last(O.wkv_recurrence(hf(rr), hf(k), hf(v), hf(decay * (torch.arange(t)[:, None] != 300) +
                                                                   (torch.arange(t)[:, None] == 300)), u.view(n, d).double()))
     assert rel(lost[-1], want[-1]) > 1e-3
-    pool = torch.zeros(1, n * d * d + 8, device=dev)
+    pool = torch.zeros(2, n * d * d + 8, device=dev)
     o = torch.zeros(t, n * d, device=dev)
     W.wkv_scan(rr.to(dev), k.to(dev), v.to(dev), dl.to(dev), w0.to(dev), u.to(dev), pool[:, :n * d * d].unflatten(1, (n, d, d)),
-               pool[:, n * d * d:], torch.zeros(t, 8, device=dev), o, runs=i32([[0, t, 0, 0]], dev))
+               pool[:, n * d * d:], torch.zeros(t, 8, device=dev), o, torch.empty(t * n * W.record(d), device=dev), runs=i32([[0, t, 0, 0]], dev))
     assert rel(o[-1], want[-1]) < 2e-5
 
 
@@ -595,7 +605,9 @@ def wide_cfg():
 
 
 CFGS = {"tiny": M.rodapel_tiny, "odd": odd_cfg, "wide": wide_cfg}
-TOL = {F32: 3e-5, BF: 6e-2}
+# bf16: the restatement with every product's inputs rounded to bf16 is off by 0.03 (tiny) and 0.10 (odd) at worst,
+# where a norm divides by a small root mean square; half of the rows stay within 0.02
+TOL = {F32: 3e-5, BF: 0.25}
 
 
 class Bench:
@@ -603,8 +615,9 @@ class Bench:
 
     def __init__(self, dev, name, dtype):
         self.cfg = CFGS[name]()
-        # router logits well apart, so that rounding does not change who is chosen
-        self.tensors = {k: (v.float() * 3 if k.endswith(".router") else v.float()).to(BF)
+        # bf16: the correction decides who is chosen, so that rounding cannot flip a close choice (the 32-bit runs
+        # and the routing tests above leave it to the scores)
+        self.tensors = {k: (v.float() * 50).to(BF) if dtype == BF and k.endswith(".correction") else v
                         for k, v in M.random_tensors(self.cfg, 11).items()}
         self.model = M.RodapelModel(M.build_weights(self.cfg, self.tensors, dev, dtype))
         self.dtype, self._ref, self._w = dtype, {}, {k: v.double() for k, v in self.tensors.items()}
@@ -622,13 +635,10 @@ class Bench:
         return ServingEngine(self.model, blocks, SchedulerConfig(max_batch_size=batch, **kw))
 
     def close(self, got, want):
-        """32-bit: every row. bf16: nearly every row (a close choice of experts may flip), and all on average."""
-        if self.dtype == F32:
-            return worst_row(got, want) < TOL[F32]
-        d = got.double().cpu() - want.double().cpu()
-        d = d - d.mean(-1, keepdim=True)
-        err = d.pow(2).mean(-1).sqrt() / want.double().pow(2).mean().sqrt()
-        return float((err > TOL[BF]).double().mean()) <= 0.06 and float(err.median()) < TOL[BF] / 2
+        want = want.double().cpu()
+        d = got.double().cpu() - want
+        err = (d - d.mean(-1, keepdim=True)).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
+        return float(err.max()) < TOL[self.dtype] and (self.dtype == F32 or len(err) < 8 or float(err.median()) < 0.06)
 
 
 @pytest.fixture(scope="module", params=[(n, d) for n in CFGS for d in (F32, BF)], ids=lambda p: f"{p[0]}-{str(p[1])[6:]}")
@@ -689,8 +699,7 @@ def test_unequal_requests_together_and_slots_again(bench):
             if live[i][1] == lens[i]:
                 eng.close_sequence(live.pop(i)[0])
     for i, toks in enumerate(reqs):
-        assert bench.close(torch.cat(got[i]), bench.ref(toks)) or len(toks) < 20, i
-    assert bench.close(torch.cat([torch.cat(got[i]) for i in range(10)]), torch.cat([bench.ref(t) for t in reqs]))
+        assert bench.close(torch.cat(got[i]), bench.ref(toks)), i
 
 
 def test_result_does_not_depend_on_company_or_pages(bench):
@@ -742,8 +751,7 @@ def test_decode_engine_buckets(bench, rows):
                 eng.set_next_tokens([p[-1] for p in prompts])
         for j in (0, 1):
             want = torch.stack([bench.ref(p)[j - 2] for p in prompts])
-            assert bench.close(got[j], want) or (bench.dtype == BF and rows < 16 and
-                                                 rel(got[j], want) < 0.3), (use_graph, j)
+            assert bench.close(got[j], want), (use_graph, j)
         assert eng.launches_per_step > 0
 
 
