@@ -259,7 +259,7 @@ def prefill_kernels(tab: Table, model: RodapelModel, t: int):
     tab.add(ph, "latent: q|latent projection", [lambda w=w: N.linear(h, w.w_in.w, raw) for _, w, _ in lat], gemm(n_in, d),
             "the same GEMM", [lambda w=w: gemm_bf16(h, w.w_in.w, out=raw) for _, w, _ in lat])
     tab.add(ph, "latent: norm + rotation + append", [lambda i=i, w=w: N.latent_append(
-        raw, w.c_norm, 1e-6, w.inv_freq, q, None, cache.k[i], c.block_table, c.positions, c.token_seq, m.heads, m.dim, m.rot_dim,
+        raw, raw[:, w.down_at:], w.c_norm, 1e-6, w.inv_freq, q, None, cache.k[i], c.block_table, c.positions, c.token_seq, m.heads, m.dim, m.rot_dim,
         m.kv_rank, w.dim_p, w.rot_p, w.lat_p) for i, w, _ in lat], (t * n_in * 4, 0), "rope + append",
         [lambda: D.rope_kv_write(qkv, q_like, cache.k[win[0][0]], cache.v[win[0][0]], c.block_table, c.positions, cos, cos,
                                  m.heads, win[0][1].spec.kv_heads, token_seq=c.token_seq) for _ in lat],
@@ -328,7 +328,7 @@ def decode_kernels(tab: Table, model: RodapelModel, b: int, ctx: int):
             [lambda w=w: D.rms_gemv(h, w.w_in, nw, 1e-6, out=out16, pdl=True) for _, w, _ in win])
     attn = torch.randn(b, m.heads, m.vdim, dtype=bf, device=dev)
     q16 = torch.randn(b, m.heads, m.dim, dtype=bf, device=dev)
-    scr = model.scratch(m.heads, m.kv_heads, m.vdim, b, model.window_splits(m, b, c.max_len))
+    scr = model.scratch(m.heads, m.kv_heads, m.vdim, b, model.attention_splits(m, b, c.max_len, m.window))
     from rmlx_b200 import _lib
     gt = _lib.cuda().rmlx_flash_decode_gtiles(m.heads, m.kv_heads)
     sp = D.default_splits(b, m.kv_heads, gt, WINDOW)
@@ -386,7 +386,7 @@ def decode_kernels(tab: Table, model: RodapelModel, b: int, ctx: int):
     q_abs = torch.randn(b, m.heads, w0.lat_p + w0.rot_p, dtype=bf, device=dev)
     o_lat, attn = torch.randn(b, m.heads, w0.lat_p, dtype=bf, device=dev), torch.randn(b, m.heads, w0.vdim_p, dtype=bf, device=dev)
     tab.add(ph, "latent: norm + rotation + append", [lambda i=i, w=w: N.latent_append(
-        raw, w.c_norm, 1e-6, w.inv_freq, q, q_abs, cache.k[i], c.block_table, c.positions, None, m.heads, m.dim, m.rot_dim,
+        raw, raw[:, w.down_at:], w.c_norm, 1e-6, w.inv_freq, q, q_abs, cache.k[i], c.block_table, c.positions, None, m.heads, m.dim, m.rot_dim,
         m.kv_rank, w.dim_p, w.rot_p, w.lat_p, pdl=True) for i, w, _ in lat], (b * w0.w_in.n * 6, 0))
     tab.add(ph, "latent: queries into the latent space", [lambda w=w: N.head_gemv(w.w_uk, q, q_abs, pdl=True) for _, w, _ in lat],
             (w0.w_uk.numel() * 2, 0), "einsum (as the latent-attention model)",

@@ -254,7 +254,8 @@ class WindowAttentionSpec:
 class LatentAttentionSpec:
     """Attention over one latent of ``kv_rank`` values and one rotated key part of ``rot_dim`` values per
     token; heads have ``dim`` unrotated and ``rot_dim`` rotated query / key values, of which the first
-    ``rot_dims`` turn, and ``vdim`` value channels."""
+    ``rot_dims`` turn, and ``vdim`` value channels. ``q_rank``: queries go through a normed latent of that size (0:
+    they do not). ``kv_from``: the layer whose cached latents and key parts this one reads (None: its own)."""
     heads: int
     dim: int
     rot_dim: int
@@ -263,6 +264,8 @@ class LatentAttentionSpec:
     scale: float
     rot_base: float = 10000.0
     rot_dims: Optional[int] = None       # default: all of rot_dim
+    q_rank: int = 0
+    kv_from: Optional[int] = None
 
     kind = "latent_attention"
 
@@ -276,6 +279,7 @@ class LatentAttentionSpec:
                  "rotated dimensions come in pairs, at most rot_dim of them")
         _require(self.kv_rank <= 1024, "kv_rank must be <= 1024")
         _require(self.rot_base > 0, "rot_base must be positive")
+        _require(self.q_rank >= 0, "q_rank must be >= 0 (0: no query latent)")
         return self
 
     @staticmethod
@@ -283,11 +287,17 @@ class LatentAttentionSpec:
         rot = m.get("rot") or {}
         rot_dim = int(m["rot_dim"])
         return LatentAttentionSpec(int(m["heads"]), int(m["dim"]), rot_dim, int(m["vdim"]), int(m["kv_rank"]),
-                                   float(m["scale"]), float(rot.get("base", 10000.0)), int(rot.get("dims", rot_dim)))
+                                   float(m["scale"]), float(rot.get("base", 10000.0)), int(rot.get("dims", rot_dim)),
+                                   int(m.get("q_rank") or 0), None if m.get("kv_from") is None else int(m["kv_from"]))
 
     def to_json(self) -> dict:
-        return {"heads": self.heads, "dim": self.dim, "rot_dim": self.rot_dim, "vdim": self.vdim, "kv_rank": self.kv_rank,
-                "scale": self.scale, "rot": {"base": self.rot_base, "dims": self.rot_dims}}
+        out = {"heads": self.heads, "dim": self.dim, "rot_dim": self.rot_dim, "vdim": self.vdim, "kv_rank": self.kv_rank,
+               "scale": self.scale, "rot": {"base": self.rot_base, "dims": self.rot_dims}}
+        if self.q_rank:
+            out["q_rank"] = self.q_rank
+        if self.kv_from is not None:
+            out["kv_from"] = self.kv_from
+        return out
 
 
 @dataclass
@@ -358,6 +368,8 @@ class PostNormLayerSpec:
 
     def validate(self) -> "PostNormLayerSpec":
         self.mixer.validate()
+        if isinstance(self.mixer, LatentAttentionSpec):
+            _require(not self.mixer.q_rank and self.mixer.kv_from is None, "latent attention: no query latent, no shared rows")
         if self.mlp is not None:
             self.mlp.validate()
         return self
@@ -417,6 +429,264 @@ class RodapelConfig:
     def to_json(self) -> dict:
         return {"architecture": "Rodapel", "vocab": self.vocab_size, "width": self.width,
                 "norm": {"eps": self.norm_eps}, "layers": [l.to_json() for l in self.layers]}
+
+
+@dataclass
+class RotarySpec:
+    """Rotation of the first ``dims`` values of a head; ``scaling``: None or YaRN's (factor, original, fast, slow)."""
+    base: float
+    dims: int
+    scaling: Optional[dict] = None
+
+    def validate(self, dim: int) -> "RotarySpec":
+        _require(self.base > 0 and 0 <= self.dims <= dim and self.dims % 2 == 0,
+                 "rotated dimensions come in pairs, at most the head's")
+        if self.scaling:
+            _require(all(float(self.scaling[k]) > 0 for k in ("factor", "original", "fast", "slow")), "rotation scaling: positive values")
+            _require(self.base != 1.0, "rotation scaling needs a base other than 1")
+        return self
+
+    @staticmethod
+    def from_json(r: dict) -> "RotarySpec":
+        s = r.get("scaling")
+        return RotarySpec(float(r["base"]), int(r["dims"]),
+                          None if not s else {k: float(s[k]) for k in ("factor", "original", "fast", "slow")})
+
+    def to_json(self) -> dict:
+        out = {"base": self.base, "dims": self.dims}
+        if self.scaling:
+            out["scaling"] = dict(self.scaling)
+        return out
+
+
+@dataclass
+class ChunkedAttentionSpec:
+    """Grouped-query attention with biased projections, rotated and unweightedly normed queries and keys, a soft cap
+    (0: none) and, with ``chunk`` > 0, only the keys of the query's own chunk of so many positions."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotarySpec
+    softcap: float = 0.0
+    chunk: int = 0
+
+    def validate(self) -> "ChunkedAttentionSpec":
+        _require(self.heads > 0 and self.kv_heads > 0 and self.heads % self.kv_heads == 0,
+                 "heads must be a positive multiple of kv_heads")
+        _require(self.dim > 0 and self.vdim > 0, "head sizes must be positive")
+        _require(self.softcap >= 0 and self.chunk >= 0, "softcap and chunk must be >= 0 (0: none)")
+        self.rot.validate(self.dim)
+        return self
+
+    @staticmethod
+    def from_json(m: dict) -> "ChunkedAttentionSpec":
+        return ChunkedAttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                                    RotarySpec.from_json(m["rot"]), float(m.get("softcap") or 0.0),
+                                    int((m.get("mask") or {}).get("size") or 0))
+
+    def to_json(self) -> dict:
+        return {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale,
+                "rot": self.rot.to_json(), "softcap": self.softcap or None, "mask": {"size": self.chunk} if self.chunk else None}
+
+
+@dataclass
+class StateSpaceSpec:
+    """State-space heads: ``heads`` states of ``state`` x ``vdim``, ``groups`` shared input / output vectors, a causal
+    convolution over ``conv`` tokens, the gated output normed in ``norm_groups`` equal parts."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_groups: int
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+    def validate(self) -> "StateSpaceSpec":
+        _require(self.heads > 0 and self.vdim > 0 and 0 < self.state <= 256, "state space: heads and vdim positive, state in [1, 256]")
+        _require(self.groups > 0 and self.heads % self.groups == 0, "state space: heads must be a multiple of groups")
+        _require(self.conv > 0, "state space: the convolution has at least one tap")
+        _require(self.norm_groups > 0 and self.inner % self.norm_groups == 0, "state space: norm groups must divide the inner width")
+        return self
+
+    @staticmethod
+    def from_json(m: dict) -> "StateSpaceSpec":
+        return StateSpaceSpec(*(int(m[k]) for k in ("heads", "vdim", "state", "groups", "conv", "norm_groups")))
+
+    def to_json(self) -> dict:
+        return {k: getattr(self, k) for k in ("heads", "vdim", "state", "groups", "conv", "norm_groups")}
+
+
+@dataclass
+class GlaSpec:
+    """Gated linear attention: ``heads`` states of ``dim`` x ``vdim``, decays sigmoid(z)^(1 / tau) from a low-rank
+    projection (its rank comes with the weights; ``decay_rank`` is what random weights use)."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    decay_rank: int = 16
+
+    kind = "gla"
+
+    def validate(self) -> "GlaSpec":
+        _require(self.heads > 0 and self.vdim > 0 and 0 < self.dim <= 256, "gla: heads and vdim positive, dim in [1, 256]")
+        _require(self.tau > 0, "gla: tau must be positive")
+        return self
+
+    @staticmethod
+    def from_json(m: dict) -> "GlaSpec":
+        return GlaSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["tau"]))
+
+    def to_json(self) -> dict:
+        return {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "tau": self.tau}
+
+
+@dataclass
+class PairSpec:
+    """Chunked attention and state-space heads side by side on the same input, their outputs weighted."""
+    left: ChunkedAttentionSpec
+    right: StateSpaceSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+    kind = "parallel"
+
+    def validate(self) -> "PairSpec":
+        self.left.validate()
+        self.right.validate()
+        return self
+
+    @staticmethod
+    def from_json(m: dict) -> "PairSpec":
+        return PairSpec(ChunkedAttentionSpec.from_json(m["left"]), StateSpaceSpec.from_json(m["right"]),
+                        float(m["left_scale"]), float(m["right_scale"]))
+
+    def to_json(self) -> dict:
+        return {"left": self.left.to_json(), "right": self.right.to_json(), "left_scale": self.left_scale,
+                "right_scale": self.right_scale}
+
+
+@dataclass
+class SwigluFfSpec:
+    """Gated feed-forward with silu."""
+    ff: int
+
+    limit = 0.0                      # of the gated activation: none
+
+    def validate(self) -> "SwigluFfSpec":
+        _require(self.ff > 0, "feed-forward: ff must be positive")
+        return self
+
+    def to_json(self) -> dict:
+        return {"kind": "dense", "ff": self.ff}
+
+
+@dataclass
+class ChosenFfSpec:
+    """``experts`` gated feed-forwards of width ``ff``; each token uses the ``top`` with the largest biased logits,
+    weighted by the softmax over those alone."""
+    experts: int
+    top: int
+    ff: int
+
+    limit = 0.0
+    identity = 0
+
+    def validate(self) -> "ChosenFfSpec":
+        _require(0 < self.experts <= 512 and self.ff > 0, "experts: 1 to 512, ff positive")
+        _require(1 <= self.top <= min(32, self.experts), "top must be in [1, 32] and <= experts")
+        return self
+
+    def to_json(self) -> dict:
+        return {"kind": "moe", "expert": {"ff": self.ff}, "router": {"experts": self.experts, "top": self.top}}
+
+
+_TWIN_MIXERS = {c.kind: c for c in (LatentAttentionSpec, GlaSpec, PairSpec)}
+
+
+@dataclass
+class TwinNormLayerSpec:
+    """One layer: a mixer and (unless None) a feed-forward, both reading the same residual through norms of their own."""
+    mixer: "LatentAttentionSpec | GlaSpec | PairSpec"
+    mlp: "SwigluFfSpec | ChosenFfSpec | None" = None
+
+    def validate(self) -> "TwinNormLayerSpec":
+        self.mixer.validate()
+        if isinstance(self.mixer, LatentAttentionSpec):
+            _require(self.mixer.q_rank > 0, "latent attention: queries go through a latent (q_rank)")
+        if self.mlp is not None:
+            self.mlp.validate()
+        return self
+
+    @staticmethod
+    def from_json(e: dict) -> "TwinNormLayerSpec":
+        _require(e.get("type") in _TWIN_MIXERS, f"unknown mixer type {e.get('type')!r}")
+        m, mlp = e.get("mlp"), None
+        if m is not None:
+            _require(m.get("kind") in ("dense", "moe"), f"unknown feed-forward kind {m.get('kind')!r}")
+            mlp = SwigluFfSpec(int(m["ff"])) if m["kind"] == "dense" else \
+                ChosenFfSpec(int(m["router"]["experts"]), int(m["router"]["top"]), int(m["expert"]["ff"]))
+        return TwinNormLayerSpec(_TWIN_MIXERS[e["type"]].from_json(e["mixer"]), mlp)
+
+    def to_json(self) -> dict:
+        return {"type": self.mixer.kind, "mixer": self.mixer.to_json(),
+                "mlp": None if self.mlp is None else self.mlp.to_json()}
+
+
+@dataclass
+class NugosunConfig:
+    """Nugosun: a decoder of latent attention (rows may be shared between layers), gated linear attention and pairs of
+    chunked attention and state-space heads, with the feed-forward beside the mixer; every layer states its own kind
+    and sizes."""
+    vocab_size: int
+    width: int
+    layers: "list[TwinNormLayerSpec]"
+    norm_eps: float = 1e-6
+    embedding_scale: float = 1.0
+    max_seq_len: int = 0             # 0: bounded by the cache only
+    name: str = "nugosun"
+
+    sliding_window = 0               # pages are shared by every layer: none can be dropped early
+
+    def validate(self) -> "NugosunConfig":
+        _require(self.vocab_size > 0 and self.width > 0 and len(self.layers) > 0, "bad sizes")
+        _require(self.norm_eps > 0, "norm_eps must be positive")
+        for i, layer in enumerate(self.layers):
+            layer.validate()
+            j = getattr(layer.mixer, "kv_from", None)
+            if j is not None:
+                _require(0 <= j < i and isinstance(self.layers[j].mixer, LatentAttentionSpec), f"layer {i}: kv_from names no latent layer before it")
+                a, b = layer.mixer, self.layers[j].mixer
+                _require(b.kv_from is None, f"layer {i}: kv_from names a layer without rows of its own")
+                _require((a.kv_rank, a.rot_dim, a.rot_dims, a.rot_base) == (b.kv_rank, b.rot_dim, b.rot_dims, b.rot_base),
+                         f"layer {i}: the shared rows' sizes and rotation differ")
+        return self
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def hidden_size(self) -> int:
+        return self.width
+
+    @staticmethod
+    def from_json(c: dict) -> "NugosunConfig":
+        return NugosunConfig(int(c["vocab"]), int(c["width"]), [TwinNormLayerSpec.from_json(e) for e in c["layers"]],
+                             float(c["norm"]["eps"]), float(c["embedding"]["scale"])).validate()
+
+    def to_json(self) -> dict:
+        return {"architecture": "Nugosun", "vocab": self.vocab_size, "width": self.width, "norm": {"eps": self.norm_eps},
+                "embedding": {"scale": self.embedding_scale}, "layers": [l.to_json() for l in self.layers]}
 
 
 @dataclass

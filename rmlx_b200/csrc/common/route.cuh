@@ -1,4 +1,4 @@
-// Expert choice by corrected softmax scores for one token, by one full warp (see moe_route.cu).
+// Expert choice for one token by one full warp (see moe_route.cu).
 #pragma once
 #include "ptx.cuh"
 
@@ -7,9 +7,14 @@ namespace rb {
 constexpr int kRouteMaxOutputs = 512;
 constexpr int kRouteMaxTop = 32;
 
+enum RouteRule {
+  kRouteCorrected = 0,      // by softmax + correction; weights: the softmax over all outputs
+  kRouteChosen = 1,         // by logit + correction (a bias); weights: the softmax over the chosen ones alone
+};
+
 // N: outputs a lane holds. logits, correction: fp32 [outputs], the first `experts` of them with weights of their own. Ties go to
 // the lower index. counts (may be null) gets one more for every chosen expert.
-template <int N>
+template <int N, RouteRule RULE>
 __device__ __forceinline__ void warp_route_n(const float* logits, const float* correction, int experts, int outputs,
                                              int top_k, int* idx, float* weights, float* identity, int* counts) {
   const int lane = threadIdx.x & 31;
@@ -20,16 +25,20 @@ __device__ __forceinline__ void warp_route_n(const float* logits, const float* c
     s[i] = e < outputs ? logits[e] : -INFINITY;
     m = fmaxf(m, s[i]);
   }
-  m = warp_max(m);
-  float sum = 0.f;
+  if (RULE == kRouteCorrected) {
+    m = warp_max(m);
+    float sum = 0.f;
 #pragma unroll
-  for (int i = 0; i < N; ++i) { s[i] = expf(s[i] - m); sum += s[i]; }
-  sum = warp_sum(sum);
+    for (int i = 0; i < N; ++i) { s[i] = expf(s[i] - m); sum += s[i]; }
+    sum = warp_sum(sum);
+#pragma unroll
+    for (int i = 0; i < N; ++i) s[i] = s[i] / sum;
+  }
 #pragma unroll
   for (int i = 0; i < N; ++i) {
     const int e = i * 32 + lane;
-    s[i] = s[i] / sum;
     c[i] = e < outputs ? s[i] + correction[e] : -INFINITY;
+    if (RULE == kRouteChosen) s[i] = c[i];
   }
   float my_w = 0.f, id_w = 0.f;
   int my_e = 0;
@@ -52,20 +61,25 @@ __device__ __forceinline__ void warp_route_n(const float* logits, const float* c
     if (lane == r) { my_e = be; my_w = w; }
     if (be >= experts) id_w += w;
   }
+  if (RULE == kRouteChosen) {                              // the first choice has the largest logit
+    const float top = __shfl_sync(0xffffffffu, my_w, 0);   // (by the whole warp)
+    my_w = lane < top_k ? expf(my_w - top) : 0.f;
+    my_w = my_w / warp_sum(my_w);
+  }
   if (lane < top_k) {
     idx[lane] = my_e;
     weights[lane] = my_w;
     if (counts && my_e < experts) atomicAdd(counts + my_e, 1);
   }
-  if (lane == 0) *identity = id_w;
+  if (lane == 0 && identity) *identity = id_w;
 }
 
-__device__ __forceinline__ void warp_route_corrected(const float* logits, const float* correction, int experts,
-                                                     int outputs, int top_k, int* idx, float* weights, float* identity,
-                                                     int* counts) {
-  if (outputs <= 64) warp_route_n<2>(logits, correction, experts, outputs, top_k, idx, weights, identity, counts);
-  else if (outputs <= 256) warp_route_n<8>(logits, correction, experts, outputs, top_k, idx, weights, identity, counts);
-  else warp_route_n<kRouteMaxOutputs / 32>(logits, correction, experts, outputs, top_k, idx, weights, identity, counts);
+template <RouteRule RULE>
+__device__ __forceinline__ void warp_route(const float* logits, const float* correction, int experts, int outputs, int top_k,
+                                           int* idx, float* weights, float* identity, int* counts) {
+  if (outputs <= 64) warp_route_n<2, RULE>(logits, correction, experts, outputs, top_k, idx, weights, identity, counts);
+  else if (outputs <= 256) warp_route_n<8, RULE>(logits, correction, experts, outputs, top_k, idx, weights, identity, counts);
+  else warp_route_n<kRouteMaxOutputs / 32, RULE>(logits, correction, experts, outputs, top_k, idx, weights, identity, counts);
 }
 
 }  // namespace rb

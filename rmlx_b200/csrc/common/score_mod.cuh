@@ -24,6 +24,14 @@ struct ScoreMod {
   const float* sink = nullptr;
 };
 
+// The first key a query at position `pos` sees: the last `window` keys (> 0), only its own chunk of `chunk`
+// positions counted from 0 (> 0), or every key before it.
+__device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+  int first = window > 0 ? max(0, pos - window + 1) : 0;
+  if (chunk > 0) first = max(first, pos - pos % chunk);
+  return first;
+}
+
 // Gate logits of token t, head h at gate[t * ld + h], in the activations' type.
 struct HeadGate {
   const void* gate = nullptr;

@@ -22,7 +22,7 @@ struct AaParams {
   const int* positions;     // [T]
   const int* token_seq;     // [T] row of the block table, or null: token t has row t
   void* out;                // [T, Hq, dvp]
-  int Hq, Hkv, dkp, dvp, ldk, ldv, max_blocks, page, window;
+  int Hq, Hkv, dkp, dvp, ldk, ldv, max_blocks, page, window, chunk;
   ScoreMod mod;
   HeadGate gate;
   const int* rows;          // [n] batch rows to run, or null: all
@@ -69,7 +69,7 @@ __global__ void __launch_bounds__(kAaWarps * 32) attention_any_kernel(AaParams p
   const float st = p.mod.scale * (p.mod.temp ? p.mod.temp[h] : 1.f);
   const float cap = p.mod.softcap;
   const float r1 = p.mod.r1 ? p.mod.r1[h] : 0.f, r2 = p.mod.r1 ? p.mod.r2[h] : 0.f;
-  const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int first = first_key(pos, p.window, p.chunk);
 
   float m = -INFINITY, l = 0.f, o[NV];
 #pragma unroll
@@ -154,12 +154,13 @@ RB_BOUNDS_REGISTER("attention_any.cu")
 
 // q [T, Hq, dkp], out [T, Hq, dvp], caches [blocks, Hkv, page, ldk / ldv]: fp32 (f32) or bf16; dkp, dvp, ldk
 // and ldv multiples of eight, dvp <= 1024. Token t sits at positions[t] and sees keys 0 .. positions[t]
-// (the last `window` of them when window > 0) of row token_seq[t] of the block table. rows: the n_rows
+// (the last `window` of them when window > 0, those of its own
+// chunk of `chunk` positions when chunk > 0) of row token_seq[t] of the block table. rows: the n_rows
 // batch rows to run (null: all T). gate [T, ldg] in the same type, or null.
 extern "C" int rmlx_attention_any(const void* q, const void* k_cache, const void* v_cache,
                                   const int* block_table, const int* positions, const int* token_seq,
                                   const int* rows, int n_rows, void* out, int T, int Hq, int Hkv, int dkp, int dvp,
-                                  int ldk, int ldv, int max_blocks, int page, int window, float scale, float softcap,
+                                  int ldk, int ldv, int max_blocks, int page, int window, int chunk, float scale, float softcap,
                                   const float* temp, const float* r1, const float* r2, const float* sink,
                                   const void* gate, int ldg, int f32, int pdl, cudaStream_t st) {
   if (T < 1 || Hkv < 1 || Hq % Hkv || Hq > 65535 || dkp < 8 || dkp % 8 || dvp < 8 || dvp % 8 ||
@@ -169,7 +170,7 @@ extern "C" int rmlx_attention_any(const void* q, const void* k_cache, const void
   p.q = q; p.k_cache = k_cache; p.v_cache = v_cache; p.block_table = block_table;
   p.positions = positions; p.token_seq = token_seq; p.out = out; p.rows = rows;
   p.Hq = Hq; p.Hkv = Hkv; p.dkp = dkp; p.dvp = dvp; p.ldk = ldk; p.ldv = ldv; p.max_blocks = max_blocks; p.page = page;
-  p.window = window;
+  p.window = window; p.chunk = chunk;
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2;
   p.mod.sink = sink;
   p.gate.gate = gate; p.gate.ld = ldg;

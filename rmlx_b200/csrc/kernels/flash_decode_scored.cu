@@ -1,6 +1,6 @@
 // Paged flash-decode attention with score modifiers (score_mod.cuh): one new query token per row,
 // grouped-query heads, different key and value widths, temperature / soft cap / distance bias /
-// sink / sliding window.
+// sink / sliding window / chunked visibility.
 //
 // Same decomposition as flash_decode.cu: a block owns one (row, kv head, 16-query-head tile, KV
 // split); its four warps walk the split's 16-token pages with cp.async rings into swizzled shared
@@ -61,7 +61,7 @@ struct FsParams {
   float* part_o;                 // [B, Hkv*gtiles, S, 16, DV class]
   float* part_ml;                // [B, Hkv*gtiles, S, 16, 2]
   unsigned int* tickets;         // [B * Hkv*gtiles], zero on entry, zero on exit
-  int raw_ld, max_blocks, Hq, Hkv, G, gtiles, S, window, dim, vdim, dkp, dvp;
+  int raw_ld, max_blocks, Hq, Hkv, G, gtiles, S, window, chunk, dim, vdim, dkp, dvp;
   int head_norm;                 // fused form: q_w / k_w are [dim] and every head is normed on its own
   int gate_col;                  // fused form: gate logits at raw[b][gate_col + head] (< 0: none)
   float eps;
@@ -123,7 +123,7 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   pdl_wait();
   const int b = p.rows ? p.rows[lb] : lb;
   const int len = p.positions[b] + 1;
-  const int first = (p.window > 0 && len > p.window) ? len - p.window : 0;   // first visible token
+  const int first = first_key(len - 1, p.window, p.chunk);   // first visible token
   const int pg_begin = first / kFsPage;
   const int pg_end = (len + kFsPage - 1) / kFsPage;
   const int pg_per_split = (pg_end - pg_begin + p.S - 1) / p.S;
@@ -497,7 +497,7 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
                                         const int* block_table, const int* positions, const int* rows,
                                         const int* table_rows, void* out, float* part_o, float* part_ml,
                                         unsigned int* tickets, int B, int Hq, int Hkv, int dim, int vdim,
-                                        int dkp, int dvp, int max_blocks, int splits, int window,
+                                        int dkp, int dvp, int max_blocks, int splits, int window, int chunk,
                                         float scale, float softcap, const float* temp, const float* r1,
                                         const float* r2, const float* sink, const void* gate, int ldg,
                                         int head_norm, int gate_col, int pdl, cudaStream_t st) {
@@ -513,7 +513,7 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
   p.out = static_cast<__nv_bfloat16*>(out);
   p.part_o = part_o; p.part_ml = part_ml; p.tickets = tickets;
   p.max_blocks = max_blocks; p.Hq = Hq; p.Hkv = Hkv; p.G = Hq / Hkv; p.gtiles = (p.G + 15) / 16;
-  p.S = splits; p.window = window; p.dim = dim; p.vdim = vdim; p.dkp = dkp; p.dvp = dvp;
+  p.S = splits; p.window = window; p.chunk = chunk; p.dim = dim; p.vdim = vdim; p.dkp = dkp; p.dvp = dvp;
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2; p.mod.sink = sink;
   p.gate.gate = gate; p.gate.ld = ldg; p.head_norm = head_norm; p.gate_col = gate_col;
   if (raw && gate_col >= 0 && raw_ld < gate_col + Hq) return -2;

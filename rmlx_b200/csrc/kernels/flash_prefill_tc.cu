@@ -90,6 +90,7 @@ struct TcParams {
   const int4* tiles;        // ragged batches: {first row, rows, position of the first row, table row}
   int max_blocks;
   int window;               // > 0: a query sees only its last `window` keys
+  int chunk;                // > 0: only the keys of its own chunk of so many positions
   float scale_log2;
   ScoreMod mod;             // MOD instances
   HeadGate gate;            // ragged batches
@@ -185,9 +186,9 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     bt = p.block_table;
   }
   // steps of lane L: it sees keys [0, kv_end_L); a lane that starts past the last token is idle.
-  // With a sliding window the block's steps start at j0, the step that holds the first key its
-  // first row can see (later rows mask what lies before their own window).
-  const int j0 = p.window > 0 ? max(0, pos_q0 - p.window + 1) / kTcKeys : 0;
+  // With a sliding window or chunks the block's steps start at j0, the step that holds the first key its
+  // first row can see (later rows mask what lies before their own first key).
+  const int j0 = first_key(pos_q0, p.window, p.chunk) / kTcKeys;
   int n_steps[LANES];
   int n_max = 0, kv_end_max = 1;
 #pragma unroll
@@ -382,7 +383,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     uint64_t* p_full = s_full + 4;
     uint64_t* o_done = s_full + 5;
     const int lrow = L * kTcRows + row;                // row inside the block
-    const int pos = pos_q0 + lrow;
+    const int pos = pos_q0 + lrow, first = first_key(pos, p.window, p.chunk);
     const int my_steps = n_steps[LANES == 1 ? 0 : L];
     const float sc = MOD ? 1.f : p.scale_log2;         // MOD: scores are final, in base 2
     char* prow = sP + L * kTcPTile + row * 128;
@@ -486,8 +487,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
           for (int i = 0; i < 32; ++i)
             if (c * 32 + i > vis) r[c][i] = 0xff800000u;   // -inf
       }
-      if (p.window > 0 && pos - p.window + 1 > k0) {   // keys before this row's window
-        const int lo = pos - p.window + 1 - k0;        // keys k0 .. k0+lo-1 are out of the window
+      if (first > k0) {                                // keys before this row's first one
+        const int lo = first - k0;
 #pragma unroll
         for (int c = 0; c < NC; ++c)
 #pragma unroll
@@ -692,7 +693,7 @@ extern "C" int rmlx_flash_prefill_scored_supported(int dk, int dv) {
 extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, const void* v_cache,
                                          const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                                          void* out, int T, int Hq, int Hkv, int dk, int dv, int num_blocks,
-                                         int window, float scale, float softcap, const float* temp,
+                                         int window, int chunk, float scale, float softcap, const float* temp,
                                          const float* r1, const float* r2, const float* sink, const void* gate,
                                          int ldg, int lanes, int* status, int pdl, cudaStream_t st) {
   if (T < 1 || (lanes != 1 && lanes != 2) || Hkv < 1 || Hq % Hkv || num_blocks < 1 || n_tiles < 1 || !tiles || (r1 && !r2) ||
@@ -711,7 +712,7 @@ extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, con
   p.out = static_cast<__nv_bfloat16*>(out);
   p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.pos0 = 0;
   p.dk = dk; p.dv = dv;
-  p.window = window > 0 ? window : 0;
+  p.window = window > 0 ? window : 0; p.chunk = chunk > 0 ? chunk : 0;
   p.scale_log2 = 1.f;
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2; p.mod.sink = sink;
   p.gate.gate = gate; p.gate.ld = ldg;

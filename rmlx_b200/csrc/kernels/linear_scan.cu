@@ -1,0 +1,343 @@
+// Linear recurrences beside attention, on common/scan.cuh (token by token, fp32 state):
+//
+//   gla   gated linear attention: a decay per key channel, alpha = sigmoid(z + bias)^(1 / tau);
+//         S <- diag(alpha) S + k v^T, o = S^T (q scale)
+//   ssd   state-space heads: x, B and C through a causal depthwise convolution and silu, dt = softplus(.),
+//         S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x; `H / G` heads share a group's B and C
+//
+// and what surrounds them: the convolution's carried inputs, and the norm of the outputs over equal groups of
+// columns with a silu gate before or after it. Decays, step sizes and their exponentials are fp32.
+#include "../common/launch.cuh"
+#include "../common/rows.cuh"
+#include "../common/scan.cuh"
+#include <type_traits>
+
+namespace rb {
+
+__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
+template <class T>
+struct GlaIn {
+  const T* q; const T* k; const T* v;
+  int ld;
+  const float* z;
+  int ld_z;
+  const float* bias;
+  float inv_tau, scale;
+  int dim, vdim;
+  __device__ __forceinline__ void rows4(int t, int h, int i, float (&fr)[4], float (&fk)[4], float (&fw)[4], float (&fb)[4]) const {
+    const bool vec = dim % 4 == 0 && ld % 4 == 0;
+    const size_t at = size_t(t) * ld + h * dim;
+    const float* zp = z + size_t(t) * ld_z + h * dim;
+    scan_load4(q + at, i, dim, vec, fb);
+    scan_load4(k + at, i, dim, vec, fk);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const bool in = i + j < dim;
+      const int c = in ? i + j : 0;
+      fw[j] = in ? expf(-softplus_f(-(zp[c] + bias[h * dim + c])) * inv_tau) : 1.f;
+      fb[j] *= scale;
+      fr[j] = fb[j] * fw[j];
+    }
+  }
+  __device__ __forceinline__ void cols4(int t, int h, int i, float (&fv)[4]) const {
+    scan_load4(v + size_t(t) * ld + h * vdim, i, vdim, vdim % 4 == 0 && ld % 4 == 0, fv);
+  }
+};
+
+// What a state-space layer reads: rows [.. | x: H*d | B: G*n | C: G*n at x_at | .. | dt: H at dt_at | ..].
+template <class T>
+struct SsdIn {
+  const T* raw;
+  int ld, x_at, dt_at;
+  const float* conv_w;      // [taps, channels], the last row is the current token's
+  const float* conv_b;      // [channels]
+  int taps;
+  const float* before;      // slot s: before + s * stride, [taps - 1, channels]: inputs carried over, newest last
+  long long stride;
+  const int* slots;         // [rows]
+  int each_row;             // no two rows share a sequence
+  const float* dt_bias; const float* a_log; const float* skip;      // [H]
+  int H, G, n, d;
+  __device__ __forceinline__ int channels() const { return H * d + 2 * G * n; }
+};
+
+// How many of the rows before t belong to its sequence (at most taps - 1).
+template <class T>
+__device__ __forceinline__ int ssd_back(const SsdIn<T>& in, int t) {
+  int back = 0;
+  if (!in.each_row)
+    while (back < in.taps - 1 && t - back - 1 >= 0 && in.slots[t - back - 1] == in.slots[t]) ++back;
+  return back;
+}
+// Convolution and activation of channel c for token t.
+template <class T>
+__device__ __forceinline__ float ssd_conv(const SsdIn<T>& in, int t, int c, int back) {
+  const int ch = in.channels();
+  const float* st = in.before + size_t(in.slots[t]) * in.stride;
+  float a = in.conv_b[c];
+  for (int j = in.taps - 1; j >= 0; --j) {           // j tokens back
+    const float x = j <= back ? to_f32(in.raw[size_t(t - j) * in.ld + in.x_at + c]) : st[size_t(in.taps - 1 - (j - back)) * ch + c];
+    a = fmaf(in.conv_w[size_t(in.taps - 1 - j) * ch + c], x, a);
+  }
+  return silu_f(a);
+}
+
+// One block per token: all channels' convolutions, then the records.
+template <class T, int ROWS, int LANES>
+__global__ void __launch_bounds__(kRowThreads)
+ssd_prepare_kernel(SsdIn<T> in, float* __restrict__ rec, float* __restrict__ col, int rows) {
+  using C = ScanCfg<ROWS, LANES, true>;
+  extern __shared__ __align__(16) float sm[];
+  const int t = blockIdx.x, inner = in.H * in.d, gn = in.G * in.n, ch = inner + 2 * gn;
+  float* s_own = sm + ch;            // [G] C . B
+  float* s_dt = s_own + in.G;        // [H]
+  float* s_a = s_dt + in.H;          // [H]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int back = ssd_back(in, t);
+  for (int c = threadIdx.x; c < ch; c += kRowThreads) sm[c] = ssd_conv(in, t, c, back);
+  for (int h = threadIdx.x; h < in.H; h += kRowThreads) {
+    const float dt = softplus_f(to_f32(in.raw[size_t(t) * in.ld + in.dt_at + h]) + in.dt_bias[h]);
+    s_dt[h] = dt;
+    s_a[h] = expf(-expf(in.a_log[h]) * dt);
+  }
+  __syncthreads();
+  const float* sB = sm + inner;
+  const float* sC = sB + gn;
+  for (int g = threadIdx.x >> 5; g < in.G; g += kRowThreads / 32) {
+    float s = 0.f;
+    for (int i = threadIdx.x & 31; i < in.n; i += 32) s = fmaf(sB[g * in.n + i], sC[g * in.n + i], s);
+    s = warp_sum(s);
+    if ((threadIdx.x & 31) == 0) s_own[g] = s;
+  }
+  for (int u = threadIdx.x; u < in.G * C::kRows; u += kRowThreads) {
+    const int g = u / C::kRows, i = u - g * C::kRows;
+    float* o = rec + (size_t(g) * rows + t) * C::kRec + scan_at<ROWS, LANES>(i);
+    o[0] = i < in.n ? sC[g * in.n + i] : 0.f;
+    o[C::kRows] = i < in.n ? sB[g * in.n + i] : 0.f;
+  }
+  __syncthreads();
+  const int nb = C::blocks(in.d), per = in.H / in.G, width = nb * C::kCols;
+  for (int u = threadIdx.x; u < in.H * width; u += kRowThreads) {
+    const int h = u / width, i = u - h * width;
+    const float x = i < in.d ? sm[h * in.d + i] : 0.f, v = s_dt[h] * x;
+    float* o = col + ((size_t(h) * nb + i / C::kCols) * rows + t) * C::kCol;
+    o[i % C::kCols] = v;
+    o[C::kCols + i % C::kCols] = fmaf(s_own[h / per], v, in.skip[h] * x);
+    if (i % C::kCols < 4) o[2 * C::kCols + i % C::kCols] = s_a[h];
+  }
+}
+
+// The last taps - 1 inputs of every segment's sequence become its carried ones. A thread owns a channel; it
+// writes in ascending order and reads ahead of what it writes.
+template <class T>
+__global__ void __launch_bounds__(kRowThreads)
+conv_carry_kernel(const T* __restrict__ raw, int ld, int x_at, float* __restrict__ carried, long long stride,
+                  const int4* __restrict__ segs, const int* __restrict__ slots, int ch, int keep) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x * kRowThreads + threadIdx.x;
+  if (c >= ch) return;
+  int row0 = blockIdx.y, len = 1, slot;
+  if (segs) {
+    const int4 s = segs[blockIdx.y];
+    row0 = s.x; len = s.y; slot = s.z;
+  } else {
+    slot = slots[blockIdx.y];
+  }
+  float* st = carried + size_t(slot) * stride + c;
+  for (int m = 0; m < keep; ++m) {
+    const int i = len - keep + m;
+    st[size_t(m) * ch] = i >= 0 ? to_f32(raw[size_t(row0 + i) * ld + x_at + c]) : st[size_t(m + len) * ch];
+  }
+}
+
+// out[t, c] over equal groups of columns: gate_first: f = o silu(gate), f / rms(f over the group) * w;
+// else o / rms(o over the group) * w * silu(gate). L lanes (256: a block) per (row, group).
+template <class T, int L>
+__global__ void __launch_bounds__(kRowThreads)
+gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ gate, int ld_g, const float* __restrict__ w,
+                  float eps, T* __restrict__ out, int ld_out, int rows, int groups, int size, int gate_first) {
+  __shared__ float red[kRowThreads / 32];
+  constexpr int kKeep = 2;                             // chunks of eight a lane keeps
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long unit = (blockIdx.x * (long long)(kRowThreads) + threadIdx.x) / L;
+  const int lane = threadIdx.x % L;
+  const bool live = unit < (long long)(rows) * groups;   // the lanes of a warp stay together for the sums
+  const int t = live ? int(unit / groups) : 0, at = live ? int(unit - (long long)(t) * groups) * size : 0;
+  const bool vec = size % 8 == 0 && ld_o % 8 == 0 && ld_g % 8 == 0 && ld_out % 8 == 0;
+  const float* op = o + size_t(t) * ld_o + at;
+  const T* gp = gate + size_t(t) * ld_g + at;
+  float f[kKeep][8], z[kKeep][8], ssq = 0.f;
+  auto load = [&](int i0, float (&a)[8], float (&s)[8]) {
+    load8_upto(op + i0, size - i0, vec, a);
+    load8_upto(gp + i0, size - i0, vec, s);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      s[i] = silu_f(s[i]);
+      if (gate_first) a[i] *= s[i];
+      ssq += a[i] * a[i];
+    }
+  };
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int i0 = (u * L + lane) * 8;
+    if (i0 < size) load(i0, f[u], z[u]);
+  }
+  for (int i0 = (kKeep * L + lane) * 8; i0 < size; i0 += L * 8) {
+    float a[8], s[8];
+    load(i0, a, s);
+  }
+  if (L <= 32) ssq = group_sum<L <= 32 ? L : 32>(ssq);
+  else ssq = row_block_sum(ssq, red);
+  if (!live) return;
+  const float inv = 1.f / sqrtf(ssq / float(size) + eps);
+  T* dst = out + size_t(t) * ld_out + at;
+  auto put = [&](int i0, float (&a)[8], const float (&s)[8]) {
+    float g[8];
+    load8_upto(w + at + i0, size - i0, vec, g);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) a[i] = a[i] * inv * g[i] * (gate_first ? 1.f : s[i]);
+    if (vec) {
+      store8(dst + i0, a);
+    } else {
+      for (int i = 0; i < 8 && i0 + i < size; ++i) dst[i0 + i] = from_f32<T>(a[i]);
+    }
+  };
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    const int i0 = (u * L + lane) * 8;
+    if (i0 < size) put(i0, f[u], z[u]);
+  }
+  for (int i0 = (kKeep * L + lane) * 8; i0 < size; i0 += L * 8) {
+    float a[8], s[8];
+    load(i0, a, s);                                    // (the sum is not used again)
+    put(i0, a, s);
+  }
+}
+
+template <class T>
+static int run_gla(const GlaIn<T>& in, const ScanParams& p, float* rec, int n, int pdl, cudaStream_t st) {
+#define RB_GLA(R_, L_) return launch_row_scan<GlaIn<T>, R_, L_>(in, p, rec, n, pdl, st)
+  RB_SCAN_DISPATCH(p.n, RB_GLA);
+#undef RB_GLA
+  return -2;
+}
+
+template <class T, int ROWS, int LANES>
+static int launch_ssd(const SsdIn<T>& in, ScanParams p, float* rec, int n_segs, int pdl, cudaStream_t st) {
+  using C = ScanCfg<ROWS, LANES, true>;
+  const size_t smem = size_t(in.H * in.d + 2 * in.G * in.n + in.G + 2 * in.H) * sizeof(float);
+  if (smem > 200 * 1024) return -2;
+  auto kern = ssd_prepare_kernel<T, ROWS, LANES>;
+  RB_CHECK(set_max_smem(kern, smem));
+  float* col = rec + size_t(in.G) * p.rows * C::kRec;
+  int rc = launch(kern, dim3(p.rows), dim3(kRowThreads), smem, st, pdl != 0, in, rec, col, p.rows);
+  if (rc) return rc;
+  p.rec = rec; p.col = col; p.per = in.H / in.G;
+  return launch_scan<ROWS, LANES, true>(p, n_segs, pdl, st);
+}
+template <class T>
+static int run_ssd(const SsdIn<T>& in, const ScanParams& p, float* rec, int n, int pdl, cudaStream_t st) {
+#define RB_SSD(R_, L_) return launch_ssd<T, R_, L_>(in, p, rec, n, pdl, st)
+  RB_SCAN_DISPATCH(p.n, RB_SSD);
+#undef RB_SSD
+  return -2;
+}
+
+static bool scan_args_ok(int rows, const int* segs, const int* slots, int n_segs, const float* rec, int H, int n, int d) {
+  return rows >= 1 && n_segs >= 1 && n_segs <= 65535 && H >= 1 && H <= 65535 && n >= 1 && n <= kScanMaxRows && d >= 1 &&
+         (segs || slots) && !((reinterpret_cast<uintptr_t>(segs) | reinterpret_cast<uintptr_t>(rec)) & 15);
+}
+
+}  // namespace rb
+
+using namespace rb;
+
+extern "C" int rmlx_scan_max_rows() { return kScanMaxRows; }
+// Floats of the scratch records of one (token, head); one != 0: heads with a single decay, `per` of which share
+// their row record.
+extern "C" long long rmlx_scan_record(int n, int d, int one, int per) {
+  if (per < 1) return 0;
+#define RB_REC(R_, L_) return one ? ScanCfg<R_, L_, true>::row_floats(d, per) : ScanCfg<R_, L_, false>::row_floats(d, 1)
+  RB_SCAN_DISPATCH(n, RB_REC);
+#undef RB_REC
+  return 0;
+}
+
+// q, k [rows, ld] (H x dim), v (H x vdim) fp32 (f32) or bf16, 16-byte aligned; z fp32 [rows, ld_z], bias fp32
+// [H * dim]; out fp32 [rows, ld_out] (H x vdim); state fp32, slot s at state + s * stride, [H, dim, vdim]; rec:
+// scratch, rows * H records; segs int32 [n_segs, 4] = (first row, rows, slot, -), 16-byte aligned, or null with
+// slots [n_segs]: then every row is a segment. No slot occurs twice except one that nobody reads.
+extern "C" int rmlx_gla_scan(const void* q, const void* k, const void* v, int ld, const float* z, int ld_z, const float* bias,
+                             float inv_tau, float scale, float* rec, int rows, const int* segs, const int* slots, int n_segs,
+                             float* state, long long stride, float* out, int ld_out, int H, int dim, int vdim, int f32,
+                             int* status, int pdl, cudaStream_t st) {
+  if (!scan_args_ok(rows, segs, slots, n_segs, rec, H, dim, vdim) || ld < H * dim || ld < H * vdim || ld_z < H * dim ||
+      ld_out < H * vdim ||
+      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15))
+    return -2;
+  ScanParams p{};
+  p.rows = rows; p.segs = reinterpret_cast<const int4*>(segs); p.slots = slots;
+  p.state = state; p.stride = stride; p.out = out; p.ld_out = ld_out;
+  p.H = H; p.n = dim; p.d = vdim; p.status = status;
+  auto run = [&](auto* type) {
+    using T = std::remove_pointer_t<decltype(type)>;
+    return run_gla<T>(GlaIn<T>{static_cast<const T*>(q), static_cast<const T*>(k), static_cast<const T*>(v), ld, z, ld_z, bias,
+                               inv_tau, scale, dim, vdim}, p, rec, n_segs, pdl, st);
+  };
+  return f32 ? run(static_cast<float*>(nullptr)) : run(static_cast<__nv_bfloat16*>(nullptr));
+}
+
+// raw fp32 (f32) or bf16 [rows, ld] with x | B | C at column x_at and dt at dt_at; conv_w fp32 [taps, channels],
+// conv_b [channels], dt_bias, a_log, skip [H]; carried: slot s at carried + s * stride, fp32 [taps - 1, channels];
+// state [H, n, d]; row_slots int32 [rows]: the slot of every row; segs / slots as above. Updates state and carried.
+extern "C" int rmlx_ssd_scan(const void* raw, int ld, int x_at, int dt_at, const float* conv_w, const float* conv_b, int taps,
+                             float* carried, const float* dt_bias, const float* a_log, const float* skip, float* rec, int rows,
+                             const int* segs, const int* row_slots, int n_segs, float* state, long long stride, float* out,
+                             int ld_out, int H, int G, int n, int d, int f32, int* status, int pdl, cudaStream_t st) {
+  if (!scan_args_ok(rows, segs, row_slots, n_segs, rec, H, n, d) || !row_slots || G < 1 || H % G || taps < 1 || ld_out < H * d ||
+      x_at < 0 || dt_at < 0 || ld < x_at + H * d + 2 * G * n || ld < dt_at + H || (taps > 1 && !carried))
+    return -2;
+  ScanParams p{};
+  p.rows = rows; p.segs = reinterpret_cast<const int4*>(segs); p.slots = row_slots;
+  p.state = state; p.stride = stride; p.out = out; p.ld_out = ld_out;
+  p.H = H; p.n = n; p.d = d; p.status = status;
+  auto run = [&](auto* type) -> int {
+    using T = std::remove_pointer_t<decltype(type)>;
+    const SsdIn<T> in{static_cast<const T*>(raw), ld, x_at, dt_at, conv_w, conv_b, taps, carried, stride, row_slots, !segs,
+                      dt_bias, a_log, skip, H, G, n, d};
+    const int rc = run_ssd<T>(in, p, rec, n_segs, pdl, st);
+    if (rc || taps == 1) return rc;
+    const int ch = H * d + 2 * G * n;
+    return launch(conv_carry_kernel<T>, dim3((ch + kRowThreads - 1) / kRowThreads, n_segs), dim3(kRowThreads), 0, st, pdl != 0,
+                  in.raw, ld, x_at, carried, stride, p.segs, row_slots, ch, taps - 1);
+  };
+  return f32 ? run(static_cast<float*>(nullptr)) : run(static_cast<__nv_bfloat16*>(nullptr));
+}
+
+// o fp32 [rows, ld_o], gate and out [rows, ..] fp32 (f32) or bf16, w fp32 [groups * size].
+extern "C" int rmlx_gated_norm(const float* o, int ld_o, const void* gate, int ld_g, const float* w, float eps, void* out,
+                               int ld_out, int rows, int groups, int size, int gate_first, int f32, int pdl, cudaStream_t st) {
+  if (rows < 1 || groups < 1 || size < 1 || ld_o < groups * size || ld_g < groups * size || ld_out < groups * size) return -2;
+  const int lanes = size <= 128 ? 8 : size <= 1024 ? 32 : 256;
+  const long long blocks = (1LL * rows * groups * lanes + kRowThreads - 1) / kRowThreads;
+  if (blocks > 0x7fffffffLL) return -2;
+  const dim3 grid{unsigned(blocks)};
+#define RB_GN(T_, L_)                                                                                                    \
+  return launch(gated_norm_kernel<T_, L_>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o, static_cast<const T_*>(gate), \
+                ld_g, w, eps, static_cast<T_*>(out), ld_out, rows, groups, size, gate_first)
+#define RB_GNL(T_)                   \
+  {                                  \
+    if (lanes == 8) RB_GN(T_, 8);    \
+    if (lanes == 32) RB_GN(T_, 32);  \
+    RB_GN(T_, 256);                  \
+  }
+  if (f32) RB_GNL(float)
+  RB_GNL(__nv_bfloat16)
+#undef RB_GNL
+#undef RB_GN
+}

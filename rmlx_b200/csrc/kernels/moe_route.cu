@@ -3,23 +3,25 @@
 // experts' own s, not renormalised. Everything in fp32; nothing leaves the device.
 //
 // The routed experts' histogram and offsets serve the grouped expert products; the chosen identity
-// experts appear only as one summed weight per token.
+// experts appear only as one summed weight per token. The other rule (kRouteChosen) has no identity experts: the
+// top k of z + bias, weighted by the softmax over the chosen ones alone.
 #include "../common/launch.cuh"
 #include "../common/route.cuh"
 #include "../common/rows.cuh"
 
 namespace rb {
 
+template <RouteRule RULE>
 __global__ void __launch_bounds__(256)
-route_corrected_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ correction,
+route_kernel(const float* __restrict__ logits, int ldl, const float* __restrict__ correction,
                        int* __restrict__ idx, float* __restrict__ weights, float* __restrict__ identity,
                        int* __restrict__ counts, int T, int experts, int outputs, int top_k) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x * 8 + (threadIdx.x >> 5);
   if (t < T)
-    warp_route_corrected(logits + size_t(t) * ldl, correction, experts, outputs, top_k, idx + size_t(t) * top_k,
-                         weights + size_t(t) * top_k, identity + t, counts);
+    warp_route<RULE>(logits + size_t(t) * ldl, correction, experts, outputs, top_k, idx + size_t(t) * top_k,
+                     weights + size_t(t) * top_k, identity ? identity + t : nullptr, counts);
 }
 
 // offsets[e] = counts before e, offsets[E] = their sum; counts become running cursors. One warp.
@@ -76,19 +78,34 @@ RB_BOUNDS_REGISTER("moe_route.cu")
 extern "C" int rmlx_route_max_outputs() { return kRouteMaxOutputs; }
 extern "C" int rmlx_route_max_top() { return kRouteMaxTop; }
 
+template <RouteRule RULE>
+static int launch_route(const float* logits, int ldl, const float* correction, int* idx, float* weights, float* identity,
+                        int* counts, int* offsets, int T, int experts, int outputs, int top_k, int pdl, cudaStream_t st) {
+  if (T < 1 || experts < 1 || outputs < experts || outputs > kRouteMaxOutputs || top_k < 1 || top_k > kRouteMaxTop ||
+      top_k > outputs || ldl < outputs || (!counts) != (!offsets) || !correction)
+    return -2;
+  if (counts) RB_CHECK(cudaMemsetAsync(counts, 0, sizeof(int) * experts, st));
+  const int rc = launch(route_kernel<RULE>, dim3((T + 7) / 8), dim3(256), 0, st, pdl != 0 && !counts, logits, ldl,
+                        correction, idx, weights, identity, counts, T, experts, outputs, top_k);
+  if (rc || !counts) return rc;
+  return launch(route_offsets_kernel, dim3(1), dim3(32), 0, st, pdl != 0, counts, offsets, experts);
+}
+
 // logits fp32 [T, ldl], correction fp32 [outputs]; idx, weights [T, top_k], identity [T]; counts
 // [experts] (becomes the scatter's cursors) and offsets [experts + 1], both or neither.
 extern "C" int rmlx_route_corrected(const float* logits, int ldl, const float* correction, int* idx, float* weights,
                                     float* identity, int* counts, int* offsets, int T, int experts, int outputs,
                                     int top_k, int pdl, cudaStream_t st) {
-  if (T < 1 || experts < 1 || outputs < experts || outputs > kRouteMaxOutputs || top_k < 1 || top_k > kRouteMaxTop ||
-      top_k > outputs || ldl < outputs || (!counts) != (!offsets))
-    return -2;
-  if (counts) RB_CHECK(cudaMemsetAsync(counts, 0, sizeof(int) * experts, st));
-  const int rc = launch(route_corrected_kernel, dim3((T + 7) / 8), dim3(256), 0, st, pdl != 0 && !counts, logits, ldl,
-                        correction, idx, weights, identity, counts, T, experts, outputs, top_k);
-  if (rc || !counts) return rc;
-  return launch(route_offsets_kernel, dim3(1), dim3(32), 0, st, pdl != 0, counts, offsets, experts);
+  if (!identity) return -2;
+  return launch_route<kRouteCorrected>(logits, ldl, correction, idx, weights, identity, counts, offsets, T, experts, outputs,
+                                       top_k, pdl, st);
+}
+
+// The rule without identity experts: bias fp32 [experts], the rest as above.
+extern "C" int rmlx_route_chosen(const float* logits, int ldl, const float* bias, int* idx, float* weights, int* counts,
+                                 int* offsets, int T, int experts, int top_k, int pdl, cudaStream_t st) {
+  return launch_route<kRouteChosen>(logits, ldl, bias, idx, weights, nullptr, counts, offsets, T, experts, experts, top_k, pdl,
+                                    st);
 }
 
 // x [T, ldx] -> xs [T * top_k, ldx]; ldx a multiple of eight; cursors as rmlx_route_corrected left them.

@@ -239,8 +239,8 @@ postnorm_router_kernel(Matrix<WBf16> W, PostNormIn in, const float* __restrict__
       float* z = reinterpret_cast<float*>(smem) + b * outputs;
       for (int i = lane; i < outputs; i += 32) z[i] = __ldcg(logits + size_t(b) * outputs + i);
       __syncwarp();
-      warp_route_corrected(z, correction, experts, outputs, top_k, idx + size_t(b) * top_k, weights + size_t(b) * top_k,
-                           identity + b, nullptr);
+      warp_route<kRouteCorrected>(z, correction, experts, outputs, top_k, idx + size_t(b) * top_k,
+                                  weights + size_t(b) * top_k, identity + b, nullptr);
     }
     if (threadIdx.x == 0) *ticket = 0u;
   }

@@ -7,6 +7,7 @@
 // fp32 in both. Residual rows are padded to a multiple of eight; the padding stays zero.
 #include "../common/gated.cuh"
 #include "../common/launch.cuh"
+#include "../common/row_sources.cuh"
 #include "../common/rows.cuh"
 
 namespace rb {
@@ -34,65 +35,6 @@ embed_norm_kernel(const T* __restrict__ table, const int* __restrict__ ids, cons
     h[at + i] = from_f32<T>(v);
   }
 }
-
-// Sublayer outputs the norm below takes: eight consecutive values of row t from column c * 8 on.
-template <class TY>
-struct RowSource {
-  const TY* y;
-  int ldy;
-  __device__ __forceinline__ void prepare(int) {}
-  __device__ __forceinline__ void load(int t, int c, const float (&)[8], float (&f)[8]) const {
-    load8(y + size_t(t) * ldy + c * 8, f);
-  }
-};
-// Routed experts: sum over the token's slots of weight * expert output row (identity experts, and
-// slots without a row, have row -1), plus the summed identity weight times the input itself.
-template <class TY>
-struct ExpertSource {
-  const TY* y;
-  int ldy;
-  const int* row_of_pair;     // [T, top_k]
-  const float* weights;       // [T, top_k]
-  const float* identity;      // [T] summed weight of the identity experts
-  int top_k;
-  float id_w;
-  int rows[4];                // the first four slots
-  float wts[4];
-  __device__ __forceinline__ void prepare(int t) {
-    id_w = identity[t];
-#pragma unroll
-    for (int u = 0; u < 4; ++u) {
-      rows[u] = u < top_k ? row_of_pair[t * top_k + u] : -1;
-      wts[u] = u < top_k ? weights[t * top_k + u] : 0.f;
-    }
-  }
-  __device__ __forceinline__ void load(int t, int c, const float (&x)[8], float (&f)[8]) const {
-#pragma unroll
-    for (int i = 0; i < 8; ++i) f[i] = id_w * x[i];
-    float g[4][8];
-#pragma unroll
-    for (int u = 0; u < 4; ++u) {                      // four slots' rows in flight
-      if (rows[u] >= 0) {
-        load8(y + size_t(rows[u]) * ldy + c * 8, g[u]);
-      } else {
-#pragma unroll
-        for (int i = 0; i < 8; ++i) g[u][i] = 0.f;
-      }
-    }
-#pragma unroll
-    for (int u = 0; u < 4; ++u)
-#pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = fmaf(wts[u], g[u][i], f[i]);
-    for (int s = 4; s < top_k; ++s) {
-      const int row = row_of_pair[t * top_k + s];
-      if (row < 0) continue;
-      const float a = weights[t * top_k + s];
-      load8(y + size_t(row) * ldy + c * 8, g[0]);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = fmaf(a, g[0][i], f[i]);
-    }
-  }
-};
 
 // x[t] += y[t] / rms(y[t]) * w, h[t] = x[t] in the compute type (h may be null).
 template <class SRC, class T>
@@ -213,14 +155,16 @@ head_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __re
   }
 }
 
-// raw row t = [q: H * (dim + rot) | latent: rank | shared key part: rot]. Queries go to q_out
+// q row t = [H * (dim + rot)], down row t = [latent: rank | shared key part: rot] (null: the token's cache row is
+// another layer's, only the queries are done). Queries go to q_out
 // [T, H, dimp + rotp] with their last `rot` values rotated (pairs (2i, 2i+1) of the first `dims` by
 // position * inv_freq[i]), the rotated part also behind the latent part of q_abs [T, H, latp + rotp]
 // when that is given. The latent is divided by its root mean square, times c_w; it and the rotated
 // shared key part form the token's cache row [latp | rotp | ..] of `ldc` elements. One block per token, or (grid y) several.
 template <class TR, class T>
 __global__ void __launch_bounds__(kRowThreads)
-latent_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restrict__ c_w, float eps,
+latent_append_kernel(const TR* __restrict__ qraw, int ldq, const TR* __restrict__ draw, int ldd,
+                     const float* __restrict__ c_w, float eps,
                      const float* __restrict__ inv_freq, int dims, T* __restrict__ q_out, T* __restrict__ q_abs,
                      T* __restrict__ cache, int ldc, const int* __restrict__ block_table,
                      const int* __restrict__ positions, const int* __restrict__ token_seq, int H, int dim,
@@ -230,10 +174,10 @@ latent_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restr
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, pos = positions[t];
-  const TR* row = raw + size_t(t) * ldraw;
-  const TR* down = row + H * (dim + rot);
+  const TR* row = qraw + size_t(t) * ldq;
+  const TR* down = draw ? draw + size_t(t) * ldd : nullptr;
   float ssq = 0.f;
-  for (int i = threadIdx.x; i < rank; i += kRowThreads) { const float v = to_f32(down[i]); ssq += v * v; }
+  for (int i = threadIdx.x; down && i < rank; i += kRowThreads) { const float v = to_f32(down[i]); ssq += v * v; }
   for (int i = threadIdx.x; i < dims / 2; i += kRowThreads) {
     float s, c;
     sincosf(float(pos) * inv_freq[i], &s, &c);
@@ -242,7 +186,7 @@ latent_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restr
   }
   ssq = row_block_sum(ssq, red);           // the angles are in shared memory, too
   const float inv = 1.f / sqrtf(ssq / float(rank) + eps);
-  const bool vec = dim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && ldraw % 8 == 0;
+  const bool vec = dim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && ldq % 8 == 0 && ldd % 8 == 0;
   // values i0 .. i0 + 7 of a vector whose first `dims` values turn
   auto rotate = [&](int i0, float (&f)[8]) {
 #pragma unroll
@@ -258,7 +202,7 @@ latent_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restr
   const int blk = in_table ? block_table[size_t(seq) * max_blocks + pos / page] : 0;
   T* cdst = cache + (size_t(blk) * page + pos % page) * ldc;
   const int ud = dimp >> 3, uq = (dimp + rotp) >> 3, ul = latp >> 3, uc = (latp + rotp) >> 3;
-  for (int u = blockIdx.y * kRowThreads + threadIdx.x; u < H * uq + uc; u += gridDim.y * kRowThreads) {
+  for (int u = blockIdx.y * kRowThreads + threadIdx.x; u < H * uq + (down ? uc : 0); u += gridDim.y * kRowThreads) {
     float f[8];
     if (u < H * uq) {                      // a query
       const int h = u / uq, c = u - h * uq;
@@ -416,14 +360,15 @@ extern "C" int rmlx_head_norm_append(const void* raw, int ldraw, int raw_f32, co
 #undef RB_HN_L
 }
 
-// Types as above. dims: how many of the rotated part's values turn (even, <= rot); inv_freq fp32 [dims / 2].
-extern "C" int rmlx_latent_append(const void* raw, int ldraw, int raw_f32, const float* c_w, float eps,
+// Types as above; q_raw rows ldq apart; down rows ldd apart, or null. dims: how many of the rotated part's values turn (even, <= rot); inv_freq fp32 [dims / 2].
+extern "C" int rmlx_latent_append(const void* q_raw, int ldq, const void* down, int ldd, int raw_f32, const float* c_w, float eps,
                                   const float* inv_freq, int dims, void* q_out, void* q_abs, void* cache, int ldc,
                                   const int* block_table, const int* positions, const int* token_seq, int T, int H,
                                   int dim, int rot, int rank, int dimp, int rotp, int latp, int max_blocks, int page,
                                   int f32, int pdl, cudaStream_t st) {
   if (T < 1 || H < 1 || dim < 0 || rot < 0 || rank < 1 || dims < 0 || dims % 2 || dims > rot || dimp < dim ||
-      rotp < rot || latp < rank || ldc < latp + rotp || ldraw < H * (dim + rot) + rank + rot || (f32 && !raw_f32))
+      rotp < rot || latp < rank || ldc < latp + rotp || ldq < H * (dim + rot) ||
+      (down && ldd < rank + rot) || (f32 && !raw_f32))
     return -2;
   const size_t smem = size_t(dims) * sizeof(float);
   if (smem > 32 * 1024) return -2;
@@ -431,7 +376,7 @@ extern "C" int rmlx_latent_append(const void* raw, int ldraw, int raw_f32, const
   const int split = T >= 64 ? 1 : (work + kRowThreads - 1) / kRowThreads;
 #define RB_LA(TR_, T_)                                                                                            \
   return launch(latent_append_kernel<TR_, T_>, dim3(T, split), dim3(kRowThreads), smem, st, pdl != 0,                    \
-                static_cast<const TR_*>(raw), ldraw, c_w, eps, inv_freq, dims, static_cast<T_*>(q_out),           \
+                static_cast<const TR_*>(q_raw), ldq, static_cast<const TR_*>(down), ldd, c_w, eps, inv_freq, dims, static_cast<T_*>(q_out),           \
                 static_cast<T_*>(q_abs), static_cast<T_*>(cache), ldc, block_table, positions, token_seq, H, dim, \
                 rot, rank, dimp, rotp, latp, max_blocks, page)
   if (f32) RB_LA(float, float);

@@ -101,8 +101,25 @@ def _rodapel_model(weights):
     return RodapelModel(weights)
 
 
+def _nugosun_weights(model_dir, config, device, dtype, layout):
+    from ..config import NugosunConfig
+    from ..loader.safetensors_loader import load_tensors
+    from .nugosun import build_weights
+    if layout is not None and layout.world != 1:
+        raise ValueError("Nugosun runs on one GPU")
+    cfg = NugosunConfig.from_json(config)
+    return build_weights(cfg, load_tensors(model_dir), device, dtype), cfg
+
+
+def _nugosun_model(weights):
+    from .nugosun import NugosunModel
+    return NugosunModel(weights)
+
+
 register(ModelFamily("transformer", lambda c: "num_attention_heads" in c, _transformer_weights, _transformer_model))
 register(ModelFamily("posudra", lambda c: c.get("architecture") == "Posudra", _posudra_weights, _posudra_model,
                      kernels="parallel_block"))
 register(ModelFamily("rodapel", lambda c: c.get("architecture") == "Rodapel", _rodapel_weights, _rodapel_model,
                      kernels="post_norm"))
+register(ModelFamily("nugosun", lambda c: c.get("architecture") == "Nugosun", _nugosun_weights, _nugosun_model,
+                     kernels="twin_norm"))

@@ -27,14 +27,14 @@ _lib.register_cuda_sigs({
     "rmlx_sgemm": ("pipipiiiiip", "i"),
     "rmlx_sgemm_split_xielu": ("pipipiipiffiiiip", "i"),
     "rmlx_sgemm_scaled_add": ("pipippiiiiip", "i"),
-    "rmlx_attention_any": ("pppppppipiiiiiiiiii" "ffpppp" "piiip", "i"),
+    "rmlx_attention_any": ("pppppppipiiiiiiiiiii" "ffpppp" "piiip", "i"),
     "rmlx_flash_prefill_scored_supported": ("ii", "i"),
-    "rmlx_flash_prefill_scored": ("ppppipipiiiiiiiffpppp" "piipip", "i"),
+    "rmlx_flash_prefill_scored": ("ppppipipiiiiiiiiffpppp" "piipip", "i"),
     "rmlx_flash_decode_scored_supported": ("ii", "i"),
     "rmlx_flash_decode_scored_part_o_elems": ("iiiii", "q"),
     "rmlx_flash_decode_scored_part_ml_elems": ("iiii", "q"),
     "rmlx_flash_decode_scored_ticket_elems": ("iii", "q"),
-    "rmlx_flash_decode_scored": ("ppippfpppppppppp" "iiiiiiiiii" "ffpppp" "piiiip", "i"),
+    "rmlx_flash_decode_scored": ("ppippfpppppppppp" "iiiiiiiiiii" "ffpppp" "piiiip", "i"),
 })
 
 
@@ -221,10 +221,11 @@ def decode_scored_supported(dk: int, dv: int) -> bool:
 
 def flash_prefill_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                          tiles: torch.Tensor, mods: ScoreMods, out: torch.Tensor, window: int = 0, lanes: int = 1,
-                         gate: Optional[torch.Tensor] = None, pdl: bool = False) -> torch.Tensor:
+                         gate: Optional[torch.Tensor] = None, chunk: int = 0, pdl: bool = False) -> torch.Tensor:
     """Ragged causal attention over pages on the tensor cores: q [T, H, dk] bf16; ``tiles`` int32
     [n, 4] = (first row, rows <= lanes * 128, position of the first row, row of ``block_table``).
-    ``gate`` [T, H]: logits of a sigmoid each head's output is multiplied by."""
+    ``gate`` [T, H]: logits of a sigmoid each head's output is multiplied by. ``chunk`` > 0: a query sees only the
+    keys of its own chunk of so many positions, counted from the sequence's start."""
     _lib.require_cuda_tensor(q, k_cache, v_cache, block_table, tiles, out)
     t, h, dk = q.shape
     assert q.is_contiguous() and out.is_contiguous() and tiles.dtype == torch.int32 and tiles.is_contiguous()
@@ -232,7 +233,7 @@ def flash_prefill_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
     rc = _lib.cuda().rmlx_flash_prefill_scored(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), block_table.stride(0),
         tiles.data_ptr(), tiles.shape[0], out.data_ptr(), t, h, k_cache.shape[1], dk, v_cache.shape[3],
-        k_cache.shape[0], window, *mods.args(), *_gate_args(gate, t, h, q.dtype), lanes, GemmStatus.get(q.device).data_ptr(), int(pdl),
+        k_cache.shape[0], window, chunk, *mods.args(), *_gate_args(gate, t, h, q.dtype), lanes, GemmStatus.get(q.device).data_ptr(), int(pdl),
         _lib.stream_ptr())
     _lib.check(rc, "flash_prefill_scored")
     return out
@@ -259,7 +260,7 @@ def flash_decode_scored(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tabl
                         k_w: Optional[torch.Tensor] = None, eps: float = 0.0, rows: Optional[torch.Tensor] = None,
                         table_rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None, window: int = 0,
                         gate: Optional[torch.Tensor] = None, head_norm: bool = False, gate_col: int = -1,
-                        pdl: bool = False) -> torch.Tensor:
+                        chunk: int = 0, pdl: bool = False) -> torch.Tensor:
     """One token per row: q [T, H, dk] (keys already appended) or the fused form on the un-normalised
     fp32 projection ``raw`` [T, >= q|k|v], which also appends the key and value (``head_norm``: the
     norms are per head, their weights [dim]; ``gate_col``: where the output gate's logits start in a
@@ -275,7 +276,7 @@ def flash_decode_scored(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tabl
         k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), positions.data_ptr(), _lib.ptr(rows),
         _lib.ptr(table_rows), out.data_ptr(), scratch.part_o.data_ptr(), scratch.part_ml.data_ptr(),
         scratch.tickets.data_ptr(), n, heads, k_cache.shape[1], dim, vdim, k_cache.shape[3], v_cache.shape[3],
-        block_table.stride(0), scratch.splits, window, *mods.args(),
+        block_table.stride(0), scratch.splits, window, chunk, *mods.args(),
         *_gate_args(gate, 0 if q is None else q.shape[0], heads, torch.bfloat16), int(head_norm), gate_col, int(pdl),
         _lib.stream_ptr())
     _lib.check(rc, "flash_decode_scored")
@@ -285,7 +286,7 @@ def flash_decode_scored(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tabl
 def attention_any(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                   positions: torch.Tensor, token_seq: Optional[torch.Tensor], mods: ScoreMods, out: torch.Tensor,
                   window: int = 0, gate: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
-                  pdl: bool = False) -> torch.Tensor:
+                  chunk: int = 0, pdl: bool = False) -> torch.Tensor:
     """Attention of single query tokens over pages for any head widths, bf16 or fp32 storage. Cache rows
     may be wider than the query (key) and the output (value): ``k_cache`` and ``v_cache`` may be one
     pool whose rows hold both (latent attention). ``rows``: batch rows to run (default: all)."""
@@ -297,6 +298,6 @@ def attention_any(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), positions.data_ptr(),
         _lib.ptr(token_seq), _lib.ptr(rows), 0 if rows is None else rows.numel(), out.data_ptr(), t, h,
         k_cache.shape[1], dk, out.shape[2], k_cache.shape[3], v_cache.shape[3], block_table.stride(0),
-        k_cache.shape[2], window, *mods.args(), *_gate_args(gate, t, h, q.dtype), _f32(q), int(pdl), _lib.stream_ptr())
+        k_cache.shape[2], window, chunk, *mods.args(), *_gate_args(gate, t, h, q.dtype), _f32(q), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "attention_any")
     return out

@@ -18,7 +18,7 @@ _lib.register_cuda_sigs({
     "rmlx_embed_norm": ("pppfppiiiiiip", "i"),
     "rmlx_post_norm_add": ("piipfppiiiiip", "i"),
     "rmlx_head_norm_append": ("piippfpppppp" "iiiiiiiiiiip", "i"),
-    "rmlx_latent_append": ("piipfpi" "pppippp" "iiiiiiiiiiiip", "i"),
+    "rmlx_latent_append": ("pipiipfpi" "pppippp" "iiiiiiiiiiiip", "i"),
     "rmlx_gated_act": ("ppiifiip", "i"),
     "rmlx_tanh_rows": ("ppqiip", "i"),
     "rmlx_head_gemv": ("ppiipiipiiiiiip", "i"),
@@ -73,23 +73,24 @@ def head_norm_append(raw: torch.Tensor, q_w: torch.Tensor, k_w: torch.Tensor, ep
     _lib.check(rc, "head_norm_append")
 
 
-def latent_append(raw: torch.Tensor, c_w: torch.Tensor, eps: float, inv_freq: torch.Tensor, q: torch.Tensor,
-                  q_abs: Optional[torch.Tensor], cache: torch.Tensor, block_table: torch.Tensor, positions: torch.Tensor,
-                  token_seq: Optional[torch.Tensor], heads: int, dim: int, rot: int, rank: int, dim_p: int, rot_p: int,
-                  lat_p: int, pdl: bool = False) -> None:
-    """raw [T, q | latent | key part]: rotated queries to ``q`` [T, H, dim_p + rot_p] (their rotated part
-    also behind the latent part of ``q_abs`` [T, H, lat_p + rot_p]), the normed latent and the rotated
-    key part to the token's cache row. ``inv_freq`` fp32 [rotated pairs]."""
-    _lib.require_cuda_tensor(raw, c_w, inv_freq, q, q_abs, cache, block_table, positions, token_seq)
-    t = raw.shape[0]
+def latent_append(q_raw: torch.Tensor, down: Optional[torch.Tensor], c_w: Optional[torch.Tensor], eps: float,
+                  inv_freq: torch.Tensor, q: torch.Tensor, q_abs: Optional[torch.Tensor], cache: torch.Tensor,
+                  block_table: torch.Tensor, positions: torch.Tensor, token_seq: Optional[torch.Tensor], heads: int,
+                  dim: int, rot: int, rank: int, dim_p: int, rot_p: int, lat_p: int, pdl: bool = False) -> None:
+    """Rotated queries of ``q_raw`` [T, H * (dim + rot)] to ``q`` [T, H, dim_p + rot_p] (their rotated part also
+    behind the latent part of ``q_abs`` [T, H, lat_p + rot_p]); of ``down`` [T, latent | key part] the normed
+    latent and the rotated key part to the token's cache row (None: the row is another layer's and in place).
+    ``inv_freq`` fp32 [rotated pairs]."""
+    _lib.require_cuda_tensor(q_raw, down, c_w, inv_freq, q, q_abs, cache, block_table, positions, token_seq)
+    t = q_raw.shape[0]
     assert q.shape == (t, heads, dim_p + rot_p) and q.is_contiguous() and q.dtype == cache.dtype
     assert q_abs is None or (q_abs.shape == (t, heads, lat_p + rot_p) and q_abs.is_contiguous())
-    assert c_w.numel() == rank and cache.shape[1] == 1
+    assert cache.shape[1] == 1 and (down is None or (c_w.numel() == rank and down.dtype == q_raw.dtype))
     rc = _lib.cuda().rmlx_latent_append(
-        raw.data_ptr(), raw.stride(0), _f32(raw), c_w.data_ptr(), eps, inv_freq.data_ptr(), 2 * inv_freq.numel(),
-        q.data_ptr(), _lib.ptr(q_abs), cache.data_ptr(), cache.shape[3], block_table.data_ptr(), positions.data_ptr(),
-        _lib.ptr(token_seq), t, heads, dim, rot, rank, dim_p, rot_p, lat_p, block_table.stride(0), cache.shape[2],
-        _f32(q), int(pdl), _lib.stream_ptr())
+        q_raw.data_ptr(), q_raw.stride(0), _lib.ptr(down), 0 if down is None else down.stride(0), _f32(q_raw), _lib.ptr(c_w),
+        eps, inv_freq.data_ptr(), 2 * inv_freq.numel(), q.data_ptr(), _lib.ptr(q_abs), cache.data_ptr(), cache.shape[3],
+        block_table.data_ptr(), positions.data_ptr(), _lib.ptr(token_seq), t, heads, dim, rot, rank, dim_p, rot_p, lat_p,
+        block_table.stride(0), cache.shape[2], _f32(q), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "latent_append")
 
 

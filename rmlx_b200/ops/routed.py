@@ -1,9 +1,11 @@
-"""Routing by corrected scores with identity experts (csrc/kernels/moe_route.cu) and the grouped expert
+"""Routing by corrected scores with identity experts, or by biased logits with the softmax over the chosen
+experts (csrc/kernels/moe_route.cu), and the grouped expert
 feed-forward around it for any number of tokens: route -> rows sorted by expert -> gate/up with the gated
 activation -> down. The combination with the output norm is ``combine_post_norm`` (postnorm_rows.cu)."""
 from __future__ import annotations
 
 from dataclasses import dataclass
+from typing import Optional
 
 import torch
 
@@ -19,6 +21,7 @@ _lib.register_cuda_sigs({
     "rmlx_route_max_outputs": ("", "i"),
     "rmlx_route_max_top": ("", "i"),
     "rmlx_route_corrected": ("pippppppiiiiip", "i"),
+    "rmlx_route_chosen": ("pippppp" "iiiip", "i"),
     "rmlx_route_scatter": ("pipppp" "iiiiip", "i"),
     "rmlx_moe_combine_post_norm": ("pipppipfppiiiiip", "i"),
     "rmlx_postnorm_router": ("ppppfpii" "pppppp" "iiiiip", "i"),
@@ -33,7 +36,7 @@ class Routing:
     """Device arrays of one routed batch (views of preallocated buffers)."""
     idx: torch.Tensor            # int32 [T, top]; identity experts have idx >= experts
     weights: torch.Tensor        # fp32 [T, top]
-    identity: torch.Tensor       # fp32 [T] summed weight of the identity experts
+    identity: Optional[torch.Tensor]   # fp32 [T] summed weight of the identity experts (None: there are none)
     counts: torch.Tensor         # int32 [experts]
     offsets: torch.Tensor        # int32 [experts + 1]
     row_of_pair: torch.Tensor    # int32 [T, top]; -1: no row
@@ -50,6 +53,18 @@ def route_corrected(logits: torch.Tensor, correction: torch.Tensor, experts: int
         r.identity.data_ptr(), r.counts.data_ptr() if grouped else None, r.offsets.data_ptr() if grouped else None, t,
         experts, outputs, r.idx.shape[1], int(pdl), _lib.stream_ptr())
     _lib.check(rc, "route_corrected")
+
+
+def route_chosen(logits: torch.Tensor, bias: torch.Tensor, r: Routing, grouped: bool = True, pdl: bool = False) -> None:
+    """Chooses by logits + bias, weights by the softmax over the chosen experts' alone (no identity experts)."""
+    _lib.require_cuda_tensor(logits, bias, r.idx)
+    t, experts = logits.shape
+    assert logits.dtype == bias.dtype == torch.float32 and bias.numel() == experts
+    rc = _lib.cuda().rmlx_route_chosen(
+        logits.data_ptr(), logits.stride(0), bias.data_ptr(), r.idx.data_ptr(), r.weights.data_ptr(),
+        r.counts.data_ptr() if grouped else None, r.offsets.data_ptr() if grouped else None, t, experts, r.idx.shape[1],
+        int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "route_chosen")
 
 
 def route_scatter(h: torch.Tensor, r: Routing, xs: torch.Tensor, pdl: bool = False) -> None:

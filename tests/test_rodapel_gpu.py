@@ -251,7 +251,7 @@ class LatentCase:
         q = torch.empty(t, m.heads, mw.dim_p + mw.rot_p, dtype=dt, device=dev)
         q_abs = torch.zeros(t, m.heads, mw.lat_p + mw.rot_p, dtype=dt, device=dev)
         out = torch.full((t, m.heads, mw.vdim_p), 5.0, dtype=dt, device=dev)
-        N.latent_append(raw, mw.c_norm, 1e-5, mw.inv_freq, q, q_abs, pool, table, pos, seq, m.heads, m.dim, m.rot_dim,
+        N.latent_append(raw, raw[:, mw.down_at:], mw.c_norm, 1e-5, mw.inv_freq, q, q_abs, pool, table, pos, seq, m.heads, m.dim, m.rot_dim,
                         m.kv_rank, mw.dim_p, mw.rot_p, mw.lat_p)
         if how.startswith("expanded"):
             first = [sum(self.lens[:i]) for i in range(len(self.lens))]
