@@ -57,7 +57,7 @@ SETS = {
         "host": ("host/serving.cpp", "host/sampler.cpp", "host/safetensors_io.cpp"),
     },
     "twin_norm": {
-        "cuda": ("kernels/twin_norm_rows.cu", "kernels/linear_scan.cu", "kernels/postnorm_rows.cu", "kernels/moe_route.cu",
+        "cuda": ("kernels/twin_norm_rows.cu", "kernels/twin_norm_gemv.cu", "kernels/linear_scan.cu", "kernels/postnorm_rows.cu", "kernels/moe_route.cu",
                  "kernels/head_gemv.cu", "kernels/gemm_tcgen05.cu", "kernels/xgemm_tcgen05.cu",
                  "kernels/gemm_f32.cu", "kernels/flash_prefill_tc.cu", "kernels/flash_decode_scored.cu",
                  "kernels/attention_any.cu", "kernels/mla_decode.cu", "kernels/parallel_rows.cu", "kernels/postnorm_gemv.cu",

@@ -77,6 +77,21 @@ struct XLoadBf16 {          // x (global, bf16), optionally times a per-channel 
     }
   }
 };
+// fp32 activations times a per-channel fp32 weight; tracks the sum of squares.
+struct XLoadF32 {
+  const float* x;
+  const float* scale_w;
+  float ssq;
+  __device__ __forceinline__ void operator()(int c, float (&f)[8]) {
+    const float4 a = __ldcg(reinterpret_cast<const float4*>(x + (c << 3)));
+    const float4 b = __ldcg(reinterpret_cast<const float4*>(x + (c << 3) + 4));
+    const float4 s = *reinterpret_cast<const float4*>(scale_w + (c << 3));
+    const float4 t = *reinterpret_cast<const float4*>(scale_w + (c << 3) + 4);
+    ssq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w + b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
+    f[0] = a.x * s.x; f[1] = a.y * s.y; f[2] = a.z * s.z; f[3] = a.w * s.w;
+    f[4] = b.x * t.x; f[5] = b.y * t.y; f[6] = b.z * t.z; f[7] = b.w * t.w;
+  }
+};
 struct XLoadSwiglu {        // silu(gate) * up from a [gate | up] row of 2*I bf16
   const __nv_bfloat16* gu;
   int I;

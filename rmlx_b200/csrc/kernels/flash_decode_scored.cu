@@ -63,6 +63,12 @@ struct FsParams {
   unsigned int* tickets;         // [B * Hkv*gtiles], zero on entry, zero on exit
   int raw_ld, max_blocks, Hq, Hkv, G, gtiles, S, window, chunk, dim, vdim, dkp, dvp;
   int head_norm;                 // fused form: q_w / k_w are [dim] and every head is normed on its own
+  // fused form with head_norm: bias of the projection (its layout), rotation of values i and i + rot_dims / 2 by position *
+  // inv_freq[i] with cos and sin times `grow`, both before the norm; q_w / k_w may then be null (no weight)
+  const float* bias;
+  const float* inv_freq;
+  int rot_dims;
+  float grow;
   int gate_col;                  // fused form: gate logits at raw[b][gate_col + head] (< 0: none)
   float eps;
   ScoreMod mod;
@@ -159,26 +165,56 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
     if (p.head_norm) {
       // one warp per query head in turn; the owner's last warp also takes the new key's root mean square
       constexpr int PL = DK / 32;
-      const int q_rows = min(16, p.G - gt * 16);
-      float v[4][PL];
+      const int q_rows = min(16, p.G - gt * 16), half = p.rot_dims >> 1;
+      // the rotation of this lane's places: own value times cs, partner's (at `other`) times sn
+      float cs[PL], sn[PL];
+      int other[PL];
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int r = warp * 4 + u;
-        const float* src = row + (kvh * p.G + gt * 16 + r) * p.dim;
-#pragma unroll
-        for (int i = 0; i < PL; ++i) v[u][i] = (r < q_rows && i * 32 + lane < p.dim) ? __ldcg(src + i * 32 + lane) : 0.f;
+      for (int i = 0; i < PL; ++i) {
+        const int d = i * 32 + lane;
+        cs[i] = 1.f; sn[i] = 0.f; other[i] = d;
+        if (d < p.rot_dims) {
+          float sv, cv;
+          sincosf(float(len - 1) * p.inv_freq[d < half ? d : d - half], &sv, &cv);
+          cs[i] = cv * p.grow;
+          sn[i] = (d < half ? -sv : sv) * p.grow;
+          other[i] = d < half ? d + half : d - half;
+        }
       }
+      auto load_head = [&](int at, bool live, float (&v)[PL], float (&u)[PL]) {
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int r = warp * 4 + u;
+        for (int i = 0; i < PL; ++i) {
+          const bool in = live && i * 32 + lane < p.dim;
+          v[i] = in ? __ldcg(row + at + i * 32 + lane) : 0.f;
+          u[i] = (in && i * 32 + lane < p.rot_dims) ? __ldcg(row + at + other[i]) : 0.f;
+          if (p.bias && in) {
+            v[i] += p.bias[at + i * 32 + lane];
+            if (i * 32 + lane < p.rot_dims) u[i] += p.bias[at + other[i]];
+          }
+        }
+      };
+      auto turn = [&](float (&v)[PL], const float (&u)[PL]) {     // returns 1 / rms
         float ss = 0.f;
 #pragma unroll
-        for (int i = 0; i < PL; ++i) ss += v[u][i] * v[u][i];
-        const float iq = 1.f / sqrtf(warp_sum(ss) / float(p.dim) + p.eps);
+        for (int i = 0; i < PL; ++i) {
+          v[i] = fmaf(v[i], cs[i], u[i] * sn[i]);
+          ss += v[i] * v[i];
+        }
+        return 1.f / sqrtf(warp_sum(ss) / float(p.dim) + p.eps);
+      };
+      float v[4][PL], u[4][PL];
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        const int r = warp * 4 + w;
+        load_head((kvh * p.G + gt * 16 + r) * p.dim, r < q_rows, v[w], u[w]);
+      }
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        const float iq = turn(v[w], u[w]);
 #pragma unroll
         for (int i = 0; i < PL; ++i) {
           const int d = i * 32 + lane;
-          sQ[r][d] = __float2bfloat16_rn(d < p.dim ? v[u][i] * iq * p.q_w[d] : 0.f);
+          sQ[warp * 4 + w][d] = __float2bfloat16_rn(d < p.dim ? v[w][i] * iq * (p.q_w ? p.q_w[d] : 1.f) : 0.f);
         }
       }
       if (owner && RB_BOUNDS((len - 1) / kFsPage, p.max_blocks)) {
@@ -186,21 +222,18 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
         __nv_bfloat16* kd = p.k_cache + slot * p.dkp;
         __nv_bfloat16* vd = p.v_cache + slot * p.dvp;
         if (warp == kFsWarps - 1) {
-          float f[PL], ss = 0.f;
-#pragma unroll
-          for (int i = 0; i < PL; ++i) {
-            f[i] = i * 32 + lane < p.dim ? __ldcg(row + nq + kvh * p.dim + i * 32 + lane) : 0.f;
-            ss += f[i] * f[i];
-          }
-          const float ik = 1.f / sqrtf(warp_sum(ss) / float(p.dim) + p.eps);
+          load_head(nq + kvh * p.dim, true, v[0], u[0]);
+          const float ik = turn(v[0], u[0]);
 #pragma unroll
           for (int i = 0; i < PL; ++i) {
             const int d = i * 32 + lane;
-            if (d < p.dim) kd[d] = __float2bfloat16_rn(f[i] * ik * p.k_w[d]);
+            if (d < p.dim) kd[d] = __float2bfloat16_rn(v[0][i] * ik * (p.k_w ? p.k_w[d] : 1.f));
           }
         }
-        for (int d = threadIdx.x; d < p.vdim; d += kFsThreads)
-          vd[d] = __float2bfloat16_rn(__ldcg(row + nq + nk + kvh * p.vdim + d));
+        for (int d = threadIdx.x; d < p.vdim; d += kFsThreads) {
+          const int at = nq + nk + kvh * p.vdim + d;
+          vd[d] = __float2bfloat16_rn(__ldcg(row + at) + (p.bias ? p.bias[at] : 0.f));
+        }
       }
     } else {
     // this thread's share of the tile's queries, un-normalised but weighted (independent loads)
@@ -491,7 +524,8 @@ extern "C" long long rmlx_flash_decode_scored_ticket_elems(int B, int Hq, int Hk
 
 // q (bf16) or raw (fp32, with q_w, k_w, eps: the fused form), exactly one of them. dkp / dvp: dim /
 // vdim rounded up to eight. gate: bf16 [rows, ldg] output gate logits of the plain form, or null; head_norm,
-// gate_col (-1: none): the fused form's. `tickets` is zero on the first call; the kernel leaves it zero.
+// gate_col (-1: none): the fused form's; with head_norm also bias (fp32, raw's layout, or null) and the rotation of the
+// first rot_dims values (inv_freq fp32 [rot_dims / 2]). `tickets` is zero on the first call; the kernel leaves it zero.
 extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw_ld, const float* q_w,
                                         const float* k_w, float eps, void* k_cache, void* v_cache,
                                         const int* block_table, const int* positions, const int* rows,
@@ -500,11 +534,14 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
                                         int dkp, int dvp, int max_blocks, int splits, int window, int chunk,
                                         float scale, float softcap, const float* temp, const float* r1,
                                         const float* r2, const float* sink, const void* gate, int ldg,
-                                        int head_norm, int gate_col, int pdl, cudaStream_t st) {
+                                        int head_norm, int gate_col, const float* bias, const float* inv_freq,
+                                        int rot_dims, float grow, int pdl, cudaStream_t st) {
   if (B < 1 || B > 65535 || Hkv < 1 || Hq % Hkv || splits < 1 || splits > kFsMaxSplits || (!q) == (!raw) ||
       dkp % 8 || dvp % 8 || dim > dkp || vdim > dvp || dim < 1 || vdim < 1 || (r1 && !r2))
     return -2;
-  if (raw && (!q_w || !k_w || raw_ld < (Hq + Hkv) * dim + Hkv * vdim)) return -2;
+  if (raw && (((!q_w || !k_w) && !head_norm) || raw_ld < (Hq + Hkv) * dim + Hkv * vdim)) return -2;
+  if ((bias || rot_dims) && !(raw && head_norm)) return -2;
+  if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || (rot_dims && !inv_freq)) return -2;
   if (splits > 1 && (!part_o || !part_ml || !tickets)) return -2;
   FsParams p;
   p.q = static_cast<const __nv_bfloat16*>(q); p.raw = raw; p.raw_ld = raw_ld; p.q_w = q_w; p.k_w = k_w; p.eps = eps;
@@ -516,6 +553,7 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
   p.S = splits; p.window = window; p.chunk = chunk; p.dim = dim; p.vdim = vdim; p.dkp = dkp; p.dvp = dvp;
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2; p.mod.sink = sink;
   p.gate.gate = gate; p.gate.ld = ldg; p.head_norm = head_norm; p.gate_col = gate_col;
+  p.bias = bias; p.inv_freq = inv_freq; p.rot_dims = rot_dims; p.grow = grow;
   if (raw && gate_col >= 0 && raw_ld < gate_col + Hq) return -2;
   if (p.Hkv * p.gtiles > 65535) return -2;
   const dim3 grid(splits, Hkv * p.gtiles, B);

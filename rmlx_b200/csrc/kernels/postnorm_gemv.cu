@@ -290,11 +290,11 @@ postnorm_expert_kernel(const __nv_bfloat16* __restrict__ w, int K, const float* 
   }
 }
 
-// grid (row blocks, tokens): y[b, n] = sum_s weight_s * (Wdown[e_s] act_s)[n] + identity * x[b, n], n < N.
+// grid (row blocks, tokens): y[b, n] = sum_s weight_s * (Wdown[e_s] act_s)[n] + identity * x[b, n], n < N. y may be x.
 __global__ void __launch_bounds__(kGemvThreads, 2)
 expert_out_kernel(const __nv_bfloat16* __restrict__ w, int rows_e, int K, const __nv_bfloat16* __restrict__ act, int ld_act,
                   const int* __restrict__ idx, const float* __restrict__ weights, const float* __restrict__ identity,
-                  const float* __restrict__ x, float* __restrict__ y, int ldx, int N, int top_k, int experts) {
+                  const float* x, float* y, int ldx, int N, int top_k, int experts) {
   extern __shared__ __align__(16) char smem[];        // [top_k] staged activations
   __shared__ int s_e[kRouteMaxTop];
   __shared__ float s_w[kRouteMaxTop];

@@ -41,7 +41,7 @@ class LatentWeights:
     source: int                      # the layer whose cache rows are read
     w_in: LinearWeight               # [rows, width_p]: q (or the query latent) | latent | rotated key part
     down_at: int                     # column of the latent in a row of w_in's result
-    q_norm: Optional[torch.Tensor]   # fp32 [q_rank]; None: no query latent
+    q_norm: Optional[torch.Tensor]   # fp32 [pad8(q_rank)]; None: no query latent
     w_uq: Optional[LinearWeight]     # [rows, pad8(q_rank)]
     c_norm: Optional[torch.Tensor]   # fp32 [rank]; None: the rows are another layer's
     w_uk: torch.Tensor               # [heads, lat_p, dim_p]: queries into the latent space
@@ -144,7 +144,7 @@ class WeightBuilder:
         q_norm = w_uq = None
         if m.q_rank:
             first, down_at = g("dq"), pad8(m.q_rank)
-            q_norm, w_uq = self.vec(g("dq.norm")), self.lin([g("uq")], pad8(q_cols), pad8(m.q_rank))
+            q_norm, w_uq = self.vec(g("dq.norm"), down_at), self.lin([g("uq")], pad8(q_cols), pad8(m.q_rank))
         else:
             first, down_at = g("q"), q_cols
         rows = down_at + (m.kv_rank + m.rot_dim if own else 0)
@@ -369,11 +369,13 @@ class RaggedModel:
         pool, b = c.cache.k[mw.source], c.batch
         q_raw = raw
         if mw.w_uq is not None:
-            cq = TN.rows_norm(raw, mw.q_norm, self.cfg.norm_eps, c.bufs.get("q_lat", t, mw.w_uq.k, dtype=dt), pdl=pdl)
             if raw.dtype == dt:
+                cq = TN.rows_norm(raw, mw.q_norm, self.cfg.norm_eps, m.q_rank, c.bufs.get("q_lat", t, mw.w_uq.k, dtype=dt), pdl=pdl)
                 q_raw = N.linear(cq, mw.w_uq.w, c.bufs.get("q_up", t, mw.w_uq.n, dtype=dt), pdl=pdl)
-            else:                                  # decode: raw is fp32 beside bf16 weights
-                q_raw = N.matvec_out(cq, mw.w_uq.w, c.bufs.get("q_up", t, mw.w_uq.n, dtype=torch.float32), pdl=pdl)
+            else:                                  # mat-vec decode: raw is fp32 beside bf16 weights
+                q_raw = c.bufs.get("q_up32", t, mw.w_uq.n, dtype=torch.float32)
+                P.norm_in_proj(raw[:, :mw.w_uq.k], mw.q_norm, self.cfg.norm_eps, m.q_rank, mw.w_uq.w, mw.w_uq.n, 0.0, 0.0, q_raw,
+                               None, pdl=pdl)
         down = raw[:, mw.down_at:] if mw.c_norm is not None else None
         q = c.bufs.get("q", t, m.heads, mw.dim_p + mw.rot_p, dtype=dt)
         q_abs = c.bufs.get("q_abs", t, m.heads, mw.lat_p + mw.rot_p, dtype=dt)
@@ -408,7 +410,7 @@ class RaggedModel:
         f, t = fw.spec, c.t
         i32 = dict(dtype=torch.int32)
         return R.Routing(c.bufs.get("route_idx", t, f.top, **i32), c.bufs.get("route_w", t, f.top, dtype=torch.float32),
-                         c.bufs.get("route_id", t, dtype=torch.float32) if f.identity else None, c.bufs.get("route_counts", 1, f.experts, **i32)[0],
+                         c.bufs.get("route_id", t, dtype=torch.float32), c.bufs.get("route_counts", 1, f.experts, **i32)[0],
                          c.bufs.get("route_offsets", 1, f.experts + 1, **i32)[0],
                          c.bufs.get("route_rows", t, f.top, **i32))
 

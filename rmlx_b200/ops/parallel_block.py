@@ -34,7 +34,7 @@ _lib.register_cuda_sigs({
     "rmlx_flash_decode_scored_part_o_elems": ("iiiii", "q"),
     "rmlx_flash_decode_scored_part_ml_elems": ("iiii", "q"),
     "rmlx_flash_decode_scored_ticket_elems": ("iii", "q"),
-    "rmlx_flash_decode_scored": ("ppippfpppppppppp" "iiiiiiiiiii" "ffpppp" "piiiip", "i"),
+    "rmlx_flash_decode_scored": ("ppippfpppppppppp" "iiiiiiiiiii" "ffpppp" "piii" "ppif" "ip", "i"),
 })
 
 
@@ -260,11 +260,13 @@ def flash_decode_scored(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tabl
                         k_w: Optional[torch.Tensor] = None, eps: float = 0.0, rows: Optional[torch.Tensor] = None,
                         table_rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None, window: int = 0,
                         gate: Optional[torch.Tensor] = None, head_norm: bool = False, gate_col: int = -1,
-                        chunk: int = 0, pdl: bool = False) -> torch.Tensor:
+                        chunk: int = 0, bias: Optional[torch.Tensor] = None, inv_freq: Optional[torch.Tensor] = None,
+                        grow: float = 1.0, pdl: bool = False) -> torch.Tensor:
     """One token per row: q [T, H, dk] (keys already appended) or the fused form on the un-normalised
     fp32 projection ``raw`` [T, >= q|k|v], which also appends the key and value (``head_norm``: the
-    norms are per head, their weights [dim]; ``gate_col``: where the output gate's logits start in a
-    row). ``rows`` int32: the batch rows to run (default: the first ``n_rows``)."""
+    norms are per head, their weights [dim] or None; with it ``bias`` is added to the projection, and the first
+    ``2 * inv_freq.numel()`` values of query and key heads rotate, i with i + pairs, before the norm; ``gate_col``:
+    where the output gate's logits start in a row). ``rows`` int32: the batch rows to run (default: the first ``n_rows``)."""
     _lib.require_cuda_tensor(k_cache, v_cache, block_table, positions, out, q, raw)
     src = q if q is not None else raw
     n = rows.numel() if rows is not None else (n_rows or src.shape[0])
@@ -277,8 +279,8 @@ def flash_decode_scored(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tabl
         _lib.ptr(table_rows), out.data_ptr(), scratch.part_o.data_ptr(), scratch.part_ml.data_ptr(),
         scratch.tickets.data_ptr(), n, heads, k_cache.shape[1], dim, vdim, k_cache.shape[3], v_cache.shape[3],
         block_table.stride(0), scratch.splits, window, chunk, *mods.args(),
-        *_gate_args(gate, 0 if q is None else q.shape[0], heads, torch.bfloat16), int(head_norm), gate_col, int(pdl),
-        _lib.stream_ptr())
+        *_gate_args(gate, 0 if q is None else q.shape[0], heads, torch.bfloat16), int(head_norm), gate_col,
+        _lib.ptr(bias), _lib.ptr(inv_freq), 0 if inv_freq is None else 2 * inv_freq.numel(), grow, int(pdl), _lib.stream_ptr())
     _lib.check(rc, "flash_decode_scored")
     return out
 

@@ -1,5 +1,5 @@
 """Linear recurrences token by token (csrc/kernels/linear_scan.cu): gated linear attention and state-space heads with
-their short convolution, and the norm of their outputs with a silu gate. A sequence's state is its slot's row of a
+their short convolution, and the norm of their outputs with a silu gate; their decode steps (twin_norm_gemv.cu). A sequence's state is its slot's row of a
 flat fp32 pool (``PagedKvCache.layer_state`` views)."""
 from __future__ import annotations
 
@@ -18,6 +18,9 @@ _lib.register_cuda_sigs({
     "rmlx_scan_record": ("iiii", "q"),
     "rmlx_gla_scan": ("pppi" "pip" "ff" "pippi" "pqpi" "iiii" "pip", "i"),
     "rmlx_ssd_scan": ("piii" "ppi" "pppp" "pippi" "pqpi" "iiiii" "pip", "i"),
+    "rmlx_gla_decode_supported": ("ii", "i"),
+    "rmlx_gla_decode": ("piiiii" "pipff" "pfp" "pq" "pi" "iiiiip", "i"),
+    "rmlx_ssd_decode": ("piii" "ppi" "ppppp" "pq" "pi" "pfi" "pi" "iiiii" "ip", "i"),
     "rmlx_gated_norm": ("pipipfpi" "iiiiiip", "i"),
 })
 
@@ -88,3 +91,43 @@ def gated_norm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float,
                                      _f32(out), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "gated_norm")
     return out
+
+
+# ------------------------------------------------------------------ decode (csrc/kernels/twin_norm_gemv.cu)
+def gla_decode_supported(n: int, d: int) -> bool:
+    return bool(_lib.cuda().rmlx_gla_decode_supported(n, d))
+
+
+def gla_decode(raw: torch.Tensor, at, a2: torch.Tensor, bias: torch.Tensor, tau: float, scale: float, norm: torch.Tensor,
+               eps: float, slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> None:
+    """One token per row through decay, state, head norm and gate: raw fp32 [B, ..] with q, k, v, g and the decay's first
+    factor at the columns ``at``, ``a2`` bf16 [>= H dim, rank]; out bf16 [B, >= H vdim]."""
+    _lib.require_cuda_tensor(raw, a2, bias, norm, slots, state, out)
+    _, h, n, d = state.shape
+    assert raw.dtype == torch.float32 and a2.dtype == out.dtype == torch.bfloat16 and a2.is_contiguous() and at[0] == 0
+    assert state.stride()[1:] == (n * d, d, 1) and slots.dtype == torch.int32 and bias.numel() == h * n and norm.numel() == h * d
+    rc = _lib.cuda().rmlx_gla_decode(
+        raw.data_ptr(), raw.stride(0), at[1], at[2], at[3], at[4], a2.data_ptr(), a2.shape[1], bias.data_ptr(), 1.0 / tau, scale,
+        norm.data_ptr(), eps, slots.data_ptr(), state.data_ptr(), state.stride(0), out.data_ptr(), out.stride(0), raw.shape[0], h,
+        n, d, int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "gla_decode")
+
+
+def ssd_decode(raw: torch.Tensor, x_at: int, dt_at: int, conv_w: torch.Tensor, conv_b: torch.Tensor,
+               carried: Optional[torch.Tensor], dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor, groups: int,
+               slots: torch.Tensor, state: torch.Tensor, y: torch.Tensor, norm: torch.Tensor, eps: float, norm_groups: int,
+               out: torch.Tensor, pdl: bool = False) -> None:
+    """One token per row through convolution, state, gate and grouped norm: raw fp32 [B, ..] = z at 0, x | B | C at
+    ``x_at``, dt at ``dt_at``; ``y`` fp32 scratch [B, >= H d], out bf16 [B, >= H d]."""
+    _lib.require_cuda_tensor(raw, conv_w, conv_b, dt_bias, a_log, skip, slots, state, y, norm, out)
+    _, h, n, d = state.shape
+    taps, ch = conv_w.shape
+    assert raw.dtype == y.dtype == torch.float32 and out.dtype == torch.bfloat16 and ch == h * d + 2 * groups * n
+    assert state.stride()[1:] == (n * d, d, 1) and slots.dtype == torch.int32 and norm.numel() == h * d
+    assert taps == 1 or (carried.shape[1:] == (taps - 1, ch) and carried.stride(0) == state.stride(0))
+    rc = _lib.cuda().rmlx_ssd_decode(
+        raw.data_ptr(), raw.stride(0), x_at, dt_at, conv_w.data_ptr(), conv_b.data_ptr(), taps,
+        carried.data_ptr() if taps > 1 else None, dt_bias.data_ptr(), a_log.data_ptr(), skip.data_ptr(), slots.data_ptr(),
+        state.data_ptr(), state.stride(0), y.data_ptr(), y.stride(0), norm.data_ptr(), eps, norm_groups, out.data_ptr(),
+        out.stride(0), raw.shape[0], h, groups, n, d, int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "ssd_decode")

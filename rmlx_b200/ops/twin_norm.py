@@ -1,5 +1,5 @@
 """Row operations of decoders whose mixer and feed-forward read the same residual row through norms of their own
-(csrc/kernels/twin_norm_rows.cu). Activations are bf16 or fp32; the dtype of the tensors picks the kernels."""
+(csrc/kernels/twin_norm_rows.cu), and the decode projections that read it (twin_norm_gemv.cu). Activations are bf16 or fp32; the dtype of the tensors picks the kernels."""
 from __future__ import annotations
 
 import math
@@ -14,6 +14,9 @@ from .routed import Routing
 _lib.register_cuda_sigs({
     "rmlx_twin_norm": ("ppippi" "ppppf" "iiiiip", "i"),
     "rmlx_rows_norm": ("piipfpi" "iiiip", "i"),
+    "rmlx_twin_in_max_rows": ("i", "i"),
+    "rmlx_twin_in_gated": ("pppfii" "pipi" "pipif" "iip", "i"),
+    "rmlx_twin_in_router": ("pppfii" "pipi" "ppipp" "ppip" "iip", "i"),
     "rmlx_rotary_norm_append": ("piippiff" "ppp" "ppp" "iiiiiiiiiiip", "i"),
 })
 
@@ -53,12 +56,13 @@ def twin_norm(x: torch.Tensor, w1: Optional[torch.Tensor], h1: Optional[torch.Te
     _lib.check(rc, "twin_norm")
 
 
-def rows_norm(x: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor, pdl: bool = False) -> torch.Tensor:
-    """out = RMSNorm of the first ``w.numel()`` columns of x times w, zeros in the rest of out's columns."""
+def rows_norm(x: torch.Tensor, w: torch.Tensor, eps: float, width: int, out: torch.Tensor, pdl: bool = False) -> torch.Tensor:
+    """out = RMSNorm of the first ``width`` columns of x times w, zeros in the rest of out's columns."""
     _lib.require_cuda_tensor(x, w, out)
-    assert w.dtype == torch.float32 and out.is_contiguous() and x.shape[0] == out.shape[0] and x.stride(1) == 1
+    assert w.dtype == torch.float32 and w.numel() >= width and out.is_contiguous() and x.shape[0] == out.shape[0]
+    assert x.stride(1) == 1
     rc = _lib.cuda().rmlx_rows_norm(x.data_ptr(), x.stride(0), _f32(x), w.data_ptr(), eps, out.data_ptr(), out.shape[1],
-                                    x.shape[0], w.numel(), _f32(out), int(pdl), _lib.stream_ptr())
+                                    x.shape[0], width, _f32(out), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "rows_norm")
     return out
 
@@ -79,3 +83,50 @@ def rotary_norm_append(raw: torch.Tensor, bias: Optional[torch.Tensor], inv_freq
         _lib.ptr(token_seq), t, heads, hkv, dim, vdim, k_cache.shape[3], v_cache.shape[3], block_table.stride(0),
         k_cache.shape[2], _f32(q), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "rotary_norm_append")
+
+
+# ------------------------------------------------------------------ decode projections (csrc/kernels/twin_norm_gemv.cu)
+def _row_chunks(b: int, k: int):
+    step = int(_lib.cuda().rmlx_twin_in_max_rows(k))
+    if step < 1:
+        raise _lib.NativeError(f"decode projections: {k} values do not fit a block's shared memory")
+    return [(lo, min(b, lo + step)) for lo in range(0, b, step)]
+
+
+def _twin_in_checks(x, w1, w, out):
+    _lib.require_cuda_tensor(x, w1, w, out)
+    assert x.dtype == out.dtype == w1.dtype == torch.float32 and w.dtype == torch.bfloat16 and x.is_contiguous()
+    assert w.is_contiguous() and w.shape[1] == x.shape[1] == w1.numel() and out.shape == (x.shape[0], w.shape[0])
+
+
+def twin_in(x: torch.Tensor, w1: torch.Tensor, eps: float, width: int, w: torch.Tensor, out: torch.Tensor,
+            w2: Optional[torch.Tensor] = None, w_gu: Optional[torch.Tensor] = None, act: Optional[torch.Tensor] = None,
+            limit: float = 0.0, pdl: bool = False) -> None:
+    """out = W RMSNorm(x; w1) in fp32 and, in the same launch, act = the gated activation of W_gu RMSNorm(x; w2) in bf16
+    (W_gu = [gate; up]; None: no feed-forward)."""
+    _twin_in_checks(x, w1, w, out)
+    assert w_gu is None or (w_gu.is_contiguous() and w_gu.shape == (2 * act.shape[1], x.shape[1]) and act.dtype == w_gu.dtype)
+    for lo, hi in _row_chunks(*x.shape):
+        a = None if act is None else act[lo:]
+        rc = _lib.cuda().rmlx_twin_in_gated(
+            x[lo:].data_ptr(), w1.data_ptr(), _lib.ptr(w2), eps, width, x.shape[1], w.data_ptr(), w.shape[0], out[lo:].data_ptr(),
+            out.stride(0), _lib.ptr(w_gu), 0 if act is None else act.shape[1], _lib.ptr(a), 0 if act is None else act.stride(0),
+            limit, hi - lo, int(pdl), _lib.stream_ptr())
+        _lib.check(rc, "twin_in_gated")
+
+
+def twin_in_router(x: torch.Tensor, w1: torch.Tensor, eps: float, width: int, w: torch.Tensor, out: torch.Tensor,
+                   w2: torch.Tensor, router: torch.Tensor, bias: torch.Tensor, logits: torch.Tensor, h2: torch.Tensor,
+                   ticket: torch.Tensor, r: Routing, pdl: bool = False) -> None:
+    """out = W RMSNorm(x; w1) in fp32 and, in the same launch, h2 = RMSNorm(x; w2) in fp32, its router logits and the
+    choice of experts. ``ticket``: one int32 word, zero."""
+    _twin_in_checks(x, w1, w, out)
+    assert router.dtype == torch.bfloat16 and router.is_contiguous() and bias.numel() == router.shape[0]
+    assert h2.shape == x.shape and h2.dtype == torch.float32 and h2.is_contiguous() and logits.is_contiguous()
+    for lo, hi in _row_chunks(*x.shape):
+        rc = _lib.cuda().rmlx_twin_in_router(
+            x[lo:].data_ptr(), w1.data_ptr(), w2.data_ptr(), eps, width, x.shape[1], w.data_ptr(), w.shape[0], out[lo:].data_ptr(),
+            out.stride(0), router.data_ptr(), bias.data_ptr(), router.shape[0], logits[lo:].data_ptr(), h2[lo:].data_ptr(),
+            r.idx[lo:].data_ptr(), r.weights[lo:].data_ptr(), r.idx.shape[1], ticket.data_ptr(), hi - lo, int(pdl),
+            _lib.stream_ptr())
+        _lib.check(rc, "twin_in_router")

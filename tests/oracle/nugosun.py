@@ -103,8 +103,10 @@ def chunked_attention(w, m, eps, h):
     q, k = (rms_norm(rotate_halves(proj(s, n), m["rot"]), eps) for s, n in (("q", hd), ("k", kv)))
     k, v = (s.repeat_interleave(hd // kv, 0) for s in (k, proj("v", kv)))
     s = q @ k.transpose(1, 2) * m["scale"]
-    s = m["softcap"] * torch.tanh(s / m["softcap"])
-    return heads_last(softmax_attention(s, same_chunk(len(h), m["mask"]["size"]), v)) @ w["o"].T
+    if m.get("softcap"):
+        s = m["softcap"] * torch.tanh(s / m["softcap"])
+    seen = same_chunk(len(h), m["mask"]["size"]) if m.get("mask") else visible(len(h))
+    return heads_last(softmax_attention(s, seen, v)) @ w["o"].T
 
 
 def side_by_side(w, m, eps, h):
