@@ -1,14 +1,14 @@
 // Recurrences with an fp32 matrix state per head, token by token: S [n, d] (rows: key channels, columns: value
 // channels) carried per sequence,
-//     o_t = scale_t * S^T r_t + extra_t,   S <- diag(w_t) S + k_t v_t^T.
+//     o_t = scale_t * S^T r_t + own_t * v_t,   S <- diag(w_t) S + k_t v_t^T.
 // WKV, gated linear attention and state-space heads are all of this form: what reads the state after its update
-// has the decay folded into r (or, when a head has one decay for all its rows, into scale) and the new token's
-// own share in `extra`.
+// has the decay folded into r (or, when a head has one decay for all its rows, into scale) and adds the new token's
+// own share, a multiple of its v.
 //
 // Columns are independent of each other. A prepare kernel takes the exponentials once and writes fp32 records
 // in token order: one per (head, token) with r | k | w - or, with one decay per head (ONE), one per (group of
-// heads, token) with r | k - and one per (head, column block, token) with v | extra (| scale, which is the decay,
-// too). scan_kernel: a block owns one (sequence, head, group of columns) and walks the sequence's new tokens,
+// heads, token) with r | k - and one per (head, column block, token) with v and own (ONE: x, the decay, which is
+// scale, too, the step size dt with v = dt x, and the multiple of x). scan_kernel: a block owns one (sequence, head, group of columns) and walks the sequence's new tokens,
 // whose records arrive in shared memory by two bulk copies per chunk, two chunks ahead: no instruction of the
 // scan is spent on staging (when the block converted its own inputs, that took more issue slots than the
 // recurrence). A thread holds ROWS rows of four columns in registers, so that each r, k and w it reads serves
@@ -46,7 +46,7 @@ struct ScanCfg {
   static constexpr int kCols = kScanThreads / LANES * kScanCols; // columns per block
   static constexpr int kChunk = kRows > 128 ? 8 : 16;            // tokens per chunk
   static constexpr int kRec = (ONE ? 2 : 3) * kRows;             // floats of a row record
-  static constexpr int kCol = 2 * kCols + (ONE ? 4 : 0);         // floats of a column record
+  static constexpr int kCol = kCols + 4;                         // floats of a column record: v | own, or x | decay, dt, own
   static constexpr int kStage = kChunk * (kRec + kCol);
   static constexpr int kSmem = kScanStages * kStage * 4 + 64;
   static constexpr int blocks(int d) { return (d + kCols - 1) / kCols; }
@@ -131,7 +131,7 @@ scan_prepare_kernel(IN in, float* __restrict__ rec, float* __restrict__ col, int
     in.cols4(t, h, i, v);
     float* o = col + ((size_t(h) * nb + i / C::kCols) * rows + t) * C::kCol + i % C::kCols;
     *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
-    *reinterpret_cast<float4*>(o + C::kCols) = make_float4(own * v[0], own * v[1], own * v[2], own * v[3]);
+    if (i % C::kCols == 0) *reinterpret_cast<float4*>(o + C::kCols) = make_float4(own, 0.f, 0.f, 0.f);
   }
 }
 
@@ -191,13 +191,18 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(ScanParams p) {
   // after the butterfly, the lanes of a column group hold column `mine` of the four
   const int mine = (g & (LANES / 2) ? 2 : 0) + (g & (LANES / 4) ? 1 : 0);
   const bool writer = g % (LANES / 4) == 0 && col0 + c0 + mine < dim;
-  const int at_extra = C::kCols + c0 + mine, at_one = 2 * C::kCols;
+  const int at_own = C::kCols + (ONE ? 2 : 0);
   float* op = p.out + size_t(row0) * p.ld_out + h * dim + col0 + c0 + mine;
 
   // one token: the state's part of o, then the state's update
   auto token = [&](const float* b, const float* bc, float (&o)[kScanCols]) {
-    const float4 v = *reinterpret_cast<const float4*>(bc + c0);
-    const uint64_t one = ONE ? scan_pair(bc[at_one], bc[at_one]) : 0;
+    float4 v = *reinterpret_cast<const float4*>(bc + c0);
+    uint64_t one = 0;
+    if (ONE) {
+      const float2 a = *reinterpret_cast<const float2*>(bc + C::kCols);      // decay, dt
+      one = scan_pair(a.x, a.x);
+      v.x *= a.y; v.y *= a.y; v.z *= a.y; v.w *= a.y;
+    }
     const uint64_t v2[kScanCols] = {scan_pair(v.x, v.x), scan_pair(v.y, v.y), scan_pair(v.z, v.z), scan_pair(v.w, v.w)};
     uint64_t acc[kScanCols] = {0, 0, 0, 0};
 #pragma unroll
@@ -250,7 +255,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(ScanParams p) {
 #pragma unroll
         for (int q = 0; q < TU; ++q) {
           const float* bc = buf_col + (t + q) * C::kCol;
-          oc[size_t(t + q) * p.ld_out] = ONE ? fmaf(bc[at_one], sum[q], bc[at_extra]) : sum[q] + bc[at_extra];
+          oc[size_t(t + q) * p.ld_out] = fmaf(bc[at_own], bc[c0 + mine], ONE ? bc[C::kCols] * sum[q] : sum[q]);
         }
       }
     };
@@ -276,7 +281,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(ScanParams p) {
       float o[kScanCols];
       token(buf + t * C::kRec, bc, o);
       const float sum = fold(o);
-      if (writer) oc[size_t(t) * p.ld_out] = ONE ? fmaf(bc[at_one], sum, bc[at_extra]) : sum + bc[at_extra];
+      if (writer) oc[size_t(t) * p.ld_out] = fmaf(bc[at_own], bc[c0 + mine], ONE ? bc[C::kCols] * sum : sum);
     }
     __syncthreads();                                 // the stage has been read
     if (threadIdx.x == 0 && ch + kScanStages < chunks) issue(ch + kScanStages);

@@ -122,11 +122,10 @@ ssd_prepare_kernel(SsdIn<T> in, float* __restrict__ rec, float* __restrict__ col
   const int nb = C::blocks(in.d), per = in.H / in.G, width = nb * C::kCols;
   for (int u = threadIdx.x; u < in.H * width; u += kRowThreads) {
     const int h = u / width, i = u - h * width;
-    const float x = i < in.d ? sm[h * in.d + i] : 0.f, v = s_dt[h] * x;
     float* o = col + ((size_t(h) * nb + i / C::kCols) * rows + t) * C::kCol;
-    o[i % C::kCols] = v;
-    o[C::kCols + i % C::kCols] = fmaf(s_own[h / per], v, in.skip[h] * x);
-    if (i % C::kCols < 4) o[2 * C::kCols + i % C::kCols] = s_a[h];
+    o[i % C::kCols] = i < in.d ? sm[h * in.d + i] : 0.f;
+    if (i % C::kCols == 0)
+      *reinterpret_cast<float4*>(o + C::kCols) = make_float4(s_a[h], s_dt[h], fmaf(s_own[h / per], s_dt[h], in.skip[h]), 0.f);
   }
 }
 
@@ -154,53 +153,62 @@ conv_carry_kernel(const T* __restrict__ raw, int ld, int x_at, float* __restrict
   }
 }
 
-// out[t, c] over equal groups of columns: gate_first: f = o silu(gate), f / rms(f over the group) * w;
-// else o / rms(o over the group) * w * silu(gate). L lanes (256: a block) per (row, group).
-template <class T, int L>
+// out[t, c] over equal groups of columns: FIRST: f = o silu(gate), f / rms(f over the group) * w;
+// else o / rms(o over the group) * w * silu(gate). L lanes (256: a block) per (row, group), KEEP chunks of eight a lane
+// keeps; what is left is read again.
+template <class T, int L, int KEEP, bool FIRST>
 __global__ void __launch_bounds__(kRowThreads)
 gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ gate, int ld_g, const float* __restrict__ w,
-                  float eps, T* __restrict__ out, int ld_out, int rows, int groups, int size, int gate_first) {
+                  float eps, T* __restrict__ out, int ld_out, int rows, int groups, int size) {
   __shared__ float red[kRowThreads / 32];
-  constexpr int kKeep = 2;                             // chunks of eight a lane keeps
   pdl_launch_dependents();
   pdl_wait();
-  const long long unit = (blockIdx.x * (long long)(kRowThreads) + threadIdx.x) / L;
-  const int lane = threadIdx.x % L;
-  const bool live = unit < (long long)(rows) * groups;   // the lanes of a warp stay together for the sums
-  const int t = live ? int(unit / groups) : 0, at = live ? int(unit - (long long)(t) * groups) * size : 0;
+  const int unit = (blockIdx.x * kRowThreads + threadIdx.x) / L, lane = threadIdx.x % L;
+  const bool live = unit < rows * groups;              // the lanes of a warp stay together for the sums
+  const int t = live ? unit / groups : 0, at = live ? (unit - t * groups) * size : 0;
   const bool vec = size % 8 == 0 && ld_o % 8 == 0 && ld_g % 8 == 0 && ld_out % 8 == 0;
   const float* op = o + size_t(t) * ld_o + at;
   const T* gp = gate + size_t(t) * ld_g + at;
-  float f[kKeep][8], z[kKeep][8], ssq = 0.f;
-  auto load = [&](int i0, float (&a)[8], float (&s)[8]) {
+  float f[KEEP][8], ssq = 0.f;
+  auto load = [&](int i0, float (&a)[8]) {
     load8_upto(op + i0, size - i0, vec, a);
-    load8_upto(gp + i0, size - i0, vec, s);
+    if (FIRST) {
+      float z[8];
+      load8_upto(gp + i0, size - i0, vec, z);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      s[i] = silu_f(s[i]);
-      if (gate_first) a[i] *= s[i];
-      ssq += a[i] * a[i];
+      for (int i = 0; i < 8; ++i) a[i] *= silu_f(z[i]);
     }
   };
 #pragma unroll
-  for (int u = 0; u < kKeep; ++u) {
+  for (int u = 0; u < KEEP; ++u) {
     const int i0 = (u * L + lane) * 8;
-    if (i0 < size) load(i0, f[u], z[u]);
+    if (i0 < size) {
+      load(i0, f[u]);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ssq += f[u][i] * f[u][i];
+    }
   }
-  for (int i0 = (kKeep * L + lane) * 8; i0 < size; i0 += L * 8) {
-    float a[8], s[8];
-    load(i0, a, s);
+  for (int i0 = (KEEP * L + lane) * 8; i0 < size; i0 += L * 8) {
+    float a[8];
+    load(i0, a);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ssq += a[i] * a[i];
   }
   if (L <= 32) ssq = group_sum<L <= 32 ? L : 32>(ssq);
   else ssq = row_block_sum(ssq, red);
   if (!live) return;
   const float inv = 1.f / sqrtf(ssq / float(size) + eps);
   T* dst = out + size_t(t) * ld_out + at;
-  auto put = [&](int i0, float (&a)[8], const float (&s)[8]) {
+  auto put = [&](int i0, float (&a)[8]) {
     float g[8];
     load8_upto(w + at + i0, size - i0, vec, g);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) a[i] = a[i] * inv * g[i] * (gate_first ? 1.f : s[i]);
+    for (int i = 0; i < 8; ++i) a[i] *= inv * g[i];
+    if (!FIRST) {
+      load8_upto(gp + i0, size - i0, vec, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) a[i] *= silu_f(g[i]);
+    }
     if (vec) {
       store8(dst + i0, a);
     } else {
@@ -208,14 +216,14 @@ gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ g
     }
   };
 #pragma unroll
-  for (int u = 0; u < kKeep; ++u) {
+  for (int u = 0; u < KEEP; ++u) {
     const int i0 = (u * L + lane) * 8;
-    if (i0 < size) put(i0, f[u], z[u]);
+    if (i0 < size) put(i0, f[u]);
   }
-  for (int i0 = (kKeep * L + lane) * 8; i0 < size; i0 += L * 8) {
-    float a[8], s[8];
-    load(i0, a, s);                                    // (the sum is not used again)
-    put(i0, a, s);
+  for (int i0 = (KEEP * L + lane) * 8; i0 < size; i0 += L * 8) {
+    float a[8];
+    load(i0, a);
+    put(i0, a);
   }
 }
 
@@ -323,21 +331,24 @@ extern "C" int rmlx_ssd_scan(const void* raw, int ld, int x_at, int dt_at, const
 extern "C" int rmlx_gated_norm(const float* o, int ld_o, const void* gate, int ld_g, const float* w, float eps, void* out,
                                int ld_out, int rows, int groups, int size, int gate_first, int f32, int pdl, cudaStream_t st) {
   if (rows < 1 || groups < 1 || size < 1 || ld_o < groups * size || ld_g < groups * size || ld_out < groups * size) return -2;
-  const int lanes = size <= 128 ? 8 : size <= 1024 ? 32 : 256;
-  const long long blocks = (1LL * rows * groups * lanes + kRowThreads - 1) / kRowThreads;
-  if (blocks > 0x7fffffffLL) return -2;
+  const int lanes = size <= 64 ? 8 : size <= 128 ? 16 : size <= 256 ? 32 : 256;
+  const long long units = 1LL * rows * groups, blocks = (units * lanes + kRowThreads - 1) / kRowThreads;
+  if (units * lanes > 0x7fffffffLL) return -2;
   const dim3 grid{unsigned(blocks)};
-#define RB_GN(T_, L_)                                                                                                    \
-  return launch(gated_norm_kernel<T_, L_>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o, static_cast<const T_*>(gate), \
-                ld_g, w, eps, static_cast<T_*>(out), ld_out, rows, groups, size, gate_first)
-#define RB_GNL(T_)                   \
-  {                                  \
-    if (lanes == 8) RB_GN(T_, 8);    \
-    if (lanes == 32) RB_GN(T_, 32);  \
-    RB_GN(T_, 256);                  \
+#define RB_GN(T_, L_, K_, F_)                                                                                          \
+  return launch(gated_norm_kernel<T_, L_, K_, F_>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o,                  \
+                static_cast<const T_*>(gate), ld_g, w, eps, static_cast<T_*>(out), ld_out, rows, groups, size)
+#define RB_GNL(T_, F_)                    \
+  {                                       \
+    if (lanes == 8) RB_GN(T_, 8, 1, F_);  \
+    if (lanes == 16) RB_GN(T_, 16, 1, F_); \
+    if (lanes == 32) RB_GN(T_, 32, 1, F_); \
+    RB_GN(T_, 256, 2, F_);                \
   }
-  if (f32) RB_GNL(float)
-  RB_GNL(__nv_bfloat16)
+  if (f32 && gate_first) RB_GNL(float, true)
+  if (f32) RB_GNL(float, false)
+  if (gate_first) RB_GNL(__nv_bfloat16, true)
+  RB_GNL(__nv_bfloat16, false)
 #undef RB_GNL
 #undef RB_GN
 }

@@ -339,10 +339,12 @@ struct SsdStep {
   float* out;                     // [B, ld_out] fp32
   int ld_out, H, G, n, d;
 };
-__device__ __forceinline__ float step_conv(const SsdStep& p, const float* row, const float* before, int ch, int c) {
+// Channel c's convolution without the current token.
+__device__ __forceinline__ float past_conv(const SsdStep& p, const float* before, int ch, int c) {
   float a = p.conv_b[c];
-  for (int j = 0; j < p.taps - 1; ++j) a = fmaf(p.conv_w[size_t(j) * ch + c], before[size_t(j) * ch + c], a);
-  return tn_silu(fmaf(p.conv_w[size_t(p.taps - 1) * ch + c], __ldcg(row + p.x_at + c), a));
+#pragma unroll 4
+  for (int j = 0; j < p.taps - 1; ++j) a = fmaf(p.conv_w[size_t(j) * ch + c], __ldcg(before + size_t(j) * ch + c), a);
+  return a;
 }
 
 template <int COLS, int ROWS>
@@ -362,18 +364,36 @@ ssd_decode_kernel(SsdStep p) {
   float* sp = p.state + slot + size_t(h) * n * d + col;
   float s[ROWS];
   load_state<ROWS>(sp, d, i0, i1, col < d, s);
+  // B and C of the head's group, then x of the block's columns: what earlier tokens contribute waits for nothing, either
+  const int grp = h / (p.H / p.G), last = p.taps - 1;
+  const float* before = p.carried + slot;
+  auto channel = [&](int i) {
+    if (i < n) return inner + grp * n + i;
+    if (i < 2 * n) return inner + p.G * n + grp * n + i - n;
+    return i - 2 * n < COLS && c0 + i - 2 * n < d ? h * d + c0 + i - 2 * n : -1;
+  };
+  constexpr int kKeep = 2;
+  float past[kKeep], now_w[kKeep];
+  int chan[kKeep];
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u) {
+    chan[u] = channel(u * kGemvThreads + tid);
+    past[u] = chan[u] >= 0 ? past_conv(p, before, ch, chan[u]) : 0.f;
+    now_w[u] = chan[u] >= 0 ? p.conv_w[size_t(last) * ch + chan[u]] : 0.f;
+  }
   pdl_launch_dependents();
   pdl_wait();
   const float* row = p.raw + size_t(b) * p.ld_raw;
-  const float* before = p.carried + slot;
-  const int grp = h / (p.H / p.G);
-  for (int i = tid; i < 2 * n + COLS; i += kGemvThreads) {
-    if (i < 2 * n) {
-      const int c = inner + (i < n ? grp * n + i : p.G * n + grp * n + i - n);
-      sm[i] = step_conv(p, row, before, ch, c);
-    } else if (c0 + i - 2 * n < d) {
-      sx[i - 2 * n] = step_conv(p, row, before, ch, h * d + c0 + i - 2 * n);
-    }
+  auto keep = [&](int i, float v) {
+    if (i < 2 * n) sm[i] = v;
+    else sx[i - 2 * n] = v;
+  };
+#pragma unroll
+  for (int u = 0; u < kKeep; ++u)
+    if (chan[u] >= 0) keep(u * kGemvThreads + tid, tn_silu(fmaf(now_w[u], __ldcg(row + p.x_at + chan[u]), past[u])));
+  for (int i = kKeep * kGemvThreads + tid; i < 2 * n + COLS; i += kGemvThreads) {
+    const int c = channel(i);
+    if (c >= 0) keep(i, tn_silu(fmaf(p.conv_w[size_t(last) * ch + c], __ldcg(row + p.x_at + c), past_conv(p, before, ch, c))));
   }
   const float dt = tn_softplus(__ldcg(row + p.dt_at + h) + p.dt_bias[h]), decay = expf(-expf(p.a_log[h]) * dt);
   __syncthreads();
@@ -389,16 +409,27 @@ ssd_decode_kernel(SsdStep p) {
   }
 }
 
-// grid (norm groups, batch rows): f = y silu(z), f / rms(f over the group) * norm; the row's conv inputs move up.
+// grid (norm groups + blocks of channels, batch rows): f = y silu(z), f / rms(f over the group) * norm; the channels'
+// blocks move the row's conv inputs up.
 __global__ void __launch_bounds__(kGemvThreads)
-ssd_finish_kernel(SsdStep p, const float* __restrict__ norm, float eps, int size, __nv_bfloat16* __restrict__ a, int ld_a) {
+ssd_finish_kernel(SsdStep p, const float* __restrict__ norm, float eps, int groups, int size, __nv_bfloat16* __restrict__ a,
+                  int ld_a) {
   constexpr int kKeep = 16;
   __shared__ float red[kGemvWarps];
   const int b = blockIdx.y, at = blockIdx.x * size, tid = threadIdx.x;
+  const float* row = p.raw + size_t(b) * p.ld_raw;
   pdl_launch_dependents();
   pdl_wait();
+  if (int(blockIdx.x) >= groups) {
+    const int ch = p.H * p.d + 2 * p.G * p.n, c = (blockIdx.x - groups) * kGemvThreads + tid;
+    if (c >= ch) return;
+    float* st = p.carried + size_t(p.slots[b]) * p.stride + c;
+#pragma unroll 4
+    for (int j = 0; j + 2 < p.taps; ++j) st[size_t(j) * ch] = st[size_t(j + 1) * ch];
+    st[size_t(p.taps - 2) * ch] = __ldcg(row + p.x_at + c);
+    return;
+  }
   const float* y = p.out + size_t(b) * p.ld_out + at;
-  const float* row = p.raw + size_t(b) * p.ld_raw;
   float f[kKeep], ssq = 0.f;
   auto value = [&](int i) { return __ldcg(y + i) * tn_silu(__ldcg(row + at + i)); };
 #pragma unroll
@@ -416,14 +447,6 @@ ssd_finish_kernel(SsdStep p, const float* __restrict__ norm, float eps, int size
     if (i < size) dst[i] = __float2bfloat16_rn(f[u] * inv * norm[at + i]);
   }
   for (int i = kKeep * kGemvThreads + tid; i < size; i += kGemvThreads) dst[i] = __float2bfloat16_rn(value(i) * inv * norm[at + i]);
-  if (p.taps > 1) {
-    const int ch = p.H * p.d + 2 * p.G * p.n;
-    float* st = p.carried + size_t(p.slots[b]) * p.stride;
-    for (int c = blockIdx.x * kGemvThreads + tid; c < ch; c += gridDim.x * kGemvThreads) {
-      for (int j = 0; j + 2 < p.taps; ++j) st[size_t(j) * ch + c] = st[size_t(j + 1) * ch + c];
-      st[size_t(p.taps - 2) * ch + c] = __ldcg(row + p.x_at + c);
-    }
-  }
 }
 
 }  // namespace rb
@@ -582,6 +605,7 @@ extern "C" int rmlx_ssd_decode(const float* raw, int ld_raw, int x_at, int dt_at
 #undef RB_SD
   }();
   if (rc) return rc;
-  return launch(ssd_finish_kernel, dim3(norm_groups, B), dim3(kGemvThreads), 0, st, pdl != 0, p, norm, eps, H * d / norm_groups,
-                static_cast<__nv_bfloat16*>(a), ld_a);
+  const int movers = taps > 1 ? (H * d + 2 * G * n + kGemvThreads - 1) / kGemvThreads : 0;
+  return launch(ssd_finish_kernel, dim3(norm_groups + movers, B), dim3(kGemvThreads), 0, st, pdl != 0, p, norm, eps, norm_groups,
+                H * d / norm_groups, static_cast<__nv_bfloat16*>(a), ld_a);
 }

@@ -119,7 +119,7 @@ rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __
                           T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ block_table,
                           const int* __restrict__ positions, const int* __restrict__ token_seq, int Hq, int Hkv, int dim,
                           int vdim, int dkp, int dvp, int max_blocks, int page) {
-  extern __shared__ float trig[];          // cos [dims / 2], sin [dims / 2]
+  extern __shared__ __align__(16) float trig[];          // cos [dims / 2], sin [dims / 2]
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, pos = positions[t], half = dims / 2;
@@ -145,14 +145,34 @@ rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __
     const TR* src = row + src0;
     const float* bs = bias ? bias + src0 : nullptr;
     const bool vec = width % 8 == 0 && src0 % 8 == 0 && ldraw % 8 == 0;
+    const bool pairs = vec && half % 8 == 0;           // eight values turn with eight
     auto value = [&](int d) { return to_f32(src[d]) + (bs ? bs[d] : 0.f); };
-    auto load = [&](int d0, float (&f)[8]) {
+    auto biased = [&](int d0, float (&f)[8]) {
       load8_upto(src + d0, width - d0, vec && d0 < width, f);
-      if (bs) {
+      if (!bs) return;
+      if (vec && d0 < width) {
+        float g[8];
+        load8(bs + d0, g);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] += g[i];
+      } else {
 #pragma unroll
         for (int i = 0; i < 8; ++i) f[i] += d0 + i < width ? bs[d0 + i] : 0.f;
       }
-      if (!is_v && d0 < dims) {
+    };
+    auto load = [&](int d0, float (&f)[8]) {
+      biased(d0, f);
+      if (is_v || d0 >= dims || !live) return;
+      if (pairs) {
+        const bool low = d0 < half;
+        const int j = low ? d0 : d0 - half;
+        float g[8], cs[8], sn[8];
+        biased(low ? d0 + half : j, g);
+        load8(trig + j, cs);
+        load8(trig + half + j, sn);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = fmaf(f[i], cs[i], low ? -g[i] * sn[i] : g[i] * sn[i]);
+      } else {
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
           const int d = d0 + i;
