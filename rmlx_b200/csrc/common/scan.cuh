@@ -15,6 +15,8 @@
 // four columns; LANES threads share a column and add their parts by a transposing butterfly. Arithmetic on the
 // state runs on pairs (fma.rn.f32x2).
 #pragma once
+#include <type_traits>
+
 #include "launch.cuh"
 #include "rows.cuh"
 
@@ -39,20 +41,46 @@ __device__ __forceinline__ uint64_t scan_mul(uint64_t a, uint64_t b) {
   return d;
 }
 
-constexpr int kScanThreads = 64, kScanCols = 4, kScanStages = 3;       // columns per thread; chunks in flight
-template <int ROWS, int LANES, bool ONE>
+constexpr int kScanCols = 4, kScanStages = 3;       // columns per thread; chunks in flight
+// TH threads a block: more of them share the row records a block fetches (which L2 bandwidth bounds when every block
+// of 64 fetches its own: GLA with 512 blocks at 3.9 TB/s), fewer spread a small problem over more SMs.
+template <int ROWS, int LANES, bool ONE, int TH>
 struct ScanCfg {
   static constexpr int kRows = ROWS * LANES;                     // padded rows of the state
-  static constexpr int kCols = kScanThreads / LANES * kScanCols; // columns per block
+  static constexpr int kCols = TH / LANES * kScanCols;           // columns per block
   static constexpr int kChunk = kRows > 128 ? 8 : 16;            // tokens per chunk
   static constexpr int kRec = (ONE ? 2 : 3) * kRows;             // floats of a row record
   static constexpr int kCol = kCols + 4;                         // floats of a column record: v | own, or x | decay, dt, own
   static constexpr int kStage = kChunk * (kRec + kCol);
   static constexpr int kSmem = kScanStages * kStage * 4 + 64;
   static constexpr int blocks(int d) { return (d + kCols - 1) / kCols; }
-  // Floats of the records of one token and head (ONE: `per` heads share a row record).
-  static constexpr long long row_floats(int d, int per) { return (kRec + per - 1) / per + (long long)(blocks(d)) * kCol; }
 };
+
+// Columns per block, as a power of two: what a column record's layout depends on.
+inline int scan_col_shift(int lanes, int threads) {
+  int s = 0;
+  while ((1 << s) < threads / lanes * kScanCols) ++s;
+  return s;
+}
+inline int scan_blocks(int d, int shift) { return (d + (1 << shift) - 1) >> shift; }
+// Threads per block: as many as still leave blocks for most SMs.
+inline int scan_threads(int lanes, int d, int H, int n_segs) {
+  int th = 64;
+  while (th < 256 && (1 << scan_col_shift(lanes, 2 * th)) <= (d + 7) / 8 * 8 &&
+         1LL * scan_blocks(d, scan_col_shift(lanes, 2 * th)) * H * n_segs * 10 >= 7LL * sm_count())
+    th *= 2;
+  return th;
+}
+// Floats of the records of one token and head whatever the block size; `per` heads share a row record.
+inline long long scan_row_floats(int rows, int lanes, int parts, int d, int per) {
+  long long widest = 0;
+  for (int th = 64; th <= 256; th *= 2) {
+    const int sh = scan_col_shift(lanes, th);
+    const long long n = 1LL * scan_blocks(d, sh) * ((1 << sh) + 4);
+    widest = n > widest ? n : widest;
+  }
+  return (parts * rows + per - 1) / per + widest;
+}
 
 // Where value i of r, k or w sits in a record: row group g's values four at a time, so that the 16-byte pieces
 // of consecutive groups are neighbours.
@@ -102,16 +130,16 @@ __device__ __forceinline__ void scan_load4(const T* p, int i, int dim, bool vec,
 // per record, four values each per turn.
 template <class IN, int ROWS, int LANES, int LU>
 __global__ void __launch_bounds__(kRowThreads)
-scan_prepare_kernel(IN in, float* __restrict__ rec, float* __restrict__ col, int rows, int H, int d) {
-  using C = ScanCfg<ROWS, LANES, false>;
+scan_prepare_kernel(IN in, float* __restrict__ rec, float* __restrict__ col, int rows, int H, int d, int shift) {
+  constexpr int kRows = ROWS * LANES;
   pdl_launch_dependents();
   pdl_wait();
   const int unit = (blockIdx.x * kRowThreads + threadIdx.x) / LU, lane = threadIdx.x % LU;
   const bool live = unit < rows * H;                 // the lanes of a warp stay together for the sum
   const int t = live ? unit / H : 0, h = live ? unit - t * H : 0;
-  float* out = rec + (size_t(h) * rows + t) * C::kRec;
+  float* out = rec + (size_t(h) * rows + t) * 3 * kRows;
   float own = 0.f;
-  for (int i = lane * 4; i < C::kRows; i += LU * 4) {
+  for (int i = lane * 4; i < kRows; i += LU * 4) {
     float r[4], k[4], w[4], b[4];
     in.rows4(t, h, i, r, k, w, b);
 #pragma unroll
@@ -119,25 +147,26 @@ scan_prepare_kernel(IN in, float* __restrict__ rec, float* __restrict__ col, int
     if (live) {
       float* o = out + scan_at<ROWS, LANES>(i);
       *reinterpret_cast<float4*>(o) = make_float4(r[0], r[1], r[2], r[3]);
-      *reinterpret_cast<float4*>(o + C::kRows) = make_float4(k[0], k[1], k[2], k[3]);
-      *reinterpret_cast<float4*>(o + 2 * C::kRows) = make_float4(w[0], w[1], w[2], w[3]);
+      *reinterpret_cast<float4*>(o + kRows) = make_float4(k[0], k[1], k[2], k[3]);
+      *reinterpret_cast<float4*>(o + 2 * kRows) = make_float4(w[0], w[1], w[2], w[3]);
     }
   }
   own = group_sum<LU>(own);
   if (!live) return;
-  const int nb = C::blocks(d);
-  for (int i = lane * 4; i < nb * C::kCols; i += LU * 4) {
+  const int cols = 1 << shift, nb = (d + cols - 1) >> shift;
+  for (int i = lane * 4; i < nb << shift; i += LU * 4) {
     float v[4];
     in.cols4(t, h, i, v);
-    float* o = col + ((size_t(h) * nb + i / C::kCols) * rows + t) * C::kCol + i % C::kCols;
+    const int at = i & (cols - 1);
+    float* o = col + ((size_t(h) * nb + (i >> shift)) * rows + t) * (cols + 4) + at;
     *reinterpret_cast<float4*>(o) = make_float4(v[0], v[1], v[2], v[3]);
-    if (i % C::kCols == 0) *reinterpret_cast<float4*>(o + C::kCols) = make_float4(own, 0.f, 0.f, 0.f);
+    if (at == 0) *reinterpret_cast<float4*>(o + cols) = make_float4(own, 0.f, 0.f, 0.f);
   }
 }
 
-template <int ROWS, int LANES, bool ONE>
-__global__ void __launch_bounds__(kScanThreads) scan_kernel(ScanParams p) {
-  using C = ScanCfg<ROWS, LANES, ONE>;
+template <int ROWS, int LANES, bool ONE, int TH>
+__global__ void __launch_bounds__(TH) scan_kernel(ScanParams p) {
+  using C = ScanCfg<ROWS, LANES, ONE, TH>;
   extern __shared__ __align__(128) float smem[];
   uint64_t* full = reinterpret_cast<uint64_t*>(smem + kScanStages * C::kStage);      // [stages]
   __shared__ uint32_t gave_up;
@@ -307,31 +336,37 @@ __global__ void __launch_bounds__(kScanThreads) scan_kernel(ScanParams p) {
   if (p.prev && blockIdx.x == 0 && h == 0) {
     const float* last = p.x + size_t(row0 + len - 1) * p.ldx;
     float* keep = p.prev + size_t(slot) * p.stride;
-    for (int i = threadIdx.x; i < p.ldx; i += kScanThreads) keep[i] = last[i];
+    for (int i = threadIdx.x; i < p.ldx; i += TH) keep[i] = last[i];
   }
 }
 
-// The scan over records that are in place; `p.rec` and `p.col` follow each other.
+// The scan over records that are in place, made for column blocks of th threads.
 template <int ROWS, int LANES, bool ONE>
-static int launch_scan(const ScanParams& p, int n_segs, int pdl, cudaStream_t st) {
-  using C = ScanCfg<ROWS, LANES, ONE>;
-  auto kern = scan_kernel<ROWS, LANES, ONE>;
-  RB_CHECK(set_max_smem(kern, C::kSmem));
-  return launch(kern, dim3(C::blocks(p.d), p.H, n_segs), dim3(kScanThreads), C::kSmem, st, pdl != 0, p);
+static int launch_scan(const ScanParams& p, int th, int n_segs, int pdl, cudaStream_t st) {
+  auto go = [&](auto threads) -> int {
+    constexpr int TH = decltype(threads)::value;
+    using C = ScanCfg<ROWS, LANES, ONE, TH>;
+    auto kern = scan_kernel<ROWS, LANES, ONE, TH>;
+    RB_CHECK(set_max_smem(kern, C::kSmem));
+    return launch(kern, dim3((p.d + C::kCols - 1) / C::kCols, p.H, n_segs), dim3(TH), C::kSmem, st, pdl != 0, p);
+  };
+  if (th == 256) return go(std::integral_constant<int, 256>{});
+  if (th == 128) return go(std::integral_constant<int, 128>{});
+  return go(std::integral_constant<int, 64>{});
 }
 // Records and scan of heads with a decay per row. rec: scratch, 16-byte aligned.
 template <class IN, int ROWS, int LANES>
 static int launch_row_scan(const IN& in, ScanParams p, float* rec, int n_segs, int pdl, cudaStream_t st) {
-  using C = ScanCfg<ROWS, LANES, false>;
-  constexpr int LU = C::kRows >= 128 ? 32 : C::kRows / 4;
+  constexpr int kRows = ROWS * LANES, LU = kRows >= 128 ? 32 : kRows / 4;
   const long long threads = 1LL * p.rows * p.H * LU;
   if (threads > 0x7fffffffLL) return -2;
-  float* col = rec + size_t(p.H) * p.rows * C::kRec;
+  const int th = scan_threads(LANES, p.d, p.H, n_segs);
+  float* col = rec + size_t(p.H) * p.rows * 3 * kRows;
   const int rc = launch(scan_prepare_kernel<IN, ROWS, LANES, LU>, dim3(unsigned((threads + kRowThreads - 1) / kRowThreads)),
-                        dim3(kRowThreads), 0, st, pdl != 0, in, rec, col, p.rows, p.H, p.d);
+                        dim3(kRowThreads), 0, st, pdl != 0, in, rec, col, p.rows, p.H, p.d, scan_col_shift(LANES, th));
   if (rc) return rc;
   p.rec = rec; p.col = col; p.per = 1;
-  return launch_scan<ROWS, LANES, false>(p, n_segs, pdl, st);
+  return launch_scan<ROWS, LANES, false>(p, th, n_segs, pdl, st);
 }
 
 constexpr int kScanMaxRows = 256;

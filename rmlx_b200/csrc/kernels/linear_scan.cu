@@ -60,72 +60,106 @@ struct SsdIn {
   int each_row;             // no two rows share a sequence
   const float* dt_bias; const float* a_log; const float* skip;      // [H]
   int H, G, n, d;
-  __device__ __forceinline__ int channels() const { return H * d + 2 * G * n; }
+  __host__ __device__ __forceinline__ int channels() const { return H * d + 2 * G * n; }
 };
 
-// How many of the rows before t belong to its sequence (at most taps - 1).
-template <class T>
-__device__ __forceinline__ int ssd_back(const SsdIn<T>& in, int t) {
-  int back = 0;
-  if (!in.each_row)
-    while (back < in.taps - 1 && t - back - 1 >= 0 && in.slots[t - back - 1] == in.slots[t]) ++back;
-  return back;
-}
-// Convolution and activation of channel c for token t.
-template <class T>
-__device__ __forceinline__ float ssd_conv(const SsdIn<T>& in, int t, int c, int back) {
-  const int ch = in.channels();
-  const float* st = in.before + size_t(in.slots[t]) * in.stride;
-  float a = in.conv_b[c];
-  for (int j = in.taps - 1; j >= 0; --j) {           // j tokens back
-    const float x = j <= back ? to_f32(in.raw[size_t(t - j) * in.ld + in.x_at + c]) : st[size_t(in.taps - 1 - (j - back)) * ch + c];
-    a = fmaf(in.conv_w[size_t(in.taps - 1 - j) * ch + c], x, a);
-  }
-  return silu_f(a);
+// Two consecutive inputs, 4- or 8-byte aligned.
+__device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 load2(const __nv_bfloat16* p) {
+  const uint32_t v = *reinterpret_cast<const uint32_t*>(p);
+  return make_float2(bf16lo(v), bf16hi(v));
 }
 
-// One block per token: all channels' convolutions, then the records.
-template <class T, int ROWS, int LANES>
+// All channels' convolutions and the step sizes of a block's TOKENS tokens into shared memory, then the records. Where the
+// block and the taps before it lie in one sequence, a thread asks for a pair of channels' inputs of all tokens at once
+// (TAPS 0, or elsewhere: one by one).
+template <class T, int ROWS, int LANES, int TAPS, int TOKENS>
 __global__ void __launch_bounds__(kRowThreads)
-ssd_prepare_kernel(SsdIn<T> in, float* __restrict__ rec, float* __restrict__ col, int rows) {
-  using C = ScanCfg<ROWS, LANES, true>;
+ssd_prepare_kernel(SsdIn<T> in, float* __restrict__ rec, float* __restrict__ col, int rows, int shift) {
+  constexpr int kRows = ROWS * LANES, tokens = TOKENS;
   extern __shared__ __align__(16) float sm[];
-  const int t = blockIdx.x, inner = in.H * in.d, gn = in.G * in.n, ch = inner + 2 * gn;
-  float* s_own = sm + ch;            // [G] C . B
-  float* s_dt = s_own + in.G;        // [H]
-  float* s_a = s_dt + in.H;          // [H]
+  const int t0 = blockIdx.x * tokens, nt = min(tokens, rows - t0), inner = in.H * in.d, gn = in.G * in.n, ch = inner + 2 * gn;
+  const int taps = in.taps;
+  float* s_own = sm + tokens * ch;         // [tokens, G] C . B
+  float* s_dt = s_own + tokens * in.G;     // [tokens, H]
+  float* s_a = s_dt + tokens * in.H;       // [tokens, H]
   pdl_launch_dependents();
   pdl_wait();
-  const int back = ssd_back(in, t);
-  for (int c = threadIdx.x; c < ch; c += kRowThreads) sm[c] = ssd_conv(in, t, c, back);
-  for (int h = threadIdx.x; h < in.H; h += kRowThreads) {
-    const float dt = softplus_f(to_f32(in.raw[size_t(t) * in.ld + in.dt_at + h]) + in.dt_bias[h]);
-    s_dt[h] = dt;
-    s_a[h] = expf(-expf(in.a_log[h]) * dt);
+  const bool inside = TAPS > 0 && !in.each_row && nt == tokens && t0 >= TAPS - 1 &&
+                      in.slots[t0 - (TAPS > 0 ? TAPS - 1 : 0)] == in.slots[t0 + tokens - 1] && ((ch | in.ld | in.x_at) & 1) == 0;
+  if (inside) {
+    constexpr int W = TAPS > 0 ? TAPS : 1;
+    const T* base = in.raw + size_t(t0 - (W - 1)) * in.ld + in.x_at;
+    for (int c = threadIdx.x * 2; c < ch; c += kRowThreads * 2) {
+      float2 x[tokens + W - 1], w[W];
+#pragma unroll
+      for (int i = 0; i < tokens + W - 1; ++i) x[i] = load2(base + size_t(i) * in.ld + c);
+#pragma unroll
+      for (int j = 0; j < W; ++j) w[j] = load2(in.conv_w + size_t(j) * ch + c);
+      const float2 bias = load2(in.conv_b + c);
+#pragma unroll
+      for (int i = 0; i < tokens; ++i) {
+        float2 a = bias;
+#pragma unroll
+        for (int j = 0; j < W; ++j) { a.x = fmaf(w[j].x, x[i + j].x, a.x); a.y = fmaf(w[j].y, x[i + j].y, a.y); }
+        *reinterpret_cast<float2*>(sm + i * ch + c) = make_float2(silu_f(a.x), silu_f(a.y));
+      }
+    }
+  } else {
+    for (int i = 0; i < nt; ++i) {
+      const int t = t0 + i;
+      int back = 0;                        // how many of the rows before t are its sequence's (at most taps - 1)
+      if (!in.each_row)
+        while (back < taps - 1 && t - back - 1 >= 0 && in.slots[t - back - 1] == in.slots[t]) ++back;
+      const float* before = in.before + size_t(in.slots[t]) * in.stride;
+      for (int c = threadIdx.x; c < ch; c += kRowThreads) {
+        float a = in.conv_b[c];
+        for (int j = taps - 1; j >= 0; --j) {              // j tokens back
+          const float x = j <= back ? to_f32(in.raw[size_t(t - j) * in.ld + in.x_at + c]) : before[size_t(taps - 1 - (j - back)) * ch + c];
+          a = fmaf(in.conv_w[size_t(taps - 1 - j) * ch + c], x, a);
+        }
+        sm[i * ch + c] = silu_f(a);
+      }
+    }
+  }
+  for (int u = threadIdx.x; u < nt * in.H; u += kRowThreads) {
+    const int i = u / in.H, h = u - i * in.H;
+    const float dt = softplus_f(to_f32(in.raw[size_t(t0 + i) * in.ld + in.dt_at + h]) + in.dt_bias[h]);
+    s_dt[u] = dt;
+    s_a[u] = expf(-expf(in.a_log[h]) * dt);
   }
   __syncthreads();
-  const float* sB = sm + inner;
-  const float* sC = sB + gn;
-  for (int g = threadIdx.x >> 5; g < in.G; g += kRowThreads / 32) {
+  for (int u = threadIdx.x >> 5; u < nt * in.G; u += kRowThreads / 32) {
+    const int i = u / in.G, g = u - i * in.G;
+    const float* B = sm + i * ch + inner + g * in.n;
     float s = 0.f;
-    for (int i = threadIdx.x & 31; i < in.n; i += 32) s = fmaf(sB[g * in.n + i], sC[g * in.n + i], s);
+    for (int j = threadIdx.x & 31; j < in.n; j += 32) s = fmaf(B[j], B[gn + j], s);
     s = warp_sum(s);
-    if ((threadIdx.x & 31) == 0) s_own[g] = s;
+    if ((threadIdx.x & 31) == 0) s_own[u] = s;
   }
-  for (int u = threadIdx.x; u < in.G * C::kRows; u += kRowThreads) {
-    const int g = u / C::kRows, i = u - g * C::kRows;
-    float* o = rec + (size_t(g) * rows + t) * C::kRec + scan_at<ROWS, LANES>(i);
-    o[0] = i < in.n ? sC[g * in.n + i] : 0.f;
-    o[C::kRows] = i < in.n ? sB[g * in.n + i] : 0.f;
+  for (int u = threadIdx.x; u < nt * in.G * kRows; u += kRowThreads) {
+    const int q = u / kRows, j = u - q * kRows, i = q / in.G, g = q - i * in.G;
+    const float* B = sm + i * ch + inner + g * in.n;
+    float* o = rec + (size_t(g) * rows + t0 + i) * (2 * kRows) + scan_at<ROWS, LANES>(j);
+    o[0] = j < in.n ? B[gn + j] : 0.f;
+    o[kRows] = j < in.n ? B[j] : 0.f;
   }
   __syncthreads();
-  const int nb = C::blocks(in.d), per = in.H / in.G, width = nb * C::kCols;
-  for (int u = threadIdx.x; u < in.H * width; u += kRowThreads) {
-    const int h = u / width, i = u - h * width;
-    float* o = col + ((size_t(h) * nb + i / C::kCols) * rows + t) * C::kCol;
-    o[i % C::kCols] = i < in.d ? sm[h * in.d + i] : 0.f;
-    if (i % C::kCols == 0)
-      *reinterpret_cast<float4*>(o + C::kCols) = make_float4(s_a[h], s_dt[h], fmaf(s_own[h / per], s_dt[h], in.skip[h]), 0.f);
+  // column records of a block's tokens are neighbours: four values a thread, tokens before column blocks
+  const int cols = 1 << shift, nb = (in.d + cols - 1) >> shift, per = in.H / in.G, quads = (cols + 4) >> 2;
+  for (int u = threadIdx.x; u < in.H * nb * tokens * quads; u += kRowThreads) {
+    const int v = u / quads, q = u - v * quads, i = v % tokens, hb = v / tokens, h = nb == 1 ? hb : hb / nb;
+    const int c0 = ((hb - h * nb) << shift) + q * 4;
+    if (i >= nt) continue;
+    float4 f;
+    if (q == quads - 1) {
+      const float dt = s_dt[i * in.H + h];
+      f = make_float4(s_a[i * in.H + h], dt, fmaf(s_own[i * in.G + h / per], dt, in.skip[h]), 0.f);
+    } else {
+      const float* x = sm + i * ch + h * in.d + c0;
+      f = make_float4(c0 < in.d ? x[0] : 0.f, c0 + 1 < in.d ? x[1] : 0.f, c0 + 2 < in.d ? x[2] : 0.f, c0 + 3 < in.d ? x[3] : 0.f);
+    }
+    *reinterpret_cast<float4*>(col + (size_t(hb) * rows + t0 + i) * (cols + 4) + q * 4) = f;
   }
 }
 
@@ -237,16 +271,23 @@ static int run_gla(const GlaIn<T>& in, const ScanParams& p, float* rec, int n, i
 
 template <class T, int ROWS, int LANES>
 static int launch_ssd(const SsdIn<T>& in, ScanParams p, float* rec, int n_segs, int pdl, cudaStream_t st) {
-  using C = ScanCfg<ROWS, LANES, true>;
-  const size_t smem = size_t(in.H * in.d + 2 * in.G * in.n + in.G + 2 * in.H) * sizeof(float);
-  if (smem > 200 * 1024) return -2;
-  auto kern = ssd_prepare_kernel<T, ROWS, LANES>;
-  RB_CHECK(set_max_smem(kern, smem));
-  float* col = rec + size_t(in.G) * p.rows * C::kRec;
-  int rc = launch(kern, dim3(p.rows), dim3(kRowThreads), smem, st, pdl != 0, in, rec, col, p.rows);
+  const size_t per_token = size_t(in.channels() + in.G + 2 * in.H) * sizeof(float);
+  if (per_token > 200 * 1024) return -2;
+  const int th = scan_threads(LANES, p.d, p.H, n_segs);
+  float* col = rec + size_t(in.G) * p.rows * 2 * ROWS * LANES;
+  auto prepare = [&](auto kern, int tokens) -> int {
+    const size_t smem = per_token * tokens;
+    RB_CHECK(set_max_smem(kern, smem));
+    return launch(kern, dim3((p.rows + tokens - 1) / tokens), dim3(kRowThreads), smem, st, pdl != 0, in, rec, col, p.rows,
+                  scan_col_shift(LANES, th));
+  };
+  const bool one = per_token * 4 > 200 * 1024;
+  const int rc = one ? prepare(ssd_prepare_kernel<T, ROWS, LANES, 0, 1>, 1)
+                     : in.taps == 4 ? prepare(ssd_prepare_kernel<T, ROWS, LANES, 4, 4>, 4)
+                                    : prepare(ssd_prepare_kernel<T, ROWS, LANES, 0, 4>, 4);
   if (rc) return rc;
   p.rec = rec; p.col = col; p.per = in.H / in.G;
-  return launch_scan<ROWS, LANES, true>(p, n_segs, pdl, st);
+  return launch_scan<ROWS, LANES, true>(p, th, n_segs, pdl, st);
 }
 template <class T>
 static int run_ssd(const SsdIn<T>& in, const ScanParams& p, float* rec, int n, int pdl, cudaStream_t st) {
@@ -270,7 +311,7 @@ extern "C" int rmlx_scan_max_rows() { return kScanMaxRows; }
 // their row record.
 extern "C" long long rmlx_scan_record(int n, int d, int one, int per) {
   if (per < 1) return 0;
-#define RB_REC(R_, L_) return one ? ScanCfg<R_, L_, true>::row_floats(d, per) : ScanCfg<R_, L_, false>::row_floats(d, 1)
+#define RB_REC(R_, L_) return scan_row_floats((R_) * (L_), L_, one ? 2 : 3, d, one ? per : 1)
   RB_SCAN_DISPATCH(n, RB_REC);
 #undef RB_REC
   return 0;

@@ -120,7 +120,7 @@ using namespace rb;
 extern "C" int rmlx_wkv_max_dim() { return kScanMaxRows; }
 // Floats of the scratch records of one (token, head).
 extern "C" int rmlx_wkv_record(int dim) {
-#define RB_WKV(R_, L_) return int(ScanCfg<R_, L_, false>::row_floats(dim, 1))
+#define RB_WKV(R_, L_) return int(scan_row_floats((R_) * (L_), L_, 3, dim, 1))
   RB_SCAN_DISPATCH(dim, RB_WKV);
 #undef RB_WKV
   return 0;
