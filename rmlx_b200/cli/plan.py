@@ -224,37 +224,34 @@ def plan_posudra(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, bud
     }
 
 
-def plan_rodapel(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, budget_fraction: float = 0.90,
-                 cfg=None) -> dict:
-    """A Rodapel model (bf16, one GPU): pages for its attention layers, recurrent state per sequence for its
-    WKV layers, the widest activations of a prompt chunk (with expanded keys and values of ``ctx`` tokens)."""
-    from ..config import LatentAttentionSpec, RoutedFfSpec, WkvSpec
-    from ..models.rodapel import kv_shapes, rodapel_4096, state_shapes, tensor_shapes
-    c = cfg or rodapel_4096()
+def _plan_layered(c, shapes: dict, kv_shapes, state_shapes, row: int, batch: int, ctx: int, prefill_chunk: int,
+                  budget_fraction: float) -> dict:
+    """A model with a layer list of its own (bf16, one GPU): ``shapes`` its checkpoint tensors, ``row`` activation bytes
+    per prompt token beside the expanded latents."""
+    from ..config import LatentAttentionSpec
     parts = {"attention": 0, "feed_forward": 0, "norms": 0, "embedding": 0, "lm_head": 0}
     routed, active = 0, 0
-    for name, shape in tensor_shapes(c).items():
+    for name, shape in shapes.items():
         n = math.prod(shape)
         part = {"embed": "embedding", "head": "lm_head"}.get(name) or (
             "norms" if len(shape) == 1 else "feed_forward" if ".mlp." in name else "attention")
         parts[part] += n * (4 if len(shape) == 1 else 2)               # per-channel vectors are kept in fp32
         routed += n * 2 if ".mlp.e" in name else 0
     for l in c.layers:
-        if isinstance(l.mlp, RoutedFfSpec):
+        if hasattr(l.mlp, "top"):
             active += min(l.mlp.experts, batch * l.mlp.top) * 3 * l.mlp.ff * c.width * 2
     parts["total"] = sum(parts.values())
-    kv_tok = sum(s[0] * (s[1] + s[2]) * 2 for s in kv_shapes(c) if s is not None)
-    state = sum(4 * math.prod(shape) for p in state_shapes(c) if p for shape in p.values())
+    head = parts["lm_head"] or parts["embedding"]                      # a step reads the table once as the LM head
+    kv_tok = sum(s[0] * (s[1] + s[2]) * 2 for s in kv_shapes if s is not None)
+    state = sum(4 * math.prod(shape) for p in state_shapes if p for shape in p.values())
     lat = [l.mixer for l in c.layers if isinstance(l.mixer, LatentAttentionSpec)]
-    row = 10 * c.width + max([0] + [12 * l.mixer.heads * l.mixer.dim + 10 * c.width for l in c.layers
-                                    if isinstance(l.mixer, WkvSpec)]) + \
-        max([0] + [l.mlp.top * 2 * (2 * c.width + l.mlp.ff) if isinstance(l.mlp, RoutedFfSpec) else 2 * l.mlp.ff
-                   for l in c.layers if l.mlp is not None])
+    row += max([0] + [l.mlp.top * 2 * (2 * c.width + l.mlp.ff) if hasattr(l.mlp, "top") else 2 * l.mlp.ff
+                      for l in c.layers if l.mlp is not None])
     scratch = prefill_chunk * row + ctx * max([0] + [2 * (m.heads * (m.dim + m.vdim) + m.kv_rank) for m in lat])
     budget, need = int(HBM_BYTES * budget_fraction), batch * (ctx * kv_tok + state)
-    step = parts["attention"] + parts["feed_forward"] - routed + active + need + parts["lm_head"]
+    step = parts["attention"] + parts["feed_forward"] - routed + active + need + head
     hbm = decode_hbm_gbs()
-    layer = (step - parts["lm_head"]) / c.num_layers
+    layer = (step - head) / c.num_layers
     return {
         "model": c.name, "weights": "bf16", "tp": 1, "expert_parallel": False, "batch": batch, "ctx": ctx,
         "kv_quant": "bf16", "weight_bytes_per_gpu": parts, "kv_bytes_per_token_per_gpu": kv_tok,
@@ -266,6 +263,38 @@ def plan_rodapel(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, bud
                             "tokens_per_s": batch * hbm * 1e9 / step, "hbm_gbs": hbm},
         "decode_stream_plans": {},
     }
+
+
+def plan_rodapel(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, budget_fraction: float = 0.90,
+                 cfg=None) -> dict:
+    """A Rodapel model (bf16, one GPU): pages for its attention layers, recurrent state per sequence for its
+    WKV layers, the widest activations of a prompt chunk (with expanded keys and values of ``ctx`` tokens)."""
+    from ..config import WkvSpec
+    from ..models.rodapel import kv_shapes, rodapel_4096, state_shapes, tensor_shapes
+    c = cfg or rodapel_4096()
+    row = 10 * c.width + max([0] + [12 * l.mixer.heads * l.mixer.dim + 10 * c.width for l in c.layers
+                                    if isinstance(l.mixer, WkvSpec)])
+    return _plan_layered(c, tensor_shapes(c), kv_shapes(c), state_shapes(c), row, batch, ctx, prefill_chunk, budget_fraction)
+
+
+def plan_nugosun(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, budget_fraction: float = 0.90,
+                 cfg=None) -> dict:
+    """A Nugosun model (bf16, one GPU): pages for the attention layers with rows of their own, the recurrent layers'
+    states per sequence, the widest activations of a prompt chunk (with the recurrences' records)."""
+    from ..config import GlaSpec, PairSpec
+    from ..models.nugosun import kv_shapes, nugosun_4096, state_shapes, tensor_shapes
+    c = cfg or nugosun_4096()
+
+    def mixer(m) -> int:
+        if isinstance(m, GlaSpec):         # projection, decay, fp32 output, records
+            return m.heads * (2 * (2 * m.dim + 2 * m.vdim) + 4 * m.dim + 6 * m.vdim + 4 * (3 * max(16, m.dim) + 2 * m.vdim))
+        if isinstance(m, PairSpec):
+            a, r = m.left, m.right
+            return 2 * (2 * a.heads * a.dim + 2 * a.kv_heads * a.dim + a.heads * a.vdim + r.channels + r.inner) + 14 * r.inner
+        return 2 * (m.q_rank + m.kv_rank + m.heads * (2 * (m.dim + m.rot_dim) + m.vdim))
+
+    row = 8 * c.width + max(mixer(l.mixer) for l in c.layers)
+    return _plan_layered(c, tensor_shapes(c), kv_shapes(c), state_shapes(c), row, batch, ctx, prefill_chunk, budget_fraction)
 
 
 def plan(model: str = "moe-a22b", weights: str = "q4", tp: int = 1, batch: int = 1, ctx: int = 4096,
@@ -281,6 +310,10 @@ def plan(model: str = "moe-a22b", weights: str = "q4", tp: int = 1, batch: int =
         if weights != "bf16" or tp != 1 or kv_quant is not None:
             raise ValueError("Rodapel runs on one GPU with bf16 weights and cache")
         return plan_rodapel(batch, ctx, prefill_chunk, budget_fraction)
+    if model == "nugosun-4096" and cfg is None:
+        if weights != "bf16" or tp != 1 or kv_quant is not None:
+            raise ValueError("Nugosun runs on one GPU with bf16 weights and cache")
+        return plan_nugosun(batch, ctx, prefill_chunk, budget_fraction)
     cfg = cfg or presets()[model]
     w = weight_bytes_per_gpu(cfg, weights, tp, expert_parallel)
     kv_tok = kv_bytes_per_token_per_gpu(cfg, tp, kv_quant)
@@ -344,7 +377,7 @@ def render(p: dict) -> str:
 
 def main(argv: Optional[Sequence[str]] = None) -> int:
     ap = argparse.ArgumentParser(prog="rmlx plan", description=__doc__.split("\n\n")[0])
-    ap.add_argument("--model", default="moe-a22b", choices=sorted(presets()) + ["deepseek-v3", "posudra-8b", "rodapel-4096"])
+    ap.add_argument("--model", default="moe-a22b", choices=sorted(presets()) + ["deepseek-v3", "posudra-8b", "rodapel-4096", "nugosun-4096"])
     ap.add_argument("--weights", default="q4", choices=sorted(BITS))
     ap.add_argument("--tp", type=int, default=1)
     ap.add_argument("--expert-parallel", action="store_true")
