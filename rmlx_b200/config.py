@@ -602,7 +602,7 @@ class ChosenFfSpec:
     identity = 0
 
     def validate(self) -> "ChosenFfSpec":
-        _require(0 < self.experts <= 512 and self.ff > 0, "experts: 1 to 512, ff positive")
+        _require(0 < self.experts <= 256 and self.ff > 0, "experts: 1 to 256, ff positive")
         _require(1 <= self.top <= min(32, self.experts), "top must be in [1, 32] and <= experts")
         return self
 
