@@ -52,6 +52,13 @@ __device__ __forceinline__ void load8_upto(const T* p, int n, bool aligned, floa
   for (int i = 0; i < 8; ++i) f[i] = i < n ? to_f32(p[i]) : 0.f;
 }
 
+// sin and cos of pos * freq radians: the product in double, whole turns taken off there, so that a far position costs
+// no accuracy (and no branch).
+__device__ __forceinline__ void rotary_sincos(int pos, float freq, float& s, float& c) {
+  const double turns = double(pos) * double(freq) * 0.15915494309189535;
+  sincospif(2.f * float(turns - rint(turns)), &s, &c);
+}
+
 // Sum over groups of L consecutive lanes (L a power of two).
 template <int L>
 __device__ __forceinline__ float group_sum(float v) {

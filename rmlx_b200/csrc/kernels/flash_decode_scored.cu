@@ -16,6 +16,7 @@
 // Rows in shared memory are padded to the class width (64 or 128) with zeros; global memory holds
 // dkp / dvp elements per row (multiples of eight), so narrow heads cost no extra bytes.
 #include "../common/launch.cuh"
+#include "../common/rows.cuh"
 #include "../common/score_mod.cuh"
 
 namespace rb {
@@ -175,31 +176,36 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
         cs[i] = 1.f; sn[i] = 0.f; other[i] = d;
         if (d < p.rot_dims) {
           float sv, cv;
-          sincosf(float(len - 1) * p.inv_freq[d < half ? d : d - half], &sv, &cv);
+          rotary_sincos(len - 1, p.inv_freq[d < half ? d : d - half], sv, cv);
           cs[i] = cv * p.grow;
           sn[i] = (d < half ? -sv : sv) * p.grow;
           other[i] = d < half ? d + half : d - half;
         }
       }
+      const bool rot = p.rot_dims > 0;
       auto load_head = [&](int at, bool live, float (&v)[PL], float (&u)[PL]) {
 #pragma unroll
-        for (int i = 0; i < PL; ++i) {
-          const bool in = live && i * 32 + lane < p.dim;
-          v[i] = in ? __ldcg(row + at + i * 32 + lane) : 0.f;
-          u[i] = (in && i * 32 + lane < p.rot_dims) ? __ldcg(row + at + other[i]) : 0.f;
-          if (p.bias && in) {
-            v[i] += p.bias[at + i * 32 + lane];
-            if (i * 32 + lane < p.rot_dims) u[i] += p.bias[at + other[i]];
+        for (int i = 0; i < PL; ++i) v[i] = (live && i * 32 + lane < p.dim) ? __ldcg(row + at + i * 32 + lane) : 0.f;
+        if (rot) {
+#pragma unroll
+          for (int i = 0; i < PL; ++i) u[i] = (live && i * 32 + lane < p.rot_dims) ? __ldcg(row + at + other[i]) : 0.f;
+        }
+        if (p.bias && live) {
+#pragma unroll
+          for (int i = 0; i < PL; ++i) {
+            if (i * 32 + lane < p.dim) v[i] += p.bias[at + i * 32 + lane];
+            if (rot && i * 32 + lane < p.rot_dims) u[i] += p.bias[at + other[i]];
           }
         }
       };
       auto turn = [&](float (&v)[PL], const float (&u)[PL]) {     // returns 1 / rms
+        if (rot) {
+#pragma unroll
+          for (int i = 0; i < PL; ++i) v[i] = fmaf(v[i], cs[i], u[i] * sn[i]);
+        }
         float ss = 0.f;
 #pragma unroll
-        for (int i = 0; i < PL; ++i) {
-          v[i] = fmaf(v[i], cs[i], u[i] * sn[i]);
-          ss += v[i] * v[i];
-        }
+        for (int i = 0; i < PL; ++i) ss += v[i] * v[i];
         return 1.f / sqrtf(warp_sum(ss) / float(p.dim) + p.eps);
       };
       float v[4][PL], u[4][PL];

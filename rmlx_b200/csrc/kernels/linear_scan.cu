@@ -187,10 +187,16 @@ conv_carry_kernel(const T* __restrict__ raw, int ld, int x_at, float* __restrict
   }
 }
 
+// silu of an output gate; with the hardware exponential and division where the result is rounded to bf16.
+template <class T>
+__device__ __forceinline__ float gate_silu(float z) {
+  return sizeof(T) == 2 ? __fdividef(z, 1.f + __expf(fminf(-z, 80.f))) : silu_f(z);
+}
+
 // out[t, c] over equal groups of columns: FIRST: f = o silu(gate), f / rms(f over the group) * w;
 // else o / rms(o over the group) * w * silu(gate). L lanes (256: a block) per (row, group), KEEP chunks of eight a lane
-// keeps; what is left is read again.
-template <class T, int L, int KEEP, bool FIRST>
+// keeps; what is left is read again. VEC: sizes and strides are multiples of eight.
+template <class T, int L, int KEEP, bool FIRST, bool VEC>
 __global__ void __launch_bounds__(kRowThreads)
 gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ gate, int ld_g, const float* __restrict__ w,
                   float eps, T* __restrict__ out, int ld_out, int rows, int groups, int size) {
@@ -200,17 +206,25 @@ gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ g
   const int unit = (blockIdx.x * kRowThreads + threadIdx.x) / L, lane = threadIdx.x % L;
   const bool live = unit < rows * groups;              // the lanes of a warp stay together for the sums
   const int t = live ? unit / groups : 0, at = live ? (unit - t * groups) * size : 0;
-  const bool vec = size % 8 == 0 && ld_o % 8 == 0 && ld_g % 8 == 0 && ld_out % 8 == 0;
   const float* op = o + size_t(t) * ld_o + at;
   const T* gp = gate + size_t(t) * ld_g + at;
-  float f[KEEP][8], ssq = 0.f;
+  float f[KEEP][8], g[KEEP][8], ssq = 0.f;
   auto load = [&](int i0, float (&a)[8]) {
-    load8_upto(op + i0, size - i0, vec, a);
+    load8_upto(op + i0, size - i0, VEC, a);
     if (FIRST) {
       float z[8];
-      load8_upto(gp + i0, size - i0, vec, z);
+      load8_upto(gp + i0, size - i0, VEC, z);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) a[i] *= silu_f(z[i]);
+      for (int i = 0; i < 8; ++i) a[i] *= gate_silu<T>(z[i]);
+    }
+  };
+  auto factor = [&](int i0, float (&a)[8]) {           // what the normed values are multiplied by
+    load8_upto(w + at + i0, size - i0, VEC, a);
+    if (!FIRST) {
+      float z[8];
+      load8_upto(gp + i0, size - i0, VEC, z);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) a[i] *= gate_silu<T>(z[i]);
     }
   };
 #pragma unroll
@@ -218,6 +232,7 @@ gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ g
     const int i0 = (u * L + lane) * 8;
     if (i0 < size) {
       load(i0, f[u]);
+      factor(i0, g[u]);
 #pragma unroll
       for (int i = 0; i < 8; ++i) ssq += f[u][i] * f[u][i];
     }
@@ -233,17 +248,10 @@ gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ g
   if (!live) return;
   const float inv = 1.f / sqrtf(ssq / float(size) + eps);
   T* dst = out + size_t(t) * ld_out + at;
-  auto put = [&](int i0, float (&a)[8]) {
-    float g[8];
-    load8_upto(w + at + i0, size - i0, vec, g);
+  auto put = [&](int i0, float (&a)[8], const float (&m)[8]) {
 #pragma unroll
-    for (int i = 0; i < 8; ++i) a[i] *= inv * g[i];
-    if (!FIRST) {
-      load8_upto(gp + i0, size - i0, vec, g);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) a[i] *= silu_f(g[i]);
-    }
-    if (vec) {
+    for (int i = 0; i < 8; ++i) a[i] *= inv * m[i];
+    if (VEC) {
       store8(dst + i0, a);
     } else {
       for (int i = 0; i < 8 && i0 + i < size; ++i) dst[i0 + i] = from_f32<T>(a[i]);
@@ -252,12 +260,13 @@ gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ g
 #pragma unroll
   for (int u = 0; u < KEEP; ++u) {
     const int i0 = (u * L + lane) * 8;
-    if (i0 < size) put(i0, f[u]);
+    if (i0 < size) put(i0, f[u], g[u]);
   }
   for (int i0 = (KEEP * L + lane) * 8; i0 < size; i0 += L * 8) {
-    float a[8];
+    float a[8], m[8];
     load(i0, a);
-    put(i0, a);
+    factor(i0, m);
+    put(i0, a, m);
   }
 }
 
@@ -376,20 +385,30 @@ extern "C" int rmlx_gated_norm(const float* o, int ld_o, const void* gate, int l
   const long long units = 1LL * rows * groups, blocks = (units * lanes + kRowThreads - 1) / kRowThreads;
   if (units * lanes > 0x7fffffffLL) return -2;
   const dim3 grid{unsigned(blocks)};
-#define RB_GN(T_, L_, K_, F_)                                                                                          \
-  return launch(gated_norm_kernel<T_, L_, K_, F_>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o,                  \
+  const bool vec = size % 8 == 0 && ld_o % 8 == 0 && ld_g % 8 == 0 && ld_out % 8 == 0 &&
+                   !((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out) |
+                      reinterpret_cast<uintptr_t>(w)) & 15);
+#define RB_GN(T_, L_, K_, F_, V_)                                                                                      \
+  return launch(gated_norm_kernel<T_, L_, K_, F_, V_>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o,              \
                 static_cast<const T_*>(gate), ld_g, w, eps, static_cast<T_*>(out), ld_out, rows, groups, size)
-#define RB_GNL(T_, F_)                    \
-  {                                       \
-    if (lanes == 8) RB_GN(T_, 8, 1, F_);  \
-    if (lanes == 16) RB_GN(T_, 16, 1, F_); \
-    if (lanes == 32) RB_GN(T_, 32, 1, F_); \
-    RB_GN(T_, 256, 2, F_);                \
+#define RB_GNL(T_, F_, V_)                          \
+  {                                                 \
+    if (lanes == 8) RB_GN(T_, 8, 1, F_, V_);        \
+    if (lanes == 16) RB_GN(T_, 16, 1, F_, V_);      \
+    if (lanes == 32) RB_GN(T_, 32, 1, F_, V_);      \
+    if (size <= 2048) RB_GN(T_, 256, 1, F_, V_);    \
+    RB_GN(T_, 256, 2, F_, V_);                      \
   }
-  if (f32 && gate_first) RB_GNL(float, true)
-  if (f32) RB_GNL(float, false)
-  if (gate_first) RB_GNL(__nv_bfloat16, true)
-  RB_GNL(__nv_bfloat16, false)
+#define RB_GNV(T_)                                    \
+  {                                                   \
+    if (gate_first && vec) RB_GNL(T_, true, true)     \
+    if (gate_first) RB_GNL(T_, true, false)           \
+    if (vec) RB_GNL(T_, false, true)                  \
+    RB_GNL(T_, false, false)                          \
+  }
+  if (f32) RB_GNV(float)
+  RB_GNV(__nv_bfloat16)
+#undef RB_GNV
 #undef RB_GNL
 #undef RB_GN
 }

@@ -180,7 +180,7 @@ latent_append_kernel(const TR* __restrict__ qraw, int ldq, const TR* __restrict_
   for (int i = threadIdx.x; down && i < rank; i += kRowThreads) { const float v = to_f32(down[i]); ssq += v * v; }
   for (int i = threadIdx.x; i < dims / 2; i += kRowThreads) {
     float s, c;
-    sincosf(float(pos) * inv_freq[i], &s, &c);
+    rotary_sincos(pos, inv_freq[i], s, c);
     trig[i] = c;
     trig[dims / 2 + i] = s;
   }

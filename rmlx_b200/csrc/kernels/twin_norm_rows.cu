@@ -125,7 +125,7 @@ rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __
   const int t = blockIdx.x, pos = positions[t], half = dims / 2;
   for (int i = threadIdx.x; i < half; i += kRowThreads) {
     float s, c;
-    sincosf(float(pos) * inv_freq[i], &s, &c);
+    rotary_sincos(pos, inv_freq[i], s, c);
     trig[i] = c * grow;
     trig[half + i] = s * grow;
   }

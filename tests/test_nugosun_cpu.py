@@ -178,8 +178,8 @@ def test_oracle_latent_queries_and_routing_by_hand():
 
 
 def test_rotary_frequencies_match_the_restatement():
-    for rot in ({"base": 500000.0, "dims": 24}, {"base": 1e4, "dims": 2},
-                {"base": 500000.0, "dims": 24, "scaling": {"factor": 4.0, "original": 1000.0, "fast": 30.0, "slow": 1.0}},
+    for rot in ({"base": 300000.0, "dims": 28}, {"base": 1e4, "dims": 2},
+                {"base": 70000.0, "dims": 36, "scaling": {"factor": 6.0, "original": 1500.0, "fast": 20.0, "slow": 1.5}},
                 {"base": 50.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4.0, "fast": 1.0, "slow": 0.9}},
                 {"base": 1e4, "dims": 40, "scaling": {"factor": 1.0, "original": 2048.0, "fast": 32.0, "slow": 1.0}}):
         f, grow = TN.rotary_frequencies(rot["base"], rot["dims"], rot.get("scaling"))
