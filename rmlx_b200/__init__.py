@@ -21,7 +21,7 @@ _EXPORTS = {
     "NativePrefill": "models.prefill", "enable_native_prefill": "models.prefill",
     "Qwen2Model": "models.qwen", "MixtralModel": "models.mixtral", "DeepSeekV3Model": "models.deepseek",
     "PosudraModel": "models.posudra", "PosudraConfig": "config", "RodapelModel": "models.rodapel", "RodapelConfig": "config",
-    "NugosunModel": "models.nugosun", "NugosunConfig": "config",
+    "NugosunModel": "models.nugosun", "NugosunConfig": "config", "NizoraxModel": "models.nizorax", "NizoraxConfig": "config",
     "from_pretrained": "models.registry",
     "ModelFamily": "models.registry", "Entry": "models.ragged", "ParallelBlockDecode": "models.parallel_decode",
     # weights, caches, serving

@@ -64,6 +64,14 @@ SETS = {
                  "kernels/parallel_gemv.cu", "kernels/misc.cu", "runtime/graph_exec.cu"),
         "host": ("host/serving.cpp", "host/sampler.cpp", "host/safetensors_io.cpp"),
     },
+    "sandwich": {
+        "cuda": ("kernels/sandwich_rows.cu", "kernels/sandwich_gemv.cu", "kernels/twin_norm_rows.cu", "kernels/linear_scan.cu",
+                 "kernels/postnorm_rows.cu", "kernels/moe_route.cu", "kernels/gemm_tcgen05.cu", "kernels/xgemm_tcgen05.cu",
+                 "kernels/gemm_f32.cu", "kernels/flash_prefill_tc.cu", "kernels/flash_decode_scored.cu",
+                 "kernels/attention_any.cu", "kernels/parallel_rows.cu", "kernels/postnorm_gemv.cu",
+                 "kernels/parallel_gemv.cu", "kernels/misc.cu", "runtime/graph_exec.cu"),
+        "host": ("host/serving.cpp", "host/sampler.cpp", "host/safetensors_io.cpp"),
+    },
 }
 
 

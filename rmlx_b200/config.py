@@ -433,7 +433,8 @@ class RodapelConfig:
 
 @dataclass
 class RotarySpec:
-    """Rotation of the first ``dims`` values of a head; ``scaling``: None or YaRN's (factor, original, fast, slow)."""
+    """Rotation of the first ``dims`` values of a head; ``scaling``: None, YaRN's (factor, original, fast, slow) or Llama's
+    (factor, original, high, low)."""
     base: float
     dims: int
     scaling: Optional[dict] = None
@@ -442,15 +443,23 @@ class RotarySpec:
         _require(self.base > 0 and 0 <= self.dims <= dim and self.dims % 2 == 0,
                  "rotated dimensions come in pairs, at most the head's")
         if self.scaling:
-            _require(all(float(self.scaling[k]) > 0 for k in ("factor", "original", "fast", "slow")), "rotation scaling: positive values")
-            _require(self.base != 1.0, "rotation scaling needs a base other than 1")
+            keys = self.scaling_keys(self.scaling)
+            _require(all(float(self.scaling[k]) > 0 for k in keys), "rotation scaling: positive values")
+            if "high" in keys:
+                _require(self.scaling["high"] > self.scaling["low"], "rotation scaling: high must be above low")
+            else:
+                _require(self.base != 1.0, "rotation scaling needs a base other than 1")
         return self
+
+    @staticmethod
+    def scaling_keys(s: dict) -> tuple:
+        return ("factor", "original", "high", "low") if "high" in s else ("factor", "original", "fast", "slow")
 
     @staticmethod
     def from_json(r: dict) -> "RotarySpec":
         s = r.get("scaling")
         return RotarySpec(float(r["base"]), int(r["dims"]),
-                          None if not s else {k: float(s[k]) for k in ("factor", "original", "fast", "slow")})
+                          None if not s else {k: float(s[k]) for k in RotarySpec.scaling_keys(s)})
 
     def to_json(self) -> dict:
         out = {"base": self.base, "dims": self.dims}
@@ -687,6 +696,225 @@ class NugosunConfig:
     def to_json(self) -> dict:
         return {"architecture": "Nugosun", "vocab": self.vocab_size, "width": self.width, "norm": {"eps": self.norm_eps},
                 "embedding": {"scale": self.embedding_scale}, "layers": [l.to_json() for l in self.layers]}
+
+
+@dataclass
+class DifferentialAttentionSpec:
+    """Grouped-query attention with two maps per head (a query and a key of ``dim`` values each, over the same values): the
+    first map's result minus a learned multiple of the second's, normed per head and times 1 - ``diff``. Neighbouring values
+    of queries and keys turn together; ``window`` > 0: only the last so many keys."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotarySpec
+    diff: float
+    window: int = 0
+
+    kind = "attention"
+
+    def validate(self) -> "DifferentialAttentionSpec":
+        _require(self.heads > 0 and self.kv_heads > 0 and self.heads % self.kv_heads == 0,
+                 "heads must be a positive multiple of kv_heads")
+        _require(self.dim > 0 and self.vdim > 0, "head sizes must be positive")
+        _require(self.window >= 0, "window must be >= 0 (0: none)")
+        self.rot.validate(self.dim)
+        return self
+
+    @staticmethod
+    def from_json(m: dict) -> "DifferentialAttentionSpec":
+        return DifferentialAttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                                         RotarySpec.from_json(m["rot"]) if m.get("rot") else RotarySpec(10000.0, 0),
+                                         float(m["diff"]), int((m.get("mask") or {}).get("size") or 0))
+
+    def to_json(self) -> dict:
+        return {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale,
+                "rot": self.rot.to_json(), "diff": self.diff, "mask": {"size": self.window} if self.window else None}
+
+
+@dataclass
+class LightningSpec:
+    """Lightning attention: ``heads`` states of ``dim`` x ``vdim``, each with a constant decay."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: "list[float]"
+
+    kind = "lightning"
+
+    def validate(self) -> "LightningSpec":
+        _require(self.heads > 0 and self.vdim > 0 and 0 < self.dim <= 256, "lightning: heads and vdim positive, dim in [1, 256]")
+        _require(len(self.decay) == self.heads, "lightning: one decay per head")
+        return self
+
+    @staticmethod
+    def from_json(m: dict) -> "LightningSpec":
+        return LightningSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), [float(v) for v in m["decay"]])
+
+    def to_json(self) -> dict:
+        return {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "decay": list(self.decay)}
+
+
+@dataclass
+class PolyNormFfSpec:
+    """Feed-forward without a gate, its activation a polynomial of normed powers."""
+    ff: int
+
+    def validate(self) -> "PolyNormFfSpec":
+        _require(self.ff > 0, "feed-forward: ff must be positive")
+        return self
+
+    def to_json(self) -> dict:
+        return {"kind": "dense", "ff": self.ff}
+
+
+@dataclass
+class GroupedFfSpec:
+    """``experts`` gated feed-forwards of width ``ff`` in ``groups`` equal groups; each token uses the ``top`` with the largest
+    sigmoid scores in its ``keep`` best groups, weighted by the scores times ``scale``, and (``shared`` > 0) one of width
+    ``shared`` that every token uses."""
+    experts: int
+    top: int
+    ff: int
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+    shared: int = 0
+
+    limit = 0.0
+    identity = 0
+
+    def validate(self) -> "GroupedFfSpec":
+        _require(0 < self.experts <= 256 and self.ff > 0 and self.shared >= 0, "experts: 1 to 256, ff positive")
+        _require(1 <= self.groups <= 128 and self.experts % self.groups == 0 and 1 <= self.keep <= self.groups,
+                 "experts must form 1 to 128 equal groups, of which 1 or more are kept")
+        _require(1 <= self.top <= min(31, self.keep * self.experts // self.groups), "top must be in [1, 31] and fit the kept groups")
+        return self
+
+    @property
+    def slices(self) -> tuple:
+        """(count, width) of the equal parts the shared feed-forward is cut into, which run as experts of every token, as wide
+        as the routed ones unless they would be too many."""
+        if not self.shared:
+            return 0, self.ff
+        n = min(-(-self.shared // self.ff), 32 - self.top, 512 - self.experts)
+        return n, max(self.ff, -(-self.shared // n))
+
+    def to_json(self) -> dict:
+        out = {"kind": "moe", "expert": {"ff": self.ff},
+               "router": {"experts": self.experts, "top": self.top, "scale": self.scale, "groups": {"count": self.groups, "keep": self.keep}}}
+        if self.shared:
+            out["shared"] = {"ff": self.shared}
+        return out
+
+
+_SANDWICH_MIXERS = {c.kind: c for c in (DifferentialAttentionSpec, LightningSpec)}
+
+
+@dataclass
+class SandwichLayerSpec:
+    """One layer: a mixer and (unless None) a feed-forward, each between two norms and behind a short convolution."""
+    mixer: "DifferentialAttentionSpec | LightningSpec"
+    mlp: "PolyNormFfSpec | GroupedFfSpec | None" = None
+
+    def validate(self) -> "SandwichLayerSpec":
+        self.mixer.validate()
+        if self.mlp is not None:
+            self.mlp.validate()
+        return self
+
+    @staticmethod
+    def from_json(e: dict) -> "SandwichLayerSpec":
+        _require(e.get("type") in _SANDWICH_MIXERS, f"unknown mixer type {e.get('type')!r}")
+        m, mlp = e.get("mlp"), None
+        if m is not None:
+            _require(m.get("kind") in ("dense", "moe"), f"unknown feed-forward kind {m.get('kind')!r}")
+            if m["kind"] == "dense":
+                mlp = PolyNormFfSpec(int(m["ff"]))
+            else:
+                r, g = m["router"], m["router"].get("groups") or {}
+                mlp = GroupedFfSpec(int(r["experts"]), int(r["top"]), int(m["expert"]["ff"]), int(g.get("count", 1)),
+                                    int(g.get("keep", 1)), float(r.get("scale", 1.0)), int((m.get("shared") or {}).get("ff", 0)))
+        return SandwichLayerSpec(_SANDWICH_MIXERS[e["type"]].from_json(e["mixer"]), mlp)
+
+    def to_json(self) -> dict:
+        return {"type": self.mixer.kind, "mixer": self.mixer.to_json(),
+                "mlp": None if self.mlp is None else self.mlp.to_json()}
+
+
+@dataclass
+class LoopSpec:
+    """Layers ``start`` .. ``stop`` - 1 run ``times`` times in a row, each pass with a cache of its own."""
+    start: int
+    stop: int
+    times: int
+
+    def validate(self, layers: int) -> "LoopSpec":
+        _require(0 <= self.start < self.stop <= layers and self.times >= 1, "loop: a range of layers, at least once")
+        return self
+
+
+@dataclass
+class NizoraxConfig:
+    """Nizorax: a decoder of differential attention and lightning attention between layer norms, with short convolutions over
+    what the sublayers read and a range of layers that runs several times; every layer states its own kind and sizes."""
+    vocab_size: int
+    width: int
+    layers: "list[SandwichLayerSpec]"
+    norm_eps: float = 1e-6
+    embedding_scale: float = 1.0
+    logit_scale: float = 1.0
+    taps: int = 4
+    loop: Optional[LoopSpec] = None
+    max_seq_len: int = 0             # 0: bounded by the cache only
+    name: str = "nizorax"
+
+    sliding_window = 0               # pages are shared by every layer: none can be dropped early
+
+    def validate(self) -> "NizoraxConfig":
+        _require(self.vocab_size > 0 and self.width > 0 and len(self.layers) > 0, "bad sizes")
+        _require(self.norm_eps > 0, "norm_eps must be positive")
+        _require(1 <= self.taps <= 64, "the short convolution has 1 to 64 taps")
+        for layer in self.layers:
+            layer.validate()
+        if self.loop is not None:
+            self.loop.validate(len(self.layers))
+        return self
+
+    @property
+    def runs(self) -> "list[int]":
+        """The layers in the order in which they run."""
+        order = list(range(len(self.layers)))
+        if self.loop is None:
+            return order
+        a, b = self.loop.start, self.loop.stop
+        return order[:a] + order[a:b] * self.loop.times + order[b:]
+
+    @property
+    def num_layers(self) -> int:
+        """Layer runs: what the cache holds pages and states for."""
+        return len(self.runs)
+
+    @property
+    def hidden_size(self) -> int:
+        return self.width
+
+    @staticmethod
+    def from_json(c: dict) -> "NizoraxConfig":
+        loop = c.get("loop")
+        return NizoraxConfig(int(c["vocab"]), int(c["width"]), [SandwichLayerSpec.from_json(e) for e in c["layers"]],
+                             float(c["norm"]["eps"]), float((c.get("embedding") or {}).get("scale", 1.0)),
+                             float(c.get("logit_scale", 1.0)), int(c["canon"]["taps"]),
+                             LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None).validate()
+
+    def to_json(self) -> dict:
+        out = {"architecture": "Nizorax", "vocab": self.vocab_size, "width": self.width, "norm": {"eps": self.norm_eps},
+               "embedding": {"scale": self.embedding_scale}, "logit_scale": self.logit_scale, "canon": {"taps": self.taps},
+               "layers": [l.to_json() for l in self.layers]}
+        if self.loop is not None:
+            out["loop"] = {"start": self.loop.start, "stop": self.loop.stop, "times": self.loop.times}
+        return out
 
 
 @dataclass

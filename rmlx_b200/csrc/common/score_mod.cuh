@@ -7,6 +7,9 @@
 //   weights = exp(s) / (sum exp(s) + exp(sink[h]))    sink without key or value (nullptr: none)
 //   o = o * sigmoid(gate[t, h])                 output gate, one logit per token and head (nullptr: none)
 //
+// Differential attention: a head has two maps, each a query and a key of its own over the same values, and
+//   d = softmax(map 1) v - weight * softmax(map 2) v,   o = scale * d / sqrt(mean(d^2) + eps)     (MapDiff)
+//
 // The tensor-core kernels work in base 2 (scores times log2 e), which leaves one ex2 per weight.
 #pragma once
 #include "ptx.cuh"
@@ -22,6 +25,10 @@ struct ScoreMod {
   const float* r1 = nullptr;
   const float* r2 = nullptr;
   const float* sink = nullptr;
+};
+
+struct MapDiff {
+  float weight = 0.f, scale = 1.f, eps = 0.f;
 };
 
 // The first key a query at position `pos` sees: the last `window` keys (> 0), only its own chunk of `chunk`

@@ -13,6 +13,11 @@
 // values from L2), normalises its heads' queries, and the block whose split ends the sequence
 // normalises and appends the new key and value first: norm, append and attention are one launch.
 //
+// MAPS 2: differential attention (score_mod.cuh). A tile holds eight query heads: rows 0 - 7 are their first maps'
+// queries, rows 8 - 15 their second ones'. A page's keys come as two tiles, one per map; both score products take all
+// sixteen rows (each is used for its own half), after which everything up to the merge is as with one map. The merge
+// forms the difference of rows r and r + 8, norms it and writes one head.
+//
 // Rows in shared memory are padded to the class width (64 or 128) with zeros; global memory holds
 // dkp / dvp elements per row (multiples of eight), so narrow heads cost no extra bytes.
 #include "../common/launch.cuh"
@@ -63,17 +68,19 @@ struct FsParams {
   float* part_ml;                // [B, Hkv*gtiles, S, 16, 2]
   unsigned int* tickets;         // [B * Hkv*gtiles], zero on entry, zero on exit
   int raw_ld, max_blocks, Hq, Hkv, G, gtiles, S, window, chunk, dim, vdim, dkp, dvp;
-  int head_norm;                 // fused form: q_w / k_w are [dim] and every head is normed on its own
+  int head_norm;                 // fused form: 1: q_w / k_w are [dim], every head is normed on its own; 2: no norm
   // fused form with head_norm: bias of the projection (its layout), rotation of values i and i + rot_dims / 2 by position *
-  // inv_freq[i] with cos and sin times `grow`, both before the norm; q_w / k_w may then be null (no weight)
+  // inv_freq[i] with cos and sin times `grow`, both before the norm; q_w / k_w may then be null (no weight).
+  // neighbours: values 2 i and 2 i + 1 turn together instead
   const float* bias;
   const float* inv_freq;
-  int rot_dims;
+  int rot_dims, neighbours;
   float grow;
   int gate_col;                  // fused form: gate logits at raw[b][gate_col + head] (< 0: none)
   float eps;
   ScoreMod mod;
   HeadGate gate;                 // plain form
+  MapDiff diff;                  // MAPS 2: query heads and key rows are 2 dkp wide, [map 1 | map 2]
 };
 
 __device__ __forceinline__ float fs_block_sum(float v, float* red) {
@@ -103,12 +110,24 @@ __device__ __forceinline__ void fs_copy_page(char* dst, const char* src, int chu
   }
 }
 
+// The same for rows that hold MAPS keys of `chunks` pieces side by side: a tile of its own for each.
+template <int ROW_BYTES, int MAPS>
+__device__ __forceinline__ void fs_copy_maps(char* dst, const char* src, int chunks, int lane) {
+  if (MAPS == 1) { fs_copy_page<ROW_BYTES>(dst, src, chunks, lane); return; }
+  const int per = MAPS * chunks;
+  for (int i = lane; i < kFsPage * per; i += 32) {
+    const int r = i / per, q = i - r * per, a = q / chunks, c = q - a * chunks;
+    fs_cp_async16(dst + a * (kFsPage * ROW_BYTES) + r * ROW_BYTES + ((c ^ (r & 7)) << 4), src + i * 16);
+  }
+}
+
 // MOD = false: no modifier but the scale.
-template <int DK, int DV, int NST, bool MOD>
+template <int DK, int DV, int NST, bool MOD, int MAPS>
 __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParams p) {
   constexpr int KS = DK / 16;            // k-steps of the QK^T product
   constexpr int NT = DV / 8;             // n-tiles of the PV product
-  constexpr int K_PAGE = kFsPage * DK * 2, V_PAGE = kFsPage * DV * 2;
+  constexpr int K_TILE = kFsPage * DK * 2, K_PAGE = MAPS * K_TILE, V_PAGE = kFsPage * DV * 2;
+  constexpr int HPT = 16 / MAPS;         // query heads per tile
   constexpr int STAGE = K_PAGE + V_PAGE;
   extern __shared__ __align__(128) char smem[];
   char* wsm = smem + (threadIdx.x >> 5) * (NST * STAGE);   // reused for the merges afterwards
@@ -145,7 +164,7 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
     const int blk = RB_BOUNDS(pg, p.max_blocks) ? bt[pg] : 0;
     const size_t pgi = (size_t(blk) * p.Hkv + kvh) * kFsPage;
     char* kd = wsm + stage * STAGE;
-    fs_copy_page<DK * 2>(kd, reinterpret_cast<const char*>(p.k_cache + pgi * p.dkp), kch, lane);
+    fs_copy_maps<DK * 2, MAPS>(kd, reinterpret_cast<const char*>(p.k_cache + pgi * (MAPS * p.dkp)), kch, lane);
     fs_copy_page<DV * 2>(kd + K_PAGE, reinterpret_cast<const char*>(p.v_cache + pgi * p.dvp), vch, lane);
   };
 
@@ -162,11 +181,11 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   // ---- queries of this tile: 16 rows (heads beyond G are zero) ----
   if (p.raw) {
     const float* row = p.raw + size_t(b) * p.raw_ld;
-    const int nq = p.Hq * p.dim, nk = p.Hkv * p.dim;
-    if (p.head_norm) {
+    const int nq = p.Hq * MAPS * p.dim, nk = p.Hkv * MAPS * p.dim;
+    if (MAPS > 1 || p.head_norm) {
       // one warp per query head in turn; the owner's last warp also takes the new key's root mean square
       constexpr int PL = DK / 32;
-      const int q_rows = min(16, p.G - gt * 16), half = p.rot_dims >> 1;
+      const int q_heads = min(HPT, p.G - gt * HPT), half = p.rot_dims >> 1;
       // the rotation of this lane's places: own value times cs, partner's (at `other`) times sn
       float cs[PL], sn[PL];
       int other[PL];
@@ -175,11 +194,12 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
         const int d = i * 32 + lane;
         cs[i] = 1.f; sn[i] = 0.f; other[i] = d;
         if (d < p.rot_dims) {
+          const bool low = p.neighbours ? !(d & 1) : d < half;
           float sv, cv;
-          rotary_sincos(len - 1, p.inv_freq[d < half ? d : d - half], sv, cv);
+          rotary_sincos(len - 1, p.inv_freq[p.neighbours ? d >> 1 : low ? d : d - half], sv, cv);
           cs[i] = cv * p.grow;
-          sn[i] = (d < half ? -sv : sv) * p.grow;
-          other[i] = d < half ? d + half : d - half;
+          sn[i] = (low ? -sv : sv) * p.grow;
+          other[i] = p.neighbours ? d ^ 1 : low ? d + half : d - half;
         }
       }
       const bool rot = p.rot_dims > 0;
@@ -198,11 +218,12 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
           }
         }
       };
-      auto turn = [&](float (&v)[PL], const float (&u)[PL]) {     // returns 1 / rms
+      auto turn = [&](float (&v)[PL], const float (&u)[PL]) {     // returns 1 / rms (1 without a norm)
         if (rot) {
 #pragma unroll
           for (int i = 0; i < PL; ++i) v[i] = fmaf(v[i], cs[i], u[i] * sn[i]);
         }
+        if (p.head_norm != 1) return 1.f;
         float ss = 0.f;
 #pragma unroll
         for (int i = 0; i < PL; ++i) ss += v[i] * v[i];
@@ -211,8 +232,8 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
       float v[4][PL], u[4][PL];
 #pragma unroll
       for (int w = 0; w < 4; ++w) {
-        const int r = warp * 4 + w;
-        load_head((kvh * p.G + gt * 16 + r) * p.dim, r < q_rows, v[w], u[w]);
+        const int r = warp * 4 + w, hd = r % HPT, a = r / HPT;
+        load_head(((kvh * p.G + gt * HPT + hd) * MAPS + a) * p.dim, hd < q_heads, v[w], u[w]);
       }
 #pragma unroll
       for (int w = 0; w < 4; ++w) {
@@ -225,15 +246,16 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
       }
       if (owner && RB_BOUNDS((len - 1) / kFsPage, p.max_blocks)) {
         const size_t slot = (size_t(bt[(len - 1) / kFsPage]) * p.Hkv + kvh) * kFsPage + (len - 1) % kFsPage;
-        __nv_bfloat16* kd = p.k_cache + slot * p.dkp;
+        __nv_bfloat16* kd = p.k_cache + slot * (MAPS * p.dkp);
         __nv_bfloat16* vd = p.v_cache + slot * p.dvp;
-        if (warp == kFsWarps - 1) {
-          load_head(nq + kvh * p.dim, true, v[0], u[0]);
+        if (warp >= kFsWarps - MAPS) {
+          const int a = warp - (kFsWarps - MAPS);
+          load_head(nq + (kvh * MAPS + a) * p.dim, true, v[0], u[0]);
           const float ik = turn(v[0], u[0]);
 #pragma unroll
           for (int i = 0; i < PL; ++i) {
             const int d = i * 32 + lane;
-            if (d < p.dim) kd[d] = __float2bfloat16_rn(v[0][i] * ik * (p.k_w ? p.k_w[d] : 1.f));
+            if (d < p.dim) kd[a * p.dkp + d] = __float2bfloat16_rn(v[0][i] * ik * (p.k_w ? p.k_w[d] : 1.f));
           }
         }
         for (int d = threadIdx.x; d < p.vdim; d += kFsThreads) {
@@ -296,18 +318,19 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
     }
   } else {
     for (int i = threadIdx.x; i < 16 * (DK / 8); i += kFsThreads) {
-      const int r = i / (DK / 8), c = i % (DK / 8), h = gt * 16 + r;
+      const int r = i / (DK / 8), c = i % (DK / 8), h = gt * HPT + r % HPT;
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
       if (h < p.G && c * 8 < p.dkp)
-        v = *reinterpret_cast<const uint4*>(p.q + (size_t(b) * p.Hq + kvh * p.G + h) * p.dkp + c * 8);
+        v = *reinterpret_cast<const uint4*>(p.q + ((size_t(b) * p.Hq + kvh * p.G + h) * MAPS + r / HPT) * p.dkp + c * 8);
       *reinterpret_cast<uint4*>(&sQ[r][c * 8]) = v;
     }
   }
   const float lin = p.mod.scale * kLog2e;
   HeadScore hs0{}, hs1{};
-  if (gt * 16 + g < p.G) hs0 = head_score(p.mod, kvh * p.G + gt * 16 + g);
-  if (gt * 16 + g + 8 < p.G) hs1 = head_score(p.mod, kvh * p.G + gt * 16 + g + 8);
-  if (threadIdx.x < 16) {
+  if (MAPS == 1 && gt * 16 + g < p.G) hs0 = head_score(p.mod, kvh * p.G + gt * 16 + g);
+  if (MAPS == 1 && gt * 16 + g + 8 < p.G) hs1 = head_score(p.mod, kvh * p.G + gt * 16 + g + 8);
+  if (MAPS > 1 && threadIdx.x < 16) { s_sink[threadIdx.x] = -INFINITY; s_gate[threadIdx.x] = 1.f; }
+  if (MAPS == 1 && threadIdx.x < 16) {
     const int h = gt * 16 + threadIdx.x;
     s_sink[threadIdx.x] = (h < p.G && p.mod.sink) ? p.mod.sink[kvh * p.G + h] * kLog2e : -INFINITY;
     float gate = 1.f;
@@ -355,6 +378,19 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
       fs_ldm4(kb, kbase + tok * (DK * 2) + ((c ^ (tok & 7)) << 4));
       fs_mma(s0, qa[ks], kb[0], kb[1]);
       fs_mma(s1, qa[ks], kb[2], kb[3]);
+    }
+    if (MAPS > 1) {                      // rows 8 - 15 against the second map's keys
+      float u0[4] = {0.f, 0.f, 0.f, 0.f}, u1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int ks = 0; ks < KS; ++ks) {
+        const int mi = lane >> 3, r = lane & 7;
+        const int tok = (mi >> 1) * 8 + r, c = 2 * ks + (mi & 1);
+        uint32_t kb[4];
+        fs_ldm4(kb, kbase + (MAPS - 1) * K_TILE + tok * (DK * 2) + ((c ^ (tok & 7)) << 4));
+        fs_mma(u0, qa[ks], kb[0], kb[1]);
+        fs_mma(u1, qa[ks], kb[2], kb[3]);
+      }
+      s0[2] = u0[2]; s0[3] = u0[3]; s1[2] = u1[2]; s1[3] = u1[3];
     }
     const int tok0 = pg * kFsPage + t * 2;
     float sv[8] = {s0[0], s0[1], s1[0], s1[1], s0[2], s0[3], s1[2], s1[3]};
@@ -444,7 +480,8 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
     const int h = gt * 16 + row;
     if (p.S == 1) {
       if (s_sink[row] != -INFINITY) L += ex2_approx(s_sink[row] - M);
-      if (h < p.G && d < p.dvp)
+      if (MAPS > 1) so[row * DV + d] = L > 0.f ? acc / L : 0.f;      // (this thread alone has read the place)
+      else if (h < p.G && d < p.dvp)
         p.out[(size_t(b) * p.Hq + size_t(kvh) * p.G + h) * p.dvp + d] = __float2bfloat16_rn(L > 0.f ? acc * s_gate[row] / L : 0.f);
     } else {
       p.part_o[((tile * p.S + split) * 16 + row) * DV + d] = acc;
@@ -454,7 +491,31 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
       }
     }
   }
-  if (p.S == 1) return;
+  // MAPS 2: rows r and r + 8 of `val` [16][DV] are a head's two maps
+  auto put_difference = [&](const float* val) {
+    constexpr int PL = DV / 32;
+    for (int r = warp; r < HPT && gt * HPT + r < p.G; r += kFsWarps) {
+      float v[PL], ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < PL; ++i) {
+        const int d = i * 32 + lane;
+        v[i] = val[r * DV + d] - p.diff.weight * val[(r + HPT) * DV + d];
+        if (d < p.vdim) ss += v[i] * v[i];
+      }
+      const float inv = p.diff.scale / sqrtf(warp_sum(ss) / float(p.vdim) + p.diff.eps);
+      __nv_bfloat16* dst = p.out + (size_t(b) * p.Hq + size_t(kvh) * p.G + gt * HPT + r) * p.dvp;
+#pragma unroll
+      for (int i = 0; i < PL; ++i)
+        if (i * 32 + lane < p.dvp) dst[i * 32 + lane] = __float2bfloat16_rn(v[i] * inv);
+    }
+  };
+  if (p.S == 1) {
+    if (MAPS > 1) {
+      __syncthreads();
+      put_difference(so);
+    }
+    return;
+  }
 
   // ---- last block of this tile merges the splits ----
   __threadfence();
@@ -465,6 +526,7 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   __threadfence();
   float* wgt = reinterpret_cast<float*>(smem);        // [S][16] weights exp2(m_s - M) / L
   float* mls = wgt + kFsMaxSplits * 16;               // [S][16][2] copy of the (max, sum) table
+  float* whole = mls + kFsMaxSplits * 32;             // MAPS 2: [16][DV] merged rows
   for (int i = threadIdx.x; i < p.S * 32; i += kFsThreads) mls[i] = p.part_ml[tile * p.S * 32 + i];
   __syncthreads();
   if (threadIdx.x < 16) {
@@ -487,7 +549,7 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
   for (int idx = threadIdx.x; idx < 16 * D4; idx += kFsThreads) {
     const int row = idx / D4, d4 = idx % D4;
     const int h = gt * 16 + row;
-    if (h >= p.G || d4 * 4 >= p.dvp) continue;
+    if (MAPS == 1 && (h >= p.G || d4 * 4 >= p.dvp)) continue;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int s = 0; s < p.S; s += 16) {
       float4 v[16];
@@ -501,10 +563,18 @@ __global__ void __launch_bounds__(kFsThreads) flash_decode_scored_kernel(FsParam
         acc.z = fmaf(v[j].z, w, acc.z); acc.w = fmaf(v[j].w, w, acc.w);
       }
     }
+    if (MAPS > 1) {
+      *reinterpret_cast<float4*>(whole + row * DV + d4 * 4) = acc;
+      continue;
+    }
     uint2 ov;
     ov.x = pack_bf16(acc.x, acc.y);
     ov.y = pack_bf16(acc.z, acc.w);
     *reinterpret_cast<uint2*>(p.out + (size_t(b) * p.Hq + size_t(kvh) * p.G + h) * p.dvp + d4 * 4) = ov;
+  }
+  if (MAPS > 1) {
+    __syncthreads();
+    put_difference(whole);
   }
   if (threadIdx.x == 0) p.tickets[tile] = 0u;
 }
@@ -531,7 +601,10 @@ extern "C" long long rmlx_flash_decode_scored_ticket_elems(int B, int Hq, int Hk
 // q (bf16) or raw (fp32, with q_w, k_w, eps: the fused form), exactly one of them. dkp / dvp: dim /
 // vdim rounded up to eight. gate: bf16 [rows, ldg] output gate logits of the plain form, or null; head_norm,
 // gate_col (-1: none): the fused form's; with head_norm also bias (fp32, raw's layout, or null) and the rotation of the
-// first rot_dims values (inv_freq fp32 [rot_dims / 2]). `tickets` is zero on the first call; the kernel leaves it zero.
+// first rot_dims values (inv_freq fp32 [rot_dims / 2]; neighbours: pairs (2 i, 2 i + 1) turn). `tickets` is zero on the
+// first call; the kernel leaves it zero. maps 2: differential attention with no modifier but the scale - q [rows, Hq,
+// 2 dkp], key rows of 2 dkp values, raw = [q: Hq x 2 x dim | k: Hkv x 2 x dim | v] (head_norm 1 or 2); scratch as for 2 Hq
+// query heads.
 extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw_ld, const float* q_w,
                                         const float* k_w, float eps, void* k_cache, void* v_cache,
                                         const int* block_table, const int* positions, const int* rows,
@@ -541,11 +614,14 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
                                         float scale, float softcap, const float* temp, const float* r1,
                                         const float* r2, const float* sink, const void* gate, int ldg,
                                         int head_norm, int gate_col, const float* bias, const float* inv_freq,
-                                        int rot_dims, float grow, int pdl, cudaStream_t st) {
+                                        int rot_dims, float grow, int neighbours, int maps, float map_weight, float map_scale,
+                                        float map_eps, int pdl, cudaStream_t st) {
   if (B < 1 || B > 65535 || Hkv < 1 || Hq % Hkv || splits < 1 || splits > kFsMaxSplits || (!q) == (!raw) ||
       dkp % 8 || dvp % 8 || dim > dkp || vdim > dvp || dim < 1 || vdim < 1 || (r1 && !r2))
     return -2;
-  if (raw && (((!q_w || !k_w) && !head_norm) || raw_ld < (Hq + Hkv) * dim + Hkv * vdim)) return -2;
+  if (maps < 1 || maps > 2 || head_norm < 0 || head_norm > 2) return -2;
+  if (maps == 2 && (softcap > 0.f || temp || r1 || sink || gate || gate_col >= 0 || (raw && !head_norm))) return -2;
+  if (raw && (((!q_w || !k_w) && !head_norm) || raw_ld < (Hq + Hkv) * maps * dim + Hkv * vdim)) return -2;
   if ((bias || rot_dims) && !(raw && head_norm)) return -2;
   if (rot_dims < 0 || rot_dims % 2 || rot_dims > dim || (rot_dims && !inv_freq)) return -2;
   if (splits > 1 && (!part_o || !part_ml || !tickets)) return -2;
@@ -555,32 +631,41 @@ extern "C" int rmlx_flash_decode_scored(const void* q, const float* raw, int raw
   p.block_table = block_table; p.positions = positions; p.rows = rows; p.table_rows = table_rows;
   p.out = static_cast<__nv_bfloat16*>(out);
   p.part_o = part_o; p.part_ml = part_ml; p.tickets = tickets;
-  p.max_blocks = max_blocks; p.Hq = Hq; p.Hkv = Hkv; p.G = Hq / Hkv; p.gtiles = (p.G + 15) / 16;
+  p.max_blocks = max_blocks; p.Hq = Hq; p.Hkv = Hkv; p.G = Hq / Hkv; p.gtiles = (p.G * maps + 15) / 16;
   p.S = splits; p.window = window; p.chunk = chunk; p.dim = dim; p.vdim = vdim; p.dkp = dkp; p.dvp = dvp;
   p.mod.scale = scale; p.mod.softcap = softcap; p.mod.temp = temp; p.mod.r1 = r1; p.mod.r2 = r2; p.mod.sink = sink;
   p.gate.gate = gate; p.gate.ld = ldg; p.head_norm = head_norm; p.gate_col = gate_col;
   p.bias = bias; p.inv_freq = inv_freq; p.rot_dims = rot_dims; p.grow = grow;
+  p.neighbours = neighbours; p.diff.weight = map_weight; p.diff.scale = map_scale; p.diff.eps = map_eps;
   if (raw && gate_col >= 0 && raw_ld < gate_col + Hq) return -2;
   if (p.Hkv * p.gtiles > 65535) return -2;
   const dim3 grid(splits, Hkv * p.gtiles, B);
   const bool plain = softcap <= 0.f && !temp && !r1 && !sink;
   const bool deep = size_t(splits) * Hkv * p.gtiles * B <= size_t(2 * sm_count());
   // staging (>= 4 x 2 x 4 KB) covers the warp merge (4 x 16 x DV floats) and the split tables (12 KB)
-#define RB_FS(DK_, DV_, NST_)                                                      \
-  {                                                                                \
-    constexpr size_t smem = size_t(kFsWarps) * NST_ * kFsPage * (DK_ + DV_) * 2;   \
-    static_assert(smem >= size_t(kFsWarps) * 16 * DV_ * 4, "warp merge");          \
-    static_assert(smem >= size_t(kFsMaxSplits) * 16 * 3 * 4, "split tables");      \
-    auto kern = plain ? flash_decode_scored_kernel<DK_, DV_, NST_, false>          \
-                      : flash_decode_scored_kernel<DK_, DV_, NST_, true>;          \
-    RB_CHECK(set_max_smem(kern, smem));                                            \
-    return launch(kern, grid, dim3(kFsThreads), smem, st, pdl != 0, p);            \
+#define RB_FS(DK_, DV_, NST_, MAPS_)                                                       \
+  {                                                                                        \
+    constexpr size_t smem = size_t(kFsWarps) * NST_ * kFsPage * (MAPS_ * DK_ + DV_) * 2;   \
+    static_assert(smem >= size_t(kFsWarps) * 16 * DV_ * 4, "warp merge");                  \
+    static_assert(smem >= size_t(kFsMaxSplits) * 16 * 3 * 4 + (MAPS_ - 1) * 16 * DV_ * 4, "split tables"); \
+    auto kern = plain ? flash_decode_scored_kernel<DK_, DV_, NST_, false, MAPS_>           \
+                      : flash_decode_scored_kernel<DK_, DV_, NST_, MAPS_ == 1, MAPS_>;     \
+    RB_CHECK(set_max_smem(kern, smem));                                                    \
+    return launch(kern, grid, dim3(kFsThreads), smem, st, pdl != 0, p);                    \
+  }
+#define RB_FSM(DK_, DV_)                          \
+  {                                               \
+    if (maps == 2 && deep) RB_FS(DK_, DV_, 4, 2)  \
+    if (maps == 2) RB_FS(DK_, DV_, 2, 2)          \
+    if (deep) RB_FS(DK_, DV_, 4, 1)               \
+    RB_FS(DK_, DV_, 2, 1)                         \
   }
   const int ck = fs_class(dkp), cv = fs_class(dvp);
-  if (ck == 128 && cv == 128) { if (deep) RB_FS(128, 128, 4) else RB_FS(128, 128, 2) }
-  if (ck == 128 && cv == 64) { if (deep) RB_FS(128, 64, 4) else RB_FS(128, 64, 2) }
-  if (ck == 64 && cv == 128) { if (deep) RB_FS(64, 128, 4) else RB_FS(64, 128, 2) }
-  if (ck == 64 && cv == 64) { if (deep) RB_FS(64, 64, 4) else RB_FS(64, 64, 2) }
+  if (ck == 128 && cv == 128) RB_FSM(128, 128)
+  if (ck == 128 && cv == 64) RB_FSM(128, 64)
+  if (ck == 64 && cv == 128) RB_FSM(64, 128)
+  if (ck == 64 && cv == 64) RB_FSM(64, 64)
+#undef RB_FSM
 #undef RB_FS
   return -2;
 }

@@ -11,6 +11,10 @@
 // beforehand, [context rows, H, dim + vdim] in position order, and read through three-dimensional tensor
 // maps (a head's columns past its width read as zero); the rotated key part, shared by all heads, is the
 // last panel of a key row and comes straight from the latent cache's pages.
+// Differential attention (DIFF, score_mod.cuh): the two lanes are the two maps of one query tile. Each has its own
+// query tile and, per step, its own key tile; the value tile serves both, so the values cross shared memory once. At the
+// end the lanes exchange their sums and take half of the value columns each: difference of the maps, its norm over the
+// head, one store.
 //
 // Score modifiers run between S and the softmax, in base 2: t = P(s) - bias(i - j), where P is
 // softcap * tanh(s scale temp / softcap) as s times a polynomial in s^2 with the head's constants
@@ -67,10 +71,11 @@ constexpr int kTcPTile = kTcQPanel;           // 128 rows x 64 keys bf16
 constexpr int kTcPageBytes = kTcPage * 128;   // one page inside a 64-column panel
 constexpr float kTcRescaleStep = 8.f;         // log2 of the growth tolerated before O is rescaled
 
-template <int LANES, int KP, int VP, bool MOD>
+template <int LANES, int KP, int VP, bool MOD, bool DIFF = false>
 struct TcCfg {
   static constexpr int kQTile = KP * kTcQPanel;     // 128 query rows
-  static constexpr int kKTile = KP * kTcKvPanel;    // 64 keys
+  static constexpr int kKMap = KP * kTcKvPanel;     // 64 keys of one map
+  static constexpr int kKTile = (DIFF ? 2 : 1) * kKMap;
   static constexpr int kVTile = VP * kTcKvPanel;
   static constexpr int kThreads = 64 + 128 * LANES;
   // per lane: S0 [0,64) S1 [64,128); then per lane O (VP * 64 columns)
@@ -98,6 +103,9 @@ struct TcParams {
   // a cache row, first context row of every tile's sequence
   int kn, q_rot, c_rot;
   const int* tile_ctx;
+  // DIFF instances: query rows are [head][map], values of a head that exist
+  MapDiff diff;
+  int vdim;
   int* status;
 };
 
@@ -140,13 +148,20 @@ __device__ __forceinline__ float max3_abs(float a, float b, float c) {
   return d;
 }
 
-template <int LANES, int KP, int VP, bool MOD, bool LAT>
-__global__ void __launch_bounds__(TcCfg<LANES, KP, VP, MOD>::kThreads, 1)
+// Barrier `id` among `threads` threads of the block.
+__device__ __forceinline__ void named_bar_sync(int id, int threads) {
+  asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory");
+}
+
+template <int LANES, int KP, int VP, bool MOD, bool LAT, bool DIFF>
+__global__ void __launch_bounds__(TcCfg<LANES, KP, VP, MOD, DIFF>::kThreads, 1)
 flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
                         const __grid_constant__ CUtensorMap tmap_k,
                         const __grid_constant__ CUtensorMap tmap_v,
                         const __grid_constant__ CUtensorMap tmap_kr, TcParams p) {
-  using C = TcCfg<LANES, KP, VP, MOD>;
+  using C = TcCfg<LANES, KP, VP, MOD, DIFF>;
+  static_assert(!DIFF || (LANES == 2 && !MOD && !LAT), "differential attention: one lane per map");
+  constexpr int kLaneRows = DIFF ? 0 : kTcRows;     // rows from one lane's tile to the next one's
   extern __shared__ __align__(1024) char smem[];
   if (smem_u32(smem) & 1023u) {       // the swizzled tiles need 1024-byte alignment
     if (threadIdx.x == 0 && p.status) atomicExch(p.status, kStatusBadArgument);
@@ -193,7 +208,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   int n_max = 0, kv_end_max = 1;
 #pragma unroll
   for (int L = 0; L < LANES; ++L) {
-    const int first = L * kTcRows;
+    const int first = L * kLaneRows;
     const int kv_end = pos_q0 + min(first + kTcRows, rows);
     n_steps[L] = first < rows ? (kv_end + kTcKeys - 1) / kTcKeys - j0 : 0;
     if (n_steps[L] > 0) { n_max = max(n_max, n_steps[L]); kv_end_max = max(kv_end_max, kv_end); }
@@ -247,7 +262,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
 #pragma unroll
           for (int c = 0; c < KP; ++c)
             tma_load_2d(sQ + L * C::kQTile + c * kTcQPanel, &tmap_q, q_full,
-                        h * p.dk + (LAT && c >= p.kn ? p.q_rot + (c - p.kn) * 64 : c * 64), q0 + L * kTcRows);
+                        (DIFF ? h * 2 + L : h) * p.dk + (LAT && c >= p.kn ? p.q_rot + (c - p.kn) * 64 : c * 64),
+                        q0 + L * kLaneRows);
         }
       }
       for (int j = 0; j < n_max; ++j) {
@@ -280,8 +296,11 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
 #pragma unroll
           for (int pg = 0; pg < kTcPages; ++pg)
 #pragma unroll
-            for (int c = 0; c < KP; ++c)
+            for (int c = 0; c < KP; ++c) {
               tma_load_2d(kd + c * kTcKvPanel + pg * kTcPageBytes, &tmap_k, k_full + s, c * 64, y[pg]);
+              if (DIFF)          // the second map's columns, through a tensor map of their own
+                tma_load_2d(kd + C::kKMap + c * kTcKvPanel + pg * kTcPageBytes, &tmap_kr, k_full + s, c * 64, y[pg]);
+            }
         }
         if (!mbar_wait(v_free + s, par, abort_flag)) break;
         mbar_arrive_expect_tx(v_full + s, C::kVTile);
@@ -324,10 +343,11 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         const int s = j & 1;
         const uint32_t u = (j >> 1) & 1;
         if (!mbar_wait(k_full + s, u, abort_flag)) return false;
-        const uint32_t k_addr = smem_u32(sK + s * C::kKTile);
+        const uint32_t k_tile = smem_u32(sK + s * C::kKTile);
 #pragma unroll
         for (int L = 0; L < LANES; ++L) {
           if (j >= n_steps[L]) continue;
+          const uint32_t k_addr = k_tile + (DIFF ? L * C::kKMap : 0);
           uint64_t* lb = lane_bars + 6 * L;
           if (!mbar_wait(lb + 2 + s, u ^ 1u, abort_flag)) return false;   // s_free
           tc_fence_after_sync();
@@ -382,7 +402,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
     uint64_t* s_free = s_full + 2;
     uint64_t* p_full = s_full + 4;
     uint64_t* o_done = s_full + 5;
-    const int lrow = L * kTcRows + row;                // row inside the block
+    const int lrow = L * kLaneRows + row;              // row inside the block
     const int pos = pos_q0 + lrow, first = first_key(pos, p.window, p.chunk);
     const int my_steps = n_steps[LANES == 1 ? 0 : L];
     const float sc = MOD ? 1.f : p.scale_log2;         // MOD: scores are final, in base 2
@@ -479,7 +499,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         }
         __syncwarp();
       }
-      if (k0 + kTcKeys - 1 > pos_q0 + L * kTcRows) {   // the step touches the diagonal
+      if (k0 + kTcKeys - 1 > pos_q0 + L * kLaneRows) {   // the step touches the diagonal
         const int vis = pos - k0;                      // keys k0 .. k0+vis are visible to this row
 #pragma unroll
         for (int c = 0; c < NC; ++c)
@@ -580,7 +600,50 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       ok = mbar_wait(o_done, (my_steps - 1) & 1, abort_flag);
       ok = __all_sync(0xffffffffu, ok);
     }
-    if (ok && my_steps > 0) {
+    if (DIFF) {
+      // both lanes arrive at both barriers whatever happened; this lane's P tile is free once its last product is done
+      float* mine = reinterpret_cast<float*>(sP + L * kTcPTile);
+      const float* other = reinterpret_cast<const float*>(sP + (1 - L) * kTcPTile);
+      const float own = l > 0.f ? 1.f / l : 0.f;
+      if (ok) mine[row] = own;
+      named_bar_sync(1, 256);
+      const bool whole = __all_sync(0xffffffffu, ok) && *abort_flag == 0u;
+      float v[VP * 32], ssq = 0.f;
+      if (whole) {
+        tc_fence_after_sync();
+        const float theirs = other[row];
+        const float f1 = L == 0 ? own : theirs, f2 = (L == 0 ? theirs : own) * p.diff.weight;
+        const uint32_t o1 = tmem_base + LANES * 128 + t_lane, o2 = o1 + VP * 64;
+#pragma unroll
+        for (int c = 0; c < VP; ++c) {                   // this lane's half of the value columns
+          uint32_t a[32], b[32];
+          tmem_ld_32x32(o1 + (L * VP + c) * 32, a);
+          tmem_ld_32x32(o2 + (L * VP + c) * 32, b);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {                 // (columns past the head's width are zero)
+            v[c * 32 + i] = __uint_as_float(a[i]) * f1 - __uint_as_float(b[i]) * f2;
+            ssq += v[c * 32 + i] * v[c * 32 + i];
+          }
+        }
+        mine[kTcRows + row] = ssq;
+      }
+      named_bar_sync(1, 256);
+      if (whole && lrow < rows) {
+        const float inv = p.diff.scale / sqrtf((ssq + other[kTcRows + row]) / float(p.vdim) + p.diff.eps);
+        __nv_bfloat16* dst = p.out + (size_t(q0 + lrow) * p.Hq + h) * p.dv + L * VP * 32;
+#pragma unroll
+        for (int u = 0; u < VP * 4; ++u) {
+          if (L * VP * 32 + u * 8 >= p.dv) break;        // dv is a multiple of 8
+          uint4 pk;
+          pk.x = pack_bf16(v[u * 8] * inv, v[u * 8 + 1] * inv);
+          pk.y = pack_bf16(v[u * 8 + 2] * inv, v[u * 8 + 3] * inv);
+          pk.z = pack_bf16(v[u * 8 + 4] * inv, v[u * 8 + 5] * inv);
+          pk.w = pack_bf16(v[u * 8 + 6] * inv, v[u * 8 + 7] * inv);
+          *reinterpret_cast<uint4*>(dst + u * 8) = pk;
+        }
+      }
+    } else if (ok && my_steps > 0) {
       tc_fence_after_sync();
       float inv = l > 0.f ? 1.f / l : 0.f;
       if (p.gate.gate) inv *= head_gate<__nv_bfloat16>(p.gate, size_t(q0 + min(lrow, rows - 1)), h);
@@ -617,11 +680,11 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   pdl_launch_dependents();
 }
 
-template <int LANES, int KP, int VP, bool MOD, bool LAT = false>
+template <int LANES, int KP, int VP, bool MOD, bool LAT = false, bool DIFF = false>
 static int launch_prefill_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv,
                              TcParams p, int pdl, cudaStream_t st, const CUtensorMap* tkr = nullptr) {
-  auto kern = flash_prefill_tc_kernel<LANES, KP, VP, MOD, LAT>;
-  using C = TcCfg<LANES, KP, VP, MOD>;
+  auto kern = flash_prefill_tc_kernel<LANES, KP, VP, MOD, LAT, DIFF>;
+  using C = TcCfg<LANES, KP, VP, MOD, DIFF>;
   constexpr size_t smem = C::kSmem;
   RB_CHECK(set_max_smem(kern, smem));
   if (!p.tiles) p.n_qt = (p.T + kTcRows * LANES - 1) / (kTcRows * LANES);
@@ -733,6 +796,48 @@ extern "C" int rmlx_flash_prefill_scored(const void* q, const void* k_cache, con
   if (dv > 64) { RB_FPS(1, 2); }
   RB_FPS(1, 1);
 #undef RB_FPS
+}
+
+// Differential attention over a ragged batch: q [T, Hq, 2, dk], keys [num_blocks, Hkv, 16, 2 dk] = [map 1 | map 2], values
+// [num_blocks, Hkv, 16, dv], of which vdim exist (the rest are zero); out [T, Hq, dv] = map_scale * d / rms(d), d = the
+// first map's attention - map_weight * the second's. tiles: at most 128 rows each. dk, dv as
+// rmlx_flash_prefill_scored_supported.
+extern "C" int rmlx_flash_prefill_diff(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
+                                       int max_blocks, const int* tiles, int n_tiles, void* out, int T, int Hq, int Hkv, int dk,
+                                       int dv, int vdim, int num_blocks, int window, int chunk, float scale, float map_weight,
+                                       float map_scale, float map_eps, int* status, int pdl, cudaStream_t st) {
+  if (T < 1 || Hkv < 1 || Hq % Hkv || num_blocks < 1 || n_tiles < 1 || !tiles || vdim < 1 || vdim > dv ||
+      !rmlx_flash_prefill_scored_supported(dk, dv))
+    return -2;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) |
+       reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(out) |
+       reinterpret_cast<uintptr_t>(tiles)) & 15)
+    return -2;
+  CUtensorMap tq, tk, tv, tk2;
+  int rc = make_tmap_2d_bf16(&tq, q, uint64_t(Hq) * 2 * dk, uint64_t(T), uint64_t(Hq) * 4 * dk, 64, kTcRows);
+  if (rc) return rc;
+  const uint64_t rows = uint64_t(num_blocks) * Hkv * kTcPage;
+  rc = make_tmap_2d_bf16(&tk, k_cache, uint64_t(dk), rows, uint64_t(dk) * 4, 64, kTcPage);
+  if (rc) return rc;
+  rc = make_tmap_2d_bf16(&tk2, static_cast<const __nv_bfloat16*>(k_cache) + dk, uint64_t(dk), rows, uint64_t(dk) * 4, 64, kTcPage);
+  if (rc) return rc;
+  rc = make_tmap_2d_bf16(&tv, v_cache, uint64_t(dv), rows, uint64_t(dv) * 2, 64, kTcPage);
+  if (rc) return rc;
+  TcParams p{};
+  p.block_table = block_table; p.max_blocks = max_blocks;
+  p.tiles = reinterpret_cast<const int4*>(tiles); p.n_qt = n_tiles;
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.pos0 = 0;
+  p.dk = dk; p.dv = dv; p.vdim = vdim;
+  p.window = window > 0 ? window : 0; p.chunk = chunk > 0 ? chunk : 0;
+  p.scale_log2 = scale * kLog2e;
+  p.diff.weight = map_weight; p.diff.scale = map_scale; p.diff.eps = map_eps;
+  p.status = status;
+#define RB_FPD(KP_, VP_) return launch_prefill_tc<2, KP_, VP_, false, false, true>(tq, tk, tv, p, pdl, st, &tk2)
+  if (dk > 64) { if (dv > 64) RB_FPD(2, 2); RB_FPD(2, 1); }
+  if (dv > 64) RB_FPD(1, 2);
+  RB_FPD(1, 1);
+#undef RB_FPD
 }
 
 // 1 when the latent form takes these (eight-padded) widths: unrotated, rotated, value.

@@ -4,9 +4,10 @@
 //         S <- diag(alpha) S + k v^T, o = S^T (q scale)
 //   ssd   state-space heads: x, B and C through a causal depthwise convolution and silu, dt = softplus(.),
 //         S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x; `H / G` heads share a group's B and C
+//   lightning  one constant decay per head; q, k and v through silu; S <- decay S + k v^T, o = S^T q
 //
 // and what surrounds them: the convolution's carried inputs, and the norm of the outputs over equal groups of
-// columns with a silu gate before or after it. Decays, step sizes and their exponentials are fp32.
+// columns with a silu or sigmoid gate before or after it. Decays, step sizes and their exponentials are fp32.
 #include "../common/launch.cuh"
 #include "../common/rows.cuh"
 #include "../common/scan.cuh"
@@ -163,6 +164,56 @@ ssd_prepare_kernel(SsdIn<T> in, float* __restrict__ rec, float* __restrict__ col
   }
 }
 
+template <class T>
+struct LightIn {
+  const T* q; const T* k; const T* v;
+  int ld;
+  const float* decay;       // [H]
+  int dim, vdim;
+};
+// Records of heads with a constant decay, LU lanes per (token, head).
+template <class T, int ROWS, int LANES, int LU>
+__global__ void __launch_bounds__(kRowThreads)
+lightning_prepare_kernel(LightIn<T> in, float* __restrict__ rec, float* __restrict__ col, int rows, int H, int shift) {
+  constexpr int kRows = ROWS * LANES;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int unit = (blockIdx.x * kRowThreads + threadIdx.x) / LU, lane = threadIdx.x % LU;
+  const bool live = unit < rows * H;                 // the lanes of a warp stay together for the sum
+  const int t = live ? unit / H : 0, h = live ? unit - t * H : 0;
+  const bool vec = in.dim % 4 == 0 && in.ld % 4 == 0, vec_v = in.vdim % 4 == 0 && in.ld % 4 == 0;
+  const size_t row = size_t(t) * in.ld;
+  float* out = rec + (size_t(h) * rows + t) * 2 * kRows;
+  float own = 0.f;
+  for (int i = lane * 4; i < kRows; i += LU * 4) {
+    float r[4], k[4];
+    scan_load4(in.q + row + h * in.dim, i, in.dim, vec, r);
+    scan_load4(in.k + row + h * in.dim, i, in.dim, vec, k);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      r[j] = silu_f(r[j]);
+      k[j] = silu_f(k[j]);
+      own = fmaf(r[j], k[j], own);
+    }
+    if (live) {
+      float* o = out + scan_at<ROWS, LANES>(i);
+      *reinterpret_cast<float4*>(o) = make_float4(r[0], r[1], r[2], r[3]);
+      *reinterpret_cast<float4*>(o + kRows) = make_float4(k[0], k[1], k[2], k[3]);
+    }
+  }
+  own = group_sum<LU>(own);
+  if (!live) return;
+  const int cols = 1 << shift, nb = (in.vdim + cols - 1) >> shift;
+  for (int i = lane * 4; i < nb << shift; i += LU * 4) {
+    float v[4];
+    scan_load4(in.v + row + h * in.vdim, i, in.vdim, vec_v, v);
+    const int at = i & (cols - 1);
+    float* o = col + ((size_t(h) * nb + (i >> shift)) * rows + t) * (cols + 4) + at;
+    *reinterpret_cast<float4*>(o) = make_float4(silu_f(v[0]), silu_f(v[1]), silu_f(v[2]), silu_f(v[3]));
+    if (at == 0) *reinterpret_cast<float4*>(o + cols) = make_float4(in.decay[h], 1.f, own, 0.f);
+  }
+}
+
 // The last taps - 1 inputs of every segment's sequence become its carried ones. A thread owns a channel; it
 // writes in ascending order and reads ahead of what it writes.
 template <class T>
@@ -187,19 +238,20 @@ conv_carry_kernel(const T* __restrict__ raw, int ld, int x_at, float* __restrict
   }
 }
 
-// silu of an output gate; with the hardware exponential and division where the result is rounded to bf16.
+// silu (or sigmoid) of an output gate; with the hardware exponential and division where the result is rounded to bf16.
 template <class T>
-__device__ __forceinline__ float gate_silu(float z) {
-  return sizeof(T) == 2 ? __fdividef(z, 1.f + __expf(fminf(-z, 80.f))) : silu_f(z);
+__device__ __forceinline__ float gate_value(float z, bool sigmoid) {
+  const float n = sigmoid ? 1.f : z;
+  return sizeof(T) == 2 ? __fdividef(n, 1.f + __expf(fminf(-z, 80.f))) : n / (1.f + expf(-z));
 }
 
-// out[t, c] over equal groups of columns: FIRST: f = o silu(gate), f / rms(f over the group) * w;
-// else o / rms(o over the group) * w * silu(gate). L lanes (256: a block) per (row, group), KEEP chunks of eight a lane
+// out[t, c] over equal groups of columns, g: silu or sigmoid: FIRST: f = o g(gate), f / rms(f over the group) * w;
+// else o / rms(o over the group) * w * g(gate). L lanes (256: a block) per (row, group), KEEP chunks of eight a lane
 // keeps; what is left is read again. VEC: sizes and strides are multiples of eight.
 template <class T, int L, int KEEP, bool FIRST, bool VEC>
 __global__ void __launch_bounds__(kRowThreads)
 gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ gate, int ld_g, const float* __restrict__ w,
-                  float eps, T* __restrict__ out, int ld_out, int rows, int groups, int size) {
+                  float eps, T* __restrict__ out, int ld_out, int rows, int groups, int size, bool sigmoid) {
   __shared__ float red[kRowThreads / 32];
   pdl_launch_dependents();
   pdl_wait();
@@ -215,7 +267,7 @@ gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ g
       float z[8];
       load8_upto(gp + i0, size - i0, VEC, z);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) a[i] *= gate_silu<T>(z[i]);
+      for (int i = 0; i < 8; ++i) a[i] *= gate_value<T>(z[i], sigmoid);
     }
   };
   auto factor = [&](int i0, float (&a)[8]) {           // what the normed values are multiplied by
@@ -224,7 +276,7 @@ gated_norm_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ g
       float z[8];
       load8_upto(gp + i0, size - i0, VEC, z);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) a[i] *= gate_silu<T>(z[i]);
+      for (int i = 0; i < 8; ++i) a[i] *= gate_value<T>(z[i], sigmoid);
     }
   };
 #pragma unroll
@@ -297,6 +349,26 @@ static int launch_ssd(const SsdIn<T>& in, ScanParams p, float* rec, int n_segs, 
   if (rc) return rc;
   p.rec = rec; p.col = col; p.per = in.H / in.G;
   return launch_scan<ROWS, LANES, true>(p, th, n_segs, pdl, st);
+}
+template <class T, int ROWS, int LANES>
+static int launch_lightning(const LightIn<T>& in, ScanParams p, float* rec, int n_segs, int pdl, cudaStream_t st) {
+  constexpr int kRows = ROWS * LANES, LU = kRows >= 128 ? 32 : kRows / 4;
+  const long long threads = 1LL * p.rows * p.H * LU;
+  if (threads > 0x7fffffffLL) return -2;
+  const int th = scan_threads(LANES, p.d, p.H, n_segs);
+  float* col = rec + size_t(p.H) * p.rows * 2 * kRows;
+  const int rc = launch(lightning_prepare_kernel<T, ROWS, LANES, LU>, dim3(unsigned((threads + kRowThreads - 1) / kRowThreads)),
+                        dim3(kRowThreads), 0, st, pdl != 0, in, rec, col, p.rows, p.H, scan_col_shift(LANES, th));
+  if (rc) return rc;
+  p.rec = rec; p.col = col; p.per = 1;
+  return launch_scan<ROWS, LANES, true>(p, th, n_segs, pdl, st);
+}
+template <class T>
+static int run_lightning(const LightIn<T>& in, const ScanParams& p, float* rec, int n, int pdl, cudaStream_t st) {
+#define RB_LI(R_, L_) return launch_lightning<T, R_, L_>(in, p, rec, n, pdl, st)
+  RB_SCAN_DISPATCH(p.n, RB_LI);
+#undef RB_LI
+  return -2;
 }
 template <class T>
 static int run_ssd(const SsdIn<T>& in, const ScanParams& p, float* rec, int n, int pdl, cudaStream_t st) {
@@ -377,9 +449,30 @@ extern "C" int rmlx_ssd_scan(const void* raw, int ld, int x_at, int dt_at, const
   return f32 ? run(static_cast<float*>(nullptr)) : run(static_cast<__nv_bfloat16*>(nullptr));
 }
 
+// q, k, v and the other arguments as in rmlx_gla_scan; decay fp32 [H]. rec: rmlx_scan_record(dim, vdim, 1, 1) floats per
+// (token, head).
+extern "C" int rmlx_lightning_scan(const void* q, const void* k, const void* v, int ld, const float* decay, float* rec, int rows,
+                                   const int* segs, const int* slots, int n_segs, float* state, long long stride, float* out,
+                                   int ld_out, int H, int dim, int vdim, int f32, int* status, int pdl, cudaStream_t st) {
+  if (!scan_args_ok(rows, segs, slots, n_segs, rec, H, dim, vdim) || !decay || ld < H * dim || ld < H * vdim || ld_out < H * vdim ||
+      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15))
+    return -2;
+  ScanParams p{};
+  p.rows = rows; p.segs = reinterpret_cast<const int4*>(segs); p.slots = slots;
+  p.state = state; p.stride = stride; p.out = out; p.ld_out = ld_out;
+  p.H = H; p.n = dim; p.d = vdim; p.status = status;
+  auto run = [&](auto* type) {
+    using T = std::remove_pointer_t<decltype(type)>;
+    return run_lightning<T>(LightIn<T>{static_cast<const T*>(q), static_cast<const T*>(k), static_cast<const T*>(v), ld, decay,
+                                       dim, vdim}, p, rec, n_segs, pdl, st);
+  };
+  return f32 ? run(static_cast<float*>(nullptr)) : run(static_cast<__nv_bfloat16*>(nullptr));
+}
+
 // o fp32 [rows, ld_o], gate and out [rows, ..] fp32 (f32) or bf16, w fp32 [groups * size].
 extern "C" int rmlx_gated_norm(const float* o, int ld_o, const void* gate, int ld_g, const float* w, float eps, void* out,
-                               int ld_out, int rows, int groups, int size, int gate_first, int f32, int pdl, cudaStream_t st) {
+                               int ld_out, int rows, int groups, int size, int gate_first, int sigmoid, int f32, int pdl,
+                               cudaStream_t st) {
   if (rows < 1 || groups < 1 || size < 1 || ld_o < groups * size || ld_g < groups * size || ld_out < groups * size) return -2;
   const int lanes = size <= 64 ? 8 : size <= 128 ? 16 : size <= 256 ? 32 : 256;
   const long long units = 1LL * rows * groups, blocks = (units * lanes + kRowThreads - 1) / kRowThreads;
@@ -390,7 +483,7 @@ extern "C" int rmlx_gated_norm(const float* o, int ld_o, const void* gate, int l
                       reinterpret_cast<uintptr_t>(w)) & 15);
 #define RB_GN(T_, L_, K_, F_, V_)                                                                                      \
   return launch(gated_norm_kernel<T_, L_, K_, F_, V_>, grid, dim3(kRowThreads), 0, st, pdl != 0, o, ld_o,              \
-                static_cast<const T_*>(gate), ld_g, w, eps, static_cast<T_*>(out), ld_out, rows, groups, size)
+                static_cast<const T_*>(gate), ld_g, w, eps, static_cast<T_*>(out), ld_out, rows, groups, size, sigmoid != 0)
 #define RB_GNL(T_, F_, V_)                          \
   {                                                 \
     if (lanes == 8) RB_GN(T_, 8, 1, F_, V_);        \

@@ -5,7 +5,7 @@
 //
 //   postnorm_in       out = W x: fp32 rows, or (gated) the activation of row pairs (i, n + i) in bf16, or
 //                     (shift) row segments that each read their own token-shift mix of x
-//   postnorm_router   router logits, softmax, corrected top-k (the last block to finish chooses)
+//   postnorm_router   router logits and the choice of experts by one of route.cuh's rules (the last block to finish chooses)
 //   postnorm_expert   gate / up projections of each token's chosen experts with the gated activation
 //   expert_out        y = sum over slots of weight * Wdown[e] act + identity weight * x
 //   matvec_out        y = W a
@@ -28,7 +28,7 @@ struct PostNormIn {
   const float* w;
   float eps;
   int D, ldx;
-  float* x_out;                   // written by block 0; not x itself
+  float* x_out;                   // written by block 0; not x itself (null: y is null, too, and x is only read)
 };
 // Token shift: rows seg * seg_rows .. of W read x + (prev - x) * mu[seg].
 struct ShiftIn {
@@ -142,7 +142,7 @@ postnorm_in_kernel(Matrix<WBf16> W, PostNormIn in, ShiftIn sh, float* __restrict
   const float* mu = sh.mu ? sh.mu + size_t(seg) * in.ldx : nullptr;
 #pragma unroll
   for (int b = 0; b < B; ++b)
-    stage_post_norm(in, b, smem + b * bstride, red, blockIdx.x == 0 && seg == 0, mu,
+    stage_post_norm(in, b, smem + b * bstride, red, blockIdx.x == 0 && seg == 0 && in.x_out, mu,
                     mu ? sh.prev + sh.slots[b] * sh.stride : nullptr);
   __syncthreads();
   for (bool first = true; n0 < n_hi; n0 += gridDim.x * kGemvWarps * kPnRows, first = false) {
@@ -169,11 +169,11 @@ postnorm_in_kernel(Matrix<WBf16> W, PostNormIn in, ShiftIn sh, float* __restrict
 }
 
 // One block per router output, its warps share the row; the last block to arrive chooses for every token.
-template <int B>
+template <int B, RouteRule RULE>
 __global__ void __launch_bounds__(kGemvThreads)
 postnorm_router_kernel(Matrix<WBf16> W, PostNormIn in, const float* __restrict__ correction, float* __restrict__ logits,
                        int* __restrict__ idx, float* __restrict__ weights, float* __restrict__ identity,
-                       unsigned int* __restrict__ ticket, int experts, int outputs, int top_k) {
+                       unsigned int* __restrict__ ticket, int experts, int outputs, int top_k, RouteGroups groups) {
   extern __shared__ __align__(16) char smem[];
   __shared__ float red[kGemvWarps];
   __shared__ float part[kGemvWarps][B];
@@ -192,7 +192,7 @@ postnorm_router_kernel(Matrix<WBf16> W, PostNormIn in, const float* __restrict__
   pdl_launch_dependents();
   pdl_wait();
 #pragma unroll
-  for (int b = 0; b < B; ++b) stage_post_norm(in, b, smem + b * bstride, red, n == 0, nullptr, nullptr);
+  for (int b = 0; b < B; ++b) stage_post_norm(in, b, smem + b * bstride, red, n == 0 && in.x_out, nullptr, nullptr);
   __syncthreads();
   float acc[B];
 #pragma unroll
@@ -239,8 +239,9 @@ postnorm_router_kernel(Matrix<WBf16> W, PostNormIn in, const float* __restrict__
       float* z = reinterpret_cast<float*>(smem) + b * outputs;
       for (int i = lane; i < outputs; i += 32) z[i] = __ldcg(logits + size_t(b) * outputs + i);
       __syncwarp();
-      warp_route<kRouteCorrected>(z, correction, experts, outputs, top_k, idx + size_t(b) * top_k,
-                                  weights + size_t(b) * top_k, identity + b, nullptr);
+      const int slots = top_k + groups.always;
+      warp_route<RULE>(z, correction, experts, outputs, top_k, idx + size_t(b) * slots, weights + size_t(b) * slots,
+                       identity ? identity + b : nullptr, nullptr, groups);
     }
     if (threadIdx.x == 0) *ticket = 0u;
   }
@@ -290,7 +291,8 @@ postnorm_expert_kernel(const __nv_bfloat16* __restrict__ w, int K, const float* 
   }
 }
 
-// grid (row blocks, tokens): y[b, n] = sum_s weight_s * (Wdown[e_s] act_s)[n] + identity * x[b, n], n < N. y may be x.
+// grid (row blocks, tokens): y[b, n] = sum_s weight_s * (Wdown[e_s] act_s)[n] + identity * x[b, n], n < N (identity null:
+// without the last term). y may be x.
 __global__ void __launch_bounds__(kGemvThreads, 2)
 expert_out_kernel(const __nv_bfloat16* __restrict__ w, int rows_e, int K, const __nv_bfloat16* __restrict__ act, int ld_act,
                   const int* __restrict__ idx, const float* __restrict__ weights, const float* __restrict__ identity,
@@ -350,7 +352,7 @@ expert_out_kernel(const __nv_bfloat16* __restrict__ w, int rows_e, int K, const 
   for (int r = 0; r < kPnRows; ++r) {
     const float v = warp_sum(tot[r]);
     const int n = n0 + r;
-    if (lane == r && n < N) y[size_t(b) * ldx + n] = fmaf(identity[b], __ldcg(x + size_t(b) * ldx + n), v);
+    if (lane == r && n < N) y[size_t(b) * ldx + n] = identity ? fmaf(identity[b], __ldcg(x + size_t(b) * ldx + n), v) : v;
   }
 }
 
@@ -521,13 +523,13 @@ static int launch_in(const void* w, const PostNormIn& in, const ShiftIn& sh, flo
                 static_cast<__nv_bfloat16*>(act), ld_act, N, limit);
 }
 
-// w bf16 [N, ldx]; x, y (or null) and x_out fp32 [B, ldx], norm_w fp32 [ldx]; out fp32 [B, ld_out]. mu (or
+// w bf16 [N, ldx]; x, y (or null) and x_out (or, with y, null) fp32 [B, ldx], norm_w fp32 [ldx]; out fp32 [B, ld_out]. mu (or
 // null): fp32 [5, ldx], prev rows `stride` apart by slots [B]; then w's rows are four segments of seg_rows (a
 // multiple of 16) and a fifth.
 extern "C" int rmlx_postnorm_in(const void* w, const float* x, const float* y, const float* norm_w, float eps, float* x_out,
                                 int D, int ldx, const float* mu, const float* prev, const int* slots, long long stride,
                                 int seg_rows, float* out, int ld_out, int B, int N, int pdl, cudaStream_t st) {
-  if (ldx < 8 || ldx % 8 || D < 1 || D > ldx || N < 1 || ld_out < N || !x_out || x_out == x || B > rmlx_postnorm_max_rows(ldx) ||
+  if (ldx < 8 || ldx % 8 || D < 1 || D > ldx || N < 1 || ld_out < N || (!x_out && y) || x_out == x || B > rmlx_postnorm_max_rows(ldx) ||
       (y && !norm_w) || (mu && (!prev || !slots || stride % 4 || seg_rows < 16 || seg_rows % 16)))
     return -2;
   const PostNormIn in{x, y, norm_w, eps, D, ldx, x_out};
@@ -547,17 +549,17 @@ extern "C" int rmlx_postnorm_gated(const void* w, const float* x, const float* y
   RB_PN_DISPATCH(B, (launch_in<kB, true>(w, in, sh, nullptr, 0, act, ld_act, N, limit, pdl, st)))
 }
 
-template <int B>
+template <int B, RouteRule RULE>
 static int launch_router(const void* w, const PostNormIn& in, const float* correction, float* logits, int* idx,
                          float* weights, float* identity, unsigned int* ticket, int experts, int outputs, int top_k, int pdl,
-                         cudaStream_t st) {
+                         cudaStream_t st, const RouteGroups& groups = RouteGroups{}) {
   size_t smem = XStage<WBf16>::bytes(in.ldx) * B;
   if (smem < size_t(B) * outputs * 4) smem = size_t(B) * outputs * 4;
-  auto kern = postnorm_router_kernel<B>;
+  auto kern = postnorm_router_kernel<B, RULE>;
   RB_CHECK(set_max_smem(kern, smem));
   return launch(kern, dim3(outputs), dim3(kGemvThreads), smem, st, pdl != 0,
                 Matrix<WBf16>{static_cast<const __nv_bfloat16*>(w), in.ldx}, in, correction, logits, idx, weights, identity,
-                ticket, experts, outputs, top_k);
+                ticket, experts, outputs, top_k, groups);
 }
 
 // w bf16 [outputs, ldx]; logits fp32 [B, outputs] scratch; ticket: one word, zero on entry and on exit.
@@ -569,8 +571,22 @@ extern "C" int rmlx_postnorm_router(const void* w, const float* x, const float* 
       outputs > kRouteMaxOutputs || top_k < 1 || top_k > kRouteMaxTop || top_k > outputs || B > rmlx_postnorm_max_rows(ldx))
     return -2;
   const PostNormIn in{x, y, norm_w, eps, D, ldx, x_out};
-  RB_PN_DISPATCH(B, (launch_router<kB>(w, in, correction, logits, idx, weights, identity, ticket, experts, outputs, top_k,
-                                       pdl, st)))
+  RB_PN_DISPATCH(B, (launch_router<kB, kRouteCorrected>(w, in, correction, logits, idx, weights, identity, ticket, experts,
+                                                        outputs, top_k, pdl, st)))
+}
+
+// Routing by sigmoids and groups of finished rows h fp32 [B, ldx]; idx and weights [B, top_k + always], the rest as above.
+extern "C" int rmlx_grouped_router(const void* w, const float* h, int ldx, float* logits, int* idx, float* weights,
+                                   unsigned int* ticket, int B, int experts, int top_k, int groups, int keep, int always,
+                                   float scale, int pdl, cudaStream_t st) {
+  RouteGroups g;
+  g.count = groups; g.keep = keep; g.always = always; g.scale = scale;
+  if (ldx < 8 || ldx % 8 || experts < 1 || experts > kRouteMaxOutputs || top_k < 1 || !route_groups_ok(g, experts, top_k) ||
+      B > rmlx_postnorm_max_rows(ldx))
+    return -2;
+  const PostNormIn in{h, nullptr, nullptr, 0.f, ldx, ldx, nullptr};
+  RB_PN_DISPATCH(B, (launch_router<kB, kRouteGrouped>(w, in, nullptr, logits, idx, weights, nullptr, ticket, experts, experts,
+                                                      top_k, pdl, st, g)))
 }
 
 // w bf16 [experts, 2 N, ldx]; x fp32 [B, ldx]; idx [B, top_k]; act bf16 [B * top_k, ld_act].

@@ -17,6 +17,7 @@
 #include "../common/launch.cuh"
 #include "../common/route.cuh"
 #include "../common/rows.cuh"
+#include "../common/state_step.cuh"
 
 namespace cg = cooperative_groups;
 
@@ -212,31 +213,7 @@ twin_in_kernel(TwinIn in, Matrix<WBf16> Wm, int N1, float* __restrict__ out, int
   }
 }
 
-__device__ __forceinline__ float tn_silu(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float tn_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-
-// State rows of one thread: rows i0 .. i0 + ROWS - 1 (below i1) of one column. They belong to the calling kernel alone
-// within a step, so they are asked for before the wait (the step's first kernel has waited for everything before it).
-template <int ROWS>
-__device__ __forceinline__ void load_state(const float* sp, int d, int i0, int i1, bool live, float (&s)[ROWS]) {
-#pragma unroll
-  for (int q = 0; q < ROWS; ++q) s[q] = (live && i0 + q < i1) ? __ldcg(sp + size_t(i0 + q) * d) : 0.f;
-}
-// Their part of S^T r, and S <- w S + k v (w: per row, or one for all).
-template <int ROWS, bool ONE>
-__device__ __forceinline__ float step_state(float* sp, int d, int i0, int i1, const float (&s)[ROWS], const float* r, const float* k,
-                                            const float* w, float one, float v) {
-  float o = 0.f;
-#pragma unroll
-  for (int q = 0; q < ROWS; ++q) {
-    const int i = i0 + q;
-    if (i < i1) {
-      o = fmaf(r[i], s[q], o);
-      sp[size_t(i) * d] = fmaf(ONE ? one : w[i], s[q], k[i] * v);
-    }
-  }
-  return o;
-}
 
 struct GlaStep {
   const float* raw;               // [B, ld_raw]: q, k, v, g and the decay rank at their columns
@@ -321,7 +298,7 @@ gla_decode_kernel(GlaStep p) {
   if (tid < COLS && col < d) {
     const float inv = 1.f / sqrtf(ssq / float(d) + p.eps);
     p.a[size_t(b) * p.ld_a + h * d + col] =
-        __float2bfloat16_rn(o * inv * p.norm[h * d + col] * tn_silu(__ldcg(row + p.at_g + h * d + col)));
+        __float2bfloat16_rn(o * inv * p.norm[h * d + col] * step_silu(__ldcg(row + p.at_g + h * d + col)));
   }
 }
 
@@ -390,10 +367,10 @@ ssd_decode_kernel(SsdStep p) {
   };
 #pragma unroll
   for (int u = 0; u < kKeep; ++u)
-    if (chan[u] >= 0) keep(u * kGemvThreads + tid, tn_silu(fmaf(now_w[u], __ldcg(row + p.x_at + chan[u]), past[u])));
+    if (chan[u] >= 0) keep(u * kGemvThreads + tid, step_silu(fmaf(now_w[u], __ldcg(row + p.x_at + chan[u]), past[u])));
   for (int i = kKeep * kGemvThreads + tid; i < 2 * n + COLS; i += kGemvThreads) {
     const int c = channel(i);
-    if (c >= 0) keep(i, tn_silu(fmaf(p.conv_w[size_t(last) * ch + c], __ldcg(row + p.x_at + c), past_conv(p, before, ch, c))));
+    if (c >= 0) keep(i, step_silu(fmaf(p.conv_w[size_t(last) * ch + c], __ldcg(row + p.x_at + c), past_conv(p, before, ch, c))));
   }
   const float dt = tn_softplus(__ldcg(row + p.dt_at + h) + p.dt_bias[h]), decay = expf(-expf(p.a_log[h]) * dt);
   __syncthreads();
@@ -431,7 +408,7 @@ ssd_finish_kernel(SsdStep p, const float* __restrict__ norm, float eps, int grou
   }
   const float* y = p.out + size_t(b) * p.ld_out + at;
   float f[kKeep], ssq = 0.f;
-  auto value = [&](int i) { return __ldcg(y + i) * tn_silu(__ldcg(row + at + i)); };
+  auto value = [&](int i) { return __ldcg(y + i) * step_silu(__ldcg(row + at + i)); };
 #pragma unroll
   for (int u = 0; u < kKeep; ++u) {
     const int i = u * kGemvThreads + tid;
@@ -526,46 +503,6 @@ extern "C" int rmlx_twin_in_router(const float* x, const float* w1, const float*
   RB_TN_DISPATCH(B, (launch_twin_in<kB, kTwinRouter>(in, w, N1, out, ld_out, ff, pdl, st)))
 }
 
-// Launches a (column blocks, heads, rows) grid with the column blocks of a head as one cluster.
-template <class P>
-static int launch_columns(void (*kern)(P), const P& p, int blocks, int H, int B, size_t smem, bool cluster, int pdl,
-                          cudaStream_t st) {
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(blocks, H, B);
-  cfg.blockDim = dim3(kGemvThreads);
-  cfg.dynamicSmemBytes = smem;
-  cfg.stream = st;
-  cudaLaunchAttribute attr[2];
-  int n = 0;
-  if (cluster && blocks > 1) {
-    attr[n].id = cudaLaunchAttributeClusterDimension;
-    attr[n].val.clusterDim.x = blocks; attr[n].val.clusterDim.y = 1; attr[n].val.clusterDim.z = 1;
-    ++n;
-  }
-  if (pdl) {
-    attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[n].val.programmaticStreamSerializationAllowed = 1;
-    ++n;
-    prefer_max_shared(kern);
-  }
-  cfg.attrs = attr; cfg.numAttrs = n;
-  const cudaError_t e = cudaLaunchKernelEx(&cfg, kern, p);
-  if (e != cudaSuccess) (void)cudaGetLastError();
-  return static_cast<int>(e);
-}
-
-// The instance for n state rows and d columns: CALL(COLS, ROWS); clusters hold at most eight blocks.
-#define RB_TN_STATE(n_, d_, CALL)                        \
-  if ((d_) <= 256) {                                     \
-    if ((n_) <= 32) { CALL(32, 4); }                     \
-    if ((n_) <= 64) { CALL(32, 8); }                     \
-    if ((n_) <= 128) { CALL(32, 16); }                   \
-    CALL(32, 32);                                        \
-  }                                                      \
-  if ((n_) <= 64) { CALL(64, 16); }                      \
-  if ((n_) <= 128) { CALL(64, 32); }                     \
-  CALL(64, 64)
-
 // 1 when the decode kernel of gated linear attention takes a state of n x d.
 extern "C" int rmlx_gla_decode_supported(int n, int d) { return n >= 1 && n <= 256 && d >= 1 && d <= 512; }
 
@@ -581,7 +518,7 @@ extern "C" int rmlx_gla_decode(const float* raw, int ld_raw, int at_k, int at_v,
                   norm, eps, slots, state, stride, static_cast<__nv_bfloat16*>(a), ld_a, n, d};
   const size_t smem = size_t(3 * n + rank) * sizeof(float);
 #define RB_GD(C_, R_) return launch_columns(gla_decode_kernel<C_, R_>, p, (d + C_ - 1) / C_, H, B, smem, true, pdl, st)
-  RB_TN_STATE(n, d, RB_GD);
+  RB_STATE_DISPATCH(n, d, RB_GD);
 #undef RB_GD
 }
 
@@ -601,7 +538,7 @@ extern "C" int rmlx_ssd_decode(const float* raw, int ld_raw, int x_at, int dt_at
   const int rc = [&]() -> int {
     // a head's columns need not meet in one block here
 #define RB_SD(C_, R_) return launch_columns(ssd_decode_kernel<C_, R_>, p, (d + C_ - 1) / C_, H, B, smem, false, pdl, st)
-    RB_TN_STATE(n, 1, RB_SD);
+    RB_STATE_DISPATCH(n, 1, RB_SD);
 #undef RB_SD
   }();
   if (rc) return rc;

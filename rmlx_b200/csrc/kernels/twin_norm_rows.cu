@@ -4,7 +4,8 @@
 //   twin_norm           the residual, with the routed experts' weighted rows added if there are any, and both norms
 //                       of it in one pass
 //   rows_norm           RMS norm of a slice of a projection's rows (the latent that queries go through)
-//   rotary_norm_append  bias, rotation of halves, unweighted per-head norm of queries and keys, cache append
+//   rotary_norm_append  bias, rotation (of halves or of neighbours), unweighted per-head norm of queries and keys (or
+//                       none), cache append; heads of one or of two maps
 //
 // Activations are bf16 (serving) or fp32 (the all-32-bit mode); norms, angles and the residual are fp32 in both.
 #include "../common/launch.cuh"
@@ -111,14 +112,16 @@ rows_norm_kernel(const TR* __restrict__ in, int ld, const float* __restrict__ w,
 // raw row t = [q: Hq*dim | k: Hkv*dim | v: Hkv*vdim | ..], bias (fp32, the same layout) or null. Value i of a query
 // or key head turns with value i + dims / 2 by position * inv_freq[i], cos and sin times `grow`; then every query
 // and key head is divided by its own root mean square. q goes to q_out [T, Hq, dkp], k and v to the token's slot of
-// its sequence's pages. One block per token, or (grid y) several; L lanes per head.
+// its sequence's pages. One block per token, or (grid y) several; L lanes per head. neighbours: values 2 i and 2 i + 1 turn
+// together instead. norm 0: no division. maps 2 (differential attention): every query and key head is two of `dim`
+// values, side by side also in q_out and in a key's cache row; each part turns and is normed on its own.
 template <class TR, class T, int L>
 __global__ void __launch_bounds__(kRowThreads)
 rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restrict__ bias,
                           const float* __restrict__ inv_freq, int dims, float grow, float eps, T* __restrict__ q_out,
                           T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ block_table,
                           const int* __restrict__ positions, const int* __restrict__ token_seq, int Hq, int Hkv, int dim,
-                          int vdim, int dkp, int dvp, int max_blocks, int page) {
+                          int vdim, int dkp, int dvp, int max_blocks, int page, int neighbours, int norm, int maps) {
   extern __shared__ __align__(16) float trig[];          // cos [dims / 2], sin [dims / 2]
   pdl_launch_dependents();
   pdl_wait();
@@ -134,14 +137,14 @@ rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __
   const int seq = token_seq ? token_seq[t] : t;
   const bool in_table = RB_BOUNDS(pos / page, max_blocks);
   const int blk = in_table ? block_table[size_t(seq) * max_blocks + pos / page] : 0;
-  const int per = Hq + 2 * Hkv, lane = threadIdx.x % L;
+  const int nq = Hq * maps, nk = Hkv * maps, per = nq + nk + Hkv, lane = threadIdx.x % L;
   for (int r0 = blockIdx.y * (kRowThreads / L); r0 < per; r0 += gridDim.y * (kRowThreads / L)) {
     const int r = r0 + threadIdx.x / L;
     const bool live = r < per;                         // the lanes of a warp stay together for the sums
-    const bool is_q = r < Hq, is_v = r >= Hq + Hkv;
-    const int head = is_q ? r : is_v ? r - Hq - Hkv : r - Hq;
+    const bool is_q = r < nq, is_v = r >= nq + nk;
+    const int head = is_q ? r : is_v ? r - nq - nk : r - nq;
     const int width = !live ? 0 : is_v ? vdim : dim, padded = is_v ? dvp : dkp;
-    const int src0 = !live ? 0 : is_v ? (Hq + Hkv) * dim + head * vdim : r * dim;
+    const int src0 = !live ? 0 : is_v ? (nq + nk) * dim + head * vdim : r * dim;
     const TR* src = row + src0;
     const float* bs = bias ? bias + src0 : nullptr;
     const bool vec = width % 8 == 0 && src0 % 8 == 0 && ldraw % 8 == 0;
@@ -163,7 +166,15 @@ rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __
     auto load = [&](int d0, float (&f)[8]) {
       biased(d0, f);
       if (is_v || d0 >= dims || !live) return;
-      if (pairs) {
+      if (neighbours) {
+#pragma unroll
+        for (int i = 0; i < 8; i += 2) {
+          if (d0 + i >= dims) break;
+          const float c = trig[(d0 + i) >> 1], s = trig[half + ((d0 + i) >> 1)], u = f[i], v = f[i + 1];
+          f[i] = u * c - v * s;
+          f[i + 1] = v * c + u * s;
+        }
+      } else if (pairs) {
         const bool low = d0 < half;
         const int j = low ? d0 : d0 - half;
         float g[8], cs[8], sn[8];
@@ -182,8 +193,9 @@ rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __
       }
     };
     T* dst = nullptr;
-    if (is_q) dst = q_out + (size_t(t) * Hq + head) * dkp;
-    else if (in_table) dst = (is_v ? v_cache : k_cache) + ((size_t(blk) * Hkv + head) * page + pos % page) * padded;
+    if (is_q) dst = q_out + (size_t(t) * nq + head) * dkp;
+    else if (in_table && is_v) dst = v_cache + ((size_t(blk) * Hkv + head) * page + pos % page) * dvp;
+    else if (in_table) dst = k_cache + (((size_t(blk) * Hkv + head / maps) * page + pos % page) * maps + head % maps) * dkp;
     float first[8], ssq = 0.f;
     load(lane * 8, first);
 #pragma unroll
@@ -196,7 +208,7 @@ rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __
     }
     ssq = group_sum<L>(ssq);
     if (!live || !dst) continue;
-    const float inv = is_v ? 1.f : 1.f / sqrtf(ssq / float(dim) + eps);
+    const float inv = is_v || !norm ? 1.f : 1.f / sqrtf(ssq / float(dim) + eps);
     for (int d0 = lane * 8; d0 < padded; d0 += L * 8) {
       float f[8];
       if (d0 == lane * 8) {
@@ -258,25 +270,25 @@ extern "C" int rmlx_rows_norm(const void* in, int ld, int in_f32, const float* w
 }
 
 // f32: q_out and the caches are fp32, else bf16; raw_f32: raw is fp32. dims: how many of a head's values turn (even,
-// <= dim); inv_freq fp32 [dims / 2].
+// <= dim); inv_freq fp32 [dims / 2]. maps 2: q_out [T, Hq, 2, dkp], key rows of 2 dkp values.
 extern "C" int rmlx_rotary_norm_append(const void* raw, int ldraw, int raw_f32, const float* bias, const float* inv_freq,
                                        int dims, float grow, float eps, void* q_out, void* k_cache, void* v_cache,
                                        const int* block_table, const int* positions, const int* token_seq, int T, int Hq,
-                                       int Hkv, int dim, int vdim, int dkp, int dvp, int max_blocks, int page, int f32, int pdl,
-                                       cudaStream_t st) {
+                                       int Hkv, int dim, int vdim, int dkp, int dvp, int max_blocks, int page, int neighbours,
+                                       int norm, int maps, int f32, int pdl, cudaStream_t st) {
   if (T < 1 || Hq < 1 || Hkv < 1 || dim < 1 || vdim < 1 || dkp % 8 || dvp % 8 || dkp < dim || dvp < vdim || dims < 0 ||
-      dims % 2 || dims > dim || ldraw < (Hq + Hkv) * dim + Hkv * vdim || (f32 && !raw_f32))
+      dims % 2 || dims > dim || maps < 1 || maps > 2 || ldraw < (Hq + Hkv) * maps * dim + Hkv * vdim || (f32 && !raw_f32))
     return -2;
   const size_t smem = size_t(dims) * sizeof(float);
   if (smem > 32 * 1024) return -2;
   const int widest = dkp > dvp ? dkp : dvp, lanes = widest <= 64 ? 8 : widest <= 128 ? 16 : 32;
-  const int per_block = kRowThreads / lanes, blocks = (Hq + 2 * Hkv + per_block - 1) / per_block;
+  const int per_block = kRowThreads / lanes, blocks = ((Hq + Hkv) * maps + Hkv + per_block - 1) / per_block;
   const dim3 grid(T, T >= 64 ? 1 : blocks);           // few tokens: several blocks share one
 #define RB_RA_L(TR_, T_, L_)                                                                                            \
   return launch(rotary_norm_append_kernel<TR_, T_, L_>, grid, dim3(kRowThreads), smem, st, pdl != 0,                    \
                 static_cast<const TR_*>(raw), ldraw, bias, inv_freq, dims, grow, eps, static_cast<T_*>(q_out),          \
                 static_cast<T_*>(k_cache), static_cast<T_*>(v_cache), block_table, positions, token_seq, Hq, Hkv, dim, vdim, \
-                dkp, dvp, max_blocks, page)
+                dkp, dvp, max_blocks, page, neighbours, norm, maps)
 #define RB_RA(TR_, T_)                     \
   {                                        \
     if (lanes == 8) RB_RA_L(TR_, T_, 8);   \

@@ -1,4 +1,4 @@
-"""What models with a layer list of their own share (``models/rodapel.py``, ``models/nugosun.py``): merged and padded
+"""What models with a layer list of their own share (``models/rodapel.py``, ``models/nugosun.py``, ``models/nizorax.py``): merged and padded
 weights, activation buffers, latent attention over the paged cache, gated and routed feed-forwards, and the forward
 pass over a ragged batch with its one-sequence conveniences. A model adds its mixers, ``start`` (embedding) and
 ``layer``."""
@@ -79,18 +79,19 @@ class DenseFfWeights:
 class RoutedFfWeights:
     spec: object                     # experts, identity, top, ff, limit
     router: torch.Tensor             # [experts + identity, width_p]
-    correction: torch.Tensor         # fp32 [experts + identity]: the router's correction or bias
-    w_gu: LinearWeight               # [experts, 2 * ff_p, width_p]
-    w_down: LinearWeight             # [experts, rows, ff_p], rows: width rounded up to the tile width
+    correction: Optional[torch.Tensor]   # fp32 [experts + identity]: the router's correction or bias (None: neither)
+    w_gu: LinearWeight               # [experts + always, 2 * ff_p, width_p]
+    w_down: LinearWeight             # [experts + always, rows, ff_p], rows: width rounded up to the tile width
+    always: int = 0                  # experts behind the routed ones that every token uses
 
 
 def weight_bytes(*parts) -> int:
-    """Bytes of the tensors and linear weights that the given dataclasses hold."""
+    """Bytes of the tensors and linear weights that the given dataclasses hold (one given twice counts once)."""
     def size(v) -> int:
         if isinstance(v, LinearWeight):
             return v.nbytes()
         return v.numel() * v.element_size() if isinstance(v, torch.Tensor) else 0
-    return sum(size(v) for p in parts if p is not None for v in vars(p).values())
+    return sum(size(v) for p in {id(p): p for p in parts if p is not None}.values() for v in vars(p).values())
 
 
 def check_tensors(tensors: Dict[str, torch.Tensor], shapes: Dict[str, tuple]) -> None:
@@ -318,28 +319,32 @@ class RaggedModel:
             P.prefill_scored_supported(pad8(m.dim), pad8(m.vdim))
 
     def paged_attention(self, li: int, m, mods: ScoreMods, q: torch.Tensor, c: StepContext, window: int = 0, chunk: int = 0,
-                        gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        gate: Optional[torch.Tensor] = None, diff: Optional[P.MapDiff] = None) -> torch.Tensor:
         """Attention of the batch's queries [T, heads, pad8(dim)] over the layer's pages: tensor-core prompt attention for
-        the entries of several tokens, split-KV decode attention for the others."""
+        the entries of several tokens, split-KV decode attention for the others. ``diff``: differential attention, queries
+        [T, heads, 2, pad8(dim)]; the batch's query tiles are then planned one lane wide."""
         t, b, pdl = c.t, c.batch, c.pdl
         k, v = c.cache.k[li], c.cache.v[li]
         attn = c.bufs.get("attn", t, m.heads, v.shape[3], dtype=self.dtype)
         see = dict(window=window, chunk=chunk, gate=gate)
         reach = min([r for r in (window, chunk) if r], default=0)
+        rows_per_head = 1 if diff is None else 2
         if not self.tensor_core_attention(m):
-            P.attention_any(q, k, v, c.block_table, c.positions, c.token_seq, mods, attn, pdl=pdl, **see)
+            P.attention_any(q, k, v, c.block_table, c.positions, c.token_seq, mods, attn, diff=diff, vdim=m.vdim, pdl=pdl, **see)
         elif b is None:
-            s = self.scratch(m.heads, m.kv_heads, v.shape[3], t, self.attention_splits(m, t, c.max_len, reach))
+            s = self.scratch(m.heads * rows_per_head, m.kv_heads, v.shape[3], t, self.attention_splits(m, t, c.max_len, reach))
             P.flash_decode_scored(k, v, c.block_table, c.positions, mods, attn, s, m.heads, m.dim, m.vdim, q=q, n_rows=t,
-                                  pdl=pdl, **see)
+                                  diff=diff, pdl=pdl, **see)
         else:
-            if b.tiles is not None:
+            if b.tiles is not None and diff is not None:
+                P.flash_prefill_diff(q, k, v, c.block_table, b.tiles, mods.scale, diff, m.vdim, attn, window=window, chunk=chunk)
+            elif b.tiles is not None:
                 P.flash_prefill_scored(q, k, v, c.block_table, b.tiles, mods, attn, lanes=b.lanes, **see)
             if b.single is not None:
                 n = len(b.single_host)
-                s = self.scratch(m.heads, m.kv_heads, v.shape[3], n, self.attention_splits(m, n, b.single_len, reach))
+                s = self.scratch(m.heads * rows_per_head, m.kv_heads, v.shape[3], n, self.attention_splits(m, n, b.single_len, reach))
                 P.flash_decode_scored(k, v, c.block_table, c.positions, mods, attn, s, m.heads, m.dim, m.vdim, q=q,
-                                      rows=b.single, table_rows=c.token_seq, **see)
+                                      rows=b.single, table_rows=c.token_seq, diff=diff, **see)
         return attn.view(t, -1)
 
     def latent_prefill(self, mw: LatentWeights) -> bool:
@@ -408,23 +413,22 @@ class RaggedModel:
 
     def routing(self, fw: RoutedFfWeights, c: StepContext) -> R.Routing:
         f, t = fw.spec, c.t
-        i32 = dict(dtype=torch.int32)
-        return R.Routing(c.bufs.get("route_idx", t, f.top, **i32), c.bufs.get("route_w", t, f.top, dtype=torch.float32),
-                         c.bufs.get("route_id", t, dtype=torch.float32), c.bufs.get("route_counts", 1, f.experts, **i32)[0],
-                         c.bufs.get("route_offsets", 1, f.experts + 1, **i32)[0],
-                         c.bufs.get("route_rows", t, f.top, **i32))
+        i32, slots, experts = dict(dtype=torch.int32), f.top + fw.always, f.experts + fw.always
+        return R.Routing(c.bufs.get("route_idx", t, slots, **i32), c.bufs.get("route_w", t, slots, dtype=torch.float32),
+                         c.bufs.get("route_id", t, dtype=torch.float32) if fw.correction is not None else None,
+                         c.bufs.get("route_counts", 1, experts, **i32)[0], c.bufs.get("route_offsets", 1, experts + 1, **i32)[0],
+                         c.bufs.get("route_rows", t, slots, **i32))
 
     def router_logits(self, fw: RoutedFfWeights, h: torch.Tensor, c: StepContext) -> torch.Tensor:
         return P.logits_f32(h, fw.router, c.bufs.get("route_z", c.t, fw.router.shape[0], dtype=torch.float32))
 
     def expert_rows(self, fw: RoutedFfWeights, h: torch.Tensor, r: R.Routing, c: StepContext) -> torch.Tensor:
         """The chosen experts' outputs, one row per (token, slot) sorted by expert."""
-        f, t, dt, pdl, ffp = fw.spec, c.t, self.dtype, c.pdl, fw.w_down.k
-        xs = c.bufs.get("xs", t, f.top, self.width_p, dtype=dt).view(t * f.top, self.width_p)
-        R.route_scatter(h, r, xs, pdl=pdl)
-        act = c.bufs.get("moe_act", t, f.top, ffp, dtype=dt).view(t * f.top, ffp)
-        y = c.bufs.get("moe_y", t, f.top, fw.w_down.n, dtype=dt).view(t * f.top, fw.w_down.n)
-        scratch = c.bufs.get("moe_gu", t, f.top, 2 * ffp, dtype=dt).view(t * f.top, 2 * ffp) if dt == torch.float32 else None
+        f, t, dt, pdl, ffp, slots = fw.spec, c.t, self.dtype, c.pdl, fw.w_down.k, r.idx.shape[1]
+        rows = lambda name, n: c.bufs.get(name, t, slots, n, dtype=dt).view(t * slots, n)      # noqa: E731
+        xs, act, y = rows("xs", self.width_p), rows("moe_act", ffp), rows("moe_y", fw.w_down.n)
+        R.route_scatter(h, r, xs, fw.always, pdl=pdl)
+        scratch = rows("moe_gu", 2 * ffp) if dt == torch.float32 else None
         R.grouped_gated_ffn(xs, r.offsets, fw.w_gu, fw.w_down, f.limit, t, scratch, act, y, pdl=pdl)
         return y
 
@@ -436,8 +440,12 @@ class RaggedModel:
             out = torch.empty(r, self.cfg.vocab_size, dtype=torch.float32, device=self.device)
         if h is None:
             h = torch.empty(r, self.width_p, dtype=self.dtype, device=self.device)
-        P.rms_norm_f32(x, w.final_norm, self.cfg.norm_eps, h, self.cfg.width, pdl=pdl)
+        self.final_rows(x, h, pdl=pdl)
         return P.logits_f32(h, w.lm_head.w, out=out)
+
+    def final_rows(self, x: torch.Tensor, h: torch.Tensor, pdl: bool = False) -> None:
+        """h = the final norm of the residual rows."""
+        P.rms_norm_f32(x, self.w.final_norm, self.cfg.norm_eps, h, self.cfg.width, pdl=pdl)
 
     # ------------------------------------------------------------------ ragged batches
     def _buffers(self, rows: int) -> Buffers:

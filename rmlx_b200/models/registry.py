@@ -116,6 +116,21 @@ def _nugosun_model(weights):
     return NugosunModel(weights)
 
 
+def _nizorax_weights(model_dir, config, device, dtype, layout):
+    from ..config import NizoraxConfig
+    from ..loader.safetensors_loader import load_tensors
+    from .nizorax import build_weights
+    if layout is not None and layout.world != 1:
+        raise ValueError("Nizorax runs on one GPU")
+    cfg = NizoraxConfig.from_json(config)
+    return build_weights(cfg, load_tensors(model_dir), device, dtype), cfg
+
+
+def _nizorax_model(weights):
+    from .nizorax import NizoraxModel
+    return NizoraxModel(weights)
+
+
 register(ModelFamily("transformer", lambda c: "num_attention_heads" in c, _transformer_weights, _transformer_model))
 register(ModelFamily("posudra", lambda c: c.get("architecture") == "Posudra", _posudra_weights, _posudra_model,
                      kernels="parallel_block"))
@@ -123,3 +138,5 @@ register(ModelFamily("rodapel", lambda c: c.get("architecture") == "Rodapel", _r
                      kernels="post_norm"))
 register(ModelFamily("nugosun", lambda c: c.get("architecture") == "Nugosun", _nugosun_weights, _nugosun_model,
                      kernels="twin_norm"))
+register(ModelFamily("nizorax", lambda c: c.get("architecture") == "Nizorax", _nizorax_weights, _nizorax_model,
+                     kernels="sandwich"))

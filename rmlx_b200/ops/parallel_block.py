@@ -27,14 +27,15 @@ _lib.register_cuda_sigs({
     "rmlx_sgemm": ("pipipiiiiip", "i"),
     "rmlx_sgemm_split_xielu": ("pipipiipiffiiiip", "i"),
     "rmlx_sgemm_scaled_add": ("pipippiiiiip", "i"),
-    "rmlx_attention_any": ("pppppppipiiiiiiiiiii" "ffpppp" "piiip", "i"),
+    "rmlx_attention_any": ("pppppppipiiiiiiiiiii" "ffpppp" "pi" "iifff" "iip", "i"),
     "rmlx_flash_prefill_scored_supported": ("ii", "i"),
     "rmlx_flash_prefill_scored": ("ppppipipiiiiiiiiffpppp" "piipip", "i"),
+    "rmlx_flash_prefill_diff": ("ppppipipiiiiiiiiiffff" "pip", "i"),
     "rmlx_flash_decode_scored_supported": ("ii", "i"),
     "rmlx_flash_decode_scored_part_o_elems": ("iiiii", "q"),
     "rmlx_flash_decode_scored_part_ml_elems": ("iiii", "q"),
     "rmlx_flash_decode_scored_ticket_elems": ("iii", "q"),
-    "rmlx_flash_decode_scored": ("ppippfpppppppppp" "iiiiiiiiiii" "ffpppp" "piii" "ppif" "ip", "i"),
+    "rmlx_flash_decode_scored": ("ppippfpppppppppp" "iiiiiiiiiii" "ffpppp" "piii" "ppif" "iifff" "ip", "i"),
 })
 
 
@@ -56,6 +57,21 @@ class ScoreMods:
     def args(self):
         return (self.scale, self.softcap, _lib.ptr(self.temp), _lib.ptr(self.r1), _lib.ptr(self.r2),
                 _lib.ptr(self.sink))
+
+
+@dataclass
+class MapDiff:
+    """Differential attention: a head's result is ``scale`` times the RMS norm of its first map's attention minus
+    ``weight`` times its second map's."""
+    weight: float
+    scale: float
+    eps: float
+
+    def args(self):
+        return (self.weight, self.scale, self.eps)
+
+
+NO_DIFF = MapDiff(0.0, 1.0, 0.0)
 
 
 def _f32(t: torch.Tensor) -> int:
@@ -239,8 +255,25 @@ def flash_prefill_scored(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
     return out
 
 
+def flash_prefill_diff(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
+                       tiles: torch.Tensor, scale: float, diff: MapDiff, vdim: int, out: torch.Tensor, window: int = 0,
+                       chunk: int = 0, pdl: bool = False) -> torch.Tensor:
+    """``flash_prefill_scored`` for differential attention: q [T, H, 2, dk], key rows of two keys, out [T, H, dv]; tiles of
+    at most 128 rows."""
+    _lib.require_cuda_tensor(q, k_cache, v_cache, block_table, tiles, out)
+    t, h, maps, dk = q.shape
+    assert maps == 2 and q.is_contiguous() and out.is_contiguous() and tiles.dtype == torch.int32 and tiles.is_contiguous()
+    assert k_cache.shape[2] == 16 and k_cache.shape[3] == 2 * dk and out.shape == (t, h, v_cache.shape[3])
+    rc = _lib.cuda().rmlx_flash_prefill_diff(
+        q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), block_table.stride(0),
+        tiles.data_ptr(), tiles.shape[0], out.data_ptr(), t, h, k_cache.shape[1], dk, v_cache.shape[3], vdim,
+        k_cache.shape[0], window, chunk, scale, *diff.args(), GemmStatus.get(q.device).data_ptr(), int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "flash_prefill_diff")
+    return out
+
+
 class ScoredDecodeScratch:
-    """Split-KV scratch of ``flash_decode_scored`` for up to ``rows`` rows."""
+    """Split-KV scratch of ``flash_decode_scored`` for up to ``rows`` rows (differential attention: twice the heads)."""
 
     def __init__(self, rows: int, heads: int, kv_heads: int, dv: int, splits: int, device):
         lib = _lib.cuda()
@@ -261,26 +294,32 @@ def flash_decode_scored(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tabl
                         table_rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None, window: int = 0,
                         gate: Optional[torch.Tensor] = None, head_norm: bool = False, gate_col: int = -1,
                         chunk: int = 0, bias: Optional[torch.Tensor] = None, inv_freq: Optional[torch.Tensor] = None,
-                        grow: float = 1.0, pdl: bool = False) -> torch.Tensor:
+                        grow: float = 1.0, neighbours: bool = False, normed: bool = True, diff: Optional[MapDiff] = None,
+                        pdl: bool = False) -> torch.Tensor:
     """One token per row: q [T, H, dk] (keys already appended) or the fused form on the un-normalised
     fp32 projection ``raw`` [T, >= q|k|v], which also appends the key and value (``head_norm``: the
     norms are per head, their weights [dim] or None; with it ``bias`` is added to the projection, and the first
-    ``2 * inv_freq.numel()`` values of query and key heads rotate, i with i + pairs, before the norm; ``gate_col``:
-    where the output gate's logits start in a row). ``rows`` int32: the batch rows to run (default: the first ``n_rows``)."""
+    ``2 * inv_freq.numel()`` values of query and key heads rotate, i with i + pairs or (``neighbours``) 2 i with 2 i + 1,
+    before the norm, which ``normed`` False leaves out; ``gate_col``: where the output gate's logits start in a row).
+    ``rows`` int32: the batch rows to run (default: the first ``n_rows``). ``diff``: differential attention, q [T, H, 2, dk]
+    or raw rows [q: H x 2 x dim | k: Hkv x 2 x dim | v] with ``head_norm``, key rows of two keys."""
     _lib.require_cuda_tensor(k_cache, v_cache, block_table, positions, out, q, raw)
     src = q if q is not None else raw
     n = rows.numel() if rows is not None else (n_rows or src.shape[0])
+    maps = 1 if diff is None else 2
+    dk = k_cache.shape[3] // maps
     assert k_cache.shape[2] == 16 and out.is_contiguous() and k_cache.dtype == torch.bfloat16
-    assert q is None or (q.is_contiguous() and q.shape[1:] == (heads, k_cache.shape[3]))
+    assert q is None or (q.is_contiguous() and q.shape[1:] == ((heads, dk) if maps == 1 else (heads, 2, dk)))
     assert raw is None or raw.dtype == torch.float32
     rc = _lib.cuda().rmlx_flash_decode_scored(
         _lib.ptr(q), _lib.ptr(raw), 0 if raw is None else raw.stride(0), _lib.ptr(q_w), _lib.ptr(k_w), eps,
         k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), positions.data_ptr(), _lib.ptr(rows),
         _lib.ptr(table_rows), out.data_ptr(), scratch.part_o.data_ptr(), scratch.part_ml.data_ptr(),
-        scratch.tickets.data_ptr(), n, heads, k_cache.shape[1], dim, vdim, k_cache.shape[3], v_cache.shape[3],
+        scratch.tickets.data_ptr(), n, heads, k_cache.shape[1], dim, vdim, dk, v_cache.shape[3],
         block_table.stride(0), scratch.splits, window, chunk, *mods.args(),
-        *_gate_args(gate, 0 if q is None else q.shape[0], heads, torch.bfloat16), int(head_norm), gate_col,
-        _lib.ptr(bias), _lib.ptr(inv_freq), 0 if inv_freq is None else 2 * inv_freq.numel(), grow, int(pdl), _lib.stream_ptr())
+        *_gate_args(gate, 0 if q is None else q.shape[0], heads, torch.bfloat16), (1 if normed else 2) if head_norm else 0,
+        gate_col, _lib.ptr(bias), _lib.ptr(inv_freq), 0 if inv_freq is None else 2 * inv_freq.numel(), grow, int(neighbours), maps,
+        *(diff or NO_DIFF).args(), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "flash_decode_scored")
     return out
 
@@ -288,18 +327,21 @@ def flash_decode_scored(k_cache: torch.Tensor, v_cache: torch.Tensor, block_tabl
 def attention_any(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                   positions: torch.Tensor, token_seq: Optional[torch.Tensor], mods: ScoreMods, out: torch.Tensor,
                   window: int = 0, gate: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
-                  chunk: int = 0, pdl: bool = False) -> torch.Tensor:
+                  chunk: int = 0, diff: Optional[MapDiff] = None, vdim: int = 0, pdl: bool = False) -> torch.Tensor:
     """Attention of single query tokens over pages for any head widths, bf16 or fp32 storage. Cache rows
     may be wider than the query (key) and the output (value): ``k_cache`` and ``v_cache`` may be one
-    pool whose rows hold both (latent attention). ``rows``: batch rows to run (default: all)."""
+    pool whose rows hold both (latent attention). ``rows``: batch rows to run (default: all). ``diff``: differential
+    attention, q [T, H, 2, dk], key rows of two keys, heads of ``vdim`` values."""
     _lib.require_cuda_tensor(q, k_cache, v_cache, block_table, positions, token_seq, out)
-    t, h, dk = q.shape
-    assert q.is_contiguous() and out.is_contiguous() and q.dtype == k_cache.dtype == out.dtype
-    assert k_cache.shape[3] >= dk and out.shape[:2] == (t, h) and v_cache.shape[3] >= out.shape[2]
+    t, h, dk = q.shape[0], q.shape[1], q.shape[-1]
+    maps = 1 if diff is None else 2
+    assert q.dim() == 2 + maps and q.is_contiguous() and out.is_contiguous() and q.dtype == k_cache.dtype == out.dtype
+    assert k_cache.shape[3] >= maps * dk and out.shape[:2] == (t, h) and v_cache.shape[3] >= out.shape[2]
     rc = _lib.cuda().rmlx_attention_any(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), positions.data_ptr(),
         _lib.ptr(token_seq), _lib.ptr(rows), 0 if rows is None else rows.numel(), out.data_ptr(), t, h,
         k_cache.shape[1], dk, out.shape[2], k_cache.shape[3], v_cache.shape[3], block_table.stride(0),
-        k_cache.shape[2], window, chunk, *mods.args(), *_gate_args(gate, t, h, q.dtype), _f32(q), int(pdl), _lib.stream_ptr())
+        k_cache.shape[2], window, chunk, *mods.args(), *_gate_args(gate, t, h, q.dtype), maps, vdim,
+        *(diff or NO_DIFF).args(), _f32(q), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "attention_any")
     return out

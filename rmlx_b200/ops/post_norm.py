@@ -201,6 +201,19 @@ def postnorm_gated(x: torch.Tensor, pending: Pending, eps: float, width: int, x_
         _lib.check(rc, "postnorm_gated")
 
 
+def rows_in(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, pdl: bool = False) -> torch.Tensor:
+    """out = x w^T of a few finished fp32 rows (``postnorm_in`` with nothing pending)."""
+    _lib.require_cuda_tensor(x, w, out)
+    b, k = x.shape
+    assert x.dtype == out.dtype == torch.float32 and w.dtype == torch.bfloat16 and w.is_contiguous() and w.shape[1] == k
+    assert x.is_contiguous() and out.shape == (b, w.shape[0])
+    for lo, hi in _chunks(b, k):
+        rc = _lib.cuda().rmlx_postnorm_in(w.data_ptr(), x[lo:].data_ptr(), None, None, 0.0, None, k, k, None, None, None, 0, 0,
+                                          out[lo:].data_ptr(), out.stride(0), hi - lo, w.shape[0], int(pdl), _lib.stream_ptr())
+        _lib.check(rc, "postnorm_in")
+    return out
+
+
 def matvec_out(a: torch.Tensor, w: torch.Tensor, y: torch.Tensor, pdl: bool = False) -> torch.Tensor:
     """y = a w^T, bf16 in, fp32 out, a few rows."""
     _lib.require_cuda_tensor(a, w, y)

@@ -1,5 +1,5 @@
-"""Routing by corrected scores with identity experts, or by biased logits with the softmax over the chosen
-experts (csrc/kernels/moe_route.cu), and the grouped expert
+"""Routing by corrected scores with identity experts, by biased logits with the softmax over the chosen
+experts, or by sigmoids among the best groups beside experts that every token uses (csrc/kernels/moe_route.cu), and the grouped expert
 feed-forward around it for any number of tokens: route -> rows sorted by expert -> gate/up with the gated
 activation -> down. The combination with the output norm is ``combine_post_norm`` (postnorm_rows.cu)."""
 from __future__ import annotations
@@ -22,7 +22,9 @@ _lib.register_cuda_sigs({
     "rmlx_route_max_top": ("", "i"),
     "rmlx_route_corrected": ("pippppppiiiiip", "i"),
     "rmlx_route_chosen": ("pippppp" "iiiip", "i"),
-    "rmlx_route_scatter": ("pipppp" "iiiiip", "i"),
+    "rmlx_route_grouped": ("pipppp" "iiiiiifip", "i"),
+    "rmlx_grouped_router": ("ppipppp" "iiiiiifip", "i"),
+    "rmlx_route_scatter": ("pipppp" "iiiiiip", "i"),
     "rmlx_moe_combine_post_norm": ("pipppipfppiiiiip", "i"),
     "rmlx_postnorm_router": ("ppppfpii" "pppppp" "iiiiip", "i"),
     "rmlx_postnorm_expert": ("ppippiiiiifip", "i"),
@@ -67,13 +69,37 @@ def route_chosen(logits: torch.Tensor, bias: torch.Tensor, r: Routing, grouped: 
     _lib.check(rc, "route_chosen")
 
 
-def route_scatter(h: torch.Tensor, r: Routing, xs: torch.Tensor, pdl: bool = False) -> None:
-    """Copies every routed (token, slot) row of ``h`` into ``xs`` [T * top, width], sorted by expert."""
+@dataclass
+class RouteGroups:
+    """Groups of neighbouring experts of which a token may use the ``keep`` best; the weights' factor; how many experts
+    behind the routed ones every token uses, with weight one."""
+    count: int = 1
+    keep: int = 1
+    scale: float = 1.0
+    always: int = 0
+
+
+def route_grouped(logits: torch.Tensor, g: RouteGroups, r: Routing, grouped: bool = True, pdl: bool = False) -> None:
+    """Chooses by sigmoid(logits) within the groups whose two largest have the largest sums; weights: the sigmoids times
+    ``g.scale``. ``r`` has room for the chosen and the ``g.always`` experts."""
+    _lib.require_cuda_tensor(logits, r.idx)
+    t, experts = logits.shape
+    assert logits.dtype == torch.float32 and r.counts.numel() == experts + g.always
+    rc = _lib.cuda().rmlx_route_grouped(
+        logits.data_ptr(), logits.stride(0), r.idx.data_ptr(), r.weights.data_ptr(), r.counts.data_ptr() if grouped else None,
+        r.offsets.data_ptr() if grouped else None, t, experts, r.idx.shape[1] - g.always, g.count, g.keep, g.always, g.scale,
+        int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "route_grouped")
+
+
+def route_scatter(h: torch.Tensor, r: Routing, xs: torch.Tensor, always: int = 0, pdl: bool = False) -> None:
+    """Copies every routed (token, slot) row of ``h`` into ``xs`` [T * top, width], sorted by expert. ``always``: how many
+    of the experts (the last ones) have every token's row."""
     _lib.require_cuda_tensor(h, xs)
     t, top = r.idx.shape
     assert h.is_contiguous() and xs.is_contiguous() and xs.shape == (t * top, h.shape[1]) and xs.dtype == h.dtype
     rc = _lib.cuda().rmlx_route_scatter(h.data_ptr(), h.stride(0), r.idx.data_ptr(), r.counts.data_ptr(), xs.data_ptr(),
-                                        r.row_of_pair.data_ptr(), t, top, r.counts.numel(), _f32(h), int(pdl),
+                                        r.row_of_pair.data_ptr(), t, top, r.counts.numel(), always, _f32(h), int(pdl),
                                         _lib.stream_ptr())
     _lib.check(rc, "route_scatter")
 
@@ -129,6 +155,21 @@ def postnorm_router(x: torch.Tensor, pending: Pending, eps: float, width: int, x
         _lib.check(rc, "postnorm_router")
 
 
+def grouped_router(h: torch.Tensor, w: torch.Tensor, g: RouteGroups, logits: torch.Tensor, ticket: torch.Tensor, r: Routing,
+                   pdl: bool = False) -> None:
+    """Router logits of finished rows (fp32) and ``route_grouped``'s choice. ``ticket``: one int32 word, zero."""
+    _lib.require_cuda_tensor(h, w, logits, ticket)
+    b, k = h.shape
+    assert h.dtype == torch.float32 and h.is_contiguous() and w.dtype == torch.bfloat16 and w.is_contiguous() and w.shape[1] == k
+    assert logits.is_contiguous()
+    for lo, hi in _chunks(b, k):
+        rc = _lib.cuda().rmlx_grouped_router(
+            w.data_ptr(), h[lo:].data_ptr(), k, logits[lo:].data_ptr(), r.idx[lo:].data_ptr(), r.weights[lo:].data_ptr(),
+            ticket.data_ptr(), hi - lo, w.shape[0], r.idx.shape[1] - g.always, g.count, g.keep, g.always, g.scale, int(pdl),
+            _lib.stream_ptr())
+        _lib.check(rc, "grouped_router")
+
+
 def postnorm_expert(x: torch.Tensor, w: torch.Tensor, limit: float, r: Routing, act: torch.Tensor, pdl: bool = False) -> None:
     """act [B * top, n] = gated activation of the chosen experts' [gate; up] projections of x (fp32)."""
     _lib.require_cuda_tensor(x, w, act)
@@ -140,13 +181,13 @@ def postnorm_expert(x: torch.Tensor, w: torch.Tensor, limit: float, r: Routing, 
 
 
 def expert_out(act: torch.Tensor, w: torch.Tensor, r: Routing, x: torch.Tensor, y: torch.Tensor, pdl: bool = False) -> None:
-    """y = sum of the slots' weighted down projections + identity weight * x."""
+    """y = sum of the slots' weighted down projections + identity weight * x (without identity weights: the sum alone)."""
     _lib.require_cuda_tensor(act, w, x, y)
     e, rows, k = w.shape
     b, ldx = x.shape
     assert y.shape == x.shape and act.stride(0) >= k and w.is_contiguous()
     rc = _lib.cuda().rmlx_expert_out(w.data_ptr(), rows, k, act.data_ptr(), act.stride(0), r.idx.data_ptr(),
-                                     r.weights.data_ptr(), r.identity.data_ptr(), x.data_ptr(), y.data_ptr(), ldx, b, ldx,
+                                     r.weights.data_ptr(), _lib.ptr(r.identity), x.data_ptr(), y.data_ptr(), ldx, b, ldx,
                                      r.idx.shape[1], e, int(pdl), _lib.stream_ptr())
     _lib.check(rc, "expert_out")
 

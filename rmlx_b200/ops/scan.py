@@ -1,5 +1,6 @@
-"""Linear recurrences token by token (csrc/kernels/linear_scan.cu): gated linear attention and state-space heads with
-their short convolution, and the norm of their outputs with a silu gate; their decode steps (twin_norm_gemv.cu). A sequence's state is its slot's row of a
+"""Linear recurrences token by token (csrc/kernels/linear_scan.cu): gated linear attention, state-space heads with
+their short convolution, lightning attention, and the norm of their outputs with a gate; their decode steps
+(twin_norm_gemv.cu, sandwich_gemv.cu). A sequence's state is its slot's row of a
 flat fp32 pool (``PagedKvCache.layer_state`` views)."""
 from __future__ import annotations
 
@@ -21,7 +22,9 @@ _lib.register_cuda_sigs({
     "rmlx_gla_decode_supported": ("ii", "i"),
     "rmlx_gla_decode": ("piiiii" "pipff" "pfp" "pq" "pi" "iiiiip", "i"),
     "rmlx_ssd_decode": ("piii" "ppi" "ppppp" "pq" "pi" "pfi" "pi" "iiiii" "ip", "i"),
-    "rmlx_gated_norm": ("pipipfpi" "iiiiiip", "i"),
+    "rmlx_lightning_scan": ("pppip" "pippi" "pqpi" "iiii" "pip", "i"),
+    "rmlx_lightning_step": ("piii" "ppp" "q" "pi" "iiii" "ip", "i"),
+    "rmlx_gated_norm": ("pipipfpi" "iiiiiiip", "i"),
 })
 
 
@@ -80,15 +83,33 @@ def ssd_scan(raw: torch.Tensor, x_at: int, dt_at: int, conv_w: torch.Tensor, con
     _lib.check(rc, "ssd_scan")
 
 
+def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+                   rec: torch.Tensor, runs: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None,
+                   pdl: bool = False) -> None:
+    """S <- decay S + silu(k) silu(v)^T, out = S^T silu(q) with one constant decay per head (fp32 [H]); ``rec``: scratch of
+    T * H * ``record(dim, vdim, True)`` floats, the rest as in ``gla_scan``."""
+    _lib.require_cuda_tensor(q, k, v, decay, state, out, rec, runs, slots)
+    _, h, n, d = state.shape
+    t = q.shape[0]
+    assert q.stride(0) == k.stride(0) == v.stride(0) and q.dtype == k.dtype == v.dtype
+    assert decay.dtype == out.dtype == state.dtype == torch.float32 and state.stride()[1:] == (n * d, d, 1)
+    assert decay.numel() == h and rec.is_contiguous() and rec.numel() >= t * h * record(n, d, True)
+    rc = _lib.cuda().rmlx_lightning_scan(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), decay.data_ptr(), rec.data_ptr(), t, _lib.ptr(runs), _lib.ptr(slots),
+        _segments(runs, slots), state.data_ptr(), state.stride(0), out.data_ptr(), out.stride(0), h, n, d, _f32(q),
+        GemmStatus.get(q.device).data_ptr(), int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "lightning_scan")
+
+
 def gated_norm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float, groups: int, out: torch.Tensor,
-               gate_first: bool, pdl: bool = False) -> torch.Tensor:
-    """RMS norm of the first ``w.numel()`` columns in ``groups`` equal parts, times w, with silu(gate) multiplied
-    before (``gate_first``) or after the norm."""
+               gate_first: bool, sigmoid: bool = False, pdl: bool = False) -> torch.Tensor:
+    """RMS norm of the first ``w.numel()`` columns in ``groups`` equal parts, times w, with silu(gate) (``sigmoid``:
+    sigmoid(gate)) multiplied before (``gate_first``) or after the norm."""
     _lib.require_cuda_tensor(o, gate, w, out)
     assert o.dtype == w.dtype == torch.float32 and gate.dtype == out.dtype and w.numel() % groups == 0
     rc = _lib.cuda().rmlx_gated_norm(o.data_ptr(), o.stride(0), gate.data_ptr(), gate.stride(0), w.data_ptr(), eps,
                                      out.data_ptr(), out.stride(0), o.shape[0], groups, w.numel() // groups, int(gate_first),
-                                     _f32(out), int(pdl), _lib.stream_ptr())
+                                     int(sigmoid), _f32(out), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "gated_norm")
     return out
 
@@ -131,3 +152,16 @@ def ssd_decode(raw: torch.Tensor, x_at: int, dt_at: int, conv_w: torch.Tensor, c
         state.data_ptr(), state.stride(0), y.data_ptr(), y.stride(0), norm.data_ptr(), eps, norm_groups, out.data_ptr(),
         out.stride(0), raw.shape[0], h, groups, n, d, int(pdl), _lib.stream_ptr())
     _lib.check(rc, "ssd_decode")
+
+
+def lightning_step(raw: torch.Tensor, at_k: int, at_v: int, decay: torch.Tensor, slots: torch.Tensor, state: torch.Tensor,
+                   out: torch.Tensor, pdl: bool = False) -> None:
+    """One token per row of ``lightning_scan``: raw fp32 [B, ..] = q at 0, k and v at their columns; out fp32 [B, >= H vdim]."""
+    _lib.require_cuda_tensor(raw, decay, slots, state, out)
+    _, h, n, d = state.shape
+    assert raw.dtype == out.dtype == decay.dtype == torch.float32 and state.stride()[1:] == (n * d, d, 1)
+    assert slots.dtype == torch.int32 and decay.numel() == h
+    rc = _lib.cuda().rmlx_lightning_step(
+        raw.data_ptr(), raw.stride(0), at_k, at_v, decay.data_ptr(), slots.data_ptr(), state.data_ptr(), state.stride(0),
+        out.data_ptr(), out.stride(0), raw.shape[0], h, n, d, int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "lightning_step")

@@ -17,18 +17,25 @@ _lib.register_cuda_sigs({
     "rmlx_twin_in_max_rows": ("i", "i"),
     "rmlx_twin_in_gated": ("pppfii" "pipi" "pipif" "iip", "i"),
     "rmlx_twin_in_router": ("pppfii" "pipi" "ppipp" "ppip" "iip", "i"),
-    "rmlx_rotary_norm_append": ("piippiff" "ppp" "ppp" "iiiiiiiiiiip", "i"),
+    "rmlx_rotary_norm_append": ("piippiff" "ppp" "ppp" "iiiiiiiii" "iii" "iip", "i"),
 })
 
 
 def rotary_frequencies(base: float, dims: int, scaling: Optional[dict] = None) -> Tuple[torch.Tensor, float]:
     """(angle per position of every pair, fp64 [dims / 2]; factor of cos and sin). ``scaling``: YaRN (factor, original,
     fast, slow) - pairs that turn more than ``fast`` times over ``original`` positions keep their speed, those below
-    ``slow`` turns are slowed by ``factor``, with a ramp between."""
+    ``slow`` turns are slowed by ``factor``, with a ramp over the pairs between - or Llama's (factor, original, high, low):
+    the same by ``high`` and ``low`` turns, with a ramp over the turns and no factor of cos and sin."""
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = base ** (-2.0 * i / max(dims, 1))
     if not scaling:
         return f, 1.0
+    if "high" in scaling:
+        turns = scaling["original"] * f / (2 * math.pi)
+        s = (turns - scaling["low"]) / (scaling["high"] - scaling["low"])
+        mixed = (1 - s) * f / scaling["factor"] + s * f
+        slow = torch.where(turns < scaling["low"], f / scaling["factor"], mixed)
+        return torch.where(turns > scaling["high"], f, slow), 1.0
     def dim_of(turns):
         return dims * math.log(scaling["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
     lo = max(math.floor(dim_of(scaling["fast"])), 0)
@@ -70,18 +77,22 @@ def rows_norm(x: torch.Tensor, w: torch.Tensor, eps: float, width: int, out: tor
 def rotary_norm_append(raw: torch.Tensor, bias: Optional[torch.Tensor], inv_freq: torch.Tensor, grow: float, eps: float,
                        q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                        positions: torch.Tensor, token_seq: Optional[torch.Tensor], heads: int, dim: int, vdim: int,
-                       pdl: bool = False) -> None:
-    """raw [T, q | k | v] + bias: queries and keys rotated (value i with value i + pairs, cos and sin times ``grow``) and
-    divided by their root mean square per head; queries to ``q``, keys / values to their pages."""
+                       neighbours: bool = False, norm: bool = True, maps: int = 1, pdl: bool = False) -> None:
+    """raw [T, q | k | v] + bias: queries and keys rotated (value i with value i + pairs, or (``neighbours``) 2 i with 2 i + 1;
+    cos and sin times ``grow``) and (``norm``) divided by their root mean square per head; queries to ``q``, keys / values
+    to their pages. ``maps`` 2 (differential attention): query and key heads of two parts of ``dim`` values, q [T, heads, 2,
+    ..], cache rows of two keys."""
     _lib.require_cuda_tensor(raw, bias, inv_freq, q, k_cache, v_cache, block_table, positions, token_seq)
     t, hkv = raw.shape[0], k_cache.shape[1]
-    assert q.shape == (t, heads, k_cache.shape[3]) and q.dtype == k_cache.dtype == v_cache.dtype
-    assert bias is None or (bias.dtype == torch.float32 and bias.numel() >= (heads + hkv) * dim + hkv * vdim)
+    dkp = k_cache.shape[3] // maps
+    assert q.shape == ((t, heads, dkp) if maps == 1 else (t, heads, maps, dkp)) and q.is_contiguous()
+    assert q.dtype == k_cache.dtype == v_cache.dtype
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() >= (heads + hkv) * maps * dim + hkv * vdim)
     rc = _lib.cuda().rmlx_rotary_norm_append(
         raw.data_ptr(), raw.stride(0), _f32(raw), _lib.ptr(bias), inv_freq.data_ptr(), 2 * inv_freq.numel(), grow, eps,
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr(), positions.data_ptr(),
-        _lib.ptr(token_seq), t, heads, hkv, dim, vdim, k_cache.shape[3], v_cache.shape[3], block_table.stride(0),
-        k_cache.shape[2], _f32(q), int(pdl), _lib.stream_ptr())
+        _lib.ptr(token_seq), t, heads, hkv, dim, vdim, dkp, v_cache.shape[3], block_table.stride(0),
+        k_cache.shape[2], int(neighbours), int(norm), maps, _f32(q), int(pdl), _lib.stream_ptr())
     _lib.check(rc, "rotary_norm_append")
 
 
