@@ -55,11 +55,12 @@ def parse():
     ap.add_argument("--arms", default="auto",
                     help="comma list of extra arms: bf16, nccl_cublas; 'auto' = both from 2 GPUs on, "
                          "'none' = headline only")
-    ap.add_argument("--suite", default="headline", choices=["headline", "parallel_block", "post_norm", "twin_norm"],
+    ap.add_argument("--suite", default="headline", choices=["headline", "parallel_block", "post_norm", "twin_norm", "sandwich"],
                     help="parallel_block: the parallel-block decoder beside the dense one at equal size; "
                          "post_norm: the post-norm decoder beside the mixture-of-experts one; twin_norm: the "
-                         "twin-norm decoder beside the post-norm one (benchmarks/bench_<suite>.py, which take the "
-                         "remaining options); the default is the headline workload")
+                         "twin-norm decoder beside the post-norm one; sandwich: the sandwich-norm decoder beside the "
+                         "post-norm one (benchmarks/bench_<suite>.py, which take the remaining "
+                         "options); the default is the headline workload")
     args, rest = ap.parse_known_args()
     if args.suite == "headline" and rest:
         ap.error(f"unrecognized arguments: {' '.join(rest)}")
@@ -334,6 +335,10 @@ def main():
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "benchmarks"))
         import bench_twin_norm
         return bench_twin_norm.main(args.rest)
+    if args.suite == "sandwich":
+        sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "benchmarks"))
+        import bench_sandwich
+        return bench_sandwich.main(args.rest)
     world = int(os.environ.get("WORLD_SIZE", "1"))
     if args.gpus != world and world == 1 and args.gpus > 1:
         print(f"bench.py: --gpus {args.gpus} needs torchrun with {args.gpus} ranks", file=sys.stderr)

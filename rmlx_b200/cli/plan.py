@@ -230,16 +230,19 @@ def _plan_layered(c, shapes: dict, kv_shapes, state_shapes, row: int, batch: int
     per prompt token beside the expanded latents."""
     from ..config import LatentAttentionSpec
     parts = {"attention": 0, "feed_forward": 0, "norms": 0, "embedding": 0, "lm_head": 0}
-    routed, active = 0, 0
+    routed, active, again = 0, 0, 0
+    passes = [getattr(c, "runs", list(range(len(c.layers)))).count(i) for i in range(len(c.layers))]
     for name, shape in shapes.items():
         n = math.prod(shape)
+        if name[0] == "l" and ".mlp.e" not in name and len(shape) > 1:   # weights that a looped layer reads once more per pass
+            again += (passes[int(name[1:name.index(".")])] - 1) * n * 2
         part = {"embed": "embedding", "head": "lm_head"}.get(name) or (
             "norms" if len(shape) == 1 else "feed_forward" if ".mlp." in name else "attention")
         parts[part] += n * (4 if len(shape) == 1 else 2)               # per-channel vectors are kept in fp32
         routed += n * 2 if ".mlp.e" in name else 0
-    for l in c.layers:
+    for l, times in zip(c.layers, passes):
         if hasattr(l.mlp, "top"):
-            active += min(l.mlp.experts, batch * l.mlp.top) * 3 * l.mlp.ff * c.width * 2
+            active += times * min(l.mlp.experts, batch * l.mlp.top) * 3 * l.mlp.ff * c.width * 2
     parts["total"] = sum(parts.values())
     head = parts["lm_head"] or parts["embedding"]                      # a step reads the table once as the LM head
     kv_tok = sum(s[0] * (s[1] + s[2]) * 2 for s in kv_shapes if s is not None)
@@ -249,7 +252,7 @@ def _plan_layered(c, shapes: dict, kv_shapes, state_shapes, row: int, batch: int
                       for l in c.layers if l.mlp is not None])
     scratch = prefill_chunk * row + ctx * max([0] + [2 * (m.heads * (m.dim + m.vdim) + m.kv_rank) for m in lat])
     budget, need = int(HBM_BYTES * budget_fraction), batch * (ctx * kv_tok + state)
-    step = parts["attention"] + parts["feed_forward"] - routed + active + need + head
+    step = parts["attention"] + parts["feed_forward"] - routed + again + active + need + head
     hbm = decode_hbm_gbs()
     layer = (step - head) / c.num_layers
     return {
@@ -297,6 +300,23 @@ def plan_nugosun(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, bud
     return _plan_layered(c, tensor_shapes(c), kv_shapes(c), state_shapes(c), row, batch, ctx, prefill_chunk, budget_fraction)
 
 
+def plan_nizorax(batch: int = 1, ctx: int = 4096, prefill_chunk: int = 2048, budget_fraction: float = 0.90,
+                 cfg=None) -> dict:
+    """A Nizorax model (bf16, one GPU): pages for the attention runs, matrix states and carried convolution inputs per
+    sequence, the widest activations of a prompt chunk (with the recurrence's records)."""
+    from ..config import LightningSpec
+    from ..models.nizorax import kv_shapes, nizorax_4096, state_shapes, tensor_shapes
+    c = cfg or nizorax_4096()
+
+    def mixer(m) -> int:
+        if isinstance(m, LightningSpec):   # projection, fp32 output, records, gated rows
+            return m.heads * (2 * (2 * m.dim + 2 * m.vdim) + 6 * m.vdim + 4 * (2 * max(16, m.dim) + 2 * m.vdim))
+        return 2 * (2 * (2 * m.heads + m.kv_heads) * m.dim + (m.heads + m.kv_heads) * m.vdim)
+
+    row = 10 * c.width + max(mixer(l.mixer) for l in c.layers)
+    return _plan_layered(c, tensor_shapes(c), kv_shapes(c), state_shapes(c), row, batch, ctx, prefill_chunk, budget_fraction)
+
+
 def plan(model: str = "moe-a22b", weights: str = "q4", tp: int = 1, batch: int = 1, ctx: int = 4096,
          kv_quant: Optional[str] = None, expert_parallel: bool = False, prefill_chunk: int = 2048,
          budget_fraction: float = 0.90, cfg: Optional[TransformerConfig] = None) -> dict:
@@ -314,6 +334,10 @@ def plan(model: str = "moe-a22b", weights: str = "q4", tp: int = 1, batch: int =
         if weights != "bf16" or tp != 1 or kv_quant is not None:
             raise ValueError("Nugosun runs on one GPU with bf16 weights and cache")
         return plan_nugosun(batch, ctx, prefill_chunk, budget_fraction)
+    if model == "nizorax-4096" and cfg is None:
+        if weights != "bf16" or tp != 1 or kv_quant is not None:
+            raise ValueError("Nizorax runs on one GPU with bf16 weights and cache")
+        return plan_nizorax(batch, ctx, prefill_chunk, budget_fraction)
     cfg = cfg or presets()[model]
     w = weight_bytes_per_gpu(cfg, weights, tp, expert_parallel)
     kv_tok = kv_bytes_per_token_per_gpu(cfg, tp, kv_quant)
@@ -377,7 +401,8 @@ def render(p: dict) -> str:
 
 def main(argv: Optional[Sequence[str]] = None) -> int:
     ap = argparse.ArgumentParser(prog="rmlx plan", description=__doc__.split("\n\n")[0])
-    ap.add_argument("--model", default="moe-a22b", choices=sorted(presets()) + ["deepseek-v3", "posudra-8b", "rodapel-4096", "nugosun-4096"])
+    ap.add_argument("--model", default="moe-a22b", choices=sorted(presets()) + ["deepseek-v3", "posudra-8b", "rodapel-4096", "nugosun-4096",
+                                                                                           "nizorax-4096"])
     ap.add_argument("--weights", default="q4", choices=sorted(BITS))
     ap.add_argument("--tp", type=int, default=1)
     ap.add_argument("--expert-parallel", action="store_true")

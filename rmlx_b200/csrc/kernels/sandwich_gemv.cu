@@ -78,7 +78,7 @@ struct GatedSource {
       for (int i = 0; i < 8; ++i) {
         const bool in = c * 8 + i < D;
         ssq += in ? f[i] * f[i] : 0.f;
-        f[i] = in ? f[i] * w[c * 8 + i] / (1.f + expf(-g[i])) : 0.f;
+        f[i] = in ? __fdividef(f[i] * w[c * 8 + i], 1.f + __expf(fminf(-g[i], 80.f))) : 0.f;
       }
       dst[c] = make_float4(f[0], f[1], f[2], f[3]);
       dst[chunks + c] = make_float4(f[4], f[5], f[6], f[7]);

@@ -4,18 +4,15 @@
 //                  sublayer that follows, in one pass
 //   short_conv     h + causal depthwise convolution of h over time, the last inputs carried per sequence
 //   poly_norm      a N(z) + b N(z^2) + c N(z^3) + e, N: division by the row's root mean square
-//   sandwich_step  a decode row through all of the first two: a cluster per row
+//   sandwich_step  decode rows through both of the first two in one launch
 //
 // LN(v) = (v - mean) / sqrt(mean((v - mean)^2) + eps) * w + b. Activations are bf16 (serving) or fp32 (the all-32-bit
 // mode); norms, convolutions and the residual are fp32 in both.
-#include <cooperative_groups.h>
 #include <type_traits>
 
 #include "../common/launch.cuh"
 #include "../common/row_sources.cuh"
 #include "../common/rows.cuh"
-
-namespace cg = cooperative_groups;
 
 namespace rb {
 
@@ -29,130 +26,236 @@ struct Affine {
   }
 };
 
-// x[t] += LN(source; wy); h[t] = LN(x[t]; wh) (h may be null). Columns past D are zero. KEEP chunks of eight a thread keeps;
-// rows wider than KEEP * 8 * 256 are read again.
-template <class SRC, bool ADD, class T, int KEEP>
-__global__ void __launch_bounds__(kRowThreads)
-sandwich_norm_kernel(SRC src, Affine wy, float* __restrict__ x, Affine wh, T* __restrict__ h, float eps, int D, int ldx) {
-  __shared__ float red[kRowThreads / 32];
+// A warp's share of a row: how many values, their mean, and the sum of their squared deviations from it. Shares of several
+// warps are joined by the deviations of the means, so nothing cancels and a block needs one barrier per norm.
+struct Share {
+  float n, mean, m2;
+};
+template <int WARPS>
+__device__ __forceinline__ void join_shares(const Share (&s)[WARPS], float total, float eps, float& mean, float& inv) {
+  float m = 0.f, q = 0.f;
+#pragma unroll
+  for (int w = 0; w < WARPS; ++w) m = fmaf(s[w].n, s[w].mean, m);
+  mean = m / total;
+#pragma unroll
+  for (int w = 0; w < WARPS; ++w) {
+    const float d = s[w].mean - mean;
+    q += fmaf(s[w].n * d, d, s[w].m2);
+  }
+  inv = 1.f / sqrtf(q / total + eps);
+}
+
+// Eight values as they are stored; rows pass through once, so their loads leave the first-level cache to the weights.
+template <class T>
+struct Packed;
+template <>
+struct Packed<__nv_bfloat16> {
+  uint4 v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = __ldcs(reinterpret_cast<const uint4*>(p)); }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+    f[0] = bf16lo(v.x); f[1] = bf16hi(v.x); f[2] = bf16lo(v.y); f[3] = bf16hi(v.y);
+    f[4] = bf16lo(v.z); f[5] = bf16hi(v.z); f[6] = bf16lo(v.w); f[7] = bf16hi(v.w);
+  }
+};
+template <>
+struct Packed<float> {
+  float v[8];
+  __device__ __forceinline__ void load(const float* p) {
+    const float4 a = __ldcs(reinterpret_cast<const float4*>(p)), b = __ldcs(reinterpret_cast<const float4*>(p + 4));
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) f[i] = v[i];
+  }
+};
+
+// What a thread keeps of the rows it norms.
+template <class SRC>
+struct Kept {
+  Packed<float> p;
+  __device__ __forceinline__ void load(const SRC& src, int t, int c) {
+    const float none[8] = {};
+    src.load(t, c, none, p.v);
+  }
+};
+template <class TY>
+struct Kept<RowSource<TY>> {
+  Packed<TY> p;
+  __device__ __forceinline__ void load(const RowSource<TY>& src, int t, int c) { p.load(src.y + size_t(t) * src.ldy + c * 8); }
+};
+
+// x[t] += LN(source; wy); h[t] = LN(x[t]; wh) (h may be null) for R rows a block. Columns past D are zero in the source, x
+// and the weights, so they stay zero, add nothing to a sum, and mean^2 each to a sum of squared deviations. KEEP chunks of
+// eight a thread keeps; rows wider than KEEP * 8 * 256 are read again.
+template <class SRC, bool ADD, class T, int KEEP, int R, int BLOCKS>
+__global__ void __launch_bounds__(kRowThreads, BLOCKS)
+sandwich_norm_kernel(SRC src, Affine wy, float* __restrict__ x, Affine wh, T* __restrict__ h, float eps, int rows, int D, int ldx) {
+  constexpr int kWarps = kRowThreads / 32;
+  __shared__ Share part[2][R][kWarps];
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, chunks = ldx >> 3;
-  float* row = x + size_t(t) * ldx;
-  if constexpr (ADD) src.prepare(t);
-  const float none[8] = {};
-  float f[KEEP][8];
-  // mean and 1 / deviation of the values that get(c, .) gives; keep[] holds the first ones
-  auto moments = [&](float (&keep)[KEEP][8], auto get, float& mean, float& inv) {
-    float sum = 0.f;
+  const int t0 = blockIdx.x * R, chunks = ldx >> 3;
+  auto row = [&](int r) { return min(t0 + r, rows - 1); };         // (a last odd row is done twice, the copy not stored)
+  auto chunk = [&](int u) { return u * kRowThreads + threadIdx.x; };
+  SRC from[R];
 #pragma unroll
-    for (int u = 0; u < KEEP; ++u) {
-      const int c = u * kRowThreads + threadIdx.x;
-      if (c < chunks) {
+  for (int r = 0; r < R; ++r) {
+    from[r] = src;
+    if constexpr (ADD) from[r].prepare(row(r));
+  }
+  Packed<float> f[R][KEEP];
+  float count = 0.f, pads = 0.f;
+  for (int c = threadIdx.x; c < chunks; c += kRowThreads) {
+    const int n = max(0, min(8, D - c * 8));
+    count += float(n);
+    pads += float(8 - n);
+  }
+  count = warp_sum(count);
+  pads = warp_sum(pads);
+  // mean and 1 / deviation of the rows; keep[] holds a row's first chunks, get(r, c, .) gives the others
+  auto moments = [&](auto& keep, auto get, Share (&mine)[R][kWarps], float (&mean)[R], float (&inv)[R]) {
+    float v[R];
+    auto each = [&](auto use) {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) sum += c * 8 + i < D ? keep[u][i] : 0.f;
-      }
-    }
-    for (int c = KEEP * kRowThreads + threadIdx.x; c < chunks; c += kRowThreads) {
-      float a[8];
-      get(c, a);
+      for (int u = 0; u < KEEP; ++u)
+        if (chunk(u) < chunks) {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) sum += c * 8 + i < D ? a[i] : 0.f;
-    }
-    mean = row_block_sum(sum, red) / float(D);
-    float ssq = 0.f;
-    auto dev = [&](int c, const float (&a)[8]) {
+          for (int r = 0; r < R; ++r) {
+            float a[8];
+            keep(r, u, a);
+            use(r, a);
+          }
+        }
+      for (int c = chunk(KEEP); c < chunks; c += kRowThreads)
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+          float a[8];
+          get(r, c, a);
+          use(r, a);
+        }
+    };
+#pragma unroll
+    for (int r = 0; r < R; ++r) v[r] = 0.f;
+    each([&](int r, const float (&a)[8]) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) v[r] += a[i];
+    });
+#pragma unroll
+    for (int r = 0; r < R; ++r) mean[r] = count > 0.f ? warp_sum(v[r]) / count : 0.f;
+#pragma unroll
+    for (int r = 0; r < R; ++r) v[r] = 0.f;
+    each([&](int r, const float (&a)[8]) {
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
-        const float d = a[i] - mean;
-        ssq += c * 8 + i < D ? d * d : 0.f;
+        const float d = a[i] - mean[r];
+        v[r] = fmaf(d, d, v[r]);
       }
-    };
+    });
 #pragma unroll
-    for (int u = 0; u < KEEP; ++u) {
-      const int c = u * kRowThreads + threadIdx.x;
-      if (c < chunks) dev(c, keep[u]);
+    for (int r = 0; r < R; ++r) {
+      const float q = fmaf(-pads * mean[r], mean[r], warp_sum(v[r]));
+      if ((threadIdx.x & 31) == 0) mine[r][threadIdx.x >> 5] = Share{count, mean[r], q};
     }
-    for (int c = KEEP * kRowThreads + threadIdx.x; c < chunks; c += kRowThreads) {
-      float a[8];
-      get(c, a);
-      dev(c, a);
-    }
-    inv = 1.f / sqrtf(row_block_sum(ssq, red) / float(D) + eps);
-  };
-  auto scaled = [&](const Affine& w, int c, const float (&a)[8], float mean, float inv, float (&o)[8]) {
-    float g[8], b[8];
-    w.load(c, g, b);
+    __syncthreads();
 #pragma unroll
-    for (int i = 0; i < 8; ++i) o[i] = c * 8 + i < D ? fmaf((a[i] - mean) * inv, g[i], b[i]) : 0.f;
+    for (int r = 0; r < R; ++r) join_shares<kWarps>(mine[r], float(D), eps, mean[r], inv[r]);
   };
-  float mean, inv;
+  auto scaled = [&](const float (&g)[8], const float (&b)[8], const float (&a)[8], float mean, float inv, float (&o)[8]) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) o[i] = fmaf((a[i] - mean) * inv, g[i], b[i]);
+  };
+  float mean[R], inv[R];
   if constexpr (ADD) {
-    float y[KEEP][8];
+    Kept<SRC> y[R][KEEP];
 #pragma unroll
-    for (int u = 0; u < KEEP; ++u) {
-      const int c = u * kRowThreads + threadIdx.x;
-      if (c < chunks) {
-        src.load(t, c, none, y[u]);
-        load8(row + c * 8, f[u]);
+    for (int u = 0; u < KEEP; ++u)
+      if (chunk(u) < chunks) {
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+          y[r][u].load(from[r], row(r), chunk(u));
+          f[r][u].load(x + size_t(row(r)) * ldx + chunk(u) * 8);
+        }
       }
-    }
-    moments(y, [&](int c, float (&a)[8]) { src.load(t, c, none, a); }, mean, inv);
-    auto add = [&](int c, const float (&a)[8], float (&v)[8]) {
+    auto again = [&](int r, int c, float (&a)[8]) {
+      Kept<SRC> k;
+      k.load(from[r], row(r), c);
+      k.p.get(a);
+    };
+    auto kept = [&](int r, int u, float (&a)[8]) { y[r][u].p.get(a); };
+    moments(kept, again, part[0], mean, inv);
+    auto add = [&](int r, int c, const float (&g)[8], const float (&b)[8], const float (&a)[8], float (&v)[8]) {
       float o[8];
-      scaled(wy, c, a, mean, inv, o);
+      scaled(g, b, a, mean[r], inv[r], o);
 #pragma unroll
       for (int i = 0; i < 8; ++i) v[i] += o[i];
-      store8(row + c * 8, v);
+      if (r == 0 || t0 + r < rows) store8(x + size_t(row(r)) * ldx + c * 8, v);
     };
 #pragma unroll
-    for (int u = 0; u < KEEP; ++u) {
-      const int c = u * kRowThreads + threadIdx.x;
-      if (c < chunks) add(c, y[u], f[u]);
-    }
-    for (int c = KEEP * kRowThreads + threadIdx.x; c < chunks; c += kRowThreads) {
-      float a[8], v[8];
-      src.load(t, c, none, a);
-      load8(row + c * 8, v);
-      add(c, a, v);
+    for (int u = 0; u < KEEP; ++u)
+      if (chunk(u) < chunks) {
+        float g[8], b[8];
+        wy.load(chunk(u), g, b);
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+          float a[8];
+          kept(r, u, a);
+          add(r, chunk(u), g, b, a, f[r][u].v);
+        }
+      }
+    for (int c = chunk(KEEP); c < chunks; c += kRowThreads) {
+      float g[8], b[8];
+      wy.load(c, g, b);
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        float a[8], v[8];
+        again(r, c, a);
+        load8(x + size_t(row(r)) * ldx + c * 8, v);
+        add(r, c, g, b, a, v);
+      }
     }
   } else {
 #pragma unroll
-    for (int u = 0; u < KEEP; ++u) {
-      const int c = u * kRowThreads + threadIdx.x;
-      if (c < chunks) load8(row + c * 8, f[u]);
-    }
+    for (int u = 0; u < KEEP; ++u)
+      if (chunk(u) < chunks) {
+#pragma unroll
+        for (int r = 0; r < R; ++r) f[r][u].load(x + size_t(row(r)) * ldx + chunk(u) * 8);
+      }
   }
   if (!h) return;
-  moments(f, [&](int c, float (&a)[8]) { load8(row + c * 8, a); }, mean, inv);   // (this thread wrote them)
-  T* dst = h + size_t(t) * ldx;
+  // (a thread reads again what it has written itself)
+  auto kept_x = [&](int r, int u, float (&a)[8]) { f[r][u].get(a); };
+  moments(kept_x, [&](int r, int c, float (&a)[8]) { load8(x + size_t(row(r)) * ldx + c * 8, a); }, part[1], mean, inv);
+  auto put = [&](int c, auto value) {
+    float g[8], b[8], o[8];
+    wh.load(c, g, b);
 #pragma unroll
-  for (int u = 0; u < KEEP; ++u) {
-    const int c = u * kRowThreads + threadIdx.x;
-    if (c < chunks) {
-      float o[8];
-      scaled(wh, c, f[u], mean, inv, o);
-      store8(dst + c * 8, o);
+    for (int r = 0; r < R; ++r) {
+      scaled(g, b, value(r), mean[r], inv[r], o);
+      if (r == 0 || t0 + r < rows) store8(h + size_t(row(r)) * ldx + c * 8, o);
     }
-  }
-  for (int c = KEEP * kRowThreads + threadIdx.x; c < chunks; c += kRowThreads) {
-    float a[8], o[8];
-    load8(row + c * 8, a);
-    scaled(wh, c, a, mean, inv, o);
-    store8(dst + c * 8, o);
+  };
+#pragma unroll
+  for (int u = 0; u < KEEP; ++u)
+    if (chunk(u) < chunks) put(chunk(u), [&](int r) -> const float (&)[8] { return f[r][u].v; });
+  for (int c = chunk(KEEP); c < chunks; c += kRowThreads) {
+    float a[R][8];
+#pragma unroll
+    for (int r = 0; r < R; ++r) load8(x + size_t(row(r)) * ldx + c * 8, a[r]);
+    put(c, [&](int r) -> const float (&)[8] { return a[r]; });
   }
 }
 
-// out[t] = h[t] + sum_j w[j] h[t - taps + 1 + j] within a sequence. A thread owns eight columns. Blocks y < strips: kStrip
-// rows each, of which those with all their inputs in the batch are done; the others: one run of rows each, its first
+// out[t] = h[t] + sum_j w[j] h[t - taps + 1 + j] within a sequence. A thread owns eight columns. Blocks y < strips: `strip`
+// rows each (kConvRows at a time), of which those with all their inputs in the batch are done; the others: one run of rows each, its first
 // taps - 1 rows with the help of the carried inputs, which it then replaces by the run's last ones. So a sequence's carried
 // inputs are read and written by one thread alone.
-constexpr int kConvStrip = 8;
+constexpr int kConvRows = 4;
 template <class T, int TAPS>
 __global__ void __launch_bounds__(128)
 short_conv_kernel(const T* __restrict__ h, T* __restrict__ out, int ldx, const float* __restrict__ w, int n_taps,
                   float* __restrict__ carried, long long stride, const int4* __restrict__ runs, const int* __restrict__ slots,
-                  int T_rows, int strips) {
+                  int T_rows, int strip, int strips) {
   pdl_launch_dependents();
   pdl_wait();
   const int taps = TAPS > 0 ? TAPS : n_taps, keep = taps - 1;
@@ -160,29 +263,39 @@ short_conv_kernel(const T* __restrict__ h, T* __restrict__ out, int ldx, const f
   if (c >= ldx) return;
   auto put = [&](int t, const float (&a)[8]) { store8(out + size_t(t) * ldx + c, a); };
   if (int(blockIdx.y) < strips) {
-    const int t0 = blockIdx.y * kConvStrip, n = min(kConvStrip, T_rows - t0);
+    const int t0 = blockIdx.y * strip, n = min(strip, T_rows - t0);
     if constexpr (TAPS > 0) {
-      float v[kConvStrip + TAPS - 1][8], g[TAPS][8];
-#pragma unroll
-      for (int i = 0; i < kConvStrip + TAPS - 1; ++i) {
-        const int t = t0 + i - (TAPS - 1);
-        if (t >= 0 && t < T_rows) load8(h + size_t(t) * ldx + c, v[i]);
-      }
+      constexpr int K = TAPS - 1;
+      Packed<T> v[kConvRows + K];
+      float g[TAPS][8];
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) load8(w + size_t(j) * ldx + c, g[j]);
 #pragma unroll
-      for (int i = 0; i < kConvStrip; ++i) {
-        const int t = t0 + i;
-        if (i >= n || t < keep || (keep > 0 && slots[t - keep] != slots[t])) continue;
-        float a[8];
+      for (int i = 0; i < K; ++i)
+        if (t0 + i >= K) v[i].load(h + size_t(t0 + i - K) * ldx + c);
+      // rows of one sequence are neighbours: with both ends its own, the strip is one sequence's
+      const bool inside = t0 >= K && (K == 0 || slots[max(t0 - K, 0)] == slots[t0 + n - 1]);
+      for (int at = t0; at < t0 + n; at += kConvRows) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          float s = 0.f;
+        for (int i = 0; i < kConvRows; ++i)
+          if (at + i < T_rows) v[K + i].load(h + size_t(at + i) * ldx + c);
 #pragma unroll
-          for (int j = 0; j < TAPS; ++j) s = fmaf(g[j][e], v[i + j][e], s);
-          a[e] = v[i + TAPS - 1][e] + s;
+        for (int i = 0; i < kConvRows; ++i) {
+          const int t = at + i;
+          if (t >= t0 + n || (!inside && (t < K || (K > 0 && slots[t - K] != slots[t])))) continue;
+          float a[8], s[8] = {};
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) {
+            v[i + j].get(a);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) s[e] = fmaf(g[j][e], a[e], s[e]);
+          }
+#pragma unroll
+          for (int e = 0; e < 8; ++e) a[e] += s[e];          // (the last one read is the row itself)
+          put(t, a);
         }
-        put(t, a);
+#pragma unroll
+        for (int i = 0; i < K; ++i) v[i] = v[kConvRows + i];
       }
     } else {
       for (int t = t0; t < t0 + n; ++t) {
@@ -246,9 +359,11 @@ poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ act, float e
   const int chunks = ld >> 3;
   const T* row = z + size_t(blockIdx.x) * ld;
   T* dst = out + size_t(blockIdx.x) * ld;
-  float f[KEEP][8], s2 = 0.f, s4 = 0.f, s6 = 0.f;
-  auto take = [&](int c, float (&a)[8]) {
-    load8(row + c * 8, a);
+  Packed<T> f[KEEP];
+  float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  auto take = [&](int c, const Packed<T>& p) {
+    float a[8];
+    p.get(a);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       if (c * 8 + i >= D) a[i] = 0.f;
@@ -261,11 +376,17 @@ poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ act, float e
 #pragma unroll
   for (int u = 0; u < KEEP; ++u) {
     const int c = u * kRowThreads + threadIdx.x;
+    if (c < chunks) f[u].load(row + c * 8);
+  }
+#pragma unroll
+  for (int u = 0; u < KEEP; ++u) {
+    const int c = u * kRowThreads + threadIdx.x;
     if (c < chunks) take(c, f[u]);
   }
   for (int c = KEEP * kRowThreads + threadIdx.x; c < chunks; c += kRowThreads) {
-    float a[8];
-    take(c, a);
+    Packed<T> p;
+    p.load(row + c * 8);
+    take(c, p);
   }
   s2 = warp_sum(s2); s4 = warp_sum(s4); s6 = warp_sum(s6);
   if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = s2; red[1][threadIdx.x >> 5] = s4; red[2][threadIdx.x >> 5] = s6; }
@@ -273,12 +394,15 @@ poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ act, float e
   float k[3];
 #pragma unroll
   for (int i = 0; i < 3; ++i) {
-    const float v = (threadIdx.x & 31) < kRowThreads / 32 ? red[i][threadIdx.x & 31] : 0.f;
-    k[i] = act[i] / sqrtf(warp_sum(v) / float(D) + eps);
+    float v = 0.f;
+#pragma unroll
+    for (int w = 0; w < kRowThreads / 32; ++w) v += red[i][w];
+    k[i] = act[i] / sqrtf(v / float(D) + eps);
   }
   const float e = act[3];
-  auto put = [&](int c, const float (&a)[8]) {
-    float o[8];
+  auto put = [&](int c, const Packed<T>& p) {
+    float a[8], o[8];
+    p.get(a);
 #pragma unroll
     for (int i = 0; i < 8; ++i) o[i] = c * 8 + i < D ? fmaf(a[i], fmaf(a[i], fmaf(a[i], k[2], k[1]), k[0]), e) : 0.f;
     store8(dst + c * 8, o);
@@ -289,23 +413,22 @@ poly_norm_kernel(const T* __restrict__ z, const float* __restrict__ act, float e
     if (c < chunks) put(c, f[u]);
   }
   for (int c = KEEP * kRowThreads + threadIdx.x; c < chunks; c += kRowThreads) {
-    float a[8];
-    load8(row + c * 8, a);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) a[i] = c * 8 + i < D ? a[i] : 0.f;
-    put(c, a);
+    Packed<T> p;
+    p.load(row + c * 8);
+    put(c, p);
   }
 }
 
 // ------------------------------------------------------------------ decode
-constexpr int kStepThreads = 128, kStepCols = kStepThreads * 4;
+constexpr int kStepThreads = 512;
 
+template <class SRC, class T>
 struct SandwichStep {
+  SRC src;                  // finished sublayer
+  int add;                  // 0: there is none
   float* x;                 // [B, ldx]
-  const float* y;           // [B, ldx] finished sublayer, or null
-  const float* wy;          // [2, ldx]
-  const float* wh;          // [2, ldx]
-  float* h;                 // [B, ldx]
+  Affine wy, wh;
+  T* h;                     // [B, ldx]
   const float* conv;        // [taps, ldx], or null: no convolution
   int taps;
   float* carried;           // slot s: carried + s * stride, [taps - 1, ldx]
@@ -315,140 +438,160 @@ struct SandwichStep {
   int D, ldx;
 };
 
-// A count, a mean and a sum of squared deviations, joined without cancellation.
-struct Moments {
-  float n, mean, m2;
-};
-__device__ __forceinline__ Moments join(const Moments& a, const Moments& b) {
-  const float n = a.n + b.n;
-  if (n == 0.f) return a;
-  const float d = b.mean - a.mean, f = b.n / n;
-  return Moments{n, fmaf(d, f, a.mean), a.m2 + b.m2 + d * d * a.n * f};
+__device__ __forceinline__ void step_copy32(float* dst, const float* src) {      // 32 bytes, asynchronously
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst + 4)), "l"(src + 4) : "memory");
 }
 
-// grid (column blocks = one cluster, rows). E float4 pieces a thread holds.
-template <int E>
+// One block per row, E chunks of eight columns a thread. What no kernel of the step writes is asked for before the wait: the
+// weights go to shared memory (every thread its own columns'), the carried inputs move up, and their share of the
+// convolution is taken.
+template <int E, class SRC, class T>
 __global__ void __launch_bounds__(kStepThreads)
-sandwich_step_kernel(SandwichStep p) {
-  __shared__ Moments warp_part[kStepThreads / 32];
-  __shared__ Moments part[2];
-  const int b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int col0 = (blockIdx.x * kStepThreads + tid) * 4, step = gridDim.x * kStepCols;
-  auto ld = [](const float* q) { return __ldcg(reinterpret_cast<const float4*>(q)); };
-  auto at = [&](int e) { return col0 + e * step; };
-  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  // what no kernel of this step writes before: norm weights, and the convolution's share of the carried inputs
-  float4 gy[E], by[E], gh[E], bh[E], past[E], now[E];
+sandwich_step_kernel(SandwichStep<SRC, T> p) {
+  constexpr int kWarps = kStepThreads / 32;
+  extern __shared__ __align__(16) float sw[];          // [5][chunks][8]: weight, bias of both norms, the current token's tap
+  __shared__ Share part[2][kWarps];
+  const int b = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, chunks = p.ldx >> 3;
+  auto chunk = [&](int e) { return e * kStepThreads + tid; };
+  auto own = [&](int k, int c) { return sw + (size_t(k) * chunks + c) * 8; };
   float* st = p.conv && p.taps > 1 ? p.carried + size_t(p.slots[b]) * p.stride : nullptr;
+  float count = 0.f, pads = 0.f;
 #pragma unroll
   for (int e = 0; e < E; ++e) {
-    gy[e] = by[e] = gh[e] = bh[e] = past[e] = now[e] = zero;
-    if (at(e) >= p.ldx) continue;
-    if (p.y) { gy[e] = ld(p.wy + at(e)); by[e] = ld(p.wy + p.ldx + at(e)); }
-    gh[e] = ld(p.wh + at(e));
-    bh[e] = ld(p.wh + p.ldx + at(e));
-    if (p.conv) {
-      now[e] = ld(p.conv + size_t(p.taps - 1) * p.ldx + at(e));
-      for (int j = 0; j < p.taps - 1; ++j) {
-        const float4 w = ld(p.conv + size_t(j) * p.ldx + at(e)), v = ld(st + size_t(j) * p.ldx + at(e));
-        past[e].x = fmaf(w.x, v.x, past[e].x); past[e].y = fmaf(w.y, v.y, past[e].y);
-        past[e].z = fmaf(w.z, v.z, past[e].z); past[e].w = fmaf(w.w, v.w, past[e].w);
-      }
+    const int c = chunk(e);
+    if (c >= chunks) continue;
+    const int n = max(0, min(8, p.D - c * 8));
+    count += float(n);
+    pads += float(8 - n);
+    if (p.add) {
+      step_copy32(own(0, c), p.wy.w + c * 8);
+      step_copy32(own(1, c), p.wy.w + p.ldx + c * 8);
+    }
+    step_copy32(own(2, c), p.wh.w + c * 8);
+    step_copy32(own(3, c), p.wh.w + p.ldx + c * 8);
+    if (p.conv) step_copy32(own(4, c), p.conv + size_t(p.taps - 1) * p.ldx + c * 8);
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  float past[E][8];
+#pragma unroll
+  for (int e = 0; e < E; ++e) {
+    const int c = chunk(e);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) past[e][i] = 0.f;
+    if (c >= chunks || !p.conv) continue;
+#pragma unroll 3
+    for (int j = 0; j < p.taps - 1; ++j) {
+      float w[8], v[8];
+      load8(p.conv + size_t(j) * p.ldx + c * 8, w);
+      load8(st + size_t(j) * p.ldx + c * 8, v);
+      if (j > 0) store8(st + size_t(j - 1) * p.ldx + c * 8, v);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) past[e][i] = fmaf(w[i], v[i], past[e][i]);
     }
   }
+  count = warp_sum(count);
+  pads = warp_sum(pads);
   pdl_launch_dependents();
   pdl_wait();
-  float4 x[E], y[E];
+  if (p.add) p.src.prepare(b);
+  const float none[8] = {};
+  float x[E][8], y[E][8];
 #pragma unroll
   for (int e = 0; e < E; ++e) {
-    const bool in = at(e) < p.ldx;
-    x[e] = in ? ld(p.x + size_t(b) * p.ldx + at(e)) : zero;
-    y[e] = in && p.y ? ld(p.y + size_t(b) * p.ldx + at(e)) : zero;
-  }
-  cg::cluster_group cluster = cg::this_cluster();
-  // mean and 1 / deviation over the row
-  auto moments = [&](const float4 (&v)[E], Moments* mine, float& mean, float& inv) {
-    Moments m{0.f, 0.f, 0.f};
-#pragma unroll
-    for (int e = 0; e < E; ++e) {
-      const int n = max(0, min(4, p.D - at(e)));
-      const float f[4] = {v[e].x, v[e].y, v[e].z, v[e].w};
-      float s = 0.f, q = 0.f;
-#pragma unroll
-      for (int i = 0; i < 4; ++i) s += i < n ? f[i] : 0.f;
-      const float mu = n > 0 ? s / float(n) : 0.f;
-#pragma unroll
-      for (int i = 0; i < 4; ++i) q += i < n ? (f[i] - mu) * (f[i] - mu) : 0.f;
-      m = join(m, Moments{float(n), mu, q});
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1)
-      m = join(m, Moments{__shfl_xor_sync(0xffffffffu, m.n, o), __shfl_xor_sync(0xffffffffu, m.mean, o),
-                          __shfl_xor_sync(0xffffffffu, m.m2, o)});
-    if (lane == 0) warp_part[warp] = m;
-    __syncthreads();
-    m = warp_part[0];
-#pragma unroll
-    for (int q = 1; q < kStepThreads / 32; ++q) m = join(m, warp_part[q]);
-    if (gridDim.x > 1) {
-      if (tid == 0) *mine = m;
-      cluster.sync();
-      m = *cluster.map_shared_rank(mine, 0);
-      for (unsigned r = 1; r < gridDim.x; ++r) m = join(m, *cluster.map_shared_rank(mine, r));
+    if (chunk(e) < chunks) {
+      load8(p.x + size_t(b) * p.ldx + chunk(e) * 8, x[e]);
+      if (p.add) p.src.load(b, chunk(e), none, y[e]);
     } else {
-      __syncthreads();                                 // warp_part is written again
+#pragma unroll
+      for (int i = 0; i < 8; ++i) x[e][i] = y[e][i] = 0.f;
     }
-    mean = m.mean;
-    inv = 1.f / sqrtf(m.m2 / float(p.D) + p.eps);
-  };
-  auto norm4 = [&](int e, const float4& v, float mean, float inv, const float4& g, const float4& o) {
-    const int n = p.D - at(e);
-    return make_float4(n > 0 ? fmaf((v.x - mean) * inv, g.x, o.x) : 0.f, n > 1 ? fmaf((v.y - mean) * inv, g.y, o.y) : 0.f,
-                       n > 2 ? fmaf((v.z - mean) * inv, g.z, o.z) : 0.f, n > 3 ? fmaf((v.w - mean) * inv, g.w, o.w) : 0.f);
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  // mean and 1 / deviation over the row (columns past D are zero)
+  auto moments = [&](const float (&v)[E][8], Share (&mine)[kWarps], float& mean, float& inv) {
+    float s = 0.f, q = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s += v[e][i];
+    mean = count > 0.f ? warp_sum(s) / count : 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e)
+      if (chunk(e) < chunks) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) q = fmaf(v[e][i] - mean, v[e][i] - mean, q);
+      }
+    q = fmaf(-pads * mean, mean, warp_sum(q));
+    if (lane == 0) mine[warp] = Share{count, mean, q};
+    __syncthreads();
+    join_shares<kWarps>(mine, float(p.D), p.eps, mean, inv);
   };
   float mean, inv;
-  if (p.y) {
-    moments(y, part, mean, inv);
+  if (p.add) {
+    moments(y, part[0], mean, inv);
 #pragma unroll
     for (int e = 0; e < E; ++e) {
-      const float4 a = norm4(e, y[e], mean, inv, gy[e], by[e]);
-      x[e].x += a.x; x[e].y += a.y; x[e].z += a.z; x[e].w += a.w;
-      if (at(e) < p.ldx) *reinterpret_cast<float4*>(p.x + size_t(b) * p.ldx + at(e)) = x[e];
+      const int c = chunk(e);
+      if (c >= chunks) continue;
+      float g[8], o[8];
+      load8(own(0, c), g);
+      load8(own(1, c), o);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) x[e][i] += fmaf((y[e][i] - mean) * inv, g[i], o[i]);
+      store8(p.x + size_t(b) * p.ldx + c * 8, x[e]);
     }
   }
-  moments(x, part + 1, mean, inv);
+  moments(x, part[1], mean, inv);
 #pragma unroll
   for (int e = 0; e < E; ++e) {
-    if (at(e) >= p.ldx) continue;
-    const float4 a = norm4(e, x[e], mean, inv, gh[e], bh[e]);
-    float4 o = a;
+    const int c = chunk(e);
+    if (c >= chunks) continue;
+    float g[8], o[8], a[8];
+    load8(own(2, c), g);
+    load8(own(3, c), o);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) a[i] = o[i] = fmaf((x[e][i] - mean) * inv, g[i], o[i]);
     if (p.conv) {
-      o.x += fmaf(now[e].x, a.x, past[e].x); o.y += fmaf(now[e].y, a.y, past[e].y);
-      o.z += fmaf(now[e].z, a.z, past[e].z); o.w += fmaf(now[e].w, a.w, past[e].w);
-      float* q = st + at(e);
-      for (int j = 0; j + 2 < p.taps; ++j) *reinterpret_cast<float4*>(q + size_t(j) * p.ldx) = ld(q + size_t(j + 1) * p.ldx);
-      if (p.taps > 1) *reinterpret_cast<float4*>(q + size_t(p.taps - 2) * p.ldx) = a;
+      load8(own(4, c), g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) o[i] += fmaf(g[i], a[i], past[e][i]);
+      if (p.taps > 1) store8(st + size_t(p.taps - 2) * p.ldx + c * 8, a);
     }
-    *reinterpret_cast<float4*>(p.h + size_t(b) * p.ldx + at(e)) = o;
+    store8(p.h + size_t(b) * p.ldx + c * 8, o);
   }
-  if (gridDim.x > 1) cluster.sync();                   // nobody leaves while a neighbour still reads its shared memory
 }
 
 template <class SRC, bool ADD>
 static int launch_sandwich(SRC src, const float* wy, float* x, const float* wh, void* h, float eps, int T, int D, int ldx, int f32,
                            int pdl, cudaStream_t st) {
   const Affine ay{wy, ldx}, ah{wh, ldx};
-  auto go = [&](auto kern, auto* out) -> int {
-    return launch(kern, dim3(T), dim3(kRowThreads), 0, st, pdl != 0, src, ay, x, ah, out, eps, D, ldx);
+  auto go = [&](auto kern, int per, auto* out) -> int {
+    return launch(kern, dim3((T + per - 1) / per), dim3(kRowThreads), 0, st, pdl != 0, src, ay, x, ah, out, eps, T, D, ldx);
   };
   const bool narrow = ldx <= 2 * 8 * kRowThreads;
   if (f32) {
     float* out = static_cast<float*>(h);
-    return narrow ? go(sandwich_norm_kernel<SRC, ADD, float, 2>, out) : go(sandwich_norm_kernel<SRC, ADD, float, 4>, out);
+    return narrow ? go(sandwich_norm_kernel<SRC, ADD, float, 2, 1, 2>, 1, out)
+                  : go(sandwich_norm_kernel<SRC, ADD, float, 4, 1, 2>, 1, out);
   }
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(h);
-  return narrow ? go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 2>, out)
-                : go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 4>, out);
+  if (!narrow) return go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 4, 1, 2>, 1, out);
+  // where rows are plenty, two a block share its weights and barriers; else as many blocks as the registers allow
+  constexpr bool kExperts = !std::is_same<SRC, RowSource<float>>::value && !std::is_same<SRC, RowSource<__nv_bfloat16>>::value;
+  if constexpr (kExperts) return go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 2, 1, 2>, 1, out);
+  else if (T >= 16 * sm_count()) return go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 2, 2, 3>, 2, out);
+  else return go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 2, 1, 4>, 1, out);
+}
+
+template <class SRC, class T>
+static int launch_step(const SandwichStep<SRC, T>& p, int B, int pdl, cudaStream_t st) {
+  const int pieces = (p.ldx + 8 * kStepThreads - 1) / (8 * kStepThreads);
+  auto kern = pieces <= 1 ? sandwich_step_kernel<1, SRC, T> : pieces <= 2 ? sandwich_step_kernel<2, SRC, T>
+                                                                           : sandwich_step_kernel<3, SRC, T>;
+  const size_t smem = size_t(5) * p.ldx * sizeof(float);
+  RB_CHECK(set_max_smem(kern, smem));
+  return launch(kern, dim3(B), dim3(kStepThreads), smem, st, pdl != 0, p);
 }
 
 }  // namespace rb
@@ -483,15 +626,19 @@ extern "C" int rmlx_short_conv(const void* h, void* out, int ldx, const float* w
   if (T < 1 || ldx < 8 || ldx % 8 || taps < 1 || taps > 64 || h == out || n_runs < 1 || n_runs > T || (!runs && n_runs != T) ||
       (taps > 1 && (!carried || !slots || stride % 4 || (reinterpret_cast<uintptr_t>(carried) & 15))) || (reinterpret_cast<uintptr_t>(runs) & 15))
     return -2;
-  const int strips = runs || taps == 1 ? (T + kConvStrip - 1) / kConvStrip : 0, tails = taps > 1 ? n_runs : 0;
+  // longer strips read fewer rows and weights twice, as far as there is work for every SM
+  const int wide = (ldx / 8 + 127) / 128;
+  int strip = kConvRows;
+  while (strip < 4 * kConvRows && (long long)wide * ((T + 2 * strip - 1) / (2 * strip)) >= 12 * sm_count()) strip *= 2;
+  const int strips = runs || taps == 1 ? (T + strip - 1) / strip : 0, tails = taps > 1 ? n_runs : 0;
   if (strips + tails > 65535) return -2;
-  const dim3 grid((ldx / 8 + 127) / 128, strips + tails);
+  const dim3 grid(wide, strips + tails);
   auto go = [&](auto* type) -> int {
     using T_ = std::remove_pointer_t<decltype(type)>;
     auto kern = taps == 4 ? short_conv_kernel<T_, 4> : taps == 3 ? short_conv_kernel<T_, 3>
                 : taps == 2 ? short_conv_kernel<T_, 2> : short_conv_kernel<T_, 0>;
     return launch(kern, grid, dim3(128), 0, st, pdl != 0, static_cast<const T_*>(h), static_cast<T_*>(out), ldx, w, taps, carried,
-                  stride, reinterpret_cast<const int4*>(runs), slots, T, strips);
+                  stride, reinterpret_cast<const int4*>(runs), slots, T, strip, strips);
   };
   return f32 ? go(static_cast<float*>(nullptr)) : go(static_cast<__nv_bfloat16*>(nullptr));
 }
@@ -505,46 +652,40 @@ extern "C" int rmlx_poly_norm(const void* z, const float* act, float eps, void* 
     return launch(kern, dim3(T), dim3(kRowThreads), 0, st, pdl != 0, static_cast<const T_*>(z), act, eps, static_cast<T_*>(out),
                   D, ld);
   };
-  const bool narrow = ld <= 2 * 8 * kRowThreads;
-  if (f32)
-    return narrow ? go(poly_norm_kernel<float, 2>, static_cast<float*>(nullptr)) : go(poly_norm_kernel<float, 8>, static_cast<float*>(nullptr));
-  return narrow ? go(poly_norm_kernel<__nv_bfloat16, 2>, static_cast<__nv_bfloat16*>(nullptr))
-                : go(poly_norm_kernel<__nv_bfloat16, 8>, static_cast<__nv_bfloat16*>(nullptr));
+  const int keep = (ld + 8 * kRowThreads - 1) / (8 * kRowThreads);
+  if (f32) {
+    float* type = nullptr;
+    return keep <= 2 ? go(poly_norm_kernel<float, 2>, type) : go(poly_norm_kernel<float, 6>, type);
+  }
+  __nv_bfloat16* type = nullptr;
+  return keep <= 4 ? go(poly_norm_kernel<__nv_bfloat16, 4>, type) : keep <= 7 ? go(poly_norm_kernel<__nv_bfloat16, 7>, type)
+                                                                               : go(poly_norm_kernel<__nv_bfloat16, 12>, type);
 }
 
 // Widest row the decode step takes.
-extern "C" int rmlx_sandwich_step_max_width() { return 8 * kStepCols * 4; }
+extern "C" int rmlx_sandwich_step_max_width() { return 44 * 1024 / 4; }      // five fp32 rows of shared memory
 
-// x += LN(y; wy) (y null: nothing), h = LN(x; wh), with conv (fp32 [taps, ldx]) h + its convolution; everything fp32 [B, ldx],
-// carried and slots [B] as in rmlx_short_conv.
-extern "C" int rmlx_sandwich_step(float* x, const float* y, const float* wy, const float* wh, float* h, const float* conv, int taps,
+// x fp32 [B, ldx] += LN(y; wy) (y null: nothing), h = LN(x; wh), with conv (fp32 [taps, ldx]) h + its convolution. y and h
+// [B, ldx] fp32 (f32) or bf16, y's rows ldy apart or (row_of_pair) expert rows with weights [B, top_k]; carried and slots [B] as in rmlx_short_conv.
+extern "C" int rmlx_sandwich_step(float* x, const void* y, int ldy, const int* row_of_pair, const float* weights,
+                                  int top_k, const float* wy, const float* wh, void* h, int f32, const float* conv, int taps,
                                   float* carried, long long stride, const int* slots, float eps, int B, int D, int ldx, int pdl,
                                   cudaStream_t st) {
-  if (B < 1 || B > 65535 || D < 1 || ldx < D || ldx % 8 || ldx > rmlx_sandwich_step_max_width() || !x || !wh || !h || h == x ||
-      (y && !wy) || (conv && (taps < 1 || (taps > 1 && (!carried || !slots || stride % 4)))))
+  if (B < 1 || D < 1 || ldx < D || ldx % 8 || ldx > rmlx_sandwich_step_max_width() || !x || !wh || !h || h == x ||
+      (y && (!wy || ldy % 8 || ldy < ldx)) || (row_of_pair && (!y || !weights || top_k < 1)) ||
+      (conv && (taps < 1 || (taps > 1 && (!carried || !slots || stride % 4)))))
     return -2;
-  int blocks = 1;
-  while (blocks < 8 && blocks * kStepCols < ldx) blocks *= 2;
-  const int pieces = (ldx + blocks * kStepCols - 1) / (blocks * kStepCols);
-  const SandwichStep p{x, y, wy, wh, h, conv, taps, carried, stride, slots, eps, D, ldx};
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(blocks, B);
-  cfg.blockDim = dim3(kStepThreads);
-  cfg.stream = st;
-  cudaLaunchAttribute attr[2];
-  int n = 0;
-  attr[n].id = cudaLaunchAttributeClusterDimension;
-  attr[n].val.clusterDim.x = blocks; attr[n].val.clusterDim.y = 1; attr[n].val.clusterDim.z = 1;
-  ++n;
-  auto kern = pieces <= 1 ? sandwich_step_kernel<1> : pieces <= 2 ? sandwich_step_kernel<2> : sandwich_step_kernel<4>;
-  if (pdl) {
-    attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[n].val.programmaticStreamSerializationAllowed = 1;
-    ++n;
-    prefer_max_shared(kern);
-  }
-  cfg.attrs = attr; cfg.numAttrs = n;
-  const cudaError_t e = cudaLaunchKernelEx(&cfg, kern, p);
-  if (e != cudaSuccess) (void)cudaGetLastError();
-  return static_cast<int>(e);
+  auto run = [&](auto src, auto* out) -> int {
+    using SRC = decltype(src);
+    using T = std::remove_pointer_t<decltype(out)>;
+    return launch_step(SandwichStep<SRC, T>{src, y != nullptr, x, Affine{wy, ldx}, Affine{wh, ldx}, out, conv, taps, carried, stride,
+                                            slots, eps, D, ldx}, B, pdl, st);
+  };
+  auto from = [&](auto* rows, auto* out) -> int {
+    using TY = std::remove_const_t<std::remove_pointer_t<decltype(rows)>>;
+    if (row_of_pair) return run(ExpertSource<TY>{rows, ldy, row_of_pair, weights, nullptr, top_k}, out);
+    return run(RowSource<TY>{rows, ldy}, out);
+  };
+  return f32 ? from(static_cast<const float*>(y), static_cast<float*>(h))
+             : from(static_cast<const __nv_bfloat16*>(y), static_cast<__nv_bfloat16*>(h));
 }

@@ -224,6 +224,72 @@ rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __
   }
 }
 
+// The form with neighbours, no norm and no bias: chunks of eight turn on their own, so a block deals those of kRaTokens
+// tokens to its threads in a row. Source rows, widths and strides are multiples of eight values.
+constexpr int kRaTokens = 4;
+template <class TR, class T>
+__global__ void __launch_bounds__(kRowThreads)
+rotary_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restrict__ inv_freq, int dims, float grow,
+                     T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ block_table,
+                     const int* __restrict__ positions, const int* __restrict__ token_seq, int rows, int Hq, int Hkv, int dim,
+                     int vdim, int max_blocks, int page, int maps) {
+  extern __shared__ __align__(16) float trig[];          // per token: cos [dims / 2], sin [dims / 2]
+  __shared__ int s_blk[kRaTokens], s_off[kRaTokens];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t0 = blockIdx.x * kRaTokens, n = min(kRaTokens, rows - t0), half = dims / 2;
+  for (int i = threadIdx.x; i < n * half; i += kRowThreads) {
+    const int a = i / half, j = i - a * half;
+    float s, c;
+    rotary_sincos(positions[t0 + a], inv_freq[j], s, c);
+    trig[a * dims + j] = c * grow;
+    trig[a * dims + half + j] = s * grow;
+  }
+  if (threadIdx.x < n) {
+    const int t = t0 + threadIdx.x, pos = positions[t];
+    const bool in_table = RB_BOUNDS(pos / page, max_blocks);
+    s_blk[threadIdx.x] = in_table ? block_table[size_t(token_seq ? token_seq[t] : t) * max_blocks + pos / page] : -1;
+    s_off[threadIdx.x] = pos % page;
+  }
+  __syncthreads();
+  const int nq = Hq * maps * dim, nk = Hkv * maps * dim, chunks = (nq + nk + Hkv * vdim) >> 3;
+  for (int a = 0; a < n; ++a) {
+    const TR* row = raw + size_t(t0 + a) * ldraw;
+    const float* cs = trig + a * dims;
+#pragma unroll 4
+    for (int c = threadIdx.x; c < chunks; c += kRowThreads) {
+      const int at = c * 8;
+      float f[8];
+      load8(row + at, f);
+      T* dst;
+      if (at < nq + nk) {
+        const int r = at / dim, d0 = at - r * dim;         // part (head, map) and place in it
+        if (d0 < dims) {
+#pragma unroll
+          for (int i = 0; i < 8; i += 2) {
+            if (d0 + i >= dims) break;
+            const float co = cs[(d0 + i) >> 1], si = cs[half + ((d0 + i) >> 1)], u = f[i], v = f[i + 1];
+            f[i] = u * co - v * si;
+            f[i + 1] = v * co + u * si;
+          }
+        }
+        if (at < nq) {
+          dst = q_out + size_t(t0 + a) * nq + at;
+        } else {
+          if (s_blk[a] < 0) continue;
+          const int k = r - Hq * maps;
+          dst = k_cache + (((size_t(s_blk[a]) * Hkv + k / maps) * page + s_off[a]) * maps + k % maps) * dim + d0;
+        }
+      } else {
+        if (s_blk[a] < 0) continue;
+        const int v = at - nq - nk, g = v / vdim;
+        dst = v_cache + ((size_t(s_blk[a]) * Hkv + g) * page + s_off[a]) * vdim + v - g * vdim;
+      }
+      store8(dst, f);
+    }
+  }
+}
+
 template <class SRC, bool ADD>
 static int launch_twin(SRC src, float* x, const float* w1, void* h1, const float* w2, void* h2, float eps, int T, int D, int ldx,
                        int f32, int pdl, cudaStream_t st) {
@@ -281,6 +347,17 @@ extern "C" int rmlx_rotary_norm_append(const void* raw, int ldraw, int raw_f32, 
     return -2;
   const size_t smem = size_t(dims) * sizeof(float);
   if (smem > 32 * 1024) return -2;
+  if (neighbours && !norm && !bias && dim % 8 == 0 && vdim % 8 == 0 && ldraw % 8 == 0 && dkp == dim && dvp == vdim && dims <= 2048) {
+#define RB_RF(TR_, T_)                                                                                                     \
+  return launch(rotary_append_kernel<TR_, T_>, dim3((T + kRaTokens - 1) / kRaTokens), dim3(kRowThreads), smem * kRaTokens, st, \
+                pdl != 0, static_cast<const TR_*>(raw), ldraw, inv_freq, dims, grow, static_cast<T_*>(q_out),                  \
+                static_cast<T_*>(k_cache), static_cast<T_*>(v_cache), block_table, positions, token_seq, T, Hq, Hkv, dim, vdim, \
+                max_blocks, page, maps)
+    if (f32) RB_RF(float, float);
+    if (raw_f32) RB_RF(float, __nv_bfloat16);
+    RB_RF(__nv_bfloat16, __nv_bfloat16);
+#undef RB_RF
+  }
   const int widest = dkp > dvp ? dkp : dvp, lanes = widest <= 64 ? 8 : widest <= 128 ? 16 : 32;
   const int per_block = kRowThreads / lanes, blocks = ((Hq + Hkv) * maps + Hkv + per_block - 1) / per_block;
   const dim3 grid(T, T >= 64 ? 1 : blocks);           // few tokens: several blocks share one

@@ -329,32 +329,43 @@ class NizoraxModel(RaggedModel):
         return R.RouteGroups(f.groups, f.keep, f.scale, fw.always)
 
     # ------------------------------------------------------------------ layers
-    def conv(self, li: int, name: str, w: torch.Tensor, h: torch.Tensor, c: StepContext) -> torch.Tensor:
-        return W.short_conv(h, w, self.carried(c.cache, li, name), c.bufs.get("h_conv", c.t, self.width_p, dtype=self.dtype), c.slots,
-                            runs=c.runs, pdl=c.pdl)
+    def conv(self, li: int, name: str, w: torch.Tensor, h: torch.Tensor, hc: torch.Tensor, c: StepContext) -> None:
+        W.short_conv(h, w, self.carried(c.cache, li, name), hc, c.slots, runs=c.runs, pdl=c.pdl)
 
     def layer(self, li: int, acts, c: StepContext) -> None:
-        """One layer run over the fp32 residual ``x`` and its norm ``h``, in place: the norm becomes the next run's."""
+        """One layer run over the fp32 residual ``x`` and its norm ``h``, in place: the norm becomes the next run's. In a decode
+        step the convolution that follows a norm is part of its launch (the next run then finds its input convolved)."""
         x, h = acts
         lw, eps, width, pdl = self.w.layers[li], self.cfg.norm_eps, self.cfg.width, c.pdl
-        after = self.w.layers[li + 1].norm1 if li + 1 < len(self.w.layers) else None
+        after = self.w.layers[li + 1] if li + 1 < len(self.w.layers) else None
+        step = c.batch is None and self.width_p <= W.step_max_width()
+        hc = c.bufs.get("h_conv", c.t, self.width_p, dtype=self.dtype)
         out = lambda a, w: N.linear(a, w.w, c.bufs.get("y", c.t, self.width_p, dtype=self.dtype), pdl=pdl)    # noqa: E731
 
-        hc = self.conv(li, "conv1", lw.conv1, h, c)
+        def finish(y, post, norm, run, name, w, r=None) -> None:
+            """x += post(y); the norm for what follows (of which ``step`` also does the convolution)."""
+            if step and norm is not None:
+                W.sandwich_step(x, y, post, norm, hc, eps, width, (w, self.carried(c.cache, run, name), c.slots), routing=r, pdl=pdl)
+            else:
+                W.sandwich_norm(x, y, post, norm, None if norm is None else h, eps, width, routing=r, pdl=pdl)
+
+        follow = (None, li, "", None) if after is None else (after.norm1, li + 1, "conv1", after.conv1)
+        if li == 0 or not step:
+            self.conv(li, "conv1", lw.conv1, h, hc, c)
         mixer = self.attention if isinstance(lw.mix, DiffAttentionWeights) else self.lightning
         y = out(mixer(li, lw.mix, hc, c), lw.mix.w_o)
         if lw.mlp is None:
-            W.sandwich_norm(x, y, lw.post1, after, None if after is None else h, eps, width, pdl=pdl)
+            finish(y, lw.post1, *follow)
             return
-        W.sandwich_norm(x, y, lw.post1, lw.norm2, h, eps, width, pdl=pdl)
-        hc, r = self.conv(li, "conv2", lw.conv2, h, c), None
+        finish(y, lw.post1, lw.norm2, li, "conv2", lw.conv2)
+        if not step:
+            self.conv(li, "conv2", lw.conv2, h, hc, c)
         if isinstance(lw.mlp, PolyFfWeights):
-            y = out(self.poly(lw.mlp, hc, c), lw.mlp.w_down)
+            finish(out(self.poly(lw.mlp, hc, c), lw.mlp.w_down), lw.post2, *follow)
         else:
             r = self.routing(lw.mlp, c)
             R.route_grouped(self.router_logits(lw.mlp, hc, c), self.groups(lw.mlp), r, pdl=pdl)
-            y = self.expert_rows(lw.mlp, hc, r, c)
-        W.sandwich_norm(x, y, lw.post2, after, None if after is None else h, eps, width, routing=r, pdl=pdl)
+            finish(self.expert_rows(lw.mlp, hc, r, c), lw.post2, *follow, r)
 
     def start(self, tokens: torch.Tensor, bufs: Buffers, pdl: bool = False):
         """(fp32 residual, its norm for the first layer's mixer) of the tokens."""

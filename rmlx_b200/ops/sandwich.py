@@ -3,6 +3,7 @@ reads (csrc/kernels/sandwich_rows.cu), and their decode projections (sandwich_ge
 dtype of the tensors picks the kernels. A norm's weight and bias are one fp32 tensor [2, row width]."""
 from __future__ import annotations
 
+import functools
 from typing import Optional, Tuple
 
 import torch
@@ -17,7 +18,7 @@ _lib.register_cuda_sigs({
     "rmlx_short_conv": ("ppipi" "pq" "ppiiiip", "i"),
     "rmlx_poly_norm": ("ppfp" "iiiiip", "i"),
     "rmlx_sandwich_step_max_width": ("", "i"),
-    "rmlx_sandwich_step": ("ppppp" "pi" "pqp" "fiiiip", "i"),
+    "rmlx_sandwich_step": ("ppi" "ppi" "pppi" "pi" "pqp" "fiiiip", "i"),
     "rmlx_poly_out": ("ppipfpi" "iiiiip", "i"),
     "rmlx_gated_out": ("ppipipfpi" "iiiiip", "i"),
 })
@@ -80,24 +81,28 @@ def poly_norm(z: torch.Tensor, act: torch.Tensor, eps: float, width: int, out: t
 
 
 # ------------------------------------------------------------------ decode
+@functools.lru_cache(maxsize=None)
 def step_max_width() -> int:
     return int(_lib.cuda().rmlx_sandwich_step_max_width())
 
 
 def sandwich_step(x: torch.Tensor, y: Optional[torch.Tensor], wy: Optional[torch.Tensor], wh: torch.Tensor, h: torch.Tensor,
                   eps: float, width: int, conv: Optional[Tuple[torch.Tensor, Optional[torch.Tensor], Optional[torch.Tensor]]] = None,
-                  pdl: bool = False) -> None:
-    """A decode row per sequence: x += LN(y; wy), h = LN(x; wh), with ``conv`` (weights, carried inputs, slots) h + its
-    convolution. Everything fp32."""
+                  routing: Optional[Routing] = None, pdl: bool = False) -> None:
+    """A decode row per sequence: ``sandwich_norm`` and, with ``conv`` (weights, carried inputs, slots), ``short_conv`` in one
+    launch: x += LN(y; wy), h = LN(x; wh) + its convolution. x fp32; y and h both fp32 or both bf16."""
     w, carried, slots = conv or (None, None, None)
     _lib.require_cuda_tensor(x, y, wy, wh, h, w, carried, slots)
     b, ldx = x.shape
-    assert x.dtype == h.dtype == torch.float32 and x.is_contiguous() and h.is_contiguous() and h.shape == x.shape
-    assert _affine_ok(wy, ldx) and _affine_ok(wh, ldx) and (y is None or (y.dtype == torch.float32 and y.is_contiguous() and y.shape == x.shape))
+    assert x.dtype == torch.float32 and x.is_contiguous() and h.is_contiguous() and h.shape == x.shape
+    assert _affine_ok(wy, ldx) and _affine_ok(wh, ldx)
+    assert y is None or (y.dtype == h.dtype and y.stride(1) == 1 and (routing is not None or y.shape[0] == b))
     taps = 0 if w is None else w.shape[0]
     assert w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.shape[1] == ldx and _carried_ok(carried, taps, ldx))
     rc = _lib.cuda().rmlx_sandwich_step(
-        x.data_ptr(), _lib.ptr(y), _lib.ptr(wy), wh.data_ptr(), h.data_ptr(), _lib.ptr(w), taps,
+        x.data_ptr(), _lib.ptr(y), 0 if y is None else y.stride(0),
+        None if routing is None else routing.row_of_pair.data_ptr(), None if routing is None else routing.weights.data_ptr(),
+        0 if routing is None else routing.idx.shape[1], _lib.ptr(wy), wh.data_ptr(), h.data_ptr(), _f32(h), _lib.ptr(w), taps,
         _lib.ptr(carried) if taps > 1 else None, carried.stride(0) if taps > 1 else 0, _lib.ptr(slots), eps, b, width, ldx, int(pdl),
         _lib.stream_ptr())
     _lib.check(rc, "sandwich_step")
