@@ -23,7 +23,7 @@ __device__ __forceinline__ float gated_act_fast(float g, float u, float limit) {
     u = fminf(fmaxf(u, -limit), limit);
     return __fdividef(g, 1.f + __expf(fminf(-kClampedGateSlope * g, 80.f))) * (u + 1.f);
   }
-  return g / (1.f + __expf(-g)) * u;
+  return __fdividef(g, 1.f + __expf(fminf(-g, 80.f))) * u;
 }
 
 }  // namespace rb

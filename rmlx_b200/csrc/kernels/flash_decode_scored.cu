@@ -114,6 +114,15 @@ __device__ __forceinline__ void fs_copy_page(char* dst, const char* src, int chu
 template <int ROW_BYTES, int MAPS>
 __device__ __forceinline__ void fs_copy_maps(char* dst, const char* src, int chunks, int lane) {
   if (MAPS == 1) { fs_copy_page<ROW_BYTES>(dst, src, chunks, lane); return; }
+  constexpr int FULL = ROW_BYTES / 16;
+  if (chunks == FULL) {
+#pragma unroll
+    for (int u = 0; u < kFsPage * MAPS * FULL / 32; ++u) {
+      const int i = u * 32 + lane, r = i / (MAPS * FULL), a = i / FULL % MAPS, c = i % FULL;
+      fs_cp_async16(dst + a * (kFsPage * ROW_BYTES) + r * ROW_BYTES + ((c ^ (r & 7)) << 4), src + i * 16);
+    }
+    return;
+  }
   const int per = MAPS * chunks;
   for (int i = lane; i < kFsPage * per; i += 32) {
     const int r = i / per, q = i - r * per, a = q / chunks, c = q - a * chunks;

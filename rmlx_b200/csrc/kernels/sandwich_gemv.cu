@@ -5,7 +5,9 @@
 //   gated_out       y = W (o / rms(o) * w * sigmoid(gate))
 //   lightning_step  one token: q, k, v through silu, S <- decay S + k v^T, o = S^T q
 //
-// Everything is fp32 beside bf16 weights.
+// Everything is fp32 beside bf16 weights; lightning_step also takes bf16 rows (larger batches, whose projections are GEMMs).
+#include <type_traits>
+
 #include "../common/gemv_core.cuh"
 #include "../common/launch.cuh"
 #include "../common/state_step.cuh"
@@ -128,8 +130,15 @@ staged_out_kernel(Matrix<WBf16> W, SRC src, float* __restrict__ y, int ld_y, int
   }
 }
 
+// Past the first-level cache: the launch before wrote them.
+__device__ __forceinline__ float step_load(const float* p) { return __ldcg(p); }
+__device__ __forceinline__ float step_load(const __nv_bfloat16* p) {
+  return __uint_as_float(uint32_t(__ldcg(reinterpret_cast<const unsigned short*>(p))) << 16);
+}
+
+template <class T>
 struct LightningStep {
-  const float* raw;               // [B, ld_raw]: q at 0, k and v at their columns
+  const T* raw;               // [B, ld_raw]: q at 0, k and v at their columns
   int ld_raw, at_k, at_v;
   const float* decay;             // [H]
   const int* slots;
@@ -140,9 +149,9 @@ struct LightningStep {
 };
 
 // grid (column blocks, heads, batch rows); COLS columns a block.
-template <int COLS, int ROWS>
+template <int COLS, int ROWS, class T>
 __global__ void __launch_bounds__(kGemvThreads)
-lightning_step_kernel(LightningStep p) {
+lightning_step_kernel(LightningStep<T> p) {
   constexpr int G = kGemvThreads / COLS;
   extern __shared__ float sm[];
   float* sr = sm;                    // [n] q, k
@@ -158,15 +167,15 @@ lightning_step_kernel(LightningStep p) {
   const float decay = p.decay[h];
   pdl_launch_dependents();
   pdl_wait();
-  const float* row = p.raw + size_t(b) * p.ld_raw;
+  const T* row = p.raw + size_t(b) * p.ld_raw;
   float own = 0.f;
   if (tid < n) {
-    const float q = step_silu(__ldcg(row + h * n + tid)), k = step_silu(__ldcg(row + p.at_k + h * n + tid));
+    const float q = step_silu(step_load(row + h * n + tid)), k = step_silu(step_load(row + p.at_k + h * n + tid));
     sr[tid] = q;
     sk[tid] = k;
     own = q * k;
   }
-  const float v = col < d ? step_silu(__ldcg(row + p.at_v + h * d + col)) : 0.f;
+  const float v = col < d ? step_silu(step_load(row + p.at_v + h * d + col)) : 0.f;
   own = block_sum_256(own, red);     // sr and sk are visible, too
   part[tid] = col < d ? step_state<ROWS, true>(sp, d, i0, i1, s, sr, sk, nullptr, decay, v) : 0.f;
   __syncthreads();
@@ -218,16 +227,21 @@ extern "C" int rmlx_gated_out(const void* w, const float* o, int ld_o, const flo
   return run_staged(w, GatedSource{o, gate, norm, eps, ld_o, ld_g, D}, y, ld_y, N, K, B, pdl, st);
 }
 
-// raw fp32 [B, ld_raw] with q at 0; out fp32 [B, ld_out]; n <= 256.
-extern "C" int rmlx_lightning_step(const float* raw, int ld_raw, int at_k, int at_v, const float* decay, const int* slots, float* state,
-                                   long long stride, float* out, int ld_out, int B, int H, int n, int d, int pdl, cudaStream_t st) {
+// raw fp32 (f32) or bf16 [B, ld_raw] with q at 0; out fp32 [B, ld_out]; n <= 256.
+extern "C" int rmlx_lightning_step(const void* raw, int ld_raw, int at_k, int at_v, const float* decay, const int* slots, float* state,
+                                   long long stride, float* out, int ld_out, int B, int H, int n, int d, int f32, int pdl,
+                                   cudaStream_t st) {
   if (B < 1 || B > 65535 || H < 1 || H > 65535 || n < 1 || n > 256 || d < 1 || !slots || !decay || at_k < H * n || ld_out < H * d ||
       ld_raw < at_v + H * d || ld_raw < at_k + H * n)
     return -2;
-  const LightningStep p{raw, ld_raw, at_k, at_v, decay, slots, state, stride, out, ld_out, n, d};
   const size_t smem = size_t(2 * n) * sizeof(float);
-  // a head's columns need not meet in one block
-#define RB_LS(C_, R_) return launch_columns(lightning_step_kernel<C_, R_>, p, (d + C_ - 1) / C_, H, B, smem, false, pdl, st)
-  RB_STATE_DISPATCH(n, 1, RB_LS);
+  auto run = [&](auto* rows) -> int {
+    using T = std::remove_const_t<std::remove_pointer_t<decltype(rows)>>;
+    const LightningStep<T> p{rows, ld_raw, at_k, at_v, decay, slots, state, stride, out, ld_out, n, d};
+    // a head's columns need not meet in one block
+#define RB_LS(C_, R_) return launch_columns(lightning_step_kernel<C_, R_, T>, p, (d + C_ - 1) / C_, H, B, smem, false, pdl, st)
+    RB_STATE_DISPATCH(n, 1, RB_LS);
 #undef RB_LS
+  };
+  return f32 ? run(static_cast<const float*>(raw)) : run(static_cast<const __nv_bfloat16*>(raw));
 }

@@ -96,7 +96,7 @@ sandwich_norm_kernel(SRC src, Affine wy, float* __restrict__ x, Affine wh, T* __
   pdl_launch_dependents();
   pdl_wait();
   const int t0 = blockIdx.x * R, chunks = ldx >> 3;
-  auto row = [&](int r) { return min(t0 + r, rows - 1); };         // (a last odd row is done twice, the copy not stored)
+  auto row = [&](int r) { return min(t0 + r, rows - 1); };         // (past the last row: done once more, not stored)
   auto chunk = [&](int u) { return u * kRowThreads + threadIdx.x; };
   SRC from[R];
 #pragma unroll
@@ -562,26 +562,28 @@ sandwich_step_kernel(SandwichStep<SRC, T> p) {
   }
 }
 
-template <class SRC, bool ADD>
-static int launch_sandwich(SRC src, const float* wy, float* x, const float* wh, void* h, float eps, int T, int D, int ldx, int f32,
-                           int pdl, cudaStream_t st) {
+template <class SRC, bool ADD, class TH>
+static int launch_sandwich(SRC src, const float* wy, float* x, const float* wh, TH* h, float eps, int T, int D, int ldx, int pdl,
+                           cudaStream_t st) {
   const Affine ay{wy, ldx}, ah{wh, ldx};
-  auto go = [&](auto kern, int per, auto* out) -> int {
-    return launch(kern, dim3((T + per - 1) / per), dim3(kRowThreads), 0, st, pdl != 0, src, ay, x, ah, out, eps, T, D, ldx);
+  auto go = [&](auto kern, int per) -> int {
+    return launch(kern, dim3((T + per - 1) / per), dim3(kRowThreads), 0, st, pdl != 0, src, ay, x, ah, h, eps, T, D, ldx);
   };
-  const bool narrow = ldx <= 2 * 8 * kRowThreads;
-  if (f32) {
-    float* out = static_cast<float*>(h);
-    return narrow ? go(sandwich_norm_kernel<SRC, ADD, float, 2, 1, 2>, 1, out)
-                  : go(sandwich_norm_kernel<SRC, ADD, float, 4, 1, 2>, 1, out);
+  // where rows are plenty, several a block share its weights and barriers; else as many blocks as the registers allow
+  const int keep = (ldx + 8 * kRowThreads - 1) / (8 * kRowThreads);
+  const bool some = T >= 8 * sm_count(), many = T >= 16 * sm_count();
+  if constexpr (sizeof(TH) == 4) {
+    return keep <= 2 ? go(sandwich_norm_kernel<SRC, ADD, TH, 2, 1, 2>, 1) : go(sandwich_norm_kernel<SRC, ADD, TH, 4, 1, 2>, 1);
+  } else if constexpr (!std::is_same<SRC, RowSource<float>>::value && !std::is_same<SRC, RowSource<__nv_bfloat16>>::value) {
+    if (keep > 2) return go(sandwich_norm_kernel<SRC, ADD, TH, 4, 1, 2>, 1);
+    if (keep > 1) return some ? go(sandwich_norm_kernel<SRC, ADD, TH, 2, 2, 2>, 2) : go(sandwich_norm_kernel<SRC, ADD, TH, 2, 1, 2>, 1);
+    return some ? go(sandwich_norm_kernel<SRC, ADD, TH, 1, 2, 3>, 2) : go(sandwich_norm_kernel<SRC, ADD, TH, 1, 1, 3>, 1);
+  } else {
+    if (keep > 2) return go(sandwich_norm_kernel<SRC, ADD, TH, 4, 1, 2>, 1);
+    if (keep > 1) return many ? go(sandwich_norm_kernel<SRC, ADD, TH, 2, 2, 3>, 2) : go(sandwich_norm_kernel<SRC, ADD, TH, 2, 1, 4>, 1);
+    return many ? go(sandwich_norm_kernel<SRC, ADD, TH, 1, 4, 3>, 4)
+           : some ? go(sandwich_norm_kernel<SRC, ADD, TH, 1, 2, 4>, 2) : go(sandwich_norm_kernel<SRC, ADD, TH, 1, 1, 4>, 1);
   }
-  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(h);
-  if (!narrow) return go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 4, 1, 2>, 1, out);
-  // where rows are plenty, two a block share its weights and barriers; else as many blocks as the registers allow
-  constexpr bool kExperts = !std::is_same<SRC, RowSource<float>>::value && !std::is_same<SRC, RowSource<__nv_bfloat16>>::value;
-  if constexpr (kExperts) return go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 2, 1, 2>, 1, out);
-  else if (T >= 16 * sm_count()) return go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 2, 2, 3>, 2, out);
-  else return go(sandwich_norm_kernel<SRC, ADD, __nv_bfloat16, 2, 1, 4>, 1, out);
 }
 
 template <class SRC, class T>
@@ -605,14 +607,15 @@ extern "C" int rmlx_sandwich_norm(float* x, const void* y, int ldy, const int* r
                                   const float* wy, const float* wh, void* h, float eps, int T, int D, int ldx, int f32, int pdl,
                                   cudaStream_t st) {
   if (T < 1 || D < 1 || ldx < D || ldx % 8 || (h && !wh) || (!h && !y)) return -2;
-  if (!y) return launch_sandwich<RowSource<float>, false>(RowSource<float>{nullptr, 0}, nullptr, x, wh, h, eps, T, D, ldx, f32, pdl, st);
-  if (ldy % 8 || ldy < ldx || !wy || (row_of_pair && (!weights || top_k < 1))) return -2;
+  if (y && (ldy % 8 || ldy < ldx || !wy || (row_of_pair && (!weights || top_k < 1)))) return -2;
   auto run = [&](auto* p) -> int {
     using TY = std::remove_const_t<std::remove_pointer_t<decltype(p)>>;
+    TY* out = static_cast<TY*>(h);
+    if (!p) return launch_sandwich<RowSource<TY>, false, TY>(RowSource<TY>{p, 0}, nullptr, x, wh, out, eps, T, D, ldx, pdl, st);
     if (row_of_pair)
-      return launch_sandwich<ExpertSource<TY>, true>(ExpertSource<TY>{p, ldy, row_of_pair, weights, nullptr, top_k}, wy, x, wh, h,
-                                                     eps, T, D, ldx, f32, pdl, st);
-    return launch_sandwich<RowSource<TY>, true>(RowSource<TY>{p, ldy}, wy, x, wh, h, eps, T, D, ldx, f32, pdl, st);
+      return launch_sandwich<ExpertSource<TY>, true, TY>(ExpertSource<TY>{p, ldy, row_of_pair, weights, nullptr, top_k}, wy, x, wh,
+                                                         out, eps, T, D, ldx, pdl, st);
+    return launch_sandwich<RowSource<TY>, true, TY>(RowSource<TY>{p, ldy}, wy, x, wh, out, eps, T, D, ldx, pdl, st);
   };
   return f32 ? run(static_cast<const float*>(y)) : run(static_cast<const __nv_bfloat16*>(y));
 }

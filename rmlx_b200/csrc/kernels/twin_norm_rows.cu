@@ -224,20 +224,19 @@ rotary_norm_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __
   }
 }
 
-// The form with neighbours, no norm and no bias: chunks of eight turn on their own, so a block deals those of kRaTokens
+// The form with neighbours, no norm and no bias: chunks of eight turn on their own, so a block deals those of TOKENS
 // tokens to its threads in a row. Source rows, widths and strides are multiples of eight values.
-constexpr int kRaTokens = 4;
-template <class TR, class T>
+template <class TR, class T, int TOKENS>
 __global__ void __launch_bounds__(kRowThreads)
 rotary_append_kernel(const TR* __restrict__ raw, int ldraw, const float* __restrict__ inv_freq, int dims, float grow,
                      T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ block_table,
                      const int* __restrict__ positions, const int* __restrict__ token_seq, int rows, int Hq, int Hkv, int dim,
                      int vdim, int max_blocks, int page, int maps) {
   extern __shared__ __align__(16) float trig[];          // per token: cos [dims / 2], sin [dims / 2]
-  __shared__ int s_blk[kRaTokens], s_off[kRaTokens];
+  __shared__ int s_blk[TOKENS], s_off[TOKENS];
   pdl_launch_dependents();
   pdl_wait();
-  const int t0 = blockIdx.x * kRaTokens, n = min(kRaTokens, rows - t0), half = dims / 2;
+  const int t0 = blockIdx.x * TOKENS, n = min(TOKENS, rows - t0), half = dims / 2;
   for (int i = threadIdx.x; i < n * half; i += kRowThreads) {
     const int a = i / half, j = i - a * half;
     float s, c;
@@ -348,11 +347,12 @@ extern "C" int rmlx_rotary_norm_append(const void* raw, int ldraw, int raw_f32, 
   const size_t smem = size_t(dims) * sizeof(float);
   if (smem > 32 * 1024) return -2;
   if (neighbours && !norm && !bias && dim % 8 == 0 && vdim % 8 == 0 && ldraw % 8 == 0 && dkp == dim && dvp == vdim && dims <= 2048) {
-#define RB_RF(TR_, T_)                                                                                                     \
-  return launch(rotary_append_kernel<TR_, T_>, dim3((T + kRaTokens - 1) / kRaTokens), dim3(kRowThreads), smem * kRaTokens, st, \
-                pdl != 0, static_cast<const TR_*>(raw), ldraw, inv_freq, dims, grow, static_cast<T_*>(q_out),                  \
-                static_cast<T_*>(k_cache), static_cast<T_*>(v_cache), block_table, positions, token_seq, T, Hq, Hkv, dim, vdim, \
-                max_blocks, page, maps)
+    const int per = T >= 8 * sm_count() ? 4 : 1;          // tokens a block
+#define RB_RF(TR_, T_)                                                                                                        \
+  return launch(per == 4 ? rotary_append_kernel<TR_, T_, 4> : rotary_append_kernel<TR_, T_, 1>, dim3((T + per - 1) / per),    \
+                dim3(kRowThreads), smem * per, st, pdl != 0, static_cast<const TR_*>(raw), ldraw, inv_freq, dims, grow,       \
+                static_cast<T_*>(q_out), static_cast<T_*>(k_cache), static_cast<T_*>(v_cache), block_table, positions,        \
+                token_seq, T, Hq, Hkv, dim, vdim, max_blocks, page, maps)
     if (f32) RB_RF(float, float);
     if (raw_f32) RB_RF(float, __nv_bfloat16);
     RB_RF(__nv_bfloat16, __nv_bfloat16);

@@ -313,10 +313,12 @@ class NizoraxModel(RaggedModel):
         m, t, dt, pdl = mw.spec, c.t, self.dtype, c.pdl
         raw = N.linear(h, mw.w_in.w, c.bufs.get("raw", t, mw.w_in.n, dtype=dt), pdl=pdl)
         q, k, v, g = (raw[:, a:] for a in mw.at)
-        o = c.bufs.get("scan_o", t, mw.w_o.k, dtype=torch.float32)
-        rec = c.bufs.get("scan_rec", t, m.heads, S.record(m.dim, m.vdim, True), dtype=torch.float32)
-        S.lightning_scan(q, k, v, mw.decay, c.cache.layer_state(li, "state"), o, rec, runs=c.runs,
-                         slots=None if c.runs is not None else c.slots, pdl=pdl)
+        o, state = c.bufs.get("scan_o", t, mw.w_o.k, dtype=torch.float32), c.cache.layer_state(li, "state")
+        if c.runs is None:                                 # a token of every sequence
+            S.lightning_step(raw, mw.at[1], mw.at[2], mw.decay, c.slots, state, o, pdl=pdl)
+        else:
+            rec = c.bufs.get("scan_rec", t, m.heads, S.record(m.dim, m.vdim, True), dtype=torch.float32)
+            S.lightning_scan(q, k, v, mw.decay, state, o, rec, runs=c.runs, pdl=pdl)
         return S.gated_norm(o, g, mw.norm, self.cfg.norm_eps, 1, c.bufs.get("scan_a", t, mw.w_o.k, dtype=dt), False, sigmoid=True,
                             pdl=pdl)
 
