@@ -236,7 +236,7 @@ def decode_kernels(tab: Table, model: NizoraxModel, like, b: int, ctx: int):
     _, at_k, at_v, at_g = g0.at
     raw, o, a = rnd(b, g0.w_in.n), rnd(b, g0.w_o.k), rnd(b, g0.w_o.k, dtype=BF)
     wraw, wout = rnd(b, r0.w_in.n), rnd(b, r0.inner_p, dtype=BF)
-    tab.add(ph, "lightning: state", [lambda i=i, w=w: S.lightning_step(raw, at_k, at_v, w.decay, c.slots, cache.layer_state(i, "state"),
+    tab.add(ph, "lightning: state", [lambda i=i, w=w: W.lightning_step(raw, at_k, at_v, w.decay, c.slots, cache.layer_state(i, "state"),
                                                                        o, pdl=True) for i, w, _ in light],
             (b * s.heads * s.dim * s.vdim * 8, 0), "WKV step", [lambda i=i, w=w: wkv.wkv_decode(
                 wraw, w.inner_p, w.w2, w.w0, w.u, w.norm, 1e-6, lc.slots, lcache.layer_state(i, "wkv"), lcache.layer_state(i, "prev"),

@@ -315,7 +315,7 @@ class NizoraxModel(RaggedModel):
         q, k, v, g = (raw[:, a:] for a in mw.at)
         o, state = c.bufs.get("scan_o", t, mw.w_o.k, dtype=torch.float32), c.cache.layer_state(li, "state")
         if c.runs is None:                                 # a token of every sequence
-            S.lightning_step(raw, mw.at[1], mw.at[2], mw.decay, c.slots, state, o, pdl=pdl)
+            W.lightning_step(raw, mw.at[1], mw.at[2], mw.decay, c.slots, state, o, pdl=pdl)
         else:
             rec = c.bufs.get("scan_rec", t, m.heads, S.record(m.dim, m.vdim, True), dtype=torch.float32)
             S.lightning_scan(q, k, v, mw.decay, state, o, rec, runs=c.runs, pdl=pdl)

@@ -15,7 +15,6 @@ from ..ops import parallel_block as P
 from ..ops import post_norm as N
 from ..ops import routed as R
 from ..ops import sandwich as W
-from ..ops import scan as S
 from .layered_decode import LayeredDecode
 from .nizorax import DiffAttentionWeights, PolyFfWeights
 from .ragged_model import StepContext
@@ -48,7 +47,7 @@ class SandwichDecode(LayeredDecode):
             return
         _, at_k, at_v, at_g = mw.at
         o = get("scan_o", t, mw.w_o.k, dtype=f32)
-        S.lightning_step(raw, at_k, at_v, mw.decay, c.slots, c.cache.layer_state(li, "state"), o, pdl=pdl)
+        W.lightning_step(raw, at_k, at_v, mw.decay, c.slots, c.cache.layer_state(li, "state"), o, pdl=pdl)
         W.gated_out(o, raw[:, at_g:], mw.norm, eps, mw.w_o.w, y, pdl=pdl)
 
     def _feed_forward(self, f, h: torch.Tensor, y: torch.Tensor, c: StepContext) -> None:

@@ -19,6 +19,7 @@ _lib.register_cuda_sigs({
     "rmlx_poly_norm": ("ppfp" "iiiiip", "i"),
     "rmlx_sandwich_step_max_width": ("", "i"),
     "rmlx_sandwich_step": ("ppi" "ppi" "pppi" "pi" "pqp" "fiiiip", "i"),
+    "rmlx_lightning_step": ("piii" "ppp" "q" "pi" "iiii" "iip", "i"),
     "rmlx_poly_out": ("ppipfpi" "iiiiip", "i"),
     "rmlx_gated_out": ("ppipipfpi" "iiiiip", "i"),
 })
@@ -130,3 +131,16 @@ def gated_out(o: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor, eps: floa
                                         norm.data_ptr(), eps, y[lo:].data_ptr(), y.stride(0), hi - lo, n, k, norm.numel(), int(pdl),
                                         _lib.stream_ptr())
         _lib.check(rc, "gated_out")
+
+
+def lightning_step(raw: torch.Tensor, at_k: int, at_v: int, decay: torch.Tensor, slots: torch.Tensor, state: torch.Tensor,
+                   out: torch.Tensor, pdl: bool = False) -> None:
+    """One token per row of ``scan.lightning_scan``: raw fp32 or bf16 [B, ..] = q at 0, k and v at their columns; out fp32 [B, >= H vdim]."""
+    _lib.require_cuda_tensor(raw, decay, slots, state, out)
+    _, h, n, d = state.shape
+    assert out.dtype == decay.dtype == torch.float32 and state.stride()[1:] == (n * d, d, 1)
+    assert slots.dtype == torch.int32 and decay.numel() == h
+    rc = _lib.cuda().rmlx_lightning_step(
+        raw.data_ptr(), raw.stride(0), at_k, at_v, decay.data_ptr(), slots.data_ptr(), state.data_ptr(), state.stride(0),
+        out.data_ptr(), out.stride(0), raw.shape[0], h, n, d, _f32(raw), int(pdl), _lib.stream_ptr())
+    _lib.check(rc, "lightning_step")

@@ -23,7 +23,6 @@ _lib.register_cuda_sigs({
     "rmlx_gla_decode": ("piiiii" "pipff" "pfp" "pq" "pi" "iiiiip", "i"),
     "rmlx_ssd_decode": ("piii" "ppi" "ppppp" "pq" "pi" "pfi" "pi" "iiiii" "ip", "i"),
     "rmlx_lightning_scan": ("pppip" "pippi" "pqpi" "iiii" "pip", "i"),
-    "rmlx_lightning_step": ("piii" "ppp" "q" "pi" "iiii" "iip", "i"),
     "rmlx_gated_norm": ("pipipfpi" "iiiiiiip", "i"),
 })
 
@@ -152,16 +151,3 @@ def ssd_decode(raw: torch.Tensor, x_at: int, dt_at: int, conv_w: torch.Tensor, c
         state.data_ptr(), state.stride(0), y.data_ptr(), y.stride(0), norm.data_ptr(), eps, norm_groups, out.data_ptr(),
         out.stride(0), raw.shape[0], h, groups, n, d, int(pdl), _lib.stream_ptr())
     _lib.check(rc, "ssd_decode")
-
-
-def lightning_step(raw: torch.Tensor, at_k: int, at_v: int, decay: torch.Tensor, slots: torch.Tensor, state: torch.Tensor,
-                   out: torch.Tensor, pdl: bool = False) -> None:
-    """One token per row of ``lightning_scan``: raw fp32 or bf16 [B, ..] = q at 0, k and v at their columns; out fp32 [B, >= H vdim]."""
-    _lib.require_cuda_tensor(raw, decay, slots, state, out)
-    _, h, n, d = state.shape
-    assert out.dtype == decay.dtype == torch.float32 and state.stride()[1:] == (n * d, d, 1)
-    assert slots.dtype == torch.int32 and decay.numel() == h
-    rc = _lib.cuda().rmlx_lightning_step(
-        raw.data_ptr(), raw.stride(0), at_k, at_v, decay.data_ptr(), slots.data_ptr(), state.data_ptr(), state.stride(0),
-        out.data_ptr(), out.stride(0), raw.shape[0], h, n, d, _f32(raw), int(pdl), _lib.stream_ptr())
-    _lib.check(rc, "lightning_step")

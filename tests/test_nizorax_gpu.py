@@ -529,7 +529,7 @@ def test_lightning_decode_step(dev, spec, b):
     o, y = torch.zeros(b, c.mw.w_o.k, device=dev), torch.zeros(b, pad8(c.width), device=dev)
     for t in range(6):
         raw = (padded(h[:, t], dev).double() @ c.mw.w_in.w.double().T).float()
-        S.lightning_step(raw, at_k, at_v, c.mw.decay, slots, state, o)
+        W.lightning_step(raw, at_k, at_v, c.mw.decay, slots, state, o)
         W.gated_out(o, raw[:, at_g:], c.mw.norm, 1e-5, c.mw.w_o.w, y)
         assert rel(y[:, :c.width], torch.stack([w[t] for w in want])) < 2e-5, t
     assert int((c.cache.state.abs().sum(1) > 0).sum()) == b               # other slots are untouched
