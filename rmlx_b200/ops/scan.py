@@ -1,6 +1,6 @@
 """Linear recurrences token by token (csrc/kernels/linear_scan.cu): gated linear attention, state-space heads with
-their short convolution, lightning attention, and the norm of their outputs with a gate; their decode steps
-(twin_norm_gemv.cu, sandwich_gemv.cu). A sequence's state is its slot's row of a
+their short convolution, lightning attention, and the norm of their outputs with a gate; the first two's decode steps
+(twin_norm_gemv.cu). A sequence's state is its slot's row of a
 flat fp32 pool (``PagedKvCache.layer_state`` views)."""
 from __future__ import annotations
 
